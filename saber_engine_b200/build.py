@@ -25,6 +25,9 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall", "-Xptxas", "-v",
 ]
+# Sources whose results are held to fp32 accuracy: CUDA's accurate math functions, IEEE division and
+# square root, denormals kept.
+PRECISE = {"linear.cu", "delta.cu", "mla.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-march=x86-64-v3"]
 
 
@@ -59,7 +62,8 @@ def _compile(src: Path, verbose: bool) -> tuple[Path, str]:
     obj = OBJ_DIR / (src.relative_to(CSRC).as_posix().replace("/", "__") + ".o")
     stamp = obj.with_suffix(".sha")
     if src.suffix == ".cu":
-        cmd = [str(home / "bin" / "nvcc"), *NVCC_FLAGS, "-c", str(src), "-o", str(obj)]
+        flags = [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and src.name in PRECISE)]
+        cmd = [str(home / "bin" / "nvcc"), *flags, "-c", str(src), "-o", str(obj)]
     else:
         cmd = ["g++", *CXX_FLAGS, f"-I{home / 'include'}", "-c", str(src), "-o", str(obj)]
     dg = _digest(src, cmd)

@@ -22,8 +22,11 @@
 
 #include "../comm/comm.h"
 #include "../kernels/attn.h"
+#include "../kernels/delta.h"
 #include "../kernels/gdn.h"
 #include "../kernels/gemm_i8.h"
+#include "../kernels/linear.h"
+#include "../kernels/mla.h"
 #include "../kernels/moe.h"
 #include "../kernels/rowops.h"
 #include "../kernels/sample.h"
@@ -45,8 +48,8 @@ struct OpGdnStep { saber::GdnStepParams p; int nseq; };
 struct OpGdnChunk { saber::GdnRecParams p; int nseq, max_rows; float* scratch; };
 struct OpRope { saber::RopeKvParams p; };
 struct OpAttn { saber::AttnParams p; };
-struct OpArgmax { const void* logits; int rows, ld, V, id_offset; int32_t* idx; float* val; };
-struct OpSeam { const void* logits; int rows, ld, V, id_offset; const float* temps; int32_t* ids; float* vals; float* lse; };
+struct OpArgmax { const void* logits; int f32, rows, ld, V, id_offset; int32_t* idx; float* val; };
+struct OpSeam { const void* logits; int f32, rows, ld, V, id_offset; const float* temps; int32_t* ids; float* vals; float* lse; };
 struct OpVerify { saber::VerifyParams p; };
 struct OpDraftIndex { saber::DraftIndexParams p; };
 struct OpMemset { void* dst; int value; size_t bytes; };
@@ -58,12 +61,18 @@ struct OpMoeCombine { saber::MoeCombineParams p; };
 struct OpDigest { const void* buf; size_t bytes; unsigned long long* out; };
 struct OpDigestClear { unsigned long long* out; int n; };
 struct OpSampleSeam { const int32_t* ids; const float* vals; const float* samp; const float* u; int32_t* picks; int rows; };
-struct OpLogitGather { const void* logits; int rows, ld, V, id_offset; const int32_t* ids; float* out; };
+struct OpLogitGather { const void* logits; int f32, rows, ld, V, id_offset; const int32_t* ids; float* out; };
+struct OpLinear { saber::LinParams p; };
+struct OpStreamEmbed { saber::StreamEmbedParams p; };
+struct OpStreamNorm { saber::StreamNormParams p; };
+struct OpDelta { saber::DeltaParams p; int single_row; };
+struct OpMla { saber::MlaParams p; };
 struct OpMoeGather { const int8_t* q; const float* scale; int M_pad; const int32_t* src_row; const int32_t* ntiles;
                      int8_t* q_out; float* scale_out; int rows_cap, M_pad_out, K, to_fp8; };
 
 using Op = std::variant<OpGemm, OpRow, OpEmbed, OpGdnConv, OpGdnRec, OpRope, OpAttn, OpArgmax,
-                        OpSeam, OpVerify, OpMemset, OpCopy, OpAllReduce, OpExpand, OpAdvance, OpPickMerge, OpMoeRoute, OpMoeCombine, OpMoeGather, OpDigest, OpDigestClear, OpGdnChunk, OpLogitGather, OpSampleSeam, OpGdnStep, OpSeamMerge, OpDraftIndex>;
+                        OpSeam, OpVerify, OpMemset, OpCopy, OpAllReduce, OpExpand, OpAdvance, OpPickMerge, OpMoeRoute, OpMoeCombine, OpMoeGather, OpDigest, OpDigestClear, OpGdnChunk, OpLogitGather, OpSampleSeam, OpGdnStep, OpSeamMerge, OpDraftIndex,
+                        OpLinear, OpStreamEmbed, OpStreamNorm, OpDelta, OpMla>;
 
 struct Entry {
   Op op;
@@ -102,9 +111,9 @@ int launch(const Op& op, cudaStream_t s) {
         else if constexpr (std::is_same_v<T, OpRope>) return saber_rope_kv_launch(&o.p, s);
         else if constexpr (std::is_same_v<T, OpAttn>) return saber_attn_launch(&o.p, s);
         else if constexpr (std::is_same_v<T, OpArgmax>)
-          return saber_argmax_launch(o.logits, o.rows, o.ld, o.V, o.id_offset, o.idx, o.val, s);
+          return saber_argmax_launch(o.logits, o.f32, o.rows, o.ld, o.V, o.id_offset, o.idx, o.val, s);
         else if constexpr (std::is_same_v<T, OpSeam>)
-          return saber_topk_seam_launch(o.logits, o.rows, o.ld, o.V, o.id_offset, o.temps, o.ids, o.vals, o.lse, s);
+          return saber_topk_seam_launch(o.logits, o.f32, o.rows, o.ld, o.V, o.id_offset, o.temps, o.ids, o.vals, o.lse, s);
         else if constexpr (std::is_same_v<T, OpVerify>) return saber_verify_launch(&o.p, s);
         else if constexpr (std::is_same_v<T, OpDraftIndex>) return saber_draft_index_launch(&o.p, s);
         else if constexpr (std::is_same_v<T, OpMemset>)
@@ -119,7 +128,12 @@ int launch(const Op& op, cudaStream_t s) {
         else if constexpr (std::is_same_v<T, OpDigest>) return saber_digest_launch(o.buf, o.bytes, o.out, s);
         else if constexpr (std::is_same_v<T, OpDigestClear>) return saber_digest_clear_launch(o.out, o.n, s);
         else if constexpr (std::is_same_v<T, OpSampleSeam>) return saber_sample_seam_launch(o.ids, o.vals, o.samp, o.u, o.picks, o.rows, s);
-        else if constexpr (std::is_same_v<T, OpLogitGather>) return saber_logit_gather_launch(o.logits, o.rows, o.ld, o.V, o.id_offset, o.ids, o.out, s);
+        else if constexpr (std::is_same_v<T, OpLogitGather>) return saber_logit_gather_launch(o.logits, o.f32, o.rows, o.ld, o.V, o.id_offset, o.ids, o.out, s);
+        else if constexpr (std::is_same_v<T, OpLinear>) return saber_linear_launch(&o.p, s);
+        else if constexpr (std::is_same_v<T, OpStreamEmbed>) return saber_stream_embed_launch(&o.p, s);
+        else if constexpr (std::is_same_v<T, OpStreamNorm>) return saber_stream_norm_launch(&o.p, s);
+        else if constexpr (std::is_same_v<T, OpDelta>) return saber_delta_launch(&o.p, o.single_row, s);
+        else if constexpr (std::is_same_v<T, OpMla>) return saber_mla_launch(&o.p, s);
         else if constexpr (std::is_same_v<T, OpMoeGather>)
           return saber_moe_gather_launch(o.q, o.scale, o.M_pad, o.src_row, o.ntiles, o.q_out, o.scale_out, o.rows_cap,
                                          o.M_pad_out, o.K, o.to_fp8, s);
@@ -220,13 +234,13 @@ int saber_program_add_rope(void* h, const saber::RopeKvParams* p, const char* ta
 int saber_program_add_attn(void* h, const saber::AttnParams* p, const char* tag) {
   return add(h, OpAttn{*p}, p->splits > 1 ? 2 : 1, tag);
 }
-int saber_program_add_argmax(void* h, const void* logits, int rows, int ld, int V, int id_offset,
+int saber_program_add_argmax(void* h, const void* logits, int f32, int rows, int ld, int V, int id_offset,
                              int32_t* idx, float* val, const char* tag) {
-  return add(h, OpArgmax{logits, rows, ld, V, id_offset, idx, val}, 1, tag);
+  return add(h, OpArgmax{logits, f32, rows, ld, V, id_offset, idx, val}, 1, tag);
 }
-int saber_program_add_seam(void* h, const void* logits, int rows, int ld, int V, int id_offset,
+int saber_program_add_seam(void* h, const void* logits, int f32, int rows, int ld, int V, int id_offset,
                            const float* temps, int32_t* ids, float* vals, float* lse, const char* tag) {
-  return add(h, OpSeam{logits, rows, ld, V, id_offset, temps, ids, vals, lse}, 1, tag);
+  return add(h, OpSeam{logits, f32, rows, ld, V, id_offset, temps, ids, vals, lse}, 1, tag);
 }
 int saber_program_add_verify(void* h, const saber::VerifyParams* p, const char* tag) {
   return add(h, OpVerify{*p}, 1, tag);
@@ -261,15 +275,30 @@ int saber_program_add_sample_seam(void* h, const int32_t* ids, const float* vals
                                   int32_t* picks, int rows, const char* tag) {
   return add(h, OpSampleSeam{ids, vals, samp, u, picks, rows}, 1, tag);
 }
-int saber_program_add_logit_gather(void* h, const void* logits, int rows, int ld, int V, int id_offset,
+int saber_program_add_logit_gather(void* h, const void* logits, int f32, int rows, int ld, int V, int id_offset,
                                    const int32_t* ids, float* out, const char* tag) {
-  return add(h, OpLogitGather{logits, rows, ld, V, id_offset, ids, out}, 1, tag);
+  return add(h, OpLogitGather{logits, f32, rows, ld, V, id_offset, ids, out}, 1, tag);
 }
 int saber_program_add_digest_clear(void* h, unsigned long long* out, int n, const char* tag) {
   return add(h, OpDigestClear{out, n}, 1, tag);
 }
 int saber_program_add_moe_combine(void* h, const saber::MoeCombineParams* p, const char* tag) {
   return add(h, OpMoeCombine{*p}, 1, tag);
+}
+int saber_program_add_linear(void* h, const saber::LinParams* p, const char* tag) {
+  return add(h, OpLinear{*p}, saber_linear_launches(p), tag);
+}
+int saber_program_add_stream_embed(void* h, const saber::StreamEmbedParams* p, const char* tag) {
+  return add(h, OpStreamEmbed{*p}, 1, tag);
+}
+int saber_program_add_stream_norm(void* h, const saber::StreamNormParams* p, const char* tag) {
+  return add(h, OpStreamNorm{*p}, 1, tag);
+}
+int saber_program_add_delta(void* h, const saber::DeltaParams* p, int single_row, const char* tag) {
+  return add(h, OpDelta{*p, single_row}, saber_delta_launches(single_row), tag);
+}
+int saber_program_add_mla(void* h, const saber::MlaParams* p, const char* tag) {
+  return add(h, OpMla{*p}, saber_mla_launches(p), tag);
 }
 int saber_program_add_allreduce(void* h, const saber::AllReduceParams* p, const char* tag) {
   return add(h, OpAllReduce{*p}, 1, tag);

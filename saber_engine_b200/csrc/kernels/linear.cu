@@ -1,0 +1,478 @@
+// Linears around an fp32 residual stream.
+//
+// bf16: one tcgen05 GEMM kernel, token rows on the 128 accumulator lanes and 256 weight rows on the N
+// side (the orientation and tile storage of gemm_i8.cu: pre-tiled operands, untiled bulk copies into a
+// ring of stages, one MMA-issuing thread, eight epilogue warps).  Its epilogues keep the residual stream
+// and the normalisation in fp32 without a kernel of their own: a "stream" linear adds its result to the
+// fp32 row, writes the next linear's bf16 operand norm_w * x and the row's partial sums of squares; the
+// next linear multiplies its result by the reciprocal root mean square.  A gated unit's activation is
+// computed in the epilogue of its gate | up tiles.  Split-K parts go to a workspace and the last CTA of a
+// tile to arrive adds them in order, so the result does not depend on the order of arrival.
+//
+// fp32: a CUDA-core GEMM (plain fused multiply-adds) followed by one row kernel that runs the same
+// epilogue; the bf16 linear takes this two-launch form too when fuse = 0.
+#include "launch.cuh"
+#include "linear.h"
+#include "ptx_sm100.cuh"
+
+namespace saber {
+
+constexpr int kLinThreads = 320;
+constexpr int kLinMaxStages = 8;
+constexpr uint32_t kLinTile = 32768;      // 256 weight rows x 64 bf16
+
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit, float alpha) {
+  const float g = fminf(gate, limit);
+  const float u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+
+__device__ __forceinline__ float row_rms_scale(const LinEpi& e, int m) {
+  if (e.ss == nullptr) return 1.f;
+  float s = 0.f;
+  for (int i = 0; i < e.ss_n; ++i) s += __ldcg(e.ss + static_cast<size_t>(m) * e.ss_n + i);
+  return 1.f / sqrtf(s * e.inv_width + e.eps);
+}
+
+template <int kMT>
+__global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_constant__ LinParams p, const int stages) {
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ uint64_t bars[2 * kLinMaxStages + 1];
+  __shared__ uint32_t tmem_base_s, is_last_s, abort_s;
+  __shared__ float bias_s[256], normw_s[256];
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int tile_m = blockIdx.x, tile_n = blockIdx.y, split = blockIdx.z;
+  const int KB = p.K >> 6;
+  const int kb_per = (KB + p.splits - 1) / p.splits;
+  const int kb0 = split * kb_per;
+  const int nkb = min(KB, kb0 + kb_per) - kb0;        // host guarantees >= 1
+  const int m0 = tile_m * p.nt * kMT;
+  const uint32_t abytes = static_cast<uint32_t>(p.nt) * 128u * kMT;
+  const uint32_t a_smem = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  const uint32_t w_smem = a_smem + static_cast<uint32_t>(stages) * abytes;
+  const uint32_t bar_full = smem_u32(&bars[0]);
+  const uint32_t bar_empty = smem_u32(&bars[kLinMaxStages]);
+  const uint32_t bar_acc = smem_u32(&bars[2 * kLinMaxStages]);
+  constexpr uint32_t kCols = kMT == 2 ? 512u : 256u;
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < stages; ++s) {
+      mbar_init(bar_full + 8 * s, 1);
+      mbar_init(bar_empty + 8 * s, 1);
+    }
+    mbar_init(bar_acc, 1);
+    abort_s = 0;
+    is_last_s = 1;
+    mbar_init_fence();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_s), kCols);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_d = tmem_base_s;
+
+  if (warp == 0) {
+    // ---------------------------------------------------------------- producer
+    if (lane == 0) {
+      const uint64_t pol = gridDim.x > 1 ? l2_policy_evict_normal() : l2_policy_evict_first();
+      const uint8_t* wp = static_cast<const uint8_t*>(p.w) + (static_cast<size_t>(tile_n) * KB + kb0) * kLinTile;
+      const uint8_t* ap = static_cast<const uint8_t*>(p.a) + (static_cast<size_t>(kb0) * p.M_pad + m0) * 128;
+      const size_t a_step = static_cast<size_t>(p.M_pad) * 128;
+      const int pre = min(stages, nkb);
+      for (int it = 0; it < pre; ++it) {         // weights do not depend on the predecessor kernel
+        mbar_arrive_expect_tx(bar_full + 8 * it, kLinTile + abytes);
+        bulk_g2s_hint(w_smem + it * kLinTile, wp, kLinTile, bar_full + 8 * it, pol);
+        wp += kLinTile;
+      }
+      pdl_wait();
+      for (int it = 0; it < pre; ++it) {
+        bulk_g2s(a_smem + it * abytes, ap, abytes, bar_full + 8 * it);
+        ap += a_step;
+      }
+      int issued = pre, s = pre == stages ? 0 : pre;
+      uint32_t ph = pre == stages ? 1u : 0u;
+      bool ok = true;
+      for (int it = pre; it < nkb; ++it) {
+        if (!mbar_wait(bar_empty + 8 * s, ph ^ 1u, p.err, kErrWaitEmpty)) { ok = false; break; }
+        mbar_arrive_expect_tx(bar_full + 8 * s, kLinTile + abytes);
+        bulk_g2s_hint(w_smem + s * kLinTile, wp, kLinTile, bar_full + 8 * s, pol);
+        bulk_g2s(a_smem + s * abytes, ap, abytes, bar_full + 8 * s);
+        wp += kLinTile;
+        ap += a_step;
+        issued = it + 1;
+        if (++s == stages) { s = 0; ph ^= 1u; }
+      }
+      if (!ok)                                   // do not leave while an own copy is in flight
+        for (int it = max(0, issued - stages); it < issued; ++it)
+          mbar_wait(bar_full + 8 * (it % stages), (it / stages) & 1, p.err, kErrWaitDrain);
+    }
+  } else if (warp == 1) {
+    // ---------------------------------------------------------------- MMA issuer
+    if (lane == 0) {
+      const uint32_t idesc = make_idesc(kCFmtF32, kFmtBF16, kFmtBF16, 128, 256);
+      const uint64_t desc_hi = make_desc_k128(0);
+      uint32_t a_addr = a_smem;
+      int s = 0;
+      uint32_t ph = 0;
+      bool ok = true;
+      for (int it = 0; it < nkb; ++it) {
+        if (!mbar_wait(bar_full + 8 * s, ph, p.err, kErrWaitReady)) { ok = false; break; }
+        tc_fence_after_sync();
+        const uint32_t w_addr = w_smem + s * kLinTile;
+        const uint64_t a_desc = desc_hi | static_cast<uint64_t>((a_addr & 0x3FFFFu) >> 4);
+        const uint64_t b_desc = desc_hi | static_cast<uint64_t>((w_addr & 0x3FFFFu) >> 4);
+#pragma unroll
+        for (int j2 = 0; j2 < kMT; ++j2) {
+          const uint32_t dj = tmem_d + static_cast<uint32_t>(j2) * 256u;
+          const uint64_t aj = a_desc + static_cast<uint64_t>(j2) * (static_cast<uint64_t>(p.nt) * 128u >> 4);
+          mma_f16_ss(dj, aj, b_desc, idesc, it != 0 ? 1u : 0u);
+          mma_f16_ss(dj, aj + 2, b_desc + 2, idesc, 1u);
+          mma_f16_ss(dj, aj + 4, b_desc + 4, idesc, 1u);
+          mma_f16_ss(dj, aj + 6, b_desc + 6, idesc, 1u);
+        }
+        mma_commit(bar_empty + 8 * s);
+        a_addr += abytes;
+        if (++s == stages) { s = 0; ph ^= 1u; a_addr = a_smem; }
+      }
+      mma_commit(bar_acc);
+      if (!ok) mbar_wait(bar_acc, 0, nullptr, 0);   // issued MMAs retire before the tensor memory is freed
+    }
+  } else {
+    // ---------------------------------------------------------------- epilogue (8 warps)
+    const int te = threadIdx.x - 64;              // 0..255
+    const int grp = te >> 7;                      // column half
+    const int q4 = warp & 3;                      // TMEM lane quarter of this warp
+    const LinEpi& e = p.e;
+    const int n0 = tile_n * 256;
+    if (e.stream) {
+      const bool in = n0 + te < e.width;
+      bias_s[te] = (e.bias && in) ? e.bias[n0 + te] : 0.f;
+      normw_s[te] = in ? (e.norm_w ? e.norm_w[n0 + te] : 1.f) : 0.f;
+    }
+    bool ok = mbar_wait(bar_acc, 0, p.err, kErrWaitAcc);
+    if (!ok) abort_s = 1u;
+    named_bar_sync(1, 256);
+    ok = abort_s == 0u;
+    tc_fence_after_sync();
+    pdl_wait();
+    const int rowl = q4 * 32 + lane;
+    const uint32_t t_lane = tmem_d + (static_cast<uint32_t>(q4 * 32) << 16);
+    const int tile_lin = tile_m * gridDim.y + tile_n;
+    bool from_ws = false;
+    if (p.splits > 1) {                           // (kMT == 1)
+      const int mt = min(p.nt, p.M - m0);
+      float* part = p.ws + (static_cast<size_t>(tile_lin) * p.splits + split) * p.nt * 256;
+      if (ok && q4 * 32 < mt) {
+        for (int c = grp * 128; c < grp * 128 + 128; c += 32) {
+          uint32_t r[32];
+          tmem_ld32(t_lane + c, r);
+          tmem_ld_wait();
+          if (rowl < mt) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              __stcg(reinterpret_cast<float4*>(part + (static_cast<size_t>((c >> 2) + j) * p.nt + rowl) * 4),
+                     make_float4(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]), __uint_as_float(r[4 * j + 2]),
+                                 __uint_as_float(r[4 * j + 3])));
+          }
+        }
+      }
+      __threadfence();
+      named_bar_sync(1, 256);
+      if (te == 0) {
+        const uint32_t old = atomicAdd(p.counters + tile_lin, 1u);
+        const bool last = old == static_cast<uint32_t>(p.splits) - 1u;
+        if (last) p.counters[tile_lin] = 0u;
+        __threadfence();
+        is_last_s = last ? 1u : 0u;
+      }
+      named_bar_sync(1, 256);
+      if (!is_last_s) ok = false;
+      __threadfence();
+      from_ws = true;
+    }
+    if (ok) {
+      const float* parts = p.ws + static_cast<size_t>(tile_lin) * p.splits * p.nt * 256;
+#pragma unroll 1
+      for (int j2 = 0; j2 < kMT; ++j2) {
+        const int mb = m0 + j2 * p.nt;
+        const int mt = min(p.nt, p.M - mb);
+        if (q4 * 32 >= mt) continue;              // warp-uniform
+        const bool live = rowl < mt;
+        const int m = mb + rowl;
+        // 32 accumulator columns from c on (all lanes of the warp call together)
+        auto load = [&](int c, float (&v)[32]) {
+          if (!from_ws) {
+            uint32_t r[32];
+            tmem_ld32(t_lane + static_cast<uint32_t>(j2) * 256u + c, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = 0.f;
+            if (live) {
+              for (int sp = 0; sp < p.splits; ++sp) {
+                const float* part = parts + static_cast<size_t>(sp) * p.nt * 256;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                  const float4 f = __ldcg(reinterpret_cast<const float4*>(part + (static_cast<size_t>((c >> 2) + j) * p.nt + rowl) * 4));
+                  v[4 * j] += f.x; v[4 * j + 1] += f.y; v[4 * j + 2] += f.z; v[4 * j + 3] += f.w;
+                }
+              }
+            }
+          }
+        };
+        if (!e.stream) {
+          const float sc = live ? row_rms_scale(e, m) : 0.f;
+          if (tile_n < e.act_tile0) {
+            for (int c = grp * 128; c < grp * 128 + 128; c += 32) {
+              if (n0 + c >= e.n_plain) break;
+              float v[32];
+              load(c, v);
+              if (live) {
+                float* o = e.out + static_cast<size_t>(m) * e.ldo + n0 + c;
+                if (n0 + c + 32 <= e.n_plain) {
+#pragma unroll
+                  for (int j = 0; j < 8; ++j)
+                    *reinterpret_cast<float4*>(o + 4 * j) = make_float4(v[4 * j] * sc, v[4 * j + 1] * sc, v[4 * j + 2] * sc, v[4 * j + 3] * sc);
+                } else {
+#pragma unroll
+                  for (int j = 0; j < 32; ++j)
+                    if (n0 + c + j < e.n_plain) o[j] = v[j] * sc;
+                }
+              }
+            }
+          } else {
+            const int k0 = e.act_k0 + (tile_n - e.act_tile0) * 128;
+            for (int c = grp * 64; c < grp * 64 + 64; c += 32) {
+              float g[32], u[32];
+              load(c, g);
+              load(128 + c, u);
+              if (live) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                  float y[8];
+#pragma unroll
+                  for (int i = 0; i < 8; ++i) y[i] = clamped_glu(g[8 * j + i] * sc, u[8 * j + i] * sc, e.limit, e.alpha);
+                  operand_store8(e.act, m, k0 + c + 8 * j, y);
+                }
+              }
+            }
+          }
+        } else {
+          float sq = 0.f;
+          for (int c = grp * 128; c < grp * 128 + 128; c += 32) {
+            if (n0 + c >= e.width) break;
+            float v[32];
+            load(c, v);
+            if (live) {
+              float* xr = e.x + static_cast<size_t>(m) * e.ldx + n0 + c;     // ldx is a multiple of 32: whole groups are in bounds
+#pragma unroll
+              for (int j = 0; j < 8; ++j) {
+                float4 o = e.add ? *reinterpret_cast<const float4*>(xr + 4 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
+                const float* b = bias_s + c + 4 * j;
+                o.x += v[4 * j] + b[0]; o.y += v[4 * j + 1] + b[1]; o.z += v[4 * j + 2] + b[2]; o.w += v[4 * j + 3] + b[3];
+                *reinterpret_cast<float4*>(xr + 4 * j) = o;
+                v[4 * j] = o.x; v[4 * j + 1] = o.y; v[4 * j + 2] = o.z; v[4 * j + 3] = o.w;
+              }
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                float y[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                  const float t = v[8 * j + i];
+                  sq += t * t;
+                  y[i] = t * normw_s[c + 8 * j + i];
+                }
+                operand_store8(e.op, m, e.op_k0 + n0 + c + 8 * j, y);
+              }
+            }
+          }
+          if (live && e.ss_out != nullptr && tile_n * 2 + grp < e.ss_out_n)
+            e.ss_out[static_cast<size_t>(m) * e.ss_out_n + tile_n * 2 + grp] = sq;
+        }
+      }
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tmem_d, kCols);
+}
+
+// ------------------------------------------------------------------------------------ fp32 GEMM
+// 64 x 64 output tile, 16 k per step, 4 x 4 outputs per thread; plain fused multiply-adds.
+__global__ void __launch_bounds__(256) lin_f32_kernel(const float* __restrict__ a, const float* __restrict__ w, float* __restrict__ out,
+                                                      int M, int N, int K) {
+  pdl_wait();
+  __shared__ float as[16][68], ws[16][68];
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    const float4 av = m0 + lr < M ? *reinterpret_cast<const float4*>(a + static_cast<size_t>(m0 + lr) * K + k0 + lk) : make_float4(0, 0, 0, 0);
+    const float4 wv = *reinterpret_cast<const float4*>(w + static_cast<size_t>(n0 + lr) * K + k0 + lk);   // N is a multiple of 256
+    as[lk][lr] = av.x; as[lk + 1][lr] = av.y; as[lk + 2][lr] = av.z; as[lk + 3][lr] = av.w;
+    ws[lk][lr] = wv.x; ws[lk + 1][lr] = wv.y; ws[lk + 2][lr] = wv.z; ws[lk + 3][lr] = wv.w;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      float x[4], y[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) { x[i] = as[k][ty * 4 + i]; y[i] = ws[k][tx * 4 + i]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], y[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m < M)
+      *reinterpret_cast<float4*>(out + static_cast<size_t>(m) * N + n0 + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+  }
+}
+
+// The same epilogue from the product rows [M][N_pad]: one CTA of eight warps per row.
+__global__ void __launch_bounds__(256) lin_epi_kernel(const __grid_constant__ LinParams p) {
+  pdl_wait();
+  const LinEpi& e = p.e;
+  const int m = blockIdx.x;
+  const float* acc = p.ws + static_cast<size_t>(m) * p.N_pad;
+  if (!e.stream) {
+    const float sc = row_rms_scale(e, m);
+    for (int n = threadIdx.x; n < e.n_plain; n += 256) e.out[static_cast<size_t>(m) * e.ldo + n] = acc[n] * sc;
+    const int tiles = p.N_pad / 256;
+    for (int i = threadIdx.x; i < (tiles - e.act_tile0) * 128; i += 256) {
+      const float* t = acc + static_cast<size_t>(e.act_tile0 + (i >> 7)) * 256 + (i & 127);
+      operand_store1(e.act, m, e.act_k0 + i, clamped_glu(t[0] * sc, t[128] * sc, e.limit, e.alpha));
+    }
+    return;
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int groups = (e.width + 127) / 128;
+  for (int g = warp; g < groups; g += 8) {
+    float sq = 0.f;
+    for (int n = g * 128 + lane; n < min(e.width, g * 128 + 128); n += 32) {
+      float* xr = e.x + static_cast<size_t>(m) * e.ldx + n;
+      const float v = (e.add ? *xr : 0.f) + (acc[n] + (e.bias ? e.bias[n] : 0.f));
+      *xr = v;
+      sq += v * v;
+      operand_store1(e.op, m, e.op_k0 + n, e.norm_w ? v * e.norm_w[n] : v);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    if (lane == 0 && e.ss_out != nullptr) e.ss_out[static_cast<size_t>(m) * e.ss_out_n + g] = sq;
+  }
+}
+
+// ------------------------------------------------------------------------------------ stream rows
+__global__ void __launch_bounds__(256) stream_embed_kernel(const __grid_constant__ StreamEmbedParams p) {
+  pdl_wait();
+  const int m = blockIdx.x;
+  const int id = min(max(p.ids[m], 0), p.vocab - 1);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int g = warp; g * 128 < p.width; g += 8) {
+    float sq = 0.f;
+    for (int n = g * 128 + lane; n < min(p.width, g * 128 + 128); n += 32) {
+      const size_t i = static_cast<size_t>(id) * p.width + n;
+      const float t = p.table_f32 ? static_cast<const float*>(p.table)[i] : __bfloat162float(static_cast<const __nv_bfloat16*>(p.table)[i]);
+      const float v = t * p.scale;
+      p.x[static_cast<size_t>(m) * ((p.width + 31) / 32 * 32) + n] = v;
+      sq += v * v;
+      if (p.x0_k0 >= 0) operand_store1(p.x0, m, p.x0_k0 + n, v);
+      operand_store1(p.op, m, p.op_k0 + n, p.norm_w ? v * p.norm_w[n] : v);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    if (lane == 0 && p.ss_out != nullptr) p.ss_out[static_cast<size_t>(m) * p.ss_out_n + g] = sq;
+  }
+}
+
+__global__ void __launch_bounds__(256) stream_norm_kernel(const __grid_constant__ StreamNormParams p) {
+  pdl_wait();
+  __shared__ float red[8];
+  const int i = blockIdx.x;
+  const float* x = p.x + static_cast<size_t>(p.rows ? p.rows[i] : i) * p.ldx;
+  float sq = 0.f;
+  for (int n = threadIdx.x; n < p.width; n += 256) sq += x[n] * x[n];
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
+  __syncthreads();
+  sq = 0.f;
+  for (int w = 0; w < 8; ++w) sq += red[w];
+  const float r = 1.f / sqrtf(sq / static_cast<float>(p.width) + p.eps);
+  for (int n = threadIdx.x; n < p.width; n += 256) operand_store1(p.op, i, n, x[n] * r * p.w[n]);
+}
+
+}  // namespace saber
+
+extern "C" int saber_linear_launches(const saber::LinParams* p) { return (p->fp32 || !p->fuse) ? 2 : 1; }
+
+extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t stream) {
+  using namespace saber;
+  const LinEpi& e = p->e;
+  if (p->M <= 0 || (p->N_pad & 255) || (p->K & 63) || p->K <= 0 || p->M > p->M_pad) return static_cast<int>(cudaErrorInvalidValue);
+  if (e.stream ? (e.width > p->N_pad || (e.ldx & 31) || e.x == nullptr)
+               : (e.n_plain > e.act_tile0 * 256 || e.act_tile0 * 256 > p->N_pad || (e.ldo & 3)))
+    return static_cast<int>(cudaErrorInvalidValue);
+  if (p->fp32) {
+    cudaError_t r = launch(lin_f32_kernel, dim3(p->N_pad / 64, (p->M + 63) / 64), dim3(256), 0, stream, 0, static_cast<const float*>(p->a),
+                           static_cast<const float*>(p->w), p->ws, p->M, p->N_pad, p->K);
+    if (r != cudaSuccess) return static_cast<int>(r);
+    return static_cast<int>(launch(lin_epi_kernel, dim3(p->M), dim3(256), 0, stream, 0, *p));
+  }
+  if (p->nt < 16 || p->nt > 128 || (p->nt & 15) || (p->M_pad % p->nt) || p->splits < 1) return static_cast<int>(cudaErrorInvalidValue);
+  const int KB = p->K >> 6;
+  const int kb_per = (KB + p->splits - 1) / p->splits;
+  if ((p->splits - 1) * kb_per >= KB) return static_cast<int>(cudaErrorInvalidValue);
+  LinParams q = *p;
+  if (!p->fuse) {
+    // product rows only: the split parts use the workspace behind them
+    q.e = LinEpi{};
+    q.e.out = p->ws;
+    q.e.ldo = p->N_pad;
+    q.e.n_plain = p->N_pad;
+    q.e.act_tile0 = p->N_pad / 256;
+    q.ws = p->ws + static_cast<size_t>(p->M) * p->N_pad;
+  }
+  static bool ready[64];
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
+  constexpr int kSmem = 224 * 1024;
+  if (!ready[dev]) {
+    cudaError_t r = cudaFuncSetAttribute(lin_bf16_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (r != cudaSuccess) return static_cast<int>(r);
+    ready[dev] = true;
+  }
+  const bool pair = p->mtiles == 2 && p->splits == 1 && p->nt == 128 && (p->M_pad / 128) % 2 == 0;
+  const int abytes = p->nt * 128 * (pair ? 2 : 1);
+  int stages = (kSmem - 1024) / (static_cast<int>(kLinTile) + abytes);
+  if (stages > kLinMaxStages) stages = kLinMaxStages;
+  const int smem = stages * (static_cast<int>(kLinTile) + abytes) + 1024;
+  const int tiles_m = pair ? (p->M + 255) / 256 : (p->M + p->nt - 1) / p->nt;
+  const dim3 grid(tiles_m, p->N_pad / 256, p->splits);
+  cudaError_t r = pair ? launch(lin_bf16_kernel<2>, grid, dim3(kLinThreads), smem, stream, 2, q, stages)
+                       : launch(lin_bf16_kernel<1>, grid, dim3(kLinThreads), smem, stream, 2, q, stages);
+  if (r != cudaSuccess || p->fuse) return static_cast<int>(r);
+  return static_cast<int>(launch(lin_epi_kernel, dim3(p->M), dim3(256), 0, stream, 0, *p));
+}
+
+extern "C" int saber_stream_embed_launch(const saber::StreamEmbedParams* p, cudaStream_t stream) {
+  if (p->M <= 0) return static_cast<int>(cudaErrorInvalidValue);
+  return static_cast<int>(saber::launch(saber::stream_embed_kernel, dim3(p->M), dim3(256), 0, stream, 0, *p));
+}
+
+extern "C" int saber_stream_norm_launch(const saber::StreamNormParams* p, cudaStream_t stream) {
+  if (p->n <= 0) return static_cast<int>(cudaErrorInvalidValue);
+  return static_cast<int>(saber::launch(saber::stream_norm_kernel, dim3(p->n), dim3(256), 0, stream, 0, *p));
+}

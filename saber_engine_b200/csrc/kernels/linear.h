@@ -1,0 +1,82 @@
+// Launch interface of the linears whose residual stream is fp32 (linear.cu): a bf16 x bf16 tcgen05
+// GEMM with the stream's epilogues, and the same linear in fp32 on the CUDA cores.  Plain C types only.
+#pragma once
+#include <cuda_runtime.h>
+#include <stdint.h>
+#include "operand.cuh"
+
+namespace saber {
+
+// What happens to acc[m][n] = sum_k a[m][k] w[n][k].  Two kinds:
+//   project  the operand rows are norm_w * x without the division by the root mean square, so the
+//            result is scaled by rsqrt(sum(ss[m]) * inv_width + eps) (ss: per-128-column sums of squares the
+//            stream epilogue left; null: scale 1).  Features below act_tile0 * 256 are stored as fp32
+//            (n < n_plain); from there on a 256-feature tile holds 128 gate then 128 up features of a
+//            clamped gated unit, whose products go to the operand `act`:
+//            g = min(gate, limit), u = clamp(up, -limit, limit), y = g sigmoid(alpha g) (u + 1)
+//   stream   x[m][n] = (add ? x[m][n] : 0) + bias[n] + acc, and the operand of the next linear:
+//            norm_w[n] x[m][n] with its sums of squares (ss_out), or x itself (norm_w null)
+struct LinEpi {
+  int stream;
+  const float* ss;
+  int ss_n;
+  float inv_width, eps;
+  float* out;
+  int ldo, n_plain, act_tile0;
+  Operand act;
+  int act_k0;
+  float limit, alpha;
+  float* x;
+  int ldx, width, add;
+  const float* bias;
+  const float* norm_w;
+  Operand op;
+  int op_k0;
+  float* ss_out;
+  int ss_out_n;
+};
+
+struct LinParams {
+  const void* w;        // bf16: [n_tile][k-block][32 KiB swizzled tile]; fp32: [N_pad][K]
+  const void* a;        // bf16: operand tiles; fp32: rows [M_pad][K]
+  float* ws;            // split-K partials (bf16), the [M][N_pad] product (unfused forms)
+  uint32_t* counters;   // one per output tile, zero between launches
+  uint32_t* err;
+  int M, M_pad, N_pad, K, nt, splits, fp32, fuse, mtiles;
+  LinEpi e;
+};
+
+// Rows of the stream from token ids: x = table[id] * scale, an optional second copy as the operand `x0`
+// (columns from x0_k0), and the first layer's operand as in the stream epilogue.
+struct StreamEmbedParams {
+  const void* table;    // bf16 or fp32 [vocab][width]
+  int table_f32, vocab;
+  const int32_t* ids;
+  int M, width;
+  float scale;
+  float* x;
+  Operand x0;
+  int x0_k0;            // < 0: none
+  const float* norm_w;
+  Operand op;
+  int op_k0;
+  float* ss_out;
+  int ss_out_n;
+};
+
+// Stream rows `rows[i]` (null: row i), root-mean-square normed, as an operand.
+struct StreamNormParams {
+  const float* x;
+  int ldx, width, n;
+  const int32_t* rows;
+  const float* w;
+  float eps;
+  Operand op;
+};
+
+}  // namespace saber
+
+extern "C" int saber_linear_launches(const saber::LinParams* p);
+extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t stream);
+extern "C" int saber_stream_embed_launch(const saber::StreamEmbedParams* p, cudaStream_t stream);
+extern "C" int saber_stream_norm_launch(const saber::StreamNormParams* p, cudaStream_t stream);

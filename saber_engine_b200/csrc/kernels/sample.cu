@@ -17,18 +17,40 @@ __device__ __forceinline__ bool better(float v, int i, float bv, int bi) {
   return v > bv || (v == bv && i < bi);
 }
 
+// A logit (bf16, or fp32 where the model keeps its logits in fp32) as fp32, and its order-preserving
+// unsigned key of the same width (larger key = larger value; NaN sorts lowest).
+__device__ __forceinline__ float logit_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float logit_f(float v) { return v; }
+__device__ __forceinline__ uint32_t logit_key(__nv_bfloat16 v) {
+  const uint32_t bits = __bfloat16_as_ushort(v);
+  if ((bits & 0x7FFFu) > 0x7F80u) return 0u;
+  return (bits & 0x8000u) ? (0xFFFFu ^ bits) : (bits | 0x8000u);
+}
+__device__ __forceinline__ uint32_t logit_key(float v) {
+  const uint32_t bits = __float_as_uint(v);
+  if ((bits & 0x7FFFFFFFu) > 0x7F800000u) return 0u;
+  return (bits & 0x80000000u) ? ~bits : (bits | 0x80000000u);
+}
+__device__ __forceinline__ float key_logit(uint32_t key, __nv_bfloat16) {
+  return __bfloat162float(__ushort_as_bfloat16(static_cast<uint16_t>((key & 0x8000u) ? (key & 0x7FFFu) : (0xFFFFu ^ key))));
+}
+__device__ __forceinline__ float key_logit(uint32_t key, float) {
+  return __uint_as_float((key & 0x80000000u) ? (key & 0x7FFFFFFFu) : ~key);
+}
+
 // grid = rows, block 1024. out_idx[r] = argmax (global id = local + id_offset), out_val[r] = value.
-__global__ void __launch_bounds__(1024) argmax_kernel(const __nv_bfloat16* logits, int ld, int V,
+template <typename T>
+__global__ void __launch_bounds__(1024) argmax_kernel(const T* logits, int ld, int V,
                                                       int id_offset, int32_t* out_idx,
                                                       float* out_val) {
   pdl_wait();
   __shared__ float sv[32];
   __shared__ int si[32];
   const int r = blockIdx.x;
-  const __nv_bfloat16* row = logits + static_cast<size_t>(r) * ld;
+  const T* row = logits + static_cast<size_t>(r) * ld;
   float bv = -INFINITY;
   int bi = V;  // "cols" when nothing finite/non-NaN was seen
-  const int nvec = V >> 3;
+  const int nvec = sizeof(T) == 2 ? V >> 3 : 0;
   for (int v = threadIdx.x; v < nvec; v += blockDim.x) {
     const uint4 raw = *reinterpret_cast<const uint4*>(row + v * 8);
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
@@ -40,7 +62,7 @@ __global__ void __launch_bounds__(1024) argmax_kernel(const __nv_bfloat16* logit
     }
   }
   for (int i = nvec * 8 + threadIdx.x; i < V; i += blockDim.x) {
-    const float f = __bfloat162float(row[i]);
+    const float f = logit_f(row[i]);
     if (f == f && better(f, i, bv, bi)) { bv = f; bi = i; }
   }
 #pragma unroll
@@ -69,90 +91,76 @@ __global__ void __launch_bounds__(1024) argmax_kernel(const __nv_bfloat16* logit
 }
 
 // ------------------------------------------------------------------------------- top-k seam
-// Order-preserving 16-bit key of a bf16 value (larger key = larger value; NaN sorts lowest).
-__device__ __forceinline__ uint32_t bf16_key(uint16_t bits) {
-  if ((bits & 0x7FFFu) > 0x7F80u) return 0u;  // NaN
-  return (bits & 0x8000u) ? (0xFFFFu ^ bits) & 0xFFFFu : (bits | 0x8000u);
-}
-
 // grid = rows, block 1024. Writes per row: ids[kSeamK], vals[kSeamK] (sorted: value desc, id asc),
 // lse[2] = log-sum-exp at temperature 1 and at temperature temps[r].
-__global__ void __launch_bounds__(1024) topk_seam_kernel(const __nv_bfloat16* logits, int ld, int V,
+template <typename T>
+__global__ void __launch_bounds__(1024) topk_seam_kernel(const T* logits, int ld, int V,
                                                          int id_offset, const float* temps,
                                                          int32_t* ids, float* vals, float* lse) {
   pdl_wait();
   __shared__ uint32_t hist[256];
-  __shared__ uint32_t sel_hi, sel_lo, above_hi, above_lo;
+  __shared__ uint32_t sel_prefix, sel_above;
   __shared__ float cand_v[kSeamK];
   __shared__ int cand_i[kSeamK];
   __shared__ uint32_t n_cand, n_tie;
   __shared__ int tie_i[256];
   __shared__ float red[64];
   const int r = blockIdx.x;
-  const uint16_t* row = reinterpret_cast<const uint16_t*>(logits + static_cast<size_t>(r) * ld);
+  const T* row = logits + static_cast<size_t>(r) * ld;
   const int tid = threadIdx.x;
 
-  // pass 1: histogram of the high byte of the key, row max for the lse
-  if (tid < 256) hist[tid] = 0;
-  __syncthreads();
+  // row maximum for the log-sum-exps
   float mx = -INFINITY;
   for (int i = tid; i < V; i += blockDim.x) {
-    const uint16_t bits = row[i];
-    atomicAdd(&hist[bf16_key(bits) >> 8], 1u);
-    const float f = __bfloat162float(__ushort_as_bfloat16(bits));
+    const float f = logit_f(row[i]);
     if (f == f) mx = fmaxf(mx, f);
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   if ((tid & 31) == 0) red[tid >> 5] = mx;
   __syncthreads();
-  if (tid == 0) {
-    uint32_t acc = 0;
-    int bin = 255;
-    for (; bin > 0; --bin) {
-      if (acc + hist[bin] >= kSeamK) break;
-      acc += hist[bin];
-    }
-    sel_hi = bin;
-    above_hi = acc;  // elements strictly above the selected high bin
-  }
   mx = red[0];
-  for (int w = 1; w < 32; ++w) mx = fmaxf(mx, red[w]);   // row maximum, same in every thread
-  __syncthreads();
-  const uint32_t hi = sel_hi;
-  const uint32_t above1 = above_hi;
-  __syncthreads();
-  if (tid < 256) hist[tid] = 0;
-  __syncthreads();
-  // pass 2: histogram of the low byte inside the selected high bin
-  for (int i = tid; i < V; i += blockDim.x) {
-    const uint32_t k = bf16_key(row[i]);
-    if ((k >> 8) == hi) atomicAdd(&hist[k & 255u], 1u);
-  }
-  __syncthreads();
-  if (tid == 0) {
-    uint32_t acc = above1;
-    int bin = 255;
-    for (; bin > 0; --bin) {
-      if (acc + hist[bin] >= kSeamK) break;
-      acc += hist[bin];
+  for (int w = 1; w < 32; ++w) mx = fmaxf(mx, red[w]);   // same in every thread
+  // radix select, a byte of the key per pass from the top: histogram of that byte among the keys that
+  // share the bytes selected so far
+  uint32_t prefix = 0, above = 0;                        // above: keys strictly greater than the selection
+  for (int byte = static_cast<int>(sizeof(T)) - 1; byte >= 0; --byte) {
+    __syncthreads();
+    if (tid < 256) hist[tid] = 0;
+    __syncthreads();
+    for (int i = tid; i < V; i += blockDim.x) {
+      const uint64_t k = logit_key(row[i]);
+      if ((k >> (8 * (byte + 1))) == prefix) atomicAdd(&hist[(k >> (8 * byte)) & 255u], 1u);
     }
-    sel_lo = bin;
-    above_lo = acc;  // elements with key strictly above the threshold key
+    __syncthreads();
+    if (tid == 0) {
+      uint32_t acc = above;
+      int bin = 255;
+      for (; bin > 0; --bin) {
+        if (acc + hist[bin] >= kSeamK) break;
+        acc += hist[bin];
+      }
+      sel_prefix = (prefix << 8) | static_cast<uint32_t>(bin);
+      sel_above = acc;
+    }
+    __syncthreads();
+    prefix = sel_prefix;
+    above = sel_above;
+  }
+  if (tid == 0) {
     n_cand = 0;
     n_tie = 0;
   }
   __syncthreads();
-  const uint32_t thr = (hi << 8) | sel_lo;
-  const uint32_t n_above = above_lo;
+  const uint32_t thr = prefix;
+  const uint32_t n_above = above;
   // pass 3: collect everything above the threshold key; ties at the threshold by ascending id
   float s1 = 0.f, sT = 0.f;
   const float invT = temps ? 1.f / fmaxf(temps[r], 1e-6f) : 1.f;
   const float mxs = mx == -INFINITY ? 0.f : mx;
   for (int i = tid; i < V; i += blockDim.x) {
-    const uint16_t bits = row[i];
-    const uint32_t k = bf16_key(bits);
-    const float f = __bfloat162float(__ushort_as_bfloat16(bits));
+    const uint32_t k = logit_key(row[i]);
+    const float f = logit_f(row[i]);
     if (f == f) {
       s1 += __expf(f - mxs);
       sT += __expf((f - mxs) * invT);
@@ -182,8 +190,7 @@ __global__ void __launch_bounds__(1024) topk_seam_kernel(const __nv_bfloat16* lo
     // threshold values keeps an arbitrary 256 of them, lowest ids among those)
     const int need = kSeamK - static_cast<int>(n_above);
     const int nt = min(static_cast<int>(n_tie), 256);
-    const float tv = __bfloat162float(__ushort_as_bfloat16(
-        static_cast<uint16_t>((thr & 0x8000u) ? (thr & 0x7FFFu) : (0xFFFFu ^ thr))));
+    const float tv = key_logit(thr, T{});
     for (int j = 0; j < need; ++j) {
       int best = -1;
       for (int q = 0; q < nt; ++q)
@@ -251,35 +258,44 @@ __global__ void verify_accept_kernel(const VerifyParams p) {
 
 }  // namespace saber
 
-extern "C" int saber_argmax_launch(const void* logits, int rows, int ld, int V, int id_offset,
+extern "C" int saber_argmax_launch(const void* logits, int f32, int rows, int ld, int V, int id_offset,
                                    int32_t* out_idx, float* out_val, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (ld & 7) return static_cast<int>(cudaErrorInvalidValue);
-  saber::launch(saber::argmax_kernel, dim3(rows), dim3(1024), 0, stream, 0, static_cast<const __nv_bfloat16*>(logits), ld, V,
-                                                  id_offset, out_idx, out_val);
+  if (f32)
+    saber::launch(saber::argmax_kernel<float>, dim3(rows), dim3(1024), 0, stream, 0, static_cast<const float*>(logits), ld, V, id_offset,
+                  out_idx, out_val);
+  else
+    saber::launch(saber::argmax_kernel<__nv_bfloat16>, dim3(rows), dim3(1024), 0, stream, 0, static_cast<const __nv_bfloat16*>(logits), ld, V,
+                  id_offset, out_idx, out_val);
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int saber_topk_seam_launch(const void* logits, int rows, int ld, int V, int id_offset,
+extern "C" int saber_topk_seam_launch(const void* logits, int f32, int rows, int ld, int V, int id_offset,
                                       const float* temps, int32_t* ids, float* vals, float* lse,
                                       cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (V < saber::kSeamK) return static_cast<int>(cudaErrorInvalidValue);
-  saber::launch(saber::topk_seam_kernel, dim3(rows), dim3(1024), 0, stream, 0, static_cast<const __nv_bfloat16*>(logits), ld,
-                                                     V, id_offset, temps, ids, vals, lse);
+  if (f32)
+    saber::launch(saber::topk_seam_kernel<float>, dim3(rows), dim3(1024), 0, stream, 0, static_cast<const float*>(logits), ld, V, id_offset,
+                  temps, ids, vals, lse);
+  else
+    saber::launch(saber::topk_seam_kernel<__nv_bfloat16>, dim3(rows), dim3(1024), 0, stream, 0, static_cast<const __nv_bfloat16*>(logits),
+                  ld, V, id_offset, temps, ids, vals, lse);
   return static_cast<int>(cudaGetLastError());
 }
 
 namespace saber {
 // out[m] = logits[m][ids[m] - id_offset] as fp32, or -inf when ids[m] lies outside [id_offset, id_offset + V)
 // (a row without a successor carries -1).  One thread per row.
-__global__ void logit_gather_kernel(const __nv_bfloat16* logits, int ld, int V, int id_offset,
+template <typename T>
+__global__ void logit_gather_kernel(const T* logits, int ld, int V, int id_offset,
                                     const int32_t* ids, float* out, int rows) {
   pdl_wait();
   const int m = blockIdx.x * blockDim.x + threadIdx.x;
   if (m >= rows) return;
   const int id = ids[m] - id_offset;
-  out[m] = (id >= 0 && id < V) ? __bfloat162float(logits[static_cast<size_t>(m) * ld + id]) : -INFINITY;
+  out[m] = (id >= 0 && id < V) ? logit_f(logits[static_cast<size_t>(m) * ld + id]) : -INFINITY;
 }
 }  // namespace saber
 
@@ -341,11 +357,15 @@ extern "C" int saber_sample_seam_launch(const int32_t* ids, const float* vals, c
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int saber_logit_gather_launch(const void* logits, int rows, int ld, int V, int id_offset,
+extern "C" int saber_logit_gather_launch(const void* logits, int f32, int rows, int ld, int V, int id_offset,
                                          const int32_t* ids, float* out, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  saber::launch(saber::logit_gather_kernel, dim3((rows + 127) / 128), dim3(128), 0, stream, 0,
-                static_cast<const __nv_bfloat16*>(logits), ld, V, id_offset, ids, out, rows);
+  if (f32)
+    saber::launch(saber::logit_gather_kernel<float>, dim3((rows + 127) / 128), dim3(128), 0, stream, 0,
+                  static_cast<const float*>(logits), ld, V, id_offset, ids, out, rows);
+  else
+    saber::launch(saber::logit_gather_kernel<__nv_bfloat16>, dim3((rows + 127) / 128), dim3(128), 0, stream, 0,
+                  static_cast<const __nv_bfloat16*>(logits), ld, V, id_offset, ids, out, rows);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -40,13 +40,14 @@ struct DraftIndexParams {
 
 extern "C" int saber_draft_index_launch(const saber::DraftIndexParams* p, cudaStream_t stream);
 
-extern "C" int saber_argmax_launch(const void* logits, int rows, int ld, int V, int id_offset,
+// f32: the logits are fp32 (1) or bf16 (0).
+extern "C" int saber_argmax_launch(const void* logits, int f32, int rows, int ld, int V, int id_offset,
                                    int32_t* out_idx, float* out_val, cudaStream_t stream);
-extern "C" int saber_topk_seam_launch(const void* logits, int rows, int ld, int V, int id_offset,
+extern "C" int saber_topk_seam_launch(const void* logits, int f32, int rows, int ld, int V, int id_offset,
                                       const float* temps, int32_t* ids, float* vals, float* lse,
                                       cudaStream_t stream);
 extern "C" int saber_verify_launch(const saber::VerifyParams* p, cudaStream_t stream);
 extern "C" int saber_sample_seam_launch(const int32_t* ids, const float* vals, const float* samp, const float* u,
                                         int32_t* picks, int rows, cudaStream_t stream);
-extern "C" int saber_logit_gather_launch(const void* logits, int rows, int ld, int V, int id_offset,
+extern "C" int saber_logit_gather_launch(const void* logits, int f32, int rows, int ld, int V, int id_offset,
                                          const int32_t* ids, float* out, cudaStream_t stream);

@@ -224,6 +224,12 @@ class TinyQwen3Config:
 
 
 def by_name(name: str):
+    """A built-in description, or the folder of a model described by its config.json."""
+    from . import stack_config
+    if name in stack_config.NAMED:
+        return stack_config.NAMED[name]()
+    if stack_config.is_model_dir(name):
+        return stack_config.load_dir(name)
     table = {"qwen38-27b": qwen38_27b, "flashnext-moe": flashnext_moe,
              "flashnext-ref": lambda: flashnext_moe(True), "hybrid-mini": scaled_hybrid,
              "qwen38-27b-mxfp4": lambda: dataclasses.replace(qwen38_27b(), name="qwen38-27b-mxfp4", weight_format="mxfp4"),
@@ -234,7 +240,7 @@ def by_name(name: str):
                                                              drafter=dataclasses.replace(qwen38_27b().drafter, attn_layers=1)),
              "tiny-qwen3": TinyQwen3Config}
     if name not in table:
-        raise KeyError(f"unknown model {name!r}; known: {sorted(table)}")
+        raise KeyError(f"unknown model {name!r}; known: {sorted([*table, *stack_config.NAMED])}, or a folder with a config.json")
     return table[name]()
 
 

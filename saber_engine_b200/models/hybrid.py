@@ -16,7 +16,6 @@ from __future__ import annotations
 
 import ctypes as C
 import math
-from dataclasses import dataclass, field
 from typing import Optional
 
 import torch
@@ -25,90 +24,9 @@ from ..ops import functional as F
 from ..ops import layouts as L
 from ..ops import native as N
 from .config import HybridConfig, shard
+from .step import (BlobLayout, Bucket, SeqStep, StepResult, fill_blob, finish_bucket, head_outputs, parse_result,  # noqa: F401
+                   run_bucket, seam_outputs)
 from .weights import ModelWeights, random_init
-
-
-@dataclass
-class BlobLayout:
-    """Offsets (in int32 words) of the per-step index tables inside a bucket's index blob."""
-    M: int
-    nseq: int
-    max_blocks: int
-    ids: int = 0
-    pos: int = 0
-    slot_map: int = 0
-    cu_rows: int = 0
-    slots: int = 0
-    shift: int = 0
-    kv_len: int = 0
-    seq_uid: int = 0
-    step_no: int = 0
-    last_rows: int = 0
-    temps: int = 0
-    next_ids: int = 0          # per row: the token that follows it in its prompt (-1: none), for prompt log-probabilities
-    samp: int = 0              # per HEAD row: fp32 {temperature, top_k, top_p, min_p} (temperature 0: keep the greedy pick)
-    samp_u: int = 0            # per HEAD row: the uniform number of the draw (fp32)
-    block_table: int = 0
-    words: int = 0
-
-    @staticmethod
-    def make(M: int, nseq: int, max_blocks: int) -> "BlobLayout":
-        b = BlobLayout(M, nseq, max_blocks)
-        off = 0
-        def take(n):
-            nonlocal off
-            o = off
-            off += (n + 3) // 4 * 4          # keep every table 16-byte aligned
-            return o
-        b.ids = take(M)
-        b.pos = take(3 * M)
-        b.slot_map = take(M)
-        b.cu_rows = take(nseq + 1)
-        b.slots = take(nseq)
-        b.shift = take(nseq)
-        b.kv_len = take(nseq)
-        b.seq_uid = take(nseq)
-        b.step_no = take(nseq)
-        b.last_rows = take(nseq)
-        b.temps = take(M)
-        b.next_ids = take(M)
-        b.samp = take(4 * M)
-        b.samp_u = take(M)
-        b.block_table = take(nseq * max_blocks)
-        b.words = off
-        return b
-
-    @property
-    def header_words(self) -> int:
-        return self.block_table
-
-
-@dataclass
-class Bucket:
-    """One planned shape: its program, blob layout, output tensors."""
-    kind: str                 # "decode" | "prefill"
-    nseq: int
-    width: int                # rows per sequence (decode) or rung rows (prefill, nseq sequences packed)
-    M: int
-    layout: BlobLayout
-    program: N.Program
-    blob_dev: torch.Tensor    # int32 [words]
-    blob_host: torch.Tensor   # pinned int32 [words]
-    out_dev: torch.Tensor     # int32: n_commit[nseq] | out_tokens[nseq*W] | drafts[nseq*block] | picks[M]
-    out_host: torch.Tensor    # pinned mirror
-    captured: bool = False
-    n_launches: int = 0
-    logits: Optional[torch.Tensor] = None
-    keep: list = field(default_factory=list)
-    bt_rows: dict = field(default_factory=dict)    # row j -> (blocks_key, n blocks) of the block-table row the device holds
-    last_h2d_bytes: int = 0                        # index-table bytes the last step copied to the device
-    arenas: list = field(default_factory=list)     # pure activation buffers: written before read in every step
-    digests: Optional[torch.Tensor] = None         # int64 [n_layers + 1] stage digests (race_check = "shadow")
-    sp: bool = False                               # prefill on several ranks: the sequence-parallel chain (rows owned by ranks)
-    seam_dev: Optional[torch.Tensor] = None        # int32 blob: ids [Mh*64] | values [Mh*64] fp32 bits | lse [Mh*2] (seam buckets)
-    seam_host: Optional[torch.Tensor] = None       # pinned mirror
-    plp_dev: Optional[torch.Tensor] = None         # int32 blob of a prompt-log-probability bucket (every row: candidates, lse, next-token logit)
-    plp_host: Optional[torch.Tensor] = None
 
 
 class HybridModel:
@@ -223,6 +141,24 @@ class HybridModel:
             for i in self.gdn_state:
                 self.gdn_state[i][slot].zero_()
                 self.gdn_hist[i][slot].zero_()
+
+    def page_pools(self) -> dict:
+        """Tensors addressed by physical page: what a parked or shared sequence owns page by page."""
+        return {**{f"kv.{i}": t for i, t in self.kv.items()}, **{f"draft_kv.{i}": t for i, t in self.draft_kv.items()}}
+
+    def slot_tensors(self) -> dict:
+        """Tensors addressed by state slot."""
+        out = {}
+        for i in self.gdn_state:
+            out[f"gdn_state.{i}"], out[f"gdn_stash.{i}"], out[f"gdn_hist.{i}"] = self.gdn_state[i], self.gdn_stash[i], self.gdn_hist[i]
+        return out
+
+    def snapshot_views(self, slot: int) -> dict:
+        """What of a slot a prefix-cache snapshot holds after a committed portion (the rest is zero then)."""
+        out = {}
+        for i in self.gdn_state:
+            out[f"gdn_state.{i}"], out[f"gdn_hist.{i}"] = self.gdn_state[i][slot], self.gdn_hist[i][slot, :3]
+        return out
 
     def state_bytes(self) -> dict:
         kv = sum(t.numel() for t in self.kv.values())
@@ -629,11 +565,8 @@ class HybridModel:
         W = width if decode else 1
         block = cfg.drafter.block if self.use_drafter else 0
         # outputs: n_commit[nseq] | out_tokens[nseq * W] | drafts[nseq * block] | picks[Mh]
-        n_out = nseq + nseq * W + nseq * max(block, 1) + Mh
-        out = torch.zeros(n_out, dtype=torch.int32, device=dev)
-        o_commit, o_tokens = out[:nseq], out[nseq:nseq + nseq * W]
+        out, o_commit, o_tokens, o_picks = head_outputs(nseq, W, block, Mh, dev)
         o_drafts = out[nseq + nseq * W: nseq + nseq * W + nseq * max(block, 1)]
-        o_picks = out[nseq + nseq * W + nseq * max(block, 1):]
         accept_row = torch.zeros(nseq, dtype=torch.int32, device=dev)
         bonus = torch.zeros(nseq, dtype=torch.int32, device=dev)
         pick_val = torch.zeros(Mh, dtype=torch.float32, device=dev)
@@ -666,11 +599,7 @@ class HybridModel:
             ar_site += 1
         seam_dev = None
         if self._want_seam:
-            # one int32 blob so that the read-back is one copy: ids | values (fp32 bits) | lse pairs
-            seam_dev = torch.zeros(Mh * (2 * N.SEAM_K + 2), dtype=torch.int32, device=dev)
-            s_ids = seam_dev[:Mh * N.SEAM_K]
-            s_vals = seam_dev[Mh * N.SEAM_K: 2 * Mh * N.SEAM_K].view(torch.float32)
-            s_lse = seam_dev[2 * Mh * N.SEAM_K:].view(torch.float32)
+            seam_dev, s_ids, s_vals, s_lse = seam_outputs(Mh, dev)
             prog.seam(logits, Mh, logits.stride(0), sh.vocab, sh.vocab_first, None, s_ids, s_vals, s_lse, tag="topk_seam")
             if self.tp > 1:
                 # vocabulary-sharded ranks swap their candidates through the symmetric heap and merge them
@@ -827,156 +756,5 @@ class HybridModel:
         self._flush(prog)
         if self.fuse:
             prog.link_prefetch()
-        head = self._last_head
-        out = head["out"]
-        out_host = torch.zeros(out.numel(), dtype=torch.int32).pin_memory()
-        prog.keep(*[k for k in keep if k is not None], self.w)
-        b = Bucket(kind, nseq, width, M, lay, prog, blob, blob_host, out, out_host,
-                   n_launches=prog.declared_launches, logits=head["logits"], keep=keep)
-        b.W, b.block, b.Mh = head["W"], head["block"], head["Mh"]
-        b.seam_dev = head.get("seam")
-        b.plp_dev = head.get("plp")
-        b.plp_logits = getattr(self, "_plp_logits", None) if b.plp_dev is not None else None
-        b.plp_host = torch.zeros(b.plp_dev.numel(), dtype=torch.int32).pin_memory() if b.plp_dev is not None else None
-        b.seam_host = torch.zeros(b.seam_dev.numel(), dtype=torch.int32).pin_memory() if b.seam_dev is not None else None
-        if capture:
-            # one eager walk first: sets function attributes and warms lazy module loading
-            with torch.cuda.stream(self.stream):
-                prog.run(self.stream)
-                self.stream.synchronize()
-                self.scratch.check()
-                prog.capture(self.stream)
-            self.stream.synchronize()
-            b.captured = True
-        self.buckets[self._bucket_key] = b
-        return b
-
-
-@dataclass
-class SeqStep:
-    """What one sequence contributes to a step."""
-    tokens: list              # token ids of this step's rows (decode: [last committed, drafts...])
-    pos0: int                 # position of the first row
-    slot: int                 # GDN state slot (>= 1)
-    shift: int                # rows of the previous decode step that were committed (0 after prefill)
-    blocks: list              # physical KV block ids covering positions [0, pos0 + len(tokens))
-    uid: int = 0
-    step_no: int = 0
-    rope_pos: Optional[object] = None   # int [3, rows]: three-axis rotary positions of the rows (prompts with images)
-    rope_delta: int = 0       # added to the index of every row for the rotary position (after an image)
-    next_token: int = -1      # the prompt token after this chunk's last row (-1: none), for prompt log-probabilities
-    sampling: Optional[tuple] = None   # (temperature, top_k, top_p, min_p) of a sampled sequence the device may draw for
-    uniforms: Optional[list] = None    # one uniform number per head row of this step (decode: every row; prefill: the last)
-    blocks_key: Optional[object] = None   # identity of `blocks` (same key = same list contents): the block table row is then uploaded once
-
-
-@dataclass
-class StepResult:
-    n_commit: list            # per sequence: tokens committed (decode) / 1 (prefill last chunk)
-    tokens: list              # per sequence: committed token ids
-    drafts: list              # per sequence: next block of draft tokens
-    picks: list
-
-
-def fill_blob(b: Bucket, seqs: list, page_tokens: int = 16) -> list:
-    """Write the index tables of one step into the bucket's pinned blob.  Returns the word ranges
-    [(first, count), ...] that have to reach the device: the header (every per-row and per-sequence
-    table) and the block-table rows that changed.  A sequence's KV blocks are allocated up front
-    and never change, so a row whose `blocks_key` is the one the device already holds is skipped:
-    in steady-state decode no block-table byte crosses the bus (the reference sends the table only
-    on page-crossing steps, `crates/saber-engine/src/tp2.rs:1897`)."""
-    import numpy as np
-    lay = b.layout
-    a = b.blob_host.numpy()
-    M, nseq = lay.M, lay.nseq
-    hdr = lay.header_words
-    a[:hdr] = 0
-    a[lay.slot_map:lay.slot_map + M] = -1
-    a[lay.next_ids:lay.next_ids + M] = -1
-    a[lay.slots:lay.slots + nseq] = -1
-    ranges = [(0, hdr)]
-    row = 0
-    for j, s in enumerate(seqs):
-        n = len(s.tokens)
-        a[lay.ids + row: lay.ids + row + n] = s.tokens
-        a[lay.next_ids + row: lay.next_ids + row + n] = list(s.tokens[1:]) + [s.next_token]
-        if s.sampling is not None and s.uniforms:
-            hr0, hn = (row, n) if b.kind == "decode" else (j, 1)      # head rows of this sequence
-            fa = a.view(np.float32)
-            for r in range(min(hn, len(s.uniforms))):
-                fa[lay.samp + 4 * (hr0 + r): lay.samp + 4 * (hr0 + r) + 4] = s.sampling
-                fa[lay.samp_u + hr0 + r] = s.uniforms[r]
-        pos = np.arange(s.pos0, s.pos0 + n, dtype=np.int32)
-        for ax in range(3):
-            a[lay.pos + ax * M + row: lay.pos + ax * M + row + n] = \
-                pos + s.rope_delta if s.rope_pos is None else np.asarray(s.rope_pos[ax], dtype=np.int32)[:n]
-        nblk = len(s.blocks)
-        first_page, last_page = s.pos0 // page_tokens, (s.pos0 + n - 1) // page_tokens
-        touched = np.asarray(s.blocks[first_page:last_page + 1], dtype=np.int32)     # pages this step's rows write
-        a[lay.slot_map + row: lay.slot_map + row + n] = touched[pos // page_tokens - first_page] * page_tokens + pos % page_tokens
-        a[lay.cu_rows + j] = row
-        a[lay.slots + j] = s.slot
-        a[lay.shift + j] = s.shift
-        a[lay.kv_len + j] = s.pos0 + n
-        a[lay.seq_uid + j] = s.uid
-        a[lay.step_no + j] = s.step_no
-        a[lay.last_rows + j] = row + n - 1
-        bt = lay.block_table + j * lay.max_blocks
-        sig = (s.blocks_key, nblk) if s.blocks_key is not None else None
-        held = getattr(b, "bt_rows", None)
-        if sig is None or held is None or held.get(j) != sig:
-            a[bt: bt + nblk] = np.asarray(s.blocks, dtype=np.int32)
-            ranges.append((bt, nblk))
-            if held is not None:
-                held[j] = sig
-        row += n
-    for j in range(len(seqs), nseq + 1):
-        a[lay.cu_rows + j] = row
-    assert row <= M, (row, M)
-    return ranges
-
-
-def run_bucket(model: "HybridModel", b: Bucket, seqs: list, eager: bool = False) -> StepResult:
-    """One step: index tables host->device (pinned; only what changed), the program (graph replay
-    or eager walk), results device->host, then parse."""
-    ranges = fill_blob(b, seqs, model.cfg.page_tokens)
-    st = model.stream
-    with torch.cuda.stream(st):
-        nbytes = 0
-        for first, count in ranges:
-            if count > 0:
-                b.blob_dev[first:first + count].copy_(b.blob_host[first:first + count], non_blocking=True)
-                nbytes += 4 * count
-        b.last_h2d_bytes = nbytes
-        if b.captured and not eager:
-            b.program.replay(st)
-        else:
-            b.program.run(st)
-        b.out_host.copy_(b.out_dev, non_blocking=True)
-        if getattr(b, "seam_dev", None) is not None:
-            b.seam_host.copy_(b.seam_dev, non_blocking=True)
-        if getattr(b, "plp_dev", None) is not None:
-            b.plp_host.copy_(b.plp_dev, non_blocking=True)
-    # bounded: a step that never completes (a kernel wait that did not run out, a lost peer) raises,
-    # and the scheduler's fatal law ends the engine instead of leaving this thread blocked
-    from ..runtime.device_rt import bounded_wait
-    bounded_wait(st, model.step_timeout_s, f"the {b.kind} step")
-    return parse_result(b, len(seqs))
-
-
-def parse_result(b: Bucket, n_live: int) -> StepResult:
-    o = b.out_host.numpy()
-    nseq, W, block, Mh = b.nseq, b.W, b.block, b.Mh
-    o_commit = o[:nseq]
-    o_tokens = o[nseq:nseq + nseq * W].reshape(nseq, W)
-    nd = max(block, 1)
-    o_drafts = o[nseq + nseq * W: nseq + nseq * W + nseq * nd].reshape(nseq, nd)
-    o_picks = o[nseq + nseq * W + nseq * nd:]
-    if b.kind == "decode":
-        n_commit = [int(o_commit[j]) for j in range(n_live)]
-        tokens = [o_tokens[j, :n_commit[j]].tolist() for j in range(n_live)]
-    else:
-        n_commit = [1] * n_live
-        tokens = [[int(o_picks[j])] for j in range(n_live)]
-    drafts = [o_drafts[j, :block].tolist() for j in range(n_live)]
-    return StepResult(n_commit, tokens, drafts, o_picks.tolist())
+        return finish_bucket(self, prog, self._bucket_key, kind, nseq, width, M, lay, blob, blob_host, keep, capture,
+                             dict(self._last_head, plp_logits=getattr(self, "_plp_logits", None)))

@@ -1,0 +1,339 @@
+"""A decoder assembled from a list of layers (`models.stack_config.StackConfig`) as native step programs.
+
+The parallel residual layer  x <- x + mixer(norm(x)) + ff(norm(x))  is two linears around the mixer's kernels.
+The residual stream stays fp32; a layer's output linear adds both sublayers to it and leaves the next linear's
+operand (norm weight times x) with the row's partial sums of squares, so that no normalisation, activation or
+addition needs a launch of its own.  Decode launches per layer: delta 3 (project, step, out), latent attention
+2 + 4; a pass of the looped block adds one linear.
+
+Every row of every bucket is committed (no drafter): a decode bucket is one row per sequence, a prefill bucket
+is `width` ragged rows of up to `nseq` sequences, single decoded tokens beside portions of prompts included.
+Caches and states belong to a layer RUN: the pages of a latent-attention run, the slots of a delta run.
+"""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from ..ops import functional as F
+from ..ops import layouts as L
+from ..ops import native as N
+from . import stack_weights as SW
+from .stack_config import DeltaMixer, LatentMixer, StackConfig
+from .step import BlobLayout, Bucket, finish_bucket, head_outputs, plp_outputs, seam_outputs
+
+
+class StackModel:
+    def __init__(self, cfg: StackConfig, device="cuda", max_seqs: int = 8, max_ctx: Optional[int] = None, kv_blocks: Optional[int] = None,
+                 weights: Optional[SW.StackWeights] = None, seed: int = 0, dtype: torch.dtype = torch.bfloat16, fuse: bool = True,
+                 expand_bytes: int = 24 << 30, race_check: str = "off", n_slots: Optional[int] = None):
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError("dtype must be bfloat16 or float32")
+        if race_check not in ("off", "shadow"):
+            raise ValueError("race_check must be 'off' or 'shadow'")
+        self.cfg, self.tp, self.rank, self.comm = cfg, 1, 0, None
+        self.dtype, self.f32 = dtype, dtype == torch.float32
+        self.device = torch.device(device)
+        self.max_seqs, self.max_width = max_seqs, 1
+        self.max_ctx = max_ctx or cfg.max_ctx
+        self.max_blocks = (self.max_ctx + cfg.page_tokens - 1) // cfg.page_tokens
+        self.kv_blocks = kv_blocks if kv_blocks is not None else max_seqs * self.max_blocks + 1
+        self.fuse, self.race_check, self.image_rows = bool(fuse), race_check, 0
+        self.step_timeout_s = 120.0
+        self.scratch = F.scratch(self.device)
+        dev = self.device
+        if weights is not None:
+            self.w = weights
+        elif cfg.source is not None:
+            self.w = SW.load(cfg, cfg.source, dtype, dev)
+        else:
+            self.w = SW.random_init(cfg, dtype, dev, seed)
+        self.n_slots = max_seqs + 1                       # slot 0 is the null slot
+        self.kv, self.delta_state, self.delta_hist = {}, {}, {}
+        for r in cfg.runs:
+            m = cfg.layers[r.layer].mixer
+            if isinstance(m, LatentMixer):
+                self.kv[r.index] = torch.zeros(self.kv_blocks, cfg.page_tokens, m.rank_pad + m.rot_pad, dtype=dtype, device=dev)
+            else:
+                self.delta_state[r.index] = torch.zeros(self.n_slots, m.heads, m.vdim_pad, m.dim_pad, dtype=torch.float32, device=dev)
+                self.delta_hist[r.index] = torch.zeros(self.n_slots, m.taps, m.channels, dtype=torch.float32, device=dev)
+        # expanded keys / values of the pages a prompt portion sees: scratch of one layer run at a time, in
+        # physical page order (absent when it would not fit its budget: the absorbed form serves then)
+        self.k_exp = self.v_exp = None
+        lat = [l.mixer for l in cfg.layers if isinstance(l.mixer, LatentMixer)]
+        tokens = self.kv_blocks * cfg.page_tokens
+        if lat and not self.f32 and tokens * cfg.expanded_token_bytes() <= expand_bytes:
+            self.k_exp = torch.zeros(tokens * max(m.heads * (m.dim_pad + m.rot_pad) for m in lat), dtype=dtype, device=dev)
+            self.v_exp = torch.zeros(tokens * max(m.heads * m.vdim_pad for m in lat), dtype=dtype, device=dev)
+        self.buckets: dict = {}
+        self.stream = torch.cuda.Stream(device=dev)
+        torch.cuda.synchronize(dev)                       # buckets run on a stream of their own
+
+    # ------------------------------------------------------------------------------ state
+    def reset_slot(self, slot: int) -> None:
+        with torch.cuda.stream(self.stream):
+            for i in self.delta_state:
+                self.delta_state[i][slot].zero_()
+                self.delta_hist[i][slot].zero_()
+
+    def page_pools(self) -> dict:
+        return {f"kv.{i}": t for i, t in self.kv.items()}
+
+    def slot_tensors(self) -> dict:
+        out = {}
+        for i in self.delta_state:
+            out[f"delta_state.{i}"], out[f"delta_hist.{i}"] = self.delta_state[i], self.delta_hist[i]
+        return out
+
+    def snapshot_views(self, slot: int) -> dict:
+        return {k: t[slot] for k, t in self.slot_tensors().items()}
+
+    def state_bytes(self) -> dict:
+        size = lambda d: sum(t.numel() * t.element_size() for t in d.values())    # noqa: E731
+        exp = 0 if self.k_exp is None else (self.k_exp.numel() + self.v_exp.numel()) * 2
+        return {"weights": self.w.nbytes(), "kv_pool": size(self.kv), "delta": size(self.delta_state) + size(self.delta_hist),
+                "expanded_kv_scratch": exp}
+
+    # ------------------------------------------------------------------------------ builders
+    def _operand(self, t: torch.Tensor, M: int, K: int) -> N.Operand:
+        o = N.Operand()
+        o.p, o.M_pad, o.ld, o.fmt = t.data_ptr(), L.padded_rows(M), K, int(self.f32)
+        return o
+
+    def _operand_buf(self, M: int, K: int) -> torch.Tensor:
+        """Zeroed storage of a [M, K] operand: padding rows and columns stay zero."""
+        return torch.zeros(L.padded_rows(M) * L.round_up(K, 64), dtype=self.dtype, device=self.device)
+
+    def _linear(self, prog: N.Program, lin: SW.Linear, a: torch.Tensor, M: int, e: N.LinEpi, ws: Optional[torch.Tensor], tag: str) -> None:
+        p = N.LinParams()
+        sc = self.scratch
+        p.w, p.a, p.err = lin.w.data_ptr(), a.data_ptr(), sc.err.data_ptr()
+        p.ws, p.counters = (ws if ws is not None else sc.ws).data_ptr(), sc.counters.data_ptr()
+        p.M, p.M_pad, p.N_pad, p.K = M, L.padded_rows(M), lin.N_pad, lin.K
+        p.nt, p.fp32, p.fuse, p.splits, p.mtiles = L.token_tile(M), int(self.f32), int(self.fuse), 1, 1
+        if not self.f32:
+            tiles, kb = lin.N_pad // 256 * ((M + p.nt - 1) // p.nt), lin.K // 64
+            p.splits = F.stream_splits(tiles, kb)
+            p.mtiles = 2 if (M > 128 and tiles > F.device_sms() and p.M_pad % 256 == 0) else 1
+        p.e = e
+        prog.linear(p, tag=tag)
+
+    def _row_norm(self, e: N.LinEpi, ss: torch.Tensor) -> None:
+        """The operand's rows were left undivided: scale the product by the row's reciprocal root mean square."""
+        e.ss, e.ss_n = ss.data_ptr(), ss.shape[1]
+        e.inv_width, e.eps = 1.0 / self.cfg.width, self.cfg.eps
+
+    def _stream_epi(self, x: torch.Tensor, add: bool, target: tuple, bias: Optional[torch.Tensor] = None) -> N.LinEpi:
+        """target: (operand, first column, norm weight or None, sums of squares or None) of the next linear."""
+        e = N.LinEpi()
+        op, k0, norm_w, ss = target
+        e.stream, e.x, e.ldx, e.width, e.add = 1, x.data_ptr(), x.stride(0), self.cfg.width, int(add)
+        e.bias, e.norm_w = N.ptr(bias), N.ptr(norm_w)
+        e.op, e.op_k0 = op, k0
+        if ss is not None:
+            e.ss_out, e.ss_out_n = ss.data_ptr(), ss.shape[1]
+        return e
+
+    def build_bucket(self, kind: str, nseq: int, width: int, capture: bool = True, seam: bool = False, plp: bool = False) -> Bucket:
+        """kind = 'decode': one row of each of nseq sequences.  kind = 'prefill': up to nseq sequences packed in
+        `width` rows.  seam: the best candidates of every head row for the host sampler.  plp: the head over
+        EVERY row, with the candidates and the logit of the row's successor."""
+        key = ((kind, nseq, width, "seam") if seam else (kind, nseq, width))
+        if plp:
+            if kind != "prefill":
+                raise ValueError("prompt log-probabilities: prefill buckets only")
+            key = key + ("plp",)
+        if key in self.buckets:
+            return self.buckets[key]
+        decode = kind == "decode"
+        if decode and width != 1:
+            raise ValueError("this model has no drafter: decode width 1 only")
+        cfg, dev, w = self.cfg, self.device, self.w
+        M = nseq if decode else width
+        W, KW = cfg.width, L.round_up(cfg.width, 64)
+        lay = BlobLayout.make(M, nseq, self.max_blocks)
+        blob = torch.zeros(lay.words, dtype=torch.int32, device=dev)
+        blob_host = torch.zeros(lay.words, dtype=torch.int32).pin_memory()
+        at = lambda off: blob.data_ptr() + 4 * off      # noqa: E731
+        f32 = lambda *s: torch.zeros(*s, dtype=torch.float32, device=dev)   # noqa: E731
+        prog = N.Program(f"{kind}-b{nseq}-w{width}")
+
+        # ---- activation buffers
+        x = f32(M, L.round_up(W, 32))
+        ss = f32(L.padded_rows(M), (W + 127) // 128)
+        h = self._operand_buf(M, KW)
+        loop_op = self._operand_buf(M, 2 * KW) if cfg.loop is not None else None
+        mid = self._operand_buf(M, max(l.out.K for l in w.layers))
+        ldp = max(L.round_up(l.n_plain, 8) for l in w.layers)
+        proj = f32(M, ldp)
+        big = max([l.proj.N_pad for l in w.layers] + [l.out.N_pad for l in w.layers] + [w.head.N_pad])
+        ws = None
+        if self.f32 or not self.fuse:                    # product rows (and, behind them, the split parts)
+            ws = torch.empty(M * big + (0 if self.f32 else self.scratch.capacity // 4), dtype=torch.float32, device=dev)
+        work = self._mixer_scratch(M, nseq, decode)
+        keep = [blob, x, ss, h, loop_op, mid, proj, ws, work]
+        digests = None
+        if self.race_check == "shadow":
+            digests = torch.zeros(len(cfg.runs) + 1, dtype=torch.int64, device=dev)
+            prog.digest_clear(digests, len(cfg.runs) + 1, tag="digest.clear")
+
+        h_op = self._operand(h, M, KW)
+        l_op = self._operand(loop_op, M, 2 * KW) if loop_op is not None else None
+
+        def target(run) -> tuple:
+            """What the linear ahead of a run (None: ahead of the head) leaves for it."""
+            if run is None:
+                return h_op, 0, w.final_norm, ss
+            if run.enter is not None:
+                return l_op, 0, None, None
+            return h_op, 0, w.layers[run.layer].norm, ss
+
+        # ---- embedding
+        runs = cfg.runs
+        ep = N.StreamEmbedParams()
+        ep.table, ep.table_f32, ep.vocab, ep.ids = w.embed.data_ptr(), int(self.f32), cfg.vocab, at(lay.ids)
+        ep.M, ep.width, ep.scale, ep.x = M, W, cfg.embed_scale, x.data_ptr()
+        ep.x0_k0 = -1
+        if loop_op is not None:
+            ep.x0, ep.x0_k0 = l_op, KW
+        op, k0, norm_w, s0 = target(runs[0])
+        ep.op, ep.op_k0, ep.norm_w = op, k0, N.ptr(norm_w)
+        ep.ss_out, ep.ss_out_n = N.ptr(s0), ss.shape[1]
+        prog.stream_embed(ep, tag="embed")
+
+        # ---- layers
+        for i, run in enumerate(runs):
+            lw, spec, t = w.layers[run.layer], cfg.layers[run.layer], f"R{run.index}.L{run.layer}"
+            if run.enter is not None:                    # x <- W_in [x; x0] + step
+                e = self._stream_epi(x, False, (h_op, 0, lw.norm, ss), bias=w.loop_step[run.enter])
+                self._linear(prog, w.loop_in, loop_op, M, e, ws, f"{t}.loop_in")
+            m_op = self._operand(mid, M, lw.out.K)
+            e = N.LinEpi()
+            self._row_norm(e, ss)
+            e.out, e.ldo, e.n_plain, e.act_tile0 = proj.data_ptr(), ldp, lw.n_plain, lw.act_tile0
+            if spec.mlp is not None:
+                e.act, e.act_k0, e.limit, e.alpha = m_op, lw.act_k0, spec.mlp.limit, spec.mlp.alpha
+            self._linear(prog, lw.proj, h, M, e, ws, f"{t}.project")
+            if isinstance(spec.mixer, DeltaMixer):
+                prog.delta(self._delta_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work), decode, tag=f"{t}.delta")
+            else:
+                prog.mla(self._mla_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode), tag=f"{t}.latent_attention")
+            nxt = runs[i + 1] if i + 1 < len(runs) else None
+            self._linear(prog, lw.out, mid, M, self._stream_epi(x, True, target(nxt)), ws, f"{t}.out")
+            if digests is not None:
+                prog.digest(x, x.numel() * 4, digests.data_ptr() + 8 * run.index, tag=f"{t}.digest")
+        b = self._head(prog, key, kind, nseq, width, M, lay, at, blob, blob_host, x, h, ss, ws, keep + [digests], seam, plp, capture)
+        b.arenas = [a for a in (x, ss, h, loop_op, mid, proj) if a is not None]
+        b.digests, b.x = digests, x
+        return b
+
+    # ---- mixers
+    def _mixer_scratch(self, M: int, nseq: int, decode: bool) -> dict:
+        """Scratch shared by the layers of a bucket, sized for the largest of them."""
+        f32 = lambda n: torch.zeros(max(1, n), dtype=torch.float32, device=self.device)   # noqa: E731
+        ms = [l.mixer for l in self.cfg.layers]
+        de, la = [m for m in ms if isinstance(m, DeltaMixer)], [m for m in ms if isinstance(m, LatentMixer)]
+        mx = lambda it: max(it, default=0)    # noqa: E731
+        wk = {"splits": self._splits(M, decode)}
+        if not decode:
+            wk["qn"] = f32(M * mx(m.kv_heads * m.dim_pad for m in de))
+            wk["kn"] = f32(M * mx(m.kv_heads * m.dim_pad for m in de))
+            wk["vv"] = f32(M * mx(m.heads * m.vdim_pad for m in de))
+            wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in de))
+            wk["bg"] = f32(M * mx(2 * m.heads for m in de))
+        wk["q_eff"] = torch.zeros(max(1, M * mx(m.heads * (max(m.rank_pad, m.dim_pad) + m.rot_pad) for m in la)), dtype=self.dtype, device=self.device)
+        if not self._expanded(M, decode):
+            wk["o_part"] = f32(M * wk["splits"] * mx(m.heads * m.rank_pad for m in la))
+            wk["ml"] = f32(M * wk["splits"] * mx(2 * m.heads for m in la))
+        return wk
+
+    def _expanded(self, M: int, decode: bool) -> bool:
+        return False
+
+    def _splits(self, M: int, decode: bool) -> int:
+        """Key splits of the absorbed attention: fill the SMs once."""
+        return max(1, min(32, F.device_sms() // max(1, M))) if decode or M < 64 else 1
+
+    def _delta_params(self, run, lw, m: DeltaMixer, proj, m_op, M, nseq, lay, at, wk) -> N.DeltaParams:
+        p = N.DeltaParams()
+        p.x, p.ldx = proj.data_ptr(), proj.stride(0)
+        p.q_off, p.k_off, p.v_off, p.b_off, p.a_off, p.g_off = (lw.off[k] for k in ("q", "k", "v", "b", "a", "g"))
+        p.conv_w, p.A_log, p.dt_bias, p.norm_w = (lw.extra[k].data_ptr() for k in ("conv", "A_log", "dt_bias", "norm"))
+        p.hist, p.state = self.delta_hist[run.index].data_ptr(), self.delta_state[run.index].data_ptr()
+        p.qn, p.kn, p.vv, p.bg, p.o = (N.ptr(wk.get(k)) for k in ("qn", "kn", "vv", "bg", "o"))
+        p.cu_rows, p.slots, p.pos = at(lay.cu_rows), at(lay.slots), at(lay.pos)
+        p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
+        p.H, p.HK, p.D, p.DP, p.V, p.VP, p.taps, p.n_slots = m.heads, m.kv_heads, m.dim, m.dim_pad, m.vdim, m.vdim_pad, m.taps, self.n_slots
+        p.eps, p.unit_eps, p.q_scale = self.cfg.eps, m.unit_eps, m.dim ** -0.5
+        p.err = self.scratch.err.data_ptr()
+        return p
+
+    def _mla_params(self, run, lw, m: LatentMixer, proj, m_op, M, nseq, lay, at, wk, decode) -> N.MlaParams:
+        p = N.MlaParams()
+        p.x, p.ldx = proj.data_ptr(), proj.stride(0)
+        p.q_off, p.dkv_off, p.g_off = lw.off["q"], lw.off["dkv"], lw.off["g"]
+        p.dkv_norm, p.freq, p.w_uk, p.w_uv = (lw.extra[k].data_ptr() for k in ("dkv_norm", "freq", "uk", "uv"))
+        p.cache, p.q_eff = self.kv[run.index].data_ptr(), wk["q_eff"].data_ptr()
+        p.o_part, p.ml = N.ptr(wk.get("o_part")), N.ptr(wk.get("ml"))
+        p.k_exp, p.v_exp = N.ptr(self.k_exp), N.ptr(self.v_exp)
+        p.slot_map, p.pos, p.cu_rows, p.kv_len, p.block_table = (at(o) for o in (lay.slot_map, lay.pos, lay.cu_rows, lay.kv_len, lay.block_table))
+        p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
+        p.H, p.D, p.R, p.V, p.C, p.CP, p.RP, p.DP, p.VP = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.rank_pad, m.rot_pad, m.dim_pad, m.vdim_pad
+        p.page, p.n_blocks, p.max_blocks = self.cfg.page_tokens, self.kv_blocks, self.max_blocks
+        p.splits, p.f32, p.expand, p.max_rows = wk["splits"], int(self.f32), int(self._expanded(M, decode)), 1 if decode else M
+        p.scale, p.eps, p.err = m.scale, self.cfg.eps, self.scratch.err.data_ptr()
+        return p
+
+    # ---- head and sampling
+    def _head(self, prog, key, kind, nseq, width, M, lay, at, blob, blob_host, x, h, ss, ws, keep, seam, plp, capture) -> Bucket:
+        cfg, dev, w = self.cfg, self.device, self.w
+        decode = kind == "decode"
+        Mh = M if decode else nseq
+        KW, V = L.round_up(cfg.width, 64), cfg.vocab
+        ldv = L.round_up(V, 8)
+        out, o_commit, o_tokens, o_picks = head_outputs(nseq, 1, 0, Mh, dev)
+        logits = torch.zeros(Mh, ldv, dtype=torch.float32, device=dev)
+        pick_val = torch.zeros(Mh, dtype=torch.float32, device=dev)
+
+        def head(a, rows, dst, normed: bool, tag):
+            e = N.LinEpi()
+            if not normed:
+                self._row_norm(e, ss)
+            e.out, e.ldo, e.n_plain, e.act_tile0 = dst.data_ptr(), dst.stride(0), V, w.head.N_pad // 256
+            self._linear(prog, w.head, a, rows, e, ws, tag)
+
+        if decode:
+            head(h, M, logits, False, "lm_head")
+        else:
+            last = self._operand_buf(nseq, KW)
+            np_ = N.StreamNormParams()
+            np_.x, np_.ldx, np_.width, np_.n, np_.rows = x.data_ptr(), x.stride(0), cfg.width, nseq, at(lay.last_rows)
+            np_.w, np_.eps, np_.op = w.final_norm.data_ptr(), cfg.eps, self._operand(last, nseq, KW)
+            prog.stream_norm(np_, tag="final_norm.last_rows")
+            head(last, nseq, logits, True, "lm_head")
+            keep.append(last)
+        prog.argmax(logits, Mh, ldv, V, 0, o_picks, pick_val, tag="argmax")
+        seam_dev = None
+        if seam:
+            seam_dev, s_ids, s_vals, s_lse = seam_outputs(Mh, dev)
+            prog.seam(logits, Mh, ldv, V, 0, None, s_ids, s_vals, s_lse, tag="topk_seam")
+            prog.sample_seam(s_ids, s_vals, at(lay.samp), at(lay.samp_u), o_picks, Mh, tag="sample_seam")
+        plp_dev = plp_logits = None
+        if plp:
+            plp_logits = torch.zeros(M, ldv, dtype=torch.float32, device=dev)
+            plp_dev, p_ids, p_vals, p_lse, p_next = plp_outputs(M, dev)
+            head(h, M, plp_logits, False, "plp.lm_head")
+            if V >= N.SEAM_K:
+                prog.seam(plp_logits, M, ldv, V, 0, None, p_ids, p_vals, p_lse, tag="plp.topk_seam")
+            prog.logit_gather(plp_logits, M, ldv, V, 0, at(lay.next_ids), p_next, tag="plp.logit_gather")
+        if decode:
+            vp = N.VerifyParams()
+            vp.draft, vp.target, vp.cu_rows = at(lay.ids), o_picks.data_ptr(), at(lay.cu_rows)
+            vp.seq_uid, vp.step_no = at(lay.seq_uid), at(lay.step_no)
+            vp.n_commit, vp.out_tokens = o_commit.data_ptr(), o_tokens.data_ptr()
+            vp.accept_row, vp.bonus = None, None
+            vp.nseq, vp.max_w, vp.oracle_p, vp.seed = nseq, 1, 0.0, 0
+            prog.verify(vp, tag="commit")
+        return finish_bucket(self, prog, key, kind, nseq, width, M, lay, blob, blob_host, keep + [pick_val], capture,
+                             dict(out=out, logits=logits, W=1, block=0, Mh=Mh, seam=seam_dev, plp=plp_dev, plp_logits=plp_logits))

@@ -174,6 +174,19 @@ def scratch(device) -> GemmScratch:
     return _SCRATCH[key]
 
 
+def device_sms() -> int:
+    from ..rules import default_rules
+    return int(default_rules().doc["device"]["sms"])
+
+
+def stream_splits(tiles: int, kb: int) -> int:
+    """Split-K factor of the bf16 stream linears: one wave of CTAs, at least four k-blocks each, no empty part."""
+    s = max(1, min(16, kb // 4, device_sms() // max(1, tiles)))
+    while s > 1 and (s - 1) * ((kb + s - 1) // s) >= kb:
+        s -= 1
+    return s
+
+
 def pick_splits(n_tiles: int, m_tiles: int, kb: int, sms: Optional[int] = None) -> int:
     """Split-K factor that fills the SMs when the tile grid alone does not: the law and its numbers
     are the `[gemm.splits]` table of the launch rules (one wave, at most 8 parts, no empty part)."""
@@ -372,7 +385,7 @@ def argmax(logits: torch.Tensor, id_offset: int = 0):
     R, V = logits.shape
     idx = torch.empty(R, dtype=torch.int32, device=logits.device)
     val = torch.empty(R, dtype=torch.float32, device=logits.device)
-    N.check(N.lib().saber_argmax_launch(logits.data_ptr(), R, logits.stride(0), V, id_offset,
+    N.check(N.lib().saber_argmax_launch(logits.data_ptr(), N.is_f32(logits), R, logits.stride(0), V, id_offset,
                                         idx.data_ptr(), val.data_ptr(), N.stream_handle()), "argmax")
     return idx, val
 
@@ -382,7 +395,7 @@ def topk_seam(logits: torch.Tensor, temps: Optional[torch.Tensor] = None, id_off
     ids = torch.empty(R, N.SEAM_K, dtype=torch.int32, device=logits.device)
     vals = torch.empty(R, N.SEAM_K, dtype=torch.float32, device=logits.device)
     lse = torch.empty(R, 2, dtype=torch.float32, device=logits.device)
-    N.check(N.lib().saber_topk_seam_launch(logits.data_ptr(), R, logits.stride(0), V, id_offset,
+    N.check(N.lib().saber_topk_seam_launch(logits.data_ptr(), N.is_f32(logits), R, logits.stride(0), V, id_offset,
                                            N.ptr(temps), ids.data_ptr(), vals.data_ptr(),
                                            lse.data_ptr(), N.stream_handle()), "topk_seam")
     return ids, vals, lse

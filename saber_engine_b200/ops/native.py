@@ -165,6 +165,46 @@ class VisAttnParams(C.Structure):
                 ("blocks", P), ("heads", I), ("width", I), ("scale", F)]
 
 
+class Operand(C.Structure):
+    """Token operand of a linear: bf16 GEMM tiles (fmt 0) or fp32 rows (fmt 1)."""
+    _fields_ = [("p", P), ("M_pad", I), ("ld", I), ("fmt", I)]
+
+
+class LinEpi(C.Structure):
+    _fields_ = [("stream", I), ("ss", P), ("ss_n", I), ("inv_width", F), ("eps", F), ("out", P), ("ldo", I), ("n_plain", I),
+                ("act_tile0", I), ("act", Operand), ("act_k0", I), ("limit", F), ("alpha", F), ("x", P), ("ldx", I), ("width", I),
+                ("add", I), ("bias", P), ("norm_w", P), ("op", Operand), ("op_k0", I), ("ss_out", P), ("ss_out_n", I)]
+
+
+class LinParams(C.Structure):
+    _fields_ = [("w", P), ("a", P), ("ws", P), ("counters", P), ("err", P), ("M", I), ("M_pad", I), ("N_pad", I), ("K", I), ("nt", I),
+                ("splits", I), ("fp32", I), ("fuse", I), ("mtiles", I), ("e", LinEpi)]
+
+
+class StreamEmbedParams(C.Structure):
+    _fields_ = [("table", P), ("table_f32", I), ("vocab", I), ("ids", P), ("M", I), ("width", I), ("scale", F), ("x", P), ("x0", Operand),
+                ("x0_k0", I), ("norm_w", P), ("op", Operand), ("op_k0", I), ("ss_out", P), ("ss_out_n", I)]
+
+
+class StreamNormParams(C.Structure):
+    _fields_ = [("x", P), ("ldx", I), ("width", I), ("n", I), ("rows", P), ("w", P), ("eps", F), ("op", Operand)]
+
+
+class DeltaParams(C.Structure):
+    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("k_off", I), ("v_off", I), ("b_off", I), ("a_off", I), ("g_off", I), ("conv_w", P),
+                ("A_log", P), ("dt_bias", P), ("norm_w", P), ("hist", P), ("state", P), ("qn", P), ("kn", P), ("vv", P), ("bg", P), ("o", P),
+                ("cu_rows", P), ("slots", P), ("pos", P), ("out", Operand), ("out_k0", I), ("M", I), ("nseq", I), ("H", I), ("HK", I),
+                ("D", I), ("DP", I), ("V", I), ("VP", I), ("taps", I), ("n_slots", I), ("eps", F), ("unit_eps", F), ("q_scale", F), ("err", P)]
+
+
+class MlaParams(C.Structure):
+    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("dkv_off", I), ("g_off", I), ("dkv_norm", P), ("freq", P), ("w_uk", P), ("w_uv", P),
+                ("cache", P), ("q_eff", P), ("o_part", P), ("ml", P), ("k_exp", P), ("v_exp", P), ("slot_map", P), ("pos", P),
+                ("cu_rows", P), ("kv_len", P), ("block_table", P), ("out", Operand), ("out_k0", I), ("M", I), ("nseq", I), ("H", I),
+                ("D", I), ("R", I), ("V", I), ("C", I), ("CP", I), ("RP", I), ("DP", I), ("VP", I), ("page", I), ("n_blocks", I),
+                ("max_blocks", I), ("splits", I), ("f32", I), ("expand", I), ("max_rows", I), ("scale", F), ("eps", F), ("err", P)]
+
+
 def lib() -> C.CDLL:
     """Load the native library (building it first when absent and a compiler is present)."""
     global _LIB
@@ -223,8 +263,8 @@ def _declare(L: C.CDLL) -> None:
         "saber_program_add_gdn_chunk": (I, [P, C.POINTER(GdnRecParams), I, I, P, C.c_char_p]),
         "saber_rope_kv_launch": (I, [C.POINTER(RopeKvParams), S]),
         "saber_attn_launch": (I, [C.POINTER(AttnParams), S]),
-        "saber_argmax_launch": (I, [P, I, I, I, I, P, P, S]),
-        "saber_topk_seam_launch": (I, [P, I, I, I, I, P, P, P, P, S]),
+        "saber_argmax_launch": (I, [P, I, I, I, I, I, P, P, S]),
+        "saber_topk_seam_launch": (I, [P, I, I, I, I, I, P, P, P, P, S]),
         "saber_verify_launch": (I, [C.POINTER(VerifyParams), S]),
         "saber_allreduce_launch": (I, [C.POINTER(AllReduceParams), S]),
         "saber_allreduce_chk_launch": (I, [C.POINTER(AllReduceParams), S]),
@@ -257,9 +297,9 @@ def _declare(L: C.CDLL) -> None:
         "saber_program_add_gdn_rec": (I, [P, C.POINTER(GdnRecParams), I, I, C.c_char_p]),
         "saber_program_add_rope": (I, [P, C.POINTER(RopeKvParams), C.c_char_p]),
         "saber_program_add_attn": (I, [P, C.POINTER(AttnParams), C.c_char_p]),
-        "saber_program_add_argmax": (I, [P, P, I, I, I, I, P, P, C.c_char_p]),
-        "saber_program_add_seam": (I, [P, P, I, I, I, I, P, P, P, P, C.c_char_p]),
-        "saber_program_add_logit_gather": (I, [P, P, I, I, I, I, P, P, C.c_char_p]),
+        "saber_program_add_argmax": (I, [P, P, I, I, I, I, I, P, P, C.c_char_p]),
+        "saber_program_add_seam": (I, [P, P, I, I, I, I, I, P, P, P, P, C.c_char_p]),
+        "saber_program_add_logit_gather": (I, [P, P, I, I, I, I, I, P, P, C.c_char_p]),
         "saber_program_add_sample_seam": (I, [P, P, P, P, P, P, I, C.c_char_p]),
         "saber_sample_seam_launch": (I, [P, P, P, P, P, I, S]),
         "saber_program_add_verify": (I, [P, C.POINTER(VerifyParams), C.c_char_p]),
@@ -289,6 +329,17 @@ def _declare(L: C.CDLL) -> None:
         "saber_vis_pos_add_launch": (I, [C.POINTER(VisPosAddParams), S]),
         "saber_vis_attn_launch": (I, [C.POINTER(VisAttnParams), I, S]),
         "saber_vis_rope_launch": (I, [C.POINTER(VisAttnParams), I, S]),
+        "saber_linear_launches": (I, [C.POINTER(LinParams)]),
+        "saber_linear_launch": (I, [C.POINTER(LinParams), S]),
+        "saber_stream_embed_launch": (I, [C.POINTER(StreamEmbedParams), S]),
+        "saber_stream_norm_launch": (I, [C.POINTER(StreamNormParams), S]),
+        "saber_delta_launch": (I, [C.POINTER(DeltaParams), I, S]),
+        "saber_mla_launch": (I, [C.POINTER(MlaParams), S]),
+        "saber_program_add_linear": (I, [P, C.POINTER(LinParams), C.c_char_p]),
+        "saber_program_add_stream_embed": (I, [P, C.POINTER(StreamEmbedParams), C.c_char_p]),
+        "saber_program_add_stream_norm": (I, [P, C.POINTER(StreamNormParams), C.c_char_p]),
+        "saber_program_add_delta": (I, [P, C.POINTER(DeltaParams), I, C.c_char_p]),
+        "saber_program_add_mla": (I, [P, C.POINTER(MlaParams), C.c_char_p]),
         "saber_program_num_ops": (I, [P]),
         "saber_program_declared_launches": (I, [P]),
         "saber_program_op_tag": (C.c_char_p, [P, I]),
@@ -314,6 +365,11 @@ def ptr(t: Optional[torch.Tensor]) -> Optional[int]:
     if isinstance(t, int):
         return t          # already a device address
     return t.data_ptr()
+
+
+def is_f32(t: torch.Tensor) -> int:
+    """1 for an fp32 tensor, 0 for bf16 (the two logit formats)."""
+    return int(t.dtype == torch.float32)
 
 
 def stream_handle(stream: Optional[torch.cuda.Stream] = None) -> int:
@@ -384,18 +440,18 @@ class Program:
         return self._L.saber_program_add_attn(self._h, C.byref(p), tag.encode())
 
     def argmax(self, logits, rows, ld, V, id_offset, idx, val, tag="argmax") -> int:
-        return self._L.saber_program_add_argmax(self._h, ptr(logits), rows, ld, V, id_offset,
+        return self._L.saber_program_add_argmax(self._h, ptr(logits), is_f32(logits), rows, ld, V, id_offset,
                                                 ptr(idx), ptr(val), tag.encode())
 
     def sample_seam(self, ids, vals, samp, u, picks, rows, tag="sample_seam") -> int:
         return self._L.saber_program_add_sample_seam(self._h, ptr(ids), ptr(vals), ptr(samp), ptr(u), ptr(picks), rows, tag.encode())
 
     def logit_gather(self, logits, rows, ld, V, id_offset, ids, out, tag="logit_gather") -> int:
-        return self._L.saber_program_add_logit_gather(self._h, ptr(logits), rows, ld, V, id_offset,
+        return self._L.saber_program_add_logit_gather(self._h, ptr(logits), is_f32(logits), rows, ld, V, id_offset,
                                                       ptr(ids), ptr(out), tag.encode())
 
     def seam(self, logits, rows, ld, V, id_offset, temps, ids, vals, lse, tag="seam") -> int:
-        return self._L.saber_program_add_seam(self._h, ptr(logits), rows, ld, V, id_offset,
+        return self._L.saber_program_add_seam(self._h, ptr(logits), is_f32(logits), rows, ld, V, id_offset,
                                               ptr(temps), ptr(ids), ptr(vals), ptr(lse), tag.encode())
 
     def draft_index(self, p: "DraftIndexParams", tag="draft_index") -> int:
@@ -443,6 +499,22 @@ class Program:
 
     def add_moe_combine(self, p: "MoeCombineParams", tag: str = "moe_combine") -> int:
         return self._L.saber_program_add_moe_combine(self._h, C.byref(p), tag.encode())
+
+    # linears with an fp32 residual stream, the free-size delta rule and latent attention
+    def linear(self, p: "LinParams", tag: str = "linear") -> int:
+        return self._L.saber_program_add_linear(self._h, C.byref(p), tag.encode())
+
+    def stream_embed(self, p: "StreamEmbedParams", tag: str = "stream_embed") -> int:
+        return self._L.saber_program_add_stream_embed(self._h, C.byref(p), tag.encode())
+
+    def stream_norm(self, p: "StreamNormParams", tag: str = "stream_norm") -> int:
+        return self._L.saber_program_add_stream_norm(self._h, C.byref(p), tag.encode())
+
+    def delta(self, p: "DeltaParams", single_row: bool, tag: str = "delta") -> int:
+        return self._L.saber_program_add_delta(self._h, C.byref(p), int(single_row), tag.encode())
+
+    def mla(self, p: "MlaParams", tag: str = "mla") -> int:
+        return self._L.saber_program_add_mla(self._h, C.byref(p), tag.encode())
 
     # ---- execution ---------------------------------------------------------------------------
     @property

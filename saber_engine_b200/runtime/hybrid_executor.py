@@ -1,4 +1,4 @@
-"""StepExecutor over `models.hybrid.HybridModel`: turns the scheduler's run descriptors into index
+"""StepExecutor over a model that builds buckets (`models.hybrid.HybridModel`, `models.stack.StackModel`): turns the scheduler's run descriptors into index
 blobs, replays the captured bucket, and hands back committed tokens and the next drafts.
 
 Parity: `crates/saber-engine/src/executor.rs:1-40` (RealExecutor over ForwardRunner) and the device
@@ -12,7 +12,7 @@ from typing import Optional
 
 import torch
 
-from ..models.hybrid import HybridModel, SeqStep, run_bucket
+from ..models.step import SeqStep, run_bucket
 from ..sched.buckets import DEFAULT_DECODE_BATCHES, DEFAULT_PREFILL_RUNGS, select_batch, select_rung
 from ..sched.executor import SeqOut, SeqRun
 
@@ -53,7 +53,7 @@ def gather_rank_seams(ids, vals, lse, device):
 
 
 class HybridExecutor:
-    def __init__(self, model: HybridModel, decode_batches=DEFAULT_DECODE_BATCHES, decode_widths=(1, 5, 8),
+    def __init__(self, model, decode_batches=DEFAULT_DECODE_BATCHES, decode_widths=(1, 5, 8),
                  prefill_rungs=(128, 512, 2048), prefill_pack: int = 1, capture: bool = True,
                  prebuild: bool = False):
         self.model = model
@@ -155,23 +155,37 @@ class HybridExecutor:
         return [SeqOut(res.tokens[j], res.drafts[j], seam=seams[j] if runs[j].want_seam else None)
                 for j in range(len(runs))]
 
+    def forward_logits(self, runs: list) -> torch.Tensor:
+        """One step over the given runs, every row committed, and the logits of EVERY row [rows, vocab] on the
+        host: portions of prompts and single tokens of other sequences share the step.  Runs of one token each
+        that continue a sequence take the decode bucket."""
+        rows = sum(len(r.tokens) for r in runs)
+        if all(len(r.tokens) == 1 and r.pos0 > 0 for r in runs) and 1 in self.decode_widths:
+            b = self._bucket("decode", select_batch(len(runs), self.decode_batches), 1)
+            logits = b.logits
+        else:
+            b = self._bucket("prefill", max(self.prefill_pack, len(runs)), select_rung(rows, self.prefill_rungs), plp=True)
+            logits = b.plp_logits
+        run_bucket(self.model, b, [self._step(r) for r in runs])
+        self._count(b)
+        return logits[:rows, :self.vocab].float().cpu()
+
     # ---- prefix-cache snapshots (device resident)
     def snapshot_state(self, slot: int):
         m = self.model
         with torch.cuda.stream(m.stream):      # same stream as the programs: ordered after the chunk
-            return {i: (m.gdn_state[i][slot].clone(), m.gdn_hist[i][slot, :3].clone()) for i in m.gdn_state}
+            return {k: v.clone() for k, v in m.snapshot_views(slot).items()}
 
     def restore_state(self, slot: int, snap) -> None:
         m = self.model
+        m.reset_slot(slot)
         with torch.cuda.stream(m.stream):
-            for i, (st, win) in snap.items():
-                m.gdn_state[i][slot].copy_(st)
-                m.gdn_hist[i][slot].zero_()
-                m.gdn_hist[i][slot, :3].copy_(win)
+            views = m.snapshot_views(slot)
+            for k, v in snap.items():
+                views[k].copy_(v)
 
     def snapshot_bytes(self) -> int:
-        m = self.model
-        return sum(t[0].numel() * 4 + 3 * m.gdn_hist[i].shape[2] * 2 for i, t in m.gdn_state.items())  # t[0]: one slot
+        return sum(v.numel() * v.element_size() for v in self.model.snapshot_views(0).values())
 
     def free_snapshot(self, snap) -> None:
         if isinstance(snap, dict):
@@ -193,11 +207,8 @@ class HybridExecutor:
         parts, layout, off = [], [], 0
         lane = self.copy_lane()
         with torch.cuda.stream(m.stream):          # the gathers run on the step stream (ordered after the last step) ...
-            staged = [(f"kv.{i}", kv[idx]) for i, kv in m.kv.items()]
-            staged += [(f"draft_kv.{i}", kv[idx]) for i, kv in getattr(m, "draft_kv", {}).items()]   # the drafter's context-KV store
-            for i in m.gdn_state:
-                staged += [(f"gdn_state.{i}", m.gdn_state[i][slot].clone()), (f"gdn_stash.{i}", m.gdn_stash[i][slot].clone()),
-                           (f"gdn_hist.{i}", m.gdn_hist[i][slot].clone())]
+            staged = [(k, pool[idx]) for k, pool in m.page_pools().items()]     # (the drafter's context-KV store is one of them)
+            staged += [(k, t[slot].clone()) for k, t in m.slot_tensors().items()]
         lane.after(m.stream)                       # ... and the bytes leave on the copy lane: later steps do not wait for them
         for name, t in staged:
             raw = t.contiguous().view(torch.uint8).reshape(-1)
@@ -215,14 +226,12 @@ class HybridExecutor:
         npages = header["npages"]
         idx = torch.tensor(blocks[:npages], dtype=torch.long, device=m.device)
         buf = torch.frombuffer(bytearray(payload), dtype=torch.uint8)
+        pools, slots = m.page_pools(), m.slot_tensors()
         with torch.cuda.stream(m.stream):
             for name, dtype, shape, off, nbytes in header["tensors"]:
-                kind, i = name.rsplit(".", 1)
-                i = int(i)
-                dst = {"kv": m.kv, "draft_kv": getattr(m, "draft_kv", {}), "gdn_state": m.gdn_state, "gdn_stash": m.gdn_stash,
-                       "gdn_hist": m.gdn_hist}[kind][i]
+                dst = pools[name] if name in pools else slots[name]
                 src = buf[off:off + nbytes].to(m.device).view(dst.dtype).reshape(shape)
-                if kind in ("kv", "draft_kv"):
+                if name in pools:
                     dst[idx] = src
                 else:
                     dst[slot].copy_(src)

@@ -82,6 +82,8 @@ def build_engine(a):
     """Executor + scheduler for `saber engine` (also used by tests)."""
     from ..sched.scheduler import Scheduler, SchedulerConfig
     from ..serve.sampler import HostSampler
+    if a.engine != "real" and a.engine_decode_widths is None:
+        a.engine_decode_widths = "1,5,8"
     if a.engine == "mock":
         from ..sched.mock import NullExecutor
         ex = NullExecutor(vocab=a.mock_vocab, max_seqs=a.engine_max_seqs, decode_widths=_ints(a.engine_decode_widths),
@@ -94,7 +96,11 @@ def build_engine(a):
         from ..models import config as MC
         from ..models.hybrid import HybridModel
         from ..runtime.hybrid_executor import HybridExecutor
+        from ..models.stack_config import StackConfig
         cfg = MC.by_name(a.engine_config)
+        stack = isinstance(cfg, StackConfig)
+        if a.engine_decode_widths is None:               # not given: every verify width of the drafter, or 1 without one
+            a.engine_decode_widths = "1" if stack else "1,5,8"
         widths = _ints(a.engine_decode_widths)
         # several GPUs: one process per GPU (torchrun or the self-launch in cmd_engine); rank 0 plans
         # and serves, the other ranks follow its executor calls (parallel/tp_serve.py)
@@ -143,17 +149,29 @@ def build_engine(a):
             widths = list(man.decode_widths)
         weights = None
         with boot.phase("weights"):
-            if a.pack and not a.random_init:
+            if stack:
+                from ..models import stack_weights as SW
+                folder = None if a.random_init else (a.pack or cfg.source)
+                dtype = getattr(torch, a.engine_dtype)
+                weights = SW.load(cfg, folder, dtype, dev) if folder else SW.random_init(cfg, dtype, dev, a.seed)
+            elif a.pack and not a.random_init:
                 from ..pack.build import load_weights
                 weights = load_weights(a.pack, cfg, a.engine_tp, rank, dev)
         with boot.phase("model"):
             kv_blocks = a.engine_kv_blocks or plan.kv_blocks            # the ledger's pool unless a count is forced
-            model = HybridModel(cfg, tp=a.engine_tp, rank=rank, device=dev, max_seqs=man.max_seqs, comm=comm,
-                                max_ctx=man.max_ctx, kv_blocks=kv_blocks, max_width=max(widths),
-                                weights=weights, seed=a.seed, race_check=a.engine_race_check,
-                                gdn_prefill=getattr(a, "engine_gdn_prefill", "tc"),
-                                prefill_w8=bool(getattr(man, "prefill_w8", True)),
-                                image_rows=(getattr(a, "vision_arena_patches", 0) // 4 if getattr(a, "vision", False) else 0))
+            if stack:
+                from ..models.stack import StackModel
+                if getattr(a, "vision", False):
+                    raise SystemExit("saber: --vision is not available for this model")
+                model = StackModel(cfg, device=dev, max_seqs=man.max_seqs, max_ctx=man.max_ctx, kv_blocks=kv_blocks, weights=weights,
+                                   dtype=dtype, race_check=a.engine_race_check)
+            else:
+                model = HybridModel(cfg, tp=a.engine_tp, rank=rank, device=dev, max_seqs=man.max_seqs, comm=comm,
+                                    max_ctx=man.max_ctx, kv_blocks=kv_blocks, max_width=max(widths),
+                                    weights=weights, seed=a.seed, race_check=a.engine_race_check,
+                                    gdn_prefill=getattr(a, "engine_gdn_prefill", "tc"),
+                                    prefill_w8=bool(getattr(man, "prefill_w8", True)),
+                                    image_rows=(getattr(a, "vision_arena_patches", 0) // 4 if getattr(a, "vision", False) else 0))
             if man.autotune:
                 from ..plan.autotune import TuneTable
                 model.tune_table = TuneTable.load(man.autotune)
@@ -292,8 +310,12 @@ def cmd_engine(a) -> int:
 def cmd_explain(a) -> int:
     from ..plan import launch_plan as LP
     try:
+        from ..models import config as MC
+        from ..models.stack_config import StackConfig
         man = LP.Manifest.from_toml(Path(a.manifest).read_text()) if a.manifest else LP.Manifest(
             model=a.model, tp=a.tp, allow_untuned=True, autotune=a.autotune)
+        if not a.manifest and isinstance(MC.by_name(a.model), StackConfig):
+            man.decode_widths = (1,)
         plan = LP.resolve(man, LP.DeviceProfile.measured())
         print(plan.explain())
         if a.bind:
@@ -322,7 +344,11 @@ def cmd_pack(a) -> int:
     from ..pack import format as PF
     if a.action == "build":
         from ..models import config as MC
+        from ..models.stack_config import StackConfig
         from ..pack.build import write_pack
+        if isinstance(MC.by_name(a.model), StackConfig):
+            print(f"saber: {a.model} has no pack format: it is loaded from config.json and model.safetensors", file=sys.stderr)
+            return 2
         d = write_pack(MC.by_name(a.model), a.out, a.tp, a.seed, a.device)
         print(d)
         return 0
@@ -401,12 +427,12 @@ def make_parser() -> argparse.ArgumentParser:
     e.add_argument("--engine", default="real", choices=["real", "mock", "tiny"])
     e.add_argument("--engine-tp", type=int, default=1)
     e.add_argument("--pack")
-    e.add_argument("--engine-config", default="qwen38-27b")
+    e.add_argument("--engine-config", default="qwen38-27b", help="a built-in model description, or a folder with config.json and model.safetensors")
     e.add_argument("--engine-max-ctx", type=int, default=262144)
     e.add_argument("--engine-max-seqs", type=int, default=8)
     e.add_argument("--engine-prefill-rows", default="128,512,2048")
     e.add_argument("--engine-decode-batches", default="1,2,3,4,8")
-    e.add_argument("--engine-decode-widths", default="1,5,8")
+    e.add_argument("--engine-decode-widths", default=None, help="default 1,5,8 (1 for a model without a drafter)")
     e.add_argument("--engine-draft-block", type=int, default=8)
     e.add_argument("--engine-budget-mib", type=int, default=160000)
     e.add_argument("--engine-kv-blocks", type=int, default=0, help="force the KV block count (0: what the plan's ledger derives from the budget)")
@@ -435,6 +461,8 @@ def make_parser() -> argparse.ArgumentParser:
     e.add_argument("--vision", action="store_true", help="load the vision tower and accept image parts in chat requests")
     e.add_argument("--vision-arena-patches", type=int, default=16384, help="patch rows the tower arena holds (larger images are downscaled)")
     e.add_argument("--engine-host-trace", action="store_true", help="named host phases per step (an attribution, not a published time)")
+    e.add_argument("--engine-dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                   help="compute type of a layer-by-layer model (the folder of --engine-config)")
     e.add_argument("--engine-race-check", default="off", choices=["off", "shadow"])
     e.add_argument("--engine-gdn-prefill", default="tc", choices=["tc", "rows", "chunked"],
                    help="DeltaNet prefill: 64-row chunks on the tensor cores (default), the exact fp32 row-by-row "
@@ -496,6 +524,9 @@ def main(argv=None) -> int:
         sys.argv = ["bench.py"] + argv[1:]
         runpy.run_path(str(Path(__file__).resolve().parents[2] / "bench.py"), run_name="__main__")
         return 0
+    if argv and argv[0] == "trace-run":
+        from ..runtime.trace_run import main as trace_main
+        return trace_main(argv[1:])
     if argv and argv[0] == "shadow":
         from ..shadow.__main__ import main as shadow_main
         return shadow_main(argv[1:])

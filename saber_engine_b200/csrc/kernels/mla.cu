@@ -5,8 +5,7 @@
 // independent (each knows its sequence and position), so any ragged batch is the same launch; keys may be
 // split over CTAs and are merged by the output kernel.
 #include "launch.cuh"
-#include "mla.h"
-#include "ptx_sm100.cuh"
+#include "mla_device.cuh"
 
 namespace saber {
 
@@ -16,29 +15,6 @@ template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v
 template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
-
-__device__ __forceinline__ float mla_warp_sum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-__device__ __forceinline__ float mla_warp_max(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
-  return v;
-}
-__device__ __forceinline__ int mla_seq_of_row(const int32_t* cu, int nseq, int m) {
-  for (int j = 0; j < nseq; ++j)
-    if (m < cu[j + 1]) return m >= cu[j] ? j : -1;
-  return -1;
-}
-// physical page of a key (bounds-checked: an entry outside the pool is recorded and read as page 0)
-__device__ __forceinline__ int mla_page(const MlaParams& p, int j, int key) {
-  const int b = p.block_table[static_cast<size_t>(j) * p.max_blocks + key / p.page];
-  if (b >= 0 && b < p.n_blocks) return b;
-  if (p.err) atomicCAS(p.err, 0u, static_cast<uint32_t>(kErrBadIndex));
-  return 0;
-}
 
 // grid M, 256 threads: latent norm and rotated key into the cache, rotated query part (and, in the expanded
 // form, the unrotated one) into q_eff
@@ -115,10 +91,10 @@ __global__ void __launch_bounds__(128) mla_absorb_kernel(const __grid_constant__
   if (c >= p.CP) return;
   float acc[8] = {};
   if (c < p.C) {
-    const T* w = static_cast<const T*>(p.w_uk) + static_cast<size_t>(h) * p.D * p.C + c;
+    const T* w = static_cast<const T*>(p.w_uk) + static_cast<size_t>(h) * p.D * p.CP + c;
 #pragma unroll 4
     for (int d = 0; d < p.D; ++d) {
-      const float wv = to_f<T>(w[static_cast<size_t>(d) * p.C]);
+      const float wv = to_f<T>(w[static_cast<size_t>(d) * p.CP]);
       const float4 a = *reinterpret_cast<const float4*>(sm + d * 8), b = *reinterpret_cast<const float4*>(sm + d * 8 + 4);
       acc[0] = fmaf(wv, a.x, acc[0]); acc[1] = fmaf(wv, a.y, acc[1]); acc[2] = fmaf(wv, a.z, acc[2]); acc[3] = fmaf(wv, a.w, acc[3]);
       acc[4] = fmaf(wv, b.x, acc[4]); acc[5] = fmaf(wv, b.y, acc[5]); acc[6] = fmaf(wv, b.z, acc[6]); acc[7] = fmaf(wv, b.w, acc[7]);
@@ -154,7 +130,7 @@ __global__ void __launch_bounds__(128) mla_row_attn_kernel(const __grid_constant
     __syncthreads();
     if (threadIdx.x < n) {
       const int key = kb + threadIdx.x;
-      rows_s[threadIdx.x] = static_cast<const T*>(p.cache) + (static_cast<size_t>(mla_page(p, j, key)) * p.page + key % p.page) * LD;
+      rows_s[threadIdx.x] = static_cast<const T*>(p.cache) + (static_cast<size_t>(mla_page_at(p, j, key / p.page)) * p.page + key % p.page) * LD;
     }
     __syncthreads();
     for (int k = warp; k < n; k += 4) {
@@ -192,56 +168,87 @@ __global__ void __launch_bounds__(128) mla_row_attn_kernel(const __grid_constant
   if (threadIdx.x == 0) { p.ml[row * 2] = mx; p.ml[row * 2 + 1] = l; }
 }
 
-// grid (M, H, ceil(V / 64)), 256 threads: merges the key splits, carries the latents out through W_uv, gates
+// grid (ceil(M / 8), H, ceil(V / 64)), 256 threads: merges the key splits of eight rows, carries their latents out
+// through W_uv (each weight row is read once for the eight), gates
 template <typename T>
 __global__ void __launch_bounds__(256) mla_out_kernel(const __grid_constant__ MlaParams p) {
   pdl_wait();
-  extern __shared__ float sm[];                   // [CP]
-  const int m = blockIdx.x, h = blockIdx.y;
-  if (mla_seq_of_row(p.cu_rows, p.nseq, m) < 0) return;
-  const size_t row = (static_cast<size_t>(m) * p.H + h) * p.splits;
-  float mx = -INFINITY, l = 0.f;
-  for (int s = 0; s < p.splits; ++s) mx = fmaxf(mx, p.ml[(row + s) * 2]);
-  for (int s = 0; s < p.splits; ++s) l += p.ml[(row + s) * 2 + 1] * expf(p.ml[(row + s) * 2] - mx);
-  for (int c = threadIdx.x; c < p.CP; c += 256) {
-    float v = 0.f;
-    for (int s = 0; s < p.splits; ++s) {
-      const float ms = p.ml[(row + s) * 2];
-      if (ms > -INFINITY) v = fmaf(p.o_part[(row + s) * p.CP + c], expf(ms - mx), v);
-    }
-    sm[c] = v / l;
+  extern __shared__ float sm[];                   // [8][CP] latents | [8][splits] merge weights
+  const int mb = blockIdx.x * 8, h = blockIdx.y, rows = min(8, p.M - mb);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* wt = sm + 8 * p.CP;
+  if (warp < rows) {                              // a warp per row: merge weights exp(m_s - max) / sum
+    const float* ml = p.ml + (static_cast<size_t>(mb + warp) * p.H + h) * p.splits * 2;
+    const bool live = mla_seq_of_row(p.cu_rows, p.nseq, mb + warp) >= 0;
+    float mx = -INFINITY, l = 0.f;
+    for (int s = lane; s < p.splits; s += 32) mx = fmaxf(mx, live ? ml[s * 2] : -INFINITY);
+    mx = mla_warp_max(mx);
+    for (int s = lane; s < p.splits; s += 32) l += live && ml[s * 2] > -INFINITY ? ml[s * 2 + 1] * expf(ml[s * 2] - mx) : 0.f;
+    l = mla_warp_sum(l);
+    for (int s = lane; s < p.splits; s += 32) wt[warp * p.splits + s] = live && ml[s * 2] > -INFINITY ? expf(ml[s * 2] - mx) / l : 0.f;
   }
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const float* g = p.x + static_cast<size_t>(m) * p.ldx + p.g_off + h * p.V;
+  for (int i = threadIdx.x; i < 8 * p.CP; i += 256) {
+    const int r = i / p.CP, c = i - r * p.CP;
+    float v = 0.f;
+    if (r < rows) {
+      const float* o = p.o_part + (static_cast<size_t>(mb + r) * p.H + h) * p.splits * p.CP + c;
+      for (int s = 0; s < p.splits; ++s) {
+        const float w = wt[r * p.splits + s];
+        if (w != 0.f) v = fmaf(o[static_cast<size_t>(s) * p.CP], w, v);     // (a split without keys, or a padding row, was not written)
+      }
+    }
+    sm[i] = v;
+  }
+  __syncthreads();
   const int v1 = min(p.V, static_cast<int>(blockIdx.z) * 64 + 64);
   for (int v = blockIdx.z * 64 + warp; v < v1; v += 8) {
-    const T* w = static_cast<const T*>(p.w_uv) + (static_cast<size_t>(h) * p.V + v) * p.C;
-    float s = 0.f;
-    for (int c = lane; c < p.C; c += 32) s = fmaf(to_f<T>(w[c]), sm[c], s);
-    s = mla_warp_sum(s);
-    if (lane == 0) operand_store1(p.out, m, p.out_k0 + h * p.V + v, s / (1.f + expf(-g[v])));
+    const T* w = static_cast<const T*>(p.w_uv) + (static_cast<size_t>(h) * p.V + v) * p.CP;
+    float s[8] = {};
+    for (int c = lane; c < p.C; c += 32) {
+      const float wv = to_f<T>(w[c]);
+#pragma unroll
+      for (int r = 0; r < 8; ++r) s[r] = fmaf(wv, sm[r * p.CP + c], s[r]);
+    }
+#pragma unroll
+    for (int r = 0; r < 8; ++r) s[r] = mla_warp_sum(s[r]);
+    if (lane < rows) {
+      float y = s[0];
+#pragma unroll
+      for (int r = 1; r < 8; ++r) y = lane == r ? s[r] : y;
+      const float g = p.x[static_cast<size_t>(mb + lane) * p.ldx + p.g_off + h * p.V + v];
+      operand_store1(p.out, mb + lane, p.out_k0 + h * p.V + v, y / (1.f + expf(-g)));
+    }
   }
 }
 
 template <typename T>
-static int mla_absorbed(const MlaParams& p, cudaStream_t stream) {
+static int mla_go(const MlaParams& p, cudaStream_t stream) {
   cudaError_t e = launch(mla_prep_kernel<T>, dim3(p.M), dim3(256), 0, stream, 0, p);
-  if (e == cudaSuccess) e = launch(mla_absorb_kernel<T>, dim3((p.CP + 127) / 128, p.H, (p.M + 7) / 8), dim3(128), p.D * 32, stream, 0, p);
-  if (e == cudaSuccess) e = launch(mla_row_attn_kernel<T>, dim3(p.M, p.H, p.splits), dim3(128), (p.CP + p.RP + kRowKeys) * 4, stream, 0, p);
-  if (e == cudaSuccess) e = launch(mla_out_kernel<T>, dim3(p.M, p.H, (p.V + 63) / 64), dim3(256), p.CP * 4, stream, 0, p);
-  return static_cast<int>(e);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  if (p.expand) return saber_mla_expand_attn(&p, stream);
+  e = launch(mla_absorb_kernel<T>, dim3((p.CP + 127) / 128, p.H, (p.M + 7) / 8), dim3(128), p.D * 32, stream, 0, p);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  if (saber_mla_decode_ok(&p)) {
+    const int r = saber_mla_decode_attn(&p, stream);
+    if (r != 0) return r;
+  } else {
+    e = launch(mla_row_attn_kernel<T>, dim3(p.M, p.H, p.splits), dim3(128), (p.CP + p.RP + kRowKeys) * 4, stream, 0, p);
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  return static_cast<int>(launch(mla_out_kernel<T>, dim3((p.M + 7) / 8, p.H, (p.V + 63) / 64), dim3(256), 8 * (p.CP + p.splits) * 4, stream, 0, p));
 }
 
 }  // namespace saber
 
-extern "C" int saber_mla_launches(const saber::MlaParams* p) { (void)p; return 4; }
+extern "C" int saber_mla_launches(const saber::MlaParams* p) { return p->expand ? 3 : 4; }
 
 extern "C" int saber_mla_launch(const saber::MlaParams* p, cudaStream_t stream) {
   using namespace saber;
-  if (p->M <= 0 || p->C > p->CP || p->R > p->RP || (p->R & 1) || p->CP > 128 * kRowMaxC || p->D > 1024 || p->splits < 1)
+  if (p->M <= 0 || p->C > p->CP || p->R > p->RP || (p->R & 1) || p->CP > 128 * kRowMaxC || p->D > 1024 || p->splits < 1 || p->splits > 64 ||
+      p->q_eff == nullptr || p->cache == nullptr)
     return static_cast<int>(cudaErrorInvalidValue);
-  if (p->expand || p->o_part == nullptr || p->ml == nullptr || p->q_eff == nullptr || p->cache == nullptr)
+  if (p->expand ? (p->k_exp == nullptr || p->v_exp == nullptr || !saber_mla_expand_ok(p)) : (p->o_part == nullptr || p->ml == nullptr))
     return static_cast<int>(cudaErrorInvalidValue);
-  return p->f32 ? mla_absorbed<float>(*p, stream) : mla_absorbed<__nv_bfloat16>(*p, stream);
+  return p->f32 ? mla_go<float>(*p, stream) : mla_go<__nv_bfloat16>(*p, stream);
 }

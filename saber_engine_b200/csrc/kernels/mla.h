@@ -13,8 +13,8 @@ struct MlaParams {
   int ldx, q_off, dkv_off, g_off;
   const float* dkv_norm;      // [C]
   const float* freq;          // [R / 2] rotary frequencies
-  const void* w_uk;           // [H * D][C]
-  const void* w_uv;           // [H * V][C]
+  const void* w_uk;           // [H * D][CP] (pads zero)
+  const void* w_uv;           // [H * V][CP]
   void* cache;                // [n_blocks][page][CP + RP]: latent, rotated key (pads zero)
   void* q_eff;                // scratch [M][H][max(CP, DP) + RP]
   float* o_part;              // scratch [M][H][splits][CP] (absorbed form)
@@ -39,5 +39,6 @@ struct MlaParams {
 
 }  // namespace saber
 
+extern "C" int saber_mla_expand_ok(const saber::MlaParams* p);
 extern "C" int saber_mla_launches(const saber::MlaParams* p);
 extern "C" int saber_mla_launch(const saber::MlaParams* p, cudaStream_t stream);

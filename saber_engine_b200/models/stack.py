@@ -12,6 +12,7 @@ Caches and states belong to a layer RUN: the pages of a latent-attention run, th
 """
 from __future__ import annotations
 
+import ctypes as C
 from typing import Optional
 
 import torch
@@ -243,13 +244,19 @@ class StackModel:
             wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in de))
             wk["bg"] = f32(M * mx(2 * m.heads for m in de))
         wk["q_eff"] = torch.zeros(max(1, M * mx(m.heads * (max(m.rank_pad, m.dim_pad) + m.rot_pad) for m in la)), dtype=self.dtype, device=self.device)
-        if not self._expanded(M, decode):
-            wk["o_part"] = f32(M * wk["splits"] * mx(m.heads * m.rank_pad for m in la))
-            wk["ml"] = f32(M * wk["splits"] * mx(2 * m.heads for m in la))
+        absorbed = [m for m in la if not self._expanded(m, M, decode)]
+        if absorbed:
+            wk["o_part"] = f32(M * wk["splits"] * mx(m.heads * m.rank_pad for m in absorbed))
+            wk["ml"] = f32(M * wk["splits"] * mx(2 * m.heads for m in absorbed))
         return wk
 
-    def _expanded(self, M: int, decode: bool) -> bool:
-        return False
+    def _expanded(self, m: LatentMixer, M: int, decode: bool) -> bool:
+        """Prompt portions attend over expanded keys and values; decoding, short portions and fp32 in the latent space."""
+        if decode or M < 64 or self.k_exp is None:
+            return False
+        p = N.MlaParams()
+        p.f32, p.page, p.VP, p.DP, p.RP, p.CP = int(self.f32), self.cfg.page_tokens, m.vdim_pad, m.dim_pad, m.rot_pad, m.rank_pad
+        return bool(N.lib().saber_mla_expand_ok(C.byref(p)))
 
     def _splits(self, M: int, decode: bool) -> int:
         """Key splits of the absorbed attention: fill the SMs once."""
@@ -281,7 +288,7 @@ class StackModel:
         p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
         p.H, p.D, p.R, p.V, p.C, p.CP, p.RP, p.DP, p.VP = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.rank_pad, m.rot_pad, m.dim_pad, m.vdim_pad
         p.page, p.n_blocks, p.max_blocks = self.cfg.page_tokens, self.kv_blocks, self.max_blocks
-        p.splits, p.f32, p.expand, p.max_rows = wk["splits"], int(self.f32), int(self._expanded(M, decode)), 1 if decode else M
+        p.splits, p.f32, p.expand, p.max_rows = wk["splits"], int(self.f32), int(self._expanded(m, M, decode)), 1 if decode else M
         p.scale, p.eps, p.err = m.scale, self.cfg.eps, self.scratch.err.data_ptr()
         return p
 

@@ -88,8 +88,8 @@ class LatentMixer:
         return self._pad16(self.dim)
 
     @property
-    def vdim_pad(self) -> int:
-        return self._pad16(self.vdim)
+    def vdim_pad(self) -> int:        # value sizes the expanded form is instantiated for (above: the absorbed form only)
+        return next((n for n in (32, 64, 128, 256) if n >= self.vdim), self._pad16(self.vdim))
 
     def segments(self) -> list:
         return [("q", self.heads * (self.dim + self.rot_dim)), ("dkv", self.kv_rank + self.rot_dim), ("g", self.heads * self.vdim)]

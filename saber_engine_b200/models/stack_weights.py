@@ -177,7 +177,10 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
                 extra[n] = f32(f"{p}mix.{n}")
         elif isinstance(m, LatentMixer):
             extra["dkv_norm"] = f32(p + "mix.dkv.norm")
-            extra["uk"], extra["uv"] = t(p + "mix.uk").to(dtype).contiguous(), t(p + "mix.uv").to(dtype).contiguous()
+            for n in ("uk", "uv"):                                     # row stride: the padded latent
+                full = t(f"{p}mix.{n}")
+                extra[n] = torch.zeros(full.shape[0], m.rank_pad, dtype=dtype, device=dev)
+                extra[n][:, : m.kv_rank] = full
             half = m.rot_dim // 2
             extra["freq"] = torch.tensor([m.rot_base ** (-2.0 * j / m.rot_dim) for j in range(half)] or [1.0], dtype=torch.float32, device=dev)
         layers.append(StackLayer(f32(p + "norm1"), pack_linear(r, dtype), pack_linear(o, dtype), off, n_plain, tile0, mix_k, extra))

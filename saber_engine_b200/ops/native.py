@@ -334,6 +334,7 @@ def _declare(L: C.CDLL) -> None:
         "saber_stream_embed_launch": (I, [C.POINTER(StreamEmbedParams), S]),
         "saber_stream_norm_launch": (I, [C.POINTER(StreamNormParams), S]),
         "saber_delta_launch": (I, [C.POINTER(DeltaParams), I, S]),
+        "saber_mla_expand_ok": (I, [C.POINTER(MlaParams)]),
         "saber_mla_launch": (I, [C.POINTER(MlaParams), S]),
         "saber_program_add_linear": (I, [P, C.POINTER(LinParams), C.c_char_p]),
         "saber_program_add_stream_embed": (I, [P, C.POINTER(StreamEmbedParams), C.c_char_p]),

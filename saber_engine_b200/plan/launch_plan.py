@@ -18,6 +18,7 @@ from pathlib import Path
 from typing import Optional
 
 from ..models import config as MC
+from ..models.stack_config import StackConfig
 from ..ops import layouts as L
 from .autotune import TuneTable, make_key
 
@@ -193,6 +194,8 @@ def resolve(manifest: Manifest, device: Optional[DeviceProfile] = None, table: O
         raise PlanError(problems)
     device = device or DeviceProfile()
     cfg = MC.by_name(manifest.model)
+    if isinstance(cfg, StackConfig):
+        return _resolve_stack(manifest, device, cfg)
     tp = manifest.tp
     sh = MC.shard(cfg, tp, 0)
     if table is None and manifest.autotune:
@@ -231,6 +234,11 @@ def resolve(manifest: Manifest, device: Optional[DeviceProfile] = None, table: O
     led.bill("splitk_scratch", 256 * 262144 * 4)
     led.bill("headroom", manifest.headroom_mib << 20)
     block_bytes = cfg.kv_bytes_per_token(tp) * cfg.page_tokens
+    return _finish(manifest, device, cfg, routes, missing, led, block_bytes)
+
+
+def _finish(manifest: Manifest, device: DeviceProfile, cfg, routes: dict, missing: list, led: Ledger, block_bytes: int) -> LaunchPlan:
+    """The KV pool from what the ledger leaves, and the plan's hash."""
     kv_blocks = max(0, led.remaining // block_bytes) if block_bytes else 0
     need = (manifest.max_ctx + cfg.page_tokens - 1) // cfg.page_tokens + 1
     if block_bytes and kv_blocks < need:
@@ -245,6 +253,34 @@ def resolve(manifest: Manifest, device: Optional[DeviceProfile] = None, table: O
     plan = LaunchPlan(manifest, device, routes, led, kv_blocks, kv_blocks * cfg.page_tokens, missing,
                       hashlib.sha256(json.dumps(desc, sort_keys=True).encode()).hexdigest())
     plan._block_bytes = block_bytes
+    return plan
+
+
+def _resolve_stack(manifest: Manifest, device: DeviceProfile, cfg: StackConfig) -> LaunchPlan:
+    """Layer-by-layer models: bf16 linears with one declared variant each (no measured routes), one GPU.  A page
+    holds the latents of every attention run and, where the model expands keys and values for prompts, its share
+    of that scratch; a model without attention runs has no page bytes, only block ids."""
+    problems = []
+    if manifest.tp != 1:
+        problems.append(f"{cfg.name}: tp {manifest.tp} is not supported (this model class runs on one GPU)")
+    if tuple(manifest.decode_widths) != (1,):
+        problems.append(f"{cfg.name}: decode_widths must be 1 (no drafter)")
+    if problems:
+        raise PlanError(problems)
+    rows = max(max(manifest.prefill_rows), max(manifest.decode_batches))
+    led = Ledger(manifest.budget_mib << 20)
+    led.bill("weights", cfg.param_count() * 2)
+    led.bill("delta_state_slots", (manifest.max_seqs + 1) * cfg.slot_bytes())
+    led.bill("prefix_cache_snapshots", manifest.prefix_cache_mib << 20)
+    led.bill("activation_arenas", rows * 4 * (3 * cfg.width + 3 * cfg.widest_project() + max(l.mlp.ff if l.mlp else 0 for l in cfg.layers)) * 2)
+    led.bill("logits", max(manifest.decode_batches) * cfg.vocab * 4 * 2)
+    led.bill("splitk_scratch", 256 * 262144 * 4)
+    led.bill("headroom", manifest.headroom_mib << 20)
+    block_bytes = (cfg.page_token_bytes() + cfg.expanded_token_bytes()) * cfg.page_tokens
+    plan = _finish(manifest, device, cfg, {}, [], led, block_bytes)
+    if not block_bytes:
+        plan.kv_blocks = manifest.max_seqs * ((manifest.max_ctx + cfg.page_tokens - 1) // cfg.page_tokens + 1) + 1
+        plan.kv_tokens = plan.kv_blocks * cfg.page_tokens
     return plan
 
 

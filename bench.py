@@ -110,10 +110,20 @@ def main() -> int:
     ap.add_argument("--no-tune-table", action="store_true", help="ignore the committed autotune table (A/B)")
     ap.add_argument("--no-extra-arms", action="store_true", help="skip the NVFP4 side arm of the 27B run")
     ap.add_argument("--no-single", action="store_true", help="skip the single-stream side measurement")
+    ap.add_argument("--stack", default="", metavar="NAMES", help="instead of the headline workload: prefill and decode throughput of these layer-by-layer "
+                    "models (comma separated, or 'all'), each beside the hybrid decoder at equal layer sizes, with a roofline per launch group")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
     args.warmup = max(args.warmup, 3)
+    if args.stack:
+        from saber_engine_b200.runtime.bench_stack import run
+        sampler = ClockSampler(0)
+        sampler.start()
+        res = run(args)
+        res["clocks"] = sampler.stop()
+        print(json.dumps(res))
+        return 0
 
     import torch
     from saber_engine_b200.runtime.bench_core import run_benchmark

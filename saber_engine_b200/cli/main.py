@@ -164,7 +164,7 @@ def build_engine(a):
                 if getattr(a, "vision", False):
                     raise SystemExit("saber: --vision is not available for this model")
                 model = StackModel(cfg, device=dev, max_seqs=man.max_seqs, max_ctx=man.max_ctx, kv_blocks=kv_blocks, weights=weights,
-                                   dtype=dtype, race_check=a.engine_race_check)
+                                   dtype=dtype, race_check=a.engine_race_check, expand_bytes=1 << 60)      # (the plan billed the scratch)
             else:
                 model = HybridModel(cfg, tp=a.engine_tp, rank=rank, device=dev, max_seqs=man.max_seqs, comm=comm,
                                     max_ctx=man.max_ctx, kv_blocks=kv_blocks, max_width=max(widths),

@@ -1,12 +1,18 @@
 // Gated delta rule with free head sizes, fp32 throughout.
 //
-// Prompt portions (ragged rows, any length): three launches.
-//   prep   one CTA row by row: convolution, silu, unit norms, beta and decay
-//   scan   the recurrence.  Columns of the state are independent, so a warp owns eight value columns
-//          for the whole portion: eight lanes split the key dimension, four lane groups take two columns
-//          each, the state stays in registers, and both products of a token (S^T k and S^T q; the
-//          read-out after the write is g S^T q + u (k . q)) meet in one three-step shuffle reduction.
-//          Eight tokens at a time are staged in shared memory by asynchronous copies, double buffered.
+// Prompt portions (ragged rows, any length), in blocks of four tokens: three launches.
+//   prep   convolution, silu, unit norms, beta and decay, and per block the dot products k_j . k_i and k_j . q_i
+//   scan   the recurrence.  Columns of the state are independent, so a warp owns eight value columns for the
+//          whole portion: eight lanes split the key dimension, four lane groups take two columns each, the state
+//          stays in registers.  A block of four tokens needs the products of its keys and queries with the state
+//          at its start only, S_0^T k_i and S_0^T q_i (independent of one another, one shuffle reduction for
+//          all); the rest is a triangular recurrence in scalars.  With G_i = g_1 .. g_i and
+//          D_ij = g_{j+1} .. g_i (products, no quotients):
+//              u_i = beta_i (v_i - G_i S_0^T k_i - sum_{j<i} D_ij (k_j . k_i) u_j)
+//              o_i = G_i S_0^T q_i + sum_{j<=i} D_ij (k_j . q_i) u_j
+//              S_4 = G_4 S_0 + sum_j D_4j k_j u_j^T
+//          which is the token-by-token rule written out; a block with fewer tokens is filled up with
+//          k = q = v = beta = 0, g = 1.  Blocks are staged in shared memory by asynchronous copies.
 //   out    gated norm into the operand of the output linear; the convolution inputs go to the ring
 // Decoding (one row per sequence): all of it in one launch, a CTA per (head, sequence).
 #include "delta.h"
@@ -14,8 +20,6 @@
 #include "ptx_sm100.cuh"
 
 namespace saber {
-
-constexpr int kDeltaMaxPerLane = 16;     // head sizes up to 512
 
 __device__ __forceinline__ float warp_sum_f(float v) {
 #pragma unroll
@@ -25,6 +29,10 @@ __device__ __forceinline__ float warp_sum_f(float v) {
 __device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f32(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
+
+__device__ __forceinline__ void cp_async16(float* dst, const float* src, int bytes) {    // bytes 0: zero fill
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
+}
 
 // sequence of a row (-1: a padding row), and whether its slot may be used
 __device__ __forceinline__ int seq_of_row(const int32_t* cu, int nseq, int m) {
@@ -54,47 +62,122 @@ __device__ __forceinline__ float conv_silu(const DeltaParams& p, const float* hi
   return silu_f32(acc);
 }
 
-// grid (M, ceil(items / 8)); a warp per item: q heads, k heads, v heads, then one item for beta / decay
-__global__ void __launch_bounds__(256) delta_prep_kernel(const __grid_constant__ DeltaParams p) {
+constexpr int kBlk = 4;                  // tokens per block
+constexpr int kPairs = 16;               // dot products per block: k_j . k_i (j < i: 6), k_j . q_i (j <= i: 10)
+__host__ __device__ constexpr int kk_at(int i, int j) { return i * (i - 1) / 2 + j; }
+__host__ __device__ constexpr int kq_at(int i, int j) { return 6 + i * (i + 1) / 2 + j; }
+
+// Blocks of sequence j occupy the slots from (first row / 4) + j on: disjoint for all sequences of a step.
+__device__ __forceinline__ int block_slot(int r0, int j, int c) { return (r0 >> 2) + j + c; }
+__device__ __forceinline__ bool block_of_slot(const DeltaParams& p, int slot, int& j, int& c) {
+  for (j = 0; j < p.nseq; ++j) {
+    const int r0 = p.cu_rows[j], n = p.cu_rows[j + 1] - r0;
+    c = slot - ((r0 >> 2) + j);
+    if (c >= 0 && c < (n + kBlk - 1) / kBlk) return true;
+  }
+  return false;
+}
+
+// convolution + silu of channel c for the rows of a block (m: its first row, t: that row inside its sequence)
+__device__ __forceinline__ void conv_silu4(const DeltaParams& p, const float* hist, int c, int col, int m, int t, int pos, int C, int rows,
+                                           float (&y)[kBlk]) {
+  float acc[kBlk] = {};
+  for (int back = p.taps - 1; back > -kBlk; --back) {              // input row m - back feeds rows r >= -back
+    if (-back >= rows) break;
+    float x = 0.f;
+    if (back <= t) x = p.x[static_cast<size_t>(m - back) * p.ldx + col];
+    else if (back <= pos) x = hist[static_cast<size_t>((pos - back) % p.taps) * C + c];
+#pragma unroll
+    for (int r = 0; r < kBlk; ++r) {
+      const int i = p.taps - 1 - (r + back);                        // tap of this input for row r
+      if (i >= 0 && i < p.taps) acc[r] = fmaf(x, p.conv_w[static_cast<size_t>(c) * p.taps + i], acc[r]);
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < kBlk; ++r) y[r] = r < rows ? silu_f32(acc[r]) : 0.f;
+}
+
+// grid (blocks, ceil(items / 4)), 128 threads; a warp per item: key heads (q, k and their dot products), value heads,
+// then one item for beta / decay
+template <int NI>
+__global__ void __launch_bounds__(128) delta_prep_kernel(const __grid_constant__ DeltaParams p) {
   pdl_wait();
-  const int m = blockIdx.x;
   const int lane = threadIdx.x & 31;
-  const int item = blockIdx.y * 8 + (threadIdx.x >> 5);
-  if (item > 2 * p.HK + p.H) return;
-  const int j = seq_of_row(p.cu_rows, p.nseq, m);
-  if (j < 0) return;
+  const int item = blockIdx.y * 4 + (threadIdx.x >> 5);
+  if (item > p.HK + p.H) return;
+  int j, blk;
+  if (!block_of_slot(p, blockIdx.x, j, blk)) return;
   const int slot = delta_slot(p, j);
   if (slot < 0) return;
-  const int t = m - p.cu_rows[j], pos = p.pos[m];
+  constexpr int DP = NI * 32;
+  const int t = blk * kBlk, m = p.cu_rows[j] + t, rows = min(kBlk, p.cu_rows[j + 1] - m), pos = p.pos[m];
   const int C = 2 * p.HK * p.D + p.H * p.V;
   const float* hist = p.hist + static_cast<size_t>(slot) * p.taps * C;
-  if (item < 2 * p.HK) {
-    const bool isq = item < p.HK;
-    const int h = isq ? item : item - p.HK;
-    const int c0 = (isq ? 0 : p.HK * p.D) + h * p.D, col0 = (isq ? p.q_off : p.k_off) + h * p.D;
-    float v[kDeltaMaxPerLane];
-    float sq = 0.f;
+  if (item < p.HK) {
+    const int h = item;
+    float qv[NI][kBlk], kv[NI][kBlk], sq[2][kBlk] = {};
 #pragma unroll
-    for (int i = 0; i < kDeltaMaxPerLane; ++i) {
+    for (int i = 0; i < NI; ++i) {
       const int d = i * 32 + lane;
-      v[i] = 0.f;
-      if (d < p.D) v[i] = conv_silu(p, hist, c0 + d, col0 + d, m, t, pos, C);
-      sq += v[i] * v[i];
-    }
-    const float r = 1.f / sqrtf(warp_sum_f(sq) + p.unit_eps) * (isq ? p.q_scale : 1.f);
-    float* o = (isq ? p.qn : p.kn) + (static_cast<size_t>(m) * p.HK + h) * p.DP;
 #pragma unroll
-    for (int i = 0; i < kDeltaMaxPerLane; ++i)
-      if (i * 32 + lane < p.DP) o[i * 32 + lane] = v[i] * r;
-  } else if (item < 2 * p.HK + p.H) {
-    const int h = item - 2 * p.HK;
-    float* o = p.vv + (static_cast<size_t>(m) * p.H + h) * p.VP;
-    for (int d = lane; d < p.VP; d += 32)
-      o[d] = d < p.V ? conv_silu(p, hist, 2 * p.HK * p.D + h * p.V + d, p.v_off + h * p.V + d, m, t, pos, C) : 0.f;
+      for (int r = 0; r < kBlk; ++r) qv[i][r] = kv[i][r] = 0.f;
+      if (d < p.D) {
+        conv_silu4(p, hist, h * p.D + d, p.q_off + h * p.D + d, m, t, pos, C, rows, qv[i]);
+        conv_silu4(p, hist, (p.HK + h) * p.D + d, p.k_off + h * p.D + d, m, t, pos, C, rows, kv[i]);
+      }
+#pragma unroll
+      for (int r = 0; r < kBlk; ++r) {
+        sq[0][r] += qv[i][r] * qv[i][r];
+        sq[1][r] += kv[i][r] * kv[i][r];
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < kBlk; ++r) {
+      const float a = 1.f / sqrtf(warp_sum_f(sq[0][r]) + p.unit_eps) * p.q_scale;
+      const float b = 1.f / sqrtf(warp_sum_f(sq[1][r]) + p.unit_eps);
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        qv[i][r] *= a;
+        kv[i][r] *= b;
+        if (r < rows) {
+          const size_t o = (static_cast<size_t>(m + r) * p.HK + h) * DP + i * 32 + lane;
+          p.qn[o] = qv[i][r];
+          p.kn[o] = kv[i][r];
+        }
+      }
+    }
+    float* pr = p.pairs + (static_cast<size_t>(blockIdx.x) * p.HK + h) * kPairs;
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i)
+#pragma unroll
+      for (int jj = 0; jj <= i; ++jj) {
+        float kk = 0.f, kq = 0.f;
+#pragma unroll
+        for (int n = 0; n < NI; ++n) {
+          if (jj < i) kk = fmaf(kv[n][jj], kv[n][i], kk);
+          kq = fmaf(kv[n][jj], qv[n][i], kq);
+        }
+        kq = warp_sum_f(kq);
+        if (jj < i) kk = warp_sum_f(kk);
+        if (lane == 0) {
+          pr[kq_at(i, jj)] = kq;
+          if (jj < i) pr[kk_at(i, jj)] = kk;
+        }
+      }
+  } else if (item < p.HK + p.H) {
+    const int h = item - p.HK;
+    for (int d = lane; d < p.VP; d += 32) {
+      float y[kBlk] = {};
+      if (d < p.V) conv_silu4(p, hist, 2 * p.HK * p.D + h * p.V + d, p.v_off + h * p.V + d, m, t, pos, C, rows, y);
+#pragma unroll
+      for (int r = 0; r < kBlk; ++r)
+        if (r < rows) p.vv[(static_cast<size_t>(m + r) * p.H + h) * p.VP + d] = y[r];
+    }
   } else {
-    const float* x = p.x + static_cast<size_t>(m) * p.ldx;
-    for (int h = lane; h < p.H; h += 32) {
-      float* o = p.bg + (static_cast<size_t>(m) * p.H + h) * 2;
+    for (int i = lane; i < p.H * rows; i += 32) {
+      const int r = i / p.H, h = i - r * p.H;
+      const float* x = p.x + static_cast<size_t>(m + r) * p.ldx;
+      float* o = p.bg + (static_cast<size_t>(m + r) * p.H + h) * 2;
       o[0] = sigmoid_f32(x[p.b_off + h]);
       o[1] = expf(-expf(p.A_log[h]) * softplus_f32(x[p.a_off + h] + p.dt_bias[h]));
     }
@@ -160,7 +243,7 @@ __device__ __forceinline__ void delta_state_io(float* st, float (&S)[NI][4][2], 
     }
 }
 
-constexpr int kScanRows = 8;
+constexpr int kStage = 2;                // blocks per staged buffer
 
 // grid (nseq, H, ceil(VP / 32)), 128 threads
 template <int NI>
@@ -170,6 +253,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const __grid_constant__
   float* sm = reinterpret_cast<float*>(sm4);
   constexpr int DP = NI * 32;
   constexpr int kRow = 2 * DP + 32 + 4;            // k | q | 32 value columns | beta, g
+  constexpr int kBlock = kBlk * kRow + kPairs;     // four rows, then the dot products
   const int j = blockIdx.x, h = blockIdx.y;
   const int r0 = p.cu_rows[j], n = p.cu_rows[j + 1] - r0;
   if (n <= 0) return;
@@ -183,31 +267,43 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const __grid_constant__
   float S[NI][4][2] = {};
   float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + vb + cl) * DP;
   if (on) delta_state_io<NI>(st, S, DP, lg, false);
+  const int blocks = (n + kBlk - 1) / kBlk;
 
-  auto fetch = [&](int c) {                        // rows [c * kScanRows, ...) into buffer c & 1
-    float* b = sm + (c & 1) * kScanRows * kRow;
-    const int rows = min(kScanRows, n - c * kScanRows);
-    for (int i = threadIdx.x; i < rows * (kRow / 4); i += 128) {
-      const int r = i / (kRow / 4), w = i - r * (kRow / 4);
-      const size_t m = r0 + c * kScanRows + r;
-      const float* src;
-      if (w < DP / 4) src = p.kn + (m * p.HK + hk) * DP + w * 4;
-      else if (w < DP / 2) src = p.qn + (m * p.HK + hk) * DP + (w - DP / 4) * 4;
-      else if (w < DP / 2 + 8) {
-        const int v = (w - DP / 2) * 4;
-        if (v >= nv) continue;
-        src = p.vv + (m * p.H + h) * p.VP + vb + v;
-      } else {
-        // beta, g: eight bytes
-        const float* s2 = p.bg + (m * p.H + h) * 2;
-        asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(b + r * kRow + w * 4)), "l"(s2) : "memory");
-        continue;
+  auto fetch = [&](int c) {                        // blocks [c * kStage, ...) into buffer c & 1
+    for (int bi = 0; bi < kStage; ++bi) {
+      const int blk = c * kStage + bi;
+      if (blk >= blocks) break;
+      float* b = sm + ((c & 1) * kStage + bi) * kBlock;
+      const int rows = min(kBlk, n - blk * kBlk);
+      for (int i = threadIdx.x; i < kBlk * (kRow / 4) + kPairs / 4; i += 128) {
+        const int r = i / (kRow / 4), w = i - r * (kRow / 4);
+        if (r == kBlk) {
+          cp_async16(b + kBlk * kRow + w * 4, p.pairs + (static_cast<size_t>(block_slot(r0, j, blk)) * p.HK + hk) * kPairs + w * 4, 16);
+          continue;
+        }
+        const bool live = r < rows;
+        const size_t m = r0 + blk * kBlk + (live ? r : 0);
+        const float* src;
+        int bytes = 16;
+        if (w < DP / 4) src = p.kn + (m * p.HK + hk) * DP + w * 4;
+        else if (w < DP / 2) src = p.qn + (m * p.HK + hk) * DP + (w - DP / 4) * 4;
+        else if (w < DP / 2 + 8) {
+          const int v = (w - DP / 2) * 4;
+          if (v >= nv) continue;
+          src = p.vv + (m * p.H + h) * p.VP + vb + v;
+        } else {
+          // beta, g: eight bytes (a missing token: zeros here, its g is taken as 1 below)
+          src = p.bg + (m * p.H + h) * 2;
+          asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(smem_u32(b + r * kRow + w * 4)), "l"(src), "r"(live ? 8u : 0u)
+                       : "memory");
+          continue;
+        }
+        cp_async16(b + r * kRow + w * 4, src, live ? bytes : 0);
       }
-      asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(smem_u32(b + r * kRow + w * 4)), "l"(src) : "memory");
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  const int chunks = (n + kScanRows - 1) / kScanRows;
+  const int chunks = (blocks + kStage - 1) / kStage;
   fetch(0);
   for (int c = 0; c < chunks; ++c) {
     if (c + 1 < chunks) {
@@ -218,15 +314,109 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const __grid_constant__
     }
     __syncthreads();
     if (on) {
-      const float* b = sm + (c & 1) * kScanRows * kRow;
-      const int rows = min(kScanRows, n - c * kScanRows);
-      for (int r = 0; r < rows; ++r, b += kRow) {
-        const float2 v = *reinterpret_cast<const float2*>(b + 2 * DP + cl);
-        const float2 bg = *reinterpret_cast<const float2*>(b + 2 * DP + 32);
-        float o0, o1;
-        delta_token<NI>(S, b, b + DP, lg, v.x, v.y, bg.x, bg.y, o0, o1);
-        if (lg == 0)
-          *reinterpret_cast<float2*>(p.o + (static_cast<size_t>(r0 + c * kScanRows + r) * p.H + h) * p.VP + vb + cl) = make_float2(o0, o1);
+      for (int bi = 0; bi < kStage; ++bi) {
+        const int blk = c * kStage + bi;
+        if (blk >= blocks) break;
+        const float* b = sm + ((c & 1) * kStage + bi) * kBlock;
+        const int rows = min(kBlk, n - blk * kBlk);
+        float sk[kBlk][2] = {}, sq[kBlk][2] = {};
+#pragma unroll
+        for (int r = 0; r < kBlk; ++r) {
+          const float* kr = b + r * kRow;
+#pragma unroll
+          for (int i = 0; i < NI; ++i) {
+            const float4 k4 = *reinterpret_cast<const float4*>(kr + i * 32 + lg * 4);
+            const float4 q4 = *reinterpret_cast<const float4*>(kr + DP + i * 32 + lg * 4);
+            const float ka[4] = {k4.x, k4.y, k4.z, k4.w}, qa[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+#pragma unroll
+              for (int v = 0; v < 2; ++v) {
+                sk[r][v] = fmaf(S[i][e][v], ka[e], sk[r][v]);
+                sq[r][v] = fmaf(S[i][e][v], qa[e], sq[r][v]);
+              }
+          }
+        }
+#pragma unroll
+        for (int o = 1; o < 8; o <<= 1)
+#pragma unroll
+          for (int r = 0; r < kBlk; ++r)
+#pragma unroll
+            for (int v = 0; v < 2; ++v) sk[r][v] += __shfl_xor_sync(0xffffffffu, sk[r][v], o);
+        // the read-out values: lane lg keeps token lg >> 1, column lg & 1 (halving exchange: 4 + 2 + 1 shuffles)
+        float mine;
+        {
+          float t4[4], t2[2];
+          const bool b2 = (lg & 4) != 0, b1 = (lg & 2) != 0, b0 = (lg & 1) != 0;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {            // tokens 0, 1 stay with b2 = 0; tokens 2, 3 with b2 = 1
+            const float keep = b2 ? sq[2 + (e >> 1)][e & 1] : sq[e >> 1][e & 1];
+            const float give = b2 ? sq[e >> 1][e & 1] : sq[2 + (e >> 1)][e & 1];
+            t4[e] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+          }
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float keep = b1 ? t4[2 + e] : t4[e], give = b1 ? t4[e] : t4[2 + e];
+            t2[e] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+          }
+          const float keep = b0 ? t2[1] : t2[0], give = b0 ? t2[0] : t2[1];
+          mine = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+        }
+        float beta[kBlk], g[kBlk], G[kBlk], dl[kBlk], u[kBlk][2], pr[kPairs];
+#pragma unroll
+        for (int e = 0; e < kPairs; e += 4) *reinterpret_cast<float4*>(pr + e) = *reinterpret_cast<const float4*>(b + kBlk * kRow + e);
+#pragma unroll
+        for (int r = 0; r < kBlk; ++r) {
+          const float2 bg = *reinterpret_cast<const float2*>(b + r * kRow + 2 * DP + 32);
+          beta[r] = bg.x;
+          g[r] = r < rows ? bg.y : 1.f;
+          G[r] = r == 0 ? g[0] : G[r - 1] * g[r];
+        }
+        const int tok = lg >> 1;
+        float o = 0.f;
+#pragma unroll
+        for (int i = 0; i < kBlk; ++i) {
+          const float2 v = *reinterpret_cast<const float2*>(b + i * kRow + 2 * DP + cl);
+          float a0 = v.x - G[i] * sk[i][0], a1 = v.y - G[i] * sk[i][1];
+#pragma unroll
+          for (int jj = 0; jj < i; ++jj) {
+            dl[jj] *= g[i];                        // D_ij
+            const float w = dl[jj] * pr[kk_at(i, jj)];
+            a0 = fmaf(-w, u[jj][0], a0);
+            a1 = fmaf(-w, u[jj][1], a1);
+          }
+          dl[i] = 1.f;
+          u[i][0] = beta[i] * a0;
+          u[i][1] = beta[i] * a1;
+          if (tok == i) {
+            o = G[i] * mine;
+#pragma unroll
+            for (int jj = 0; jj <= i; ++jj) o = fmaf(dl[jj] * pr[kq_at(i, jj)], (lg & 1) ? u[jj][1] : u[jj][0], o);
+          }
+        }
+        if (tok < rows) p.o[(static_cast<size_t>(r0 + blk * kBlk + tok) * p.H + h) * p.VP + vb + cl + (lg & 1)] = o;
+#pragma unroll
+        for (int jj = 0; jj < kBlk; ++jj) {        // D_4j is where the recurrence left it
+          u[jj][0] *= dl[jj];
+          u[jj][1] *= dl[jj];
+        }
+        const float G4 = G[kBlk - 1];
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) { S[i][e][0] *= G4; S[i][e][1] *= G4; }
+#pragma unroll
+        for (int r = 0; r < kBlk; ++r)
+#pragma unroll
+          for (int i = 0; i < NI; ++i) {
+            const float4 k4 = *reinterpret_cast<const float4*>(b + r * kRow + i * 32 + lg * 4);
+            const float ka[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              S[i][e][0] = fmaf(u[r][0], ka[e], S[i][e][0]);
+              S[i][e][1] = fmaf(u[r][1], ka[e], S[i][e][1]);
+            }
+          }
       }
     }
     __syncthreads();
@@ -240,6 +430,16 @@ __device__ __forceinline__ void delta_gated_norm(const DeltaParams& p, const flo
   for (int v = lane; v < p.V; v += 32) sq += o[v] * o[v];
   const float r = 1.f / sqrtf(warp_sum_f(sq) / static_cast<float>(p.V) + p.eps);
   const float* g = p.x + static_cast<size_t>(m) * p.ldx + p.g_off + h * p.V;
+  if ((p.V & 3) == 0) {                            // (the gate's columns start at a multiple of 8, VP is one too)
+    for (int v = lane * 4; v < p.V; v += 128) {
+      const float4 a = *reinterpret_cast<const float4*>(o + v), b = *reinterpret_cast<const float4*>(g + v),
+                   w = *reinterpret_cast<const float4*>(p.norm_w + v);
+      operand_store4(p.out, m, p.out_k0 + h * p.V + v,
+                     make_float4(a.x * r * w.x * silu_f32(b.x), a.y * r * w.y * silu_f32(b.y), a.z * r * w.z * silu_f32(b.z),
+                                 a.w * r * w.w * silu_f32(b.w)));
+    }
+    return;
+  }
   for (int v = lane; v < p.V; v += 32) operand_store1(p.out, m, p.out_k0 + h * p.V + v, o[v] * r * p.norm_w[v] * silu_f32(g[v]));
 }
 
@@ -367,7 +567,7 @@ static int delta_go(const DeltaParams& p, bool single, cudaStream_t stream) {
     const int smem = (2 * NI * 32 + 2 * p.VP) * 4;
     return static_cast<int>(launch(delta_step_kernel<NI>, dim3(p.H, p.nseq), dim3(32 * warps), smem, stream, 0, p));
   }
-  const int smem = 2 * kScanRows * (2 * NI * 32 + 36) * 4;
+  const int smem = 2 * kStage * (kBlk * (2 * NI * 32 + 36) + kPairs) * 4;
   static bool ready[64];
   int dev = 0;
   cudaGetDevice(&dev);
@@ -377,7 +577,7 @@ static int delta_go(const DeltaParams& p, bool single, cudaStream_t stream) {
     if (e != cudaSuccess) return static_cast<int>(e);
     ready[dev] = true;
   }
-  cudaError_t e = launch(delta_prep_kernel, dim3(p.M, (2 * p.HK + p.H + 8) / 8), dim3(256), 0, stream, 0, p);
+  cudaError_t e = launch(delta_prep_kernel<NI>, dim3(p.M / kBlk + p.nseq, (p.HK + p.H + 4) / 4), dim3(128), 0, stream, 0, p);
   if (e == cudaSuccess) e = launch(delta_scan_kernel<NI>, dim3(p.nseq, p.H, (p.VP + 31) / 32), dim3(128), smem, stream, 0, p);
   if (e == cudaSuccess) e = launch(delta_out_kernel, dim3(p.M + p.nseq, (p.H + 7) / 8), dim3(256), 0, stream, 0, p);
   return static_cast<int>(e);

@@ -27,6 +27,7 @@ struct DeltaParams {
   float* kn;               // scratch [M][HK][DP]
   float* vv;               // scratch [M][H][VP]
   float* bg;               // scratch [M][H][2]: beta, g
+  float* pairs;            // scratch [M / 4 + nseq][HK][16]: dot products inside each block of four tokens
   float* o;                // scratch [M][H][VP]
   const int32_t* cu_rows;  // [nseq + 1]
   const int32_t* slots;    // [nseq], < 0: padding sequence

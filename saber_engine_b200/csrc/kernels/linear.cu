@@ -19,6 +19,7 @@ namespace saber {
 
 constexpr int kLinThreads = 320;
 constexpr int kLinMaxStages = 8;
+constexpr int kLinRow = 260;              // floats per staged accumulator row (16-byte accesses of eight lanes hit all banks)
 constexpr uint32_t kLinTile = 32768;      // 256 weight rows x 64 bf16
 
 __device__ __forceinline__ float clamped_glu(float gate, float up, float limit, float alpha) {
@@ -27,11 +28,73 @@ __device__ __forceinline__ float clamped_glu(float gate, float up, float limit, 
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
 }
 
-__device__ __forceinline__ float row_rms_scale(const LinEpi& e, int m) {
+// reciprocal root mean square of the stream row behind operand row m (all lanes of a warp call together)
+__device__ __forceinline__ float row_rms_scale(const LinEpi& e, int m, int lane) {
   if (e.ss == nullptr) return 1.f;
   float s = 0.f;
-  for (int i = 0; i < e.ss_n; ++i) s += __ldcg(e.ss + static_cast<size_t>(m) * e.ss_n + i);
+  for (int i = lane; i < e.ss_n; i += 32) s += __ldcg(e.ss + static_cast<size_t>(m) * e.ss_n + i);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
   return 1.f / sqrtf(s * e.inv_width + e.eps);
+}
+
+// One finished row of a 256-column tile, by a warp.  acc(c): the eight (project, stream) or four (gated unit)
+// accumulators from column c on.
+template <typename Acc>
+__device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& acc, int m, int tile_n, int lane) {
+  const int n0 = tile_n * 256;
+  if (!e.stream) {
+    const float sc = row_rms_scale(e, m, lane);
+    if (tile_n < e.act_tile0) {
+      const int n = n0 + lane * 8;
+      if (n >= e.n_plain) return;
+      const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+      float* o = e.out + static_cast<size_t>(m) * e.ldo + n;
+      if (n + 8 <= e.n_plain) {
+        *reinterpret_cast<float4*>(o) = make_float4(a.x * sc, a.y * sc, a.z * sc, a.w * sc);
+        *reinterpret_cast<float4*>(o + 4) = make_float4(b.x * sc, b.y * sc, b.z * sc, b.w * sc);
+      } else {
+        const float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (n + j < e.n_plain) o[j] = v[j] * sc;
+      }
+    } else {
+      const float4 g = acc(lane * 4), u = acc(128 + lane * 4);
+      operand_store4(e.act, m, e.act_k0 + (tile_n - e.act_tile0) * 128 + lane * 4,
+                     make_float4(clamped_glu(g.x * sc, u.x * sc, e.limit, e.alpha), clamped_glu(g.y * sc, u.y * sc, e.limit, e.alpha),
+                                 clamped_glu(g.z * sc, u.z * sc, e.limit, e.alpha), clamped_glu(g.w * sc, u.w * sc, e.limit, e.alpha)));
+    }
+    return;
+  }
+  const int n = n0 + lane * 8;
+  float sq = 0.f;
+  if (n < e.width) {                              // ldx is a multiple of 32: whole groups of eight are in bounds
+    float* xr = e.x + static_cast<size_t>(m) * e.ldx + n;
+    const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+    float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+    if (e.add) {
+      const float4 x0 = *reinterpret_cast<const float4*>(xr), x1 = *reinterpret_cast<const float4*>(xr + 4);
+      v[0] += x0.x; v[1] += x0.y; v[2] += x0.z; v[3] += x0.w;
+      v[4] += x1.x; v[5] += x1.y; v[6] += x1.z; v[7] += x1.w;
+    }
+    float y[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const bool in = n + j < e.width;
+      if (e.bias && in) v[j] += e.bias[n + j];
+      sq += v[j] * v[j];
+      y[j] = e.norm_w ? (in ? v[j] * e.norm_w[n + j] : 0.f) : v[j];
+    }
+    *reinterpret_cast<float4*>(xr) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(xr + 4) = make_float4(v[4], v[5], v[6], v[7]);
+    operand_store8(e.op, m, e.op_k0 + n, y);
+  }
+  if (e.ss_out == nullptr) return;
+#pragma unroll
+  for (int o = 8; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);       // per half warp: 128 columns
+  const int g = tile_n * 2 + (lane >> 4);
+  if ((lane & 15) == 0 && g < e.ss_out_n) e.ss_out[static_cast<size_t>(m) * e.ss_out_n + g] = sq;
 }
 
 template <int kMT>
@@ -39,7 +102,6 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t bars[2 * kLinMaxStages + 1];
   __shared__ uint32_t tmem_base_s, is_last_s, abort_s;
-  __shared__ float bias_s[256], normw_s[256];
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tile_m = blockIdx.x, tile_n = blockIdx.y, split = blockIdx.z;
@@ -143,16 +205,12 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
     }
   } else {
     // ---------------------------------------------------------------- epilogue (8 warps)
+    // The accumulator arrives a row per lane; it is staged in shared memory (the operand ring is idle by then) so
+    // that a warp finishes a whole 256-column row at a time with contiguous global accesses.
     const int te = threadIdx.x - 64;              // 0..255
-    const int grp = te >> 7;                      // column half
+    const int grp = te >> 7;                      // column half this warp reads out
     const int q4 = warp & 3;                      // TMEM lane quarter of this warp
     const LinEpi& e = p.e;
-    const int n0 = tile_n * 256;
-    if (e.stream) {
-      const bool in = n0 + te < e.width;
-      bias_s[te] = (e.bias && in) ? e.bias[n0 + te] : 0.f;
-      normw_s[te] = in ? (e.norm_w ? e.norm_w[n0 + te] : 1.f) : 0.f;
-    }
     bool ok = mbar_wait(bar_acc, 0, p.err, kErrWaitAcc);
     if (!ok) abort_s = 1u;
     named_bar_sync(1, 256);
@@ -162,7 +220,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
     const int rowl = q4 * 32 + lane;
     const uint32_t t_lane = tmem_d + (static_cast<uint32_t>(q4 * 32) << 16);
     const int tile_lin = tile_m * gridDim.y + tile_n;
-    bool from_ws = false;
+    float* tile_s = reinterpret_cast<float*>(smem_raw + (a_smem - smem_u32(smem_raw)));
     if (p.splits > 1) {                           // (kMT == 1)
       const int mt = min(p.nt, p.M - m0);
       float* part = p.ws + (static_cast<size_t>(tile_lin) * p.splits + split) * p.nt * 256;
@@ -192,109 +250,47 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
       named_bar_sync(1, 256);
       if (!is_last_s) ok = false;
       __threadfence();
-      from_ws = true;
-    }
-    if (ok) {
-      const float* parts = p.ws + static_cast<size_t>(tile_lin) * p.splits * p.nt * 256;
+      if (ok) {                                   // the parts in order, a 16-byte group per thread
+        const float* parts = p.ws + static_cast<size_t>(tile_lin) * p.splits * p.nt * 256;
+        const size_t step = static_cast<size_t>(p.nt) * 256;
+        for (int i = te; i < 64 * mt; i += 256) {
+          const int c4 = i / mt, r = i - c4 * mt;
+          const float* src = parts + (static_cast<size_t>(c4) * p.nt + r) * 4;
+          float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+          for (int sp = 0; sp < p.splits; ++sp) {
+            const float4 f = __ldcg(reinterpret_cast<const float4*>(src + sp * step));
+            s.x += f.x; s.y += f.y; s.z += f.z; s.w += f.w;
+          }
+          *reinterpret_cast<float4*>(tile_s + r * kLinRow + c4 * 4) = s;
+        }
+        named_bar_sync(1, 256);
+        for (int r = warp - 2; r < mt; r += 8)
+          linear_row_epilogue(e, [&](int c) { return *reinterpret_cast<const float4*>(tile_s + r * kLinRow + c); }, m0 + r, tile_n, lane);
+      }
+    } else if (ok) {
 #pragma unroll 1
       for (int j2 = 0; j2 < kMT; ++j2) {
         const int mb = m0 + j2 * p.nt;
         const int mt = min(p.nt, p.M - mb);
-        if (q4 * 32 >= mt) continue;              // warp-uniform
-        const bool live = rowl < mt;
-        const int m = mb + rowl;
-        // 32 accumulator columns from c on (all lanes of the warp call together)
-        auto load = [&](int c, float (&v)[32]) {
-          if (!from_ws) {
+        if (mt <= 0) break;                       // uniform
+        if (j2 > 0) named_bar_sync(1, 256);
+        if (q4 * 32 < mt) {
+          for (int c = grp * 128; c < grp * 128 + 128; c += 32) {
             uint32_t r[32];
             tmem_ld32(t_lane + static_cast<uint32_t>(j2) * 256u + c, r);
             tmem_ld_wait();
+            if (rowl < mt) {
 #pragma unroll
-            for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
-          } else {
-#pragma unroll
-            for (int j = 0; j < 32; ++j) v[j] = 0.f;
-            if (live) {
-              for (int sp = 0; sp < p.splits; ++sp) {
-                const float* part = parts + static_cast<size_t>(sp) * p.nt * 256;
-#pragma unroll
-                for (int j = 0; j < 8; ++j) {
-                  const float4 f = __ldcg(reinterpret_cast<const float4*>(part + (static_cast<size_t>((c >> 2) + j) * p.nt + rowl) * 4));
-                  v[4 * j] += f.x; v[4 * j + 1] += f.y; v[4 * j + 2] += f.z; v[4 * j + 3] += f.w;
-                }
-              }
+              for (int j = 0; j < 8; ++j)
+                *reinterpret_cast<float4*>(tile_s + rowl * kLinRow + c + 4 * j) =
+                    make_float4(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]), __uint_as_float(r[4 * j + 2]), __uint_as_float(r[4 * j + 3]));
             }
           }
-        };
-        if (!e.stream) {
-          const float sc = live ? row_rms_scale(e, m) : 0.f;
-          if (tile_n < e.act_tile0) {
-            for (int c = grp * 128; c < grp * 128 + 128; c += 32) {
-              if (n0 + c >= e.n_plain) break;
-              float v[32];
-              load(c, v);
-              if (live) {
-                float* o = e.out + static_cast<size_t>(m) * e.ldo + n0 + c;
-                if (n0 + c + 32 <= e.n_plain) {
-#pragma unroll
-                  for (int j = 0; j < 8; ++j)
-                    *reinterpret_cast<float4*>(o + 4 * j) = make_float4(v[4 * j] * sc, v[4 * j + 1] * sc, v[4 * j + 2] * sc, v[4 * j + 3] * sc);
-                } else {
-#pragma unroll
-                  for (int j = 0; j < 32; ++j)
-                    if (n0 + c + j < e.n_plain) o[j] = v[j] * sc;
-                }
-              }
-            }
-          } else {
-            const int k0 = e.act_k0 + (tile_n - e.act_tile0) * 128;
-            for (int c = grp * 64; c < grp * 64 + 64; c += 32) {
-              float g[32], u[32];
-              load(c, g);
-              load(128 + c, u);
-              if (live) {
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                  float y[8];
-#pragma unroll
-                  for (int i = 0; i < 8; ++i) y[i] = clamped_glu(g[8 * j + i] * sc, u[8 * j + i] * sc, e.limit, e.alpha);
-                  operand_store8(e.act, m, k0 + c + 8 * j, y);
-                }
-              }
-            }
-          }
-        } else {
-          float sq = 0.f;
-          for (int c = grp * 128; c < grp * 128 + 128; c += 32) {
-            if (n0 + c >= e.width) break;
-            float v[32];
-            load(c, v);
-            if (live) {
-              float* xr = e.x + static_cast<size_t>(m) * e.ldx + n0 + c;     // ldx is a multiple of 32: whole groups are in bounds
-#pragma unroll
-              for (int j = 0; j < 8; ++j) {
-                float4 o = e.add ? *reinterpret_cast<const float4*>(xr + 4 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
-                const float* b = bias_s + c + 4 * j;
-                o.x += v[4 * j] + b[0]; o.y += v[4 * j + 1] + b[1]; o.z += v[4 * j + 2] + b[2]; o.w += v[4 * j + 3] + b[3];
-                *reinterpret_cast<float4*>(xr + 4 * j) = o;
-                v[4 * j] = o.x; v[4 * j + 1] = o.y; v[4 * j + 2] = o.z; v[4 * j + 3] = o.w;
-              }
-#pragma unroll
-              for (int j = 0; j < 4; ++j) {
-                float y[8];
-#pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                  const float t = v[8 * j + i];
-                  sq += t * t;
-                  y[i] = t * normw_s[c + 8 * j + i];
-                }
-                operand_store8(e.op, m, e.op_k0 + n0 + c + 8 * j, y);
-              }
-            }
-          }
-          if (live && e.ss_out != nullptr && tile_n * 2 + grp < e.ss_out_n)
-            e.ss_out[static_cast<size_t>(m) * e.ss_out_n + tile_n * 2 + grp] = sq;
         }
+        named_bar_sync(1, 256);
+        for (int r = warp - 2; r < mt; r += 8)
+          linear_row_epilogue(e, [&](int c) { return *reinterpret_cast<const float4*>(tile_s + r * kLinRow + c); }, mb + r, tile_n, lane);
       }
     }
   }
@@ -346,7 +342,7 @@ __global__ void __launch_bounds__(256) lin_epi_kernel(const __grid_constant__ Li
   const int m = blockIdx.x;
   const float* acc = p.ws + static_cast<size_t>(m) * p.N_pad;
   if (!e.stream) {
-    const float sc = row_rms_scale(e, m);
+    const float sc = row_rms_scale(e, m, threadIdx.x & 31);
     for (int n = threadIdx.x; n < e.n_plain; n += 256) e.out[static_cast<size_t>(m) * e.ldo + n] = acc[n] * sc;
     const int tiles = p.N_pad / 256;
     for (int i = threadIdx.x; i < (tiles - e.act_tile0) * 128; i += 256) {
@@ -458,7 +454,7 @@ extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t strea
   const int abytes = p->nt * 128 * (pair ? 2 : 1);
   int stages = (kSmem - 1024) / (static_cast<int>(kLinTile) + abytes);
   if (stages > kLinMaxStages) stages = kLinMaxStages;
-  const int smem = stages * (static_cast<int>(kLinTile) + abytes) + 1024;
+  const int smem = stages * (static_cast<int>(kLinTile) + abytes) + 1024;      // (at least 3 stages: a staged tile of 128 rows fits)
   const int tiles_m = pair ? (p->M + 255) / 256 : (p->M + p->nt - 1) / p->nt;
   const dim3 grid(tiles_m, p->N_pad / 256, p->splits);
   cudaError_t r = pair ? launch(lin_bf16_kernel<2>, grid, dim3(kLinThreads), smem, stream, 2, q, stages)

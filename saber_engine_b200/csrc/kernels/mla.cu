@@ -22,11 +22,18 @@ template <typename T>
 __global__ void __launch_bounds__(256) mla_prep_kernel(const __grid_constant__ MlaParams p) {
   pdl_wait();
   __shared__ float red[8];
+  extern __shared__ float rot[];                  // [R / 2] cosines, [R / 2] sines of this position
   const int m = blockIdx.x;
   if (mla_seq_of_row(p.cu_rows, p.nseq, m) < 0) return;
   const float* x = p.x + static_cast<size_t>(m) * p.ldx;
   const float pos = static_cast<float>(p.pos[m]);
   const int half = p.R / 2, LD = p.CP + p.RP;
+  for (int f = threadIdx.x; f < half; f += 256) {
+    float sn, cs;
+    sincosf(pos * p.freq[f], &sn, &cs);
+    rot[f] = cs;
+    rot[half + f] = sn;
+  }
   const float* d = x + p.dkv_off;
   float sq = 0.f;
   for (int i = threadIdx.x; i < p.C; i += 256) sq += d[i] * d[i];
@@ -44,8 +51,7 @@ __global__ void __launch_bounds__(256) mla_prep_kernel(const __grid_constant__ M
       float v = 0.f;
       if (i < p.R) {
         const int f = i < half ? i : i - half;
-        float sn, cs;
-        sincosf(pos * p.freq[f], &sn, &cs);
+        const float cs = rot[f], sn = rot[half + f];
         const float a = d[p.C + f], b = d[p.C + f + half];
         v = i < half ? a * cs - b * sn : b * cs + a * sn;
       }
@@ -61,8 +67,7 @@ __global__ void __launch_bounds__(256) mla_prep_kernel(const __grid_constant__ M
     float v = 0.f;
     if (k < p.R) {
       const int f = k < half ? k : k - half;
-      float sn, cs;
-      sincosf(pos * p.freq[f], &sn, &cs);
+      const float cs = rot[f], sn = rot[half + f];
       const float* qr = x + p.q_off + h * (p.D + p.R) + p.D;
       const float a = qr[f], b = qr[f + half];
       v = k < half ? a * cs - b * sn : b * cs + a * sn;
@@ -76,34 +81,65 @@ __global__ void __launch_bounds__(256) mla_prep_kernel(const __grid_constant__ M
     }
 }
 
-// grid (ceil(CP / 128), H, ceil(M / 8)), 128 threads: q_eff[m][h][r] = sum_d W_uk[h D + d][r] q[m][h][d]
+// grid (ceil(CP / 128), H, ceil(M / 8)), 256 threads: q_eff[m][h][r] = sum_d W_uk[h D + d][r] q[m][h][d] for eight rows.
+// 64 column pairs; four thread groups take a quarter of the d each and meet in shared memory.
+template <typename T> struct Pair;
+template <> struct Pair<float> {
+  static __device__ __forceinline__ float2 load(const float* p) { return *reinterpret_cast<const float2*>(p); }
+  static __device__ __forceinline__ void store(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+};
+template <> struct Pair<__nv_bfloat16> {
+  static __device__ __forceinline__ float2 load(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+};
+
 template <typename T>
-__global__ void __launch_bounds__(128) mla_absorb_kernel(const __grid_constant__ MlaParams p) {
+__global__ void __launch_bounds__(256) mla_absorb_kernel(const __grid_constant__ MlaParams p) {
   pdl_wait();
-  extern __shared__ float sm[];                   // [D][8]
+  extern __shared__ float sm[];                   // q [D][8] | partial sums [3][64][16]
+  float* part = sm + p.D * 8;
   const int h = blockIdx.y, mb = blockIdx.z * 8, rows = min(8, p.M - mb);
-  for (int i = threadIdx.x; i < p.D * 8; i += 128) {
-    const int d = i >> 3, r = i & 7;
-    sm[i] = r < rows ? p.x[static_cast<size_t>(mb + r) * p.ldx + p.q_off + h * (p.D + p.R) + d] : 0.f;
+  for (int i = threadIdx.x; i < p.D * 8; i += 256) {
+    const int r = i / p.D, d = i - r * p.D;
+    sm[d * 8 + r] = r < rows ? p.x[static_cast<size_t>(mb + r) * p.ldx + p.q_off + h * (p.D + p.R) + d] : 0.f;
   }
   __syncthreads();
-  const int c = blockIdx.x * 128 + threadIdx.x;
-  if (c >= p.CP) return;
-  float acc[8] = {};
-  if (c < p.C) {
+  const int cp = threadIdx.x & 63, quarter = threadIdx.x >> 6;
+  const int c = blockIdx.x * 128 + cp * 2;         // CP is even
+  const int per = (p.D + 3) / 4, d0 = quarter * per, d1 = min(p.D, d0 + per);
+  float acc[8][2] = {};
+  if (c < p.CP) {
     const T* w = static_cast<const T*>(p.w_uk) + static_cast<size_t>(h) * p.D * p.CP + c;
-#pragma unroll 4
-    for (int d = 0; d < p.D; ++d) {
-      const float wv = to_f<T>(w[static_cast<size_t>(d) * p.CP]);
+#pragma unroll 8
+    for (int d = d0; d < d1; ++d) {
+      const float2 wv = Pair<T>::load(w + static_cast<size_t>(d) * p.CP);
       const float4 a = *reinterpret_cast<const float4*>(sm + d * 8), b = *reinterpret_cast<const float4*>(sm + d * 8 + 4);
-      acc[0] = fmaf(wv, a.x, acc[0]); acc[1] = fmaf(wv, a.y, acc[1]); acc[2] = fmaf(wv, a.z, acc[2]); acc[3] = fmaf(wv, a.w, acc[3]);
-      acc[4] = fmaf(wv, b.x, acc[4]); acc[5] = fmaf(wv, b.y, acc[5]); acc[6] = fmaf(wv, b.z, acc[6]); acc[7] = fmaf(wv, b.w, acc[7]);
+      const float q[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        acc[r][0] = fmaf(wv.x, q[r], acc[r][0]);
+        acc[r][1] = fmaf(wv.y, q[r], acc[r][1]);
+      }
     }
   }
+  if (quarter > 0) {
+#pragma unroll
+    for (int r = 0; r < 8; ++r) *reinterpret_cast<float2*>(part + ((quarter - 1) * 8 + r) * 128 + cp * 2) = make_float2(acc[r][0], acc[r][1]);
+  }
+  __syncthreads();
+  if (quarter > 0 || c >= p.CP) return;
   const int LD = p.CP + p.RP;
 #pragma unroll
-  for (int r = 0; r < 8; ++r)
-    if (r < rows) static_cast<T*>(p.q_eff)[(static_cast<size_t>(mb + r) * p.H + h) * LD + c] = from_f<T>(acc[r]);
+  for (int r = 0; r < 8; ++r) {
+    if (r >= rows) break;
+#pragma unroll
+    for (int g = 0; g < 3; ++g) {
+      const float2 v = *reinterpret_cast<const float2*>(part + (g * 8 + r) * 128 + cp * 2);
+      acc[r][0] += v.x;
+      acc[r][1] += v.y;
+    }
+    Pair<T>::store(static_cast<T*>(p.q_eff) + (static_cast<size_t>(mb + r) * p.H + h) * LD + c, acc[r][0], acc[r][1]);
+  }
 }
 
 // grid (M, H, splits), 128 threads: one query row of one head over its share of the keys, 64 at a time
@@ -168,47 +204,65 @@ __global__ void __launch_bounds__(128) mla_row_attn_kernel(const __grid_constant
   if (threadIdx.x == 0) { p.ml[row * 2] = mx; p.ml[row * 2 + 1] = l; }
 }
 
-// grid (ceil(M / 8), H, ceil(V / 64)), 256 threads: merges the key splits of eight rows, carries their latents out
-// through W_uv (each weight row is read once for the eight), gates
+// grid (M, H), 128 threads: merges the key splits of a row's head into split 0's place, divided by the sum
+__global__ void __launch_bounds__(128) mla_merge_kernel(const __grid_constant__ MlaParams p) {
+  pdl_wait();
+  __shared__ float wt[64];
+  const int m = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
+  if (mla_seq_of_row(p.cu_rows, p.nseq, m) < 0) return;
+  const size_t row = (static_cast<size_t>(m) * p.H + h) * p.splits;
+  if (threadIdx.x < 32) {
+    const float* ml = p.ml + row * 2;
+    float mx = -INFINITY, l = 0.f;
+    for (int s = lane; s < p.splits; s += 32) mx = fmaxf(mx, ml[s * 2]);
+    mx = mla_warp_max(mx);
+    for (int s = lane; s < p.splits; s += 32) l += ml[s * 2] > -INFINITY ? ml[s * 2 + 1] * expf(ml[s * 2] - mx) : 0.f;
+    l = mla_warp_sum(l);
+    for (int s = lane; s < p.splits; s += 32) wt[s] = ml[s * 2] > -INFINITY ? expf(ml[s * 2] - mx) / l : 0.f;
+  }
+  __syncthreads();
+  float* o = p.o_part + row * p.CP;
+  for (int c = threadIdx.x * 4; c < p.CP; c += 512) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 6
+    for (int s = 0; s < p.splits; ++s) {
+      const float4 a = __ldcg(reinterpret_cast<const float4*>(o + static_cast<size_t>(s) * p.CP + c));
+      const float w = wt[s];
+      v.x = fmaf(a.x, w, v.x); v.y = fmaf(a.y, w, v.y); v.z = fmaf(a.z, w, v.z); v.w = fmaf(a.w, w, v.w);
+    }
+    *reinterpret_cast<float4*>(o + c) = v;         // read by this thread alone
+  }
+}
+
+// grid (ceil(M / 8), H, ceil(V / 16)), 256 threads: the latents of eight rows through W_uv (a weight row is read once
+// for the eight), gated
 template <typename T>
 __global__ void __launch_bounds__(256) mla_out_kernel(const __grid_constant__ MlaParams p) {
   pdl_wait();
-  extern __shared__ float sm[];                   // [8][CP] latents | [8][splits] merge weights
+  extern __shared__ float sm[];                   // [8][CP]
   const int mb = blockIdx.x * 8, h = blockIdx.y, rows = min(8, p.M - mb);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float* wt = sm + 8 * p.CP;
-  if (warp < rows) {                              // a warp per row: merge weights exp(m_s - max) / sum
-    const float* ml = p.ml + (static_cast<size_t>(mb + warp) * p.H + h) * p.splits * 2;
-    const bool live = mla_seq_of_row(p.cu_rows, p.nseq, mb + warp) >= 0;
-    float mx = -INFINITY, l = 0.f;
-    for (int s = lane; s < p.splits; s += 32) mx = fmaxf(mx, live ? ml[s * 2] : -INFINITY);
-    mx = mla_warp_max(mx);
-    for (int s = lane; s < p.splits; s += 32) l += live && ml[s * 2] > -INFINITY ? ml[s * 2 + 1] * expf(ml[s * 2] - mx) : 0.f;
-    l = mla_warp_sum(l);
-    for (int s = lane; s < p.splits; s += 32) wt[warp * p.splits + s] = live && ml[s * 2] > -INFINITY ? expf(ml[s * 2] - mx) / l : 0.f;
-  }
-  __syncthreads();
-  for (int i = threadIdx.x; i < 8 * p.CP; i += 256) {
+  for (int i = threadIdx.x * 4; i < 8 * p.CP; i += 1024) {
     const int r = i / p.CP, c = i - r * p.CP;
-    float v = 0.f;
-    if (r < rows) {
-      const float* o = p.o_part + (static_cast<size_t>(mb + r) * p.H + h) * p.splits * p.CP + c;
-      for (int s = 0; s < p.splits; ++s) {
-        const float w = wt[r * p.splits + s];
-        if (w != 0.f) v = fmaf(o[static_cast<size_t>(s) * p.CP], w, v);     // (a split without keys, or a padding row, was not written)
-      }
-    }
-    sm[i] = v;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (r < rows && mla_seq_of_row(p.cu_rows, p.nseq, mb + r) >= 0)
+      v = *reinterpret_cast<const float4*>(p.o_part + (static_cast<size_t>(mb + r) * p.H + h) * p.splits * p.CP + c);
+    *reinterpret_cast<float4*>(sm + i) = v;
   }
   __syncthreads();
-  const int v1 = min(p.V, static_cast<int>(blockIdx.z) * 64 + 64);
-  for (int v = blockIdx.z * 64 + warp; v < v1; v += 8) {
+  const int v1 = min(p.V, static_cast<int>(blockIdx.z) * 16 + 16);
+  for (int v = blockIdx.z * 16 + warp; v < v1; v += 8) {
     const T* w = static_cast<const T*>(p.w_uv) + (static_cast<size_t>(h) * p.V + v) * p.CP;
     float s[8] = {};
-    for (int c = lane; c < p.C; c += 32) {
-      const float wv = to_f<T>(w[c]);
+#pragma unroll 8
+    for (int c = lane * 2; c < p.CP; c += 64) {
+      const float2 wv = Pair<T>::load(w + c);
 #pragma unroll
-      for (int r = 0; r < 8; ++r) s[r] = fmaf(wv, sm[r * p.CP + c], s[r]);
+      for (int r = 0; r < 8; ++r) {
+        const float2 o = *reinterpret_cast<const float2*>(sm + r * p.CP + c);
+        s[r] = fmaf(wv.x, o.x, s[r]);
+        s[r] = fmaf(wv.y, o.y, s[r]);
+      }
     }
 #pragma unroll
     for (int r = 0; r < 8; ++r) s[r] = mla_warp_sum(s[r]);
@@ -224,10 +278,10 @@ __global__ void __launch_bounds__(256) mla_out_kernel(const __grid_constant__ Ml
 
 template <typename T>
 static int mla_go(const MlaParams& p, cudaStream_t stream) {
-  cudaError_t e = launch(mla_prep_kernel<T>, dim3(p.M), dim3(256), 0, stream, 0, p);
+  cudaError_t e = launch(mla_prep_kernel<T>, dim3(p.M), dim3(256), p.R * 4 + 16, stream, 0, p);
   if (e != cudaSuccess) return static_cast<int>(e);
   if (p.expand) return saber_mla_expand_attn(&p, stream);
-  e = launch(mla_absorb_kernel<T>, dim3((p.CP + 127) / 128, p.H, (p.M + 7) / 8), dim3(128), p.D * 32, stream, 0, p);
+  e = launch(mla_absorb_kernel<T>, dim3((p.CP + 127) / 128, p.H, (p.M + 7) / 8), dim3(256), (p.D * 8 + 3 * 8 * 128) * 4, stream, 0, p);
   if (e != cudaSuccess) return static_cast<int>(e);
   if (saber_mla_decode_ok(&p)) {
     const int r = saber_mla_decode_attn(&p, stream);
@@ -236,12 +290,14 @@ static int mla_go(const MlaParams& p, cudaStream_t stream) {
     e = launch(mla_row_attn_kernel<T>, dim3(p.M, p.H, p.splits), dim3(128), (p.CP + p.RP + kRowKeys) * 4, stream, 0, p);
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  return static_cast<int>(launch(mla_out_kernel<T>, dim3((p.M + 7) / 8, p.H, (p.V + 63) / 64), dim3(256), 8 * (p.CP + p.splits) * 4, stream, 0, p));
+  e = launch(mla_merge_kernel, dim3(p.M, p.H), dim3(128), 0, stream, 0, p);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  return static_cast<int>(launch(mla_out_kernel<T>, dim3((p.M + 7) / 8, p.H, (p.V + 15) / 16), dim3(256), 8 * p.CP * 4, stream, 0, p));
 }
 
 }  // namespace saber
 
-extern "C" int saber_mla_launches(const saber::MlaParams* p) { return p->expand ? 3 : 4; }
+extern "C" int saber_mla_launches(const saber::MlaParams* p) { return p->expand ? 3 : 5; }
 
 extern "C" int saber_mla_launch(const saber::MlaParams* p, cudaStream_t stream) {
   using namespace saber;

@@ -31,8 +31,8 @@ __global__ void __launch_bounds__(256) mla_decode_kernel(const __grid_constant__
   const uint32_t q_s = smem_u32(smem);
   const uint32_t k_s = q_s + MT * 16 * rs;                          // two tiles of 64 rows
   const uint32_t p_s = k_s + 2 * kKeys * rs;                        // probabilities, bf16 [MT * 16][64 + 8]
-  float* s_f = reinterpret_cast<float*>(smem + (MT * 16 + 2 * kKeys) * rs + MT * 16 * 144);   // scores [MT * 16][64 + 4]
-  float* corr_s = s_f + MT * 16 * 68;                               // [MT * 16]
+  float* s_f = reinterpret_cast<float*>(smem + (MT * 16 + 2 * kKeys) * rs + MT * 16 * 144);   // partial scores [2][MT * 16][64 + 4]
+  float* corr_s = s_f + 2 * MT * 16 * 68;                           // [MT * 16]
   const int keys = p.pos[m] + 1;
   const int per = ((keys + p.splits - 1) / p.splits + kKeys - 1) / kKeys * kKeys;
   const int k0 = sp * per, k1 = min(keys, k0 + per);
@@ -75,40 +75,36 @@ __global__ void __launch_bounds__(256) mla_decode_kernel(const __grid_constant__
     }
     __syncthreads();
     const uint32_t kt = k_s + buf * kKeys * rs;
-    // scores of this warp's eight keys for every head tile
+    // scores of 16 keys (warp & 3) over one half of the score dimension (warp >> 2) for every head tile
     {
-      float s[MT][4] = {};
+      float s[MT][2][4] = {};
+      const int steps = LD / 16, half0 = (steps + 1) / 2;
+      const int s0 = warp < 4 ? 0 : half0, s1 = warp < 4 ? half0 : steps;
+      const int kg = (warp & 3) * 16;
       const uint32_t a_row = q_s + (lane & 15) * rs + ((lane >> 4) << 4);
-      const uint32_t b_row = kt + (warp * 8 + (lane & 7)) * rs + ((lane >> 3) << 4);
-      int kk = 0;
-      for (; kk + 32 <= LD; kk += 32) {
+      const uint32_t b_row = kt + (kg + ((lane >> 4) << 3) + (lane & 7)) * rs + (((lane >> 3) & 1) << 4);
+#pragma unroll 4
+      for (int st = s0; st < s1; ++st) {
         uint32_t b[4];
-        ldsm4(b, b_row + kk * 2);
+        ldsm4(b, b_row + st * 32);
 #pragma unroll
         for (int t = 0; t < MT; ++t) {
           uint32_t a[4];
-          ldsm4(a, a_row + t * 16 * rs + kk * 2);
-          mma16816(s[t], a, b[0], b[1]);
-          ldsm4(a, a_row + t * 16 * rs + kk * 2 + 32);
-          mma16816(s[t], a, b[2], b[3]);
+          ldsm4(a, a_row + t * 16 * rs + st * 32);
+          mma16816(s[t][0], a, b[0], b[1]);
+          mma16816(s[t][1], a, b[2], b[3]);
         }
       }
-      if (kk < LD) {                                                // one 16-wide step left (its b[2], b[3] are row padding)
-        uint32_t b[4];
-        ldsm4(b, kt + (warp * 8 + (lane & 7)) * rs + (((lane >> 3) & 1) << 4) + kk * 2);
+      float* dst = s_f + (warp >> 2) * MT * 16 * 68;
+      const int r = lane >> 2;
 #pragma unroll
-        for (int t = 0; t < MT; ++t) {
-          uint32_t a[4];
-          ldsm4(a, a_row + t * 16 * rs + kk * 2);
-          mma16816(s[t], a, b[0], b[1]);
+      for (int t = 0; t < MT; ++t)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int c = kg + i * 8 + (lane & 3) * 2;
+          *reinterpret_cast<float2*>(dst + (t * 16 + r) * 68 + c) = make_float2(s[t][i][0], s[t][i][1]);
+          *reinterpret_cast<float2*>(dst + (t * 16 + r + 8) * 68 + c) = make_float2(s[t][i][2], s[t][i][3]);
         }
-      }
-      const int c = warp * 8 + (lane & 3) * 2, r = lane >> 2;
-#pragma unroll
-      for (int t = 0; t < MT; ++t) {
-        *reinterpret_cast<float2*>(s_f + (t * 16 + r) * 68 + c) = make_float2(s[t][0], s[t][1]);
-        *reinterpret_cast<float2*>(s_f + (t * 16 + r + 8) * 68 + c) = make_float2(s[t][2], s[t][3]);
-      }
     }
     __syncthreads();
     // running softmax: warp w owns rows w, w + 8, ...
@@ -116,7 +112,10 @@ __global__ void __launch_bounds__(256) mla_decode_kernel(const __grid_constant__
 #pragma unroll
     for (int i = 0; i < 2 * MT; ++i) {
       const int r = warp + 8 * i;
-      const float2 v = *reinterpret_cast<const float2*>(s_f + r * 68 + lane * 2);
+      float2 v = *reinterpret_cast<const float2*>(s_f + r * 68 + lane * 2);
+      const float2 v2 = *reinterpret_cast<const float2*>(s_f + (MT * 16 + r) * 68 + lane * 2);
+      v.x += v2.x;
+      v.y += v2.y;
       const float a = lane * 2 < n ? v.x * p.scale : -INFINITY, b = lane * 2 + 1 < n ? v.y * p.scale : -INFINITY;
       const float mn = fmaxf(mx[i], mla_warp_max(fmaxf(a, b)));
       const float ea = exp2f((a - mn) * kLog2e), eb = exp2f((b - mn) * kLog2e);
@@ -180,10 +179,13 @@ __global__ void __launch_bounds__(256) mla_decode_kernel(const __grid_constant__
   }
 }
 
-static int decode_tiles(const MlaParams& p) { return p.H <= 16 ? 1 : (p.H <= 32 || p.H > 48 ? 2 : 3); }
 static int decode_smem(const MlaParams& p, int mt) {
   const int rs = (p.CP + p.RP) * 2 + 16;
-  return (mt * 16 + 2 * kKeys) * rs + mt * 16 * (144 + 68 * 4 + 4);
+  return (mt * 16 + 2 * kKeys) * rs + mt * 16 * (144 + 2 * 68 * 4 + 4);
+}
+static int decode_tiles(const MlaParams& p) {
+  const int mt = p.H <= 16 ? 1 : (p.H <= 32 || p.H > 48 ? 2 : 3);
+  return mt == 3 && decode_smem(p, 3) > 226 * 1024 ? 2 : mt;
 }
 template <int MT, int NC>
 static int decode_go(const MlaParams& p, cudaStream_t stream) {

@@ -1,0 +1,217 @@
+"""Throughput of a layer-by-layer model beside the int4 hybrid decoder at equal layer sizes.
+
+Prefill: a cold prompt in portions of one rung (device-timed).  Decode: `streams` sequences at the prompt's length,
+one row each (no drafter on either side).  Then every group of launches of one step on its own: the group's
+launches between two events after an L2 flush (a write of 256 MB), the median over repetitions, and the fraction
+of its roofline: the slower of algorithmic bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate.
+"""
+from __future__ import annotations
+
+import json
+import os
+import statistics
+
+import torch
+
+from ..models import config as C
+from ..models.hybrid import HybridModel
+from ..models.stack import StackModel
+from ..models.stack_config import DeltaMixer, LatentMixer, StackConfig
+from ..models.step import SeqStep, run_bucket
+
+SIZES = ("renosun-2k", "renosun-4k", "renosun-5k")
+
+
+def peaks() -> tuple:
+    path = os.path.join(os.path.dirname(os.path.abspath(__file__)), "..", "..", "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        d = json.load(open(path))
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12
+    return 6.65e12, 1.59e15
+
+
+def like_hybrid(cfg: StackConfig) -> C.HybridConfig:
+    """The hybrid decoder with the same width, feed-forward, delta heads and number of layer runs; its gated GQA
+    attention has the same query width in heads of 256 and a quarter as many key heads."""
+    d = next(l.mixer for l in cfg.layers if isinstance(l.mixer, DeltaMixer))
+    a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, LatentMixer))
+    nq = max(4, a.heads * a.dim // 256)
+    return C.HybridConfig(name=f"hybrid-like-{cfg.name}", n_layers=len(cfg.runs), hidden=cfg.width, n_q_heads=nq, n_kv_heads=max(1, nq // 4),
+                          head_dim=256, ffn_inter=cfg.layers[0].mlp.ff, vocab=cfg.vocab, gdn_k_heads=d.kv_heads, gdn_v_heads=d.heads,
+                          gdn_head_dim=128, max_ctx=cfg.max_ctx)
+
+
+def _groups(model, b) -> dict:
+    """Launch ranges of one layer run per group, by tag."""
+    tags = b.program.tags()
+    out = {}
+    if isinstance(model, StackModel):
+        for g in ("project", "delta", "latent_attention", "out", "loop_in"):
+            idx = [i for i, t in enumerate(tags) if t.endswith("." + g)]
+            if idx:
+                out[g] = [(i, i + 1) for i in idx]
+        out["lm_head"] = [(i, i + 1) for i, t in enumerate(tags) if t == "lm_head"]
+        return out
+    layers = sorted({int(t[1:].split(".")[0]) for t in tags if t[0] == "L" and t[1].isdigit()})
+    span = lambda li, keys: [i for i, t in enumerate(tags) if t.startswith(f"L{li}.") and any(k in t for k in keys)]   # noqa: E731
+    spec = {"delta": ("gdn.conv", "gdn.rec", "gdn.norm", "gdn.step"), "attention": ("attn.rope", "attn.core", "attn.gate", "attn.quant"),
+            "linears": ("in_norm", "in_proj", "attn.qkv", "out_proj", "o_proj", "post_norm", "mlp")}
+    for g, keys in spec.items():
+        out[g] = []
+        for li in layers:
+            idx = span(li, keys)
+            runs = []
+            for i in idx:
+                if runs and runs[-1][1] == i:
+                    runs[-1][1] = i + 1
+                else:
+                    runs.append([i, i + 1])
+            if runs:
+                out[g].append([tuple(r) for r in runs])
+    out["linears"] = [r for r in out["linears"] if r]
+    return out
+
+
+def _time(model, b, ranges, flush, reps: int = 7) -> float:
+    """Median microseconds of the launches in `ranges`."""
+    st, res = model.stream, []
+    with torch.cuda.stream(st):
+        for k in range(reps + 2):
+            flush.zero_()
+            tot = []
+            for lo, hi in ranges:
+                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                e0.record(st)
+                b.program.run(st, lo, hi)
+                e1.record(st)
+                tot.append((e0, e1))
+            st.synchronize()
+            if k >= 2:
+                res.append(sum(a.elapsed_time(c) for a, c in tot) * 1e3)
+    return statistics.median(res)
+
+
+def _roof(nbytes: float, flops: float) -> float:
+    hbm, mm = peaks()
+    return max(nbytes / hbm, flops / mm) * 1e6
+
+
+def stack_costs(cfg: StackConfig, M: int, nseq: int, ctx_pairs: float, ctx_tokens: float) -> dict:
+    """Algorithmic (bytes, FLOPs) per launch of each group.  ctx_pairs: visible (row, key) pairs; ctx_tokens: keys read."""
+    W, out = cfg.width, {}
+    d = next(l for l in cfg.layers if isinstance(l.mixer, DeltaMixer))
+    a = next(l for l in cfg.layers if isinstance(l.mixer, LatentMixer))
+    segs = sum(n for _, n in d.mixer.segments())
+    n = segs + 2 * d.mlp.ff
+    out["project"] = (2 * n * W + M * (2 * W + 4 * segs + 2 * d.mlp.ff), 2.0 * M * n * W)
+    k = d.mixer.out_features + d.mlp.ff
+    out["out"] = (2 * k * W + M * (2 * k + 8 * W + 2 * W), 2.0 * M * k * W)
+    out["loop_in"] = (4 * W * W + M * (4 * W + 6 * W), 4.0 * M * W * W)
+    m = d.mixer
+    out["delta"] = (2 * 4 * nseq * m.heads * m.dim * m.vdim + M * (4 * (segs + m.out_features) + 2 * m.out_features),
+                    M * m.heads * m.dim * m.vdim * 8.0)
+    m = a.mixer
+    pair = 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim)
+    carry = 2.0 * ctx_tokens * m.heads * (m.dim + m.vdim) * m.kv_rank if M > 64 else 2.0 * M * m.heads * (m.dim + m.vdim) * m.kv_rank
+    if M <= 64:
+        pair = 2.0 * m.heads * (2 * m.kv_rank + m.rot_dim)
+    out["latent_attention"] = (2 * ctx_tokens * (m.kv_rank + m.rot_dim) + 2 * m.heads * (m.dim + m.vdim) * m.kv_rank
+                               + M * (4 * m.heads * (m.dim + m.rot_dim + m.vdim) + 2 * m.heads * m.vdim), ctx_pairs * pair + carry)
+    out["lm_head"] = (2 * cfg.vocab * W, 2.0 * min(M, 8) * cfg.vocab * W)
+    return out
+
+
+def hybrid_costs(cfg: C.HybridConfig, M: int, nseq: int, ctx_pairs: float, ctx_tokens: float) -> dict:
+    sh = C.shard(cfg, 1, 0)
+    H, D = cfg.hidden, 128
+    lin = H * (sh.gdn_in_n + 2 * sh.ffn_inter) + H * (sh.gdn_out_k + sh.ffn_inter)
+    out = {"linears": (0.5 * lin + M * (2 * sh.gdn_in_n + sh.gdn_out_k + sh.ffn_inter + 12 * H), 2.0 * M * lin)}
+    out["delta"] = (2 * 4 * nseq * sh.gdn_v_heads * D * D + M * (2 * sh.gdn_in_n + sh.gdn_out_k), M * sh.gdn_v_heads * D * D * 8.0)
+    out["attention"] = (2 * ctx_tokens * sh.n_kv_heads * cfg.head_dim + M * (2 * sh.qkv_n + sh.o_k), ctx_pairs * 4.0 * sh.n_q_heads * cfg.head_dim)
+    return out
+
+
+def measure(cfg, prompt: int, streams: int, rung: int, steps: int, warmup: int, detail: bool) -> dict:
+    stack = isinstance(cfg, StackConfig)
+    ctx = prompt + 64 * ((steps + warmup) // 64 + 4)
+    if stack:
+        model = StackModel(cfg, max_seqs=streams, max_ctx=ctx, seed=5)
+    else:
+        model = HybridModel(cfg, max_seqs=streams, max_ctx=ctx, max_width=1, seed=5, use_drafter=False)
+    page = cfg.page_tokens
+    per = (ctx + page - 1) // page
+    g = torch.Generator().manual_seed(3)
+    toks = torch.randint(0, cfg.vocab, (streams, prompt), generator=g).tolist()
+    blocks = [list(range(1 + j * per, 1 + (j + 1) * per)) for j in range(streams)]
+    pb = model.build_bucket("prefill", 1, rung)
+    ms, last = [], [0] * streams
+    for j in range(streams):
+        model.reset_slot(j + 1)
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(model.stream)
+        for pos in range(0, prompt, rung):
+            r = run_bucket(model, pb, [SeqStep(toks[j][pos:pos + rung], pos, j + 1, 0, blocks[j])])
+        e1.record(model.stream)
+        torch.cuda.synchronize()
+        last[j] = r.tokens[0][0]
+        ms.append(e0.elapsed_time(e1))
+    model.scratch.check()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    res = {"prefill_ms": statistics.median(ms), "prefill_tok_s": prompt / statistics.median(ms) * 1e3, "prefill_launches": pb.n_launches}
+    if detail:      # the last portion again, group by group (the tables of that step are still on the device)
+        lo = prompt - rung
+        costs = (stack_costs if stack else hybrid_costs)(cfg, rung, 1, rung * lo + rung * (rung + 1) / 2.0, prompt)
+        res["prefill_groups"] = _detail(model, pb, costs, flush)
+    db = model.build_bucket("decode", streams, 1)
+    pos = prompt
+
+    def step():
+        nonlocal pos, last
+        r = run_bucket(model, db, [SeqStep([last[j]], pos, j + 1, 1 if (pos > prompt and not stack) else 0, blocks[j], uid=j, step_no=pos,
+                                           blocks_key=("b", j)) for j in range(streams)])
+        last = [t[0] for t in r.tokens]
+        pos += 1
+    for _ in range(warmup):
+        step()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record(model.stream)
+    for _ in range(steps):
+        step()
+    e1.record(model.stream)
+    torch.cuda.synchronize()
+    model.scratch.check()
+    t = e0.elapsed_time(e1) / steps
+    res.update(decode_ms_per_step=t, decode_tok_s=streams / t * 1e3, decode_launches=db.n_launches)
+    if detail:
+        costs = (stack_costs if stack else hybrid_costs)(cfg, streams, streams, streams * pos, streams * pos)
+        res["decode_groups"] = _detail(model, db, costs, flush)
+    res["state_bytes"] = model.state_bytes()
+    return res
+
+
+def _detail(model, b, costs: dict, flush) -> dict:
+    out = {}
+    for g, ranges in _groups(model, b).items():
+        if not ranges:
+            continue
+        one = ranges[len(ranges) // 2]
+        us = _time(model, b, one if isinstance(one, list) else [one], flush)
+        nb, fl = costs.get(g, (0, 0))
+        roof = _roof(nb, fl)
+        out[g] = {"us": round(us, 1), "roofline_us": round(roof, 1), "of_roofline": round(roof / us, 3), "per_step": len(ranges)}
+    return out
+
+
+def run(args) -> dict:
+    names = SIZES if args.stack == "all" else tuple(args.stack.split(","))
+    out = {"metric": "layer_stack_prefill_decode_tok_s", "n_gpus": 1, "data": "synthetic", "dtype": "bf16", "steps": args.steps,
+           "config": {"prompt": args.prompt, "streams": args.streams, "rung": args.rung, "l2": "flushed between group timings; weights of a step exceed L2"},
+           "models": {}}
+    for n in names:
+        cfg = C.by_name(n)
+        for c in (cfg, like_hybrid(cfg)):
+            out["models"][c.name] = measure(c, args.prompt, args.streams, args.rung, args.steps, args.warmup, True)
+            torch.cuda.empty_cache()
+    return out

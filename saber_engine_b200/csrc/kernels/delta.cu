@@ -2,8 +2,8 @@
 //
 // Prompt portions (ragged rows, any length), in blocks of four tokens: three launches.
 //   prep   convolution, silu, unit norms, beta and decay, and per block the dot products k_j . k_i and k_j . q_i
-//   scan   the recurrence.  Columns of the state are independent, so a warp owns eight value columns for the
-//          whole portion: eight lanes split the key dimension, four lane groups take two columns each, the state
+//   scan   the recurrence.  Columns of the state are independent, so a warp owns four value columns for the
+//          whole portion: sixteen lanes split the key dimension, two lane groups take two columns each, the state
 //          stays in registers.  A block of four tokens needs the products of its keys and queries with the state
 //          at its start only, S_0^T k_i and S_0^T q_i (independent of one another, one shuffle reduction for
 //          all); the rest is a triangular recurrence in scalars.  With G_i = g_1 .. g_i and
@@ -12,7 +12,7 @@
 //              o_i = G_i S_0^T q_i + sum_{j<=i} D_ij (k_j . q_i) u_j
 //              S_4 = G_4 S_0 + sum_j D_4j k_j u_j^T
 //          which is the token-by-token rule written out; a block with fewer tokens is filled up with
-//          k = q = v = beta = 0, g = 1.  Blocks are staged in shared memory by asynchronous copies.
+//          k = q = v = beta = 0, g = 1.  Blocks arrive in shared memory by bulk copies, four in flight.
 //   out    gated norm into the operand of the output linear; the convolution inputs go to the ring
 // Decoding (one row per sequence): all of it in one launch, a CTA per (head, sequence).
 #include "delta.h"
@@ -29,10 +29,6 @@ __device__ __forceinline__ float warp_sum_f(float v) {
 __device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f32(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
-
-__device__ __forceinline__ void cp_async16(float* dst, const float* src, int bytes) {    // bytes 0: zero fill
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
-}
 
 // sequence of a row (-1: a padding row), and whether its slot may be used
 __device__ __forceinline__ int seq_of_row(const int32_t* cu, int nseq, int m) {
@@ -78,33 +74,61 @@ __device__ __forceinline__ bool block_of_slot(const DeltaParams& p, int slot, in
   return false;
 }
 
-// convolution + silu of channel c for the rows of a block (m: its first row, t: that row inside its sequence)
+// convolution + silu of channel c for the rows of a block (m: its first row, t: that row inside its sequence).
+// TAPS: the number of taps when known at compile time (every input and weight is then loaded at once), else 0.
+template <int TAPS>
 __device__ __forceinline__ void conv_silu4(const DeltaParams& p, const float* hist, int c, int col, int m, int t, int pos, int C, int rows,
                                            float (&y)[kBlk]) {
   float acc[kBlk] = {};
-  for (int back = p.taps - 1; back > -kBlk; --back) {              // input row m - back feeds rows r >= -back
-    if (-back >= rows) break;
-    float x = 0.f;
-    if (back <= t) x = p.x[static_cast<size_t>(m - back) * p.ldx + col];
-    else if (back <= pos) x = hist[static_cast<size_t>((pos - back) % p.taps) * C + c];
+  const float* cw = p.conv_w + static_cast<size_t>(c) * p.taps;
+  if constexpr (TAPS > 0) {
+    float x[TAPS + kBlk - 1], w[TAPS];
 #pragma unroll
-    for (int r = 0; r < kBlk; ++r) {
-      const int i = p.taps - 1 - (r + back);                        // tap of this input for row r
-      if (i >= 0 && i < p.taps) acc[r] = fmaf(x, p.conv_w[static_cast<size_t>(c) * p.taps + i], acc[r]);
+    for (int i = 0; i < TAPS; ++i) w[i] = cw[i];
+#pragma unroll
+    for (int i = 0; i < TAPS + kBlk - 1; ++i) {                     // input row m - (TAPS - 1) + i
+      const int back = TAPS - 1 - i;
+      x[i] = 0.f;
+      if (-back < rows) {
+        if (back <= t) x[i] = p.x[static_cast<size_t>(m - back) * p.ldx + col];
+        else if (back <= pos) x[i] = hist[static_cast<size_t>((pos - back) % TAPS) * C + c];
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < kBlk; ++r)
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) acc[r] = fmaf(x[r + i], w[i], acc[r]);
+  } else {
+    for (int back = p.taps - 1; back > -kBlk; --back) {             // input row m - back feeds rows r >= -back
+      if (-back >= rows) break;
+      float x = 0.f;
+      if (back <= t) x = p.x[static_cast<size_t>(m - back) * p.ldx + col];
+      else if (back <= pos) x = hist[static_cast<size_t>((pos - back) % p.taps) * C + c];
+#pragma unroll
+      for (int r = 0; r < kBlk; ++r) {
+        const int i = p.taps - 1 - (r + back);                      // tap of this input for row r
+        if (i >= 0 && i < p.taps) acc[r] = fmaf(x, cw[i], acc[r]);
+      }
     }
   }
 #pragma unroll
   for (int r = 0; r < kBlk; ++r) y[r] = r < rows ? silu_f32(acc[r]) : 0.f;
 }
 
-// grid (blocks, ceil(items / 4)), 128 threads; a warp per item: key heads (q, k and their dot products), value heads,
-// then one item for beta / decay
-template <int NI>
+// Scratch records of a block, each contiguous (one bulk copy):
+//   key head   k rows [4][DP] | q rows [4][DP] | 16 dot products
+//   value head, per 32 columns   v [4][32] | beta [4] | g [4]
+// Missing tokens of the last block are written as k = q = v = beta = 0, g = 1.
+__host__ __device__ constexpr int kq_words(int DP) { return 2 * kBlk * DP + kPairs; }
+constexpr int kVWords = kBlk * 32 + 2 * kBlk;
+
+// grid (blocks, ceil((HK + H) / 4)), 128 threads; a warp per item: key heads (q, k and their dot products), value heads
+template <int NI, int TAPS>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const __grid_constant__ DeltaParams p) {
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int item = blockIdx.y * 4 + (threadIdx.x >> 5);
-  if (item > p.HK + p.H) return;
+  if (item >= p.HK + p.H) return;
   int j, blk;
   if (!block_of_slot(p, blockIdx.x, j, blk)) return;
   const int slot = delta_slot(p, j);
@@ -122,8 +146,8 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const __grid_constant__
 #pragma unroll
       for (int r = 0; r < kBlk; ++r) qv[i][r] = kv[i][r] = 0.f;
       if (d < p.D) {
-        conv_silu4(p, hist, h * p.D + d, p.q_off + h * p.D + d, m, t, pos, C, rows, qv[i]);
-        conv_silu4(p, hist, (p.HK + h) * p.D + d, p.k_off + h * p.D + d, m, t, pos, C, rows, kv[i]);
+        conv_silu4<TAPS>(p, hist, h * p.D + d, p.q_off + h * p.D + d, m, t, pos, C, rows, qv[i]);
+        conv_silu4<TAPS>(p, hist, (p.HK + h) * p.D + d, p.k_off + h * p.D + d, m, t, pos, C, rows, kv[i]);
       }
 #pragma unroll
       for (int r = 0; r < kBlk; ++r) {
@@ -131,6 +155,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const __grid_constant__
         sq[1][r] += kv[i][r] * kv[i][r];
       }
     }
+    float* o = p.kq + (static_cast<size_t>(blockIdx.x) * p.HK + h) * kq_words(DP);
 #pragma unroll
     for (int r = 0; r < kBlk; ++r) {
       const float a = 1.f / sqrtf(warp_sum_f(sq[0][r]) + p.unit_eps) * p.q_scale;
@@ -139,14 +164,11 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const __grid_constant__
       for (int i = 0; i < NI; ++i) {
         qv[i][r] *= a;
         kv[i][r] *= b;
-        if (r < rows) {
-          const size_t o = (static_cast<size_t>(m + r) * p.HK + h) * DP + i * 32 + lane;
-          p.qn[o] = qv[i][r];
-          p.kn[o] = kv[i][r];
-        }
+        o[r * DP + i * 32 + lane] = kv[i][r];
+        o[(kBlk + r) * DP + i * 32 + lane] = qv[i][r];
       }
     }
-    float* pr = p.pairs + (static_cast<size_t>(blockIdx.x) * p.HK + h) * kPairs;
+    float mine = 0.f;                              // lane n keeps dot product n
 #pragma unroll
     for (int i = 0; i < kBlk; ++i)
 #pragma unroll
@@ -158,28 +180,32 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const __grid_constant__
           kq = fmaf(kv[n][jj], qv[n][i], kq);
         }
         kq = warp_sum_f(kq);
-        if (jj < i) kk = warp_sum_f(kk);
-        if (lane == 0) {
-          pr[kq_at(i, jj)] = kq;
-          if (jj < i) pr[kk_at(i, jj)] = kk;
+        if (lane == kq_at(i, jj)) mine = kq;
+        if (jj < i) {
+          kk = warp_sum_f(kk);
+          if (lane == kk_at(i, jj)) mine = kk;
         }
       }
-  } else if (item < p.HK + p.H) {
-    const int h = item - p.HK;
-    for (int d = lane; d < p.VP; d += 32) {
-      float y[kBlk] = {};
-      if (d < p.V) conv_silu4(p, hist, 2 * p.HK * p.D + h * p.V + d, p.v_off + h * p.V + d, m, t, pos, C, rows, y);
-#pragma unroll
-      for (int r = 0; r < kBlk; ++r)
-        if (r < rows) p.vv[(static_cast<size_t>(m + r) * p.H + h) * p.VP + d] = y[r];
-    }
+    if (lane < kPairs) o[2 * kBlk * DP + lane] = mine;
   } else {
-    for (int i = lane; i < p.H * rows; i += 32) {
-      const int r = i / p.H, h = i - r * p.H;
-      const float* x = p.x + static_cast<size_t>(m + r) * p.ldx;
-      float* o = p.bg + (static_cast<size_t>(m + r) * p.H + h) * 2;
-      o[0] = sigmoid_f32(x[p.b_off + h]);
-      o[1] = expf(-expf(p.A_log[h]) * softplus_f32(x[p.a_off + h] + p.dt_bias[h]));
+    const int h = item - p.HK, groups = (p.VP + 31) / 32;
+    float beta = 0.f, g = 1.f;                     // lanes 0 .. 3: one token each
+    if (lane < rows) {
+      const float* x = p.x + static_cast<size_t>(m + lane) * p.ldx;
+      beta = sigmoid_f32(x[p.b_off + h]);
+      g = expf(-expf(p.A_log[h]) * softplus_f32(x[p.a_off + h] + p.dt_bias[h]));
+    }
+    for (int gr = 0; gr < groups; ++gr) {
+      const int d = gr * 32 + lane;
+      float y[kBlk] = {};
+      if (d < p.V) conv_silu4<TAPS>(p, hist, 2 * p.HK * p.D + h * p.V + d, p.v_off + h * p.V + d, m, t, pos, C, rows, y);
+      float* o = p.vb + ((static_cast<size_t>(blockIdx.x) * p.H + h) * groups + gr) * kVWords;
+#pragma unroll
+      for (int r = 0; r < kBlk; ++r) o[r * 32 + lane] = y[r];
+      if (lane < kBlk) {
+        o[kBlk * 32 + lane] = beta;
+        o[kBlk * 32 + kBlk + lane] = g;
+      }
     }
   }
 }
@@ -243,185 +269,172 @@ __device__ __forceinline__ void delta_state_io(float* st, float (&S)[NI][4][2], 
     }
 }
 
-constexpr int kStage = 2;                // blocks per staged buffer
+constexpr int kScanStages = 4;           // blocks of four tokens in flight
 
-// grid (nseq, H, ceil(VP / 32)), 128 threads
-template <int NI>
-__global__ void __launch_bounds__(128) delta_scan_kernel(const __grid_constant__ DeltaParams p) {
-  pdl_wait();
+// grid (nseq, H, ceil(VP / 32)), 256 threads: a warp per four value columns (two lane groups of two), 16 lanes along the keys
+template <int NJ>
+__global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__ DeltaParams p) {
+  constexpr int DP = NJ * 64;
+  constexpr int kKq = kq_words(DP);
+  constexpr int kStageWords = kKq + kVWords;
   extern __shared__ float4 sm4[];
   float* sm = reinterpret_cast<float*>(sm4);
-  constexpr int DP = NI * 32;
-  constexpr int kRow = 2 * DP + 32 + 4;            // k | q | 32 value columns | beta, g
-  constexpr int kBlock = kBlk * kRow + kPairs;     // four rows, then the dot products
+  __shared__ uint64_t bars[kScanStages];
+  pdl_wait();
   const int j = blockIdx.x, h = blockIdx.y;
   const int r0 = p.cu_rows[j], n = p.cu_rows[j + 1] - r0;
   if (n <= 0) return;
   const int slot = delta_slot(p, j);
   if (slot < 0) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 7;
-  const int vb = blockIdx.z * 32, nv = min(32, p.VP - vb);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
+  const int vb = blockIdx.z * 32, groups = (p.VP + 31) / 32;
   const int hk = h / (p.H / p.HK);
-  const int cl = warp * 8 + (lane >> 3) * 2;       // column inside the CTA's 32
-  const bool on = warp * 8 < nv;                   // VP is a multiple of 8
-  float S[NI][4][2] = {};
-  float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + vb + cl) * DP;
-  if (on) delta_state_io<NI>(st, S, DP, lg, false);
+  const int cl = warp * 4 + (lane >> 4) * 2;       // column inside the CTA's 32
+  const bool on = vb + warp * 4 < p.VP;            // VP is a multiple of 8
   const int blocks = (n + kBlk - 1) / kBlk;
-
-  auto fetch = [&](int c) {                        // blocks [c * kStage, ...) into buffer c & 1
-    for (int bi = 0; bi < kStage; ++bi) {
-      const int blk = c * kStage + bi;
-      if (blk >= blocks) break;
-      float* b = sm + ((c & 1) * kStage + bi) * kBlock;
-      const int rows = min(kBlk, n - blk * kBlk);
-      for (int i = threadIdx.x; i < kBlk * (kRow / 4) + kPairs / 4; i += 128) {
-        const int r = i / (kRow / 4), w = i - r * (kRow / 4);
-        if (r == kBlk) {
-          cp_async16(b + kBlk * kRow + w * 4, p.pairs + (static_cast<size_t>(block_slot(r0, j, blk)) * p.HK + hk) * kPairs + w * 4, 16);
-          continue;
-        }
-        const bool live = r < rows;
-        const size_t m = r0 + blk * kBlk + (live ? r : 0);
-        const float* src;
-        int bytes = 16;
-        if (w < DP / 4) src = p.kn + (m * p.HK + hk) * DP + w * 4;
-        else if (w < DP / 2) src = p.qn + (m * p.HK + hk) * DP + (w - DP / 4) * 4;
-        else if (w < DP / 2 + 8) {
-          const int v = (w - DP / 2) * 4;
-          if (v >= nv) continue;
-          src = p.vv + (m * p.H + h) * p.VP + vb + v;
-        } else {
-          // beta, g: eight bytes (a missing token: zeros here, its g is taken as 1 below)
-          src = p.bg + (m * p.H + h) * 2;
-          asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(smem_u32(b + r * kRow + w * 4)), "l"(src), "r"(live ? 8u : 0u)
-                       : "memory");
-          continue;
-        }
-        cp_async16(b + r * kRow + w * 4, src, live ? bytes : 0);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+  const uint32_t bar = smem_u32(bars);
+  const uint32_t sm_u = smem_u32(sm);
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kScanStages; ++i) mbar_init(bar + 8 * i, 1);
+    mbar_init_fence();
+  }
+  __syncthreads();
+  const size_t bs0 = static_cast<size_t>(block_slot(r0, j, 0));
+  auto fetch = [&](int blk) {                      // one thread
+    const int s = blk % kScanStages;
+    mbar_arrive_expect_tx(bar + 8 * s, kStageWords * 4);
+    bulk_g2s(sm_u + s * kStageWords * 4, p.kq + ((bs0 + blk) * p.HK + hk) * kKq, kKq * 4, bar + 8 * s);
+    bulk_g2s(sm_u + (s * kStageWords + kKq) * 4, p.vb + (((bs0 + blk) * p.H + h) * groups + blockIdx.z) * kVWords, kVWords * 4, bar + 8 * s);
   };
-  const int chunks = (blocks + kStage - 1) / kStage;
-  fetch(0);
-  for (int c = 0; c < chunks; ++c) {
-    if (c + 1 < chunks) {
-      fetch(c + 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
+  if (threadIdx.x == 0)
+    for (int i = 0; i < min(kScanStages, blocks); ++i) fetch(i);
+  float S[NJ][4][2] = {};
+  float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + vb + cl) * DP;
+  if (on) {
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+      for (int i = 0; i < NJ; ++i) {
+        const float4 f = *reinterpret_cast<const float4*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4);
+        S[i][0][c] = f.x; S[i][1][c] = f.y; S[i][2][c] = f.z; S[i][3][c] = f.w;
+      }
+  }
+  const int tok = lg >> 2, col = (lg >> 1) & 1;    // whose read-out value this lane keeps (lanes 2i, 2i + 1 share one)
+  float* out = p.o + (static_cast<size_t>(r0 + tok) * p.H + h) * p.VP + vb + cl + col;
+  const size_t out_step = static_cast<size_t>(kBlk) * p.H * p.VP;
+  bool ok = true;
+  for (int blk = 0; blk < blocks; ++blk) {
+    const int s = blk % kScanStages;
+    if (ok && !mbar_wait(bar + 8 * s, (blk / kScanStages) & 1, p.err, kErrWaitFull)) {
+      ok = false;                                  // copies of this thread still in flight land before the CTA leaves
+      if (threadIdx.x == 0)
+        for (int i = blk; i < min(blocks, blk + kScanStages); ++i)
+          mbar_wait(bar + 8 * (i % kScanStages), (i / kScanStages) & 1, p.err, kErrWaitDrain);
     }
-    __syncthreads();
-    if (on) {
-      for (int bi = 0; bi < kStage; ++bi) {
-        const int blk = c * kStage + bi;
-        if (blk >= blocks) break;
-        const float* b = sm + ((c & 1) * kStage + bi) * kBlock;
-        const int rows = min(kBlk, n - blk * kBlk);
-        float sk[kBlk][2] = {}, sq[kBlk][2] = {};
+    const float* b = sm + s * kStageWords;
+    const float* vrec = b + kKq;
+    if (on && ok) {
+      float sk[kBlk][2] = {}, sq[kBlk][2] = {};
 #pragma unroll
-        for (int r = 0; r < kBlk; ++r) {
-          const float* kr = b + r * kRow;
+      for (int r = 0; r < kBlk; ++r)
 #pragma unroll
-          for (int i = 0; i < NI; ++i) {
-            const float4 k4 = *reinterpret_cast<const float4*>(kr + i * 32 + lg * 4);
-            const float4 q4 = *reinterpret_cast<const float4*>(kr + DP + i * 32 + lg * 4);
-            const float ka[4] = {k4.x, k4.y, k4.z, k4.w}, qa[4] = {q4.x, q4.y, q4.z, q4.w};
+        for (int i = 0; i < NJ; ++i) {
+          const float4 k4 = *reinterpret_cast<const float4*>(b + r * DP + i * 64 + lg * 4);
+          const float4 q4 = *reinterpret_cast<const float4*>(b + (kBlk + r) * DP + i * 64 + lg * 4);
+          const float ka[4] = {k4.x, k4.y, k4.z, k4.w}, qa[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
+          for (int e = 0; e < 4; ++e)
 #pragma unroll
-              for (int v = 0; v < 2; ++v) {
-                sk[r][v] = fmaf(S[i][e][v], ka[e], sk[r][v]);
-                sq[r][v] = fmaf(S[i][e][v], qa[e], sq[r][v]);
-              }
-          }
+            for (int v = 0; v < 2; ++v) {
+              sk[r][v] = fmaf(S[i][e][v], ka[e], sk[r][v]);
+              sq[r][v] = fmaf(S[i][e][v], qa[e], sq[r][v]);
+            }
         }
 #pragma unroll
-        for (int o = 1; o < 8; o <<= 1)
-#pragma unroll
-          for (int r = 0; r < kBlk; ++r)
-#pragma unroll
-            for (int v = 0; v < 2; ++v) sk[r][v] += __shfl_xor_sync(0xffffffffu, sk[r][v], o);
-        // the read-out values: lane lg keeps token lg >> 1, column lg & 1 (halving exchange: 4 + 2 + 1 shuffles)
-        float mine;
-        {
-          float t4[4], t2[2];
-          const bool b2 = (lg & 4) != 0, b1 = (lg & 2) != 0, b0 = (lg & 1) != 0;
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {            // tokens 0, 1 stay with b2 = 0; tokens 2, 3 with b2 = 1
-            const float keep = b2 ? sq[2 + (e >> 1)][e & 1] : sq[e >> 1][e & 1];
-            const float give = b2 ? sq[e >> 1][e & 1] : sq[2 + (e >> 1)][e & 1];
-            t4[e] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
-          }
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const float keep = b1 ? t4[2 + e] : t4[e], give = b1 ? t4[e] : t4[2 + e];
-            t2[e] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
-          }
-          const float keep = b0 ? t2[1] : t2[0], give = b0 ? t2[0] : t2[1];
-          mine = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-        }
-        float beta[kBlk], g[kBlk], G[kBlk], dl[kBlk], u[kBlk][2], pr[kPairs];
-#pragma unroll
-        for (int e = 0; e < kPairs; e += 4) *reinterpret_cast<float4*>(pr + e) = *reinterpret_cast<const float4*>(b + kBlk * kRow + e);
-#pragma unroll
-        for (int r = 0; r < kBlk; ++r) {
-          const float2 bg = *reinterpret_cast<const float2*>(b + r * kRow + 2 * DP + 32);
-          beta[r] = bg.x;
-          g[r] = r < rows ? bg.y : 1.f;
-          G[r] = r == 0 ? g[0] : G[r - 1] * g[r];
-        }
-        const int tok = lg >> 1;
-        float o = 0.f;
-#pragma unroll
-        for (int i = 0; i < kBlk; ++i) {
-          const float2 v = *reinterpret_cast<const float2*>(b + i * kRow + 2 * DP + cl);
-          float a0 = v.x - G[i] * sk[i][0], a1 = v.y - G[i] * sk[i][1];
-#pragma unroll
-          for (int jj = 0; jj < i; ++jj) {
-            dl[jj] *= g[i];                        // D_ij
-            const float w = dl[jj] * pr[kk_at(i, jj)];
-            a0 = fmaf(-w, u[jj][0], a0);
-            a1 = fmaf(-w, u[jj][1], a1);
-          }
-          dl[i] = 1.f;
-          u[i][0] = beta[i] * a0;
-          u[i][1] = beta[i] * a1;
-          if (tok == i) {
-            o = G[i] * mine;
-#pragma unroll
-            for (int jj = 0; jj <= i; ++jj) o = fmaf(dl[jj] * pr[kq_at(i, jj)], (lg & 1) ? u[jj][1] : u[jj][0], o);
-          }
-        }
-        if (tok < rows) p.o[(static_cast<size_t>(r0 + blk * kBlk + tok) * p.H + h) * p.VP + vb + cl + (lg & 1)] = o;
-#pragma unroll
-        for (int jj = 0; jj < kBlk; ++jj) {        // D_4j is where the recurrence left it
-          u[jj][0] *= dl[jj];
-          u[jj][1] *= dl[jj];
-        }
-        const float G4 = G[kBlk - 1];
-#pragma unroll
-        for (int i = 0; i < NI; ++i)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) { S[i][e][0] *= G4; S[i][e][1] *= G4; }
+      for (int o = 1; o < 16; o <<= 1)
 #pragma unroll
         for (int r = 0; r < kBlk; ++r)
 #pragma unroll
-          for (int i = 0; i < NI; ++i) {
-            const float4 k4 = *reinterpret_cast<const float4*>(b + r * kRow + i * 32 + lg * 4);
-            const float ka[4] = {k4.x, k4.y, k4.z, k4.w};
+          for (int v = 0; v < 2; ++v) sk[r][v] += __shfl_xor_sync(0xffffffffu, sk[r][v], o);
+      // read-out values by halving exchange (4 + 2 + 1 + 1 shuffles)
+      float mine;
+      {
+        float t4[4], t2[2];
+        const bool b3 = (lg & 8) != 0, b2 = (lg & 4) != 0, b1 = (lg & 2) != 0;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              S[i][e][0] = fmaf(u[r][0], ka[e], S[i][e][0]);
-              S[i][e][1] = fmaf(u[r][1], ka[e], S[i][e][1]);
-            }
-          }
+        for (int e = 0; e < 4; ++e) {              // tokens 0, 1 stay with b3 = 0; tokens 2, 3 with b3 = 1
+          const float keep = b3 ? sq[2 + (e >> 1)][e & 1] : sq[e >> 1][e & 1];
+          const float give = b3 ? sq[e >> 1][e & 1] : sq[2 + (e >> 1)][e & 1];
+          t4[e] = keep + __shfl_xor_sync(0xffffffffu, give, 8);
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float keep = b2 ? t4[2 + e] : t4[e], give = b2 ? t4[e] : t4[2 + e];
+          t2[e] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+        }
+        const float keep = b1 ? t2[1] : t2[0], give = b1 ? t2[0] : t2[1];
+        mine = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+        mine += __shfl_xor_sync(0xffffffffu, mine, 1);
       }
+      float dl[kBlk], u[kBlk][2], pr[kPairs];
+#pragma unroll
+      for (int e = 0; e < kPairs; e += 4) *reinterpret_cast<float4*>(pr + e) = *reinterpret_cast<const float4*>(b + 2 * kBlk * DP + e);
+      const float4 be4 = *reinterpret_cast<const float4*>(vrec + kBlk * 32), g4 = *reinterpret_cast<const float4*>(vrec + kBlk * 32 + kBlk);
+      const float beta[4] = {be4.x, be4.y, be4.z, be4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
+      float G = 1.f, o = 0.f;
+#pragma unroll
+      for (int i = 0; i < kBlk; ++i) {
+        const float2 v = *reinterpret_cast<const float2*>(vrec + i * 32 + cl);
+        G *= g[i];
+        float a0 = v.x - G * sk[i][0], a1 = v.y - G * sk[i][1];
+#pragma unroll
+        for (int jj = 0; jj < i; ++jj) {
+          dl[jj] *= g[i];                          // D_ij
+          const float w = dl[jj] * pr[kk_at(i, jj)];
+          a0 = fmaf(-w, u[jj][0], a0);
+          a1 = fmaf(-w, u[jj][1], a1);
+        }
+        dl[i] = 1.f;
+        u[i][0] = beta[i] * a0;
+        u[i][1] = beta[i] * a1;
+        float t = G * mine;
+#pragma unroll
+        for (int jj = 0; jj <= i; ++jj) t = fmaf(dl[jj] * pr[kq_at(i, jj)], col ? u[jj][1] : u[jj][0], t);
+        o = tok == i ? t : o;
+      }
+      if ((lg & 1) == 0 && blk * kBlk + tok < n) out[blk * out_step] = o;
+#pragma unroll
+      for (int jj = 0; jj < kBlk; ++jj) {          // D_4j is where the recurrence left it
+        u[jj][0] *= dl[jj];
+        u[jj][1] *= dl[jj];
+      }
+#pragma unroll
+      for (int i = 0; i < NJ; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { S[i][e][0] *= G; S[i][e][1] *= G; }
+#pragma unroll
+      for (int r = 0; r < kBlk; ++r)
+#pragma unroll
+        for (int i = 0; i < NJ; ++i) {
+          const float4 k4 = *reinterpret_cast<const float4*>(b + r * DP + i * 64 + lg * 4);
+          const float ka[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            S[i][e][0] = fmaf(u[r][0], ka[e], S[i][e][0]);
+            S[i][e][1] = fmaf(u[r][1], ka[e], S[i][e][1]);
+          }
+        }
     }
-    __syncthreads();
+    __syncthreads();                               // the stage is free again
+    if (threadIdx.x == 0 && ok && blk + kScanStages < blocks) fetch(blk + kScanStages);
   }
-  if (on) delta_state_io<NI>(st, S, DP, lg, true);
+  if (on) {
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+      for (int i = 0; i < NJ; ++i)
+        *reinterpret_cast<float4*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4) = make_float4(S[i][0][c], S[i][1][c], S[i][2][c], S[i][3][c]);
+  }
 }
 
 // Gated norm of one head row (o: V values, shared or global memory) by a warp.
@@ -560,25 +573,31 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__
     operand_store1(p.out, m, p.out_k0 + h * p.V + v, os[v] * r * p.norm_w[v] * silu_f32(x[p.g_off + h * p.V + v]));
 }
 
-template <int NI>
+template <int NI, int TAPS>
+static cudaError_t delta_prep(const DeltaParams& p, cudaStream_t stream) {
+  return launch(delta_prep_kernel<NI, TAPS>, dim3(p.M / kBlk + p.nseq, (p.HK + p.H + 3) / 4), dim3(128), 0, stream, 0, p);
+}
+
+template <int NJ>
 static int delta_go(const DeltaParams& p, bool single, cudaStream_t stream) {
+  constexpr int NI = NJ * 2;
   if (single) {
     const int warps = min(8, p.VP / 8);
     const int smem = (2 * NI * 32 + 2 * p.VP) * 4;
     return static_cast<int>(launch(delta_step_kernel<NI>, dim3(p.H, p.nseq), dim3(32 * warps), smem, stream, 0, p));
   }
-  const int smem = 2 * kStage * (kBlk * (2 * NI * 32 + 36) + kPairs) * 4;
+  const int smem = kScanStages * (kq_words(NI * 32) + kVWords) * 4;
   static bool ready[64];
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
   if (!ready[dev]) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NI>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
     ready[dev] = true;
   }
-  cudaError_t e = launch(delta_prep_kernel<NI>, dim3(p.M / kBlk + p.nseq, (p.HK + p.H + 4) / 4), dim3(128), 0, stream, 0, p);
-  if (e == cudaSuccess) e = launch(delta_scan_kernel<NI>, dim3(p.nseq, p.H, (p.VP + 31) / 32), dim3(128), smem, stream, 0, p);
+  cudaError_t e = p.taps == 4 ? delta_prep<NI, 4>(p, stream) : delta_prep<NI, 0>(p, stream);
+  if (e == cudaSuccess) e = launch(delta_scan_kernel<NJ>, dim3(p.nseq, p.H, (p.VP + 31) / 32), dim3(256), smem, stream, 0, p);
   if (e == cudaSuccess) e = launch(delta_out_kernel, dim3(p.M + p.nseq, (p.H + 7) / 8), dim3(256), 0, stream, 0, p);
   return static_cast<int>(e);
 }
@@ -592,14 +611,12 @@ extern "C" int saber_delta_launch(const saber::DeltaParams* p, int single_row, c
   if (p->M <= 0 || p->nseq <= 0 || p->HK <= 0 || p->H % p->HK || p->D > p->DP || (p->VP & 7) || p->V > p->VP || p->VP > 4096 || p->taps < 1)
     return static_cast<int>(cudaErrorInvalidValue);
   switch (p->DP) {
-    case 32: return delta_go<1>(*p, single_row != 0, stream);
-    case 64: return delta_go<2>(*p, single_row != 0, stream);
-    case 96: return delta_go<3>(*p, single_row != 0, stream);
-    case 128: return delta_go<4>(*p, single_row != 0, stream);
-    case 192: return delta_go<6>(*p, single_row != 0, stream);
-    case 256: return delta_go<8>(*p, single_row != 0, stream);
-    case 384: return delta_go<12>(*p, single_row != 0, stream);
-    case 512: return delta_go<16>(*p, single_row != 0, stream);
+    case 64: return delta_go<1>(*p, single_row != 0, stream);
+    case 128: return delta_go<2>(*p, single_row != 0, stream);
+    case 192: return delta_go<3>(*p, single_row != 0, stream);
+    case 256: return delta_go<4>(*p, single_row != 0, stream);
+    case 384: return delta_go<6>(*p, single_row != 0, stream);
+    case 512: return delta_go<8>(*p, single_row != 0, stream);
     default: return static_cast<int>(cudaErrorInvalidValue);
   }
 }

@@ -23,11 +23,8 @@ struct DeltaParams {
   // step only overwrites rows that no later token reads.
   float* hist;             // [nslots][taps][C]
   float* state;            // [nslots][H][VP][DP] (pads stay zero)
-  float* qn;               // scratch [M][HK][DP]
-  float* kn;               // scratch [M][HK][DP]
-  float* vv;               // scratch [M][H][VP]
-  float* bg;               // scratch [M][H][2]: beta, g
-  float* pairs;            // scratch [M / 4 + nseq][HK][16]: dot products inside each block of four tokens
+  float* kq;               // scratch [M / 4 + nseq][HK][8 DP + 16]: blocks of four tokens, see delta.cu
+  float* vb;               // scratch [M / 4 + nseq][H][ceil(VP / 32)][136]
   float* o;                // scratch [M][H][VP]
   const int32_t* cu_rows;  // [nseq + 1]
   const int32_t* slots;    // [nseq], < 0: padding sequence

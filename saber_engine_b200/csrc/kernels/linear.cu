@@ -39,12 +39,12 @@ __device__ __forceinline__ float row_rms_scale(const LinEpi& e, int m, int lane)
 }
 
 // One finished row of a 256-column tile, by a warp.  acc(c): the eight (project, stream) or four (gated unit)
-// accumulators from column c on.
+// accumulators from column c on.  sc: the row's scale (project); x0, x1: this lane's eight values of the stream row
+// (stream, when the linear adds to it), fetched by the caller ahead of time.
 template <typename Acc>
-__device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& acc, int m, int tile_n, int lane) {
+__device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& acc, int m, int tile_n, int lane, float sc, float4 x0, float4 x1) {
   const int n0 = tile_n * 256;
   if (!e.stream) {
-    const float sc = row_rms_scale(e, m, lane);
     if (tile_n < e.act_tile0) {
       const int n = n0 + lane * 8;
       if (n >= e.n_plain) return;
@@ -74,7 +74,6 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
     const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
     float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
     if (e.add) {
-      const float4 x0 = *reinterpret_cast<const float4*>(xr), x1 = *reinterpret_cast<const float4*>(xr + 4);
       v[0] += x0.x; v[1] += x0.y; v[2] += x0.z; v[3] += x0.w;
       v[4] += x1.x; v[5] += x1.y; v[6] += x1.z; v[7] += x1.w;
     }
@@ -97,11 +96,40 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
   if ((lane & 15) == 0 && g < e.ss_out_n) e.ss_out[static_cast<size_t>(m) * e.ss_out_n + g] = sq;
 }
 
+// The staged rows of a tile (shared memory, kLinRow floats apart), four per warp and round: their stream rows are
+// requested together.
+__device__ __forceinline__ void linear_tile_epilogue(const LinEpi& e, const float* tile_s, const float* scale_s, int mb, int rows, int tile_n,
+                                                     int w, int lane) {
+  const int n = tile_n * 256 + lane * 8;
+  const bool addx = e.stream && e.add && n < e.width;
+  for (int r0 = w; r0 < rows; r0 += 32) {
+    float4 x[4][2];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = r0 + 8 * i;
+      x[i][0] = x[i][1] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (addx && r < rows) {
+        const float4* xr = reinterpret_cast<const float4*>(e.x + static_cast<size_t>(mb + r) * e.ldx + n);
+        x[i][0] = xr[0];
+        x[i][1] = xr[1];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = r0 + 8 * i;
+      if (r < rows)
+        linear_row_epilogue(e, [&](int c) { return *reinterpret_cast<const float4*>(tile_s + r * kLinRow + c); }, mb + r, tile_n, lane,
+                            scale_s[r], x[i][0], x[i][1]);
+    }
+  }
+}
+
 template <int kMT>
 __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_constant__ LinParams p, const int stages) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t bars[2 * kLinMaxStages + 1];
   __shared__ uint32_t tmem_base_s, is_last_s, abort_s;
+  __shared__ float scale_s[256];
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tile_m = blockIdx.x, tile_n = blockIdx.y, split = blockIdx.z;
@@ -211,12 +239,24 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
     const int grp = te >> 7;                      // column half this warp reads out
     const int q4 = warp & 3;                      // TMEM lane quarter of this warp
     const LinEpi& e = p.e;
+    pdl_wait();
+    // row scales while the main loop runs: a thread per row
+    if (te < p.nt * kMT) {
+      float sc = 1.f;
+      if (e.ss != nullptr && m0 + te < p.M) {
+        const float* q = e.ss + static_cast<size_t>(m0 + te) * e.ss_n;
+        float s = 0.f;
+#pragma unroll 8
+        for (int i = 0; i < e.ss_n; ++i) s += __ldcg(q + i);
+        sc = 1.f / sqrtf(s * e.inv_width + e.eps);
+      }
+      scale_s[te] = sc;
+    }
     bool ok = mbar_wait(bar_acc, 0, p.err, kErrWaitAcc);
     if (!ok) abort_s = 1u;
     named_bar_sync(1, 256);
     ok = abort_s == 0u;
     tc_fence_after_sync();
-    pdl_wait();
     const int rowl = q4 * 32 + lane;
     const uint32_t t_lane = tmem_d + (static_cast<uint32_t>(q4 * 32) << 16);
     const int tile_lin = tile_m * gridDim.y + tile_n;
@@ -265,8 +305,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
           *reinterpret_cast<float4*>(tile_s + r * kLinRow + c4 * 4) = s;
         }
         named_bar_sync(1, 256);
-        for (int r = warp - 2; r < mt; r += 8)
-          linear_row_epilogue(e, [&](int c) { return *reinterpret_cast<const float4*>(tile_s + r * kLinRow + c); }, m0 + r, tile_n, lane);
+        linear_tile_epilogue(e, tile_s, scale_s, m0, mt, tile_n, warp - 2, lane);
       }
     } else if (ok) {
 #pragma unroll 1
@@ -289,8 +328,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
           }
         }
         named_bar_sync(1, 256);
-        for (int r = warp - 2; r < mt; r += 8)
-          linear_row_epilogue(e, [&](int c) { return *reinterpret_cast<const float4*>(tile_s + r * kLinRow + c); }, mb + r, tile_n, lane);
+        linear_tile_epilogue(e, tile_s, scale_s + j2 * p.nt, mb, mt, tile_n, warp - 2, lane);
       }
     }
   }

@@ -238,12 +238,10 @@ class StackModel:
         mx = lambda it: max(it, default=0)    # noqa: E731
         wk = {"splits": self._splits(M, decode)}
         if not decode:
-            wk["qn"] = f32(M * mx(m.kv_heads * m.dim_pad for m in de))
-            wk["kn"] = f32(M * mx(m.kv_heads * m.dim_pad for m in de))
-            wk["vv"] = f32(M * mx(m.heads * m.vdim_pad for m in de))
+            blk = M // 4 + nseq                           # blocks of four tokens
+            wk["kq"] = f32(blk * mx(m.kv_heads * (8 * m.dim_pad + 16) for m in de))
+            wk["vb"] = f32(blk * mx(m.heads * ((m.vdim_pad + 31) // 32) * 136 for m in de))
             wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in de))
-            wk["pairs"] = f32((M // 4 + nseq) * 16 * mx(m.kv_heads for m in de))
-            wk["bg"] = f32(M * mx(2 * m.heads for m in de))
         wk["q_eff"] = torch.zeros(max(1, M * mx(m.heads * (max(m.rank_pad, m.dim_pad) + m.rot_pad) for m in la)), dtype=self.dtype, device=self.device)
         absorbed = [m for m in la if not self._expanded(m, M, decode)]
         if absorbed:
@@ -269,7 +267,7 @@ class StackModel:
         p.q_off, p.k_off, p.v_off, p.b_off, p.a_off, p.g_off = (lw.off[k] for k in ("q", "k", "v", "b", "a", "g"))
         p.conv_w, p.A_log, p.dt_bias, p.norm_w = (lw.extra[k].data_ptr() for k in ("conv", "A_log", "dt_bias", "norm"))
         p.hist, p.state = self.delta_hist[run.index].data_ptr(), self.delta_state[run.index].data_ptr()
-        p.qn, p.kn, p.vv, p.bg, p.pairs, p.o = (N.ptr(wk.get(k)) for k in ("qn", "kn", "vv", "bg", "pairs", "o"))
+        p.kq, p.vb, p.o = (N.ptr(wk.get(k)) for k in ("kq", "vb", "o"))
         p.cu_rows, p.slots, p.pos = at(lay.cu_rows), at(lay.slots), at(lay.pos)
         p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
         p.H, p.HK, p.D, p.DP, p.V, p.VP, p.taps, p.n_slots = m.heads, m.kv_heads, m.dim, m.dim_pad, m.vdim, m.vdim_pad, m.taps, self.n_slots

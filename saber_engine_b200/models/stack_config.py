@@ -34,7 +34,7 @@ class DeltaMixer:
 
     @property
     def dim_pad(self) -> int:         # key sizes the kernels are instantiated for
-        for n in (32, 64, 96, 128, 192, 256, 384, 512):
+        for n in (64, 128, 192, 256, 384, 512):
             if n >= self.dim:
                 return n
         raise ValueError(f"delta mixer: key size {self.dim} is above 512")

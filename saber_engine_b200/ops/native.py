@@ -192,7 +192,7 @@ class StreamNormParams(C.Structure):
 
 class DeltaParams(C.Structure):
     _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("k_off", I), ("v_off", I), ("b_off", I), ("a_off", I), ("g_off", I), ("conv_w", P),
-                ("A_log", P), ("dt_bias", P), ("norm_w", P), ("hist", P), ("state", P), ("qn", P), ("kn", P), ("vv", P), ("bg", P), ("pairs", P), ("o", P),
+                ("A_log", P), ("dt_bias", P), ("norm_w", P), ("hist", P), ("state", P), ("kq", P), ("vb", P), ("o", P),
                 ("cu_rows", P), ("slots", P), ("pos", P), ("out", Operand), ("out_k0", I), ("M", I), ("nseq", I), ("H", I), ("HK", I),
                 ("D", I), ("DP", I), ("V", I), ("VP", I), ("taps", I), ("n_slots", I), ("eps", F), ("unit_eps", F), ("q_scale", F), ("err", P)]
 

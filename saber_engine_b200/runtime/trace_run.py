@@ -35,23 +35,27 @@ class _Request:
 
 
 class TraceEngine:
-    def __init__(self, model_dir: str, dtype: str, max_tokens: int):
+    """Replay over one model: its executor, and the scheduler's allocators for its pages and slots."""
+
+    def __init__(self, model, prefill_rungs: tuple = PREFILL_RUNGS, capture: bool = True):
+        from ..sched.alloc import Arenas, GdnStateAllocator, PagedKvAllocator
+        from .hybrid_executor import HybridExecutor
+        self.model = model
+        self.ex = HybridExecutor(model, decode_batches=tuple(range(1, model.max_seqs + 1)), decode_widths=(1,), prefill_rungs=prefill_rungs,
+                                 prefill_pack=model.max_seqs, capture=capture)
+        self.arenas = Arenas(PagedKvAllocator(model.kv_blocks, model.cfg.page_tokens), GdnStateAllocator(model.max_seqs + 1))
+        self.live: dict = {}
+        self.admitted = 0
+
+    @staticmethod
+    def open(model_dir: str, dtype: str, max_tokens: int) -> "TraceEngine":
         import torch
         from ..models import config as MC
         from ..models.stack import StackModel
-        from ..sched.alloc import Arenas, GdnStateAllocator, PagedKvAllocator
-        from .hybrid_executor import HybridExecutor
-        torch.backends.cuda.matmul.allow_tf32 = False
         cfg = MC.by_name(model_dir)
-        page = cfg.page_tokens
-        n_blocks = (max_tokens + page - 1) // page + 1            # block 0 is the null block
-        self.model = StackModel(cfg, device="cuda", max_seqs=MAX_LIVE, max_ctx=max(page, (n_blocks - 1) * page), kv_blocks=n_blocks,
-                                dtype=getattr(torch, dtype))
-        self.ex = HybridExecutor(self.model, decode_batches=tuple(range(1, MAX_LIVE + 1)), decode_widths=(1,), prefill_rungs=PREFILL_RUNGS,
-                                 prefill_pack=MAX_LIVE)
-        self.arenas = Arenas(PagedKvAllocator(n_blocks, page), GdnStateAllocator(MAX_LIVE + 1))
-        self.live: dict = {}
-        self.admitted = 0
+        pages = (max_tokens + cfg.page_tokens - 1) // cfg.page_tokens
+        return TraceEngine(StackModel(cfg, device="cuda", max_seqs=MAX_LIVE, max_ctx=max(1, pages) * cfg.page_tokens, kv_blocks=pages + 1,
+                                      dtype=getattr(torch, dtype)))      # block 0 is the null block
 
     def _admit(self, rid) -> _Request:
         self.admitted += 1
@@ -110,7 +114,7 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True, help="tokens that live requests hold at most (sizes the page pool)")
     a = ap.parse_args(argv)
     import torch
-    eng = TraceEngine(a.model, a.dtype, a.max_tokens)
+    eng = TraceEngine.open(a.model, a.dtype, a.max_tokens)
     for line in sys.stdin:
         if not line.strip():
             continue

@@ -145,8 +145,8 @@ class Oracle:
         """(tokens, smallest gap between the best and the second logit on the way)."""
         ids, out, gap = list(prompt), [], float("inf")
         for _ in range(n):
-            top = torch.topk(self.forward(ids)[-1], 2).values
-            gap = min(gap, float(top[0] - top[1]))
-            out.append(int(self.forward(ids)[-1].argmax()))
+            top = torch.topk(self.forward(ids)[-1], 2)
+            gap = min(gap, float(top.values[0] - top.values[1]))
+            out.append(int(top.indices[0]))
             ids.append(out[-1])
         return out, gap

@@ -117,10 +117,11 @@ __device__ __forceinline__ void conv_silu4(const DeltaParams& p, const float* hi
 
 // Scratch records of a block, each contiguous (one bulk copy):
 //   key head   k rows [4][DP] | q rows [4][DP] | 16 dot products
-//   value head, per 32 columns   v [4][32] | beta [4] | g [4]
+//   value head, per 16 columns   v [4][16] | beta [4] | g [4]
 // Missing tokens of the last block are written as k = q = v = beta = 0, g = 1.
 __host__ __device__ constexpr int kq_words(int DP) { return 2 * kBlk * DP + kPairs; }
-constexpr int kVWords = kBlk * 32 + 2 * kBlk;
+constexpr int kCols = 16;                // value columns of a scan CTA
+constexpr int kVWords = kBlk * kCols + 2 * kBlk;
 
 // grid (blocks, ceil((HK + H) / 4)), 128 threads; a warp per item: key heads (q, k and their dot products), value heads
 template <int NI, int TAPS>
@@ -188,25 +189,26 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const __grid_constant__
       }
     if (lane < kPairs) o[2 * kBlk * DP + lane] = mine;
   } else {
-    const int h = item - p.HK, groups = (p.VP + 31) / 32;
+    const int h = item - p.HK, groups = (p.VP + kCols - 1) / kCols;
     float beta = 0.f, g = 1.f;                     // lanes 0 .. 3: one token each
     if (lane < rows) {
       const float* x = p.x + static_cast<size_t>(m + lane) * p.ldx;
       beta = sigmoid_f32(x[p.b_off + h]);
       g = expf(-expf(p.A_log[h]) * softplus_f32(x[p.a_off + h] + p.dt_bias[h]));
     }
-    for (int gr = 0; gr < groups; ++gr) {
-      const int d = gr * 32 + lane;
+    for (int d = lane; d < groups * kCols; d += 32) {
       float y[kBlk] = {};
       if (d < p.V) conv_silu4<TAPS>(p, hist, 2 * p.HK * p.D + h * p.V + d, p.v_off + h * p.V + d, m, t, pos, C, rows, y);
-      float* o = p.vb + ((static_cast<size_t>(blockIdx.x) * p.H + h) * groups + gr) * kVWords;
+      float* o = p.vb + ((static_cast<size_t>(blockIdx.x) * p.H + h) * groups + d / kCols) * kVWords + d % kCols;
 #pragma unroll
-      for (int r = 0; r < kBlk; ++r) o[r * 32 + lane] = y[r];
-      if (lane < kBlk) {
-        o[kBlk * 32 + lane] = beta;
-        o[kBlk * 32 + kBlk + lane] = g;
-      }
+      for (int r = 0; r < kBlk; ++r) o[r * kCols] = y[r];
     }
+    float* o = p.vb + (static_cast<size_t>(blockIdx.x) * p.H + h) * groups * kVWords + kBlk * kCols;
+    for (int gr = 0; gr < groups; ++gr)
+      if (lane < kBlk) {
+        o[gr * kVWords + lane] = beta;
+        o[gr * kVWords + kBlk + lane] = g;
+      }
   }
 }
 
@@ -271,15 +273,18 @@ __device__ __forceinline__ void delta_state_io(float* st, float (&S)[NI][4][2], 
 
 constexpr int kScanStages = 4;           // blocks of four tokens in flight
 
-// grid (nseq, H, ceil(VP / 32)), 256 threads: a warp per four value columns (two lane groups of two), 16 lanes along the keys
+// grid (nseq, H, ceil(VP / 16)), 160 threads: four warps of four value columns (two lane groups of two columns, 16 lanes
+// along the keys), each at its own pace, and a warp whose first lane keeps the copies going
+constexpr int kScanThreads = 160;
+
 template <int NJ>
-__global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__ DeltaParams p) {
+__global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_constant__ DeltaParams p) {
   constexpr int DP = NJ * 64;
   constexpr int kKq = kq_words(DP);
   constexpr int kStageWords = kKq + kVWords;
   extern __shared__ float4 sm4[];
   float* sm = reinterpret_cast<float*>(sm4);
-  __shared__ uint64_t bars[kScanStages];
+  __shared__ uint64_t bars[2 * kScanStages];
   pdl_wait();
   const int j = blockIdx.x, h = blockIdx.y;
   const int r0 = p.cu_rows[j], n = p.cu_rows[j + 1] - r0;
@@ -287,27 +292,40 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__
   const int slot = delta_slot(p, j);
   if (slot < 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
-  const int vb = blockIdx.z * 32, groups = (p.VP + 31) / 32;
+  const int vb = blockIdx.z * kCols, groups = (p.VP + kCols - 1) / kCols;
   const int hk = h / (p.H / p.HK);
-  const int cl = warp * 4 + (lane >> 4) * 2;       // column inside the CTA's 32
+  const int cl = warp * 4 + (lane >> 4) * 2;       // column inside the CTA's 16
   const bool on = vb + warp * 4 < p.VP;            // VP is a multiple of 8
   const int blocks = (n + kBlk - 1) / kBlk;
-  const uint32_t bar = smem_u32(bars);
+  const uint32_t bar = smem_u32(bars), bar_free = bar + 8 * kScanStages;
   const uint32_t sm_u = smem_u32(sm);
   if (threadIdx.x == 0) {
-    for (int i = 0; i < kScanStages; ++i) mbar_init(bar + 8 * i, 1);
+    for (int i = 0; i < kScanStages; ++i) {
+      mbar_init(bar + 8 * i, 1);
+      mbar_init(bar_free + 8 * i, 4);
+    }
     mbar_init_fence();
   }
   __syncthreads();
-  const size_t bs0 = static_cast<size_t>(block_slot(r0, j, 0));
-  auto fetch = [&](int blk) {                      // one thread
-    const int s = blk % kScanStages;
-    mbar_arrive_expect_tx(bar + 8 * s, kStageWords * 4);
-    bulk_g2s(sm_u + s * kStageWords * 4, p.kq + ((bs0 + blk) * p.HK + hk) * kKq, kKq * 4, bar + 8 * s);
-    bulk_g2s(sm_u + (s * kStageWords + kKq) * 4, p.vb + (((bs0 + blk) * p.H + h) * groups + blockIdx.z) * kVWords, kVWords * 4, bar + 8 * s);
-  };
-  if (threadIdx.x == 0)
-    for (int i = 0; i < min(kScanStages, blocks); ++i) fetch(i);
+  if (warp == 4) {                                 // ---- copies
+    if (lane == 0) {
+      const size_t bs0 = static_cast<size_t>(block_slot(r0, j, 0));
+      const float* kq = p.kq + (bs0 * p.HK + hk) * kKq;
+      const float* vr = p.vb + ((bs0 * p.H + h) * groups + blockIdx.z) * kVWords;
+      const size_t kq_step = static_cast<size_t>(p.HK) * kKq, v_step = static_cast<size_t>(p.H) * groups * kVWords;
+      int blk = 0;
+      for (; blk < blocks; ++blk) {
+        const int s = blk % kScanStages;
+        if (blk >= kScanStages && !mbar_wait(bar_free + 8 * s, ((blk / kScanStages) & 1) ^ 1, p.err, kErrWaitEmpty)) break;
+        mbar_arrive_expect_tx(bar + 8 * s, kStageWords * 4);
+        bulk_g2s(sm_u + s * kStageWords * 4, kq + blk * kq_step, kKq * 4, bar + 8 * s);
+        bulk_g2s(sm_u + (s * kStageWords + kKq) * 4, vr + blk * v_step, kVWords * 4, bar + 8 * s);
+      }
+      for (int i = max(0, blk - kScanStages); i < blk; ++i)        // the CTA does not leave before its copies have landed
+        mbar_wait(bar + 8 * (i % kScanStages), (i / kScanStages) & 1, p.err, kErrWaitDrain);
+    }
+    return;
+  }
   float S[NJ][4][2] = {};
   float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + vb + cl) * DP;
   if (on) {
@@ -322,18 +340,12 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__
   const int tok = lg >> 2, col = (lg >> 1) & 1;    // whose read-out value this lane keeps (lanes 2i, 2i + 1 share one)
   float* out = p.o + (static_cast<size_t>(r0 + tok) * p.H + h) * p.VP + vb + cl + col;
   const size_t out_step = static_cast<size_t>(kBlk) * p.H * p.VP;
-  bool ok = true;
   for (int blk = 0; blk < blocks; ++blk) {
     const int s = blk % kScanStages;
-    if (ok && !mbar_wait(bar + 8 * s, (blk / kScanStages) & 1, p.err, kErrWaitFull)) {
-      ok = false;                                  // copies of this thread still in flight land before the CTA leaves
-      if (threadIdx.x == 0)
-        for (int i = blk; i < min(blocks, blk + kScanStages); ++i)
-          mbar_wait(bar + 8 * (i % kScanStages), (i / kScanStages) & 1, p.err, kErrWaitDrain);
-    }
+    if (!mbar_wait(bar + 8 * s, (blk / kScanStages) & 1, p.err, kErrWaitFull)) break;
     const float* b = sm + s * kStageWords;
     const float* vrec = b + kKq;
-    if (on && ok) {
+    if (on) {
       float sk[kBlk][2] = {}, sq[kBlk][2] = {};
 #pragma unroll
       for (int r = 0; r < kBlk; ++r)
@@ -379,12 +391,12 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__
       float dl[kBlk], u[kBlk][2], pr[kPairs];
 #pragma unroll
       for (int e = 0; e < kPairs; e += 4) *reinterpret_cast<float4*>(pr + e) = *reinterpret_cast<const float4*>(b + 2 * kBlk * DP + e);
-      const float4 be4 = *reinterpret_cast<const float4*>(vrec + kBlk * 32), g4 = *reinterpret_cast<const float4*>(vrec + kBlk * 32 + kBlk);
+      const float4 be4 = *reinterpret_cast<const float4*>(vrec + kBlk * kCols), g4 = *reinterpret_cast<const float4*>(vrec + kBlk * kCols + kBlk);
       const float beta[4] = {be4.x, be4.y, be4.z, be4.w}, g[4] = {g4.x, g4.y, g4.z, g4.w};
       float G = 1.f, o = 0.f;
 #pragma unroll
       for (int i = 0; i < kBlk; ++i) {
-        const float2 v = *reinterpret_cast<const float2*>(vrec + i * 32 + cl);
+        const float2 v = *reinterpret_cast<const float2*>(vrec + i * kCols + cl);
         G *= g[i];
         float a0 = v.x - G * sk[i][0], a1 = v.y - G * sk[i][1];
 #pragma unroll
@@ -425,8 +437,8 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(const __grid_constant__
           }
         }
     }
-    __syncthreads();                               // the stage is free again
-    if (threadIdx.x == 0 && ok && blk + kScanStages < blocks) fetch(blk + kScanStages);
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar_free + 8 * s);  // this warp is done with the stage
   }
   if (on) {
 #pragma unroll
@@ -597,7 +609,7 @@ static int delta_go(const DeltaParams& p, bool single, cudaStream_t stream) {
     ready[dev] = true;
   }
   cudaError_t e = p.taps == 4 ? delta_prep<NI, 4>(p, stream) : delta_prep<NI, 0>(p, stream);
-  if (e == cudaSuccess) e = launch(delta_scan_kernel<NJ>, dim3(p.nseq, p.H, (p.VP + 31) / 32), dim3(256), smem, stream, 0, p);
+  if (e == cudaSuccess) e = launch(delta_scan_kernel<NJ>, dim3(p.nseq, p.H, (p.VP + kCols - 1) / kCols), dim3(kScanThreads), smem, stream, 0, p);
   if (e == cudaSuccess) e = launch(delta_out_kernel, dim3(p.M + p.nseq, (p.H + 7) / 8), dim3(256), 0, stream, 0, p);
   return static_cast<int>(e);
 }

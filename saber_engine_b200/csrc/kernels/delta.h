@@ -24,7 +24,7 @@ struct DeltaParams {
   float* hist;             // [nslots][taps][C]
   float* state;            // [nslots][H][VP][DP] (pads stay zero)
   float* kq;               // scratch [M / 4 + nseq][HK][8 DP + 16]: blocks of four tokens, see delta.cu
-  float* vb;               // scratch [M / 4 + nseq][H][ceil(VP / 32)][136]
+  float* vb;               // scratch [M / 4 + nseq][H][ceil(VP / 16)][72]
   float* o;                // scratch [M][H][VP]
   const int32_t* cu_rows;  // [nseq + 1]
   const int32_t* slots;    // [nseq], < 0: padding sequence

@@ -240,7 +240,7 @@ class StackModel:
         if not decode:
             blk = M // 4 + nseq                           # blocks of four tokens
             wk["kq"] = f32(blk * mx(m.kv_heads * (8 * m.dim_pad + 16) for m in de))
-            wk["vb"] = f32(blk * mx(m.heads * ((m.vdim_pad + 31) // 32) * 136 for m in de))
+            wk["vb"] = f32(blk * mx(m.heads * ((m.vdim_pad + 15) // 16) * 72 for m in de))
             wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in de))
         wk["q_eff"] = torch.zeros(max(1, M * mx(m.heads * (max(m.rank_pad, m.dim_pad) + m.rot_pad) for m in la)), dtype=self.dtype, device=self.device)
         absorbed = [m for m in la if not self._expanded(m, M, decode)]

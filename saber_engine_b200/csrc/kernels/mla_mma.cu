@@ -118,8 +118,8 @@ __global__ void __launch_bounds__(256) mla_decode_kernel(const __grid_constant__
       v.y += v2.y;
       const float a = lane * 2 < n ? v.x * p.scale : -INFINITY, b = lane * 2 + 1 < n ? v.y * p.scale : -INFINITY;
       const float mn = fmaxf(mx[i], mla_warp_max(fmaxf(a, b)));
-      const float ea = exp2f((a - mn) * kLog2e), eb = exp2f((b - mn) * kLog2e);
-      const float corr = exp2f((mx[i] - mn) * kLog2e);
+      const float ea = ex2((a - mn) * kLog2e), eb = ex2((b - mn) * kLog2e);
+      const float corr = ex2((mx[i] - mn) * kLog2e);
       l[i] = l[i] * corr + mla_warp_sum(ea + eb);
       mx[i] = mn;
       asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_s + r * 144 + lane * 4), "r"(pack2(ea, eb)) : "memory");
@@ -357,19 +357,22 @@ __global__ void __launch_bounds__(256) mla_flash_kernel(const __grid_constant__ 
     const int r = i / kch, c = i - r * kch;
     cp16(q_s + r * ks_ + c * 16, qg + static_cast<size_t>(min(r, rows - 1)) * p.H * DK + c * 8, r < rows);
   }
+  int next_page = mla_page_at(p, j, 0);                             // looked up one block ahead of its copies
   auto fetch = [&](int b) {
-    const size_t pg = static_cast<size_t>(mla_page_at(p, j, b)) * p.H + h;
+    const size_t pg = static_cast<size_t>(next_page) * p.H + h;
+    if (b + 1 < blocks) next_page = mla_page_at(p, j, b + 1);
     const __nv_bfloat16* kg = ke + pg * kKeys * DK;
     const __nv_bfloat16* vg = ve + pg * kKeys * VP;
     const uint32_t kd = kv_s + (b & 1) * stage, vd = kd + kKeys * ks_;
-    for (int i = threadIdx.x; i < kKeys * kch; i += 256) {
-      const int r = i / kch, c = i - r * kch;
-      cp16(kd + r * ks_ + c * 16, kg + i * 8, true);
-    }
-    for (int i = threadIdx.x; i < kKeys * vch; i += 256) {
-      const int r = i / vch, c = i - r * vch;
+#pragma unroll 4
+    for (int r = warp; r < kKeys; r += 8)                           // a warp per key row
+      for (int c = lane; c < kch; c += 32) cp16(kd + r * ks_ + c * 16, kg + r * DK + c * 8, true);
+    constexpr int kPer = vch < 32 ? 32 / vch : 1;                   // value rows a warp copies at a time
+#pragma unroll
+    for (int r0v = 0; r0v < kKeys; r0v += 8 * kPer) {
+      const int r = r0v + warp * kPer + lane / (vch < 32 ? vch : 32);
       const bool live = b * kKeys + r < keys;                       // rows never written must not reach a product (0 x NaN)
-      cp16(vd + r * vs_ + c * 16, vg + i * 8, live);
+      for (int c = lane % (vch < 32 ? vch : 32); c < vch; c += 32) cp16(vd + r * vs_ + c * 16, vg + r * VP + c * 8, live);
     }
     cp_commit();
   };
@@ -390,35 +393,52 @@ __global__ void __launch_bounds__(256) mla_flash_kernel(const __grid_constant__ 
     float s[8][4] = {};
     const uint32_t a_row = q_s + (warp * 16 + (lane & 15)) * ks_ + ((lane >> 4) << 4);
     const uint32_t b_row = kd + (((lane >> 4) << 3) + (lane & 7)) * ks_ + (((lane >> 3) & 1) << 4);
-#pragma unroll 2
-    for (int kk = 0; kk < DK; kk += 16) {
-      uint32_t a[4];
-      ldsm4(a, a_row + kk * 2);
+    // fragments of the next step are requested before the products of this one
+    uint32_t fa[4], fb[4][4];
+    ldsm4(fa, a_row);
 #pragma unroll
-      for (int i = 0; i < 8; i += 2) {
-        uint32_t bb[4];
-        ldsm4(bb, b_row + i * 8 * ks_ + kk * 2);
-        mma16816(s[i], a, bb[0], bb[1]);
-        mma16816(s[i + 1], a, bb[2], bb[3]);
+    for (int i = 0; i < 4; ++i) ldsm4(fb[i], b_row + i * 16 * ks_);
+#pragma unroll 4
+    for (int kk = 16; kk <= DK; kk += 16) {
+      uint32_t ca[4], cb[4][4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        ca[x] = fa[x];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) cb[i][x] = fb[i][x];
+      }
+      // (past the last step: the first fragments again, unused)
+      ldsm4(fa, a_row + (kk < DK ? kk : 0) * 2);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) ldsm4(fb[i], b_row + i * 16 * ks_ + (kk < DK ? kk : 0) * 2);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        mma16816(s[2 * i], ca, cb[i][0], cb[i][1]);
+        mma16816(s[2 * i + 1], ca, cb[i][2], cb[i][3]);
       }
     }
     const int kb = b * kKeys;
     const bool edge = kb + kKeys - 1 > pos0 + warp * 16;            // some key lies past some row of this warp
+    if (edge) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (kb + i * 8 + (lane & 3) * 2 + (e & 1) > pos0 + row + (e >> 1) * 8) s[i][e] = -INFINITY;
+    }
+    // running maximum in unscaled scores: needs scale > 0 (checked on the host)
     float mn[2] = {mx[0], mx[1]};
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        s[i][e] *= sc;
-        if (edge && kb + i * 8 + (lane & 3) * 2 + (e & 1) > pos0 + row + (e >> 1) * 8) s[i][e] = -INFINITY;
-        mn[e >> 1] = fmaxf(mn[e >> 1], s[i][e]);
-      }
-    float corr[2];
+      for (int e = 0; e < 4; ++e) mn[e >> 1] = fmaxf(mn[e >> 1], s[i][e]);
+    float corr[2], base[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       mn[r] = fmaxf(mn[r], __shfl_xor_sync(0xffffffffu, mn[r], 1));
       mn[r] = fmaxf(mn[r], __shfl_xor_sync(0xffffffffu, mn[r], 2));
-      corr[r] = exp2f(mx[r] - mn[r]);                               // (key 0 is visible to every row: finite)
+      corr[r] = ex2((mx[r] - mn[r]) * sc);                          // (key 0 is visible to every row: mn is finite)
+      base[r] = mn[r] * sc;
       mx[r] = mn[r];
     }
     float sum[2] = {0.f, 0.f};
@@ -428,7 +448,7 @@ __global__ void __launch_bounds__(256) mla_flash_kernel(const __grid_constant__ 
       float e4[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        e4[e] = exp2f(s[i][e] - mn[e >> 1]);
+        e4[e] = ex2(fmaf(s[i][e], sc, -base[e >> 1]));
         sum[e >> 1] += e4[e];
       }
       pa[i >> 1][(i & 1) * 2] = pack2(e4[0], e4[1]);
@@ -436,8 +456,10 @@ __global__ void __launch_bounds__(256) mla_flash_kernel(const __grid_constant__ 
     }
 #pragma unroll
     for (int r = 0; r < 2; ++r) l[r] = l[r] * corr[r] + sum[r];
+    if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
 #pragma unroll
-    for (int i = 0; i < NV; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+      for (int i = 0; i < NV; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+    }
     const uint32_t v_row = vd + (lane & 15) * vs_ + ((lane >> 4) << 4);
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks)
@@ -505,7 +527,7 @@ int saber_mla_decode_attn(const saber::MlaParams* p, cudaStream_t s) {
 // Largest value sizes and shared-memory needs the expanded form takes on (the absorbed form has no such limit).
 extern "C" int saber_mla_expand_ok(const saber::MlaParams* p) {
   const bool vp = p->VP == 32 || p->VP == 64 || p->VP == 128 || p->VP == 256;
-  return !p->f32 && vp && p->page == saber::kKeys && ((p->DP | p->RP | p->CP) & 15) == 0 && saber::flash_smem(*p) <= 226 * 1024;
+  return !p->f32 && p->scale > 0.f && vp && p->page == saber::kKeys && ((p->DP | p->RP | p->CP) & 15) == 0 && saber::flash_smem(*p) <= 226 * 1024;
 }
 
 int saber_mla_expand_attn(const saber::MlaParams* p, cudaStream_t s) {

@@ -254,7 +254,7 @@ class StackModel:
         if decode or M < 64 or self.k_exp is None:
             return False
         p = N.MlaParams()
-        p.f32, p.page, p.VP, p.DP, p.RP, p.CP = int(self.f32), self.cfg.page_tokens, m.vdim_pad, m.dim_pad, m.rot_pad, m.rank_pad
+        p.f32, p.page, p.VP, p.DP, p.RP, p.CP, p.scale = int(self.f32), self.cfg.page_tokens, m.vdim_pad, m.dim_pad, m.rot_pad, m.rank_pad, m.scale
         return bool(N.lib().saber_mla_expand_ok(C.byref(p)))
 
     def _splits(self, M: int, decode: bool) -> int:

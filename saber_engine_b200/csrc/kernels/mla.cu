@@ -304,7 +304,7 @@ extern "C" int saber_mla_launch(const saber::MlaParams* p, cudaStream_t stream) 
   if (p->M <= 0 || p->C > p->CP || p->R > p->RP || (p->R & 1) || p->CP > 128 * kRowMaxC || p->D > 1024 || p->splits < 1 || p->splits > 64 ||
       p->q_eff == nullptr || p->cache == nullptr)
     return static_cast<int>(cudaErrorInvalidValue);
-  if (p->expand ? (p->k_exp == nullptr || p->v_exp == nullptr || !saber_mla_expand_ok(p)) : (p->o_part == nullptr || p->ml == nullptr))
+  if (p->expand ? (p->k_exp == nullptr || p->v_exp == nullptr || saber_mla_expand_ok(p) < p->expand) : (p->o_part == nullptr || p->ml == nullptr))
     return static_cast<int>(cudaErrorInvalidValue);
   return p->f32 ? mla_go<float>(*p, stream) : mla_go<__nv_bfloat16>(*p, stream);
 }

@@ -20,8 +20,8 @@ struct MlaParams {
   float* o_part;              // scratch [M][H][splits][CP] (absorbed form)
   float* ml;                  // scratch [M][H][splits][2]
   // expanded form (prompt portions, bf16): keys and values of the pages this step sees, in physical page order
-  void* k_exp;                // [n_blocks][H][page][DP + RP]
-  void* v_exp;                // [n_blocks][H][page][VP]
+  void* k_exp;                // [n_blocks][H][page][DP + RP]; expand = 2: tiles [n_blocks][H][ceil((DP + RP) / 64)][page][64]
+  void* v_exp;                // [n_blocks][H][page][VP]; expand = 2: transposed [n_blocks][H][VP][page]
   const int32_t* slot_map;    // [M] page * page_tokens + offset, -1: padding row
   const int32_t* pos;         // [M]
   const int32_t* cu_rows;     // [nseq + 1]
@@ -31,7 +31,7 @@ struct MlaParams {
   int out_k0;
   int M, nseq, H, D, R, V, C, CP, RP, DP, VP, page, n_blocks, max_blocks, splits;
   int f32;                    // element type of cache, weights and q_eff: fp32 or bf16
-  int expand;                 // 1: expanded form
+  int expand;                 // expanded form: 1 mma.sync, 2 tcgen05; 0: absorbed form
   int max_rows;               // rows one sequence may bring
   float scale, eps;
   uint32_t* err;

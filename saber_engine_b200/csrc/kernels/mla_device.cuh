@@ -64,3 +64,6 @@ template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.as
 int saber_mla_decode_attn(const saber::MlaParams* p, cudaStream_t stream);
 int saber_mla_expand_attn(const saber::MlaParams* p, cudaStream_t stream);
 bool saber_mla_decode_ok(const saber::MlaParams* p);
+// mla_flash_tc.cu
+bool saber_mla_flash_tc_ok(const saber::MlaParams* p);
+int saber_mla_flash_tc(const saber::MlaParams* p, cudaStream_t stream);

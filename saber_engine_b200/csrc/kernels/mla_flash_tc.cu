@@ -1,0 +1,295 @@
+// Causal attention of prompt portions over expanded keys and values, on tcgen05.
+//
+// A CTA owns 128 query rows of one head and walks the keys 128 (two pages) at a time.
+//   warp 0     bulk copies: key tiles [k-block of 64][128 keys][128 bytes] and transposed value tiles
+//              [page][value row][64 keys], both stored swizzled by the expand kernel, two stages each
+//   warp 1     one lane issues S = Q K^T into one of two 128-column score buffers, a tile ahead of the softmax,
+//              and O += P V with P in tensor memory
+//   warps 2-5  softmax, a query row per thread: scores from tensor memory, running maximum, bf16 probabilities
+//              back to tensor memory.  O is rescaled only when a row's maximum has grown by more than 2^8 since the
+//              factor in use was chosen (the factor cancels in the division at the end).
+#include "launch.cuh"
+#include "mla_device.cuh"
+
+namespace saber {
+
+constexpr int kTcThreads = 192;
+constexpr int kTcKeys = 128;
+constexpr float kTcLog2e = 1.4426950408889634f;
+constexpr float kTcSlack = 8.f;
+
+__device__ __forceinline__ void mma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "}\n" ::"r"(d_tmem),
+      "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+
+// grid (query tiles of the longest possible portion, H, nseq)
+__global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_constant__ MlaParams p) {
+  pdl_wait();
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ uint64_t bars[16];
+  __shared__ uint32_t tmem_base_s;
+  const int h = blockIdx.y, j = blockIdx.z;
+  const int r0 = p.cu_rows[j], nrows = p.cu_rows[j + 1] - r0;
+  const int tiles = (nrows + 127) / 128;
+  if (static_cast<int>(blockIdx.x) >= tiles) return;
+  const int qt = tiles - 1 - static_cast<int>(blockIdx.x);          // long rows of keys first
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int DK = p.DP + p.RP, KB = (DK + 63) >> 6, VP = p.VP;
+  const int m0 = r0 + qt * 128, rows = min(128, nrows - qt * 128);
+  const int pos0 = p.kv_len[j] - nrows + qt * 128;                  // position of the tile's first row
+  const int keys = pos0 + rows;
+  const int blocks = (keys + kTcKeys - 1) / kTcKeys;
+  const uint32_t q_s = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  const uint32_t kbytes = static_cast<uint32_t>(KB) * 16384u, vbytes = static_cast<uint32_t>(VP) * 256u;
+  const uint32_t k_s = q_s + kbytes, v_s = k_s + 2 * kbytes;
+  const uint32_t bar = smem_u32(bars);
+  const uint32_t kfull = bar, kfree = bar + 16, vfull = bar + 32, vfree = bar + 48, sfull = bar + 64, sfree = bar + 80, pfull = bar + 96,
+                 odone = bar + 104, bend = bar + 112;
+
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(kfull + 8 * i, 1);
+      mbar_init(kfree + 8 * i, 1);
+      mbar_init(vfull + 8 * i, 1);
+      mbar_init(vfree + 8 * i, 1);
+      mbar_init(sfull + 8 * i, 1);
+      mbar_init(sfree + 8 * i, 4);
+    }
+    mbar_init(pfull, 4);
+    mbar_init(odone, 1);
+    mbar_init(bend, 1);
+    mbar_init_fence();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_s), 512);
+    tmem_relinquish();
+  }
+  // query tile, swizzled; columns past DK and rows past the live ones are zeros
+  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q_eff) + (static_cast<size_t>(m0) * p.H + h) * DK;
+  for (int r = warp; r < 128; r += 6)
+    for (int c = lane; c < KB * 8; c += 32) {
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (r < rows && c * 8 < DK) v = *reinterpret_cast<const uint4*>(qg + static_cast<size_t>(r) * p.H * DK + c * 8);
+      asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(q_s + (c >> 3) * 16384 + sw128_offset(r, (c & 7) * 16)), "r"(v.x), "r"(v.y),
+                   "r"(v.z), "r"(v.w) : "memory");
+    }
+  fence_proxy_async_smem();
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tm = tmem_base_s, tm_o = tm + 256, tm_p = tm + 384;
+
+  if (warp == 0) {
+    // ---------------------------------------------------------------- copies
+    if (lane == 0) {
+      const uint8_t* ke = static_cast<const uint8_t*>(p.k_exp);
+      const uint8_t* ve = static_cast<const uint8_t*>(p.v_exp);
+      const size_t kpage = static_cast<size_t>(KB) * 8192, vpage = static_cast<size_t>(VP) * 128;
+      const int last = (keys - 1) / 64;
+      int b = 0;
+      bool ok = true;
+      for (; b < blocks; ++b) {
+        const int s = b & 1;
+        const uint32_t ph = ((b >> 1) & 1) ^ 1;                     // of the use before this one
+        size_t at[2];                                               // (a missing second page: the first again, its keys are masked)
+        at[0] = static_cast<size_t>(mla_page_at(p, j, b * 2)) * p.H + h;
+        at[1] = b * 2 + 1 <= last ? static_cast<size_t>(mla_page_at(p, j, b * 2 + 1)) * p.H + h : at[0];
+        if (b >= 2 && !mbar_wait(kfree + 8 * s, ph, p.err, kErrWaitEmpty)) { ok = false; break; }
+        mbar_arrive_expect_tx(kfull + 8 * s, kbytes);
+        for (int kb = 0; kb < KB; ++kb)
+          for (int g = 0; g < 2; ++g)
+            bulk_g2s(k_s + s * kbytes + kb * 16384 + g * 8192, ke + at[g] * kpage + static_cast<size_t>(kb) * 8192, 8192, kfull + 8 * s);
+        if (b >= 2 && !mbar_wait(vfree + 8 * s, ph, p.err, kErrWaitEmpty)) {
+          mbar_wait(kfull + 8 * s, (b >> 1) & 1, p.err, kErrWaitDrain);
+          ok = false;
+          break;
+        }
+        mbar_arrive_expect_tx(vfull + 8 * s, vbytes);
+        for (int g = 0; g < 2; ++g) bulk_g2s(v_s + s * vbytes + g * (vbytes >> 1), ve + at[g] * vpage, vbytes >> 1, vfull + 8 * s);
+      }
+      if (!ok)                                                      // do not leave while an own copy is in flight
+        for (int i = max(0, b - 2); i < b; ++i) {
+          mbar_wait(kfull + 8 * (i & 1), (i >> 1) & 1, p.err, kErrWaitDrain);
+          mbar_wait(vfull + 8 * (i & 1), (i >> 1) & 1, p.err, kErrWaitDrain);
+        }
+    }
+  } else if (warp == 1) {
+    // ---------------------------------------------------------------- MMA issuer
+    if (lane == 0) {
+      const uint32_t id_s = make_idesc(kCFmtF32, kFmtBF16, kFmtBF16, 128, 128);
+      const uint32_t id_o = make_idesc(kCFmtF32, kFmtBF16, kFmtBF16, 128, static_cast<uint32_t>(VP));
+      const int steps = DK >> 4;
+      auto score = [&](int b) -> bool {                             // S of block b
+        const int s = b & 1;
+        if (!mbar_wait(kfull + 8 * s, (b >> 1) & 1, p.err, kErrWaitReady)) return false;
+        if (b >= 2 && !mbar_wait(sfree + 8 * s, ((b >> 1) & 1) ^ 1, p.err, kErrWaitReady)) return false;
+        tc_fence_after_sync();
+        for (int t = 0; t < steps; ++t) {
+          const uint32_t off = static_cast<uint32_t>(t >> 2) * 16384u + static_cast<uint32_t>(t & 3) * 32u;
+          mma_f16_ss(tm + s * 128, make_desc_k128(q_s) + (off >> 4), make_desc_k128(k_s + s * kbytes) + (off >> 4), id_s, t != 0 ? 1u : 0u);
+        }
+        mma_commit(sfull + 8 * s);
+        mma_commit(kfree + 8 * s);
+        return true;
+      };
+      bool ok = score(0);
+      for (int b = 0; ok && b < blocks; ++b) {
+        if (b + 1 < blocks && !score(b + 1)) { ok = false; break; }
+        const int s = b & 1;
+        if (!mbar_wait(vfull + 8 * s, (b >> 1) & 1, p.err, kErrWaitReady) || !mbar_wait(pfull, b & 1, p.err, kErrWaitReady)) { ok = false; break; }
+        tc_fence_after_sync();
+        for (int t = 0; t < 8; ++t) {
+          const uint32_t off = static_cast<uint32_t>(t >> 2) * (vbytes >> 1) + static_cast<uint32_t>(t & 3) * 32u;
+          mma_bf16_ts(tm_o, tm_p + t * 8, make_desc_k128(v_s + s * vbytes) + (off >> 4), id_o, (b != 0 || t != 0) ? 1u : 0u);
+        }
+        mma_commit(odone);
+        mma_commit(vfree + 8 * s);
+      }
+      mma_commit(bend);                                             // everything issued has retired before the tensor memory goes back
+      mbar_wait(bend, 0, p.err, kErrWaitDrain);
+    }
+  } else {
+    // ---------------------------------------------------------------- softmax
+    const int q4 = warp & 3, row = q4 * 32 + lane;
+    const uint32_t lane_off = static_cast<uint32_t>(q4 * 32) << 16;
+    const float sc = p.scale * kTcLog2e;
+    float mx = -INFINITY, used = -INFINITY, l = 0.f;
+    bool ok = true;
+    for (int b = 0; b < blocks; ++b) {
+      const int s = b & 1;
+      // (waits are decided by the warp as a whole: tensor-memory accesses need all its lanes together)
+      ok = __all_sync(0xffffffffu, mbar_wait(sfull + 8 * s, (b >> 1) & 1, p.err, kErrWaitAcc));
+      if (!ok) break;
+      tc_fence_after_sync();
+      float v[128];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        uint32_t r[32];
+        tmem_ld32(tm + lane_off + s * 128 + c * 32, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) v[c * 32 + i] = __uint_as_float(r[i]);
+      }
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(sfree + 8 * s);
+      const int vis = pos0 + row - b * kTcKeys;                     // last visible key of this row inside the block
+      if (b * kTcKeys + kTcKeys - 1 > pos0 + q4 * 32) {
+#pragma unroll
+        for (int i = 0; i < 128; ++i)
+          if (i > vis) v[i] = -INFINITY;
+      }
+      float m4[4] = {mx, mx, mx, mx};
+#pragma unroll
+      for (int i = 0; i < 128; ++i) m4[i & 3] = fmaxf(m4[i & 3], v[i]);
+      mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));         // (key 0 is visible to every row: finite from the first block on)
+      // P and O of the block before are consumed
+      ok = __all_sync(0xffffffffu, b == 0 || mbar_wait(odone, (b - 1) & 1, p.err, kErrWaitAcc));
+      if (!ok) break;
+      const bool grow = b == 0 || (mx - used) * sc > kTcSlack;
+      if (__any_sync(0xffffffffu, grow)) {
+        const float f = (grow && b > 0) ? ex2((used - mx) * sc) : 1.f;
+        if (grow) used = mx;
+        l *= b > 0 ? f : 0.f;
+        if (b > 0) {
+          tc_fence_after_sync();
+          for (int c = 0; c < VP; c += 32) {
+            uint32_t r[32];
+            tmem_ld32(tm_o + lane_off + c, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * f);
+            tmem_st32(tm_o + lane_off + c, r);
+          }
+          tmem_st_wait();
+        }
+      }
+      const float base = used * sc;
+      float sum[4] = {};
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        uint32_t r[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const float a = ex2(fmaf(v[c * 64 + 2 * i], sc, -base)), e = ex2(fmaf(v[c * 64 + 2 * i + 1], sc, -base));
+          sum[i & 3] += a + e;
+          r[i] = pack2(a, e);
+        }
+        tmem_st32(tm_p + lane_off + c * 32, r);
+      }
+      tmem_st_wait();
+      l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(pfull);
+    }
+    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(odone, (blocks - 1) & 1, p.err, kErrWaitAcc));
+    if (ok) {
+      tc_fence_after_sync();
+      const int m = m0 + row;
+      const bool live = row < rows;
+      const float inv = 1.f / l;
+      const float* g = p.x + static_cast<size_t>(live ? m : m0) * p.ldx + p.g_off + h * p.V;
+      const int k0 = p.out_k0 + h * p.V;
+      for (int c = 0; c < VP; c += 32) {
+        uint32_t r[32];
+        __syncwarp();
+        tmem_ld32(tm_o + lane_off + c, r);
+        tmem_ld_wait();
+        if (!live) continue;
+        if ((p.V & 7) == 0) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            if (c + i * 8 >= p.V) break;
+            const float4 ga = *reinterpret_cast<const float4*>(g + c + i * 8), gb = *reinterpret_cast<const float4*>(g + c + i * 8 + 4);
+            const float gg[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
+            float y[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) y[e] = __uint_as_float(r[i * 8 + e]) * inv / (1.f + expf(-gg[e]));
+            operand_store8(p.out, m, k0 + c + i * 8, y);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c + i < p.V) operand_store1(p.out, m, k0 + c + i, __uint_as_float(r[i]) * inv / (1.f + expf(-g[c + i])));
+        }
+      }
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tm, 512);
+}
+
+static int flash_tc_smem(const MlaParams& p) {
+  const int KB = (p.DP + p.RP + 63) / 64;
+  return 3 * KB * 16384 + 2 * p.VP * 256 + 1024;
+}
+
+}  // namespace saber
+
+bool saber_mla_flash_tc_ok(const saber::MlaParams* p) {
+  return !p->f32 && p->scale > 0.f && p->page == 64 && (p->VP == 32 || p->VP == 64 || p->VP == 128) && ((p->DP | p->RP) & 15) == 0 &&
+         saber::flash_tc_smem(*p) <= 226 * 1024;
+}
+
+int saber_mla_flash_tc(const saber::MlaParams* p, cudaStream_t stream) {
+  using namespace saber;
+  static bool ready[64];
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
+  if (!ready[dev]) {
+    const cudaError_t e = cudaFuncSetAttribute(mla_flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    ready[dev] = true;
+  }
+  return static_cast<int>(launch(mla_flash_tc_kernel, dim3((p->max_rows + 127) / 128, p->H, p->nseq), dim3(kTcThreads), flash_tc_smem(*p), stream, 0, *p));
+}

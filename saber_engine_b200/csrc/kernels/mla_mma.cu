@@ -209,6 +209,12 @@ static int decode_mt(const MlaParams& p, int mt, cudaStream_t s) {
 // ------------------------------------------------------------------------------------ expand
 // Work items, dealt round-robin to a resident grid: (two pages of a sequence) x (128 weight rows of W_uk, then of
 // W_uv, then one item that copies the rotated part and clears padding columns).
+// Element of a key row in the tiles of the tcgen05 kernel: [page][head][k-block of 64][64 keys][128 bytes], 16-byte chunks
+// XOR (key & 7).
+__device__ __forceinline__ size_t k_tile_at(const MlaParams& p, int pg, int h, int key, int d) {
+  const int KB = (p.DP + p.RP + 63) >> 6;
+  return ((static_cast<size_t>(pg) * p.H + h) * KB + (d >> 6)) * 4096 + key * 64 + (((((d & 63) >> 3) ^ key) & 7) << 3) + (d & 7);
+}
 constexpr int kExpStride = 144;                    // 64 bf16 + 16 bytes
 constexpr int kExpStage = 2 * 128 * kExpStride;    // latents, weights
 
@@ -245,6 +251,11 @@ __global__ void __launch_bounds__(256) mla_expand_kernel(const __grid_constant__
         const int r = i / p.H, h = i - r * p.H, pg = page[r >> 6];
         if (pg < 0) continue;
         const __nv_bfloat16* src = cache + (static_cast<size_t>(pg) * 64 + (r & 63)) * LD + p.CP;
+        if (p.expand == 2) {
+          for (int c = 0; c < rot8; ++c)
+            *reinterpret_cast<uint4*>(ke + k_tile_at(p, pg, h, r & 63, p.DP + c * 8)) = reinterpret_cast<const uint4*>(src)[c];
+          continue;
+        }
         __nv_bfloat16* d = ke + ((static_cast<size_t>(pg) * p.H + h) * 64 + (r & 63)) * DK;
         for (int c = 0; c < rot8; ++c) reinterpret_cast<uint4*>(d + p.DP)[c] = reinterpret_cast<const uint4*>(src)[c];
         for (int c = p.D; c < p.DP; ++c) d[c] = __float2bfloat16(0.f);
@@ -256,6 +267,7 @@ __global__ void __launch_bounds__(256) mla_expand_kernel(const __grid_constant__
     const bool isk = tile < nk;
     const int n0 = (isk ? tile : tile - nk) * 128, N = p.H * (isk ? p.D : p.V), per_h = isk ? p.D : p.V;
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(isk ? p.w_uk : p.w_uv);
+    const bool vt = !isk && p.expand == 2;         // values transposed: weight rows are the rows of the product
     auto fetch = [&](int c, int buf) {
       const uint32_t dst = base + buf * kExpStage;
       for (int i = threadIdx.x; i < 2048; i += 256) {
@@ -276,7 +288,8 @@ __global__ void __launch_bounds__(256) mla_expand_kernel(const __grid_constant__
       if (c + 2 < kc) fetch(c + 2, (c + 2) % 3);
       if (c + 2 < kc) cp_wait<2>(); else if (c + 1 < kc) cp_wait<1>(); else cp_wait<0>();
       __syncthreads();
-      const uint32_t a_s = base + (c % 3) * kExpStage, b_s = a_s + 128 * kExpStride;
+      const uint32_t lat_s = base + (c % 3) * kExpStage, wgt_s = lat_s + 128 * kExpStride;
+      const uint32_t a_s = vt ? wgt_s : lat_s, b_s = vt ? lat_s : wgt_s;
 #pragma unroll
       for (int ks = 0; ks < 4; ++ks) {
         uint32_t a[2][4];
@@ -294,6 +307,35 @@ __global__ void __launch_bounds__(256) mla_expand_kernel(const __grid_constant__
         }
       }
       __syncthreads();
+    }
+    if (p.expand == 2) {
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int r = wm * 32 + t * 16 + (lane >> 2) + half * 8;
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const int q = wn * 64 + i * 8 + (lane & 3) * 2;
+            const int n = n0 + (vt ? r : q), key = vt ? q : r, pg = page[key >> 6];
+            if (pg < 0 || n >= N) continue;
+            const int h = n / per_h, d = n - h * per_h;
+            const float x = acc[t][i][half * 2], y = acc[t][i][half * 2 + 1];
+            if (vt) {
+              __nv_bfloat16* o = ve + ((static_cast<size_t>(pg) * p.H + h) * p.VP + d) * 64 + (((((key & 63) >> 3) ^ d) & 7) << 3) + (key & 7);
+              *reinterpret_cast<uint32_t*>(o) = pack2(x, y);
+            } else if ((per_h & 1) == 0) {
+              *reinterpret_cast<uint32_t*>(ke + k_tile_at(p, pg, h, key & 63, d)) = pack2(x, y);
+            } else {
+              ke[k_tile_at(p, pg, h, key & 63, d)] = __float2bfloat16(x);
+              if (n + 1 < N) {
+                const int h1 = (n + 1) / per_h;
+                ke[k_tile_at(p, pg, h1, key & 63, n + 1 - h1 * per_h)] = __float2bfloat16(y);
+              }
+            }
+          }
+        }
+      continue;
     }
     const bool even = (per_h & 1) == 0;
 #pragma unroll
@@ -507,6 +549,7 @@ static int flash_go(const MlaParams& p, cudaStream_t stream) {
     ready[dev] = true;
   }
   cudaError_t e = launch(mla_expand_kernel, dim3(2 * 148), dim3(256), 3 * kExpStage, stream, 0, p);
+  if (e == cudaSuccess && p.expand == 2) return saber_mla_flash_tc(&p, stream);
   if (e == cudaSuccess)
     e = launch(mla_flash_kernel<NV>, dim3((p.max_rows + kQRows - 1) / kQRows, p.H, p.nseq), dim3(256), flash_smem(p), stream, 0, p);
   return static_cast<int>(e);
@@ -524,9 +567,11 @@ int saber_mla_decode_attn(const saber::MlaParams* p, cudaStream_t s) {
   return p->CP <= 128 ? saber::decode_mt<2>(*p, mt, s) : p->CP <= 256 ? saber::decode_mt<4>(*p, mt, s) : saber::decode_mt<8>(*p, mt, s);
 }
 
-// Largest value sizes and shared-memory needs the expanded form takes on (the absorbed form has no such limit).
+// Value sizes and shared-memory needs the expanded form takes on: 2 on tcgen05, 1 on mma.sync, 0 not at all (the
+// absorbed form has no such limit).
 extern "C" int saber_mla_expand_ok(const saber::MlaParams* p) {
   const bool vp = p->VP == 32 || p->VP == 64 || p->VP == 128 || p->VP == 256;
+  if (saber_mla_flash_tc_ok(p) && (p->CP & 15) == 0) return 2;
   return !p->f32 && p->scale > 0.f && vp && p->page == saber::kKeys && ((p->DP | p->RP | p->CP) & 15) == 0 && saber::flash_smem(*p) <= 226 * 1024;
 }
 

@@ -28,9 +28,12 @@ from .step import BlobLayout, Bucket, finish_bucket, head_outputs, plp_outputs, 
 class StackModel:
     def __init__(self, cfg: StackConfig, device="cuda", max_seqs: int = 8, max_ctx: Optional[int] = None, kv_blocks: Optional[int] = None,
                  weights: Optional[SW.StackWeights] = None, seed: int = 0, dtype: torch.dtype = torch.bfloat16, fuse: bool = True,
-                 expand_bytes: int = 24 << 30, race_check: str = "off", n_slots: Optional[int] = None):
+                 expand_bytes: int = 24 << 30, race_check: str = "off", attn_impl: str = "tc"):
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("dtype must be bfloat16 or float32")
+        if attn_impl not in ("tc", "mma"):
+            raise ValueError("attn_impl must be 'tc' or 'mma'")
+        self.attn_impl = attn_impl
         if race_check not in ("off", "shadow"):
             raise ValueError("race_check must be 'off' or 'shadow'")
         self.cfg, self.tp, self.rank, self.comm = cfg, 1, 0, None
@@ -65,7 +68,7 @@ class StackModel:
         lat = [l.mixer for l in cfg.layers if isinstance(l.mixer, LatentMixer)]
         tokens = self.kv_blocks * cfg.page_tokens
         if lat and not self.f32 and tokens * cfg.expanded_token_bytes() <= expand_bytes:
-            self.k_exp = torch.zeros(tokens * max(m.heads * (m.dim_pad + m.rot_pad) for m in lat), dtype=dtype, device=dev)
+            self.k_exp = torch.zeros(tokens * max(m.heads * m.key_tile for m in lat), dtype=dtype, device=dev)
             self.v_exp = torch.zeros(tokens * max(m.heads * m.vdim_pad for m in lat), dtype=dtype, device=dev)
         self.buckets: dict = {}
         self.stream = torch.cuda.Stream(device=dev)
@@ -249,13 +252,14 @@ class StackModel:
             wk["ml"] = f32(M * wk["splits"] * mx(2 * m.heads for m in absorbed))
         return wk
 
-    def _expanded(self, m: LatentMixer, M: int, decode: bool) -> bool:
+    def _expanded(self, m: LatentMixer, M: int, decode: bool) -> int:
         """Prompt portions attend over expanded keys and values; decoding, short portions and fp32 in the latent space."""
         if decode or M < 64 or self.k_exp is None:
-            return False
+            return 0
         p = N.MlaParams()
         p.f32, p.page, p.VP, p.DP, p.RP, p.CP, p.scale = int(self.f32), self.cfg.page_tokens, m.vdim_pad, m.dim_pad, m.rot_pad, m.rank_pad, m.scale
-        return bool(N.lib().saber_mla_expand_ok(C.byref(p)))
+        form = N.lib().saber_mla_expand_ok(C.byref(p))       # 2: tcgen05, 1: mma.sync, 0: neither takes these sizes
+        return form if self.attn_impl == "tc" else min(form, 1)
 
     def _splits(self, M: int, decode: bool) -> int:
         """Key splits of the absorbed attention: fill the SMs once."""
@@ -287,7 +291,7 @@ class StackModel:
         p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
         p.H, p.D, p.R, p.V, p.C, p.CP, p.RP, p.DP, p.VP = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.rank_pad, m.rot_pad, m.dim_pad, m.vdim_pad
         p.page, p.n_blocks, p.max_blocks = self.cfg.page_tokens, self.kv_blocks, self.max_blocks
-        p.splits, p.f32, p.expand, p.max_rows = wk["splits"], int(self.f32), int(self._expanded(m, M, decode)), 1 if decode else M
+        p.splits, p.f32, p.expand, p.max_rows = wk["splits"], int(self.f32), self._expanded(m, M, decode), 1 if decode else M
         p.scale, p.eps, p.err = m.scale, self.cfg.eps, self.scratch.err.data_ptr()
         return p
 

@@ -100,8 +100,12 @@ class LatentMixer:
     def page_token_bytes(self, elem: int) -> int:
         return elem * (self.rank_pad + self.rot_pad)
 
+    @property
+    def key_tile(self) -> int:        # an expanded key in whole 64-wide tiles
+        return (self.dim_pad + self.rot_pad + 63) // 64 * 64
+
     def expanded_token_bytes(self, elem: int) -> int:
-        return elem * self.heads * (self.dim_pad + self.rot_pad + self.vdim_pad)
+        return elem * self.heads * (self.key_tile + self.vdim_pad)
 
 
 @dataclass(frozen=True)

@@ -163,9 +163,9 @@ def test_expanded_and_absorbed_prompts_agree():
     t = R.tensors(cfg, seed=9)
     toks = R.tokens(cfg, 333)
     want = O.Oracle(cfg, t).forward(toks)
-    for kw in ({}, {"expand_bytes": 0}):                         # without the scratch pages prompts stay in the latent space
+    for kw, form in (({}, 2), ({"attn_impl": "mma"}, 1), ({"expand_bytes": 0}, 0)):      # without the scratch pages prompts stay in the latent space
         eng = R.engine(cfg, t, BF16, **kw)
-        assert (eng.model.k_exp is None) == bool(kw)
+        assert eng.model._expanded(eng.model.cfg.layers[0].mixer, 256, False) == form
         assert R.error(R.feed(eng, "r", toks, [333]), want) < R.TOL[BF16]
         assert R.error(R.feed(eng, "r", toks, [70, 130, 2]), want) < R.TOL[BF16]
 
@@ -212,6 +212,22 @@ def test_one_key_far_away_and_at_page_borders(dtype, place):
     assert R.error(R.feed(eng, "r", toks, [n])[-1:], want[-1:]) < tol                   # asked in the prompt
     assert R.error(R.feed(eng, "r", toks, [n - 1, 1])[-1:], want[-1:]) < tol            # asked by a decoded token
     assert R.error(R.feed(eng, "r", toks, [place + 1, 1, 200, 255, 1])[-1:], want[-1:]) < tol
+
+
+@pytest.mark.parametrize("scale", [0.05, 1.5])
+@pytest.mark.parametrize("lens", [(300,), (129, 64, 1, 257), (128, 640)])
+def test_prompt_attention_over_growing_scores(lens, scale):
+    """Scores that rise along the keys (the running maximum moves in every block) and unequal prompts side by side."""
+    cfg = R.config([R.latent(heads=3, dim=48, rot_dim=16, vdim=56, kv_rank=80, scale=scale, ff=None)], vocab=800)
+    t = R.tensors(cfg, 5)
+    t["embed"] = (t["embed"].float() * torch.linspace(0.2, 1.0, 800)[:, None]).bfloat16()
+    toks = [sorted(R.tokens(cfg, n, seed=i)) for i, n in enumerate(lens)]
+    orc = O.Oracle(cfg, t)
+    for kw in ({}, {"attn_impl": "mma"}):
+        eng = R.engine(cfg, t, BF16, rungs=(1024,), **kw)
+        got = eng.step([(i, x) for i, x in enumerate(toks)])
+        for g, x in zip(got, toks):
+            assert R.error(g, orc.forward(x)) < 0.06 * max(1.0, scale)
 
 
 def test_keys_reached_by_position_only():

@@ -271,6 +271,29 @@ __device__ __forceinline__ void delta_state_io(float* st, float (&S)[NI][4][2], 
     }
 }
 
+// Pairs of fp32 in one register pair: the two halves of an instruction are two ordinary fp32 operations.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack_f2(float a, float b) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unpack_f2(f32x2 v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma_f2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul_f2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
 constexpr int kScanStages = 4;           // blocks of four tokens in flight
 
 // grid (nseq, H, ceil(VP / 16)), 160 threads: four warps of four value columns (two lane groups of two columns, 16 lanes
@@ -326,15 +349,16 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
     }
     return;
   }
-  float S[NJ][4][2] = {};
+  f32x2 S[NJ][2][2] = {};                          // [64 keys][pair of keys][column]
   float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + vb + cl) * DP;
   if (on) {
 #pragma unroll
     for (int c = 0; c < 2; ++c)
 #pragma unroll
       for (int i = 0; i < NJ; ++i) {
-        const float4 f = *reinterpret_cast<const float4*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4);
-        S[i][0][c] = f.x; S[i][1][c] = f.y; S[i][2][c] = f.z; S[i][3][c] = f.w;
+        const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4);
+        S[i][0][c] = f.x;
+        S[i][1][c] = f.y;
       }
   }
   const int tok = lg >> 2, col = (lg >> 1) & 1;    // whose read-out value this lane keeps (lanes 2i, 2i + 1 share one)
@@ -346,22 +370,35 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
     const float* b = sm + s * kStageWords;
     const float* vrec = b + kKq;
     if (on) {
-      float sk[kBlk][2] = {}, sq[kBlk][2] = {};
+      constexpr bool kHold = NJ <= 2;              // the keys stay in registers for the update
+      f32x2 kr[kHold ? kBlk : 1][kHold ? NJ : 1][2];
+      float sk[kBlk][2], sq[kBlk][2];
 #pragma unroll
-      for (int r = 0; r < kBlk; ++r)
+      for (int r = 0; r < kBlk; ++r) {
+        f32x2 a[2] = {}, c[2] = {};
 #pragma unroll
         for (int i = 0; i < NJ; ++i) {
-          const float4 k4 = *reinterpret_cast<const float4*>(b + r * DP + i * 64 + lg * 4);
-          const float4 q4 = *reinterpret_cast<const float4*>(b + (kBlk + r) * DP + i * 64 + lg * 4);
-          const float ka[4] = {k4.x, k4.y, k4.z, k4.w}, qa[4] = {q4.x, q4.y, q4.z, q4.w};
+          const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(b + r * DP + i * 64 + lg * 4);
+          const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(b + (kBlk + r) * DP + i * 64 + lg * 4);
+          if constexpr (kHold) {
+            kr[r][i][0] = k4.x;
+            kr[r][i][1] = k4.y;
+          }
 #pragma unroll
-          for (int e = 0; e < 4; ++e)
-#pragma unroll
-            for (int v = 0; v < 2; ++v) {
-              sk[r][v] = fmaf(S[i][e][v], ka[e], sk[r][v]);
-              sq[r][v] = fmaf(S[i][e][v], qa[e], sq[r][v]);
-            }
+          for (int v = 0; v < 2; ++v) {
+            a[v] = fma_f2(S[i][0][v], k4.x, a[v]);
+            c[v] = fma_f2(S[i][0][v], q4.x, c[v]);
+            a[v] = fma_f2(S[i][1][v], k4.y, a[v]);
+            c[v] = fma_f2(S[i][1][v], q4.y, c[v]);
+          }
         }
+#pragma unroll
+        for (int v = 0; v < 2; ++v) {
+          const float2 x = unpack_f2(a[v]), y = unpack_f2(c[v]);
+          sk[r][v] = x.x + x.y;
+          sq[r][v] = y.x + y.y;
+        }
+      }
 #pragma unroll
       for (int o = 1; o < 16; o <<= 1)
 #pragma unroll
@@ -415,27 +452,35 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
         o = tok == i ? t : o;
       }
       if ((lg & 1) == 0 && blk * kBlk + tok < n) out[blk * out_step] = o;
-#pragma unroll
-      for (int jj = 0; jj < kBlk; ++jj) {          // D_4j is where the recurrence left it
-        u[jj][0] *= dl[jj];
-        u[jj][1] *= dl[jj];
-      }
+      const f32x2 G2 = pack_f2(G, G);
 #pragma unroll
       for (int i = 0; i < NJ; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) { S[i][e][0] *= G; S[i][e][1] *= G; }
+        for (int e = 0; e < 2; ++e) {
+          S[i][e][0] = mul_f2(S[i][e][0], G2);
+          S[i][e][1] = mul_f2(S[i][e][1], G2);
+        }
 #pragma unroll
-      for (int r = 0; r < kBlk; ++r)
+      for (int r = 0; r < kBlk; ++r) {             // D_4r is where the recurrence left it
+        const float w0 = u[r][0] * dl[r], w1 = u[r][1] * dl[r];
+        const f32x2 u0 = pack_f2(w0, w0), u1 = pack_f2(w1, w1);
 #pragma unroll
         for (int i = 0; i < NJ; ++i) {
-          const float4 k4 = *reinterpret_cast<const float4*>(b + r * DP + i * 64 + lg * 4);
-          const float ka[4] = {k4.x, k4.y, k4.z, k4.w};
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            S[i][e][0] = fmaf(u[r][0], ka[e], S[i][e][0]);
-            S[i][e][1] = fmaf(u[r][1], ka[e], S[i][e][1]);
+          f32x2 ka, kb;
+          if constexpr (kHold) {
+            ka = kr[r][i][0];
+            kb = kr[r][i][1];
+          } else {
+            const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(b + r * DP + i * 64 + lg * 4);
+            ka = k4.x;
+            kb = k4.y;
           }
+          S[i][0][0] = fma_f2(u0, ka, S[i][0][0]);
+          S[i][0][1] = fma_f2(u1, ka, S[i][0][1]);
+          S[i][1][0] = fma_f2(u0, kb, S[i][1][0]);
+          S[i][1][1] = fma_f2(u1, kb, S[i][1][1]);
         }
+      }
     }
     __syncwarp();
     if (lane == 0) mbar_arrive(bar_free + 8 * s);  // this warp is done with the stage
@@ -445,7 +490,7 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
     for (int c = 0; c < 2; ++c)
 #pragma unroll
       for (int i = 0; i < NJ; ++i)
-        *reinterpret_cast<float4*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4) = make_float4(S[i][0][c], S[i][1][c], S[i][2][c], S[i][3][c]);
+        *reinterpret_cast<ulonglong2*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4) = make_ulonglong2(S[i][0][c], S[i][1][c]);
   }
 }
 

@@ -13,6 +13,7 @@ Parity: the reference's vision executor (`crates/saber-kernels/hip/vision.hip:1-
 from __future__ import annotations
 
 import ctypes as C
+import gc
 import math
 from typing import Optional, Sequence
 
@@ -198,8 +199,17 @@ class VisionTowerGPU:
             g = torch.cuda.CUDAGraph()
             # thread-local capture mode: the engine's step loop keeps synchronising its own stream in
             # another thread while an image of a new shape is captured here
-            with torch.cuda.graph(g, stream=side, capture_error_mode="thread_local"):
-                self._run(px, Lr, meta, ob, False)
+            # (no garbage collection while capturing: an unreachable model of this thread would give device memory,
+            # events or graphs back in the middle of it, which ends the capture)
+            gc.collect()
+            was = gc.isenabled()
+            gc.disable()
+            try:
+                with torch.cuda.graph(g, stream=side, capture_error_mode="thread_local"):
+                    self._run(px, Lr, meta, ob, False)
+            finally:
+                if was:
+                    gc.enable()
             cur.wait_stream(side)
             if len(self._graphs) >= self.max_graphs:
                 self._graphs.pop(next(iter(self._graphs)))

@@ -407,3 +407,20 @@ def test_trace_replay_process(tmp_path, dtype):
     for k, w in want.items():
         got = torch.from_numpy(np.fromfile(tmp_path / f"{k}.f32", dtype="<f4").reshape(-1, cfg["vocab"]))
         assert R.error(got, w) < R.TOL[getattr(torch, dtype)]
+
+
+def test_engine_command_serves_a_model_folder(tmp_path):
+    """`saber engine --engine-config DIR`: plan, weights, scheduler; greedy ids of the oracle."""
+    from saber_engine_b200.cli.main import build_engine, make_parser
+    cfg = R.CASES["no_loop"]
+    t = R.tensors(cfg, 15)
+    R.write_model(tmp_path / "m", cfg, t)
+    a = make_parser().parse_args(["engine", "--engine-config", str(tmp_path / "m"), "--engine-dtype", "float32", "--engine-max-ctx", "512",
+                                  "--engine-max-seqs", "2", "--engine-prefill-rows", "64", "--engine-decode-batches", "1,2",
+                                  "--engine-budget-mib", "12000", "--engine-race-check", "shadow"])
+    ex, sched = build_engine(a)
+    prompts = [R.tokens(cfg, n, seed=50 + n) for n in (5, 70, 33)]
+    want = [O.Oracle(cfg, t).greedy(p, 8)[0] for p in prompts]
+    assert [g[0] for g in _greedy(sched, prompts, 8)] == want
+    b = ex.model.buckets[("decode", 2, 1)]
+    assert int((b.digests.cpu() != 0).sum()) >= len(cfg["layers"])

@@ -18,24 +18,11 @@
 #include "delta.h"
 #include "launch.cuh"
 #include "ptx_sm100.cuh"
+#include "scan_records.cuh"
 
 namespace saber {
 
-__device__ __forceinline__ float warp_sum_f(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-__device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplus_f32(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
-
-// sequence of a row (-1: a padding row), and whether its slot may be used
-__device__ __forceinline__ int seq_of_row(const int32_t* cu, int nseq, int m) {
-  for (int j = 0; j < nseq; ++j)
-    if (m < cu[j + 1]) return m >= cu[j] ? j : -1;
-  return -1;
-}
+// slot of a sequence (< 0: none)
 __device__ __forceinline__ int delta_slot(const DeltaParams& p, int j) {
   const int s = p.slots[j];
   if (s >= p.n_slots) {
@@ -58,13 +45,6 @@ __device__ __forceinline__ float conv_silu(const DeltaParams& p, const float* hi
   return silu_f32(acc);
 }
 
-constexpr int kBlk = 4;                  // tokens per block
-constexpr int kPairs = 16;               // dot products per block: k_j . k_i (j < i: 6), k_j . q_i (j <= i: 10)
-__host__ __device__ constexpr int kk_at(int i, int j) { return i * (i - 1) / 2 + j; }
-__host__ __device__ constexpr int kq_at(int i, int j) { return 6 + i * (i + 1) / 2 + j; }
-
-// Blocks of sequence j occupy the slots from (first row / 4) + j on: disjoint for all sequences of a step.
-__device__ __forceinline__ int block_slot(int r0, int j, int c) { return (r0 >> 2) + j + c; }
 __device__ __forceinline__ bool block_of_slot(const DeltaParams& p, int slot, int& j, int& c) {
   for (j = 0; j < p.nseq; ++j) {
     const int r0 = p.cu_rows[j], n = p.cu_rows[j + 1] - r0;
@@ -115,13 +95,6 @@ __device__ __forceinline__ void conv_silu4(const DeltaParams& p, const float* hi
   for (int r = 0; r < kBlk; ++r) y[r] = r < rows ? silu_f32(acc[r]) : 0.f;
 }
 
-// Scratch records of a block, each contiguous (one bulk copy):
-//   key head   k rows [4][DP] | q rows [4][DP] | 16 dot products
-//   value head, per 16 columns   v [4][16] | beta [4] | g [4]
-// Missing tokens of the last block are written as k = q = v = beta = 0, g = 1.
-__host__ __device__ constexpr int kq_words(int DP) { return 2 * kBlk * DP + kPairs; }
-constexpr int kCols = 16;                // value columns of a scan CTA
-constexpr int kVWords = kBlk * kCols + 2 * kBlk;
 
 // grid (blocks, ceil((HK + H) / 4)), 128 threads; a warp per item: key heads (q, k and their dot products), value heads
 template <int NI, int TAPS>
@@ -300,7 +273,8 @@ constexpr int kScanStages = 4;           // blocks of four tokens in flight
 // along the keys), each at its own pace, and a warp whose first lane keeps the copies going
 constexpr int kScanThreads = 160;
 
-template <int NJ>
+// kCorrect = false: u_i = beta_i v_i, the rule without correction.
+template <int NJ, bool kCorrect>
 __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_constant__ DeltaParams p) {
   constexpr int DP = NJ * 64;
   constexpr int kKq = kq_words(DP);
@@ -364,6 +338,7 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
   const int tok = lg >> 2, col = (lg >> 1) & 1;    // whose read-out value this lane keeps (lanes 2i, 2i + 1 share one)
   float* out = p.o + (static_cast<size_t>(r0 + tok) * p.H + h) * p.VP + vb + cl + col;
   const size_t out_step = static_cast<size_t>(kBlk) * p.H * p.VP;
+  const float skip = !kCorrect && p.skip != nullptr ? p.skip[h] : 0.f;
   for (int blk = 0; blk < blocks; ++blk) {
     const int s = blk % kScanStages;
     if (!mbar_wait(bar + 8 * s, (blk / kScanStages) & 1, p.err, kErrWaitFull)) break;
@@ -386,9 +361,11 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
           }
 #pragma unroll
           for (int v = 0; v < 2; ++v) {
-            a[v] = fma_f2(S[i][0][v], k4.x, a[v]);
+            if constexpr (kCorrect) {
+              a[v] = fma_f2(S[i][0][v], k4.x, a[v]);
+              a[v] = fma_f2(S[i][1][v], k4.y, a[v]);
+            }
             c[v] = fma_f2(S[i][0][v], q4.x, c[v]);
-            a[v] = fma_f2(S[i][1][v], k4.y, a[v]);
             c[v] = fma_f2(S[i][1][v], q4.y, c[v]);
           }
         }
@@ -399,12 +376,14 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
           sq[r][v] = y.x + y.y;
         }
       }
+      if constexpr (kCorrect) {
 #pragma unroll
-      for (int o = 1; o < 16; o <<= 1)
+        for (int o = 1; o < 16; o <<= 1)
 #pragma unroll
-        for (int r = 0; r < kBlk; ++r)
+          for (int r = 0; r < kBlk; ++r)
 #pragma unroll
-          for (int v = 0; v < 2; ++v) sk[r][v] += __shfl_xor_sync(0xffffffffu, sk[r][v], o);
+            for (int v = 0; v < 2; ++v) sk[r][v] += __shfl_xor_sync(0xffffffffu, sk[r][v], o);
+      }
       // read-out values by halving exchange (4 + 2 + 1 + 1 shuffles)
       float mine;
       {
@@ -435,18 +414,25 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const __grid_c
       for (int i = 0; i < kBlk; ++i) {
         const float2 v = *reinterpret_cast<const float2*>(vrec + i * kCols + cl);
         G *= g[i];
-        float a0 = v.x - G * sk[i][0], a1 = v.y - G * sk[i][1];
+        float a0 = v.x, a1 = v.y;
+        if constexpr (kCorrect) {
+          a0 -= G * sk[i][0];
+          a1 -= G * sk[i][1];
+        }
 #pragma unroll
         for (int jj = 0; jj < i; ++jj) {
           dl[jj] *= g[i];                          // D_ij
-          const float w = dl[jj] * pr[kk_at(i, jj)];
-          a0 = fmaf(-w, u[jj][0], a0);
-          a1 = fmaf(-w, u[jj][1], a1);
+          if constexpr (kCorrect) {
+            const float w = dl[jj] * pr[kk_at(i, jj)];
+            a0 = fmaf(-w, u[jj][0], a0);
+            a1 = fmaf(-w, u[jj][1], a1);
+          }
         }
         dl[i] = 1.f;
         u[i][0] = beta[i] * a0;
         u[i][1] = beta[i] * a1;
         float t = G * mine;
+        if constexpr (!kCorrect) t = fmaf(skip, col ? v.y : v.x, t);
 #pragma unroll
         for (int jj = 0; jj <= i; ++jj) t = fmaf(dl[jj] * pr[kq_at(i, jj)], col ? u[jj][1] : u[jj][0], t);
         o = tok == i ? t : o;
@@ -635,6 +621,22 @@ static cudaError_t delta_prep(const DeltaParams& p, cudaStream_t stream) {
   return launch(delta_prep_kernel<NI, TAPS>, dim3(p.M / kBlk + p.nseq, (p.HK + p.H + 3) / 4), dim3(128), 0, stream, 0, p);
 }
 
+template <int NJ, bool kCorrect>
+static int delta_scan(const DeltaParams& p, cudaStream_t stream) {
+  constexpr int smem = kScanStages * (kq_words(NJ * 64) + kVWords) * 4;
+  static bool ready[64];
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
+  if (!ready[dev]) {
+    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ, kCorrect>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    ready[dev] = true;
+  }
+  return static_cast<int>(launch(delta_scan_kernel<NJ, kCorrect>, dim3(p.nseq, p.H, (p.VP + kCols - 1) / kCols), dim3(kScanThreads), smem,
+                                 stream, 0, p));
+}
+
 template <int NJ>
 static int delta_go(const DeltaParams& p, bool single, cudaStream_t stream) {
   constexpr int NI = NJ * 2;
@@ -643,20 +645,10 @@ static int delta_go(const DeltaParams& p, bool single, cudaStream_t stream) {
     const int smem = (2 * NI * 32 + 2 * p.VP) * 4;
     return static_cast<int>(launch(delta_step_kernel<NI>, dim3(p.H, p.nseq), dim3(32 * warps), smem, stream, 0, p));
   }
-  const int smem = kScanStages * (kq_words(NI * 32) + kVWords) * 4;
-  static bool ready[64];
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
-  if (!ready[dev]) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    ready[dev] = true;
-  }
-  cudaError_t e = p.taps == 4 ? delta_prep<NI, 4>(p, stream) : delta_prep<NI, 0>(p, stream);
-  if (e == cudaSuccess) e = launch(delta_scan_kernel<NJ>, dim3(p.nseq, p.H, (p.VP + kCols - 1) / kCols), dim3(kScanThreads), smem, stream, 0, p);
-  if (e == cudaSuccess) e = launch(delta_out_kernel, dim3(p.M + p.nseq, (p.H + 7) / 8), dim3(256), 0, stream, 0, p);
-  return static_cast<int>(e);
+  int e = static_cast<int>(p.taps == 4 ? delta_prep<NI, 4>(p, stream) : delta_prep<NI, 0>(p, stream));
+  if (e == 0) e = delta_scan<NJ, true>(p, stream);
+  if (e == 0) e = static_cast<int>(launch(delta_out_kernel, dim3(p.M + p.nseq, (p.H + 7) / 8), dim3(256), 0, stream, 0, p));
+  return e;
 }
 
 }  // namespace saber
@@ -674,6 +666,19 @@ extern "C" int saber_delta_launch(const saber::DeltaParams* p, int single_row, c
     case 256: return delta_go<4>(*p, single_row != 0, stream);
     case 384: return delta_go<6>(*p, single_row != 0, stream);
     case 512: return delta_go<8>(*p, single_row != 0, stream);
+    default: return static_cast<int>(cudaErrorInvalidValue);
+  }
+}
+
+int saber_outer_scan_launch(const saber::DeltaParams* p, cudaStream_t stream) {
+  using namespace saber;
+  switch (p->DP) {
+    case 64: return delta_scan<1, false>(*p, stream);
+    case 128: return delta_scan<2, false>(*p, stream);
+    case 192: return delta_scan<3, false>(*p, stream);
+    case 256: return delta_scan<4, false>(*p, stream);
+    case 384: return delta_scan<6, false>(*p, stream);
+    case 512: return delta_scan<8, false>(*p, stream);
     default: return static_cast<int>(cudaErrorInvalidValue);
   }
 }

@@ -33,6 +33,7 @@ struct DeltaParams {
   int out_k0;
   int M, nseq, H, HK, D, DP, V, VP, taps, n_slots;
   float eps, unit_eps, q_scale;
+  const float* skip;       // [H] or null: the scan without correction adds skip * v to the read-out
   uint32_t* err;
 };
 
@@ -41,3 +42,6 @@ struct DeltaParams {
 // rows = 1: every sequence brings at most one row (one fused launch); else three launches
 extern "C" int saber_delta_launches(int single_row);
 extern "C" int saber_delta_launch(const saber::DeltaParams* p, int single_row, cudaStream_t stream);
+// The scan by itself over records that another kernel has prepared, with the rule S <- g S + beta k v^T (no
+// correction of v by what the state holds): decayed outer products (ssd.cu).
+int saber_outer_scan_launch(const saber::DeltaParams* p, cudaStream_t stream);

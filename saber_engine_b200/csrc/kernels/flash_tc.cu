@@ -1,13 +1,15 @@
-// Causal attention of prompt portions over expanded keys and values, on tcgen05.
+// Causal attention of prompt portions over tiled keys and values, on tcgen05: expanded latents (mla.cu) and
+// grouped-query pages (gqa.cu).
 //
-// A CTA owns 128 query rows of one head and walks the keys 128 (two pages) at a time.
+// A CTA owns 128 query rows of one head and walks the keys its rows can see 128 (two pages) at a time.
 //   warp 0     bulk copies: key tiles [k-block of 64][128 keys][128 bytes] and transposed value tiles
-//              [page][value row][64 keys], both stored swizzled by the expand kernel, two stages each
+//              [page][value row][64 keys], both stored swizzled, two stages each
 //   warp 1     one lane issues S = Q K^T into one of two 128-column score buffers, a tile ahead of the softmax,
 //              and O += P V with P in tensor memory
 //   warps 2-5  softmax, a query row per thread: scores from tensor memory, running maximum, bf16 probabilities
 //              back to tensor memory.  O is rescaled only when a row's maximum has grown by more than 2^8 since the
 //              factor in use was chosen (the factor cancels in the division at the end).
+#include "flash_tc.h"
 #include "launch.cuh"
 #include "mla_device.cuh"
 
@@ -17,6 +19,7 @@ constexpr int kTcThreads = 192;
 constexpr int kTcKeys = 128;
 constexpr float kTcLog2e = 1.4426950408889634f;
 constexpr float kTcSlack = 8.f;
+constexpr float kTcNone = -1e30f;          // no key seen yet
 
 __device__ __forceinline__ void mma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
   asm volatile(
@@ -29,8 +32,11 @@ __device__ __forceinline__ void mma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, ui
       : "memory");
 }
 
+// cap tanh(z s) from 2^(2 z s log2 e): zs is 2 z log2 e.  (Large sums give cap, tiny ones -cap.)
+__device__ __forceinline__ float soft_cap(float s, float zs, float cap) { return cap - __fdividef(2.f * cap, 1.f + ex2(s * zs)); }
+
 // grid (query tiles of the longest possible portion, H, nseq)
-__global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_constant__ MlaParams p) {
+__global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_constant__ FlashParams p) {
   pdl_wait();
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t bars[16];
@@ -41,11 +47,12 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
   if (static_cast<int>(blockIdx.x) >= tiles) return;
   const int qt = tiles - 1 - static_cast<int>(blockIdx.x);          // long rows of keys first
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int DK = p.DP + p.RP, KB = (DK + 63) >> 6, VP = p.VP;
+  const int DK = p.DK, KB = (DK + 63) >> 6, VP = p.VP;
   const int m0 = r0 + qt * 128, rows = min(128, nrows - qt * 128);
   const int pos0 = p.kv_len[j] - nrows + qt * 128;                  // position of the tile's first row
   const int keys = pos0 + rows;
-  const int blocks = (keys + kTcKeys - 1) / kTcKeys;
+  const int first = p.chunk > 0 ? pos0 - pos0 % p.chunk : 0;        // first key any row of the tile sees
+  const int b0 = first / kTcKeys, blocks = (keys + kTcKeys - 1) / kTcKeys - b0;
   const uint32_t q_s = (smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t kbytes = static_cast<uint32_t>(KB) * 16384u, vbytes = static_cast<uint32_t>(VP) * 256u;
   const uint32_t k_s = q_s + kbytes, v_s = k_s + 2 * kbytes;
@@ -72,7 +79,7 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
     tmem_relinquish();
   }
   // query tile, swizzled; columns past DK and rows past the live ones are zeros
-  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q_eff) + (static_cast<size_t>(m0) * p.H + h) * DK;
+  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + (static_cast<size_t>(m0) * p.H + h) * DK;
   for (int r = warp; r < 128; r += 6)
     for (int c = lane; c < KB * 8; c += 32) {
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
@@ -84,35 +91,35 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  const uint32_t tm = tmem_base_s, tm_o = tm + 256, tm_p = tm + 384;
+  const uint32_t tm = tmem_base_s, tm_o = tm + 256, tm_p = tm + 448;
 
   if (warp == 0) {
     // ---------------------------------------------------------------- copies
     if (lane == 0) {
-      const uint8_t* ke = static_cast<const uint8_t*>(p.k_exp);
-      const uint8_t* ve = static_cast<const uint8_t*>(p.v_exp);
-      const size_t kpage = static_cast<size_t>(KB) * 8192, vpage = static_cast<size_t>(VP) * 128;
-      const int last = (keys - 1) / 64;
+      const uint8_t* ke = static_cast<const uint8_t*>(p.k);
+      const uint8_t* ve = static_cast<const uint8_t*>(p.v);
+      const int last = (keys - 1) / 64, g = h / (p.H / p.G);
       int b = 0;
       bool ok = true;
       for (; b < blocks; ++b) {
         const int s = b & 1;
         const uint32_t ph = ((b >> 1) & 1) ^ 1;                     // of the use before this one
         size_t at[2];                                               // (a missing second page: the first again, its keys are masked)
-        at[0] = static_cast<size_t>(mla_page_at(p, j, b * 2)) * p.H + h;
-        at[1] = b * 2 + 1 <= last ? static_cast<size_t>(mla_page_at(p, j, b * 2 + 1)) * p.H + h : at[0];
+        const int pg = (b0 + b) * 2;
+        at[0] = static_cast<size_t>(page_at(p, j, pg)) * p.G + g;
+        at[1] = pg + 1 <= last ? static_cast<size_t>(page_at(p, j, pg + 1)) * p.G + g : at[0];
         if (b >= 2 && !mbar_wait(kfree + 8 * s, ph, p.err, kErrWaitEmpty)) { ok = false; break; }
         mbar_arrive_expect_tx(kfull + 8 * s, kbytes);
         for (int kb = 0; kb < KB; ++kb)
-          for (int g = 0; g < 2; ++g)
-            bulk_g2s(k_s + s * kbytes + kb * 16384 + g * 8192, ke + at[g] * kpage + static_cast<size_t>(kb) * 8192, 8192, kfull + 8 * s);
+          for (int i = 0; i < 2; ++i)
+            bulk_g2s(k_s + s * kbytes + kb * 16384 + i * 8192, ke + at[i] * p.k_stride + static_cast<size_t>(kb) * 8192, 8192, kfull + 8 * s);
         if (b >= 2 && !mbar_wait(vfree + 8 * s, ph, p.err, kErrWaitEmpty)) {
           mbar_wait(kfull + 8 * s, (b >> 1) & 1, p.err, kErrWaitDrain);
           ok = false;
           break;
         }
         mbar_arrive_expect_tx(vfull + 8 * s, vbytes);
-        for (int g = 0; g < 2; ++g) bulk_g2s(v_s + s * vbytes + g * (vbytes >> 1), ve + at[g] * vpage, vbytes >> 1, vfull + 8 * s);
+        for (int i = 0; i < 2; ++i) bulk_g2s(v_s + s * vbytes + i * (vbytes >> 1), ve + at[i] * p.v_stride, vbytes >> 1, vfull + 8 * s);
       }
       if (!ok)                                                      // do not leave while an own copy is in flight
         for (int i = max(0, b - 2); i < b; ++i) {
@@ -159,8 +166,12 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
     // ---------------------------------------------------------------- softmax
     const int q4 = warp & 3, row = q4 * 32 + lane;
     const uint32_t lane_off = static_cast<uint32_t>(q4 * 32) << 16;
-    const float sc = p.scale * kTcLog2e;
-    float mx = -INFINITY, used = -INFINITY, l = 0.f;
+    const bool capped = p.softcap > 0.f;
+    const float sc = capped ? kTcLog2e : p.scale * kTcLog2e, zs = capped ? 2.f * kTcLog2e * p.scale / p.softcap : 0.f;
+    // (a row may meet blocks ahead of its first key: the maximum starts finite so that differences stay numbers)
+    float mx = kTcNone, used = kTcNone, l = 0.f;
+    const int low = p.chunk > 0 ? (pos0 + row) - (pos0 + row) % p.chunk : 0;   // first key of this row
+    const int low_last = p.chunk > 0 ? (pos0 + q4 * 32 + 31) - (pos0 + q4 * 32 + 31) % p.chunk : 0;
     bool ok = true;
     for (int b = 0; b < blocks; ++b) {
       const int s = b & 1;
@@ -180,16 +191,26 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(sfree + 8 * s);
-      const int vis = pos0 + row - b * kTcKeys;                     // last visible key of this row inside the block
-      if (b * kTcKeys + kTcKeys - 1 > pos0 + q4 * 32) {
+      if (capped) {
+#pragma unroll
+        for (int i = 0; i < 128; ++i) v[i] = soft_cap(v[i], zs, p.softcap);
+      }
+      const int key0 = (b0 + b) * kTcKeys;
+      const int vis = pos0 + row - key0, low_v = low - key0;        // last and first visible key of this row inside the block
+      if (key0 + kTcKeys - 1 > pos0 + q4 * 32) {
 #pragma unroll
         for (int i = 0; i < 128; ++i)
           if (i > vis) v[i] = -INFINITY;
       }
+      if (low_last > key0) {
+#pragma unroll
+        for (int i = 0; i < 128; ++i)
+          if (i < low_v) v[i] = -INFINITY;
+      }
       float m4[4] = {mx, mx, mx, mx};
 #pragma unroll
       for (int i = 0; i < 128; ++i) m4[i & 3] = fmaxf(m4[i & 3], v[i]);
-      mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));         // (key 0 is visible to every row: finite from the first block on)
+      mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
       // P and O of the block before are consumed
       ok = __all_sync(0xffffffffu, b == 0 || mbar_wait(odone, (b - 1) & 1, p.err, kErrWaitAcc));
       if (!ok) break;
@@ -236,7 +257,7 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
       const int m = m0 + row;
       const bool live = row < rows;
       const float inv = 1.f / l;
-      const float* g = p.x + static_cast<size_t>(live ? m : m0) * p.ldx + p.g_off + h * p.V;
+      const float* g = p.gate == nullptr ? nullptr : p.gate + static_cast<size_t>(live ? m : m0) * p.ldg + h * p.V;
       const int k0 = p.out_k0 + h * p.V;
       for (int c = 0; c < VP; c += 32) {
         uint32_t r[32];
@@ -248,17 +269,24 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             if (c + i * 8 >= p.V) break;
-            const float4 ga = *reinterpret_cast<const float4*>(g + c + i * 8), gb = *reinterpret_cast<const float4*>(g + c + i * 8 + 4);
-            const float gg[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
             float y[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[e] = __uint_as_float(r[i * 8 + e]) * inv / (1.f + expf(-gg[e]));
+            for (int e = 0; e < 8; ++e) y[e] = __uint_as_float(r[i * 8 + e]) * inv;
+            if (g != nullptr) {
+              const float4 ga = *reinterpret_cast<const float4*>(g + c + i * 8), gb = *reinterpret_cast<const float4*>(g + c + i * 8 + 4);
+              const float gg[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
+#pragma unroll
+              for (int e = 0; e < 8; ++e) y[e] = y[e] / (1.f + expf(-gg[e]));
+            }
             operand_store8(p.out, m, k0 + c + i * 8, y);
           }
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (c + i < p.V) operand_store1(p.out, m, k0 + c + i, __uint_as_float(r[i]) * inv / (1.f + expf(-g[c + i])));
+            if (c + i < p.V) {
+              const float y = __uint_as_float(r[i]) * inv;
+              operand_store1(p.out, m, k0 + c + i, g != nullptr ? y / (1.f + expf(-g[c + i])) : y);
+            }
         }
       }
     }
@@ -268,28 +296,26 @@ __global__ void __launch_bounds__(kTcThreads) mla_flash_tc_kernel(const __grid_c
   if (warp == 1) tmem_dealloc(tm, 512);
 }
 
-static int flash_tc_smem(const MlaParams& p) {
-  const int KB = (p.DP + p.RP + 63) / 64;
-  return 3 * KB * 16384 + 2 * p.VP * 256 + 1024;
-}
+static int flash_tc_smem(int DK, int VP) { return 3 * ((DK + 63) / 64) * 16384 + 2 * VP * 256 + 1024; }
 
 }  // namespace saber
 
-bool saber_mla_flash_tc_ok(const saber::MlaParams* p) {
-  return !p->f32 && p->scale > 0.f && p->page == 64 && (p->VP == 32 || p->VP == 64 || p->VP == 128) && ((p->DP | p->RP) & 15) == 0 &&
-         saber::flash_tc_smem(*p) <= 226 * 1024;
+// VP: the accumulator shares tensor memory with two score buffers (256 columns) and the probabilities (64)
+bool saber_flash_tc_ok(int page, int DK, int VP, float scale, float softcap) {
+  return (scale > 0.f || softcap > 0.f) && page == 64 && (VP & 31) == 0 && VP <= 192 && (DK & 15) == 0 && saber::flash_tc_smem(DK, VP) <= 226 * 1024;
 }
 
-int saber_mla_flash_tc(const saber::MlaParams* p, cudaStream_t stream) {
+int saber_flash_tc(const saber::FlashParams* p, cudaStream_t stream) {
   using namespace saber;
   static bool ready[64];
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
   if (!ready[dev]) {
-    const cudaError_t e = cudaFuncSetAttribute(mla_flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+    const cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
     ready[dev] = true;
   }
-  return static_cast<int>(launch(mla_flash_tc_kernel, dim3((p->max_rows + 127) / 128, p->H, p->nseq), dim3(kTcThreads), flash_tc_smem(*p), stream, 0, *p));
+  return static_cast<int>(launch(flash_tc_kernel, dim3((p->max_rows + 127) / 128, p->H, p->nseq), dim3(kTcThreads),
+                                 flash_tc_smem(p->DK, p->VP), stream, 0, *p));
 }

@@ -1,0 +1,484 @@
+// Grouped-query attention over tiled pages.
+//
+//   append   keys (normed) and values of this step's rows into their pages; for the tcgen05 form also the queries
+//   form 2   flash_tc.cu: prompt portions
+//   form 1   decoding and short portions: the query heads of a key head are the rows of an `mma.sync` tile, pages arrive
+//            by bulk copies, keys are split over CTAs and the last CTA of a row to finish merges the parts.  A step
+//            with one row per sequence appends its own key and value, so that it is the only launch.
+//   form 0   a CTA per (row, head) on the CUDA cores: fp32 models and sizes the other forms do not take
+#include "flash_tc.h"
+#include "gqa.h"
+#include "launch.cuh"
+#include "mla_device.cuh"
+
+namespace saber {
+
+constexpr float kGqaLog2e = 1.4426950408889634f;
+constexpr int kPage = 64;
+
+// element of a page's key / value head block
+__device__ __forceinline__ int bf16_key_at(int key, int d) { return (d >> 6) * 4096 + key * 64 + (((((d & 63) >> 3) ^ key) & 7) << 3) + (d & 7); }
+__device__ __forceinline__ int bf16_val_at(int KP, int key, int v) { return kPage * KP + v * 64 + ((((key >> 3) ^ v) & 7) << 3) + (key & 7); }
+template <typename T> struct Page;
+template <> struct Page<__nv_bfloat16> {
+  static __device__ __forceinline__ int key(const GqaParams&, int t, int d) { return bf16_key_at(t, d); }
+  static __device__ __forceinline__ int val(const GqaParams& p, int t, int v) { return bf16_val_at(p.KP, t, v); }
+  static __device__ __forceinline__ float load(const void* b, size_t i) { return __bfloat162float(static_cast<const __nv_bfloat16*>(b)[i]); }
+  static __device__ __forceinline__ void store(void* b, size_t i, float x) { static_cast<__nv_bfloat16*>(b)[i] = __float2bfloat16(x); }
+};
+template <> struct Page<float> {
+  static __device__ __forceinline__ int key(const GqaParams& p, int t, int d) { return t * p.KP + d; }
+  static __device__ __forceinline__ int val(const GqaParams& p, int t, int v) { return kPage * p.KP + t * p.VP + v; }
+  static __device__ __forceinline__ float load(const void* b, size_t i) { return static_cast<const float*>(b)[i]; }
+  static __device__ __forceinline__ void store(void* b, size_t i, float x) { static_cast<float*>(b)[i] = x; }
+};
+__device__ __forceinline__ size_t page_block(const GqaParams& p, int page, int g) {
+  return (static_cast<size_t>(page) * p.G + g) * kPage * (p.KP + p.VP);
+}
+// reciprocal root mean square of D values (a warp), 1 without the norm
+__device__ __forceinline__ float head_scale(const GqaParams& p, const float* x, int lane) {
+  if (!p.qk_norm) return 1.f;
+  float sq = 0.f;
+  for (int d = lane; d < p.D; d += 32) sq = fmaf(x[d], x[d], sq);
+  return 1.f / sqrtf(mla_warp_sum(sq) / static_cast<float>(p.D) + p.eps);
+}
+
+// grid (ceil(M / 8), ceil(items / 8)), 256 threads; a warp per (head, eight rows): query heads (tcgen05 form only), then
+// key heads, then value heads.  Eight values of neighbouring tokens leave as one 16-byte piece where a page allows it.
+template <typename T>
+__global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__ GqaParams p) {
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  int item = blockIdx.y * 8 + (threadIdx.x >> 5);
+  const int m0 = blockIdx.x * 8, n = min(8, p.M - m0);
+  if (p.form == 2) {
+    if (item < p.H) {
+      for (int r = 0; r < n; ++r) {
+        const float* x = p.x + static_cast<size_t>(m0 + r) * p.ldx + p.q_off + item * p.D;
+        const float s = head_scale(p, x, lane);
+        __nv_bfloat16* q = static_cast<__nv_bfloat16*>(p.q) + (static_cast<size_t>(m0 + r) * p.H + item) * p.DK;
+        for (int d = lane; d < p.DK; d += 32) q[d] = __float2bfloat16(d < p.D ? x[d] * s : 0.f);
+      }
+      return;
+    }
+    item -= p.H;
+  }
+  if (p.k_off < 0 || item >= 2 * p.G) return;
+  const bool isv = item >= p.G;
+  const int g = isv ? item - p.G : item;
+  int slot[8];
+#pragma unroll
+  for (int r = 0; r < 8; ++r) {
+    slot[r] = r < n ? p.slot_map[m0 + r] : -1;
+    if (slot[r] >= p.n_blocks * kPage) {
+      if (lane == 0 && p.err) atomicCAS(p.err, 0u, static_cast<uint32_t>(kErrBadIndex));
+      slot[r] = -1;
+    }
+  }
+  if (!isv) {
+    for (int r = 0; r < n; ++r) {
+      const int s = p.slot_map[m0 + r];
+      if (s < 0 || s >= p.n_blocks * kPage) continue;
+      const float* x = p.x + static_cast<size_t>(m0 + r) * p.ldx + p.k_off + g * p.D;
+      const float sc = head_scale(p, x, lane);
+      const size_t b = page_block(p, s / kPage, g);
+      for (int d = lane; d < p.D; d += 32) Page<T>::store(p.cache, b + Page<T>::key(p, s % kPage, d), x[d] * sc);
+    }
+    return;
+  }
+  bool whole = sizeof(T) == 2 && slot[0] >= 0 && (slot[0] & 7) == 0;
+#pragma unroll
+  for (int r = 1; r < 8; ++r) whole = whole && slot[r] == slot[0] + r;
+  const float* x = p.x + static_cast<size_t>(m0) * p.ldx + p.v_off + g * p.V;
+  for (int v = lane; v < p.V; v += 32) {
+    float y[8];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) y[r] = slot[r] >= 0 ? x[static_cast<size_t>(r) * p.ldx + v] : 0.f;
+    if (whole) {
+      __nv_bfloat16* c = static_cast<__nv_bfloat16*>(p.cache) + page_block(p, slot[0] / kPage, g) + bf16_val_at(p.KP, slot[0] % kPage, v);
+      *reinterpret_cast<uint4*>(c) = make_uint4(pack2(y[0], y[1]), pack2(y[2], y[3]), pack2(y[4], y[5]), pack2(y[6], y[7]));
+    } else {
+#pragma unroll
+      for (int r = 0; r < 8; ++r)
+        if (slot[r] >= 0) Page<T>::store(p.cache, page_block(p, slot[r] / kPage, g) + Page<T>::val(p, slot[r] % kPage, v), y[r]);
+    }
+  }
+}
+
+// grid (M, H), 128 threads: one query row of one head, 64 keys at a time
+template <typename T>
+__global__ void __launch_bounds__(128) gqa_row_kernel(const __grid_constant__ GqaParams p) {
+  pdl_wait();
+  extern __shared__ float sm[];                   // q [D] | scores [64] | output [V]
+  __shared__ float scale_s;
+  const int m = blockIdx.x, h = blockIdx.y, g = h / (p.H / p.G);
+  const int j = mla_seq_of_row(p.cu_rows, p.nseq, m);
+  if (j < 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* sc = sm + p.D;
+  float* o = sc + kPage;
+  const float* x = p.x + static_cast<size_t>(m) * p.ldx + p.q_off + h * p.D;
+  if (warp == 0) {
+    const float s = head_scale(p, x, lane);
+    if (lane == 0) scale_s = s;
+  }
+  __syncthreads();
+  // (queries are rounded like the keys they meet)
+  for (int d = threadIdx.x; d < p.D; d += 128) sm[d] = sizeof(T) == 2 ? __bfloat162float(__float2bfloat16(x[d] * scale_s)) : x[d] * scale_s;
+  for (int v = threadIdx.x; v < p.V; v += 128) o[v] = 0.f;
+  const int pos = p.pos[m], low = p.chunk > 0 ? pos - pos % p.chunk : 0;
+  float mx = -INFINITY, l = 0.f;
+  for (int pg = low / kPage; pg <= pos / kPage; ++pg) {
+    const size_t b = page_block(p, page_at(p, j, pg), g);
+    const int t0 = max(0, low - pg * kPage), t1 = min(kPage, pos + 1 - pg * kPage);
+    __syncthreads();
+    for (int t = t0 + warp; t < t1; t += 4) {
+      float s = 0.f;
+      for (int d = lane; d < p.D; d += 32) s = fmaf(sm[d], Page<T>::load(p.cache, b + Page<T>::key(p, t, d)), s);
+      s = mla_warp_sum(s) * p.scale;
+      if (lane == 0) sc[t] = p.softcap > 0.f ? p.softcap * tanhf(s / p.softcap) : s;
+    }
+    __syncthreads();
+    const float a = lane >= t0 && lane < t1 ? sc[lane] : -INFINITY, c = lane + 32 >= t0 && lane + 32 < t1 ? sc[lane + 32] : -INFINITY;
+    const float mn = fmaxf(mx, mla_warp_max(fmaxf(a, c)));          // (every page of the walk has a visible key)
+    const float ea = expf(a - mn), ec = expf(c - mn), corr = expf(mx - mn);
+    l = l * corr + mla_warp_sum(ea + ec);
+    mx = mn;
+    __syncthreads();
+    if (warp == 0) { sc[lane] = ea; sc[lane + 32] = ec; }
+    __syncthreads();
+    for (int v = threadIdx.x; v < p.V; v += 128) {
+      float s = o[v] * corr;
+      for (int t = t0; t < t1; ++t) s = fmaf(sc[t], Page<T>::load(p.cache, b + Page<T>::val(p, t, v)), s);
+      o[v] = s;
+    }
+  }
+  for (int v = threadIdx.x; v < p.V; v += 128) operand_store1(p.out, m, p.out_k0 + h * p.V + v, o[v] / l);
+}
+
+// grid (M, G, splits), 128 threads.  MT: 16-row tiles of query heads.  NC: 8-column groups of a value per warp.
+template <int MT, int NC>
+__global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ GqaParams p) {
+  pdl_wait();
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  __shared__ uint64_t bars[2];
+  __shared__ float corr_s[MT * 16], l_s[MT * 16];
+  __shared__ uint32_t last_s;
+  const int m = blockIdx.x, g = blockIdx.y, sp = blockIdx.z;
+  const int j = mla_seq_of_row(p.cu_rows, p.nseq, m);
+  if (j < 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hq = p.H / p.G;
+  const int pos = p.pos[m], low = p.chunk > 0 ? pos - pos % p.chunk : 0;
+  const int page0 = low / kPage, pages = pos / kPage + 1 - page0;
+  const int per = (pages + p.splits - 1) / p.splits;
+  const int pa = page0 + sp * per, n = min(per, page0 + pages - pa);       // this CTA's pages (n <= 0: none)
+  const uint32_t stage = 128u * static_cast<uint32_t>(p.KP + p.VP);
+  const uint32_t kv_s = (smem_u32(smem_raw) + 127u) & ~127u;
+  const uint32_t qs = static_cast<uint32_t>(p.DK) * 2u + 16u;              // row stride: an odd number of 16-byte units
+  const uint32_t q_s = kv_s + 2 * stage;
+  const uint32_t p_s = q_s + MT * 16 * qs;                                 // probabilities, bf16 [MT * 16][64 + 8]
+  uint8_t* const base = smem_raw + (kv_s - smem_u32(smem_raw));
+  float* s_f = reinterpret_cast<float*>(base + 2 * stage + MT * 16 * qs + MT * 16 * 144);      // scores [MT * 16][64 + 4]
+  const bool append = p.max_rows == 1 && p.k_off >= 0 && n > 0 && pa + n == page0 + pages;     // the new token's page is mine
+  __nv_bfloat16* new_s = reinterpret_cast<__nv_bfloat16*>(s_f + MT * 16 * 68);                 // key [KP] | value [VP] of the new token
+  const uint32_t bar = smem_u32(bars);
+  const uint8_t* cache = static_cast<const uint8_t*>(p.cache);
+  auto fetch = [&](int it) {
+    mbar_arrive_expect_tx(bar + 8 * (it & 1), stage);
+    bulk_g2s(kv_s + (it & 1) * stage, cache + page_block(p, page_at(p, j, pa + it), g) * 2, stage, bar + 8 * (it & 1));
+  };
+  int issued = 0;
+  if (threadIdx.x == 0) {
+    mbar_init(bar, 1);
+    mbar_init(bar + 8, 1);
+    mbar_init_fence();
+    for (; issued < min(2, n); ++issued) fetch(issued);
+  }
+  const float* xr = p.x + static_cast<size_t>(m) * p.ldx;
+  for (int r = warp; r < MT * 16; r += 4) {
+    const float* x = xr + p.q_off + (g * hq + min(r, hq - 1)) * p.D;
+    const float s = head_scale(p, x, lane);
+    for (int d = lane * 2; d < p.DK; d += 64) {
+      const float a = r < hq && d < p.D ? x[d] * s : 0.f, b = r < hq && d + 1 < p.D ? x[d + 1] * s : 0.f;
+      asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_s + r * qs + d * 2), "r"(pack2(a, b)) : "memory");
+    }
+  }
+  for (int i = threadIdx.x; i < MT * 16 * 36; i += 128) asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_s + i * 4), "r"(0) : "memory");
+  if (threadIdx.x < MT * 16) corr_s[threadIdx.x] = 1.f;
+  if (append) {
+    const int slot = p.slot_map[m];
+    const bool live = slot >= 0 && slot < p.n_blocks * kPage;
+    __nv_bfloat16* c = static_cast<__nv_bfloat16*>(p.cache) + (live ? page_block(p, slot / kPage, g) : 0);
+    if (warp == 0) {
+      const float* x = xr + p.k_off + g * p.D;
+      const float s = head_scale(p, x, lane);
+      for (int d = lane; d < p.D; d += 32) {
+        new_s[d] = __float2bfloat16(x[d] * s);
+        if (live) c[bf16_key_at(slot % kPage, d)] = new_s[d];
+      }
+    } else {
+      for (int v = threadIdx.x - 32; v < p.V; v += 96) {
+        new_s[p.KP + v] = __float2bfloat16(xr[p.v_off + g * p.V + v]);
+        if (live) c[bf16_val_at(p.KP, slot % kPage, v)] = new_s[p.KP + v];
+      }
+    }
+  }
+  __syncthreads();
+  const bool capped = p.softcap > 0.f;
+  const float zs = capped ? 2.f * kGqaLog2e * p.scale / p.softcap : 0.f;
+  float o[MT][NC][4] = {};
+  float mx[4 * MT], l[4 * MT];                                      // rows warp, warp + 4, ... of the tile
+#pragma unroll
+  for (int i = 0; i < 4 * MT; ++i) { mx[i] = -INFINITY; l[i] = 0.f; }
+  bool ok = true;
+  int it = 0;
+  for (; it < n; ++it) {
+    const uint32_t kt = kv_s + (it & 1) * stage, vt = kt + kPage * 2 * p.KP;
+    ok = __syncthreads_and(mbar_wait(bar + 8 * (it & 1), (it >> 1) & 1, p.err, kErrWaitFull)) != 0;
+    if (!ok) break;
+    if (append && it == n - 1) {
+      __nv_bfloat16* c = reinterpret_cast<__nv_bfloat16*>(base + (it & 1) * stage);
+      for (int d = threadIdx.x; d < p.D; d += 128) c[bf16_key_at(pos % kPage, d)] = new_s[d];
+      for (int v = threadIdx.x; v < p.V; v += 128) c[bf16_val_at(p.KP, pos % kPage, v)] = new_s[p.KP + v];
+      __syncthreads();
+    }
+    // scores: 16 keys per warp
+    {
+      float s[MT][2][4] = {};
+      const uint32_t a_row = q_s + (lane & 15) * qs + ((lane >> 4) << 4);
+      const int key = warp * 16 + ((lane >> 4) << 3) + (lane & 7);
+      for (int st = 0; st < p.DK / 16; ++st) {
+        const int c = st * 2 + ((lane >> 3) & 1);
+        uint32_t b[4];
+        ldsm4(b, kt + (c >> 3) * 8192 + key * 128 + (((c ^ key) & 7) << 4));
+#pragma unroll
+        for (int t = 0; t < MT; ++t) {
+          uint32_t a[4];
+          ldsm4(a, a_row + t * 16 * qs + st * 32);
+          mma16816(s[t][0], a, b[0], b[1]);
+          mma16816(s[t][1], a, b[2], b[3]);
+        }
+      }
+      const int r = lane >> 2;
+#pragma unroll
+      for (int t = 0; t < MT; ++t)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int c = warp * 16 + i * 8 + (lane & 3) * 2;
+          *reinterpret_cast<float2*>(s_f + (t * 16 + r) * 68 + c) = make_float2(s[t][i][0], s[t][i][1]);
+          *reinterpret_cast<float2*>(s_f + (t * 16 + r + 8) * 68 + c) = make_float2(s[t][i][2], s[t][i][3]);
+        }
+    }
+    __syncthreads();
+    // running softmax
+    const int key0 = (pa + it) * kPage + lane * 2;
+#pragma unroll
+    for (int i = 0; i < 4 * MT; ++i) {
+      const int r = warp + 4 * i;
+      if (r >= hq) continue;
+      const float2 v = *reinterpret_cast<const float2*>(s_f + r * 68 + lane * 2);
+      float a = v.x * p.scale, b = v.y * p.scale;
+      if (capped) {
+        a = p.softcap - __fdividef(2.f * p.softcap, 1.f + ex2(v.x * zs));
+        b = p.softcap - __fdividef(2.f * p.softcap, 1.f + ex2(v.y * zs));
+      }
+      if (key0 < low || key0 > pos) a = -INFINITY;
+      if (key0 + 1 < low || key0 + 1 > pos) b = -INFINITY;
+      const float mn = fmaxf(mx[i], mla_warp_max(fmaxf(a, b)));     // (every page of the walk has a visible key)
+      const float ea = ex2((a - mn) * kGqaLog2e), eb = ex2((b - mn) * kGqaLog2e), corr = ex2((mx[i] - mn) * kGqaLog2e);
+      l[i] = l[i] * corr + mla_warp_sum(ea + eb);
+      mx[i] = mn;
+      asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_s + r * 144 + lane * 4), "r"(pack2(ea, eb)) : "memory");
+      if (lane == 0) corr_s[r] = corr;
+    }
+    __syncthreads();
+    // values: this warp's columns
+#pragma unroll
+    for (int t = 0; t < MT; ++t) {
+      const float c0 = corr_s[t * 16 + (lane >> 2)], c1 = corr_s[t * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int i = 0; i < NC; ++i) { o[t][i][0] *= c0; o[t][i][1] *= c0; o[t][i][2] *= c1; o[t][i][3] *= c1; }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {                          // 32 keys
+      uint32_t a[MT][2][4];
+#pragma unroll
+      for (int t = 0; t < MT; ++t)
+#pragma unroll
+        for (int k = 0; k < 2; ++k) ldsm4(a[t][k], p_s + (t * 16 + (lane & 15)) * 144 + (half * 2 + k) * 32 + ((lane >> 4) << 4));
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        const int col = (warp * NC + i) * 8;
+        if (col >= p.VP) break;
+        const int v = col + (lane & 7), c = half * 4 + (lane >> 3);
+        uint32_t b[4];
+        ldsm4(b, vt + v * 128 + (((c ^ v) & 7) << 4));
+#pragma unroll
+        for (int t = 0; t < MT; ++t) {
+          mma16816(o[t][i], a[t][0], b[0], b[1]);
+          mma16816(o[t][i], a[t][1], b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();
+    if (threadIdx.x == 0 && it + 2 < n) { fetch(it + 2); ++issued; }
+  }
+  if (!ok && threadIdx.x == 0)                                      // do not leave while an own copy is in flight
+    for (int i = it; i < issued; ++i) mbar_wait(bar + 8 * (i & 1), (i >> 1) & 1, p.err, kErrWaitDrain);
+#pragma unroll
+  for (int i = 0; i < 4 * MT; ++i) {
+    const int r = warp + 4 * i;
+    if (r >= hq || lane != 0) continue;
+    l_s[r] = l[i];
+    if (p.splits > 1) {
+      float* d = p.ml + ((static_cast<size_t>(m) * p.H + g * hq + r) * p.splits + sp) * 2;
+      __stcg(d, mx[i]);
+      __stcg(d + 1, l[i]);
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int t = 0; t < MT; ++t)
+#pragma unroll
+    for (int e2 = 0; e2 < 2; ++e2) {
+      const int r = t * 16 + (lane >> 2) + e2 * 8;
+      if (r >= hq) continue;
+      const int h = g * hq + r;
+      const float inv = 1.f / l_s[r];
+      float* d = p.splits > 1 ? p.o_part + ((static_cast<size_t>(m) * p.H + h) * p.splits + sp) * p.VP : nullptr;
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        const int v = (warp * NC + i) * 8 + (lane & 3) * 2;
+        if (v >= p.VP) break;
+        const float a = o[t][i][e2 * 2], b = o[t][i][e2 * 2 + 1];
+        if (d != nullptr) {
+          if (n > 0) __stcg(reinterpret_cast<float2*>(d + v), make_float2(a, b));
+        } else {
+          if (v < p.V) operand_store1(p.out, m, p.out_k0 + h * p.V + v, a * inv);
+          if (v + 1 < p.V) operand_store1(p.out, m, p.out_k0 + h * p.V + v + 1, b * inv);
+        }
+      }
+    }
+  if (p.splits == 1) return;
+  // the last part of the row to arrive merges them, in order
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    uint32_t* c = p.counters + static_cast<size_t>(m) * p.G + g;
+    const bool last = atomicAdd(c, 1u) == static_cast<uint32_t>(p.splits) - 1u;
+    if (last) *c = 0u;
+    __threadfence();
+    last_s = last ? 1u : 0u;
+  }
+  __syncthreads();
+  if (!last_s) return;
+  const float* ml = p.ml + (static_cast<size_t>(m) * p.H + g * hq) * p.splits * 2;
+  for (int r = warp; r < hq; r += 4) {                              // weights of the parts (splits <= 32: a lane each)
+    const float pm = lane < p.splits ? __ldcg(ml + (r * p.splits + lane) * 2) : -INFINITY;
+    const float pl = lane < p.splits ? __ldcg(ml + (r * p.splits + lane) * 2 + 1) : 0.f;
+    const float mm = mla_warp_max(pm);
+    const float w = pm > -INFINITY ? ex2((pm - mm) * kGqaLog2e) : 0.f;
+    const float tot = mla_warp_sum(w * pl);
+    s_f[r * 33 + lane] = w / tot;
+  }
+  __syncthreads();
+  const float* part = p.o_part + (static_cast<size_t>(m) * p.H + g * hq) * p.splits * p.VP;
+  for (int i = threadIdx.x; i < hq * p.V; i += 128) {
+    const int r = i / p.V, v = i - r * p.V;
+    float y = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < p.splits; ++s) {
+      const float w = s_f[r * 33 + s];
+      if (w > 0.f) y = fmaf(w, __ldcg(part + (static_cast<size_t>(r) * p.splits + s) * p.VP + v), y);
+    }
+    operand_store1(p.out, m, p.out_k0 + (g * hq + r) * p.V + v, y);
+  }
+}
+
+static int split_tiles(const GqaParams& p) {
+  const int hq = p.H / p.G;
+  return hq <= 16 ? 1 : hq <= 32 ? 2 : 4;
+}
+static int split_smem(const GqaParams& p) {
+  const int rows = split_tiles(p) * 16;
+  return 2 * 128 * (p.KP + p.VP) + rows * (p.DK * 2 + 16 + 144 + 68 * 4) + 2 * (p.KP + p.VP) + 128;
+}
+template <int MT, int NC>
+static int split_go(const GqaParams& p, cudaStream_t stream) {
+  static bool ready[64];
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
+  if (!ready[dev]) {
+    const cudaError_t e = cudaFuncSetAttribute(gqa_split_kernel<MT, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    ready[dev] = true;
+  }
+  return static_cast<int>(launch(gqa_split_kernel<MT, NC>, dim3(p.M, p.G, p.splits), dim3(128), split_smem(p), stream, 0, p));
+}
+template <int NC>
+static int split_mt(const GqaParams& p, cudaStream_t s) {
+  const int mt = split_tiles(p);
+  return mt == 1 ? split_go<1, NC>(p, s) : mt == 2 ? split_go<2, NC>(p, s) : split_go<4, NC>(p, s);
+}
+
+static int append_items(const GqaParams& p) {
+  if (p.form == 1 && p.max_rows == 1) return 0;                     // the attention kernel appends by itself
+  return (p.form == 2 ? p.H : 0) + (p.k_off >= 0 ? 2 * p.G : 0);
+}
+
+template <typename T>
+static int gqa_go(const GqaParams& p, cudaStream_t stream) {
+  if (const int items = append_items(p)) {
+    const cudaError_t e = launch(gqa_append_kernel<T>, dim3((p.M + 7) / 8, (items + 7) / 8), dim3(256), 0, stream, 0, p);
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  if (p.form == 0)
+    return static_cast<int>(launch(gqa_row_kernel<T>, dim3(p.M, p.H), dim3(128), (p.D + kPage + p.V) * 4, stream, 0, p));
+  if (p.form == 1)
+    return p.VP <= 32 ? split_mt<1>(p, stream) : p.VP <= 64 ? split_mt<2>(p, stream) : p.VP <= 128 ? split_mt<4>(p, stream) : split_mt<8>(p, stream);
+  FlashParams f = {};
+  f.q = p.q;
+  f.k = p.cache;
+  f.v = static_cast<const uint8_t*>(p.cache) + static_cast<size_t>(kPage) * p.KP * 2;
+  f.k_stride = f.v_stride = static_cast<size_t>(kPage) * (p.KP + p.VP) * 2;
+  f.cu_rows = p.cu_rows;
+  f.kv_len = p.kv_len;
+  f.block_table = p.block_table;
+  f.out = p.out;
+  f.out_k0 = p.out_k0;
+  f.nseq = p.nseq;
+  f.H = p.H;
+  f.G = p.G;
+  f.DK = p.DK;
+  f.V = p.V;
+  f.VP = p.VP;
+  f.n_blocks = p.n_blocks;
+  f.max_blocks = p.max_blocks;
+  f.max_rows = p.max_rows;
+  f.chunk = p.chunk;
+  f.scale = p.scale;
+  f.softcap = p.softcap;
+  f.err = p.err;
+  return saber_flash_tc(&f, stream);
+}
+
+}  // namespace saber
+
+extern "C" int saber_gqa_form(const saber::GqaParams* p) {
+  if (p->f32 || p->page != saber::kPage || p->H / p->G > 64 || p->VP > 256 || (p->VP & 31) || (p->DK & 15) || (p->KP & 63) ||
+      saber::split_smem(*p) > 224 * 1024)
+    return 0;
+  return saber_flash_tc_ok(p->page, p->DK, p->VP, p->scale, p->softcap) ? 2 : 1;
+}
+
+extern "C" int saber_gqa_launches(const saber::GqaParams* p) { return saber::append_items(*p) ? 2 : 1; }
+
+extern "C" int saber_gqa_launch(const saber::GqaParams* p, cudaStream_t stream) {
+  using namespace saber;
+  if (p->M <= 0 || p->G <= 0 || p->H % p->G || p->page != kPage || p->D > p->DK || p->DK > p->KP || p->V > p->VP || p->cache == nullptr ||
+      p->D > 2048 || p->V > 2048 || p->form < 0 || p->form > saber_gqa_form(p) || (p->form == 2 && p->q == nullptr) ||
+      (p->form == 1 && (p->splits < 1 || p->splits > 32 || (p->splits > 1 && (p->o_part == nullptr || p->ml == nullptr || p->counters == nullptr)))))
+    return static_cast<int>(cudaErrorInvalidValue);
+  return p->f32 ? gqa_go<float>(*p, stream) : gqa_go<__nv_bfloat16>(*p, stream);
+}

@@ -1,0 +1,46 @@
+// Launch interface of grouped-query attention over tiled pages (gqa.cu): H query heads share G key / value heads,
+// fp32 scores.  Plain C types only.
+//
+//   q, k    optionally divided by their root mean square over D (qk_norm)
+//   score   scale q . k, then cap tanh(score / cap) when softcap > 0
+//   mask    keys j <= i; chunk > 0: of the same chunk of positions as i only, j >= i - i % chunk
+//
+// A page holds, per key / value head, the keys and then the values of its 64 tokens.  bf16: in the order the
+// tensor-core kernels multiply in place, keys [D / 64][64 tokens][128 bytes], values transposed [VP][64 tokens], both
+// with 16-byte pieces XOR (row & 7).  fp32: keys [64][KP], values [64][VP].
+#pragma once
+#include <cuda_runtime.h>
+#include <stdint.h>
+#include "operand.cuh"
+
+namespace saber {
+
+struct GqaParams {
+  const float* x;             // [M][ldx] projections of this step's rows
+  int ldx, q_off, k_off, v_off;   // k_off < 0: the cache is another layer's, nothing is appended
+  void* cache;                // [n_blocks][G][64 (KP + VP)]
+  void* q;                    // scratch [M][H][DK] bf16 (tcgen05 form)
+  float* o_part;              // scratch [M][H][splits][VP]
+  float* ml;                  // scratch [M][H][splits][2]
+  uint32_t* counters;         // [M][G], zero between launches
+  const int32_t* slot_map;    // [M] page * 64 + offset, -1: padding row
+  const int32_t* pos;         // [M]
+  const int32_t* cu_rows;     // [nseq + 1]
+  const int32_t* kv_len;      // [nseq]
+  const int32_t* block_table; // [nseq][max_blocks]
+  Operand out;
+  int out_k0;
+  int M, nseq, H, G, D, DK, KP, V, VP, page, n_blocks, max_blocks, splits;
+  int f32;                    // element type of the cache
+  int form;                   // 0: a CTA per (row, head), any size; 1: mma.sync over split keys; 2: tcgen05
+  int max_rows;               // rows one sequence may bring (1: the split form appends the row's key by itself)
+  int qk_norm, chunk;
+  float scale, softcap, eps;
+  uint32_t* err;
+};
+
+}  // namespace saber
+
+extern "C" int saber_gqa_form(const saber::GqaParams* p);     // the best form for these sizes
+extern "C" int saber_gqa_launches(const saber::GqaParams* p);
+extern "C" int saber_gqa_launch(const saber::GqaParams* p, cudaStream_t stream);

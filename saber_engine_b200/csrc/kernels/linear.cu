@@ -28,6 +28,11 @@ __device__ __forceinline__ float clamped_glu(float gate, float up, float limit, 
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
 }
 
+__device__ __forceinline__ float relu_squared(float x) {
+  const float r = fmaxf(x, 0.f);
+  return r * r;
+}
+
 // reciprocal root mean square of the stream row behind operand row m (all lanes of a warp call together)
 __device__ __forceinline__ float row_rms_scale(const LinEpi& e, int m, int lane) {
   if (e.ss == nullptr) return 1.f;
@@ -48,17 +53,30 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
     if (tile_n < e.act_tile0) {
       const int n = n0 + lane * 8;
       if (n >= e.n_plain) return;
-      const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+      float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
       float* o = e.out + static_cast<size_t>(m) * e.ldo + n;
+      a = make_float4(a.x * sc, a.y * sc, a.z * sc, a.w * sc);
+      b = make_float4(b.x * sc, b.y * sc, b.z * sc, b.w * sc);
       if (n + 8 <= e.n_plain) {
-        *reinterpret_cast<float4*>(o) = make_float4(a.x * sc, a.y * sc, a.z * sc, a.w * sc);
-        *reinterpret_cast<float4*>(o + 4) = make_float4(b.x * sc, b.y * sc, b.z * sc, b.w * sc);
+        if (e.bias) {
+          const float4 c = *reinterpret_cast<const float4*>(e.bias + n), d = *reinterpret_cast<const float4*>(e.bias + n + 4);
+          a = make_float4(a.x + c.x, a.y + c.y, a.z + c.z, a.w + c.w);
+          b = make_float4(b.x + d.x, b.y + d.y, b.z + d.z, b.w + d.w);
+        }
+        *reinterpret_cast<float4*>(o) = a;
+        *reinterpret_cast<float4*>(o + 4) = b;
       } else {
         const float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
 #pragma unroll
         for (int j = 0; j < 8; ++j)
-          if (n + j < e.n_plain) o[j] = v[j] * sc;
+          if (n + j < e.n_plain) o[j] = v[j] + (e.bias ? e.bias[n + j] : 0.f);
       }
+    } else if (e.act_kind == 1) {
+      const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+      const float y[8] = {relu_squared(a.x * sc), relu_squared(a.y * sc), relu_squared(a.z * sc), relu_squared(a.w * sc),
+                          relu_squared(b.x * sc), relu_squared(b.y * sc), relu_squared(b.z * sc), relu_squared(b.w * sc)};
+      const int k = e.act_k0 + (tile_n - e.act_tile0) * 256 + lane * 8;
+      if (k < e.act.ld) operand_store8(e.act, m, k, y);              // (the operand ends at a multiple of 64 columns, the tile of 256)
     } else {
       const float4 g = acc(lane * 4), u = acc(128 + lane * 4);
       operand_store4(e.act, m, e.act_k0 + (tile_n - e.act_tile0) * 128 + lane * 4,
@@ -381,8 +399,13 @@ __global__ void __launch_bounds__(256) lin_epi_kernel(const __grid_constant__ Li
   const float* acc = p.ws + static_cast<size_t>(m) * p.N_pad;
   if (!e.stream) {
     const float sc = row_rms_scale(e, m, threadIdx.x & 31);
-    for (int n = threadIdx.x; n < e.n_plain; n += 256) e.out[static_cast<size_t>(m) * e.ldo + n] = acc[n] * sc;
+    for (int n = threadIdx.x; n < e.n_plain; n += 256) e.out[static_cast<size_t>(m) * e.ldo + n] = acc[n] * sc + (e.bias ? e.bias[n] : 0.f);
     const int tiles = p.N_pad / 256;
+    if (e.act_kind == 1) {
+      for (int i = threadIdx.x; i < min((tiles - e.act_tile0) * 256, e.act.ld - e.act_k0); i += 256)
+        operand_store1(e.act, m, e.act_k0 + i, relu_squared(acc[e.act_tile0 * 256 + i] * sc));
+      return;
+    }
     for (int i = threadIdx.x; i < (tiles - e.act_tile0) * 128; i += 256) {
       const float* t = acc + static_cast<size_t>(e.act_tile0 + (i >> 7)) * 256 + (i & 127);
       operand_store1(e.act, m, e.act_k0 + i, clamped_glu(t[0] * sc, t[128] * sc, e.limit, e.alpha));

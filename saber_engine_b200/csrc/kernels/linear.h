@@ -10,10 +10,12 @@ namespace saber {
 // What happens to acc[m][n] = sum_k a[m][k] w[n][k].  Two kinds:
 //   project  the operand rows are norm_w * x without the division by the root mean square, so the
 //            result is scaled by rsqrt(sum(ss[m]) * inv_width + eps) (ss: per-128-column sums of squares the
-//            stream epilogue left; null: scale 1).  Features below act_tile0 * 256 are stored as fp32
-//            (n < n_plain); from there on a 256-feature tile holds 128 gate then 128 up features of a
-//            clamped gated unit, whose products go to the operand `act`:
-//            g = min(gate, limit), u = clamp(up, -limit, limit), y = g sigmoid(alpha g) (u + 1)
+//            stream epilogue left; null: scale 1).  Features below act_tile0 * 256 are stored as fp32,
+//            plus bias[n] (n < n_plain); those from there on are the feed-forward's and their activations go to
+//            the operand `act`:
+//              act_kind 0  a 256-feature tile holds 128 gate then 128 up features of a clamped gated unit,
+//                          g = min(gate, limit), u = clamp(up, -limit, limit), y = g sigmoid(alpha g) (u + 1)
+//              act_kind 1  y = max(up, 0)^2, 256 features a tile
 //   stream   x[m][n] = (add ? x[m][n] : 0) + bias[n] + acc, and the operand of the next linear:
 //            norm_w[n] x[m][n] with its sums of squares (ss_out), or x itself (norm_w null)
 struct LinEpi {
@@ -24,7 +26,7 @@ struct LinEpi {
   float* out;
   int ldo, n_plain, act_tile0;
   Operand act;
-  int act_k0;
+  int act_k0, act_kind;
   float limit, alpha;
   float* x;
   int ldx, width, add;

@@ -166,7 +166,7 @@ __global__ void __launch_bounds__(128) mla_row_attn_kernel(const __grid_constant
     __syncthreads();
     if (threadIdx.x < n) {
       const int key = kb + threadIdx.x;
-      rows_s[threadIdx.x] = static_cast<const T*>(p.cache) + (static_cast<size_t>(mla_page_at(p, j, key / p.page)) * p.page + key % p.page) * LD;
+      rows_s[threadIdx.x] = static_cast<const T*>(p.cache) + (static_cast<size_t>(page_at(p, j, key / p.page)) * p.page + key % p.page) * LD;
     }
     __syncthreads();
     for (int k = warp; k < n; k += 4) {

@@ -23,7 +23,8 @@ __device__ __forceinline__ int mla_seq_of_row(const int32_t* cu, int nseq, int m
   return -1;
 }
 // physical page of the i-th page of sequence j (bounds-checked: an entry outside the pool is recorded and read as page 0)
-__device__ __forceinline__ int mla_page_at(const MlaParams& p, int j, int i) {
+template <typename Params>
+__device__ __forceinline__ int page_at(const Params& p, int j, int i) {
   const int b = i < p.max_blocks ? p.block_table[static_cast<size_t>(j) * p.max_blocks + i] : -1;
   if (b >= 0 && b < p.n_blocks) return b;
   if (p.err) atomicCAS(p.err, 0u, static_cast<uint32_t>(kErrBadIndex));
@@ -64,6 +65,3 @@ template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.as
 int saber_mla_decode_attn(const saber::MlaParams* p, cudaStream_t stream);
 int saber_mla_expand_attn(const saber::MlaParams* p, cudaStream_t stream);
 bool saber_mla_decode_ok(const saber::MlaParams* p);
-// mla_flash_tc.cu
-bool saber_mla_flash_tc_ok(const saber::MlaParams* p);
-int saber_mla_flash_tc(const saber::MlaParams* p, cudaStream_t stream);

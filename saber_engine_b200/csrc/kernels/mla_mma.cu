@@ -6,6 +6,7 @@
 // expand  keys and values of the pages a step sees, [W_uk c | rotated part] and W_uv c, into scratch pages.
 // flash   causal attention of prompt portions over the scratch pages: 128 query rows of one head per CTA,
 //         16 per warp, one page of 64 keys at a time, running softmax in the base-2 domain.
+#include "flash_tc.h"
 #include "launch.cuh"
 #include "mla_device.cuh"
 
@@ -50,7 +51,7 @@ __global__ void __launch_bounds__(256) mla_decode_kernel(const __grid_constant__
       const int key = kb + r;
       const bool live = key < k1;
       const int at = live ? key : k0;
-      const __nv_bfloat16* src = cache + (static_cast<size_t>(mla_page_at(p, j, at / p.page)) * p.page + at % p.page) * LD;
+      const __nv_bfloat16* src = cache + (static_cast<size_t>(page_at(p, j, at / p.page)) * p.page + at % p.page) * LD;
       for (int c = lane; c < chunks; c += 32) cp16(dst + r * rs + c * 16, src + c * 8, live);
     }
     cp_commit();
@@ -243,8 +244,8 @@ __global__ void __launch_bounds__(256) mla_expand_kernel(const __grid_constant__
     }
     const int len = p.kv_len[j];
     int page[2];
-    page[0] = mla_page_at(p, j, pr * 2);
-    page[1] = pr * 128 + 64 < len ? mla_page_at(p, j, pr * 2 + 1) : -1;
+    page[0] = page_at(p, j, pr * 2);
+    page[1] = pr * 128 + 64 < len ? page_at(p, j, pr * 2 + 1) : -1;
     if (tile == per - 1) {
       const int rot8 = p.RP / 8;
       for (int i = threadIdx.x; i < 128 * p.H; i += 256) {
@@ -399,10 +400,10 @@ __global__ void __launch_bounds__(256) mla_flash_kernel(const __grid_constant__ 
     const int r = i / kch, c = i - r * kch;
     cp16(q_s + r * ks_ + c * 16, qg + static_cast<size_t>(min(r, rows - 1)) * p.H * DK + c * 8, r < rows);
   }
-  int next_page = mla_page_at(p, j, 0);                             // looked up one block ahead of its copies
+  int next_page = page_at(p, j, 0);                             // looked up one block ahead of its copies
   auto fetch = [&](int b) {
     const size_t pg = static_cast<size_t>(next_page) * p.H + h;
-    if (b + 1 < blocks) next_page = mla_page_at(p, j, b + 1);
+    if (b + 1 < blocks) next_page = page_at(p, j, b + 1);
     const __nv_bfloat16* kg = ke + pg * kKeys * DK;
     const __nv_bfloat16* vg = ve + pg * kKeys * VP;
     const uint32_t kd = kv_s + (b & 1) * stage, vd = kd + kKeys * ks_;
@@ -549,7 +550,32 @@ static int flash_go(const MlaParams& p, cudaStream_t stream) {
     ready[dev] = true;
   }
   cudaError_t e = launch(mla_expand_kernel, dim3(2 * 148), dim3(256), 3 * kExpStage, stream, 0, p);
-  if (e == cudaSuccess && p.expand == 2) return saber_mla_flash_tc(&p, stream);
+  if (e == cudaSuccess && p.expand == 2) {
+    FlashParams f = {};
+    f.q = p.q_eff;
+    f.k = p.k_exp;
+    f.v = p.v_exp;
+    f.k_stride = static_cast<size_t>((p.DP + p.RP + 63) / 64) * 8192;
+    f.v_stride = static_cast<size_t>(p.VP) * 128;
+    f.gate = p.x + p.g_off;
+    f.ldg = p.ldx;
+    f.cu_rows = p.cu_rows;
+    f.kv_len = p.kv_len;
+    f.block_table = p.block_table;
+    f.out = p.out;
+    f.out_k0 = p.out_k0;
+    f.nseq = p.nseq;
+    f.H = f.G = p.H;
+    f.DK = p.DP + p.RP;
+    f.V = p.V;
+    f.VP = p.VP;
+    f.n_blocks = p.n_blocks;
+    f.max_blocks = p.max_blocks;
+    f.max_rows = p.max_rows;
+    f.scale = p.scale;
+    f.err = p.err;
+    return saber_flash_tc(&f, stream);
+  }
   if (e == cudaSuccess)
     e = launch(mla_flash_kernel<NV>, dim3((p.max_rows + kQRows - 1) / kQRows, p.H, p.nseq), dim3(256), flash_smem(p), stream, 0, p);
   return static_cast<int>(e);
@@ -571,7 +597,7 @@ int saber_mla_decode_attn(const saber::MlaParams* p, cudaStream_t s) {
 // absorbed form has no such limit).
 extern "C" int saber_mla_expand_ok(const saber::MlaParams* p) {
   const bool vp = p->VP == 32 || p->VP == 64 || p->VP == 128 || p->VP == 256;
-  if (saber_mla_flash_tc_ok(p) && (p->CP & 15) == 0) return 2;
+  if (!p->f32 && p->VP <= 128 && saber_flash_tc_ok(p->page, p->DP + p->RP, p->VP, p->scale, 0.f) && ((p->DP | p->RP | p->CP) & 15) == 0) return 2;
   return !p->f32 && p->scale > 0.f && vp && p->page == saber::kKeys && ((p->DP | p->RP | p->CP) & 15) == 0 && saber::flash_smem(*p) <= 226 * 1024;
 }
 

@@ -1,14 +1,17 @@
 """A decoder assembled from a list of layers (`models.stack_config.StackConfig`) as native step programs.
 
-The parallel residual layer  x <- x + mixer(norm(x)) + ff(norm(x))  is two linears around the mixer's kernels.
-The residual stream stays fp32; a layer's output linear adds both sublayers to it and leaves the next linear's
-operand (norm weight times x) with the row's partial sums of squares, so that no normalisation, activation or
-addition needs a launch of its own.  Decode launches per layer: delta 3 (project, step, out), latent attention
-2 + 4; a pass of the looped block adds one linear.
+The residual stream stays fp32; a linear that ends a sublayer adds its result to it and leaves the next linear's operand
+(norm weight times x) with the row's partial sums of squares, so that no normalisation, activation or addition needs a
+launch of its own.
+  parallel    x <- x + mixer(norm(x)) + ff(norm(x)): two linears around the mixer's kernels
+  sequential  x <- x + mixer(norm1(x)); x <- x + ff(norm2(x)): two linears around the mixer, two for the feed-forward
+Launches of a mixer in decoding: delta rule 1, decayed outer products 1, grouped-query attention 1, latent attention 4;
+a pass of a looped block adds one linear.
 
 Every row of every bucket is committed (no drafter): a decode bucket is one row per sequence, a prefill bucket
 is `width` ragged rows of up to `nseq` sequences, single decoded tokens beside portions of prompts included.
-Caches and states belong to a layer RUN: the pages of a latent-attention run, the slots of a delta run.
+Caches and states belong to a layer RUN: the pages of an attention run (a run may read those of an earlier one), the
+slots of a recurrent run.
 """
 from __future__ import annotations
 
@@ -21,7 +24,7 @@ from ..ops import functional as F
 from ..ops import layouts as L
 from ..ops import native as N
 from . import stack_weights as SW
-from .stack_config import DeltaMixer, LatentMixer, StackConfig
+from .stack_config import DeltaMixer, GroupedMixer, LatentMixer, OuterMixer, StackConfig
 from .step import BlobLayout, Bucket, finish_bucket, head_outputs, plp_outputs, seam_outputs
 
 
@@ -54,14 +57,18 @@ class StackModel:
         else:
             self.w = SW.random_init(cfg, dtype, dev, seed)
         self.n_slots = max_seqs + 1                       # slot 0 is the null slot
-        self.kv, self.delta_state, self.delta_hist = {}, {}, {}
+        self.kv, self.state, self.hist = {}, {}, {}
         for r in cfg.runs:
             m = cfg.layers[r.layer].mixer
             if isinstance(m, LatentMixer):
                 self.kv[r.index] = torch.zeros(self.kv_blocks, cfg.page_tokens, m.rank_pad + m.rot_pad, dtype=dtype, device=dev)
+            elif isinstance(m, GroupedMixer):
+                if m.kv_from is None:                     # the padding of a page stays zero: the kernels multiply it
+                    self.kv[r.index] = torch.zeros(self.kv_blocks, m.kv_heads, cfg.page_tokens * (m.key_pad + m.vdim_pad), dtype=dtype, device=dev)
             else:
-                self.delta_state[r.index] = torch.zeros(self.n_slots, m.heads, m.vdim_pad, m.dim_pad, dtype=torch.float32, device=dev)
-                self.delta_hist[r.index] = torch.zeros(self.n_slots, m.taps, m.channels, dtype=torch.float32, device=dev)
+                self.state[r.index] = torch.zeros(self.n_slots, m.heads, m.vdim_pad, m.dim_pad, dtype=torch.float32, device=dev)
+                if m.taps:
+                    self.hist[r.index] = torch.zeros(self.n_slots, m.taps, m.channels, dtype=torch.float32, device=dev)
         # expanded keys / values of the pages a prompt portion sees: scratch of one layer run at a time, in
         # physical page order (absent when it would not fit its budget: the absorbed form serves then)
         self.k_exp = self.v_exp = None
@@ -77,18 +84,14 @@ class StackModel:
     # ------------------------------------------------------------------------------ state
     def reset_slot(self, slot: int) -> None:
         with torch.cuda.stream(self.stream):
-            for i in self.delta_state:
-                self.delta_state[i][slot].zero_()
-                self.delta_hist[i][slot].zero_()
+            for t in self.slot_tensors().values():
+                t[slot].zero_()
 
     def page_pools(self) -> dict:
         return {f"kv.{i}": t for i, t in self.kv.items()}
 
     def slot_tensors(self) -> dict:
-        out = {}
-        for i in self.delta_state:
-            out[f"delta_state.{i}"], out[f"delta_hist.{i}"] = self.delta_state[i], self.delta_hist[i]
-        return out
+        return {**{f"state.{i}": t for i, t in self.state.items()}, **{f"hist.{i}": t for i, t in self.hist.items()}}
 
     def snapshot_views(self, slot: int) -> dict:
         return {k: t[slot] for k, t in self.slot_tensors().items()}
@@ -96,7 +99,7 @@ class StackModel:
     def state_bytes(self) -> dict:
         size = lambda d: sum(t.numel() * t.element_size() for t in d.values())    # noqa: E731
         exp = 0 if self.k_exp is None else (self.k_exp.numel() + self.v_exp.numel()) * 2
-        return {"weights": self.w.nbytes(), "kv_pool": size(self.kv), "delta": size(self.delta_state) + size(self.delta_hist),
+        return {"weights": self.w.nbytes(), "kv_pool": size(self.kv), "state": size(self.state) + size(self.hist),
                 "expanded_kv_scratch": exp}
 
     # ------------------------------------------------------------------------------ builders
@@ -169,14 +172,16 @@ class StackModel:
         h = self._operand_buf(M, KW)
         loop_op = self._operand_buf(M, 2 * KW) if cfg.loop is not None else None
         mid = self._operand_buf(M, max(l.out.K for l in w.layers))
+        ups = [l for l in w.layers if l.up is not None]
+        ff = self._operand_buf(M, max(l.down.K for l in ups)) if ups else None
         ldp = max(L.round_up(l.n_plain, 8) for l in w.layers)
         proj = f32(M, ldp)
-        big = max([l.proj.N_pad for l in w.layers] + [l.out.N_pad for l in w.layers] + [w.head.N_pad])
+        big = max([x.N_pad for l in w.layers for x in (l.proj, l.out, l.up) if x is not None] + [w.head.N_pad])
         ws = None
         if self.f32 or not self.fuse:                    # product rows (and, behind them, the split parts)
             ws = torch.empty(M * big + (0 if self.f32 else self.scratch.capacity // 4), dtype=torch.float32, device=dev)
         work = self._mixer_scratch(M, nseq, decode)
-        keep = [blob, x, ss, h, loop_op, mid, proj, ws, work]
+        keep = [blob, x, ss, h, loop_op, mid, ff, proj, ws, work]
         digests = None
         if self.race_check == "shadow":
             digests = torch.zeros(len(cfg.runs) + 1, dtype=torch.int64, device=dev)
@@ -216,19 +221,33 @@ class StackModel:
             e = N.LinEpi()
             self._row_norm(e, ss)
             e.out, e.ldo, e.n_plain, e.act_tile0 = proj.data_ptr(), ldp, lw.n_plain, lw.act_tile0
-            if spec.mlp is not None:
+            e.bias = N.ptr(lw.bias)
+            if spec.mlp is not None and cfg.parallel:
                 e.act, e.act_k0, e.limit, e.alpha = m_op, lw.act_k0, spec.mlp.limit, spec.mlp.alpha
             self._linear(prog, lw.proj, h, M, e, ws, f"{t}.project")
             if isinstance(spec.mixer, DeltaMixer):
                 prog.delta(self._delta_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work), decode, tag=f"{t}.delta")
+            elif isinstance(spec.mixer, OuterMixer):
+                prog.ssd(self._outer_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode), decode, tag=f"{t}.outer")
+            elif isinstance(spec.mixer, GroupedMixer):
+                prog.gqa(self._gqa_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode), tag=f"{t}.attention")
             else:
                 prog.mla(self._mla_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode), tag=f"{t}.latent_attention")
             nxt = runs[i + 1] if i + 1 < len(runs) else None
-            self._linear(prog, lw.out, mid, M, self._stream_epi(x, True, target(nxt)), ws, f"{t}.out")
+            tgt = target(nxt)
+            if lw.up is None:
+                self._linear(prog, lw.out, mid, M, self._stream_epi(x, True, tgt), ws, f"{t}.out")
+            else:
+                self._linear(prog, lw.out, mid, M, self._stream_epi(x, True, (h_op, 0, lw.norm2, ss)), ws, f"{t}.out")
+                e = N.LinEpi()
+                self._row_norm(e, ss)
+                e.act, e.act_kind = self._operand(ff, M, lw.down.K), 1         # (squared ReLU)
+                self._linear(prog, lw.up, h, M, e, ws, f"{t}.up")
+                self._linear(prog, lw.down, ff, M, self._stream_epi(x, True, tgt), ws, f"{t}.down")
             if digests is not None:
                 prog.digest(x, x.numel() * 4, digests.data_ptr() + 8 * run.index, tag=f"{t}.digest")
         b = self._head(prog, key, kind, nseq, width, M, lay, at, blob, blob_host, x, h, ss, ws, keep + [digests], seam, plp, capture)
-        b.arenas = [a for a in (x, ss, h, loop_op, mid, proj) if a is not None]
+        b.arenas = [a for a in (x, ss, h, loop_op, mid, ff, proj) if a is not None]
         b.digests, b.x = digests, x
         return b
 
@@ -237,14 +256,29 @@ class StackModel:
         """Scratch shared by the layers of a bucket, sized for the largest of them."""
         f32 = lambda n: torch.zeros(max(1, n), dtype=torch.float32, device=self.device)   # noqa: E731
         ms = [l.mixer for l in self.cfg.layers]
-        de, la = [m for m in ms if isinstance(m, DeltaMixer)], [m for m in ms if isinstance(m, LatentMixer)]
+        de, la = [m for m in ms if isinstance(m, (DeltaMixer, OuterMixer))], [m for m in ms if isinstance(m, LatentMixer)]
+        outer, gr = [m for m in ms if isinstance(m, OuterMixer)], [m for m in ms if isinstance(m, GroupedMixer)]
         mx = lambda it: max(it, default=0)    # noqa: E731
         wk = {"splits": self._splits(M, decode)}
         if not decode:
+            floats = {id(m): self._chunk_floats(m, M, nseq) for m in outer}
+            scan = [m for m in de if not floats.get(id(m))]
             blk = M // 4 + nseq                           # blocks of four tokens
-            wk["kq"] = f32(blk * mx(m.kv_heads * (8 * m.dim_pad + 16) for m in de))
-            wk["vb"] = f32(blk * mx(m.heads * ((m.vdim_pad + 15) // 16) * 72 for m in de))
+            wk["kq"] = f32(blk * mx(m.kv_heads * (8 * m.dim_pad + 16) for m in scan))
+            wk["vb"] = f32(blk * mx(m.heads * ((m.vdim_pad + 15) // 16) * 72 for m in scan))
             wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in de))
+            wk["chunk"] = f32(mx(floats.values()))
+        elif outer:
+            wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in outer))
+        if outer or gr:                                   # arrivals at the end of a row: zero between launches
+            wk["counters"] = torch.zeros(max(nseq, M * mx(m.kv_heads for m in gr)), dtype=torch.int32, device=self.device)
+        if gr:
+            split = [m for m in gr if self._gqa_form(m, M, decode) == 1]
+            sp = {id(m): self._gqa_splits(m, M) for m in split}
+            wk["gqa_q"] = torch.zeros(max(1, M * mx(m.heads * m.score_dim for m in gr if self._gqa_form(m, M, decode) == 2)), dtype=self.dtype,
+                                      device=self.device)
+            wk["gqa_o"] = f32(M * mx(m.heads * m.vdim_pad * sp[id(m)] for m in split))
+            wk["gqa_ml"] = f32(M * mx(2 * m.heads * sp[id(m)] for m in split))
         wk["q_eff"] = torch.zeros(max(1, M * mx(m.heads * (max(m.rank_pad, m.dim_pad) + m.rot_pad) for m in la)), dtype=self.dtype, device=self.device)
         absorbed = [m for m in la if not self._expanded(m, M, decode)]
         if absorbed:
@@ -265,12 +299,66 @@ class StackModel:
         """Key splits of the absorbed attention: fill the SMs once."""
         return max(1, min(32, F.device_sms() // max(1, M))) if decode or M < 64 else 1
 
+    def _chunk_floats(self, m: OuterMixer, M: int, nseq: int) -> int:
+        """Scratch of the chunk form for prompt portions (0: the scan serves: fp32, or sizes it does not take)."""
+        if self.f32:
+            return 0
+        p = N.SsdParams()
+        p.M, p.nseq, p.H, p.HK, p.N, p.DP, p.V, p.VP, p.taps = M, nseq, m.heads, m.kv_heads, m.dim, m.dim_pad, m.vdim, m.vdim_pad, m.taps
+        return N.lib().saber_ssd_chunk_floats(C.byref(p))
+
+    def _gqa_sizes(self, m: GroupedMixer) -> N.GqaParams:
+        p = N.GqaParams()
+        p.H, p.G, p.D, p.DK, p.KP, p.V, p.VP = m.heads, m.kv_heads, m.dim, m.score_dim, m.key_pad, m.vdim, m.vdim_pad
+        p.page, p.f32, p.scale, p.softcap = self.cfg.page_tokens, int(self.f32), m.scale, m.softcap
+        return p
+
+    def _gqa_form(self, m: GroupedMixer, M: int, decode: bool) -> int:
+        """2: tcgen05 (prompt portions), 1: split keys on mma.sync, 0: any size on the CUDA cores."""
+        form = N.lib().saber_gqa_form(C.byref(self._gqa_sizes(m)))
+        return min(form, 2 if (self.attn_impl == "tc" and not decode and M >= 64) else 1)
+
+    def _gqa_splits(self, m: GroupedMixer, M: int) -> int:
+        """Key splits: fill the SMs twice, never more parts than pages a row can see."""
+        span = self.max_ctx if m.chunk == 0 else min(self.max_ctx, m.chunk + self.cfg.page_tokens - 1)
+        pages = (span + self.cfg.page_tokens - 1) // self.cfg.page_tokens
+        return max(1, min(32, pages, 2 * F.device_sms() // max(1, M * m.kv_heads)))
+
+    def _outer_params(self, run, lw, m: OuterMixer, proj, m_op, M, nseq, lay, at, wk, decode) -> N.SsdParams:
+        p, x = N.SsdParams(), lw.extra
+        p.x, p.ldx = proj.data_ptr(), proj.stride(0)
+        p.q_off, p.k_off, p.v_off, p.g_off, p.dt_off = lw.off["q"], lw.off["k"], lw.off["v"], lw.off["g"], lw.off.get("dt", -1)
+        p.conv_w, p.conv_b, p.decay, p.A_log, p.dt_bias, p.skip = (N.ptr(x.get(k)) for k in ("conv", "conv_b", "decay", "A_log", "dt_bias", "D"))
+        p.norm_w, p.state, p.hist = x["norm"].data_ptr(), self.state[run.index].data_ptr(), N.ptr(self.hist.get(run.index))
+        p.kq, p.vb, p.o, p.counters = N.ptr(wk.get("kq")), N.ptr(wk.get("vb")), wk["o"].data_ptr(), wk["counters"].data_ptr()
+        if not decode and self._chunk_floats(m, M, nseq):
+            p.chunk = wk["chunk"].data_ptr()
+        p.cu_rows, p.slots, p.pos = at(lay.cu_rows), at(lay.slots), at(lay.pos)
+        p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
+        p.H, p.HK, p.N, p.DP, p.V, p.VP, p.taps, p.n_slots = m.heads, m.kv_heads, m.dim, m.dim_pad, m.vdim, m.vdim_pad, m.taps, self.n_slots
+        p.groups, p.gate_first, p.eps, p.err = m.norm_groups, int(m.gate_first), self.cfg.eps, self.scratch.err.data_ptr()
+        return p
+
+    def _gqa_params(self, run, lw, m: GroupedMixer, proj, m_op, M, nseq, lay, at, wk, decode) -> N.GqaParams:
+        p = self._gqa_sizes(m)
+        p.x, p.ldx = proj.data_ptr(), proj.stride(0)
+        p.q_off, p.k_off, p.v_off = lw.off["q"], lw.off.get("k", -1), lw.off.get("v", -1)
+        p.cache, p.q = self.kv[self.cfg.pages_of(run)].data_ptr(), wk["gqa_q"].data_ptr()
+        p.o_part, p.ml, p.counters = wk["gqa_o"].data_ptr(), wk["gqa_ml"].data_ptr(), wk["counters"].data_ptr()
+        p.slot_map, p.pos, p.cu_rows, p.kv_len, p.block_table = (at(o) for o in (lay.slot_map, lay.pos, lay.cu_rows, lay.kv_len, lay.block_table))
+        p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
+        p.n_blocks, p.max_blocks, p.max_rows = self.kv_blocks, self.max_blocks, 1 if decode else M
+        p.form = self._gqa_form(m, M, decode)
+        p.splits = self._gqa_splits(m, M) if p.form == 1 else 1
+        p.qk_norm, p.chunk, p.eps, p.err = int(m.qk_norm), m.chunk, self.cfg.eps, self.scratch.err.data_ptr()
+        return p
+
     def _delta_params(self, run, lw, m: DeltaMixer, proj, m_op, M, nseq, lay, at, wk) -> N.DeltaParams:
         p = N.DeltaParams()
         p.x, p.ldx = proj.data_ptr(), proj.stride(0)
         p.q_off, p.k_off, p.v_off, p.b_off, p.a_off, p.g_off = (lw.off[k] for k in ("q", "k", "v", "b", "a", "g"))
         p.conv_w, p.A_log, p.dt_bias, p.norm_w = (lw.extra[k].data_ptr() for k in ("conv", "A_log", "dt_bias", "norm"))
-        p.hist, p.state = self.delta_hist[run.index].data_ptr(), self.delta_state[run.index].data_ptr()
+        p.hist, p.state = self.hist[run.index].data_ptr(), self.state[run.index].data_ptr()
         p.kq, p.vb, p.o = (N.ptr(wk.get(k)) for k in ("kq", "vb", "o"))
         p.cu_rows, p.slots, p.pos = at(lay.cu_rows), at(lay.slots), at(lay.pos)
         p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq

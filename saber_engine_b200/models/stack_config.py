@@ -1,19 +1,58 @@
-"""Decoders described layer by layer: an ordered list of layers, each with its mixer and feed-forward, an
-optional block of layers that runs several times, and the constants of both.  `models.stack.StackModel` runs
+"""Decoders described layer by layer: an ordered list of layers, each with its mixer and feed-forward (side by
+side behind one norm, or one after the other), an optional block of layers that runs several times, and the
+constants of all of them.  `models.stack.StackModel` runs
 any such description; an architecture is a reader of its `config.json` (ARCHITECTURES) and the order and
 names of its tensors (`models.stack_weights`).
 """
 from __future__ import annotations
 
+import dataclasses
 import json
+import math
 import os
 from dataclasses import dataclass
 from pathlib import Path
 from typing import Optional
 
 
+class Mixer:
+    """What a layer asks of its mixer.  `segments` are the rows of the input projection, in order."""
+    kind = ""
+    kv_from: Optional[int] = None     # layer whose pages this mixer reads (it has none of its own)
+
+    def segments(self) -> list:
+        """(name, rows)"""
+        raise NotImplementedError
+
+    def sources(self) -> list:
+        """(segment, tensor, first row of the tensor): where the projection's rows come from."""
+        return [(name, name, 0) for name, _ in self.segments()]
+
+    def biases(self) -> list:
+        """Segments whose tensor has a bias beside it (its name with '.b')."""
+        return []
+
+    def extra_shapes(self) -> dict:
+        """Tensors beside the projections, name -> shape."""
+        return {}
+
+    def slot_bytes(self) -> int:
+        return 0
+
+    def page_token_bytes(self, elem: int) -> int:
+        return 0
+
+
+def _scan_width(n: int, what: str) -> int:
+    """Key sizes the recurrence kernels are instantiated for."""
+    for w in (64, 128, 192, 256, 384, 512):
+        if w >= n:
+            return w
+    raise ValueError(f"{what}: key size {n} is above 512")
+
+
 @dataclass(frozen=True)
-class DeltaMixer:
+class DeltaMixer(Mixer):
     """Gated delta rule: `kv_heads` query / key heads of size dim, `heads` value heads of size vdim, a causal
     convolution of `taps` over q, k and v."""
     heads: int
@@ -33,11 +72,8 @@ class DeltaMixer:
         return 2 * self.kv_heads * self.dim + self.heads * self.vdim
 
     @property
-    def dim_pad(self) -> int:         # key sizes the kernels are instantiated for
-        for n in (64, 128, 192, 256, 384, 512):
-            if n >= self.dim:
-                return n
-        raise ValueError(f"delta mixer: key size {self.dim} is above 512")
+    def dim_pad(self) -> int:
+        return _scan_width(self.dim, "delta mixer")
 
     @property
     def vdim_pad(self) -> int:
@@ -48,15 +84,16 @@ class DeltaMixer:
         return [("q", self.kv_heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.heads * self.vdim),
                 ("b", self.heads), ("a", self.heads), ("g", self.heads * self.vdim)]
 
+    def extra_shapes(self) -> dict:
+        t = {f"{name}.conv": (rows, self.taps) for name, rows in self.segments()[:3]}
+        return {**t, "A_log": (self.heads,), "dt_bias": (self.heads,), "norm": (self.vdim,)}
+
     def slot_bytes(self) -> int:
         return 4 * (self.heads * self.vdim_pad * self.dim_pad + self.taps * self.channels)
 
-    def page_token_bytes(self, elem: int) -> int:
-        return 0
-
 
 @dataclass(frozen=True)
-class LatentMixer:
+class LatentMixer(Mixer):
     """Latent attention: a cached latent of kv_rank values and one rotated key part of rot_dim per token."""
     heads: int
     dim: int
@@ -94,8 +131,8 @@ class LatentMixer:
     def segments(self) -> list:
         return [("q", self.heads * (self.dim + self.rot_dim)), ("dkv", self.kv_rank + self.rot_dim), ("g", self.heads * self.vdim)]
 
-    def slot_bytes(self) -> int:
-        return 0
+    def extra_shapes(self) -> dict:
+        return {"dkv.norm": (self.kv_rank,), "uk": (self.heads * self.dim, self.kv_rank), "uv": (self.heads * self.vdim, self.kv_rank)}
 
     def page_token_bytes(self, elem: int) -> int:
         return elem * (self.rank_pad + self.rot_pad)
@@ -109,6 +146,109 @@ class LatentMixer:
 
 
 @dataclass(frozen=True)
+class OuterMixer(Mixer):
+    """Decayed outer products: S <- a S + k (w v)^T, o = S^T q, fp32 state of `heads` heads (dim x vdim).
+
+    decay given     constant per head, w = 1; q, k, v are silu of the projection (linear attention)
+    decay None      a and w follow from a step size per token and head, a skip connection, q | k | v pass a causal
+                    convolution of `taps` with a bias (state-space duality)
+    The read-out is normed in `norm_groups` parts; gate_first: silu(gate) ahead of the norm, else sigmoid(gate) after it."""
+    heads: int
+    kv_heads: int                     # key / query heads; value heads share them in equal groups
+    dim: int
+    vdim: int
+    taps: int = 0                     # 0: no convolution
+    decay: Optional[tuple] = None
+    norm_groups: int = 1
+    gate_first: bool = False
+    packed: Optional[str] = None      # one tensor holds gate | v | k | q | dt
+    kind = "outer"
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:        # convolution channels q | k | v
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    @property
+    def dim_pad(self) -> int:
+        return _scan_width(self.dim, "decayed outer products")
+
+    @property
+    def vdim_pad(self) -> int:
+        return (self.vdim + 7) // 8 * 8
+
+    def segments(self) -> list:
+        kd, vd = self.kv_heads * self.dim, self.heads * self.vdim
+        return [("q", kd), ("k", kd), ("v", vd), ("g", vd)] + ([("dt", self.heads)] if self.decay is None else [])
+
+    def sources(self) -> list:
+        if self.packed is None:
+            return super().sources()
+        n, at, out = dict(self.segments()), 0, []
+        for name in ("g", "v", "k", "q", "dt"):
+            out.append((name, self.packed, at))
+            at += n[name]
+        return out
+
+    def extra_shapes(self) -> dict:
+        t = {"norm": (self.heads * self.vdim,)}
+        if self.taps:
+            t["conv"], t["conv.b"] = (self.channels, self.taps), (self.channels,)
+        if self.decay is None:
+            t["dt_bias"] = t["A_log"] = t["D"] = (self.heads,)
+        return t
+
+    def slot_bytes(self) -> int:
+        return 4 * (self.heads * self.vdim_pad * self.dim_pad + self.taps * self.channels)
+
+
+@dataclass(frozen=True)
+class GroupedMixer(Mixer):
+    """Grouped-query attention without rotation: q and k over their root mean square per head, capped scores, keys of the
+    query's own chunk of positions.  kv_from: the pages of that layer are read, with this layer's queries and mask."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float = 0.0              # 0: scores are not capped
+    chunk: int = 0                    # 0: every earlier key
+    qk_norm: bool = True
+    bias: bool = True
+    kv_from: Optional[int] = None
+    kind = "attention"
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def score_dim(self) -> int:       # in whole steps of the tensor cores
+        return (self.dim + 15) // 16 * 16
+
+    @property
+    def key_pad(self) -> int:         # a cached key in whole 64-wide tiles
+        return (self.dim + 63) // 64 * 64
+
+    @property
+    def vdim_pad(self) -> int:
+        return (self.vdim + 31) // 32 * 32
+
+    def segments(self) -> list:
+        q = [("q", self.heads * self.dim)]
+        return q if self.kv_from is not None else q + [("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
+
+    def biases(self) -> list:
+        return [name for name, _ in self.segments()] if self.bias else []
+
+    def page_token_bytes(self, elem: int) -> int:
+        return 0 if self.kv_from is not None else elem * self.kv_heads * (self.key_pad + self.vdim_pad)
+
+
+@dataclass(frozen=True)
 class ClampedGlu:
     """g = min(gate, limit), u = clamp(up, -limit, limit), y = g sigmoid(alpha g) (u + 1)."""
     ff: int
@@ -117,9 +257,15 @@ class ClampedGlu:
 
 
 @dataclass(frozen=True)
+class SquaredRelu:
+    """y = max(up, 0)^2, no gate."""
+    ff: int
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: object
-    mlp: Optional[ClampedGlu] = None
+    mixer: Mixer
+    mlp: object = None                # ClampedGlu, SquaredRelu or None
 
 
 @dataclass(frozen=True)
@@ -147,6 +293,8 @@ class StackConfig:
     layers: tuple
     eps: float = 1e-6
     embed_scale: float = 1.0
+    parallel: bool = True             # mixer and feed-forward side by side behind one norm; else one after the other, a norm each
+    norm_offset: float = 0.0          # norms multiply by offset + weight
     loop: Optional[LoopSpec] = None
     page_tokens: int = 64
     max_ctx: int = 32768
@@ -180,8 +328,30 @@ class StackConfig:
             m = l.mixer
             if isinstance(m, DeltaMixer) and (m.heads % m.kv_heads or m.taps < 1):
                 raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / taps {m.taps}")
+            if isinstance(m, OuterMixer) and (m.heads % m.kv_heads or m.out_features % m.norm_groups or m.taps < 0
+                                              or (m.decay is not None and len(m.decay) != m.heads)):
+                raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / norm_groups {m.norm_groups} / decay {m.decay}")
+            if isinstance(m, GroupedMixer):
+                self._check_grouped(i, m)
+            if self.parallel and l.mlp is not None and not isinstance(l.mlp, ClampedGlu):
+                raise ValueError(f"{self.name}: layer {i}: a feed-forward beside its mixer is a clamped gated unit")
             if isinstance(m, LatentMixer) and (m.rot_dim % 2 or m.kv_rank > 1024 or m.dim > 1024):
                 raise ValueError(f"{self.name}: layer {i}: rot_dim {m.rot_dim}, kv_rank {m.kv_rank}, dim {m.dim}")
+
+    def _check_grouped(self, i: int, m: GroupedMixer) -> None:
+        if m.heads % m.kv_heads or m.chunk < 0 or m.dim > 2048 or m.vdim > 2048:
+            raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / chunk {m.chunk} / dim {m.dim} / vdim {m.vdim}")
+        if m.kv_from is None:
+            return
+        s = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
+        if self.loop is not None or not isinstance(s, GroupedMixer) or s.kv_from is not None or \
+                (s.kv_heads, s.dim, s.vdim) != (m.kv_heads, m.dim, m.vdim):
+            raise ValueError(f"{self.name}: layer {i} cannot read the keys and values of layer {m.kv_from}")
+
+    def pages_of(self, run: LayerRun) -> int:
+        """The run whose pages a run reads."""
+        src = self.layers[run.layer].mixer.kv_from
+        return run.index if src is None else src      # (no loop: runs and layers are the same)
 
     # ---- byte accounting (launch plan)
     def page_token_bytes(self, elem: int = 2) -> int:
@@ -232,7 +402,31 @@ def renosun_from_json(doc: dict, name: str = "renosun", source: Optional[str] = 
                        source=source, max_ctx=max_ctx)
 
 
-ARCHITECTURES = {"Renosun": renosun_from_json}
+# ------------------------------------------------------------------------------------ Tepavik
+def tepavik_from_json(doc: dict, name: str = "tepavik", source: Optional[str] = None, max_ctx: int = 32768) -> StackConfig:
+    layers = []
+    for i, l in enumerate(doc["layers"]):
+        m = l["mixer"]
+        if l["type"] == "lightning":
+            mixer = OuterMixer(m["heads"], m["heads"], m["dim"], m["vdim"], decay=tuple(float(x) for x in m["decay"]))
+        elif l["type"] == "mamba2":
+            mixer = OuterMixer(m["heads"], m["groups"], m["state"], m["vdim"], taps=m["conv"], norm_groups=m["norm_groups"], gate_first=True, packed="in")
+        elif l["type"] == "attention":
+            mixer = GroupedMixer(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), float(m["softcap"]), m["mask"]["size"],
+                                 kv_from=m.get("kv_from"))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
+        mlp = None
+        if l.get("mlp") is not None:
+            if l["mlp"]["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {l['mlp']['kind']!r}")
+            mlp = SquaredRelu(l["mlp"]["ff"])
+        layers.append(LayerSpec(mixer, mlp))
+    return StackConfig(name=name, arch="Tepavik", vocab=doc["vocab"], width=doc["width"], layers=tuple(layers), eps=float(doc["norm"]["eps"]),
+                       parallel=False, norm_offset=1.0, source=source, max_ctx=max_ctx)
+
+
+ARCHITECTURES = {"Renosun": renosun_from_json, "Tepavik": tepavik_from_json}
 
 
 def from_json(doc: dict, **kw) -> StackConfig:
@@ -269,7 +463,38 @@ def renosun_bench(name: str, width: int, ff: int, kv_heads: int, heads: int, att
     return StackConfig(name, "Renosun", vocab=vocab, width=width, layers=layers, embed_scale=width ** 0.5, loop=LoopSpec(n_layers // 4, n_layers // 2, 2))
 
 
-NAMED = {"renosun-mini": renosun_mini,
+def _decays(heads: int) -> tuple:
+    return tuple(math.exp(-2.0 ** (-8.0 * (h + 1) / heads)) for h in range(heads))
+
+
+def tepavik_mini() -> StackConfig:
+    """Small sizes for smoke tests and demos."""
+    ff = SquaredRelu(448)
+    s = LayerSpec(OuterMixer(6, 2, 40, 32, taps=4, norm_groups=3, gate_first=True, packed="in"), ff)
+    r = LayerSpec(OuterMixer(5, 5, 48, 40, decay=_decays(5)), ff)
+    a = GroupedMixer(6, 2, 48, 56, 0.14, 25.0, 192)
+    return StackConfig("tepavik-mini", "Tepavik", vocab=1024, width=288, parallel=False, norm_offset=1.0, max_ctx=4096,
+                       layers=(s, LayerSpec(a, ff), r, LayerSpec(dataclasses.replace(a, kv_from=1, chunk=320), ff)))
+
+
+def tepavik_bench(name: str, width: int, ff: int, heads: int, kv_heads: int, chunk: int = 8192, n_layers: int = 10, vocab: int = 65536) -> StackConfig:
+    """Layers of a real model's size, two rounds of: two state-space layers (inner size 2 x width), attention, linear
+    attention, attention over the keys of the first."""
+    mlp = SquaredRelu(ff)
+    s = LayerSpec(OuterMixer(2 * width // 64, 8, 128, 64, taps=4, norm_groups=8, gate_first=True, packed="in"), mlp)
+    r = LayerSpec(OuterMixer(heads, heads, 128, 128, decay=_decays(heads)), mlp)
+    layers = []
+    for i in range(n_layers):
+        a = GroupedMixer(heads, kv_heads, 128, 128, 128 ** -0.5, 30.0, chunk, kv_from=i - 2 if i % 5 == 4 else None)
+        layers.append({2: LayerSpec(a, mlp), 3: r, 4: LayerSpec(a, mlp)}.get(i % 5, s))
+    return StackConfig(name, "Tepavik", vocab=vocab, width=width, layers=tuple(layers), parallel=False, norm_offset=1.0)
+
+
+NAMED = {"tepavik-mini": tepavik_mini,
+         "tepavik-2k": lambda: tepavik_bench("tepavik-2k", 2048, 8192, 16, 4),
+         "tepavik-4k": lambda: tepavik_bench("tepavik-4k", 4096, 16384, 32, 8),
+         "tepavik-5k": lambda: tepavik_bench("tepavik-5k", 5120, 20480, 40, 8),
+         "renosun-mini": renosun_mini,
          "renosun-2k": lambda: renosun_bench("renosun-2k", 2048, 6144, 8, 16, 16),
          "renosun-4k": lambda: renosun_bench("renosun-4k", 4096, 12288, 16, 32, 32),
          "renosun-5k": lambda: renosun_bench("renosun-5k", 5120, 17408, 16, 48, 40)}

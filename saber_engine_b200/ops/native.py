@@ -172,7 +172,7 @@ class Operand(C.Structure):
 
 class LinEpi(C.Structure):
     _fields_ = [("stream", I), ("ss", P), ("ss_n", I), ("inv_width", F), ("eps", F), ("out", P), ("ldo", I), ("n_plain", I),
-                ("act_tile0", I), ("act", Operand), ("act_k0", I), ("limit", F), ("alpha", F), ("x", P), ("ldx", I), ("width", I),
+                ("act_tile0", I), ("act", Operand), ("act_k0", I), ("act_kind", I), ("limit", F), ("alpha", F), ("x", P), ("ldx", I), ("width", I),
                 ("add", I), ("bias", P), ("norm_w", P), ("op", Operand), ("op_k0", I), ("ss_out", P), ("ss_out_n", I)]
 
 
@@ -194,7 +194,7 @@ class DeltaParams(C.Structure):
     _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("k_off", I), ("v_off", I), ("b_off", I), ("a_off", I), ("g_off", I), ("conv_w", P),
                 ("A_log", P), ("dt_bias", P), ("norm_w", P), ("hist", P), ("state", P), ("kq", P), ("vb", P), ("o", P),
                 ("cu_rows", P), ("slots", P), ("pos", P), ("out", Operand), ("out_k0", I), ("M", I), ("nseq", I), ("H", I), ("HK", I),
-                ("D", I), ("DP", I), ("V", I), ("VP", I), ("taps", I), ("n_slots", I), ("eps", F), ("unit_eps", F), ("q_scale", F), ("err", P)]
+                ("D", I), ("DP", I), ("V", I), ("VP", I), ("taps", I), ("n_slots", I), ("eps", F), ("unit_eps", F), ("q_scale", F), ("skip", P), ("err", P)]
 
 
 class MlaParams(C.Structure):
@@ -203,6 +203,22 @@ class MlaParams(C.Structure):
                 ("cu_rows", P), ("kv_len", P), ("block_table", P), ("out", Operand), ("out_k0", I), ("M", I), ("nseq", I), ("H", I),
                 ("D", I), ("R", I), ("V", I), ("C", I), ("CP", I), ("RP", I), ("DP", I), ("VP", I), ("page", I), ("n_blocks", I),
                 ("max_blocks", I), ("splits", I), ("f32", I), ("expand", I), ("max_rows", I), ("scale", F), ("eps", F), ("err", P)]
+
+
+class SsdParams(C.Structure):
+    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("k_off", I), ("v_off", I), ("dt_off", I), ("g_off", I), ("conv_w", P), ("conv_b", P),
+                ("decay", P), ("A_log", P), ("dt_bias", P), ("skip", P), ("norm_w", P), ("hist", P), ("state", P), ("kq", P), ("vb", P),
+                ("o", P), ("chunk", P), ("counters", P), ("cu_rows", P), ("slots", P), ("pos", P), ("out", Operand), ("out_k0", I),
+                ("M", I), ("nseq", I), ("H", I), ("HK", I), ("N", I), ("DP", I), ("V", I), ("VP", I), ("taps", I), ("groups", I),
+                ("gate_first", I), ("n_slots", I), ("eps", F), ("err", P)]
+
+
+class GqaParams(C.Structure):
+    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("k_off", I), ("v_off", I), ("cache", P), ("q", P), ("o_part", P), ("ml", P),
+                ("counters", P), ("slot_map", P), ("pos", P), ("cu_rows", P), ("kv_len", P), ("block_table", P), ("out", Operand),
+                ("out_k0", I), ("M", I), ("nseq", I), ("H", I), ("G", I), ("D", I), ("DK", I), ("KP", I), ("V", I), ("VP", I), ("page", I),
+                ("n_blocks", I), ("max_blocks", I), ("splits", I), ("f32", I), ("form", I), ("max_rows", I), ("qk_norm", I), ("chunk", I),
+                ("scale", F), ("softcap", F), ("eps", F), ("err", P)]
 
 
 def lib() -> C.CDLL:
@@ -336,6 +352,12 @@ def _declare(L: C.CDLL) -> None:
         "saber_delta_launch": (I, [C.POINTER(DeltaParams), I, S]),
         "saber_mla_expand_ok": (I, [C.POINTER(MlaParams)]),
         "saber_mla_launch": (I, [C.POINTER(MlaParams), S]),
+        "saber_ssd_launch": (I, [C.POINTER(SsdParams), I, S]),
+        "saber_ssd_chunk_floats": (C.c_size_t, [C.POINTER(SsdParams)]),
+        "saber_gqa_form": (I, [C.POINTER(GqaParams)]),
+        "saber_gqa_launch": (I, [C.POINTER(GqaParams), S]),
+        "saber_program_add_ssd": (I, [P, C.POINTER(SsdParams), I, C.c_char_p]),
+        "saber_program_add_gqa": (I, [P, C.POINTER(GqaParams), C.c_char_p]),
         "saber_program_add_linear": (I, [P, C.POINTER(LinParams), C.c_char_p]),
         "saber_program_add_stream_embed": (I, [P, C.POINTER(StreamEmbedParams), C.c_char_p]),
         "saber_program_add_stream_norm": (I, [P, C.POINTER(StreamNormParams), C.c_char_p]),
@@ -516,6 +538,13 @@ class Program:
 
     def mla(self, p: "MlaParams", tag: str = "mla") -> int:
         return self._L.saber_program_add_mla(self._h, C.byref(p), tag.encode())
+
+    # decayed outer products (linear attention, state space) and grouped-query attention over tiled pages
+    def ssd(self, p: "SsdParams", single_row: bool, tag: str = "ssd") -> int:
+        return self._L.saber_program_add_ssd(self._h, C.byref(p), int(single_row), tag.encode())
+
+    def gqa(self, p: "GqaParams", tag: str = "gqa") -> int:
+        return self._L.saber_program_add_gqa(self._h, C.byref(p), tag.encode())
 
     # ---- execution ---------------------------------------------------------------------------
     @property

@@ -258,7 +258,7 @@ def _finish(manifest: Manifest, device: DeviceProfile, cfg, routes: dict, missin
 
 def _resolve_stack(manifest: Manifest, device: DeviceProfile, cfg: StackConfig) -> LaunchPlan:
     """Layer-by-layer models: bf16 linears with one declared variant each (no measured routes), one GPU.  A page
-    holds the latents of every attention run and, where the model expands keys and values for prompts, its share
+    holds the latents, or the keys and values, of every attention run and, where the model expands keys and values for prompts, its share
     of that scratch; a model without attention runs has no page bytes, only block ids."""
     problems = []
     if manifest.tp != 1:
@@ -270,7 +270,7 @@ def _resolve_stack(manifest: Manifest, device: DeviceProfile, cfg: StackConfig) 
     rows = max(max(manifest.prefill_rows), max(manifest.decode_batches))
     led = Ledger(manifest.budget_mib << 20)
     led.bill("weights", cfg.param_count() * 2)
-    led.bill("delta_state_slots", (manifest.max_seqs + 1) * cfg.slot_bytes())
+    led.bill("recurrent_state_slots", (manifest.max_seqs + 1) * cfg.slot_bytes())
     led.bill("prefix_cache_snapshots", manifest.prefix_cache_mib << 20)
     led.bill("activation_arenas", rows * 4 * (3 * cfg.width + 3 * cfg.widest_project() + max(l.mlp.ff if l.mlp else 0 for l in cfg.layers)) * 2)
     led.bill("logits", max(manifest.decode_batches) * cfg.vocab * 4 * 2)

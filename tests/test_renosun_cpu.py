@@ -104,7 +104,7 @@ def test_oracle_prefix_law():
 def test_plan_registry_and_command_line(capsys):
     man = LP.Manifest(model="renosun-mini", max_ctx=2048, max_seqs=4, decode_batches=(1, 4), decode_widths=(1,), prefill_rows=(64,), budget_mib=12000)
     plan = LP.bind(LP.resolve(man))
-    assert plan.kv_blocks >= 2048 // 64 + 1 and plan.ledger.items["delta_state_slots"] == 5 * MC.by_name("renosun-mini").slot_bytes()
+    assert plan.kv_blocks >= 2048 // 64 + 1 and plan.ledger.items["recurrent_state_slots"] == 5 * MC.by_name("renosun-mini").slot_bytes()
     man.decode_widths, man.tp = (1, 5), 2
     with pytest.raises(LP.PlanError) as ei:
         LP.resolve(man)

@@ -412,7 +412,7 @@ def tepavik_from_json(doc: dict, name: str = "tepavik", source: Optional[str] = 
         elif l["type"] == "mamba2":
             mixer = OuterMixer(m["heads"], m["groups"], m["state"], m["vdim"], taps=m["conv"], norm_groups=m["norm_groups"], gate_first=True, packed="in")
         elif l["type"] == "attention":
-            mixer = GroupedMixer(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), float(m["softcap"]), m["mask"]["size"],
+            mixer = GroupedMixer(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), float(m.get("softcap") or 0.0), (m.get("mask") or {}).get("size", 0),
                                  kv_from=m.get("kv_from"))
         else:
             raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")

@@ -1,4 +1,5 @@
-"""Throughput of a layer-by-layer model beside the int4 hybrid decoder at equal layer sizes.
+"""Throughput of a layer-by-layer model beside its closest relatives at equal layer sizes: Renosun beside the int4
+hybrid decoder, Tepavik beside Renosun and the hybrid decoder.
 
 Prefill: a cold prompt in portions of one rung (device-timed).  Decode: `streams` sequences at the prompt's length,
 one row each (no drafter on either side).  Then every group of launches of one step on its own: the group's
@@ -16,10 +17,10 @@ import torch
 from ..models import config as C
 from ..models.hybrid import HybridModel
 from ..models.stack import StackModel
-from ..models.stack_config import DeltaMixer, LatentMixer, StackConfig
+from ..models.stack_config import (ClampedGlu, DeltaMixer, GroupedMixer, LatentMixer, LayerSpec, OuterMixer, StackConfig)
 from ..models.step import SeqStep, run_bucket
 
-SIZES = ("renosun-2k", "renosun-4k", "renosun-5k")
+SIZES = ("renosun-2k", "renosun-4k", "renosun-5k", "tepavik-2k", "tepavik-4k", "tepavik-5k")
 
 
 def peaks() -> tuple:
@@ -30,27 +31,53 @@ def peaks() -> tuple:
     return 6.65e12, 1.59e15
 
 
+def like_models(cfg: StackConfig) -> list:
+    return [like_hybrid(cfg)] if cfg.arch == "Renosun" else [like_renosun(cfg), like_hybrid(cfg)]
+
+
+def like_renosun(cfg: StackConfig) -> StackConfig:
+    """Renosun with the same width, vocabulary, layers of each sort and attention heads; its gated feed-forward has three
+    matrices where the other has two."""
+    a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, GroupedMixer))
+    mlp = ClampedGlu(cfg.layers[0].mlp.ff * 2 // 3 // 128 * 128, 7.0)
+    d = LayerSpec(DeltaMixer(a.heads, a.heads // 2, 128, 128, 4), mlp)
+    la = LayerSpec(LatentMixer(a.heads, 128, 64, 128, 512, 192 ** -0.5, 1e6), mlp)
+    return StackConfig(f"renosun-like-{cfg.name}", "Renosun", vocab=cfg.vocab, width=cfg.width,
+                       layers=tuple(la if isinstance(l.mixer, GroupedMixer) else d for l in cfg.layers), max_ctx=cfg.max_ctx)
+
+
 def like_hybrid(cfg: StackConfig) -> C.HybridConfig:
-    """The hybrid decoder with the same width, feed-forward, delta heads and number of layer runs; its gated GQA
+    """The hybrid decoder with the same width, feed-forward, recurrent heads of 128 and number of layer runs; its gated GQA
     attention has the same query width in heads of 256 and a quarter as many key heads."""
-    d = next(l.mixer for l in cfg.layers if isinstance(l.mixer, DeltaMixer))
-    a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, LatentMixer))
+    a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, (LatentMixer, GroupedMixer)))
+    d = next((l.mixer for l in cfg.layers if isinstance(l.mixer, DeltaMixer)), None)
+    kh, vh, ff = (d.kv_heads, d.heads, cfg.layers[0].mlp.ff) if d else (a.heads // 2, a.heads, cfg.layers[0].mlp.ff * 2 // 3 // 256 * 256)
     nq = max(4, a.heads * a.dim // 256)
     return C.HybridConfig(name=f"hybrid-like-{cfg.name}", n_layers=len(cfg.runs), hidden=cfg.width, n_q_heads=nq, n_kv_heads=max(1, nq // 4),
-                          head_dim=256, ffn_inter=cfg.layers[0].mlp.ff, vocab=cfg.vocab, gdn_k_heads=d.kv_heads, gdn_v_heads=d.heads,
+                          head_dim=256, ffn_inter=ff, vocab=cfg.vocab, gdn_k_heads=kh, gdn_v_heads=vh,
                           gdn_head_dim=128, max_ctx=cfg.max_ctx)
 
 
+def mixer_name(m) -> str:
+    if isinstance(m, OuterMixer):
+        return "state_space" if m.decay is None else "linear_attention"
+    return m.kind + ("_shared_keys" if m.kv_from is not None else "")
+
+
 def _groups(model, b) -> dict:
-    """Launch ranges of one layer run per group, by tag."""
+    """Launch ranges per group, by tag.  A layer-by-layer model: (group, mixer) of every layer run, "mixer" its kernels."""
     tags = b.program.tags()
     out = {}
     if isinstance(model, StackModel):
-        for g in ("project", "delta", "latent_attention", "out", "loop_in"):
-            idx = [i for i, t in enumerate(tags) if t.endswith("." + g)]
-            if idx:
-                out[g] = [(i, i + 1) for i in idx]
-        out["lm_head"] = [(i, i + 1) for i, t in enumerate(tags) if t == "lm_head"]
+        for i, t in enumerate(tags):
+            part = t.split(".")
+            if part[0][0] == "R" and part[0][1:].isdigit() and part[-1] != "digest":
+                m = model.cfg.layers[int(part[1][1:])].mixer
+                label = part[2] if part[2] in ("project", "out", "up", "down", "loop_in") else "mixer"
+                key = label if label in ("up", "down", "loop_in") else f"{label}:{mixer_name(m)}"
+                out.setdefault(key, []).append((i, i + 1))
+            elif t == "lm_head":
+                out["lm_head"] = [(i, i + 1)]
         return out
     layers = sorted({int(t[1:].split(".")[0]) for t in tags if t[0] == "L" and t[1].isdigit()})
     span = lambda li, keys: [i for i, t in enumerate(tags) if t.startswith(f"L{li}.") and any(k in t for k in keys)]   # noqa: E731
@@ -97,26 +124,30 @@ def _roof(nbytes: float, flops: float) -> float:
 
 
 def stack_costs(cfg: StackConfig, M: int, nseq: int, ctx_pairs: float, ctx_tokens: float) -> dict:
-    """Algorithmic (bytes, FLOPs) per launch of each group.  ctx_pairs: visible (row, key) pairs; ctx_tokens: keys read."""
-    W, out = cfg.width, {}
-    d = next(l for l in cfg.layers if isinstance(l.mixer, DeltaMixer))
-    a = next(l for l in cfg.layers if isinstance(l.mixer, LatentMixer))
-    segs = sum(n for _, n in d.mixer.segments())
-    n = segs + 2 * d.mlp.ff
-    out["project"] = (2 * n * W + M * (2 * W + 4 * segs + 2 * d.mlp.ff), 2.0 * M * n * W)
-    k = d.mixer.out_features + d.mlp.ff
-    out["out"] = (2 * k * W + M * (2 * k + 8 * W + 2 * W), 2.0 * M * k * W)
-    out["loop_in"] = (4 * W * W + M * (4 * W + 6 * W), 4.0 * M * W * W)
-    m = d.mixer
-    out["delta"] = (2 * 4 * nseq * m.heads * m.dim * m.vdim + M * (4 * (segs + m.out_features) + 2 * m.out_features),
-                    M * m.heads * m.dim * m.vdim * 8.0)
-    m = a.mixer
-    pair = 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim)
-    carry = 2.0 * ctx_tokens * m.heads * (m.dim + m.vdim) * m.kv_rank if M > 64 else 2.0 * M * m.heads * (m.dim + m.vdim) * m.kv_rank
-    if M <= 64:
-        pair = 2.0 * m.heads * (2 * m.kv_rank + m.rot_dim)
-    out["latent_attention"] = (2 * ctx_tokens * (m.kv_rank + m.rot_dim) + 2 * m.heads * (m.dim + m.vdim) * m.kv_rank
-                               + M * (4 * m.heads * (m.dim + m.rot_dim + m.vdim) + 2 * m.heads * m.vdim), ctx_pairs * pair + carry)
+    """Algorithmic (bytes, FLOPs) per launch group.  ctx_pairs: visible (row, key) pairs; ctx_tokens: keys read."""
+    W, out = cfg.width, {"loop_in": (4 * cfg.width ** 2 + M * 10 * cfg.width, 4.0 * M * cfg.width ** 2)}
+    for l in cfg.layers:
+        m, ff = l.mixer, l.mlp.ff
+        name = mixer_name(m)
+        segs = sum(n for _, n in m.segments())
+        n, k = (segs + 2 * ff, m.out_features + ff) if cfg.parallel else (segs, m.out_features)
+        out[f"project:{name}"] = (2 * n * W + M * (2 * W + 4 * segs + (2 * ff if cfg.parallel else 0)), 2.0 * M * n * W)
+        out[f"out:{name}"] = (2 * k * W + M * (2 * k + 8 * W + 2 * W), 2.0 * M * k * W)
+        out["up"] = (2 * ff * W + M * (2 * W + 2 * ff), 2.0 * M * ff * W)
+        out["down"] = (2 * ff * W + M * (2 * ff + 8 * W + 2 * W), 2.0 * M * ff * W)
+        if isinstance(m, (DeltaMixer, OuterMixer)):
+            out[f"mixer:{name}"] = (2 * 4 * nseq * m.heads * m.dim * m.vdim + M * (4 * segs + 2 * m.out_features),
+                                    M * m.heads * m.dim * m.vdim * (8.0 if isinstance(m, DeltaMixer) else 4.0))
+        elif isinstance(m, GroupedMixer):
+            out[f"mixer:{name}"] = (2 * ctx_tokens * m.kv_heads * (m.dim + m.vdim) + M * (4 * segs + 2 * m.out_features),
+                                    ctx_pairs * 2.0 * m.heads * (m.dim + m.vdim))
+        else:
+            pair = 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim)
+            carry = 2.0 * ctx_tokens * m.heads * (m.dim + m.vdim) * m.kv_rank if M > 64 else 2.0 * M * m.heads * (m.dim + m.vdim) * m.kv_rank
+            if M <= 64:
+                pair = 2.0 * m.heads * (2 * m.kv_rank + m.rot_dim)
+            out[f"mixer:{name}"] = (2 * ctx_tokens * (m.kv_rank + m.rot_dim) + 2 * m.heads * (m.dim + m.vdim) * m.kv_rank
+                                    + M * (4 * m.heads * (m.dim + m.rot_dim + m.vdim) + 2 * m.heads * m.vdim), ctx_pairs * pair + carry)
     out["lm_head"] = (2 * cfg.vocab * W, 2.0 * min(M, 8) * cfg.vocab * W)
     return out
 
@@ -211,7 +242,7 @@ def run(args) -> dict:
            "models": {}}
     for n in names:
         cfg = C.by_name(n)
-        for c in (cfg, like_hybrid(cfg)):
+        for c in (cfg, *like_models(cfg)):
             out["models"][c.name] = measure(c, args.prompt, args.streams, args.rung, args.steps, args.warmup, True)
             torch.cuda.empty_cache()
     return out

@@ -414,7 +414,7 @@ static int split_go(const GqaParams& p, cudaStream_t stream) {
     if (e != cudaSuccess) return static_cast<int>(e);
     ready[dev] = true;
   }
-  return static_cast<int>(launch(gqa_split_kernel<MT, NC>, dim3(p.M, p.G, p.splits), dim3(128), split_smem(p), stream, 0, p));
+  return static_cast<int>(launch(gqa_split_kernel<MT, NC>, dim3(p.M, p.G, p.splits), dim3(128), split_smem(p), stream, 2, p));
 }
 template <int NC>
 static int split_mt(const GqaParams& p, cudaStream_t s) {

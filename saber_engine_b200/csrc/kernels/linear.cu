@@ -145,6 +145,9 @@ __device__ __forceinline__ void linear_tile_epilogue(const LinEpi& e, const floa
 template <int kMT>
 __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_constant__ LinParams p, const int stages) {
   extern __shared__ uint8_t smem_raw[];
+  // one round of CTAs: the successor may take the SMs this grid leaves idle or frees (until its own wait it touches
+  // weights only)
+  if (gridDim.x == 1) pdl_trigger();
   __shared__ uint64_t bars[2 * kLinMaxStages + 1];
   __shared__ uint32_t tmem_base_s, is_last_s, abort_s;
   __shared__ float scale_s[256];

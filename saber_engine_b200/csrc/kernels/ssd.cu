@@ -5,8 +5,8 @@
 //   scan   that scan without its correction term: four tokens at a time, a warp per four value columns, the state in
 //          registers (fp32 models and sizes the chunk form of ssd_chunk.cu does not take)
 //   out    gate and grouped norm into the operand of the output linear; the convolution inputs go to the ring
-// Decoding (one row per sequence): one launch, a CTA per (head, sequence); the last CTA of a sequence to finish norms
-// its row.
+// Decoding (one row per sequence): one launch, a CTA per (head, sequence); the last CTA of a norm group to
+// finish norms it.
 #include "delta.h"
 #include "launch.cuh"
 #include "ssd_chunk.h"
@@ -97,21 +97,62 @@ __device__ __forceinline__ float block_sum(float v, float* red, int nw) {
   return v;
 }
 
-// Gate and norm of one group of a row: val(i) gives read-out value i of the group's n.
-template <typename Val>
-__device__ __forceinline__ void ssd_gated_norm(const SsdParams& p, const Val& val, int m, int grp, int n, float* red) {
-  const int nt = blockDim.x;
-  const float* g = p.x + static_cast<size_t>(m) * p.ldx + p.g_off + grp * n;
-  auto gated = [&](int i) { return p.gate_first ? val(i) * silu_f32(g[i]) : val(i); };
+// Gate and norm of one group of a row (o: the row's read-outs [H][VP], n values of the group).
+__device__ __forceinline__ void ssd_gated_norm(const SsdParams& p, const float* o, int m, int grp, int n, float* red) {
+  const int nt = blockDim.x, c0 = grp * n, k0 = p.out_k0 + c0;
+  const float* g = p.x + static_cast<size_t>(m) * p.ldx + p.g_off + c0;
+  const float* w = p.norm_w + c0;
+  constexpr int kHeld = 4;                         // values held per thread, in groups of four
+  if (((p.V | n) & 3) == 0 && n <= 4 * kHeld * nt) {
+    float4 v[kHeld], gate[kHeld];
+#pragma unroll
+    for (int u = 0; u < kHeld; ++u) {
+      const int i = (u * nt + threadIdx.x) * 4, c = c0 + i, h = c / p.V;
+      v[u] = gate[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < n) {
+        v[u] = __ldcg(reinterpret_cast<const float4*>(o + h * p.VP + c - h * p.V));
+        gate[u] = *reinterpret_cast<const float4*>(g + i);
+      }
+    }
+    float sq = 0.f;
+#pragma unroll
+    for (int u = 0; u < kHeld; ++u) {
+      if (p.gate_first) {
+        v[u].x *= silu_f32(gate[u].x);
+        v[u].y *= silu_f32(gate[u].y);
+        v[u].z *= silu_f32(gate[u].z);
+        v[u].w *= silu_f32(gate[u].w);
+      }
+      sq += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+    }
+    const float r = 1.f / sqrtf(block_sum(sq, red, nt >> 5) / static_cast<float>(n) + p.eps);
+#pragma unroll
+    for (int u = 0; u < kHeld; ++u) {
+      const int i = (u * nt + threadIdx.x) * 4;
+      if (i >= n) break;
+      const float4 wt = *reinterpret_cast<const float4*>(w + i);
+      float4 y = make_float4(v[u].x * r * wt.x, v[u].y * r * wt.y, v[u].z * r * wt.z, v[u].w * r * wt.w);
+      if (!p.gate_first) {
+        y.x *= sigmoid_f32(gate[u].x);
+        y.y *= sigmoid_f32(gate[u].y);
+        y.z *= sigmoid_f32(gate[u].z);
+        y.w *= sigmoid_f32(gate[u].w);
+      }
+      operand_store4(p.out, m, k0 + i, y);
+    }
+    return;
+  }
+  auto gated = [&](int i) {
+    const int c = c0 + i, h = c / p.V;
+    const float v = __ldcg(o + h * p.VP + c - h * p.V);
+    return p.gate_first ? v * silu_f32(g[i]) : v;
+  };
   float sq = 0.f;
   for (int i = threadIdx.x; i < n; i += nt) {
     const float v = gated(i);
     sq += v * v;
   }
-  sq = block_sum(sq, red, nt >> 5);
-  const float r = 1.f / sqrtf(sq / static_cast<float>(n) + p.eps);
-  const float* w = p.norm_w + grp * n;
-  const int k0 = p.out_k0 + grp * n;
+  const float r = 1.f / sqrtf(block_sum(sq, red, nt >> 5) / static_cast<float>(n) + p.eps);
   for (int i = threadIdx.x; i < n; i += nt) {
     const float y = gated(i) * r * w[i];
     operand_store1(p.out, m, k0 + i, p.gate_first ? y : y * sigmoid_f32(g[i]));
@@ -123,10 +164,9 @@ __global__ void __launch_bounds__(256) ssd_out_kernel(const __grid_constant__ Ss
   pdl_wait();
   __shared__ float red[8];
   if (static_cast<int>(blockIdx.x) < p.M) {
-    const int m = blockIdx.x, n = p.H * p.V / p.groups, c0 = blockIdx.y * n;
+    const int m = blockIdx.x;
     if (seq_of_row(p.cu_rows, p.nseq, m) < 0) return;
-    const float* o = p.o + static_cast<size_t>(m) * p.H * p.VP;
-    ssd_gated_norm(p, [&](int i) { const int c = c0 + i, h = c / p.V; return o[h * p.VP + c - h * p.V]; }, m, blockIdx.y, n, red);
+    ssd_gated_norm(p, p.o + static_cast<size_t>(m) * p.H * p.VP, m, blockIdx.y, p.H * p.V / p.groups, red);
     return;
   }
   if (p.taps == 0) return;
@@ -147,7 +187,7 @@ __global__ void __launch_bounds__(256) ssd_out_kernel(const __grid_constant__ Ss
 
 // One row per sequence: grid (H, nseq), 32 * min(8, VP / 8) threads.  A warp owns eight value columns at a time, eight
 // lanes along the keys and two columns each.
-template <int NI>
+template <int NI, int TAPS>
 __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ SsdParams p) {
   pdl_wait();
   extern __shared__ float4 sm4[];
@@ -186,7 +226,7 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ S
     float y[1] = {0.f};
     if (n < p.N) {
       const int c = (isk * p.HK + hk) * p.N + n;
-      ssd_inputs<1, 0>(p, hist, c, m, 0, pos, C, 1, y);
+      ssd_inputs<1, TAPS>(p, hist, c, m, 0, pos, C, 1, y);
       if (p.taps && h % share == 0) hist[now + c] = x[ssd_column(p, c)];      // ring row of this token: no head of this step reads it
     }
     (isk ? ks : qs)[n] = y[0];
@@ -195,7 +235,7 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ S
     float y[1] = {0.f};
     if (d < p.V) {
       const int c = 2 * p.HK * p.N + h * p.V + d;
-      ssd_inputs<1, 0>(p, hist, c, m, 0, pos, C, 1, y);
+      ssd_inputs<1, TAPS>(p, hist, c, m, 0, pos, C, 1, y);
       if (p.taps) hist[now + c] = x[ssd_column(p, c)];
     }
     vs[d] = y[0];
@@ -231,28 +271,28 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ S
     }
     if (lg < 2) __stcg(row + cb + cl + lg, fmaf(skip, vs[cb + cl + lg], lg ? o[1] : o[0]));
   }
-  // the last head of the sequence to arrive norms the row
+  // the last head to arrive norms the row, or the norm group where groups hold whole heads
+  const int parts = p.H % p.groups == 0 ? p.groups : 1, per = p.H / parts, part = h / per;
   __threadfence();
   __syncthreads();
   if (threadIdx.x == 0) {
-    const bool last = atomicAdd(p.counters + j, 1u) == static_cast<uint32_t>(p.H) - 1u;
-    if (last) p.counters[j] = 0u;
+    uint32_t* cnt = p.counters + j * parts + part;
+    const bool last = atomicAdd(cnt, 1u) == static_cast<uint32_t>(per) - 1u;
+    if (last) *cnt = 0u;
     __threadfence();
     last_s = last ? 1u : 0u;
   }
   __syncthreads();
   if (!last_s) return;
-  const int n = p.H * p.V / p.groups;
-  const float* o = p.o + static_cast<size_t>(m) * p.H * p.VP;
-  for (int g = 0; g < p.groups; ++g) {
-    const int c0 = g * n;
-    ssd_gated_norm(p, [&](int i) { const int c = c0 + i, hh = c / p.V; return __ldcg(o + hh * p.VP + c - hh * p.V); }, m, g, n, red);
-  }
+  for (int g = part; g < p.groups; g += parts)
+    ssd_gated_norm(p, p.o + static_cast<size_t>(m) * p.H * p.VP, m, g, p.H * p.V / p.groups, red);
 }
 
 template <int NI>
 static cudaError_t ssd_step(const SsdParams& p, cudaStream_t stream) {
-  return launch(ssd_step_kernel<NI>, dim3(p.H, p.nseq), dim3(32 * (p.VP / 8 < 8 ? p.VP / 8 : 8)), (2 * NI * 32 + p.VP) * 4, stream, 0, p);
+  const dim3 grid(p.H, p.nseq), block(32 * (p.VP / 8 < 8 ? p.VP / 8 : 8));
+  const int smem = (2 * NI * 32 + p.VP) * 4;
+  return p.taps == 4 ? launch(ssd_step_kernel<NI, 4>, grid, block, smem, stream, 2, p) : launch(ssd_step_kernel<NI, 0>, grid, block, smem, stream, 2, p);
 }
 template <int NI>
 static cudaError_t ssd_prep(const SsdParams& p, cudaStream_t stream) {

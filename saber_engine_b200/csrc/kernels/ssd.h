@@ -32,7 +32,7 @@ struct SsdParams {
   float* vb;
   float* o;                // scratch [M][H][VP]
   float* chunk;            // scratch of the chunk form (null: the scan)
-  uint32_t* counters;      // [nseq], zero between launches
+  uint32_t* counters;      // [nseq][groups], zero between launches
   const int32_t* cu_rows;  // [nseq + 1]
   const int32_t* slots;    // [nseq], < 0: padding sequence
   const int32_t* pos;      // [M]

@@ -271,7 +271,7 @@ class StackModel:
         elif outer:
             wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in outer))
         if outer or gr:                                   # arrivals at the end of a row: zero between launches
-            wk["counters"] = torch.zeros(max(nseq, M * mx(m.kv_heads for m in gr)), dtype=torch.int32, device=self.device)
+            wk["counters"] = torch.zeros(max(nseq * mx(m.norm_groups for m in outer), M * mx(m.kv_heads for m in gr)), dtype=torch.int32, device=self.device)
         if gr:
             split = [m for m in gr if self._gqa_form(m, M, decode) == 1]
             sp = {id(m): self._gqa_splits(m, M) for m in split}

@@ -104,6 +104,79 @@ def test_linear_bias_and_squared_relu(M, N, K, splits, fuse):
     assert (got[:, :ff].double() - sq).abs().max() < 0.01 * sq.abs().max() and torch.all(got[:, ff:] == 0)
 
 
+@pytest.mark.parametrize("H,HK,N,V,lens", [(4, 2, 24, 40, (200,)), (3, 3, 128, 100, (64, 1, 130)), (2, 1, 200, 24, (63, 65)), (2, 2, 250, 64, (150,))])
+def test_chunk_form_keeps_fp32_digits(H, HK, N, V, lens):
+    """q, k, v in bf16 and everything else in fp32: against float64 on the rounded inputs, the chunk form is as close as
+    fp32 sums are, with decays from none to total inside one chunk, and carries the state over."""
+    from saber_engine_b200.models.stack_config import OuterMixer
+    from saber_engine_b200.ops import functional as F
+    from saber_engine_b200.ops import native as NN
+    g = torch.Generator().manual_seed(H + N)
+    mix = OuterMixer(H, HK, N, V)
+    DP, VP, M, nseq = mix.dim_pad, mix.vdim_pad, sum(lens), len(lens)
+    cols, off = 0, {}
+    for name, n in mix.segments():
+        off[name] = cols
+        cols = (cols + n + 7) // 8 * 8
+    x = torch.randn(M, cols, generator=g)
+    end = off["v"] + H * V                                       # inputs whose silu is a bf16 number: no doubt about its rounding
+    y = O.silu(x[:, :end].double().clamp(min=-1.0)).bfloat16().double()
+    z = x[:, :end].double().clamp(min=-1.0)
+    for _ in range(30):
+        sg = torch.sigmoid(z)
+        z = z - (z * sg - y) / (sg * (1 + z * (1 - sg)))
+    x[:, :end] = z.float()
+    x[:, off["dt"]:off["dt"] + H] = torch.randn(M, H, generator=g) * 4
+    A_log, dt_bias, skip = torch.randn(H, generator=g) * 2, torch.randn(H, generator=g), torch.randn(H, generator=g)
+    S0 = torch.randn(nseq, H, V, N, generator=g)
+    state = torch.zeros(nseq + 1, H, VP, DP)
+    state[1:, :, :V, :N] = S0
+    dev = {k: v.float().cuda() for k, v in dict(x=x, A=A_log, b=dt_bias, d=skip, st=state, nw=torch.ones(H * V)).items()}
+    cu = torch.tensor([0] + [sum(lens[:i + 1]) for i in range(nseq)], dtype=torch.int32).cuda()
+    slots = torch.arange(1, nseq + 1, dtype=torch.int32).cuda()
+    pos = torch.cat([torch.arange(n) for n in lens]).int().cuda()
+    o, out = torch.zeros(M, H, VP, device="cuda"), torch.zeros(M, H * V, device="cuda")
+    p = NN.SsdParams()
+    p.x, p.ldx, p.q_off, p.k_off, p.v_off, p.dt_off, p.g_off = dev["x"].data_ptr(), cols, off["q"], off["k"], off["v"], off["dt"], off["g"]
+    p.A_log, p.dt_bias, p.skip, p.norm_w, p.state, p.o = (t.data_ptr() for t in (dev["A"], dev["b"], dev["d"], dev["nw"], dev["st"], o))
+    p.cu_rows, p.slots, p.pos, p.M, p.nseq = cu.data_ptr(), slots.data_ptr(), pos.data_ptr(), M, nseq
+    p.out.p, p.out.M_pad, p.out.ld, p.out.fmt = out.data_ptr(), M, H * V, 1
+    p.H, p.HK, p.N, p.DP, p.V, p.VP, p.taps, p.groups, p.n_slots, p.eps = H, HK, N, DP, V, VP, 0, 1, nseq + 1, 1e-5
+    sc = F.scratch("cuda")
+    p.err = sc.err.data_ptr()
+    chunk = torch.zeros(NN.lib().saber_ssd_chunk_floats(C.byref(p)), device="cuda")
+    p.chunk = chunk.data_ptr()
+    NN.check(NN.lib().saber_ssd_launch(C.byref(p), 0, NN.stream_handle()), "ssd")
+    torch.cuda.synchronize()
+    sc.check()
+    xd = x.double()
+    act = lambda n, h, d: O.silu(x[:, off[n]:off[n] + h * d]).bfloat16().double().view(M, h, d)      # noqa: E731
+    q, k, v = (a[:, torch.arange(H) // (H // a.shape[1])] for a in (act("q", HK, N), act("k", HK, N), act("v", H, V)))
+    dt = O.softplus(xd[:, off["dt"]:off["dt"] + H] + dt_bias.double())
+    a = torch.exp(-torch.exp(A_log.double()) * dt)
+    for s, n in enumerate(lens):
+        r0, S = int(cu[s]), S0[s].double()
+        want = torch.zeros(n, H, V).double()
+        for t in range(n):
+            S = a[r0 + t][:, None, None] * S + (dt[r0 + t][:, None] * v[r0 + t])[:, :, None] * k[r0 + t][:, None, :]
+            want[t] = torch.einsum("hvn,hn->hv", S, q[r0 + t]) + skip.double()[:, None] * v[r0 + t]
+        got = o[r0: r0 + n, :, :V].cpu().double()
+        assert (got - want).abs().max() < 2e-6 * want.abs().max(), s
+        back = dev["st"][s + 1, :, :V, :N].cpu().double()
+        assert (back - S).abs().max() < 2e-6 * S.abs().max(), s
+
+
+def test_scan_serves_sizes_the_chunk_form_does_not():
+    cfg = R.config([R.mamba(heads=2, groups=1, state=300, ff=None)])
+    t = R.tensors(cfg, 4)
+    toks = R.tokens(cfg, 130)
+    eng = R.engine(cfg, t, BF16)
+    assert eng.model._chunk_floats(eng.model.cfg.layers[0].mixer, 256, 4) == 0
+    want = O.Oracle(cfg, t).forward(toks)
+    for cuts in ([130], [70, 1]):
+        assert R.error(R.feed(eng, "r", toks, cuts), want) < R.TOL[BF16]
+
+
 # ------------------------------------------------------------------------------ whole models
 @pytest.fixture(scope="module", params=list(R.CASES))
 def case(request):

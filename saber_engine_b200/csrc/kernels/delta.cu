@@ -244,29 +244,6 @@ __device__ __forceinline__ void delta_state_io(float* st, float (&S)[NI][4][2], 
     }
 }
 
-// Pairs of fp32 in one register pair: the two halves of an instruction are two ordinary fp32 operations.
-typedef unsigned long long f32x2;
-__device__ __forceinline__ f32x2 pack_f2(float a, float b) {
-  f32x2 r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ float2 unpack_f2(f32x2 v) {
-  float2 r;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-  return r;
-}
-__device__ __forceinline__ f32x2 fma_f2(f32x2 a, f32x2 b, f32x2 c) {
-  f32x2 r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-__device__ __forceinline__ f32x2 mul_f2(f32x2 a, f32x2 b) {
-  f32x2 r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-
 constexpr int kScanStages = 4;           // blocks of four tokens in flight
 
 // grid (nseq, H, ceil(VP / 16)), 160 threads: four warps of four value columns (two lane groups of two columns, 16 lanes

@@ -6,8 +6,8 @@
 //              [page][value row][64 keys], both stored swizzled, two stages each
 //   warp 1     one lane issues S = Q K^T into one of two 128-column score buffers, a tile ahead of the softmax,
 //              and O += P V with P in tensor memory
-//   warps 2-5  softmax, a query row per thread: scores from tensor memory, running maximum, bf16 probabilities
-//              back to tensor memory.  O is rescaled only when a row's maximum has grown by more than 2^8 since the
+//   warps 2-9  softmax, two threads per query row, half of the keys each: scores from tensor memory, running maximum
+//              (the halves meet in shared memory), bf16 probabilities back to tensor memory.  O is rescaled only when a row's maximum has grown by more than 2^8 since the
 //              factor in use was chosen (the factor cancels in the division at the end).
 #include "flash_tc.h"
 #include "launch.cuh"
@@ -15,7 +15,7 @@
 
 namespace saber {
 
-constexpr int kTcThreads = 192;
+constexpr int kTcThreads = 320;
 constexpr int kTcKeys = 128;
 constexpr float kTcLog2e = 1.4426950408889634f;
 constexpr float kTcSlack = 8.f;
@@ -35,12 +35,20 @@ __device__ __forceinline__ void mma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, ui
 // cap tanh(z s) from 2^(2 z s log2 e): zs is 2 z log2 e.  (Large sums give cap, tiny ones -cap.)
 __device__ __forceinline__ float soft_cap(float s, float zs, float cap) { return cap - __fdividef(2.f * cap, 1.f + ex2(s * zs)); }
 
+// tanh(z) = z P(z^2) for |z| <= 0.75 to a relative error of 1e-7: interpolation of tanh(z) / z in the Chebyshev points
+// of z^2, in powers of z^2
+constexpr float kTanhReach = 0.75f;
+constexpr int kTanhTerms = 7;
+__constant__ float kTanh[kTanhTerms] = {1.f, -0.33333307505f, 0.13332590461f, -0.05388652161f, 0.02143389918f, -0.00763178663f, 0.00172316108f};
+
 // grid (query tiles of the longest possible portion, H, nseq)
 __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_constant__ FlashParams p) {
   pdl_wait();
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t bars[16];
   __shared__ uint32_t tmem_base_s;
+  __shared__ volatile uint32_t abort_s[4];          // per pair of softmax warps
+  __shared__ float half_s[2][2][128];               // [block parity][half of the keys][row]
   const int h = blockIdx.y, j = blockIdx.z;
   const int r0 = p.cu_rows[j], nrows = p.cu_rows[j + 1] - r0;
   const int tiles = (nrows + 127) / 128;
@@ -67,9 +75,10 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
       mbar_init(vfull + 8 * i, 1);
       mbar_init(vfree + 8 * i, 1);
       mbar_init(sfull + 8 * i, 1);
-      mbar_init(sfree + 8 * i, 4);
+      mbar_init(sfree + 8 * i, 8);
     }
-    mbar_init(pfull, 4);
+    for (int i = 0; i < 4; ++i) abort_s[i] = 0u;
+    mbar_init(pfull, 8);
     mbar_init(odone, 1);
     mbar_init(bend, 1);
     mbar_init_fence();
@@ -80,7 +89,7 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
   }
   // query tile, swizzled; columns past DK and rows past the live ones are zeros
   const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + (static_cast<size_t>(m0) * p.H + h) * DK;
-  for (int r = warp; r < 128; r += 6)
+  for (int r = warp; r < 128; r += 10)
     for (int c = lane; c < KB * 8; c += 32) {
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (r < rows && c * 8 < DK) v = *reinterpret_cast<const uint4*>(qg + static_cast<size_t>(r) * p.H * DK + c * 8);
@@ -164,26 +173,43 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
     }
   } else {
     // ---------------------------------------------------------------- softmax
-    const int q4 = warp & 3, row = q4 * 32 + lane;
+    const int q4 = warp & 3, row = q4 * 32 + lane, half = (warp - 2) >> 2;
     const uint32_t lane_off = static_cast<uint32_t>(q4 * 32) << 16;
-    const bool capped = p.softcap > 0.f;
-    const float sc = capped ? kTcLog2e : p.scale * kTcLog2e, zs = capped ? 2.f * kTcLog2e * p.scale / p.softcap : 0.f;
+    const bool capped = p.softcap > 0.f, series = capped && p.bound > 0.f && fabsf(p.scale) * p.bound <= kTanhReach * p.softcap;
+    // scores in the base-2 domain: sc times what v holds (1 where the cap already brought them there)
+    const float sc = series ? 1.f : capped ? kTcLog2e : p.scale * kTcLog2e, zs = capped ? 2.f * kTcLog2e * p.scale / p.softcap : 0.f;
+    f32x2 co[kTanhTerms];
+    {
+      const float z2 = capped ? (p.scale / p.softcap) * (p.scale / p.softcap) : 0.f;
+      float f = p.scale * kTcLog2e;
+#pragma unroll
+      for (int i = 0; i < kTanhTerms; ++i) {
+        co[i] = pack_f2(kTanh[i] * f, kTanh[i] * f);
+        f *= z2;
+      }
+    }
     // (a row may meet blocks ahead of its first key: the maximum starts finite so that differences stay numbers)
     float mx = kTcNone, used = kTcNone, l = 0.f;
     const int low = p.chunk > 0 ? (pos0 + row) - (pos0 + row) % p.chunk : 0;   // first key of this row
     const int low_last = p.chunk > 0 ? (pos0 + q4 * 32 + 31) - (pos0 + q4 * 32 + 31) % p.chunk : 0;
+    // A wait that runs out ends both warps of a row: the one that gives up arrives at their next meeting without waiting.
+    auto give_up = [&]() {
+      abort_s[q4] = 1u;
+      __threadfence_block();
+      named_bar_arrive(1 + q4, 64);
+    };
     bool ok = true;
     for (int b = 0; b < blocks; ++b) {
       const int s = b & 1;
       // (waits are decided by the warp as a whole: tensor-memory accesses need all its lanes together)
       ok = __all_sync(0xffffffffu, mbar_wait(sfull + 8 * s, (b >> 1) & 1, p.err, kErrWaitAcc));
-      if (!ok) break;
+      if (!ok) { give_up(); break; }
       tc_fence_after_sync();
-      float v[128];
+      float v[64];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < 2; ++c) {
         uint32_t r[32];
-        tmem_ld32(tm + lane_off + s * 128 + c * 32, r);
+        tmem_ld32(tm + lane_off + s * 128 + half * 64 + c * 32, r);
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 32; ++i) v[c * 32 + i] = __uint_as_float(r[i]);
@@ -191,29 +217,44 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(sfree + 8 * s);
-      if (capped) {
+      if (series) {
 #pragma unroll
-        for (int i = 0; i < 128; ++i) v[i] = soft_cap(v[i], zs, p.softcap);
+        for (int i = 0; i < 64; i += 2) {
+          const f32x2 x = pack_f2(v[i], v[i + 1]), u = mul_f2(x, x);
+          f32x2 y = co[kTanhTerms - 1];
+#pragma unroll
+          for (int t = kTanhTerms - 2; t >= 0; --t) y = fma_f2(y, u, co[t]);
+          const float2 f = unpack_f2(mul_f2(x, y));
+          v[i] = f.x;
+          v[i + 1] = f.y;
+        }
+      } else if (capped) {
+#pragma unroll
+        for (int i = 0; i < 64; ++i) v[i] = soft_cap(v[i], zs, p.softcap);
       }
-      const int key0 = (b0 + b) * kTcKeys;
-      const int vis = pos0 + row - key0, low_v = low - key0;        // last and first visible key of this row inside the block
-      if (key0 + kTcKeys - 1 > pos0 + q4 * 32) {
+      const int key0 = (b0 + b) * kTcKeys + half * 64;
+      const int vis = pos0 + row - key0, low_v = low - key0;        // last and first visible key of this row inside the half block
+      if (key0 + 63 > pos0 + q4 * 32) {
 #pragma unroll
-        for (int i = 0; i < 128; ++i)
+        for (int i = 0; i < 64; ++i)
           if (i > vis) v[i] = -INFINITY;
       }
       if (low_last > key0) {
 #pragma unroll
-        for (int i = 0; i < 128; ++i)
+        for (int i = 0; i < 64; ++i)
           if (i < low_v) v[i] = -INFINITY;
       }
       float m4[4] = {mx, mx, mx, mx};
 #pragma unroll
-      for (int i = 0; i < 128; ++i) m4[i & 3] = fmaxf(m4[i & 3], v[i]);
+      for (int i = 0; i < 64; ++i) m4[i & 3] = fmaxf(m4[i & 3], v[i]);
       mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+      half_s[s][half][row] = mx;
+      named_bar_sync(1 + q4, 64);
+      if (abort_s[q4] != 0u) { ok = false; break; }
+      mx = fmaxf(mx, half_s[s][half ^ 1][row]);
       // P and O of the block before are consumed
       ok = __all_sync(0xffffffffu, b == 0 || mbar_wait(odone, (b - 1) & 1, p.err, kErrWaitAcc));
-      if (!ok) break;
+      if (!ok) { give_up(); break; }
       const bool grow = b == 0 || (mx - used) * sc > kTcSlack;
       if (__any_sync(0xffffffffu, grow)) {
         const float f = (grow && b > 0) ? ex2((used - mx) * sc) : 1.f;
@@ -221,7 +262,7 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
         l *= b > 0 ? f : 0.f;
         if (b > 0) {
           tc_fence_after_sync();
-          for (int c = 0; c < VP; c += 32) {
+          for (int c = half * 32; c < VP; c += 64) {                // (the halves take turns over the columns)
             uint32_t r[32];
             tmem_ld32(tm_o + lane_off + c, r);
             tmem_ld_wait();
@@ -234,16 +275,15 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
       }
       const float base = used * sc;
       float sum[4] = {};
-#pragma unroll
-      for (int c = 0; c < 2; ++c) {
+      {
         uint32_t r[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          const float a = ex2(fmaf(v[c * 64 + 2 * i], sc, -base)), e = ex2(fmaf(v[c * 64 + 2 * i + 1], sc, -base));
+          const float a = ex2(fmaf(v[2 * i], sc, -base)), e = ex2(fmaf(v[2 * i + 1], sc, -base));
           sum[i & 3] += a + e;
           r[i] = pack2(a, e);
         }
-        tmem_st32(tm_p + lane_off + c * 32, r);
+        tmem_st32(tm_p + lane_off + half * 32, r);
       }
       tmem_st_wait();
       l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
@@ -251,15 +291,23 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
       __syncwarp();
       if (lane == 0) mbar_arrive(pfull);
     }
-    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(odone, (blocks - 1) & 1, p.err, kErrWaitAcc));
+    if (ok) {
+      ok = __all_sync(0xffffffffu, mbar_wait(odone, (blocks - 1) & 1, p.err, kErrWaitAcc));
+      if (!ok) give_up();
+    }
+    if (ok) {
+      half_s[blocks & 1][half][row] = l;
+      named_bar_sync(1 + q4, 64);
+      ok = abort_s[q4] == 0u;
+    }
     if (ok) {
       tc_fence_after_sync();
       const int m = m0 + row;
       const bool live = row < rows;
-      const float inv = 1.f / l;
+      const float inv = 1.f / (half_s[blocks & 1][0][row] + half_s[blocks & 1][1][row]);
       const float* g = p.gate == nullptr ? nullptr : p.gate + static_cast<size_t>(live ? m : m0) * p.ldg + h * p.V;
       const int k0 = p.out_k0 + h * p.V;
-      for (int c = 0; c < VP; c += 32) {
+      for (int c = half * 32; c < VP; c += 64) {
         uint32_t r[32];
         __syncwarp();
         tmem_ld32(tm_o + lane_off + c, r);
@@ -302,7 +350,7 @@ static int flash_tc_smem(int DK, int VP) { return 3 * ((DK + 63) / 64) * 16384 +
 
 // VP: the accumulator shares tensor memory with two score buffers (256 columns) and the probabilities (64)
 bool saber_flash_tc_ok(int page, int DK, int VP, float scale, float softcap) {
-  return (scale > 0.f || softcap > 0.f) && page == 64 && (VP & 31) == 0 && VP <= 192 && (DK & 15) == 0 && saber::flash_tc_smem(DK, VP) <= 226 * 1024;
+  return (scale > 0.f || softcap > 0.f) && page == 64 && (VP & 31) == 0 && VP <= 192 && (DK & 15) == 0 && saber::flash_tc_smem(DK, VP) <= 224 * 1024;
 }
 
 int saber_flash_tc(const saber::FlashParams* p, cudaStream_t stream) {
@@ -312,7 +360,7 @@ int saber_flash_tc(const saber::FlashParams* p, cudaStream_t stream) {
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
   if (!ready[dev]) {
-    const cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+    const cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
     ready[dev] = true;
   }

@@ -43,6 +43,39 @@ __device__ __forceinline__ float head_scale(const GqaParams& p, const float* x, 
   return 1.f / sqrtf(mla_warp_sum(sq) / static_cast<float>(p.D) + p.eps);
 }
 
+// Four rows of a head from x on (rows past n repeat the last), divided by their root mean square; put(row, d, four values)
+// takes the pieces.  D a multiple of 4, at most 256.
+template <typename Put>
+__device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x, int n, int lane, const Put& put) {
+  float4 v[4][2];
+  float sq[4];
+#pragma unroll
+  for (int r = 0; r < 4; ++r)
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int d = u * 128 + lane * 4;
+      v[r][u] = d < p.D ? *reinterpret_cast<const float4*>(x + static_cast<size_t>(min(r, n - 1)) * p.ldx + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    sq[r] = 0.f;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) sq[r] += v[r][u].x * v[r][u].x + v[r][u].y * v[r][u].y + v[r][u].z * v[r][u].z + v[r][u].w * v[r][u].w;
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int r = 0; r < 4; ++r) sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], o);
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    if (r >= n) break;
+    const float s = p.qk_norm ? 1.f / sqrtf(sq[r] / static_cast<float>(p.D) + p.eps) : 1.f;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) put(r, u * 128 + lane * 4, make_float4(v[r][u].x * s, v[r][u].y * s, v[r][u].z * s, v[r][u].w * s));
+  }
+}
+__device__ __forceinline__ uint2 pack4(float4 v) { return make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
+
 // grid (ceil(M / 8), ceil(items / 8)), 256 threads; a warp per (head, eight rows): query heads (tcgen05 form only), then
 // key heads, then value heads.  Eight values of neighbouring tokens leave as one 16-byte piece where a page allows it.
 template <typename T>
@@ -51,13 +84,22 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
   const int lane = threadIdx.x & 31;
   int item = blockIdx.y * 8 + (threadIdx.x >> 5);
   const int m0 = blockIdx.x * 8, n = min(8, p.M - m0);
+  const bool fast = sizeof(T) == 2 && (p.D & 3) == 0 && p.D <= 256;
   if (p.form == 2) {
     if (item < p.H) {
+      __nv_bfloat16* q0 = static_cast<__nv_bfloat16*>(p.q) + (static_cast<size_t>(m0) * p.H + item) * p.DK;
+      const float* x0 = p.x + static_cast<size_t>(m0) * p.ldx + p.q_off + item * p.D;
+      if (fast) {
+        for (int r0 = 0; r0 < n; r0 += 4)
+          normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, [&](int r, int d, float4 v) {
+            if (d < p.DK) *reinterpret_cast<uint2*>(q0 + static_cast<size_t>(r0 + r) * p.H * p.DK + d) = pack4(v);      // (zeros from D on)
+          });
+        return;
+      }
       for (int r = 0; r < n; ++r) {
-        const float* x = p.x + static_cast<size_t>(m0 + r) * p.ldx + p.q_off + item * p.D;
+        const float* x = x0 + static_cast<size_t>(r) * p.ldx;
         const float s = head_scale(p, x, lane);
-        __nv_bfloat16* q = static_cast<__nv_bfloat16*>(p.q) + (static_cast<size_t>(m0 + r) * p.H + item) * p.DK;
-        for (int d = lane; d < p.DK; d += 32) q[d] = __float2bfloat16(d < p.D ? x[d] * s : 0.f);
+        for (int d = lane; d < p.DK; d += 32) q0[static_cast<size_t>(r) * p.H * p.DK + d] = __float2bfloat16(d < p.D ? x[d] * s : 0.f);
       }
       return;
     }
@@ -76,10 +118,23 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
     }
   }
   if (!isv) {
+    const float* x0 = p.x + static_cast<size_t>(m0) * p.ldx + p.k_off + g * p.D;
+    if (fast) {
+#pragma unroll
+      for (int r0 = 0; r0 < 8; r0 += 4) {
+        if (r0 >= n) break;
+        normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, [&](int r, int d, float4 v) {
+          const int s = r == 0 ? slot[r0] : r == 1 ? slot[r0 + 1] : r == 2 ? slot[r0 + 2] : slot[r0 + 3];
+          if (s >= 0 && d < p.D)
+            *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.cache) + page_block(p, s / kPage, g) + bf16_key_at(s % kPage, d)) = pack4(v);
+        });
+      }
+      return;
+    }
     for (int r = 0; r < n; ++r) {
       const int s = p.slot_map[m0 + r];
       if (s < 0 || s >= p.n_blocks * kPage) continue;
-      const float* x = p.x + static_cast<size_t>(m0 + r) * p.ldx + p.k_off + g * p.D;
+      const float* x = x0 + static_cast<size_t>(r) * p.ldx;
       const float sc = head_scale(p, x, lane);
       const size_t b = page_block(p, s / kPage, g);
       for (int d = lane; d < p.D; d += 32) Page<T>::store(p.cache, b + Page<T>::key(p, s % kPage, d), x[d] * sc);
@@ -459,6 +514,7 @@ static int gqa_go(const GqaParams& p, cudaStream_t stream) {
   f.chunk = p.chunk;
   f.scale = p.scale;
   f.softcap = p.softcap;
+  f.bound = p.qk_norm ? 1.02f * p.D : 0.f;        // (two vectors of root mean square one, and the rounding to bf16)
   f.err = p.err;
   return saber_flash_tc(&f, stream);
 }

@@ -159,26 +159,77 @@ __device__ __forceinline__ void ssd_gated_norm(const SsdParams& p, const float* 
   }
 }
 
-// grid (M + nseq, groups), 256 threads: a CTA per (row, norm group); the last nseq rows of the grid update the rings
-__global__ void __launch_bounds__(256) ssd_out_kernel(const __grid_constant__ SsdParams p) {
+// The same by a warp, for groups of up to 1024 values.
+__device__ __forceinline__ void ssd_gated_norm_warp(const SsdParams& p, const float* o, int m, int grp, int n, int lane) {
+  const int c0 = grp * n, k0 = p.out_k0 + c0;
+  const float* g = p.x + static_cast<size_t>(m) * p.ldx + p.g_off + c0;
+  float4 v[8], gate[8];
+#pragma unroll
+  for (int u = 0; u < 8; ++u) {
+    const int i = (u * 32 + lane) * 4, c = c0 + i, h = c / p.V;
+    v[u] = gate[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n) {
+      v[u] = *reinterpret_cast<const float4*>(o + h * p.VP + c - h * p.V);
+      gate[u] = *reinterpret_cast<const float4*>(g + i);
+    }
+  }
+  float sq = 0.f;
+#pragma unroll
+  for (int u = 0; u < 8; ++u) {
+    if (p.gate_first) {
+      v[u].x *= silu_f32(gate[u].x);
+      v[u].y *= silu_f32(gate[u].y);
+      v[u].z *= silu_f32(gate[u].z);
+      v[u].w *= silu_f32(gate[u].w);
+    }
+    sq += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+  }
+  const float r = 1.f / sqrtf(warp_sum_f(sq) / static_cast<float>(n) + p.eps);
+#pragma unroll
+  for (int u = 0; u < 8; ++u) {
+    const int i = (u * 32 + lane) * 4;
+    if (i >= n) break;
+    const float4 wt = *reinterpret_cast<const float4*>(p.norm_w + c0 + i);
+    float4 y = make_float4(v[u].x * r * wt.x, v[u].y * r * wt.y, v[u].z * r * wt.z, v[u].w * r * wt.w);
+    if (!p.gate_first) {
+      y.x *= sigmoid_f32(gate[u].x);
+      y.y *= sigmoid_f32(gate[u].y);
+      y.z *= sigmoid_f32(gate[u].z);
+      y.w *= sigmoid_f32(gate[u].w);
+    }
+    operand_store4(p.out, m, k0 + i, y);
+  }
+}
+
+// Items 0 .. items - 1 of the grid norm the rows: a warp per (row, group) (small = 1) or a CTA (small = 0); the last
+// nseq * kRingBlocks CTAs update the rings.  256 threads.
+constexpr int kRingBlocks = 8;
+
+__global__ void __launch_bounds__(256) ssd_out_kernel(const __grid_constant__ SsdParams p, const int items, const int small) {
   pdl_wait();
   __shared__ float red[8];
-  if (static_cast<int>(blockIdx.x) < p.M) {
-    const int m = blockIdx.x;
-    if (seq_of_row(p.cu_rows, p.nseq, m) < 0) return;
-    ssd_gated_norm(p, p.o + static_cast<size_t>(m) * p.H * p.VP, m, blockIdx.y, p.H * p.V / p.groups, red);
+  const int n = p.H * p.V / p.groups;
+  if (static_cast<int>(blockIdx.x) < items) {
+    const int item = small ? blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x;
+    const int m = item / p.groups, g = item - m * p.groups;
+    if (m >= p.M || seq_of_row(p.cu_rows, p.nseq, m) < 0) return;
+    const float* o = p.o + static_cast<size_t>(m) * p.H * p.VP;
+    if (small)
+      ssd_gated_norm_warp(p, o, m, g, n, threadIdx.x & 31);
+    else
+      ssd_gated_norm(p, o, m, g, n, red);
     return;
   }
   if (p.taps == 0) return;
-  const int j = blockIdx.x - p.M;
-  const int r0 = p.cu_rows[j], n = p.cu_rows[j + 1] - r0;
-  const int slot = n > 0 ? ssd_slot(p, j) : -1;
+  const int rb = blockIdx.x - items, j = rb / kRingBlocks;
+  const int r0 = p.cu_rows[j], rows = p.cu_rows[j + 1] - r0;
+  const int slot = rows > 0 ? ssd_slot(p, j) : -1;
   if (slot < 0) return;
   const int C = ssd_channels(p);
   float* hist = p.hist + static_cast<size_t>(slot) * p.taps * C;
-  for (int c = blockIdx.y * 256 + threadIdx.x; c < C; c += gridDim.y * 256) {
+  for (int c = (rb % kRingBlocks) * 256 + threadIdx.x; c < C; c += kRingBlocks * 256) {
     const int col = ssd_column(p, c);
-    for (int t = max(0, n - p.taps); t < n; ++t) {
+    for (int t = max(0, rows - p.taps); t < rows; ++t) {
       const int m = r0 + t;
       hist[static_cast<size_t>(p.pos[m] % p.taps) * C + c] = p.x[static_cast<size_t>(m) * p.ldx + col];
     }
@@ -189,7 +240,6 @@ __global__ void __launch_bounds__(256) ssd_out_kernel(const __grid_constant__ Ss
 // lanes along the keys and two columns each.
 template <int NI, int TAPS>
 __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ SsdParams p) {
-  pdl_wait();
   extern __shared__ float4 sm4[];
   constexpr int DP = NI * 32;
   float* ks = reinterpret_cast<float*>(sm4);       // DP
@@ -203,10 +253,6 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ S
   const int slot = ssd_slot(p, j);
   if (slot < 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 7, nt = blockDim.x, nw = nt >> 5;
-  const int pos = p.pos[m], share = p.H / p.HK, hk = h / share;
-  const int C = ssd_channels(p);
-  float* hist = p.hist + static_cast<size_t>(slot) * p.taps * C;
-  const float* x = p.x + static_cast<size_t>(m) * p.ldx;
   const size_t st0 = (static_cast<size_t>(slot) * p.H + h) * p.VP;
   const int cl = (lane >> 3) * 2;
   float4 S[2][NI];                                 // [column][32 keys]
@@ -217,7 +263,14 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ S
 #pragma unroll
       for (int i = 0; i < NI; ++i) S[c][i] = *state_at(cb, c, i);
   };
-  load(warp * 8);                                  // requested before anything else (the block has VP / 8 warps at most)
+  // the state is requested ahead of the wait: the index tables and this layer's state were complete before the step began
+  // (the block has VP / 8 warps at most)
+  load(warp * 8);
+  pdl_wait();
+  const int pos = p.pos[m], share = p.H / p.HK, hk = h / share;
+  const int C = ssd_channels(p);
+  float* hist = p.hist + static_cast<size_t>(slot) * p.taps * C;
+  const float* x = p.x + static_cast<size_t>(m) * p.ldx;
   float a, w, la;
   ssd_gates(p, m, h, a, w, la);
   const size_t now = p.taps ? static_cast<size_t>(pos % p.taps) * C : 0;
@@ -292,12 +345,14 @@ template <int NI>
 static cudaError_t ssd_step(const SsdParams& p, cudaStream_t stream) {
   const dim3 grid(p.H, p.nseq), block(32 * (p.VP / 8 < 8 ? p.VP / 8 : 8));
   const int smem = (2 * NI * 32 + p.VP) * 4;
-  return p.taps == 4 ? launch(ssd_step_kernel<NI, 4>, grid, block, smem, stream, 2, p) : launch(ssd_step_kernel<NI, 0>, grid, block, smem, stream, 2, p);
+  return p.taps == 4   ? launch(ssd_step_kernel<NI, 4>, grid, block, smem, stream, 2, p)
+         : p.taps == 0 ? launch(ssd_step_kernel<NI, -1>, grid, block, smem, stream, 2, p)
+                       : launch(ssd_step_kernel<NI, 0>, grid, block, smem, stream, 2, p);
 }
 template <int NI>
 static cudaError_t ssd_prep(const SsdParams& p, cudaStream_t stream) {
   const dim3 grid(p.M / kBlk + p.nseq, (p.HK + p.H + 3) / 4);
-  return p.taps == 4 ? launch(ssd_prep_kernel<NI, 4>, grid, dim3(128), 0, stream, 0, p)
+  return p.taps == 0 ? launch(ssd_prep_kernel<NI, -1>, grid, dim3(128), 0, stream, 0, p)
                      : launch(ssd_prep_kernel<NI, 0>, grid, dim3(128), 0, stream, 0, p);
 }
 
@@ -352,5 +407,7 @@ extern "C" int saber_ssd_launch(const saber::SsdParams* p, int single_row, cudaS
     }
   }
   if (e != 0 || single_row) return e;
-  return static_cast<int>(launch(ssd_out_kernel, dim3(p->M + p->nseq, p->groups), dim3(256), 0, stream, 0, *p));
+  const int n = p->H * p->V / p->groups, small = n <= 1024 && ((p->V | n) & 3) == 0 ? 1 : 0;
+  const int items = small ? (p->M * p->groups + 7) / 8 : p->M * p->groups;
+  return static_cast<int>(launch(ssd_out_kernel, dim3(items + p->nseq * kRingBlocks), dim3(256), 0, stream, 0, *p, items, small));
 }

@@ -10,9 +10,10 @@
 // fp32 factors meet bf16 ones in `mma.sync`: they are written as a sum of three bf16 values (24 bits, the fp32
 // mantissa), three products with fp32 accumulation.  Those are the pair weights P_ij, the state, and B_j w_j v_j.
 //
-//   prep   convolution, silu -> q, k, v tiles in the order the scan's fragments want them; log decays and weights
-//   scan   a CTA per (sequence, head, 64 value columns), 16 columns a warp; the accumulator fragments of the state are
-//          the operand fragments of the next read-out.  Tiles of the next chunk arrive by bulk copies meanwhile.
+//   prep   convolution, silu -> q, k, v tiles in the order the scan's fragments want them; the tables of decays
+//   scan   a CTA per (sequence, head, 64 value columns); a pair of warps holds 16 columns of the state, half of the keys
+//          each, as accumulator fragments that are the operand fragments of the next read-out (the halves of a read-out
+//          meet in shared memory).  Tiles of the next chunk arrive by bulk copies meanwhile.
 #include "launch.cuh"
 #include "mla_device.cuh"
 #include "ssd_chunk.h"
@@ -29,6 +30,16 @@ __device__ __forceinline__ int chunk_slot(int r0, int j) { return r0 / kTok + j;
 // element of a tile of 64 rows: [64-column block][row][128 bytes], 16-byte pieces XOR (row & 7)
 __device__ __forceinline__ int tile_at(int row, int c) { return ((c >> 6) * kTok + row) * 64 + (((((c & 63) >> 3) ^ row) & 7) << 3) + (c & 7); }
 
+// Decays of a chunk, weights included (a bulk copy).
+struct ChunkTables {
+  float diag[4][16][20];                 // [sixteen][i][j] D_ij w_j of two tokens of the same sixteen, 0 above the diagonal
+  float row[kTok];                       // from the start of a token's sixteen to it
+  float start[kTok];                     // A_i
+  float col[3][kTok];                    // from token j of an earlier sixteen to the start of sixteen a + 1, times w_j
+  float end[kTok];                       // B_j w_j
+};
+static_assert(sizeof(ChunkTables) % 16 == 0, "");
+
 struct ChunkLayout {                     // of a slot, in bytes
   size_t v, gates, bytes;
 };
@@ -37,7 +48,7 @@ __host__ __device__ inline ChunkLayout chunk_layout(const SsdParams& p) {
   ChunkLayout l;
   l.v = static_cast<size_t>(p.HK) * 2 * p.DP * kTok * 2;            // [HK][q | k][DP / 64] tiles
   l.gates = l.v + static_cast<size_t>(p.H) * vs * kTok * kSlice * 2;    // [H][slices] tiles
-  l.bytes = l.gates + static_cast<size_t>(p.H) * 2 * kTok * 4;          // [H][log decay 64 | weight 64]
+  l.bytes = l.gates + static_cast<size_t>(p.H) * sizeof(ChunkTables);   // [H]
   return l;
 }
 
@@ -61,13 +72,39 @@ __global__ void __launch_bounds__(128) ssd_chunk_prep_kernel(const __grid_consta
   const int vs = (p.VP + kSlice - 1) / kSlice, nk = p.HK * p.DP, total = 2 * nk + p.H * vs * kSlice;
   const int groups = (total + 127) / 128;
   if (static_cast<int>(blockIdx.y) >= groups) {
-    const int h = (blockIdx.y - groups) * 8 + blockIdx.z * 2 + threadIdx.x / kTok, r = threadIdx.x % kTok;
-    if (h >= p.H) return;
-    float a, w = 0.f, la = 0.f;
-    if (r < live) ssd_gates(p, m0 + r, h, a, w, la);
-    float* g = reinterpret_cast<float*>(base + lay.gates) + h * 2 * kTok;
-    g[r] = la;
-    g[kTok + r] = w;
+    __shared__ float la_s[2][kTok], total_s[2][4];
+    const int hh = threadIdx.x / kTok, h = (blockIdx.y - groups) * 8 + blockIdx.z * 2 + hh, r = threadIdx.x % kTok;
+    float w = 0.f, la = 0.f, decay;
+    if (h < p.H && r < live) ssd_gates(p, m0 + r, h, decay, w, la);
+    la_s[hh][r] = la;
+    __syncthreads();
+    ChunkTables* tb = reinterpret_cast<ChunkTables*>(base + lay.gates) + min(h, p.H - 1);
+    const bool mine = h < p.H;
+    const int a = r >> 4, l = r & 15;
+    const float* q = la_s[hh] + a * 16;
+    float d = 0.f, g = 0.f;
+    for (int i = 0; i < l; ++i)
+      if (mine) tb->diag[a][i][l] = 0.f;
+    if (mine) tb->diag[a][l][l] = w;
+    for (int i = l + 1; i < 16; ++i) {
+      d += q[i];
+      if (mine) tb->diag[a][i][l] = expf(d) * w;
+    }
+    for (int i = 0; i <= l; ++i) g += q[i];
+    if (mine) tb->row[r] = expf(g);
+    if (l == 15) total_s[hh][a] = g;
+    __syncthreads();
+    if (!mine) return;
+    const float* tot = total_s[hh];
+    float before = 0.f;
+    for (int x = 0; x < a; ++x) before += tot[x];
+    tb->start[r] = expf(g + before);
+    for (int x = a + 1; x < 4; ++x) {
+      if (x > a + 1) d += tot[x - 1];
+      tb->col[x - 1][r] = expf(d) * w;
+    }
+    if (a < 3) d += tot[3];
+    tb->end[r] = expf(d) * w;
     return;
   }
   const int i = blockIdx.y * 128 + threadIdx.x;
@@ -108,23 +145,12 @@ __device__ __forceinline__ void split3(float a, float b, uint32_t (&s)[3]) {
   s[2] = pack2(a, b);
 }
 
-struct ScanTables {                      // decays of the chunk at hand (shared memory)
-  float diag[4][16][17];                 // D_ij w_j of the sixteen tokens i and j share, plus skip for i = j
-  float row[kTok];                       // from the start of a token's sixteen to it
-  float start[kTok];                     // A_i
-  float pre[kTok];                       // suffix sums: logarithms after a token inside its sixteen
-  float col[4][kTok];                    // from token j (an earlier sixteen) to the start of sixteen a, times w_j
-  float end[kTok];                       // B_j w_j
-  float total[4];                        // sums of logarithms of the sixteens
-};
-
-// grid (nseq, H, ceil(VP / 64)), 128 threads.  NJ: 64-wide blocks of the key size.
+// grid (nseq, H, ceil(VP / 64)), 256 threads.  NJ: 64-wide blocks of the key size.
 template <int NJ>
-__global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(const __grid_constant__ SsdParams p) {
-  constexpr int DP = NJ * 64, kKS = DP / 16, kQK = DP * kTok * 2;          // bytes of a q or k tile
-  constexpr uint32_t kStage = 2 * kQK + kTok * kSlice * 2 + 2 * kTok * 4;
+__global__ void __launch_bounds__(256, 1) ssd_chunk_scan_kernel(const __grid_constant__ SsdParams p) {
+  constexpr int DP = NJ * 64, kKS = DP / 32, kQK = DP * kTok * 2;          // 16-wide key steps of a warp; bytes of a q or k tile
+  constexpr uint32_t kV = kTok * kSlice * 2, kStage = 2 * kQK + kV + sizeof(ChunkTables);
   extern __shared__ uint8_t smem_raw[];
-  __shared__ ScanTables tb;
   __shared__ uint64_t bars[2];
   pdl_wait();
   const int j = blockIdx.x, h = blockIdx.y;
@@ -132,10 +158,11 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
   if (n <= 0) return;
   const int slot = ssd_slot(p, j);
   if (slot < 0) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wv = warp & 3, hn = warp >> 2;
   const int chunks = (n + kTok - 1) / kTok;
   const uint32_t st0 = (smem_u32(smem_raw) + 1023u) & ~1023u, p_s = st0 + 2 * kStage;      // P: three tiles of 8 KiB
-  const uint8_t* gen = smem_raw + (st0 - smem_u32(smem_raw));
+  uint8_t* const gen = smem_raw + (st0 - smem_u32(smem_raw));
+  float4* red = reinterpret_cast<float4*>(gen + 2 * kStage + 3 * 8192) + wv * 256 + lane;     // [16 columns][tokens, columns][lane]
   const uint32_t bar = smem_u32(bars);
   const ChunkLayout lay = chunk_layout(p);
   const int vslices = (p.VP + kSlice - 1) / kSlice, hk = h / (p.H / p.HK);
@@ -145,8 +172,8 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
     const uint8_t* s = src + c * lay.bytes;
     mbar_arrive_expect_tx(b, kStage);
     bulk_g2s(dst, s + static_cast<size_t>(hk) * 2 * kQK, 2 * kQK, b);
-    bulk_g2s(dst + 2 * kQK, s + lay.v + (static_cast<size_t>(h) * vslices + blockIdx.z) * kTok * kSlice * 2, kTok * kSlice * 2, b);
-    bulk_g2s(dst + 2 * kQK + kTok * kSlice * 2, s + lay.gates + static_cast<size_t>(h) * 2 * kTok * 4, 2 * kTok * 4, b);
+    bulk_g2s(dst + 2 * kQK, s + lay.v + (static_cast<size_t>(h) * vslices + blockIdx.z) * kV, kV, b);
+    bulk_g2s(dst + 2 * kQK + kV, s + lay.gates + static_cast<size_t>(h) * sizeof(ChunkTables), sizeof(ChunkTables), b);
   };
   int issued = 0;
   if (threadIdx.x == 0) {
@@ -157,13 +184,13 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
   }
   __syncthreads();
   const float skip = p.skip ? p.skip[h] : 0.f;
-  // this warp's value columns and the state fragments: S[8 keys][column lane / 4 | + 8, keys (lane % 4) 2 + {0, 1}]
-  const int v0 = blockIdx.z * kSlice + warp * 16, q2 = (lane & 3) * 2, l4 = lane >> 2;
+  // this warp's value columns and state fragments: S[8 keys][column lane / 4 | + 8, keys (lane % 4) 2 + {0, 1}]
+  const int v0 = blockIdx.z * kSlice + wv * 16, q2 = (lane & 3) * 2, l4 = lane >> 2;
   const bool on = v0 < p.VP;
-  float S[DP / 8][4];
-  float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + v0) * DP;
+  float S[2 * kKS][4];
+  float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + v0) * DP + hn * (DP / 2);
 #pragma unroll
-  for (int t = 0; t < DP / 8; ++t)
+  for (int t = 0; t < 2 * kKS; ++t)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int v = l4 + half * 8;
@@ -175,115 +202,74 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
   int c = 0;
   for (; c < chunks; ++c) {
     const uint32_t qt = st0 + (c & 1) * kStage, kt = qt + kQK, vt = kt + kQK;
-    const float* la = reinterpret_cast<const float*>(gen + (c & 1) * kStage + 2 * kQK + kTok * kSlice * 2);
-    const float* w = la + kTok;
+    const ChunkTables& tb = *reinterpret_cast<const ChunkTables*>(gen + (c & 1) * kStage + 2 * kQK + kV);
     ok = __syncthreads_and(mbar_wait(bar + 8 * (c & 1), (c >> 1) & 1, p.err, kErrWaitFull)) != 0;
     if (!ok) break;
-    // ---- decays
-    if (threadIdx.x < kTok) {
-      const int a = threadIdx.x >> 4, jj = threadIdx.x & 15;
-      const float wj = w[threadIdx.x];
-      float d = 0.f;
-      for (int i = 0; i < jj; ++i) tb.diag[a][i][jj] = 0.f;
-      tb.diag[a][jj][jj] = wj;
-      for (int i = jj + 1; i < 16; ++i) {
-        d += la[a * 16 + i];
-        tb.diag[a][i][jj] = expf(d) * wj;
+    // ---- pair weights: the ten 16 x 16 tiles on and below the diagonal, dealt to the warps
+    for (int tile = warp; tile < 10; tile += 8) {
+      const int mi = tile >= 6 ? 3 : tile >= 3 ? 2 : tile >= 1 ? 1 : 0, nt = tile - mi * (mi + 1) / 2;
+      const int ar = mi * 16 + (lane & 15), br = nt * 16 + ((lane >> 4) << 3) + (lane & 7);
+      float s[2][2][4] = {};                       // [even | odd steps]: two chains
+#pragma unroll
+      for (int ks = 0; ks < 2 * kKS; ++ks) {
+        uint32_t a[4], b[4];
+        const int ac = ks * 2 + (lane >> 4), bc = ks * 2 + ((lane >> 3) & 1);
+        ldsm4(a, qt + (ac >> 3) * 8192 + ar * 128 + (((ac ^ ar) & 7) << 4));
+        ldsm4(b, kt + (bc >> 3) * 8192 + br * 128 + (((bc ^ br) & 7) << 4));
+        mma16816(s[ks & 1][0], a, b[0], b[1]);
+        mma16816(s[ks & 1][1], a, b[2], b[3]);
       }
-      tb.pre[threadIdx.x] = d;                     // everything after j inside its sixteen
-    } else {
-      const int i = threadIdx.x - kTok, a = i >> 4;
-      float g = 0.f;
-      for (int t = a * 16; t <= i; ++t) g += la[t];
-      tb.row[i] = expf(g);
-      tb.start[i] = g;
-      if ((i & 15) == 15) tb.total[a] = g;
-    }
-    __syncthreads();
-    if (threadIdx.x < kTok) {
-      const int b = threadIdx.x >> 4;
-      const float wj = w[threadIdx.x];
-      float r = tb.pre[threadIdx.x];
 #pragma unroll
-      for (int a = 1; a < 4; ++a)
-        if (a > b) {
-          if (a > b + 1) r += tb.total[a - 1];
-          tb.col[a][threadIdx.x] = expf(r) * wj;
-        }
-      if (b < 3) r += tb.total[3];
-      tb.end[threadIdx.x] = expf(r) * wj;
-    } else {
-      const int i = threadIdx.x - kTok;
-      float g = 0.f;
-      for (int a = 0; a < (i >> 4); ++a) g += tb.total[a];
-      tb.start[i] = expf(tb.start[i] + g);
-    }
-    __syncthreads();
-    // ---- pair weights of this warp's sixteen tokens
-    {
-      const int ar = warp * 16 + (lane & 15);
-      for (int nt = 0; nt <= warp; ++nt) {
-        float s[2][4] = {};
-        const int br = nt * 16 + ((lane >> 4) << 3) + (lane & 7);
+      for (int half = 0; half < 2; ++half) {
+        const int il = l4 + half * 8, i = mi * 16 + il;
+        const float ri = tb.row[i];
 #pragma unroll
-        for (int ks = 0; ks < kKS; ++ks) {
-          uint32_t a[4], b[4];
-          const int ac = ks * 2 + (lane >> 4), bc = ks * 2 + ((lane >> 3) & 1);
-          ldsm4(a, qt + (ac >> 3) * 8192 + ar * 128 + (((ac ^ ar) & 7) << 4));
-          ldsm4(b, kt + (bc >> 3) * 8192 + br * 128 + (((bc ^ br) & 7) << 4));
-          mma16816(s[0], a, b[0], b[1]);
-          mma16816(s[1], a, b[2], b[3]);
-        }
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int il = l4 + half * 8, i = warp * 16 + il;
-          const float ri = tb.row[i];
-#pragma unroll
-          for (int t = 0; t < 2; ++t) {
-            const int jl = t * 8 + q2, jc = nt * 16 + jl;
-            float f0, f1;
-            if (nt == warp) {
-              f0 = tb.diag[warp][il][jl];
-              f1 = tb.diag[warp][il][jl + 1];
-            } else {
-              f0 = ri * tb.col[warp][jc];
-              f1 = ri * tb.col[warp][jc + 1];
-            }
-            float x = s[t][half * 2] * f0, y = s[t][half * 2 + 1] * f1;
-            if (nt == warp) {
-              if (il == jl) x += skip;
-              if (il == jl + 1) y += skip;
-            }
-            uint32_t sp[3];
-            split3(x, y, sp);
-#pragma unroll
-            for (int e = 0; e < 3; ++e)
-              asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_s + e * 8192 + i * 128 + ((((jc >> 3) ^ i) & 7) << 4) + q2 * 2), "r"(sp[e]) : "memory");
+        for (int t = 0; t < 2; ++t) {
+          const int jl = t * 8 + q2, jc = nt * 16 + jl;
+          float2 f;
+          if (nt == mi) {
+            f = *reinterpret_cast<const float2*>(&tb.diag[mi][il][jl]);
+          } else {
+            f = *reinterpret_cast<const float2*>(&tb.col[mi - 1][jc]);
+            f.x *= ri;
+            f.y *= ri;
           }
+          float x = (s[0][t][half * 2] + s[1][t][half * 2]) * f.x, y = (s[0][t][half * 2 + 1] + s[1][t][half * 2 + 1]) * f.y;
+          if (nt == mi) {
+            if (il == jl) x += skip;
+            if (il == jl + 1) y += skip;
+          }
+          uint32_t sp[3];
+          split3(x, y, sp);
+#pragma unroll
+          for (int e = 0; e < 3; ++e)
+            asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_s + e * 8192 + i * 128 + ((((jc >> 3) ^ i) & 7) << 4) + q2 * 2), "r"(sp[e]) : "memory");
         }
       }
     }
-    // ---- read-out of the state at the chunk's start
+    // ---- read-out of the state at the chunk's start, this warp's half of the keys
     float o[4][2][4] = {};
     if (on) {
 #pragma unroll
       for (int ks = 0; ks < kKS; ++ks) {
-        uint32_t b[2][2][3];                       // [8 columns][k half][part]
+        uint32_t b[2][2][3];                       // [8 columns][8 keys][part]
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
           split3(S[2 * ks][2 * t], S[2 * ks][2 * t + 1], b[t][0]);
           split3(S[2 * ks + 1][2 * t], S[2 * ks + 1][2 * t + 1], b[t][1]);
         }
+        uint32_t a[4][4];
 #pragma unroll
         for (int mt = 0; mt < 4; ++mt) {
-          uint32_t a[4];
-          const int ar = mt * 16 + (lane & 15), ac = ks * 2 + (lane >> 4);
-          ldsm4(a, qt + (ac >> 3) * 8192 + ar * 128 + (((ac ^ ar) & 7) << 4));
-#pragma unroll
-          for (int e = 2; e >= 0; --e)
-#pragma unroll
-            for (int t = 0; t < 2; ++t) mma16816(o[mt][t], a, b[t][0][e], b[t][1][e]);
+          const int ar = mt * 16 + (lane & 15), ac = (hn * kKS + ks) * 2 + (lane >> 4);
+          ldsm4(a[mt], qt + (ac >> 3) * 8192 + ar * 128 + (((ac ^ ar) & 7) << 4));
         }
+#pragma unroll
+        for (int e = 2; e >= 0; --e)
+#pragma unroll
+          for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+            for (int t = 0; t < 2; ++t) mma16816(o[mt][t], a[mt], b[t][0][e], b[t][1][e]);
       }
 #pragma unroll
       for (int mt = 0; mt < 4; ++mt) {
@@ -294,14 +280,16 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
     }
     __syncthreads();                               // every warp's pair weights are in place
     if (on) {
-      // ---- products inside the chunk
+      // ---- products inside the chunk: sixteens 0 and 3 of the keys by one half, 1 and 2 by the other
 #pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
+      for (int u = 0; u < 2; ++u) {
+        const int ks = u == 0 ? hn : 3 - hn;
         uint32_t b[4];
-        const int br = ks * 16 + (lane & 15), bc = warp * 2 + (lane >> 4);
+        const int br = ks * 16 + (lane & 15), bc = wv * 2 + (lane >> 4);
         ldsm4_t(b, vt + br * 128 + (((bc ^ br) & 7) << 4));
 #pragma unroll
-        for (int mt = ks; mt < 4; ++mt) {
+        for (int mt = 0; mt < 4; ++mt) {
+          if (mt < ks) continue;                   // (uniform)
           const int ar = mt * 16 + (lane & 15), ac = ks * 2 + (lane >> 4);
 #pragma unroll
           for (int e = 2; e >= 0; --e) {
@@ -312,22 +300,28 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
           }
         }
       }
+      if (hn == 1) {
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+          for (int t = 0; t < 2; ++t) red[(mt * 2 + t) * 32] = make_float4(o[mt][t][0], o[mt][t][1], o[mt][t][2], o[mt][t][3]);
+      }
       // ---- state at the chunk's end
       const float at = tb.start[kTok - 1];
 #pragma unroll
-      for (int t = 0; t < DP / 8; ++t) { S[t][0] *= at; S[t][1] *= at; S[t][2] *= at; S[t][3] *= at; }
+      for (int t = 0; t < 2 * kKS; ++t) { S[t][0] *= at; S[t][1] *= at; S[t][2] *= at; S[t][3] *= at; }
 #pragma unroll
       for (int ks = 0; ks < 4; ++ks) {
         uint32_t vr[4], a[3][4];
         {
-          const int r = ks * 16 + (lane & 7) + ((lane >> 4) << 3), vc = warp * 2 + ((lane >> 3) & 1);
+          const int r = ks * 16 + (lane & 7) + ((lane >> 4) << 3), vc = wv * 2 + ((lane >> 3) & 1);
           ldsm4_t(vr, vt + r * 128 + (((vc ^ r) & 7) << 4));
         }
-        const float e0 = tb.end[ks * 16 + q2], e1 = tb.end[ks * 16 + q2 + 1], e8 = tb.end[ks * 16 + q2 + 8], e9 = tb.end[ks * 16 + q2 + 9];
+        const float2 e0 = *reinterpret_cast<const float2*>(&tb.end[ks * 16 + q2]), e8 = *reinterpret_cast<const float2*>(&tb.end[ks * 16 + q2 + 8]);
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
           uint32_t sp[3];
-          split3(__uint_as_float(vr[x] << 16) * (x < 2 ? e0 : e8), __uint_as_float(vr[x] & 0xffff0000u) * (x < 2 ? e1 : e9), sp);
+          split3(__uint_as_float(vr[x] << 16) * (x < 2 ? e0.x : e8.x), __uint_as_float(vr[x] & 0xffff0000u) * (x < 2 ? e0.y : e8.y), sp);
           a[0][x] = sp[0];
           a[1][x] = sp[1];
           a[2][x] = sp[2];
@@ -335,7 +329,7 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
 #pragma unroll
         for (int nt = 0; nt < kKS; ++nt) {
           uint32_t b[4];
-          const int r = ks * 16 + (lane & 15), kc = nt * 2 + (lane >> 4);
+          const int r = ks * 16 + (lane & 15), kc = (hn * kKS + nt) * 2 + (lane >> 4);
           ldsm4_t(b, kt + (kc >> 3) * 8192 + r * 128 + (((kc ^ r) & 7) << 4));
 #pragma unroll
           for (int e = 2; e >= 0; --e) {
@@ -345,21 +339,22 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
         }
       }
     }
-    __syncthreads();                               // the stage, the pair weights and the tables are free
+    __syncthreads();                               // the stage and the pair weights are free, the second halves in place
     if (threadIdx.x == 0 && c + 2 < chunks) { fetch(c + 2); ++issued; }
-    if (on) {
+    if (on && hn == 0) {
       const int live = n - c * kTok;
       float* out = p.o + (static_cast<size_t>(r0 + c * kTok) * p.H + h) * p.VP + v0;
 #pragma unroll
       for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int i = mt * 16 + l4 + half * 8;
-          if (i >= live) continue;
-#pragma unroll
-          for (int t = 0; t < 2; ++t)
-            if (v0 + t * 8 < p.VP)
-              *reinterpret_cast<float2*>(out + static_cast<size_t>(i) * p.H * p.VP + t * 8 + q2) = make_float2(o[mt][t][half * 2], o[mt][t][half * 2 + 1]);
+        for (int t = 0; t < 2; ++t) {
+          const float4 x = red[(mt * 2 + t) * 32];
+          if (v0 + t * 8 >= p.VP) continue;
+          const int i = mt * 16 + l4;
+          float* d = out + static_cast<size_t>(i) * p.H * p.VP + t * 8 + q2;
+          if (i < live) *reinterpret_cast<float2*>(d) = make_float2(o[mt][t][0] + x.x, o[mt][t][1] + x.y);
+          if (i + 8 < live)
+            *reinterpret_cast<float2*>(d + static_cast<size_t>(8) * p.H * p.VP) = make_float2(o[mt][t][2] + x.z, o[mt][t][3] + x.w);
         }
     }
   }
@@ -367,7 +362,7 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
     for (int i = c; i < issued; ++i) mbar_wait(bar + 8 * (i & 1), (i >> 1) & 1, p.err, kErrWaitDrain);
   if (!ok) return;
 #pragma unroll
-  for (int t = 0; t < DP / 8; ++t)
+  for (int t = 0; t < 2 * kKS; ++t)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int v = l4 + half * 8;
@@ -377,7 +372,7 @@ __global__ void __launch_bounds__(128, NJ <= 2 ? 2 : 1) ssd_chunk_scan_kernel(co
 
 template <int NJ>
 static int chunk_go(const SsdParams& p, cudaStream_t stream) {
-  constexpr int smem = 2 * (2 * NJ * 64 * kTok * 2 + kTok * kSlice * 2 + 2 * kTok * 4) + 3 * 8192 + 1024;
+  constexpr int smem = 2 * (2 * NJ * 64 * kTok * 2 + kTok * kSlice * 2 + static_cast<int>(sizeof(ChunkTables))) + 3 * 8192 + 4 * 4096 + 1024;
   static bool ready[64];
   int dev = 0;
   cudaGetDevice(&dev);
@@ -389,10 +384,11 @@ static int chunk_go(const SsdParams& p, cudaStream_t stream) {
   }
   const int vs = (p.VP + kSlice - 1) / kSlice, channels = 2 * p.HK * p.DP + p.H * vs * kSlice;
   const dim3 grid(p.M / kTok + p.nseq, (channels + 127) / 128 + (p.H + 7) / 8, kTok / kRun);
-  const cudaError_t e = p.taps == 4 ? launch(ssd_chunk_prep_kernel<4>, grid, dim3(128), 0, stream, 0, p)
-                                    : launch(ssd_chunk_prep_kernel<0>, grid, dim3(128), 0, stream, 0, p);
+  const cudaError_t e = p.taps == 4   ? launch(ssd_chunk_prep_kernel<4>, grid, dim3(128), 0, stream, 0, p)
+                        : p.taps == 0 ? launch(ssd_chunk_prep_kernel<-1>, grid, dim3(128), 0, stream, 0, p)
+                                      : launch(ssd_chunk_prep_kernel<0>, grid, dim3(128), 0, stream, 0, p);
   if (e != cudaSuccess) return static_cast<int>(e);
-  return static_cast<int>(launch(ssd_chunk_scan_kernel<NJ>, dim3(p.nseq, p.H, vs), dim3(128), smem, stream, 0, p));
+  return static_cast<int>(launch(ssd_chunk_scan_kernel<NJ>, dim3(p.nseq, p.H, vs), dim3(256), smem, stream, 0, p));
 }
 
 }  // namespace saber

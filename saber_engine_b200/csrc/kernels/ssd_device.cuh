@@ -33,13 +33,15 @@ __device__ __forceinline__ void ssd_gates(const SsdParams& p, int m, int h, floa
   a = expf(log_a);
 }
 // silu of channel c's input at the ROWS rows from m on (m is row t of its sequence, at position pos); rows past
-// `rows` give 0.  TAPS > 0: the number of taps when known at compile time.
+// `rows` (>= 1) give 0.  TAPS > 0: the number of taps when known at compile time; -1: no convolution; 0: p.taps of them.
 template <int ROWS, int TAPS>
 __device__ __forceinline__ void ssd_inputs(const SsdParams& p, const float* hist, int c, int m, int t, int pos, int C, int rows, float (&y)[ROWS]) {
   const int col = ssd_column(p, c);
-  if (p.taps == 0) {
+  if constexpr (TAPS < 0) {
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) y[r] = r < rows ? silu_f32(p.x[static_cast<size_t>(m + r) * p.ldx + col]) : 0.f;
+    for (int r = 0; r < ROWS; ++r) y[r] = p.x[static_cast<size_t>(m + min(r, rows - 1)) * p.ldx + col];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) y[r] = r < rows ? silu_f32(y[r]) : 0.f;
     return;
   }
   float acc[ROWS];

@@ -11,8 +11,9 @@ __device__ __forceinline__ float warp_sum_f(float v) {
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
   return v;
 }
-__device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
+// (approximate division: two units in the last place; a denominator above 2^126 gives 0)
+__device__ __forceinline__ float silu_f32(float x) { return __fdividef(x, 1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f32(float x) { return __fdividef(1.f, 1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f32(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
 
 // sequence of a row (-1: a padding row)

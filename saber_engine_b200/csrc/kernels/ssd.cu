@@ -97,55 +97,63 @@ __device__ __forceinline__ float block_sum(float v, float* red, int nw) {
   return v;
 }
 
-// Gate and norm of one group of a row (o: the row's read-outs [H][VP], n values of the group).
+struct Silu { __device__ __forceinline__ float operator()(float x) const { return silu_f32(x); } };
+struct Sigmoid { __device__ __forceinline__ float operator()(float x) const { return sigmoid_f32(x); } };
+// v times f(g) where it applies
+template <typename Fn>
+__device__ __forceinline__ float4 gate4(bool on, float4 v, float4 g, Fn f) {
+  if (!on) return v;
+  return make_float4(v.x * f(g.x), v.y * f(g.y), v.z * f(g.z), v.w * f(g.w));
+}
+__device__ __forceinline__ float square4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// Gate and norm of one group of a row (o: the row's read-outs [H][VP], n values of the group) by a block.
 __device__ __forceinline__ void ssd_gated_norm(const SsdParams& p, const float* o, int m, int grp, int n, float* red) {
   const int nt = blockDim.x, c0 = grp * n, k0 = p.out_k0 + c0;
   const float* g = p.x + static_cast<size_t>(m) * p.ldx + p.g_off + c0;
   const float* w = p.norm_w + c0;
-  constexpr int kHeld = 4;                         // values held per thread, in groups of four
-  if (((p.V | n) & 3) == 0 && n <= 4 * kHeld * nt) {
+  const bool first = p.gate_first != 0;
+  if (((p.V | n) & 3) == 0) {                      // sixteen values a thread at a time, held where that is all
+    constexpr int kHeld = 4;
     float4 v[kHeld], gate[kHeld];
+    auto load = [&](int base) {
 #pragma unroll
-    for (int u = 0; u < kHeld; ++u) {
-      const int i = (u * nt + threadIdx.x) * 4, c = c0 + i, h = c / p.V;
-      v[u] = gate[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (i < n) {
-        v[u] = __ldcg(reinterpret_cast<const float4*>(o + h * p.VP + c - h * p.V));
-        gate[u] = *reinterpret_cast<const float4*>(g + i);
+      for (int u = 0; u < kHeld; ++u) {
+        const int i = base + (u * nt + threadIdx.x) * 4, c = c0 + i, h = c / p.V;
+        v[u] = gate[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n) {
+          v[u] = __ldcg(reinterpret_cast<const float4*>(o + h * p.VP + c - h * p.V));
+          gate[u] = *reinterpret_cast<const float4*>(g + i);
+        }
       }
-    }
+#pragma unroll
+      for (int u = 0; u < kHeld; ++u) v[u] = gate4(first, v[u], gate[u], Silu{});
+    };
+    const int span = 4 * kHeld * nt;
     float sq = 0.f;
+    for (int base = 0; base < n; base += span) {
+      load(base);
 #pragma unroll
-    for (int u = 0; u < kHeld; ++u) {
-      if (p.gate_first) {
-        v[u].x *= silu_f32(gate[u].x);
-        v[u].y *= silu_f32(gate[u].y);
-        v[u].z *= silu_f32(gate[u].z);
-        v[u].w *= silu_f32(gate[u].w);
-      }
-      sq += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+      for (int u = 0; u < kHeld; ++u) sq += square4(v[u]);
     }
     const float r = 1.f / sqrtf(block_sum(sq, red, nt >> 5) / static_cast<float>(n) + p.eps);
+    for (int base = 0; base < n; base += span) {
+      if (n > span) load(base);
 #pragma unroll
-    for (int u = 0; u < kHeld; ++u) {
-      const int i = (u * nt + threadIdx.x) * 4;
-      if (i >= n) break;
-      const float4 wt = *reinterpret_cast<const float4*>(w + i);
-      float4 y = make_float4(v[u].x * r * wt.x, v[u].y * r * wt.y, v[u].z * r * wt.z, v[u].w * r * wt.w);
-      if (!p.gate_first) {
-        y.x *= sigmoid_f32(gate[u].x);
-        y.y *= sigmoid_f32(gate[u].y);
-        y.z *= sigmoid_f32(gate[u].z);
-        y.w *= sigmoid_f32(gate[u].w);
+      for (int u = 0; u < kHeld; ++u) {
+        const int i = base + (u * nt + threadIdx.x) * 4;
+        if (i >= n) break;
+        const float4 wt = *reinterpret_cast<const float4*>(w + i);
+        operand_store4(p.out, m, k0 + i,
+                       gate4(!first, make_float4(v[u].x * r * wt.x, v[u].y * r * wt.y, v[u].z * r * wt.z, v[u].w * r * wt.w), gate[u], Sigmoid{}));
       }
-      operand_store4(p.out, m, k0 + i, y);
     }
     return;
   }
   auto gated = [&](int i) {
     const int c = c0 + i, h = c / p.V;
     const float v = __ldcg(o + h * p.VP + c - h * p.V);
-    return p.gate_first ? v * silu_f32(g[i]) : v;
+    return first ? v * silu_f32(g[i]) : v;
   };
   float sq = 0.f;
   for (int i = threadIdx.x; i < n; i += nt) {
@@ -155,7 +163,7 @@ __device__ __forceinline__ void ssd_gated_norm(const SsdParams& p, const float* 
   const float r = 1.f / sqrtf(block_sum(sq, red, nt >> 5) / static_cast<float>(n) + p.eps);
   for (int i = threadIdx.x; i < n; i += nt) {
     const float y = gated(i) * r * w[i];
-    operand_store1(p.out, m, k0 + i, p.gate_first ? y : y * sigmoid_f32(g[i]));
+    operand_store1(p.out, m, k0 + i, first ? y : y * sigmoid_f32(g[i]));
   }
 }
 
@@ -173,16 +181,12 @@ __device__ __forceinline__ void ssd_gated_norm_warp(const SsdParams& p, const fl
       gate[u] = *reinterpret_cast<const float4*>(g + i);
     }
   }
+  const bool first = p.gate_first != 0;
   float sq = 0.f;
 #pragma unroll
   for (int u = 0; u < 8; ++u) {
-    if (p.gate_first) {
-      v[u].x *= silu_f32(gate[u].x);
-      v[u].y *= silu_f32(gate[u].y);
-      v[u].z *= silu_f32(gate[u].z);
-      v[u].w *= silu_f32(gate[u].w);
-    }
-    sq += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+    v[u] = gate4(first, v[u], gate[u], Silu{});
+    sq += square4(v[u]);
   }
   const float r = 1.f / sqrtf(warp_sum_f(sq) / static_cast<float>(n) + p.eps);
 #pragma unroll
@@ -190,14 +194,8 @@ __device__ __forceinline__ void ssd_gated_norm_warp(const SsdParams& p, const fl
     const int i = (u * 32 + lane) * 4;
     if (i >= n) break;
     const float4 wt = *reinterpret_cast<const float4*>(p.norm_w + c0 + i);
-    float4 y = make_float4(v[u].x * r * wt.x, v[u].y * r * wt.y, v[u].z * r * wt.z, v[u].w * r * wt.w);
-    if (!p.gate_first) {
-      y.x *= sigmoid_f32(gate[u].x);
-      y.y *= sigmoid_f32(gate[u].y);
-      y.z *= sigmoid_f32(gate[u].z);
-      y.w *= sigmoid_f32(gate[u].w);
-    }
-    operand_store4(p.out, m, k0 + i, y);
+    operand_store4(p.out, m, k0 + i,
+                   gate4(!first, make_float4(v[u].x * r * wt.x, v[u].y * r * wt.y, v[u].z * r * wt.z, v[u].w * r * wt.w), gate[u], Sigmoid{}));
   }
 }
 
@@ -205,7 +203,7 @@ __device__ __forceinline__ void ssd_gated_norm_warp(const SsdParams& p, const fl
 // nseq * kRingBlocks CTAs update the rings.  256 threads.
 constexpr int kRingBlocks = 8;
 
-__global__ void __launch_bounds__(256) ssd_out_kernel(const __grid_constant__ SsdParams p, const int items, const int small) {
+__global__ void __launch_bounds__(256, 3) ssd_out_kernel(const __grid_constant__ SsdParams p, const int items, const int small) {
   pdl_wait();
   __shared__ float red[8];
   const int n = p.H * p.V / p.groups;

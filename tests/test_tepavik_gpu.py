@@ -22,6 +22,8 @@ REPO = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 ALONE = {
     "lightning": [R.lightning(ff=None)],
     "lightning_one_head": [R.lightning(heads=1, dim=128, vdim=8, decay=(0.97,), ff=None)],
+    "lightning_wide_norm": [R.lightning(heads=70, dim=8, vdim=64, decay=[0.9 + h / 1000 for h in range(70)], ff=None)],
+    "lightning_small_heads": [R.lightning(heads=80, dim=16, vdim=8, decay=[0.9 + h / 1000 for h in range(80)], ff=None)],
     "mamba": [R.mamba(ff=None)],
     "mamba_one_group_no_history": [R.mamba(heads=4, groups=1, conv=1, norm_groups=1, ff=None)],
     "mamba_groups_across_heads": [R.mamba(heads=6, groups=6, vdim=8, conv=6, norm_groups=16, state=130, ff=None)],

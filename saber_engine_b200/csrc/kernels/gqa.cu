@@ -214,6 +214,7 @@ __global__ void __launch_bounds__(128) gqa_row_kernel(const __grid_constant__ Gq
 // grid (M, G, splits), 128 threads.  MT: 16-row tiles of query heads.  NC: 8-column groups of a value per warp.
 template <int MT, int NC>
 __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ GqaParams p) {
+  pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(128) uint8_t smem_raw[];
   __shared__ uint64_t bars[2];

@@ -3,10 +3,12 @@
 // Every kernel of the engine starts with pdl_wait(): launched with the programmatic
 // stream-serialization attribute, a kernel's CTAs may become resident while its predecessor in the
 // stream is still running, and block in pdl_wait() until that predecessor has completed and its
-// writes are visible.  Only the light row kernels call pdl_trigger() (at their top): their
-// successor is a GEMM, one CTA per SM, which cannot be misplaced by starting early.  Nothing a predecessor produced is read, and nothing is written, before the
-// wait, so the result is that of a fully serialised stream; what overlaps is the launch latency,
-// the prologue and -- in the GEMM -- the first weight tiles, which no kernel ever writes.
+// writes are visible.  pdl_trigger() (at a kernel's top) lets the successor start as soon as every CTA of the
+// grid has started: light row kernels and decode mixers, whose successor is a GEMM, one CTA per SM, which cannot be
+// misplaced by starting early, and decode linears of one round of CTAs, whose successor takes the SMs they leave idle.
+// Nothing a kernel of the same step produced is read, and nothing is written, before the wait, so the result is that of a
+// fully serialised stream; what overlaps is the launch latency, the prologue and -- in the GEMM -- the first weight tiles,
+// which no kernel ever writes, or a recurrent state that only an earlier step wrote.
 // Captured into a CUDA graph the same launches become programmatic edges.
 #pragma once
 #include <cuda_runtime.h>

@@ -204,6 +204,7 @@ __device__ __forceinline__ void ssd_gated_norm_warp(const SsdParams& p, const fl
 constexpr int kRingBlocks = 8;
 
 __global__ void __launch_bounds__(256, 3) ssd_out_kernel(const __grid_constant__ SsdParams p, const int items, const int small) {
+  pdl_trigger();
   pdl_wait();
   __shared__ float red[8];
   const int n = p.H * p.V / p.groups;
@@ -264,6 +265,7 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const __grid_constant__ S
   // the state is requested ahead of the wait: the index tables and this layer's state were complete before the step began
   // (the block has VP / 8 warps at most)
   load(warp * 8);
+  pdl_trigger();                                   // the output linear fetches its first weights beside the last CTAs of this grid
   pdl_wait();
   const int pos = p.pos[m], share = p.H / p.HK, hk = h / share;
   const int C = ssd_channels(p);

@@ -304,8 +304,14 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
       tc_fence_after_sync();
       const int m = m0 + row;
       const bool live = row < rows;
-      const float inv = 1.f / (half_s[blocks & 1][0][row] + half_s[blocks & 1][1][row]);
-      const float* g = p.gate == nullptr ? nullptr : p.gate + static_cast<size_t>(live ? m : m0) * p.ldg + h * p.V;
+      float den = half_s[blocks & 1][0][row] + half_s[blocks & 1][1][row];
+      if (p.sink != nullptr) den += ex2(p.sink[h] * kTcLog2e - used * sc);        // (infinite: the sink takes everything)
+      float inv = 1.f / den;
+      const float* g = p.gate == nullptr ? nullptr : p.gate + static_cast<size_t>(live ? m : m0) * p.ldg + (p.gate_heads ? h : h * p.V);
+      if (g != nullptr && p.gate_heads) {
+        inv /= 1.f + expf(-g[0]);
+        g = nullptr;
+      }
       const int k0 = p.out_k0 + h * p.V;
       for (int c = half * 32; c < VP; c += 64) {
         uint32_t r[32];

@@ -12,8 +12,9 @@ struct FlashParams {
   const void* k;              // of page p and key / value head g: k + (p G + g) k_stride bytes
   const void* v;
   size_t k_stride, v_stride;
-  const float* gate;          // [M][ldg] (column h V + v) through a sigmoid onto the output, or null
-  int ldg;
+  const float* gate;          // [M][ldg] (column h V + v, or h where gate_heads) through a sigmoid onto the output, or null
+  int ldg, gate_heads;
+  const float* sink;          // [H]: exp(sink) joins the denominator, or null
   const int32_t* cu_rows;     // [nseq + 1]
   const int32_t* kv_len;      // [nseq]
   const int32_t* block_table; // [nseq][max_blocks]

@@ -10,6 +10,7 @@
 #include "gqa.h"
 #include "launch.cuh"
 #include "mla_device.cuh"
+#include "rotary.cuh"
 
 namespace saber {
 
@@ -43,10 +44,15 @@ __device__ __forceinline__ float head_scale(const GqaParams& p, const float* x, 
   return 1.f / sqrtf(mla_warp_sum(sq) / static_cast<float>(p.D) + p.eps);
 }
 
-// Four rows of a head from x on (rows past n repeat the last), divided by their root mean square; put(row, d, four values)
-// takes the pieces.  D a multiple of 4, at most 256.
+__device__ __forceinline__ float gated(const GqaParams& p, int m, int h, int v, float y) {
+  if (p.g_off < 0) return y;
+  return y / (1.f + expf(-p.x[static_cast<size_t>(m) * p.ldx + p.g_off + h * p.V + v]));
+}
+
+// Four rows of a head from x on (rows past n repeat the last), divided by their root mean square and rotated by the tables
+// at t (rot floats a row); put(row, d, four values) takes the pieces.  D a multiple of 4, at most 256; rot a multiple of 8.
 template <typename Put>
-__device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x, int n, int lane, const Put& put) {
+__device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x, int n, int lane, const float* t, const Put& put) {
   float4 v[4][2];
   float sq[4];
 #pragma unroll
@@ -58,14 +64,33 @@ __device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x,
     }
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
+    if (!p.qk_norm) break;
     sq[r] = 0.f;
 #pragma unroll
     for (int u = 0; u < 2; ++u) sq[r] += v[r][u].x * v[r][u].x + v[r][u].y * v[r][u].y + v[r][u].z * v[r][u].z + v[r][u].w * v[r][u].w;
   }
+  if (p.qk_norm)
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1)
+    for (int o = 16; o > 0; o >>= 1)
 #pragma unroll
-    for (int r = 0; r < 4; ++r) sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], o);
+      for (int r = 0; r < 4; ++r) sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], o);
+  if (p.rot > 0) {                                // (the partner's four values: another lane's, read again)
+    const int half = p.rot / 2;
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int d = u * 128 + lane * 4;
+        if (d >= p.rot) continue;
+        const bool lo = d < half;
+        const float* tr = t + min(r, n - 1) * p.rot + (lo ? d : d - half);
+        const float4 o4 = *reinterpret_cast<const float4*>(x + static_cast<size_t>(min(r, n - 1)) * p.ldx + (lo ? d + half : d - half));
+        const float4 c = *reinterpret_cast<const float4*>(tr), s = *reinterpret_cast<const float4*>(tr + half);
+        const float sg = lo ? -1.f : 1.f;
+        float4& w = v[r][u];
+        w = make_float4(w.x * c.x + sg * o4.x * s.x, w.y * c.y + sg * o4.y * s.y, w.z * c.z + sg * o4.z * s.z, w.w * c.w + sg * o4.w * s.w);
+      }
+  }
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
     if (r >= n) break;
@@ -81,17 +106,22 @@ __device__ __forceinline__ uint2 pack4(float4 v) { return make_uint2(pack2(v.x, 
 template <typename T>
 __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__ GqaParams p) {
   pdl_wait();
+  extern __shared__ __align__(16) float rot_s[];  // rotation tables of the eight rows
   const int lane = threadIdx.x & 31;
   int item = blockIdx.y * 8 + (threadIdx.x >> 5);
   const int m0 = blockIdx.x * 8, n = min(8, p.M - m0);
-  const bool fast = sizeof(T) == 2 && (p.D & 3) == 0 && p.D <= 256;
+  const bool fast = sizeof(T) == 2 && (p.D & 3) == 0 && p.D <= 256 && (p.rot & 7) == 0;
+  if (p.rot > 0) {
+    for (int r = threadIdx.x >> 5; r < n; r += 8) rotary_table(rot_s + r * p.rot, p.freq, p.rot, p.rot_amp, p.pos[m0 + r], lane, 32);
+    __syncthreads();
+  }
   if (p.form == 2) {
     if (item < p.H) {
       __nv_bfloat16* q0 = static_cast<__nv_bfloat16*>(p.q) + (static_cast<size_t>(m0) * p.H + item) * p.DK;
       const float* x0 = p.x + static_cast<size_t>(m0) * p.ldx + p.q_off + item * p.D;
       if (fast) {
         for (int r0 = 0; r0 < n; r0 += 4)
-          normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, [&](int r, int d, float4 v) {
+          normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
             if (d < p.DK) *reinterpret_cast<uint2*>(q0 + static_cast<size_t>(r0 + r) * p.H * p.DK + d) = pack4(v);      // (zeros from D on)
           });
         return;
@@ -99,7 +129,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
       for (int r = 0; r < n; ++r) {
         const float* x = x0 + static_cast<size_t>(r) * p.ldx;
         const float s = head_scale(p, x, lane);
-        for (int d = lane; d < p.DK; d += 32) q0[static_cast<size_t>(r) * p.H * p.DK + d] = __float2bfloat16(d < p.D ? x[d] * s : 0.f);
+        for (int d = lane; d < p.DK; d += 32) q0[static_cast<size_t>(r) * p.H * p.DK + d] = __float2bfloat16(d < p.D ? rotary_half(x, d, rot_s + r * p.rot, p.rot) * s : 0.f);
       }
       return;
     }
@@ -123,7 +153,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
 #pragma unroll
       for (int r0 = 0; r0 < 8; r0 += 4) {
         if (r0 >= n) break;
-        normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, [&](int r, int d, float4 v) {
+        normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
           const int s = r == 0 ? slot[r0] : r == 1 ? slot[r0 + 1] : r == 2 ? slot[r0 + 2] : slot[r0 + 3];
           if (s >= 0 && d < p.D)
             *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.cache) + page_block(p, s / kPage, g) + bf16_key_at(s % kPage, d)) = pack4(v);
@@ -137,7 +167,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
       const float* x = x0 + static_cast<size_t>(r) * p.ldx;
       const float sc = head_scale(p, x, lane);
       const size_t b = page_block(p, s / kPage, g);
-      for (int d = lane; d < p.D; d += 32) Page<T>::store(p.cache, b + Page<T>::key(p, s % kPage, d), x[d] * sc);
+      for (int d = lane; d < p.D; d += 32) Page<T>::store(p.cache, b + Page<T>::key(p, s % kPage, d), rotary_half(x, d, rot_s + r * p.rot, p.rot) * sc);
     }
     return;
   }
@@ -164,7 +194,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
 template <typename T>
 __global__ void __launch_bounds__(128) gqa_row_kernel(const __grid_constant__ GqaParams p) {
   pdl_wait();
-  extern __shared__ float sm[];                   // q [D] | scores [64] | output [V]
+  extern __shared__ float sm[];                   // q [D] | scores [64] | output [V] | rotation table
   __shared__ float scale_s;
   const int m = blockIdx.x, h = blockIdx.y, g = h / (p.H / p.G);
   const int j = mla_seq_of_row(p.cu_rows, p.nseq, m);
@@ -173,13 +203,18 @@ __global__ void __launch_bounds__(128) gqa_row_kernel(const __grid_constant__ Gq
   float* sc = sm + p.D;
   float* o = sc + kPage;
   const float* x = p.x + static_cast<size_t>(m) * p.ldx + p.q_off + h * p.D;
+  float* rot_s = o + p.V;
   if (warp == 0) {
     const float s = head_scale(p, x, lane);
     if (lane == 0) scale_s = s;
   }
+  if (p.rot > 0) rotary_table(rot_s, p.freq, p.rot, p.rot_amp, p.pos[m], threadIdx.x, 128);
   __syncthreads();
   // (queries are rounded like the keys they meet)
-  for (int d = threadIdx.x; d < p.D; d += 128) sm[d] = sizeof(T) == 2 ? __bfloat162float(__float2bfloat16(x[d] * scale_s)) : x[d] * scale_s;
+  for (int d = threadIdx.x; d < p.D; d += 128) {
+    const float q = rotary_half(x, d, rot_s, p.rot) * scale_s;
+    sm[d] = sizeof(T) == 2 ? __bfloat162float(__float2bfloat16(q)) : q;
+  }
   for (int v = threadIdx.x; v < p.V; v += 128) o[v] = 0.f;
   const int pos = p.pos[m], low = p.chunk > 0 ? pos - pos % p.chunk : 0;
   float mx = -INFINITY, l = 0.f;
@@ -208,7 +243,8 @@ __global__ void __launch_bounds__(128) gqa_row_kernel(const __grid_constant__ Gq
       o[v] = s;
     }
   }
-  for (int v = threadIdx.x; v < p.V; v += 128) operand_store1(p.out, m, p.out_k0 + h * p.V + v, o[v] / l);
+  if (p.sink != nullptr) l += expf(p.sink[h] - mx);                 // (infinite: the sink takes everything)
+  for (int v = threadIdx.x; v < p.V; v += 128) operand_store1(p.out, m, p.out_k0 + h * p.V + v, gated(p, m, h, v, o[v] / l));
 }
 
 // grid (M, G, splits), 128 threads.  MT: 16-row tiles of query heads.  NC: 8-column groups of a value per warp.
@@ -237,6 +273,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
   float* s_f = reinterpret_cast<float*>(base + 2 * stage + MT * 16 * qs + MT * 16 * 144);      // scores [MT * 16][64 + 4]
   const bool append = p.max_rows == 1 && p.k_off >= 0 && n > 0 && pa + n == page0 + pages;     // the new token's page is mine
   __nv_bfloat16* new_s = reinterpret_cast<__nv_bfloat16*>(s_f + MT * 16 * 68);                 // key [KP] | value [VP] of the new token
+  float* rot_s = reinterpret_cast<float*>(new_s + p.KP + p.VP);                                // rotation table of the position
   const uint32_t bar = smem_u32(bars);
   const uint8_t* cache = static_cast<const uint8_t*>(p.cache);
   auto fetch = [&](int it) {
@@ -251,11 +288,15 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
     for (; issued < min(2, n); ++issued) fetch(issued);
   }
   const float* xr = p.x + static_cast<size_t>(m) * p.ldx;
+  if (p.rot > 0) {
+    rotary_table(rot_s, p.freq, p.rot, p.rot_amp, pos, threadIdx.x, 128);
+    __syncthreads();
+  }
   for (int r = warp; r < MT * 16; r += 4) {
     const float* x = xr + p.q_off + (g * hq + min(r, hq - 1)) * p.D;
     const float s = head_scale(p, x, lane);
     for (int d = lane * 2; d < p.DK; d += 64) {
-      const float a = r < hq && d < p.D ? x[d] * s : 0.f, b = r < hq && d + 1 < p.D ? x[d + 1] * s : 0.f;
+      const float a = r < hq && d < p.D ? rotary_half(x, d, rot_s, p.rot) * s : 0.f, b = r < hq && d + 1 < p.D ? rotary_half(x, d + 1, rot_s, p.rot) * s : 0.f;
       asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_s + r * qs + d * 2), "r"(pack2(a, b)) : "memory");
     }
   }
@@ -269,7 +310,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
       const float* x = xr + p.k_off + g * p.D;
       const float s = head_scale(p, x, lane);
       for (int d = lane; d < p.D; d += 32) {
-        new_s[d] = __float2bfloat16(x[d] * s);
+        new_s[d] = __float2bfloat16(rotary_half(x, d, rot_s, p.rot) * s);
         if (live) c[bf16_key_at(slot % kPage, d)] = new_s[d];
       }
     } else {
@@ -385,7 +426,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
   for (int i = 0; i < 4 * MT; ++i) {
     const int r = warp + 4 * i;
     if (r >= hq || lane != 0) continue;
-    l_s[r] = l[i];
+    l_s[r] = p.sink != nullptr ? l[i] + ex2((p.sink[g * hq + r] - mx[i]) * kGqaLog2e) : l[i];    // (infinite: the sink takes everything)
     if (p.splits > 1) {
       float* d = p.ml + ((static_cast<size_t>(m) * p.H + g * hq + r) * p.splits + sp) * 2;
       __stcg(d, mx[i]);
@@ -410,8 +451,8 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
         if (d != nullptr) {
           if (n > 0) __stcg(reinterpret_cast<float2*>(d + v), make_float2(a, b));
         } else {
-          if (v < p.V) operand_store1(p.out, m, p.out_k0 + h * p.V + v, a * inv);
-          if (v + 1 < p.V) operand_store1(p.out, m, p.out_k0 + h * p.V + v + 1, b * inv);
+          if (v < p.V) operand_store1(p.out, m, p.out_k0 + h * p.V + v, gated(p, m, h, v, a * inv));
+          if (v + 1 < p.V) operand_store1(p.out, m, p.out_k0 + h * p.V + v + 1, gated(p, m, h, v + 1, b * inv));
         }
       }
     }
@@ -434,7 +475,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
     const float pl = lane < p.splits ? __ldcg(ml + (r * p.splits + lane) * 2 + 1) : 0.f;
     const float mm = mla_warp_max(pm);
     const float w = pm > -INFINITY ? ex2((pm - mm) * kGqaLog2e) : 0.f;
-    const float tot = mla_warp_sum(w * pl);
+    const float tot = mla_warp_sum(w * pl) + (p.sink != nullptr ? ex2((p.sink[g * hq + r] - mm) * kGqaLog2e) : 0.f);
     s_f[r * 33 + lane] = w / tot;
   }
   __syncthreads();
@@ -447,7 +488,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
       const float w = s_f[r * 33 + s];
       if (w > 0.f) y = fmaf(w, __ldcg(part + (static_cast<size_t>(r) * p.splits + s) * p.VP + v), y);
     }
-    operand_store1(p.out, m, p.out_k0 + (g * hq + r) * p.V + v, y);
+    operand_store1(p.out, m, p.out_k0 + (g * hq + r) * p.V + v, gated(p, m, g * hq + r, v, y));
   }
 }
 
@@ -457,7 +498,7 @@ static int split_tiles(const GqaParams& p) {
 }
 static int split_smem(const GqaParams& p) {
   const int rows = split_tiles(p) * 16;
-  return 2 * 128 * (p.KP + p.VP) + rows * (p.DK * 2 + 16 + 144 + 68 * 4) + 2 * (p.KP + p.VP) + 128;
+  return 2 * 128 * (p.KP + p.VP) + rows * (p.DK * 2 + 16 + 144 + 68 * 4) + 2 * (p.KP + p.VP) + p.rot * 4 + 128;
 }
 template <int MT, int NC>
 static int split_go(const GqaParams& p, cudaStream_t stream) {
@@ -486,11 +527,11 @@ static int append_items(const GqaParams& p) {
 template <typename T>
 static int gqa_go(const GqaParams& p, cudaStream_t stream) {
   if (const int items = append_items(p)) {
-    const cudaError_t e = launch(gqa_append_kernel<T>, dim3((p.M + 7) / 8, (items + 7) / 8), dim3(256), 0, stream, 0, p);
+    const cudaError_t e = launch(gqa_append_kernel<T>, dim3((p.M + 7) / 8, (items + 7) / 8), dim3(256), 8 * p.rot * 4, stream, 0, p);
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   if (p.form == 0)
-    return static_cast<int>(launch(gqa_row_kernel<T>, dim3(p.M, p.H), dim3(128), (p.D + kPage + p.V) * 4, stream, 0, p));
+    return static_cast<int>(launch(gqa_row_kernel<T>, dim3(p.M, p.H), dim3(128), (p.D + kPage + p.V + p.rot) * 4, stream, 0, p));
   if (p.form == 1)
     return p.VP <= 32 ? split_mt<1>(p, stream) : p.VP <= 64 ? split_mt<2>(p, stream) : p.VP <= 128 ? split_mt<4>(p, stream) : split_mt<8>(p, stream);
   FlashParams f = {};
@@ -515,6 +556,9 @@ static int gqa_go(const GqaParams& p, cudaStream_t stream) {
   f.chunk = p.chunk;
   f.scale = p.scale;
   f.softcap = p.softcap;
+  f.gate = p.g_off < 0 ? nullptr : p.x + p.g_off;
+  f.ldg = p.ldx;
+  f.sink = p.sink;
   f.bound = p.qk_norm ? 1.02f * p.D : 0.f;        // (two vectors of root mean square one, and the rounding to bf16)
   f.err = p.err;
   return saber_flash_tc(&f, stream);
@@ -534,7 +578,7 @@ extern "C" int saber_gqa_launches(const saber::GqaParams* p) { return saber::app
 extern "C" int saber_gqa_launch(const saber::GqaParams* p, cudaStream_t stream) {
   using namespace saber;
   if (p->M <= 0 || p->G <= 0 || p->H % p->G || p->page != kPage || p->D > p->DK || p->DK > p->KP || p->V > p->VP || p->cache == nullptr ||
-      p->D > 2048 || p->V > 2048 || p->form < 0 || p->form > saber_gqa_form(p) || (p->form == 2 && p->q == nullptr) ||
+      p->D > 2048 || p->V > 2048 || p->rot < 0 || (p->rot & 1) || p->rot > p->D || p->rot > 1024 || (p->rot > 0 && p->freq == nullptr) || p->form < 0 || p->form > saber_gqa_form(p) || (p->form == 2 && p->q == nullptr) ||
       (p->form == 1 && (p->splits < 1 || p->splits > 32 || (p->splits > 1 && (p->o_part == nullptr || p->ml == nullptr || p->counters == nullptr)))))
     return static_cast<int>(cudaErrorInvalidValue);
   return p->f32 ? gqa_go<float>(*p, stream) : gqa_go<__nv_bfloat16>(*p, stream);

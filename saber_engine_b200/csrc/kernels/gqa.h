@@ -1,8 +1,11 @@
 // Launch interface of grouped-query attention over tiled pages (gqa.cu): H query heads share G key / value heads,
 // fp32 scores.  Plain C types only.
 //
-//   q, k    optionally divided by their root mean square over D (qk_norm)
+//   q, k    optionally divided by their root mean square over D (qk_norm), then rotated (rot > 0: the first rot values, halves
+//           layout)
 //   score   scale q . k, then cap tanh(score / cap) when softcap > 0
+//   sink    exp(sink[h]) joins the denominator of head h
+//   gate    the output times sigmoid of column g_off + h V + v of x
 //   mask    keys j <= i; chunk > 0: of the same chunk of positions as i only, j >= i - i % chunk
 //
 // A page holds, per key / value head, the keys and then the values of its 64 tokens.  bf16: in the order the
@@ -18,6 +21,11 @@ namespace saber {
 struct GqaParams {
   const float* x;             // [M][ldx] projections of this step's rows
   int ldx, q_off, k_off, v_off;   // k_off < 0: the cache is another layer's, nothing is appended
+  int g_off;                      // < 0: no gate
+  int rot;
+  float rot_amp;
+  const float* freq;          // [rot / 2]
+  const float* sink;          // [H] or null
   void* cache;                // [n_blocks][G][64 (KP + VP)]
   void* q;                    // scratch [M][H][DK] bf16 (tcgen05 form)
   float* o_part;              // scratch [M][H][splits][VP]

@@ -11,6 +11,10 @@
 //
 // fp32: a CUDA-core GEMM (plain fused multiply-adds) followed by one row kernel that runs the same
 // epilogue; the bf16 linear takes this two-launch form too when fuse = 0.
+//
+// A grouped product (mixtures of experts) is the same kernel over a table of row tiles, each against the weights of its
+// expert.  Where the operand rows are tokens out of order, the eight epilogue warps, idle until the accumulator is done, copy them
+// into the ring row by row (16-byte asynchronous copies, swizzled for their place in the tile).
 #include "launch.cuh"
 #include "linear.h"
 #include "ptx_sm100.cuh"
@@ -33,6 +37,39 @@ __device__ __forceinline__ float relu_squared(float x) {
   return r * r;
 }
 
+__device__ __forceinline__ float gelu(float x) { return 0.5f * x * (1.f + erff(x * 0.70710678118654752f)); }
+
+__device__ __forceinline__ float stored(const LinEpi& e, int n, float v) {      // bias and cap of a stored column
+  if (e.bias) v += e.bias[n];
+  return e.cap > 0.f ? e.cap * tanhf(v / e.cap) : v;
+}
+
+constexpr int kGatedTile = 248;           // features of a tile of act_kind 2; row 248 of the tile is their gate
+
+// v[0..7] += sum over the routes of token m of their weight times the expert's row, columns from n on
+__device__ __forceinline__ void add_routes(const LinEpi& e, int m, int n, float (&v)[8]) {
+#pragma unroll 4
+  for (int k = 0; k < e.routes; ++k) {
+    const int r = e.slot_of[m * e.routes + k];
+    if (r < 0) continue;
+    const float w = e.route_w[m * e.routes + k];
+    if (e.y_f32) {
+      const float4* y = reinterpret_cast<const float4*>(static_cast<const float*>(e.y) + static_cast<size_t>(r) * e.ldy + n);
+      const float4 a = __ldcg(y), b = __ldcg(y + 1);
+      v[0] = fmaf(w, a.x, v[0]); v[1] = fmaf(w, a.y, v[1]); v[2] = fmaf(w, a.z, v[2]); v[3] = fmaf(w, a.w, v[3]);
+      v[4] = fmaf(w, b.x, v[4]); v[5] = fmaf(w, b.y, v[5]); v[6] = fmaf(w, b.z, v[6]); v[7] = fmaf(w, b.w, v[7]);
+    } else {
+      const uint4 q = __ldcg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(e.y) + static_cast<size_t>(r) * e.ldy + n));
+      const uint32_t u[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        v[2 * i] = fmaf(w, __uint_as_float(u[i] << 16), v[2 * i]);
+        v[2 * i + 1] = fmaf(w, __uint_as_float(u[i] & 0xFFFF0000u), v[2 * i + 1]);
+      }
+    }
+  }
+}
+
 // reciprocal root mean square of the stream row behind operand row m (all lanes of a warp call together)
 __device__ __forceinline__ float row_rms_scale(const LinEpi& e, int m, int lane) {
   if (e.ss == nullptr) return 1.f;
@@ -50,14 +87,44 @@ template <typename Acc>
 __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& acc, int m, int tile_n, int lane, float sc, float4 x0, float4 x1) {
   const int n0 = tile_n * 256;
   if (!e.stream) {
+    if (tile_n < e.lat_tiles) {
+      const int n = n0 + lane * 8;
+      const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+      const float v[8] = {a.x * sc, a.y * sc, a.z * sc, a.w * sc, b.x * sc, b.y * sc, b.z * sc, b.w * sc};
+      float y[8], sq = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const bool in = n + j < e.lat_n;
+        sq += in ? v[j] * v[j] : 0.f;
+        y[j] = in ? v[j] * e.lat_w[n + j] : 0.f;
+      }
+      if (n < e.lat.ld) operand_store8(e.lat, m, n, y);              // (the operand ends at a multiple of 64 columns)
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      const int g = tile_n * 2 + (lane >> 4);
+      if ((lane & 15) == 0 && g < e.lat_ss_n) e.lat_ss[static_cast<size_t>(m) * e.lat_ss_n + g] = sq;
+      return;
+    }
     if (tile_n < e.act_tile0) {
       const int n = n0 + lane * 8;
       if (n >= e.n_plain) return;
       float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+      if (e.out_bf16) {                                              // (rows of whole groups of eight)
+        const float v[8] = {a.x * sc, a.y * sc, a.z * sc, a.w * sc, b.x * sc, b.y * sc, b.z * sc, b.w * sc};
+        uint4 q;
+        uint32_t* u = reinterpret_cast<uint32_t*>(&q);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+          u[j] = *reinterpret_cast<const uint32_t*>(&h);
+        }
+        *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(e.out) + static_cast<size_t>(m) * e.ldo + n) = q;
+        return;
+      }
       float* o = e.out + static_cast<size_t>(m) * e.ldo + n;
       a = make_float4(a.x * sc, a.y * sc, a.z * sc, a.w * sc);
       b = make_float4(b.x * sc, b.y * sc, b.z * sc, b.w * sc);
-      if (n + 8 <= e.n_plain) {
+      if (n + 8 <= e.n_plain && !(e.cap > 0.f)) {
         if (e.bias) {
           const float4 c = *reinterpret_cast<const float4*>(e.bias + n), d = *reinterpret_cast<const float4*>(e.bias + n + 4);
           a = make_float4(a.x + c.x, a.y + c.y, a.z + c.z, a.w + c.w);
@@ -69,7 +136,7 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
         const float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
 #pragma unroll
         for (int j = 0; j < 8; ++j)
-          if (n + j < e.n_plain) o[j] = v[j] + (e.bias ? e.bias[n + j] : 0.f);
+          if (n + j < e.n_plain) o[j] = stored(e, n + j, v[j]);
       }
     } else if (e.act_kind == 1) {
       const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
@@ -77,6 +144,25 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
                           relu_squared(b.x * sc), relu_squared(b.y * sc), relu_squared(b.z * sc), relu_squared(b.w * sc)};
       const int k = e.act_k0 + (tile_n - e.act_tile0) * 256 + lane * 8;
       if (k < e.act.ld) operand_store8(e.act, m, k, y);              // (the operand ends at a multiple of 64 columns, the tile of 256)
+    } else if (e.act_kind == 2) {
+      const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+      const float gate = 1.f / (1.f + expf(-__shfl_sync(0xffffffffu, a.x * sc, 31)));
+      const float y[8] = {gate * relu_squared(a.x * sc), gate * relu_squared(a.y * sc), gate * relu_squared(a.z * sc), gate * relu_squared(a.w * sc),
+                          gate * relu_squared(b.x * sc), gate * relu_squared(b.y * sc), gate * relu_squared(b.z * sc), gate * relu_squared(b.w * sc)};
+      const int k = e.act_k0 + (tile_n - e.act_tile0) * kGatedTile + lane * 8;
+      if (lane < 31 && k < e.act.ld) operand_store8(e.act, m, k, y);
+    } else if (e.act_kind == 3) {
+      const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
+      const int f = (tile_n - e.act_tile0) * 256 + lane * 8, k = e.act_k0 + f;
+      if (k >= e.act.ld) return;
+      float4 c = make_float4(0.f, 0.f, 0.f, 0.f), d = c;
+      if (e.act_bias) {
+        c = *reinterpret_cast<const float4*>(e.act_bias + f);
+        d = *reinterpret_cast<const float4*>(e.act_bias + f + 4);
+      }
+      const float y[8] = {gelu(fmaf(a.x, sc, c.x)), gelu(fmaf(a.y, sc, c.y)), gelu(fmaf(a.z, sc, c.z)), gelu(fmaf(a.w, sc, c.w)),
+                          gelu(fmaf(b.x, sc, d.x)), gelu(fmaf(b.y, sc, d.y)), gelu(fmaf(b.z, sc, d.z)), gelu(fmaf(b.w, sc, d.w))};
+      operand_store8(e.act, m, k, y);
     } else {
       const float4 g = acc(lane * 4), u = acc(128 + lane * 4);
       operand_store4(e.act, m, e.act_k0 + (tile_n - e.act_tile0) * 128 + lane * 4,
@@ -91,6 +177,7 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
     float* xr = e.x + static_cast<size_t>(m) * e.ldx + n;
     const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
     float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+    if (e.y != nullptr) add_routes(e, m, n, v);
     if (e.add) {
       v[0] += x0.x; v[1] += x0.y; v[2] += x0.z; v[3] += x0.w;
       v[4] += x1.x; v[5] += x1.y; v[6] += x1.z; v[7] += x1.w;
@@ -106,6 +193,11 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
     *reinterpret_cast<float4*>(xr) = make_float4(v[0], v[1], v[2], v[3]);
     *reinterpret_cast<float4*>(xr + 4) = make_float4(v[4], v[5], v[6], v[7]);
     operand_store8(e.op, m, e.op_k0 + n, y);
+    if (e.norm_w2 != nullptr) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) y[j] = n + j < e.width ? v[j] * e.norm_w2[n + j] : 0.f;
+      operand_store8(e.op2, m, n, y);
+    }
   }
   if (e.ss_out == nullptr) return;
 #pragma unroll
@@ -142,12 +234,19 @@ __device__ __forceinline__ void linear_tile_epilogue(const LinEpi& e, const floa
   }
 }
 
-template <int kMT>
+// kGroup: 0 a plain product, 1 a grouped one, 2 a grouped one whose operand rows are gathered by the epilogue warps
+template <int kMT, int kGroup>
 __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_constant__ LinParams p, const int stages) {
   extern __shared__ uint8_t smem_raw[];
   // one round of CTAs: the successor may take the SMs this grid leaves idle or frees (until its own wait it touches
   // weights only)
-  if (gridDim.x == 1) pdl_trigger();
+  if (kGroup != 0 || gridDim.x == 1) pdl_trigger();
+  int4 group = make_int4(0, 0, 0, 0);
+  if constexpr (kGroup != 0) {
+    pdl_wait();
+    if (static_cast<int>(blockIdx.x) >= p.group_ntiles[0]) return;
+    group = p.group_tiles[blockIdx.x];
+  }
   __shared__ uint64_t bars[2 * kLinMaxStages + 1];
   __shared__ uint32_t tmem_base_s, is_last_s, abort_s;
   __shared__ float scale_s[256];
@@ -158,7 +257,8 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
   const int kb_per = (KB + p.splits - 1) / p.splits;
   const int kb0 = split * kb_per;
   const int nkb = min(KB, kb0 + kb_per) - kb0;        // host guarantees >= 1
-  const int m0 = tile_m * p.nt * kMT;
+  const int m0 = kGroup != 0 ? group.y : tile_m * p.nt * kMT;
+  const int m_end = kGroup != 0 ? group.y + group.z : p.M;
   const uint32_t abytes = static_cast<uint32_t>(p.nt) * 128u * kMT;
   const uint32_t a_smem = (smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t w_smem = a_smem + static_cast<uint32_t>(stages) * abytes;
@@ -169,7 +269,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < stages; ++s) {
-      mbar_init(bar_full + 8 * s, 1);
+      mbar_init(bar_full + 8 * s, kGroup == 2 ? 9 : 1);
       mbar_init(bar_empty + 8 * s, 1);
     }
     mbar_init(bar_acc, 1);
@@ -189,29 +289,33 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
   if (warp == 0) {
     // ---------------------------------------------------------------- producer
     if (lane == 0) {
+      constexpr bool kCopyA = kGroup != 2;
+      const uint32_t tx = kLinTile + (kCopyA ? abytes : 0u);
       const uint64_t pol = gridDim.x > 1 ? l2_policy_evict_normal() : l2_policy_evict_first();
-      const uint8_t* wp = static_cast<const uint8_t*>(p.w) + (static_cast<size_t>(tile_n) * KB + kb0) * kLinTile;
-      const uint8_t* ap = static_cast<const uint8_t*>(p.a) + (static_cast<size_t>(kb0) * p.M_pad + m0) * 128;
+      const uint8_t* wp = static_cast<const uint8_t*>(p.w) + group.x * p.group_w_stride + (static_cast<size_t>(tile_n) * KB + kb0) * kLinTile;
+      const uint8_t* ap = static_cast<const uint8_t*>(p.a2 != nullptr && tile_n >= p.a2_tile0 ? p.a2 : p.a) +
+                          (static_cast<size_t>(kb0) * p.M_pad + m0) * 128;
       const size_t a_step = static_cast<size_t>(p.M_pad) * 128;
       const int pre = min(stages, nkb);
       for (int it = 0; it < pre; ++it) {         // weights do not depend on the predecessor kernel
-        mbar_arrive_expect_tx(bar_full + 8 * it, kLinTile + abytes);
+        mbar_arrive_expect_tx(bar_full + 8 * it, tx);
         bulk_g2s_hint(w_smem + it * kLinTile, wp, kLinTile, bar_full + 8 * it, pol);
         wp += kLinTile;
       }
       pdl_wait();
-      for (int it = 0; it < pre; ++it) {
-        bulk_g2s(a_smem + it * abytes, ap, abytes, bar_full + 8 * it);
-        ap += a_step;
-      }
+      if constexpr (kCopyA)
+        for (int it = 0; it < pre; ++it) {
+          bulk_g2s(a_smem + it * abytes, ap, abytes, bar_full + 8 * it);
+          ap += a_step;
+        }
       int issued = pre, s = pre == stages ? 0 : pre;
       uint32_t ph = pre == stages ? 1u : 0u;
       bool ok = true;
       for (int it = pre; it < nkb; ++it) {
         if (!mbar_wait(bar_empty + 8 * s, ph ^ 1u, p.err, kErrWaitEmpty)) { ok = false; break; }
-        mbar_arrive_expect_tx(bar_full + 8 * s, kLinTile + abytes);
+        mbar_arrive_expect_tx(bar_full + 8 * s, tx);
         bulk_g2s_hint(w_smem + s * kLinTile, wp, kLinTile, bar_full + 8 * s, pol);
-        bulk_g2s(a_smem + s * abytes, ap, abytes, bar_full + 8 * s);
+        if constexpr (kCopyA) bulk_g2s(a_smem + s * abytes, ap, abytes, bar_full + 8 * s);
         wp += kLinTile;
         ap += a_step;
         issued = it + 1;
@@ -261,11 +365,53 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
     const int q4 = warp & 3;                      // TMEM lane quarter of this warp
     const LinEpi& e = p.e;
     pdl_wait();
+    if constexpr (kGroup == 2) {
+      // operand rows: up to four 16-byte pieces of every k-block per thread, three k-blocks in flight
+      constexpr int kLag = 2;                     // (below the number of stages)
+      const uint8_t* src[4];
+      uint32_t dst[4];
+      bool live[4];
+      const size_t a_step = static_cast<size_t>(p.M_pad) * 128;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int r = (te + 256 * i) >> 3, c = te & 7;
+        live[i] = r < group.z;
+        const int m = live[i] ? max(p.src_row[m0 + r], 0) : 0;
+        src[i] = static_cast<const uint8_t*>(p.a) + static_cast<size_t>(m) * 128 + (((c ^ m) & 7) << 4);
+        dst[i] = a_smem + static_cast<uint32_t>(r) * 128u + (((c ^ r) & 7) << 4);
+      }
+      int s = 0, done = 0;                        // done: k-blocks handed to the tensor cores
+      uint32_t ph = 0;
+      bool ok = true;
+      auto hand_over = [&](int it) {
+        fence_proxy_async_smem();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(bar_full + 8 * (it % stages));
+      };
+      for (int it = 0; it < nkb; ++it) {
+        if (it >= stages) ok = __all_sync(0xffffffffu, mbar_wait(bar_empty + 8 * s, ph ^ 1u, p.err, kErrWaitEmpty));
+        if (!ok) break;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          if (live[i]) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst[i] + s * abytes), "l"(src[i]) : "memory");
+          src[i] += a_step;
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (it >= kLag) {
+          asm volatile("cp.async.wait_group %0;" ::"n"(kLag) : "memory");
+          hand_over(done++);
+        }
+        if (++s == stages) { s = 0; ph ^= 1u; }
+      }
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      if (ok)
+        while (done < nkb) hand_over(done++);
+    }
     // row scales while the main loop runs: a thread per row
     if (te < p.nt * kMT) {
       float sc = 1.f;
-      if (e.ss != nullptr && m0 + te < p.M) {
-        const float* q = e.ss + static_cast<size_t>(m0 + te) * e.ss_n;
+      if (e.ss != nullptr && m0 + te < m_end) {
+        const float* q = e.ss + static_cast<size_t>(kGroup == 2 ? max(p.src_row[m0 + te], 0) : m0 + te) * e.ss_n;
         float s = 0.f;
 #pragma unroll 8
         for (int i = 0; i < e.ss_n; ++i) s += __ldcg(q + i);
@@ -283,7 +429,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
     const int tile_lin = tile_m * gridDim.y + tile_n;
     float* tile_s = reinterpret_cast<float*>(smem_raw + (a_smem - smem_u32(smem_raw)));
     if (p.splits > 1) {                           // (kMT == 1)
-      const int mt = min(p.nt, p.M - m0);
+      const int mt = min(p.nt, m_end - m0);
       float* part = p.ws + (static_cast<size_t>(tile_lin) * p.splits + split) * p.nt * 256;
       if (ok && q4 * 32 < mt) {
         for (int c = grp * 128; c < grp * 128 + 128; c += 32) {
@@ -332,7 +478,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
 #pragma unroll 1
       for (int j2 = 0; j2 < kMT; ++j2) {
         const int mb = m0 + j2 * p.nt;
-        const int mt = min(p.nt, p.M - mb);
+        const int mt = min(p.nt, m_end - mb);
         if (mt <= 0) break;                       // uniform
         if (j2 > 0) named_bar_sync(1, 256);
         if (q4 * 32 < mt) {
@@ -360,16 +506,28 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
 
 // ------------------------------------------------------------------------------------ fp32 GEMM
 // 64 x 64 output tile, 16 k per step, 4 x 4 outputs per thread; plain fused multiply-adds.
-__global__ void __launch_bounds__(256) lin_f32_kernel(const float* __restrict__ a, const float* __restrict__ w, float* __restrict__ out,
-                                                      int M, int N, int K) {
+__global__ void __launch_bounds__(256) lin_f32_kernel(const __grid_constant__ LinParams p) {
   pdl_wait();
   __shared__ float as[16][68], ws[16][68];
-  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const int N = p.N_pad, K = p.K, n0 = blockIdx.x * 64;
+  int m0 = blockIdx.y * 64, m_end = p.M;
+  const float* w = static_cast<const float*>(p.w);
+  const float* a = static_cast<const float*>(p.a2 != nullptr && n0 >= p.a2_tile0 * 256 ? p.a2 : p.a);
+  if (p.group_tiles != nullptr) {
+    if (static_cast<int>(blockIdx.y) >= p.group_ntiles[0]) return;
+    const int4 g = p.group_tiles[blockIdx.y];
+    m0 = g.y;
+    m_end = g.y + g.z;
+    w += g.x * (p.group_w_stride / sizeof(float));
+  }
+  float* out = p.ws;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
   float acc[4][4] = {};
+  const bool live = m0 + lr < m_end;
+  const int row = live && p.src_row != nullptr ? max(p.src_row[m0 + lr], 0) : m0 + lr;
   for (int k0 = 0; k0 < K; k0 += 16) {
-    const float4 av = m0 + lr < M ? *reinterpret_cast<const float4*>(a + static_cast<size_t>(m0 + lr) * K + k0 + lk) : make_float4(0, 0, 0, 0);
+    const float4 av = live ? *reinterpret_cast<const float4*>(a + static_cast<size_t>(row) * K + k0 + lk) : make_float4(0, 0, 0, 0);
     const float4 wv = *reinterpret_cast<const float4*>(w + static_cast<size_t>(n0 + lr) * K + k0 + lk);   // N is a multiple of 256
     as[lk][lr] = av.x; as[lk + 1][lr] = av.y; as[lk + 2][lr] = av.z; as[lk + 3][lr] = av.w;
     ws[lk][lr] = wv.x; ws[lk + 1][lr] = wv.y; ws[lk + 2][lr] = wv.z; ws[lk + 3][lr] = wv.w;
@@ -389,7 +547,7 @@ __global__ void __launch_bounds__(256) lin_f32_kernel(const float* __restrict__ 
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
-    if (m < M)
+    if (m < m_end)
       *reinterpret_cast<float4*>(out + static_cast<size_t>(m) * N + n0 + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
   }
 }
@@ -400,10 +558,43 @@ __global__ void __launch_bounds__(256) lin_epi_kernel(const __grid_constant__ Li
   const LinEpi& e = p.e;
   const int m = blockIdx.x;
   const float* acc = p.ws + static_cast<size_t>(m) * p.N_pad;
+  int token = m;
+  if (p.group_tiles != nullptr) {                   // padding between the experts' rows: rows of no token
+    token = p.group_rows[m];
+    if (token < 0) return;
+  }
   if (!e.stream) {
-    const float sc = row_rms_scale(e, m, threadIdx.x & 31);
-    for (int n = threadIdx.x; n < e.n_plain; n += 256) e.out[static_cast<size_t>(m) * e.ldo + n] = acc[n] * sc + (e.bias ? e.bias[n] : 0.f);
+    const float sc = row_rms_scale(e, p.src_row != nullptr ? token : m, threadIdx.x & 31);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int g = warp; g < e.lat_tiles * 2; g += 8) {
+      float sq = 0.f;
+      for (int n = g * 128 + lane; n < min(e.lat_n, g * 128 + 128); n += 32) {
+        const float v = acc[n] * sc;
+        sq += v * v;
+        operand_store1(e.lat, m, n, v * e.lat_w[n]);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      if (lane == 0 && g < e.lat_ss_n) e.lat_ss[static_cast<size_t>(m) * e.lat_ss_n + g] = sq;
+    }
+    for (int n = e.lat_tiles * 256 + threadIdx.x; n < e.n_plain; n += 256) {
+      const size_t at = static_cast<size_t>(m) * e.ldo + n;
+      if (e.out_bf16) reinterpret_cast<__nv_bfloat16*>(e.out)[at] = __float2bfloat16(acc[n] * sc);
+      else e.out[at] = stored(e, n, acc[n] * sc);
+    }
     const int tiles = p.N_pad / 256;
+    if (e.act_kind == 2) {
+      for (int i = threadIdx.x; i < min((tiles - e.act_tile0) * kGatedTile, e.act.ld - e.act_k0); i += 256) {
+        const float* t = acc + static_cast<size_t>(e.act_tile0 + i / kGatedTile) * 256;
+        operand_store1(e.act, m, e.act_k0 + i, relu_squared(t[i % kGatedTile] * sc) / (1.f + expf(-t[kGatedTile] * sc)));
+      }
+      return;
+    }
+    if (e.act_kind == 3) {
+      for (int i = threadIdx.x; i < min((tiles - e.act_tile0) * 256, e.act.ld - e.act_k0); i += 256)
+        operand_store1(e.act, m, e.act_k0 + i, gelu(fmaf(acc[e.act_tile0 * 256 + i], sc, e.act_bias ? e.act_bias[i] : 0.f)));
+      return;
+    }
     if (e.act_kind == 1) {
       for (int i = threadIdx.x; i < min((tiles - e.act_tile0) * 256, e.act.ld - e.act_k0); i += 256)
         operand_store1(e.act, m, e.act_k0 + i, relu_squared(acc[e.act_tile0 * 256 + i] * sc));
@@ -415,16 +606,24 @@ __global__ void __launch_bounds__(256) lin_epi_kernel(const __grid_constant__ Li
     }
     return;
   }
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int groups = (e.width + 127) / 128;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = (e.width + 127) / 128;
   for (int g = warp; g < groups; g += 8) {
     float sq = 0.f;
     for (int n = g * 128 + lane; n < min(e.width, g * 128 + 128); n += 32) {
       float* xr = e.x + static_cast<size_t>(m) * e.ldx + n;
-      const float v = (e.add ? *xr : 0.f) + (acc[n] + (e.bias ? e.bias[n] : 0.f));
+      float y = acc[n] + (e.bias ? e.bias[n] : 0.f);
+      if (e.y != nullptr)
+        for (int k = 0; k < e.routes; ++k) {
+          const int r = e.slot_of[m * e.routes + k];
+          if (r < 0) continue;
+          const size_t at = static_cast<size_t>(r) * e.ldy + n;
+          y = fmaf(e.route_w[m * e.routes + k], e.y_f32 ? static_cast<const float*>(e.y)[at] : __bfloat162float(static_cast<const __nv_bfloat16*>(e.y)[at]), y);
+        }
+      const float v = (e.add ? *xr : 0.f) + y;
       *xr = v;
       sq += v * v;
       operand_store1(e.op, m, e.op_k0 + n, e.norm_w ? v * e.norm_w[n] : v);
+      if (e.norm_w2 != nullptr) operand_store1(e.op2, m, n, v * e.norm_w2[n]);
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -448,6 +647,7 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(const __grid_constant
       sq += v * v;
       if (p.x0_k0 >= 0) operand_store1(p.x0, m, p.x0_k0 + n, v);
       operand_store1(p.op, m, p.op_k0 + n, p.norm_w ? v * p.norm_w[n] : v);
+      if (p.norm_w2 != nullptr) operand_store1(p.op2, m, n, v * p.norm_w2[n]);
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -479,17 +679,21 @@ extern "C" int saber_linear_launches(const saber::LinParams* p) { return (p->fp3
 extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t stream) {
   using namespace saber;
   const LinEpi& e = p->e;
-  if (p->M <= 0 || (p->N_pad & 255) || (p->K & 63) || p->K <= 0 || p->M > p->M_pad) return static_cast<int>(cudaErrorInvalidValue);
+  if (p->M <= 0 || (p->N_pad & 255) || (p->K & 63) || p->K <= 0 || (p->M > p->M_pad && p->group_tiles == nullptr)) return static_cast<int>(cudaErrorInvalidValue);
   if (e.stream ? (e.width > p->N_pad || (e.ldx & 31) || e.x == nullptr)
                : (e.n_plain > e.act_tile0 * 256 || e.act_tile0 * 256 > p->N_pad || (e.ldo & 3)))
     return static_cast<int>(cudaErrorInvalidValue);
+  const bool grouped = p->group_tiles != nullptr;
+  if (grouped && (p->group_ntiles == nullptr || p->group_rows == nullptr || p->group_max < 1 || p->splits != 1 || e.stream || p->a2 != nullptr ||
+                  (p->src_row != nullptr && p->src_row != p->group_rows)))
+    return static_cast<int>(cudaErrorInvalidValue);
+  if (!e.stream && (e.lat_tiles > e.act_tile0 || e.lat_n > e.lat_tiles * 256 || (e.out_bf16 && (e.n_plain & 7)))) return static_cast<int>(cudaErrorInvalidValue);
   if (p->fp32) {
-    cudaError_t r = launch(lin_f32_kernel, dim3(p->N_pad / 64, (p->M + 63) / 64), dim3(256), 0, stream, 0, static_cast<const float*>(p->a),
-                           static_cast<const float*>(p->w), p->ws, p->M, p->N_pad, p->K);
+    cudaError_t r = launch(lin_f32_kernel, dim3(p->N_pad / 64, grouped ? p->group_max : (p->M + 63) / 64), dim3(256), 0, stream, 0, *p);
     if (r != cudaSuccess) return static_cast<int>(r);
     return static_cast<int>(launch(lin_epi_kernel, dim3(p->M), dim3(256), 0, stream, 0, *p));
   }
-  if (p->nt < 16 || p->nt > 128 || (p->nt & 15) || (p->M_pad % p->nt) || p->splits < 1) return static_cast<int>(cudaErrorInvalidValue);
+  if (p->nt < 16 || p->nt > 128 || (p->nt & 15) || (p->M_pad % p->nt && !grouped) || p->splits < 1) return static_cast<int>(cudaErrorInvalidValue);
   const int KB = p->K >> 6;
   const int kb_per = (KB + p->splits - 1) / p->splits;
   if ((p->splits - 1) * kb_per >= KB) return static_cast<int>(cudaErrorInvalidValue);
@@ -509,20 +713,25 @@ extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t strea
   if (dev < 0 || dev >= 64) return static_cast<int>(cudaErrorInvalidDevice);
   constexpr int kSmem = 224 * 1024;
   if (!ready[dev]) {
-    cudaError_t r = cudaFuncSetAttribute(lin_bf16_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
-    if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    cudaError_t r = cudaFuncSetAttribute(lin_bf16_kernel<1, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<2, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<1, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
     if (r != cudaSuccess) return static_cast<int>(r);
     ready[dev] = true;
   }
-  const bool pair = p->mtiles == 2 && p->splits == 1 && p->nt == 128 && (p->M_pad / 128) % 2 == 0;
+  const bool pair = !grouped && p->mtiles == 2 && p->splits == 1 && p->nt == 128 && (p->M_pad / 128) % 2 == 0;
   const int abytes = p->nt * 128 * (pair ? 2 : 1);
   int stages = (kSmem - 1024) / (static_cast<int>(kLinTile) + abytes);
   if (stages > kLinMaxStages) stages = kLinMaxStages;
   const int smem = stages * (static_cast<int>(kLinTile) + abytes) + 1024;      // (at least 3 stages: a staged tile of 128 rows fits)
   const int tiles_m = pair ? (p->M + 255) / 256 : (p->M + p->nt - 1) / p->nt;
   const dim3 grid(tiles_m, p->N_pad / 256, p->splits);
-  cudaError_t r = pair ? launch(lin_bf16_kernel<2>, grid, dim3(kLinThreads), smem, stream, 2, q, stages)
-                       : launch(lin_bf16_kernel<1>, grid, dim3(kLinThreads), smem, stream, 2, q, stages);
+  const dim3 ggrid(grouped ? p->group_max : 1, p->N_pad / 256, 1);
+  cudaError_t r = grouped && p->src_row ? launch(lin_bf16_kernel<1, 2>, ggrid, dim3(kLinThreads), smem, stream, 2, q, stages)
+                  : grouped             ? launch(lin_bf16_kernel<1, 1>, ggrid, dim3(kLinThreads), smem, stream, 2, q, stages)
+                  : pair                ? launch(lin_bf16_kernel<2, 0>, grid, dim3(kLinThreads), smem, stream, 2, q, stages)
+                                        : launch(lin_bf16_kernel<1, 0>, grid, dim3(kLinThreads), smem, stream, 2, q, stages);
   if (r != cudaSuccess || p->fuse) return static_cast<int>(r);
   return static_cast<int>(launch(lin_epi_kernel, dim3(p->M), dim3(256), 0, stream, 0, *p));
 }

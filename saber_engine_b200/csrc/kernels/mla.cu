@@ -6,6 +6,7 @@
 // split over CTAs and are merged by the output kernel.
 #include "launch.cuh"
 #include "mla_device.cuh"
+#include "rotary.cuh"
 
 namespace saber {
 
@@ -26,58 +27,41 @@ __global__ void __launch_bounds__(256) mla_prep_kernel(const __grid_constant__ M
   const int m = blockIdx.x;
   if (mla_seq_of_row(p.cu_rows, p.nseq, m) < 0) return;
   const float* x = p.x + static_cast<size_t>(m) * p.ldx;
-  const float pos = static_cast<float>(p.pos[m]);
-  const int half = p.R / 2, LD = p.CP + p.RP;
-  for (int f = threadIdx.x; f < half; f += 256) {
-    float sn, cs;
-    sincosf(pos * p.freq[f], &sn, &cs);
-    rot[f] = cs;
-    rot[half + f] = sn;
-  }
-  const float* d = x + p.dkv_off;
-  float sq = 0.f;
-  for (int i = threadIdx.x; i < p.C; i += 256) sq += d[i] * d[i];
-  sq = mla_warp_sum(sq);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
-  __syncthreads();
-  sq = 0.f;
-  for (int w = 0; w < 8; ++w) sq += red[w];
-  const float r = 1.f / sqrtf(sq / static_cast<float>(p.C) + p.eps);
-  const int slot = p.slot_map[m];
-  if (slot >= 0 && slot < p.n_blocks * p.page) {
-    T* c = static_cast<T*>(p.cache) + static_cast<size_t>(slot) * LD;
-    for (int i = threadIdx.x; i < p.CP; i += 256) c[i] = from_f<T>(i < p.C ? d[i] * r * p.dkv_norm[i] : 0.f);
-    for (int i = threadIdx.x; i < p.RP; i += 256) {
-      float v = 0.f;
-      if (i < p.R) {
-        const int f = i < half ? i : i - half;
-        const float cs = rot[f], sn = rot[half + f];
-        const float a = d[p.C + f], b = d[p.C + f + half];
-        v = i < half ? a * cs - b * sn : b * cs + a * sn;
-      }
-      c[p.CP + i] = from_f<T>(v);
+  const float* qx = p.q + static_cast<size_t>(m) * p.ldq + p.q_off;
+  const int LD = p.CP + p.RP;
+  const bool il = p.interleaved != 0;
+  rotary_table(rot, p.freq, p.R, p.rot_amp, p.pos[m], threadIdx.x, 256);
+  if (p.dkv_off >= 0) {
+    const float* d = x + p.dkv_off;
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < p.C; i += 256) sq += d[i] * d[i];
+    sq = mla_warp_sum(sq);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
+    __syncthreads();
+    sq = 0.f;
+    for (int w = 0; w < 8; ++w) sq += red[w];
+    const float r = 1.f / sqrtf(sq / static_cast<float>(p.C) + p.eps);
+    const int slot = p.slot_map[m];
+    if (slot >= 0 && slot < p.n_blocks * p.page) {
+      T* c = static_cast<T*>(p.cache) + static_cast<size_t>(slot) * LD;
+      for (int i = threadIdx.x; i < p.CP; i += 256) c[i] = from_f<T>(i < p.C ? d[i] * r * p.dkv_norm[i] : 0.f);
+      for (int i = threadIdx.x; i < p.RP; i += 256) c[p.CP + i] = from_f<T>(i < p.R ? rotary_value(d + p.C, i, rot, p.R, il) : 0.f);
+    } else if (slot >= 0 && threadIdx.x == 0 && p.err) {
+      atomicCAS(p.err, 0u, static_cast<uint32_t>(kErrBadIndex));
     }
-  } else if (slot >= 0 && threadIdx.x == 0 && p.err) {
-    atomicCAS(p.err, 0u, static_cast<uint32_t>(kErrBadIndex));
+  } else {
+    __syncthreads();
   }
   const int KP = p.expand ? p.DP : p.CP;
   T* q = static_cast<T*>(p.q_eff) + static_cast<size_t>(m) * p.H * (KP + p.RP);
   for (int i = threadIdx.x; i < p.H * p.RP; i += 256) {
     const int h = i / p.RP, k = i - h * p.RP;
-    float v = 0.f;
-    if (k < p.R) {
-      const int f = k < half ? k : k - half;
-      const float cs = rot[f], sn = rot[half + f];
-      const float* qr = x + p.q_off + h * (p.D + p.R) + p.D;
-      const float a = qr[f], b = qr[f + half];
-      v = k < half ? a * cs - b * sn : b * cs + a * sn;
-    }
-    q[static_cast<size_t>(h) * (KP + p.RP) + KP + k] = from_f<T>(v);
+    q[static_cast<size_t>(h) * (KP + p.RP) + KP + k] = from_f<T>(k < p.R ? rotary_value(qx + h * (p.D + p.R) + p.D, k, rot, p.R, il) : 0.f);
   }
   if (p.expand)
     for (int i = threadIdx.x; i < p.H * p.DP; i += 256) {
       const int h = i / p.DP, k = i - h * p.DP;
-      q[static_cast<size_t>(h) * (KP + p.RP) + k] = from_f<T>(k < p.D ? x[p.q_off + h * (p.D + p.R) + k] : 0.f);
+      q[static_cast<size_t>(h) * (KP + p.RP) + k] = from_f<T>(k < p.D ? qx[h * (p.D + p.R) + k] : 0.f);
     }
 }
 
@@ -101,7 +85,7 @@ __global__ void __launch_bounds__(256) mla_absorb_kernel(const __grid_constant__
   const int h = blockIdx.y, mb = blockIdx.z * 8, rows = min(8, p.M - mb);
   for (int i = threadIdx.x; i < p.D * 8; i += 256) {
     const int r = i / p.D, d = i - r * p.D;
-    sm[d * 8 + r] = r < rows ? p.x[static_cast<size_t>(mb + r) * p.ldx + p.q_off + h * (p.D + p.R) + d] : 0.f;
+    sm[d * 8 + r] = r < rows ? p.q[static_cast<size_t>(mb + r) * p.ldq + p.q_off + h * (p.D + p.R) + d] : 0.f;
   }
   __syncthreads();
   const int cp = threadIdx.x & 63, quarter = threadIdx.x >> 6;
@@ -270,7 +254,7 @@ __global__ void __launch_bounds__(256) mla_out_kernel(const __grid_constant__ Ml
       float y = s[0];
 #pragma unroll
       for (int r = 1; r < 8; ++r) y = lane == r ? s[r] : y;
-      const float g = p.x[static_cast<size_t>(mb + lane) * p.ldx + p.g_off + h * p.V + v];
+      const float g = mla_gate(p, mb + lane, h, v);
       operand_store1(p.out, mb + lane, p.out_k0 + h * p.V + v, y / (1.f + expf(-g)));
     }
   }
@@ -302,7 +286,7 @@ extern "C" int saber_mla_launches(const saber::MlaParams* p) { return p->expand 
 extern "C" int saber_mla_launch(const saber::MlaParams* p, cudaStream_t stream) {
   using namespace saber;
   if (p->M <= 0 || p->C > p->CP || p->R > p->RP || (p->R & 1) || p->CP > 128 * kRowMaxC || p->D > 1024 || p->splits < 1 || p->splits > 64 ||
-      p->q_eff == nullptr || p->cache == nullptr)
+      p->q_eff == nullptr || p->cache == nullptr || p->q == nullptr)
     return static_cast<int>(cudaErrorInvalidValue);
   if (p->expand ? (p->k_exp == nullptr || p->v_exp == nullptr || saber_mla_expand_ok(p) < p->expand) : (p->o_part == nullptr || p->ml == nullptr))
     return static_cast<int>(cudaErrorInvalidValue);

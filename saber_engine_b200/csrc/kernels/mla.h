@@ -10,7 +10,12 @@ namespace saber {
 
 struct MlaParams {
   const float* x;             // [M][ldx] projections of this step's rows
-  int ldx, q_off, dkv_off, g_off;
+  int ldx, q_off, dkv_off, g_off;   // dkv_off < 0: the cache is another layer's, nothing is appended
+  const float* q;             // [M][ldq] queries (column q_off on)
+  int ldq;
+  int gate_heads;             // 1: one gate per head (column g_off + h), 0: one per value (g_off + h V + v)
+  int interleaved;            // layout of a rotated pair (rotary.cuh)
+  float rot_amp;
   const float* dkv_norm;      // [C]
   const float* freq;          // [R / 2] rotary frequencies
   const void* w_uk;           // [H * D][CP] (pads zero)

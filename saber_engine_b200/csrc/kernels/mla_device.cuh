@@ -22,6 +22,9 @@ __device__ __forceinline__ int mla_seq_of_row(const int32_t* cu, int nseq, int m
     if (m < cu[j + 1]) return m >= cu[j] ? j : -1;
   return -1;
 }
+__device__ __forceinline__ float mla_gate(const MlaParams& p, int m, int h, int v) {
+  return p.x[static_cast<size_t>(m) * p.ldx + p.g_off + (p.gate_heads ? h : h * p.V + v)];
+}
 // physical page of the i-th page of sequence j (bounds-checked: an entry outside the pool is recorded and read as page 0)
 template <typename Params>
 __device__ __forceinline__ int page_at(const Params& p, int j, int i) {

@@ -522,13 +522,12 @@ __global__ void __launch_bounds__(256) mla_flash_kernel(const __grid_constant__ 
     const int rr = row + r * 8;
     if (rr >= rows) continue;
     const float inv = 1.f / l[r];
-    const float* g = p.x + static_cast<size_t>(m0 + rr) * p.ldx + p.g_off + h * p.V;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int v = i * 8 + (lane & 3) * 2;
 #pragma unroll
       for (int e = 0; e < 2; ++e)
-        if (v + e < p.V) operand_store1(p.out, m0 + rr, p.out_k0 + h * p.V + v + e, o[i][r * 2 + e] * inv / (1.f + expf(-g[v + e])));
+        if (v + e < p.V) operand_store1(p.out, m0 + rr, p.out_k0 + h * p.V + v + e, o[i][r * 2 + e] * inv / (1.f + expf(-mla_gate(p, m0 + rr, h, v + e))));
     }
   }
 }
@@ -559,6 +558,7 @@ static int flash_go(const MlaParams& p, cudaStream_t stream) {
     f.v_stride = static_cast<size_t>(p.VP) * 128;
     f.gate = p.x + p.g_off;
     f.ldg = p.ldx;
+    f.gate_heads = p.gate_heads;
     f.cu_rows = p.cu_rows;
     f.kv_len = p.kv_len;
     f.block_table = p.block_table;

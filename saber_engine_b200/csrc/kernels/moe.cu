@@ -18,61 +18,92 @@ constexpr int kMoeTpMaxTiles = kTpMaxTiles;   // same flag regions as the row-pa
 
 __device__ __forceinline__ float e_safe(float x, float mx) { return x == -INFINITY ? 0.f : __expf(x - mx); }
 
-// grid = ceil(M / 8), block 256: one warp per token.
-__global__ void __launch_bounds__(256) moe_topk_kernel(const MoeRouteParams p) {
-  pdl_wait();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int m = blockIdx.x * 8 + warp;
-  if (m >= p.M) return;
-  constexpr int kPerLane = 32;                 // up to 1024 experts
-  float v[kPerLane];
-  const int per = (p.E + 31) / 32;
+// The routes of token m, by one warp; kPer * 32 experts at most.  add(expert) counts a route of a local expert.
+template <int kPer, typename Add>
+__device__ __forceinline__ void moe_topk_row(const MoeRouteParams& p, int m, int lane, const Add& add) {
+  if (p.live != nullptr && m >= *p.live) {
+    for (int k = lane; k < p.top_k; k += 32) {
+      p.topk_id[m * p.top_k + k] = -1;
+      p.topk_w[m * p.top_k + k] = 0.f;
+    }
+    return;
+  }
+  float v[kPer];
   float mx = -INFINITY;
-  for (int i = 0; i < per; ++i) {
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
     const int e = i * 32 + lane;
-    v[i] = e < p.E ? __bfloat162float(p.logits[static_cast<size_t>(m) * p.ld + e]) : -INFINITY;
+    const size_t at = static_cast<size_t>(m) * p.ld + e;
+    v[i] = e >= p.E ? -INFINITY : p.logits_f32 != nullptr ? p.logits_f32[at] : __bfloat162float(p.logits[at]);
     mx = fmaxf(mx, v[i]);
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   float sum = 0.f;
-  for (int i = 0; i < per; ++i) {
-    v[i] = e_safe(v[i], mx);
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
+    v[i] = v[i] == -INFINITY ? 0.f : p.logits_f32 != nullptr ? expf(v[i] - mx) : e_safe(v[i], mx);
     sum += v[i];
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-  const float inv = 1.f / sum;
-  float picked_w[kMoeMaxTopK];
-  int picked_e[kMoeMaxTopK];
-  float wsum = 0.f;
-  for (int k = 0; k < p.top_k; ++k) {
-    float bv = -1.f;
-    int be = p.E;
-    for (int i = 0; i < per; ++i) {
-      const int e = i * 32 + lane;
-      if (v[i] > bv) { bv = v[i]; be = e; }     // ascending e per lane: the lower id wins ties
-    }
+  uint32_t open = kPer == 32 ? 0xffffffffu : (1u << kPer) - 1u;     // bit i: expert i * 32 + lane may be chosen
+  auto best = [&](uint32_t among, float& bv, int& be) {             // largest score, the lower id wins ties
+    bv = -1.f;
+    be = p.E;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i)
+      if ((among >> i & 1u) && i * 32 + lane < p.E && v[i] > bv) { bv = v[i]; be = i * 32 + lane; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
       const int oe = __shfl_xor_sync(0xffffffffu, be, o);
       if (ov > bv || (ov == bv && oe < be)) { bv = ov; be = oe; }
     }
-    picked_w[k] = bv * inv;
-    picked_e[k] = be;
-    wsum += picked_w[k];
-    if ((be & 31) == lane) v[be >> 5] = -1.f;   // taken
-  }
-  if (lane == 0) {
-    const float rn = p.norm_topk ? 1.f / wsum : 1.f;
-    for (int k = 0; k < p.top_k; ++k) {
-      p.topk_id[m * p.top_k + k] = picked_e[k];
-      p.topk_w[m * p.top_k + k] = picked_w[k] * rn;
-      const int le = picked_e[k] - p.e_lo;
-      if (le >= 0 && le < p.e_n) atomicAdd(p.counts + le, 1);
+  };
+  if (p.groups > 1 && p.keep < p.groups) {
+    // the best expert outside the groups kept so far names the next group to keep
+    const int size = p.E / p.groups;
+    uint32_t kept = 0u;
+    for (int k = 0; k < p.keep; ++k) {
+      float bv;
+      int be;
+      best(~kept, bv, be);
+      if (be >= p.E) break;                         // (scores that are no numbers)
+      const int lo = be / size * size;
+#pragma unroll
+      for (int i = 0; i < kPer; ++i) {
+        const int e = i * 32 + lane;
+        if (e >= lo && e < lo + size) kept |= 1u << i;
+      }
     }
+    open = kept;
   }
+  float wsum = 0.f, mine_w = 0.f;
+  int mine_e = -1;                                  // lane k holds route k
+  for (int k = 0; k < p.top_k; ++k) {
+    float bv;
+    int be;
+    best(open, bv, be);
+    if (be >= p.E) break;
+    wsum += bv;
+    if (lane == k) { mine_w = bv; mine_e = be; }
+    if ((be & 31) == lane) open &= ~(1u << (be >> 5));
+  }
+  if (lane < p.top_k) {
+    p.topk_id[m * p.top_k + lane] = mine_e;
+    p.topk_w[m * p.top_k + lane] = mine_w / (p.norm_topk ? wsum : sum);
+    const int le = mine_e - p.e_lo;
+    if (mine_e >= 0 && le >= 0 && le < p.e_n) add(le);
+  }
+}
+
+// grid = ceil(M / 8), block 256: one warp per token.
+template <int kPer>
+__global__ void __launch_bounds__(256) moe_topk_kernel(const MoeRouteParams p) {
+  pdl_wait();
+  const int m = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (m < p.M) moe_topk_row<kPer>(p, m, threadIdx.x & 31, [&](int e) { atomicAdd(p.counts + e, 1); });
 }
 
 // One block of 1024 threads (one per local expert): exclusive scans of the padded row counts and of
@@ -126,13 +157,46 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const MoeRouteParams p) 
   for (int i = t; i < p.rows_cap; i += blockDim.x) p.src_row[i] = -1;
 }
 
+// One block for a few tokens: scores, plan and placement in one launch.
+template <int kPer>
+__global__ void __launch_bounds__(1024) moe_route_few_kernel(const MoeRouteParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ int warp_tot[32], counts[1024], at[1024];
+  const int t = threadIdx.x;
+  counts[t] = 0;
+  for (int i = t; i < p.rows_cap; i += 1024) p.src_row[i] = -1;
+  __syncthreads();
+  for (int m = t >> 5; m < p.M; m += 32) moe_topk_row<kPer>(p, m, t & 31, [&](int e) { atomicAdd(counts + e, 1); });
+  __syncthreads();
+  const int c = counts[t];
+  int rows_total, tiles_total;
+  const int off = block_excl_scan_1024((c + 15) & ~15, warp_tot, rows_total);
+  const int toff = block_excl_scan_1024((c + p.nt - 1) / p.nt, warp_tot, tiles_total);
+  at[t] = off;
+  int i = toff;
+  for (int r = 0; r < c; r += p.nt) p.tiles[i++] = make_int4(t, off + r, min(p.nt, c - r), 0);
+  if (t == 0) {
+    p.ntiles[0] = tiles_total;
+    p.ntiles[1] = rows_total;
+  }
+  __syncthreads();
+  for (int r = t; r < p.M * p.top_k; r += 1024) {
+    const int le = p.topk_id[r] - p.e_lo;
+    const bool mine = p.topk_id[r] >= 0 && le >= 0 && le < p.e_n;
+    const int pos = mine ? atomicAdd(at + le, 1) : -1;
+    p.slot_of[r] = pos;
+    if (mine) p.src_row[pos] = r / p.top_k;
+  }
+}
+
 // thread per route: claim a row in the expert's segment.
 __global__ void moe_place_kernel(const MoeRouteParams p) {
   pdl_wait();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= p.M * p.top_k) return;
   const int le = p.topk_id[i] - p.e_lo;
-  if (le < 0 || le >= p.e_n) { p.slot_of[i] = -1; return; }
+  if (p.topk_id[i] < 0 || le < 0 || le >= p.e_n) { p.slot_of[i] = -1; return; }
   const int pos = p.offsets[le] + atomicAdd(p.cursors + le, 1);
   p.slot_of[i] = pos;
   p.src_row[pos] = i / p.top_k;
@@ -241,14 +305,28 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const MoeCombineParams
 
 }  // namespace saber
 
+namespace saber {
+static bool moe_few(const MoeRouteParams& p) { return p.logits_f32 != nullptr && p.M <= 64; }
+
+template <int kPer>
+static int moe_route_go(const MoeRouteParams& p, cudaStream_t stream) {
+  if (moe_few(p)) return static_cast<int>(launch(moe_route_few_kernel<kPer>, dim3(1), dim3(1024), 0, stream, 2, p));
+  launch(moe_topk_kernel<kPer>, dim3((p.M + 7) / 8), dim3(256), 0, stream, 0, p);
+  launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, 0, p);
+  launch(moe_place_kernel, dim3((p.M * p.top_k + 255) / 256), dim3(256), 0, stream, 0, p);
+  return static_cast<int>(cudaGetLastError());
+}
+}  // namespace saber
+
+extern "C" int saber_moe_route_launches(const saber::MoeRouteParams* p) { return saber::moe_few(*p) ? 1 : 3; }
+
 extern "C" int saber_moe_route_launch(const saber::MoeRouteParams* p, cudaStream_t stream) {
   using namespace saber;
-  if (p->E > 1024 || p->e_n > 1024 || p->top_k > kMoeMaxTopK || p->top_k < 1 || p->nt < 16 || (p->nt & 15))
+  if (p->E < 1 || p->E > 1024 || p->e_n > 1024 || p->top_k > kMoeMaxTopK || p->top_k < 1 || p->nt < 16 || (p->nt & 15) ||
+      (p->groups > 1 && (p->E % p->groups || p->keep < 1 || p->keep * (p->E / p->groups) < p->top_k)))
     return static_cast<int>(cudaErrorInvalidValue);
-  saber::launch(moe_topk_kernel, dim3((p->M + 7) / 8), dim3(256), 0, stream, 0, *p);
-  saber::launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, 0, *p);
-  saber::launch(moe_place_kernel, dim3((p->M * p->top_k + 255) / 256), dim3(256), 0, stream, 0, *p);
-  return static_cast<int>(cudaGetLastError());
+  const int per = (p->E + 31) / 32;
+  return per <= 1 ? moe_route_go<1>(*p, stream) : per <= 4 ? moe_route_go<4>(*p, stream) : per <= 16 ? moe_route_go<16>(*p, stream) : moe_route_go<32>(*p, stream);
 }
 
 extern "C" int saber_moe_gather_launch(const int8_t* q, const float* scale, int M_pad, const int32_t* src_row,

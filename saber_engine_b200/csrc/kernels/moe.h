@@ -6,7 +6,7 @@
 
 namespace saber {
 
-constexpr int kMoeMaxTopK = 16;
+constexpr int kMoeMaxTopK = 32;
 
 struct MoeRouteParams {
   const __nv_bfloat16* logits;   // [M][ld] router logits
@@ -22,6 +22,10 @@ struct MoeRouteParams {
   int M, ld, E, top_k, nt, rows_cap;
   int e_lo, e_n;                 // this rank's experts are [e_lo, e_lo + e_n)
   int norm_topk;
+  // fp32 logits (instead of `logits`), softmax with the accurate exponential
+  const float* logits_f32;
+  const int32_t* live;           // rows from *live on are padding and take no route (null: every row is live)
+  int groups, keep;              // groups > 1: only experts of the `keep` groups of neighbours whose best score is best
 };
 
 struct MoeCombineParams {
@@ -47,5 +51,6 @@ struct MoeCombineParams {
 extern "C" int saber_moe_gather_launch(const int8_t* q, const float* scale, int M_pad, const int32_t* src_row,
                                        const int32_t* ntiles, int8_t* q_out, float* scale_out, int rows_cap,
                                        int M_pad_out, int K, int to_fp8, cudaStream_t stream);
+extern "C" int saber_moe_route_launches(const saber::MoeRouteParams* p);
 extern "C" int saber_moe_route_launch(const saber::MoeRouteParams* p, cudaStream_t stream);
 extern "C" int saber_moe_combine_launch(const saber::MoeCombineParams* p, cudaStream_t stream);

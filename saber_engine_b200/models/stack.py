@@ -3,10 +3,12 @@
 The residual stream stays fp32; a linear that ends a sublayer adds its result to it and leaves the next linear's operand
 (norm weight times x) with the row's partial sums of squares, so that no normalisation, activation or addition needs a
 launch of its own.
-  parallel    x <- x + mixer(norm(x)) + ff(norm(x)): two linears around the mixer's kernels
+  parallel    x <- x + mixer(norm(x)) + ff(norm(x)): two linears around the mixer's kernels.  Two norms: the same, the rows of the
+              feed-forward multiply a second operand
   sequential  x <- x + mixer(norm1(x)); x <- x + ff(norm2(x)): two linears around the mixer, two for the feed-forward
-Launches of a mixer in decoding: delta rule 1, decayed outer products 1, grouped-query attention 1, latent attention 4;
-a pass of a looped block adds one linear.
+Launches of a mixer in decoding: delta rule 1, decayed outer products 1, grouped-query attention 1, latent attention 5 (6 where
+queries come from a latent of their own); a pass of a looped block adds one linear, routed experts add 3 (routing and two grouped
+products: the output linear's epilogue adds the experts' rows to the stream).
 
 Every row of every bucket is committed (no drafter): a decode bucket is one row per sequence, a prefill bucket
 is `width` ragged rows of up to `nseq` sequences, single decoded tokens beside portions of prompts included.
@@ -24,7 +26,7 @@ from ..ops import functional as F
 from ..ops import layouts as L
 from ..ops import native as N
 from . import stack_weights as SW
-from .stack_config import DeltaMixer, GroupedMixer, LatentMixer, OuterMixer, StackConfig
+from .stack_config import DeltaMixer, ExpertMix, GroupedMixer, LatentMixer, OuterMixer, StackConfig
 from .step import BlobLayout, Bucket, finish_bucket, head_outputs, plp_outputs, seam_outputs
 
 
@@ -61,7 +63,8 @@ class StackModel:
         for r in cfg.runs:
             m = cfg.layers[r.layer].mixer
             if isinstance(m, LatentMixer):
-                self.kv[r.index] = torch.zeros(self.kv_blocks, cfg.page_tokens, m.rank_pad + m.rot_pad, dtype=dtype, device=dev)
+                if m.kv_from is None:
+                    self.kv[r.index] = torch.zeros(self.kv_blocks, cfg.page_tokens, m.rank_pad + m.rot_pad, dtype=dtype, device=dev)
             elif isinstance(m, GroupedMixer):
                 if m.kv_from is None:                     # the padding of a page stays zero: the kernels multiply it
                     self.kv[r.index] = torch.zeros(self.kv_blocks, m.kv_heads, cfg.page_tokens * (m.key_pad + m.vdim_pad), dtype=dtype, device=dev)
@@ -112,8 +115,12 @@ class StackModel:
         """Zeroed storage of a [M, K] operand: padding rows and columns stay zero."""
         return torch.zeros(L.padded_rows(M) * L.round_up(K, 64), dtype=self.dtype, device=self.device)
 
-    def _linear(self, prog: N.Program, lin: SW.Linear, a: torch.Tensor, M: int, e: N.LinEpi, ws: Optional[torch.Tensor], tag: str) -> None:
+    def _linear(self, prog: N.Program, lin: SW.Linear, a: torch.Tensor, M: int, e: N.LinEpi, ws: Optional[torch.Tensor], tag: str,
+                second: Optional[tuple] = None) -> None:
+        """second: (operand, first weight tile that reads it)."""
         p = N.LinParams()
+        if second is not None:
+            p.a2, p.a2_tile0 = second[0].data_ptr(), second[1]
         sc = self.scratch
         p.w, p.a, p.err = lin.w.data_ptr(), a.data_ptr(), sc.err.data_ptr()
         p.ws, p.counters = (ws if ws is not None else sc.ws).data_ptr(), sc.counters.data_ptr()
@@ -126,15 +133,32 @@ class StackModel:
         p.e = e
         prog.linear(p, tag=tag)
 
+    def _grouped_linear(self, prog: N.Program, lin: SW.Linear, a: torch.Tensor, a_rows: int, ew: dict, gather: bool, e: N.LinEpi,
+                        ws: Optional[torch.Tensor], tag: str) -> None:
+        """The routed rows of a step against the stack of experts.  gather: the operand's rows are tokens."""
+        p, sc = N.LinParams(), self.scratch
+        p.w, p.a, p.err, p.counters = lin.w.data_ptr(), a.data_ptr(), sc.err.data_ptr(), sc.counters.data_ptr()
+        p.ws = (ws if ws is not None else sc.ws).data_ptr()
+        p.M, p.M_pad, p.N_pad, p.K, p.splits, p.mtiles = ew["rows"], a_rows, lin.N_pad, lin.K, 1, 1
+        p.nt, p.fp32, p.fuse = ew["nt"], int(self.f32), int(self.fuse)
+        p.group_tiles, p.group_ntiles, p.group_rows, p.group_max = (*(ew[k].data_ptr() for k in ("tiles", "ntiles", "src_row")), ew["max_tiles"])
+        p.src_row = ew["src_row"].data_ptr() if gather else None
+        p.group_w_stride = lin.N_pad * lin.K * lin.w.element_size() if self.f32 else lin.N_pad * lin.K * 2
+        p.e = e
+        prog.linear(p, tag=tag)
+
     def _row_norm(self, e: N.LinEpi, ss: torch.Tensor) -> None:
         """The operand's rows were left undivided: scale the product by the row's reciprocal root mean square."""
         e.ss, e.ss_n = ss.data_ptr(), ss.shape[1]
         e.inv_width, e.eps = 1.0 / self.cfg.width, self.cfg.eps
 
     def _stream_epi(self, x: torch.Tensor, add: bool, target: tuple, bias: Optional[torch.Tensor] = None) -> N.LinEpi:
-        """target: (operand, first column, norm weight or None, sums of squares or None) of the next linear."""
+        """target: (operand, first column, norm weight or None, sums of squares or None) of the next linear, and the same stream's
+        second operand with its norm weight (or None)."""
         e = N.LinEpi()
-        op, k0, norm_w, ss = target
+        op, k0, norm_w, ss, op2, norm_w2 = target
+        if norm_w2 is not None:
+            e.op2, e.norm_w2 = op2, norm_w2.data_ptr()
         e.stream, e.x, e.ldx, e.width, e.add = 1, x.data_ptr(), x.stride(0), self.cfg.width, int(add)
         e.bias, e.norm_w = N.ptr(bias), N.ptr(norm_w)
         e.op, e.op_k0 = op, k0
@@ -170,33 +194,39 @@ class StackModel:
         x = f32(M, L.round_up(W, 32))
         ss = f32(L.padded_rows(M), (W + 127) // 128)
         h = self._operand_buf(M, KW)
+        h2 = self._operand_buf(M, KW) if cfg.two_norms else None
         loop_op = self._operand_buf(M, 2 * KW) if cfg.loop is not None else None
         mid = self._operand_buf(M, max(l.out.K for l in w.layers))
         ups = [l for l in w.layers if l.up is not None]
         ff = self._operand_buf(M, max(l.down.K for l in ups)) if ups else None
         ldp = max(L.round_up(l.n_plain, 8) for l in w.layers)
         proj = f32(M, ldp)
-        big = max([x.N_pad for l in w.layers for x in (l.proj, l.out, l.up) if x is not None] + [w.head.N_pad])
+        work = self._mixer_scratch(M, nseq, decode)
+        experts = self._expert_scratch(M)
+        big = max([x.N_pad for l in w.layers for x in (l.proj, l.out, l.up, l.carry) if x is not None] + [w.head.N_pad]) * M
+        if experts:
+            big = max([big] + [x.N_pad * experts["rows"] for l in w.layers for x in (l.experts_up, l.experts_down) if x is not None])
         ws = None
         if self.f32 or not self.fuse:                    # product rows (and, behind them, the split parts)
-            ws = torch.empty(M * big + (0 if self.f32 else self.scratch.capacity // 4), dtype=torch.float32, device=dev)
-        work = self._mixer_scratch(M, nseq, decode)
-        keep = [blob, x, ss, h, loop_op, mid, ff, proj, ws, work]
+            ws = torch.empty(big + (0 if self.f32 else self.scratch.capacity // 4), dtype=torch.float32, device=dev)
+        keep = [blob, x, ss, h, h2, loop_op, mid, ff, proj, ws, work, experts]
         digests = None
         if self.race_check == "shadow":
             digests = torch.zeros(len(cfg.runs) + 1, dtype=torch.int64, device=dev)
             prog.digest_clear(digests, len(cfg.runs) + 1, tag="digest.clear")
 
         h_op = self._operand(h, M, KW)
+        h2_op = self._operand(h2, M, KW) if h2 is not None else None
         l_op = self._operand(loop_op, M, 2 * KW) if loop_op is not None else None
 
         def target(run) -> tuple:
             """What the linear ahead of a run (None: ahead of the head) leaves for it."""
             if run is None:
-                return h_op, 0, w.final_norm, ss
+                return h_op, 0, w.final_norm, ss, None, None
             if run.enter is not None:
-                return l_op, 0, None, None
-            return h_op, 0, w.layers[run.layer].norm, ss
+                return l_op, 0, None, None, None, None
+            lw = w.layers[run.layer]
+            return h_op, 0, lw.norm, ss, h2_op, lw.norm2 if cfg.two_norms else None
 
         # ---- embedding
         runs = cfg.runs
@@ -206,8 +236,10 @@ class StackModel:
         ep.x0_k0 = -1
         if loop_op is not None:
             ep.x0, ep.x0_k0 = l_op, KW
-        op, k0, norm_w, s0 = target(runs[0])
+        op, k0, norm_w, s0, op2, norm_w2 = target(runs[0])
         ep.op, ep.op_k0, ep.norm_w = op, k0, N.ptr(norm_w)
+        if norm_w2 is not None:
+            ep.op2, ep.norm_w2 = op2, norm_w2.data_ptr()
         ep.ss_out, ep.ss_out_n = N.ptr(s0), ss.shape[1]
         prog.stream_embed(ep, tag="embed")
 
@@ -215,7 +247,7 @@ class StackModel:
         for i, run in enumerate(runs):
             lw, spec, t = w.layers[run.layer], cfg.layers[run.layer], f"R{run.index}.L{run.layer}"
             if run.enter is not None:                    # x <- W_in [x; x0] + step
-                e = self._stream_epi(x, False, (h_op, 0, lw.norm, ss), bias=w.loop_step[run.enter])
+                e = self._stream_epi(x, False, (h_op, 0, lw.norm, ss, None, None), bias=w.loop_step[run.enter])
                 self._linear(prog, w.loop_in, loop_op, M, e, ws, f"{t}.loop_in")
             m_op = self._operand(mid, M, lw.out.K)
             e = N.LinEpi()
@@ -223,8 +255,16 @@ class StackModel:
             e.out, e.ldo, e.n_plain, e.act_tile0 = proj.data_ptr(), ldp, lw.n_plain, lw.act_tile0
             e.bias = N.ptr(lw.bias)
             if spec.mlp is not None and cfg.parallel:
-                e.act, e.act_k0, e.limit, e.alpha = m_op, lw.act_k0, spec.mlp.limit, spec.mlp.alpha
-            self._linear(prog, lw.proj, h, M, e, ws, f"{t}.project")
+                e.act, e.act_k0, e.act_kind, e.limit, e.alpha = m_op, lw.act_k0, spec.mlp.act_kind, spec.mlp.limit, spec.mlp.alpha
+                e.act_bias = N.ptr(lw.act_bias)
+            if lw.lat_tiles:
+                e.lat_tiles, e.lat_n, e.lat, e.lat_w = lw.lat_tiles, spec.mixer.q_rank, self._operand(work["lat"], M, lw.carry.K), lw.extra["dq_norm"].data_ptr()
+                e.lat_ss, e.lat_ss_n = work["lat_ss"].data_ptr(), 2 * lw.lat_tiles
+            self._linear(prog, lw.proj, h, M, e, ws, f"{t}.project", second=(h2, lw.tile2) if cfg.two_norms and spec.mlp is not None else None)
+            if lw.experts_up is not None:
+                self._experts(prog, lw, spec.mlp, h2, ss, proj, M, at(lay.cu_rows + nseq), experts, ws, t)
+            if lw.carry is not None:
+                self._carry_queries(prog, lw, spec.mixer, work, M, ws, f"{t}.carry")
             if isinstance(spec.mixer, DeltaMixer):
                 prog.delta(self._delta_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work), decode, tag=f"{t}.delta")
             elif isinstance(spec.mixer, OuterMixer):
@@ -236,9 +276,13 @@ class StackModel:
             nxt = runs[i + 1] if i + 1 < len(runs) else None
             tgt = target(nxt)
             if lw.up is None:
-                self._linear(prog, lw.out, mid, M, self._stream_epi(x, True, tgt), ws, f"{t}.out")
+                e = self._stream_epi(x, True, tgt, bias=lw.out_bias)
+                if lw.experts_up is not None:
+                    e.y, e.slot_of, e.route_w = (experts[k].data_ptr() for k in ("y", "slot_of", "topk_w"))
+                    e.routes, e.ldy, e.y_f32 = spec.mlp.top, L.round_up(W, 8), int(self.f32)
+                self._linear(prog, lw.out, mid, M, e, ws, f"{t}.out")
             else:
-                self._linear(prog, lw.out, mid, M, self._stream_epi(x, True, (h_op, 0, lw.norm2, ss)), ws, f"{t}.out")
+                self._linear(prog, lw.out, mid, M, self._stream_epi(x, True, (h_op, 0, lw.norm2, ss, None, None)), ws, f"{t}.out")
                 e = N.LinEpi()
                 self._row_norm(e, ss)
                 e.act, e.act_kind = self._operand(ff, M, lw.down.K), 1         # (squared ReLU)
@@ -247,11 +291,53 @@ class StackModel:
             if digests is not None:
                 prog.digest(x, x.numel() * 4, digests.data_ptr() + 8 * run.index, tag=f"{t}.digest")
         b = self._head(prog, key, kind, nseq, width, M, lay, at, blob, blob_host, x, h, ss, ws, keep + [digests], seam, plp, capture)
-        b.arenas = [a for a in (x, ss, h, loop_op, mid, ff, proj) if a is not None]
+        b.arenas = [a for a in (x, ss, h, h2, loop_op, mid, ff, proj) if a is not None]
         b.digests, b.x = digests, x
         return b
 
+    # ---- routed experts
+    def _expert_scratch(self, M: int) -> dict:
+        """Routing tables and routed rows of a bucket, sized for the largest mixture.  Every expert's rows start at a multiple of 16."""
+        ms = [l.mlp for l in self.cfg.layers if isinstance(l.mlp, ExpertMix)]
+        if not ms:
+            return {}
+        dev, W = self.device, self.cfg.width
+        i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=dev)       # noqa: E731
+        nt = 64 if self.f32 else L.token_tile(M)
+        per = [(M * f.top, min(f.experts, M * f.top)) for f in ms]            # routes, experts that can have one
+        rows = L.round_up(max(r + 15 * e for r, e in per), 16)
+        pad = rows + 128                                                      # (a tile's copies may run past the live rows)
+        top, E, ff = max(f.top for f in ms), max(f.experts for f in ms), max(L.round_up(f.ff, 64) for f in ms)
+        return {"nt": nt, "rows": rows, "pad": pad, "max_tiles": max(e + r // nt for r, e in per), "tiles": i32(max(e + r // nt for r, e in per), 4),
+                "ntiles": i32(2), "src_row": i32(pad), "topk_id": i32(M * top), "slot_of": i32(M * top), "counts": i32(E), "offsets": i32(E + 1), "cursors": i32(E),
+                "topk_w": torch.zeros(M * top, dtype=torch.float32, device=dev), "act": torch.zeros(pad * ff, dtype=self.dtype, device=dev),
+                "y": torch.zeros(rows * L.round_up(W, 8), dtype=self.dtype, device=dev)}
+
+    def _experts(self, prog, lw, f: ExpertMix, h2, ss, proj, M: int, live, ew: dict, ws, tag: str) -> None:
+        """Routes of the step, then the experts' rows; their weighted sum is left to the output linear."""
+        p = N.MoeRouteParams()
+        p.logits_f32, p.ld, p.M, p.E, p.top_k = proj.data_ptr() + 4 * lw.off["router"], proj.stride(0), M, f.experts, f.top
+        p.topk_id, p.topk_w, p.counts, p.offsets, p.cursors, p.tiles, p.ntiles, p.src_row, p.slot_of = \
+            (ew[k].data_ptr() for k in ("topk_id", "topk_w", "counts", "offsets", "cursors", "tiles", "ntiles", "src_row", "slot_of"))
+        p.nt, p.rows_cap, p.e_lo, p.e_n, p.live, p.groups, p.keep = ew["nt"], ew["src_row"].numel(), 0, f.experts, live, f.groups, f.keep
+        prog.add_moe_route(p, tag=f"{tag}.route")
+        e = N.LinEpi()
+        self._row_norm(e, ss)
+        e.act, e.act_kind = N.Operand(ew["act"].data_ptr(), ew["pad"], lw.experts_down.K, int(self.f32)), 1
+        self._grouped_linear(prog, lw.experts_up, h2, L.padded_rows(M), ew, True, e, ws, f"{tag}.experts_up")
+        e = N.LinEpi()
+        e.out, e.ldo, e.n_plain, e.act_tile0 = ew["y"].data_ptr(), L.round_up(self.cfg.width, 8), L.round_up(self.cfg.width, 8), lw.experts_down.N_pad // 256
+        e.out_bf16 = int(not self.f32)
+        self._grouped_linear(prog, lw.experts_down, ew["act"], ew["pad"], ew, False, e, ws, f"{tag}.experts_down")
+
     # ---- mixers
+    def _carry_queries(self, prog, lw, m: LatentMixer, wk: dict, M: int, ws, tag: str) -> None:
+        """Queries from their normed latent (its rows were left undivided, like the stream's)."""
+        e = N.LinEpi()
+        e.ss, e.ss_n, e.inv_width, e.eps = wk["lat_ss"].data_ptr(), 2 * lw.lat_tiles, 1.0 / m.q_rank, self.cfg.eps
+        e.out, e.ldo, e.n_plain, e.act_tile0 = wk["queries"].data_ptr(), wk["queries"].stride(0), m.query_rows, lw.carry.N_pad // 256
+        self._linear(prog, lw.carry, wk["lat"], M, e, ws, tag)
+
     def _mixer_scratch(self, M: int, nseq: int, decode: bool) -> dict:
         """Scratch shared by the layers of a bucket, sized for the largest of them."""
         f32 = lambda n: torch.zeros(max(1, n), dtype=torch.float32, device=self.device)   # noqa: E731
@@ -279,6 +365,11 @@ class StackModel:
                                       device=self.device)
             wk["gqa_o"] = f32(M * mx(m.heads * m.vdim_pad * sp[id(m)] for m in split))
             wk["gqa_ml"] = f32(M * mx(2 * m.heads * sp[id(m)] for m in split))
+        carried = [m for m in la if m.q_rank]
+        if carried:
+            wk["lat"] = self._operand_buf(M, max(m.q_rank for m in carried))
+            wk["lat_ss"] = f32(L.padded_rows(M) * 2 * mx((m.q_rank + 255) // 256 for m in carried))
+            wk["queries"] = f32(M * mx(L.round_up(m.query_rows, 8) for m in carried)).view(M, -1)
         wk["q_eff"] = torch.zeros(max(1, M * mx(m.heads * (max(m.rank_pad, m.dim_pad) + m.rot_pad) for m in la)), dtype=self.dtype, device=self.device)
         absorbed = [m for m in la if not self._expanded(m, M, decode)]
         if absorbed:
@@ -311,6 +402,8 @@ class StackModel:
         p = N.GqaParams()
         p.H, p.G, p.D, p.DK, p.KP, p.V, p.VP = m.heads, m.kv_heads, m.dim, m.score_dim, m.key_pad, m.vdim, m.vdim_pad
         p.page, p.f32, p.scale, p.softcap = self.cfg.page_tokens, int(self.f32), m.scale, m.softcap
+        if m.rot is not None:
+            p.rot, p.rot_amp = m.rot.dims, m.rot.amplitude
         return p
 
     def _gqa_form(self, m: GroupedMixer, M: int, decode: bool) -> int:
@@ -342,7 +435,8 @@ class StackModel:
     def _gqa_params(self, run, lw, m: GroupedMixer, proj, m_op, M, nseq, lay, at, wk, decode) -> N.GqaParams:
         p = self._gqa_sizes(m)
         p.x, p.ldx = proj.data_ptr(), proj.stride(0)
-        p.q_off, p.k_off, p.v_off = lw.off["q"], lw.off.get("k", -1), lw.off.get("v", -1)
+        p.q_off, p.k_off, p.v_off, p.g_off = lw.off["q"], lw.off.get("k", -1), lw.off.get("v", -1), lw.off.get("g", -1)
+        p.freq, p.sink = N.ptr(lw.extra.get("freq")), N.ptr(lw.extra.get("sink"))
         p.cache, p.q = self.kv[self.cfg.pages_of(run)].data_ptr(), wk["gqa_q"].data_ptr()
         p.o_part, p.ml, p.counters = wk["gqa_o"].data_ptr(), wk["gqa_ml"].data_ptr(), wk["counters"].data_ptr()
         p.slot_map, p.pos, p.cu_rows, p.kv_len, p.block_table = (at(o) for o in (lay.slot_map, lay.pos, lay.cu_rows, lay.kv_len, lay.block_table))
@@ -370,9 +464,12 @@ class StackModel:
     def _mla_params(self, run, lw, m: LatentMixer, proj, m_op, M, nseq, lay, at, wk, decode) -> N.MlaParams:
         p = N.MlaParams()
         p.x, p.ldx = proj.data_ptr(), proj.stride(0)
-        p.q_off, p.dkv_off, p.g_off = lw.off["q"], lw.off["dkv"], lw.off["g"]
-        p.dkv_norm, p.freq, p.w_uk, p.w_uv = (lw.extra[k].data_ptr() for k in ("dkv_norm", "freq", "uk", "uv"))
-        p.cache, p.q_eff = self.kv[run.index].data_ptr(), wk["q_eff"].data_ptr()
+        p.q_off, p.dkv_off, p.g_off, p.q, p.ldq = lw.off.get("q", 0), lw.off.get("dkv", -1), lw.off["g"], proj.data_ptr(), proj.stride(0)
+        if m.q_rank:
+            p.q, p.ldq = wk["queries"].data_ptr(), wk["queries"].stride(0)
+        p.gate_heads, p.interleaved, p.rot_amp = int(m.gate_heads), int(m.rot.interleaved), m.rot.amplitude
+        p.dkv_norm, p.freq, p.w_uk, p.w_uv = (N.ptr(lw.extra.get(k)) for k in ("dkv_norm", "freq", "uk", "uv"))
+        p.cache, p.q_eff = self.kv[self.cfg.pages_of(run)].data_ptr(), wk["q_eff"].data_ptr()
         p.o_part, p.ml = N.ptr(wk.get("o_part")), N.ptr(wk.get("ml"))
         p.k_exp, p.v_exp = N.ptr(self.k_exp), N.ptr(self.v_exp)
         p.slot_map, p.pos, p.cu_rows, p.kv_len, p.block_table = (at(o) for o in (lay.slot_map, lay.pos, lay.cu_rows, lay.kv_len, lay.block_table))
@@ -398,7 +495,7 @@ class StackModel:
             e = N.LinEpi()
             if not normed:
                 self._row_norm(e, ss)
-            e.out, e.ldo, e.n_plain, e.act_tile0 = dst.data_ptr(), dst.stride(0), V, w.head.N_pad // 256
+            e.out, e.ldo, e.n_plain, e.act_tile0, e.cap = dst.data_ptr(), dst.stride(0), V, w.head.N_pad // 256, cfg.logit_cap
             self._linear(prog, w.head, a, rows, e, ws, tag)
 
         if decode:

@@ -1,5 +1,5 @@
 """Decoders described layer by layer: an ordered list of layers, each with its mixer and feed-forward (side by
-side behind one norm, or one after the other), an optional block of layers that runs several times, and the
+side behind one norm or a norm each, or one after the other), an optional block of layers that runs several times, and the
 constants of all of them.  `models.stack.StackModel` runs
 any such description; an architecture is a reader of its `config.json` (ARCHITECTURES) and the order and
 names of its tensors (`models.stack_weights`).
@@ -15,10 +15,44 @@ from pathlib import Path
 from typing import Optional
 
 
+@dataclass(frozen=True)
+class Rotation:
+    """Rotary positions on the first `dims` values of a head: pair i turns by position * f_i, f_i = base^(-2 i / dims) / factor.
+    yarn = (original, fast, slow): only the slow pairs are divided by the factor.  Pair i makes original f_i / 2 pi turns over
+    `original` positions; those with more than `fast` keep f_i, those with fewer than `slow` are divided, a ramp over whole pair
+    numbers lies between, and the rotated vector grows by 0.1 ln(factor) + 1."""
+    base: float
+    dims: int
+    interleaved: bool = False         # pair i is (x[2 i], x[2 i + 1]) instead of (x[i], x[i + dims / 2])
+    factor: float = 1.0
+    yarn: Optional[tuple] = None
+
+    def frequencies(self) -> list:
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if self.yarn is None:
+            return [x / self.factor for x in f]
+        original, fast, slow = self.yarn
+        pair = lambda turns: self.dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(self.base))    # noqa: E731
+        lo, hi = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(f))]
+        return [x / self.factor * r + x * (1.0 - r) for x, r in zip(f, ramp)]
+
+    @property
+    def amplitude(self) -> float:
+        return 1.0 if self.yarn is None else 0.1 * math.log(self.factor) + 1.0
+
+    @staticmethod
+    def from_json(d: dict, interleaved: bool = False) -> "Rotation":
+        s = d.get("scaling") or {}
+        yarn = (float(s["original"]), float(s["fast"]), float(s["slow"])) if "original" in s else None
+        return Rotation(float(d["base"]), d["dims"], interleaved, float(s.get("factor", 1.0)), yarn)
+
+
 class Mixer:
     """What a layer asks of its mixer.  `segments` are the rows of the input projection, in order."""
     kind = ""
     kv_from: Optional[int] = None     # layer whose pages this mixer reads (it has none of its own)
+    q_rank = 0                        # > 0: the first segment is a latent of this size, normed and carried on by a linear of its own
 
     def segments(self) -> list:
         """(name, rows)"""
@@ -94,14 +128,18 @@ class DeltaMixer(Mixer):
 
 @dataclass(frozen=True)
 class LatentMixer(Mixer):
-    """Latent attention: a cached latent of kv_rank values and one rotated key part of rot_dim per token."""
+    """Latent attention: a cached latent of kv_rank values and one rotated key part of rot_dim per token.  q_rank: queries come from
+    a normed latent of their own.  kv_from: that layer's latents and key parts, with this layer's own carriers."""
     heads: int
     dim: int
     rot_dim: int
     vdim: int
     kv_rank: int
     scale: float
-    rot_base: float
+    rot: Rotation
+    q_rank: int = 0
+    gate_heads: bool = False          # output gate: one per head, else one per value
+    kv_from: Optional[int] = None
     kind = "latent_attention"
 
     @property
@@ -129,13 +167,22 @@ class LatentMixer(Mixer):
         return next((n for n in (32, 64, 128, 256) if n >= self.vdim), self._pad16(self.vdim))
 
     def segments(self) -> list:
-        return [("q", self.heads * (self.dim + self.rot_dim)), ("dkv", self.kv_rank + self.rot_dim), ("g", self.heads * self.vdim)]
+        q = ("dq", self.q_rank) if self.q_rank else ("q", self.query_rows)
+        kv = [] if self.kv_from is not None else [("dkv", self.kv_rank + self.rot_dim)]
+        return [q, *kv, ("g", self.heads if self.gate_heads else self.heads * self.vdim)]
+
+    @property
+    def query_rows(self) -> int:
+        return self.heads * (self.dim + self.rot_dim)
 
     def extra_shapes(self) -> dict:
-        return {"dkv.norm": (self.kv_rank,), "uk": (self.heads * self.dim, self.kv_rank), "uv": (self.heads * self.vdim, self.kv_rank)}
+        t = {"dq.norm": (self.q_rank,), "uq": (self.query_rows, self.q_rank)} if self.q_rank else {}
+        if self.kv_from is None:
+            t["dkv.norm"] = (self.kv_rank,)
+        return {**t, "uk": (self.heads * self.dim, self.kv_rank), "uv": (self.heads * self.vdim, self.kv_rank)}
 
     def page_token_bytes(self, elem: int) -> int:
-        return elem * (self.rank_pad + self.rot_pad)
+        return 0 if self.kv_from is not None else elem * (self.rank_pad + self.rot_pad)
 
     @property
     def key_tile(self) -> int:        # an expanded key in whole 64-wide tiles
@@ -207,8 +254,9 @@ class OuterMixer(Mixer):
 
 @dataclass(frozen=True)
 class GroupedMixer(Mixer):
-    """Grouped-query attention without rotation: q and k over their root mean square per head, capped scores, keys of the
-    query's own chunk of positions.  kv_from: the pages of that layer are read, with this layer's queries and mask."""
+    """Grouped-query attention: q and k over their root mean square per head, rotated, capped scores, keys of the query's own
+    chunk of positions, a learned number per head in the denominator, an output gate; each where asked for.  kv_from: the pages
+    of that layer are read, with this layer's queries and mask."""
     heads: int
     kv_heads: int
     dim: int
@@ -219,6 +267,9 @@ class GroupedMixer(Mixer):
     qk_norm: bool = True
     bias: bool = True
     kv_from: Optional[int] = None
+    rot: Optional[Rotation] = None
+    sink: bool = False
+    gate: bool = False                # sigmoid of a projection, value by value
     kind = "attention"
 
     @property
@@ -238,34 +289,99 @@ class GroupedMixer(Mixer):
         return (self.vdim + 31) // 32 * 32
 
     def segments(self) -> list:
-        q = [("q", self.heads * self.dim)]
-        return q if self.kv_from is not None else q + [("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
+        q, g = [("q", self.heads * self.dim)], [("g", self.heads * self.vdim)] if self.gate else []
+        return q + g if self.kv_from is not None else q + [("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)] + g
 
     def biases(self) -> list:
-        return [name for name, _ in self.segments()] if self.bias else []
+        return [name for name, _ in self.segments() if name != "g"] if self.bias else []
+
+    def extra_shapes(self) -> dict:
+        return {"sink": (self.heads,)} if self.sink else {}
 
     def page_token_bytes(self, elem: int) -> int:
         return 0 if self.kv_from is not None else elem * self.kv_heads * (self.key_pad + self.vdim_pad)
 
 
+class FeedForward:
+    """What a layer asks of its feed-forward.  Its rows are tiles of 256 behind the mixer's: `per_tile` features each."""
+    act_kind = 0                      # the linear epilogue's activation
+    per_tile = 256
+    limit = alpha = 0.0
+
+    @property
+    def inner(self) -> int:
+        """Width of the activation that one linear produces and the next consumes (0: none)."""
+        return self.ff
+
+    @property
+    def tiles(self) -> int:
+        return (self.inner + self.per_tile - 1) // self.per_tile
+
+    def shapes(self, width: int) -> dict:
+        return {"up": (self.ff, width), "down": (width, self.ff)}
+
+
 @dataclass(frozen=True)
-class ClampedGlu:
+class ClampedGlu(FeedForward):
     """g = min(gate, limit), u = clamp(up, -limit, limit), y = g sigmoid(alpha g) (u + 1)."""
     ff: int
     limit: float
     alpha: float = 1.702
+    per_tile = 128
+
+    def shapes(self, width: int) -> dict:
+        return {"gate": (self.ff, width), **super().shapes(width)}
 
 
 @dataclass(frozen=True)
-class SquaredRelu:
+class SquaredRelu(FeedForward):
     """y = max(up, 0)^2, no gate."""
     ff: int
+    act_kind = 1
+
+
+@dataclass(frozen=True)
+class Gelu(FeedForward):
+    """y = gelu(up + b) by the error function; a bias behind either matrix."""
+    ff: int
+    act_kind = 3
+
+    def shapes(self, width: int) -> dict:
+        return {"up": (self.ff, width), "up.b": (self.ff,), "down": (width, self.ff), "down.b": (width,)}
+
+
+@dataclass(frozen=True)
+class ExpertMix(FeedForward):
+    """Mixture of squared-ReLU experts: softmax over `experts` scores, the `top` best of the `keep` groups of neighbours whose best
+    score is best, weighted by their scores as they are.  shared: the size of one more expert for every token, times the
+    sigmoid of a number of its own."""
+    experts: int
+    top: int
+    ff: int
+    groups: int = 1
+    keep: int = 1
+    shared: int = 0
+    act_kind = 2
+    per_tile = 248                    # and the shared expert's gate row behind them
+
+    @property
+    def inner(self) -> int:
+        return self.shared
+
+    def shapes(self, width: int) -> dict:
+        t = {}
+        for e in range(self.experts):
+            t[f"e{e}.up"], t[f"e{e}.down"] = (self.ff, width), (width, self.ff)
+        t["router"] = (self.experts, width)
+        if self.shared:
+            t.update({"shared.up": (self.shared, width), "shared.down": (width, self.shared), "shared.sg": (1, width)})
+        return t
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: Mixer
-    mlp: object = None                # ClampedGlu, SquaredRelu or None
+    mlp: Optional[FeedForward] = None
 
 
 @dataclass(frozen=True)
@@ -293,7 +409,9 @@ class StackConfig:
     layers: tuple
     eps: float = 1e-6
     embed_scale: float = 1.0
-    parallel: bool = True             # mixer and feed-forward side by side behind one norm; else one after the other, a norm each
+    parallel: bool = True             # mixer and feed-forward side by side; else one after the other, a norm each
+    two_norms: bool = False           # side by side: the feed-forward reads a norm of its own
+    logit_cap: float = 0.0            # logits become cap tanh(logits / cap)
     norm_offset: float = 0.0          # norms multiply by offset + weight
     loop: Optional[LoopSpec] = None
     page_tokens: int = 64
@@ -333,20 +451,38 @@ class StackConfig:
                 raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / norm_groups {m.norm_groups} / decay {m.decay}")
             if isinstance(m, GroupedMixer):
                 self._check_grouped(i, m)
-            if self.parallel and l.mlp is not None and not isinstance(l.mlp, ClampedGlu):
-                raise ValueError(f"{self.name}: layer {i}: a feed-forward beside its mixer is a clamped gated unit")
-            if isinstance(m, LatentMixer) and (m.rot_dim % 2 or m.kv_rank > 1024 or m.dim > 1024):
-                raise ValueError(f"{self.name}: layer {i}: rot_dim {m.rot_dim}, kv_rank {m.kv_rank}, dim {m.dim}")
+            if not self.parallel and isinstance(l.mlp, (Gelu, ExpertMix)):
+                raise ValueError(f"{self.name}: layer {i}: {type(l.mlp).__name__} stands beside its mixer only")
+            if isinstance(l.mlp, ExpertMix):
+                self._check_experts(i, l.mlp)
+            if isinstance(m, LatentMixer):
+                if m.rot_dim % 2 or m.kv_rank > 1024 or m.dim > 1024 or m.rot.dims != m.rot_dim:
+                    raise ValueError(f"{self.name}: layer {i}: rot_dim {m.rot_dim} (rotated {m.rot.dims}), kv_rank {m.kv_rank}, dim {m.dim}")
+                self._check_source(i, m, lambda s: (s.kv_rank, s.rot_dim, s.rot))
+        if self.two_norms and (not self.parallel or self.loop is not None):
+            raise ValueError(f"{self.name}: a second norm needs layers side by side and no loop")
+
+    def _check_experts(self, i: int, f: ExpertMix) -> None:
+        if not (1 <= f.experts <= 1024 and 1 <= f.top <= 32 and f.groups >= 1 and f.experts % f.groups == 0 and 1 <= f.keep <= f.groups
+                and f.top <= f.experts // f.groups * f.keep):
+            raise ValueError(f"{self.name}: layer {i}: top {f.top} of {f.experts} experts in {f.keep} of {f.groups} groups")
+        if not self.two_norms:
+            raise ValueError(f"{self.name}: layer {i}: a mixture of experts reads a norm of its own")
+
+    def _check_source(self, i: int, m: Mixer, sizes) -> None:
+        """A layer that reads another's pages finds a layer of its kind and sizes there."""
+        if m.kv_from is None:
+            return
+        s = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
+        if self.loop is not None or type(s) is not type(m) or s.kv_from is not None or sizes(s) != sizes(m):
+            raise ValueError(f"{self.name}: layer {i} cannot read the keys and values of layer {m.kv_from}")
 
     def _check_grouped(self, i: int, m: GroupedMixer) -> None:
         if m.heads % m.kv_heads or m.chunk < 0 or m.dim > 2048 or m.vdim > 2048:
             raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / chunk {m.chunk} / dim {m.dim} / vdim {m.vdim}")
-        if m.kv_from is None:
-            return
-        s = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
-        if self.loop is not None or not isinstance(s, GroupedMixer) or s.kv_from is not None or \
-                (s.kv_heads, s.dim, s.vdim) != (m.kv_heads, m.dim, m.vdim):
-            raise ValueError(f"{self.name}: layer {i} cannot read the keys and values of layer {m.kv_from}")
+        if m.rot is not None and (m.rot.dims % 2 or m.rot.dims > min(m.dim, 1024) or m.rot.interleaved):
+            raise ValueError(f"{self.name}: layer {i}: rotation of {m.rot.dims} of {m.dim} values")
+        self._check_source(i, m, lambda s: (s.kv_heads, s.dim, s.vdim, s.rot))
 
     def pages_of(self, run: LayerRun) -> int:
         """The run whose pages a run reads."""
@@ -364,7 +500,11 @@ class StackConfig:
         return max([l.mixer.expanded_token_bytes(elem) for l in self.layers if isinstance(l.mixer, LatentMixer)], default=0)
 
     def widest_project(self) -> int:
-        return max(sum(n for _, n in l.mixer.segments()) for l in self.layers)
+        return max(sum(n for _, n in l.mixer.segments()) + (l.mixer.query_rows if l.mixer.q_rank else 0) for l in self.layers)
+
+    def expert_row_bytes(self, rows: int, elem: int = 2) -> int:
+        """Scratch of the routed rows of a step (one layer at a time)."""
+        return max([rows * l.mlp.top * elem * (l.mlp.ff + self.width) for l in self.layers if isinstance(l.mlp, ExpertMix)], default=0)
 
     def param_count(self) -> int:
         from .stack_weights import tensor_shapes
@@ -387,7 +527,7 @@ def renosun_from_json(doc: dict, name: str = "renosun", source: Optional[str] = 
         elif l["type"] == "latent_attention":
             if m["rot"]["dims"] != m["rot_dim"]:
                 raise ValueError(f"layer {i}: rot.dims {m['rot']['dims']} is not rot_dim {m['rot_dim']}")
-            mixer = LatentMixer(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], float(m["scale"]), float(m["rot"]["base"]))
+            mixer = LatentMixer(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], float(m["scale"]), Rotation.from_json(m["rot"]))
         else:
             raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
         mlp = None
@@ -426,7 +566,35 @@ def tepavik_from_json(doc: dict, name: str = "tepavik", source: Optional[str] = 
                        parallel=False, norm_offset=1.0, source=source, max_ctx=max_ctx)
 
 
-ARCHITECTURES = {"Renosun": renosun_from_json, "Tepavik": tepavik_from_json}
+# ------------------------------------------------------------------------------------ Fitatar
+def fitatar_from_json(doc: dict, name: str = "fitatar", source: Optional[str] = None, max_ctx: int = 32768) -> StackConfig:
+    layers = []
+    for i, l in enumerate(doc["layers"]):
+        m, f = l["mixer"], l.get("mlp")
+        if l["type"] == "latent_attention":
+            mixer = LatentMixer(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], float(m["scale"]), Rotation.from_json(m["rot"], interleaved=True),
+                                q_rank=m["q_rank"], gate_heads=True, kv_from=m.get("kv_from"))
+        elif l["type"] == "attention":
+            mixer = GroupedMixer(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), qk_norm=False, bias=False,
+                                 rot=Rotation.from_json(m["rot"]), sink=True, gate=True)
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
+        if f is None:
+            mlp = None
+        elif f["kind"] == "dense":
+            mlp = Gelu(f["ff"])
+        elif f["kind"] == "moe":
+            r, g = f["router"], f["router"].get("groups") or {}
+            mlp = ExpertMix(r["experts"], r["top"], f["expert"]["ff"], g.get("count", 1), g.get("keep", 1), (f.get("shared") or {}).get("ff", 0))
+        else:
+            raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+        layers.append(LayerSpec(mixer, mlp))
+    return StackConfig(name=name, arch="Fitatar", vocab=doc["vocab"], width=doc["width"], layers=tuple(layers), eps=float(doc["norm"]["eps"]),
+                       embed_scale=float(doc["embedding"]["scale"]), two_norms=True, logit_cap=float(doc.get("logit_softcap") or 0.0),
+                       source=source, max_ctx=max_ctx)
+
+
+ARCHITECTURES = {"Renosun": renosun_from_json, "Tepavik": tepavik_from_json, "Fitatar": fitatar_from_json}
 
 
 def from_json(doc: dict, **kw) -> StackConfig:
@@ -450,7 +618,7 @@ def load_dir(path: str) -> StackConfig:
 def renosun_mini() -> StackConfig:
     """Small sizes for smoke tests and demos."""
     d = LayerSpec(DeltaMixer(6, 2, 64, 48, 3), ClampedGlu(384, 4.0))
-    a = LayerSpec(LatentMixer(3, 64, 32, 40, 96, 96 ** -0.5, 1e4), ClampedGlu(384, 4.0))
+    a = LayerSpec(LatentMixer(3, 64, 32, 40, 96, 96 ** -0.5, Rotation(1e4, 32)), ClampedGlu(384, 4.0))
     return StackConfig("renosun-mini", "Renosun", vocab=1024, width=320, layers=(a, d, d, a, d), embed_scale=8.0, loop=LoopSpec(1, 4, 2),
                        max_ctx=4096)
 
@@ -458,7 +626,7 @@ def renosun_mini() -> StackConfig:
 def renosun_bench(name: str, width: int, ff: int, kv_heads: int, heads: int, attn_heads: int, n_layers: int = 8, vocab: int = 65536) -> StackConfig:
     """Layers of a real model's size: three delta layers to one attention layer."""
     d = LayerSpec(DeltaMixer(heads, kv_heads, 128, 128, 4), ClampedGlu(ff, 7.0))
-    a = LayerSpec(LatentMixer(attn_heads, 128, 64, 128, 512, 192 ** -0.5, 1e6), ClampedGlu(ff, 7.0))
+    a = LayerSpec(LatentMixer(attn_heads, 128, 64, 128, 512, 192 ** -0.5, Rotation(1e6, 64)), ClampedGlu(ff, 7.0))
     layers = tuple(a if i % 4 == 3 else d for i in range(n_layers))
     return StackConfig(name, "Renosun", vocab=vocab, width=width, layers=layers, embed_scale=width ** 0.5, loop=LoopSpec(n_layers // 4, n_layers // 2, 2))
 
@@ -490,7 +658,34 @@ def tepavik_bench(name: str, width: int, ff: int, heads: int, kv_heads: int, chu
     return StackConfig(name, "Tepavik", vocab=vocab, width=width, layers=tuple(layers), parallel=False, norm_offset=1.0)
 
 
-NAMED = {"tepavik-mini": tepavik_mini,
+def fitatar_mini() -> StackConfig:
+    """Small sizes for smoke tests and demos."""
+    a = GroupedMixer(6, 2, 48, 40, 0.15, qk_norm=False, bias=False, rot=Rotation(1e4, 24, factor=2.0), sink=True, gate=True)
+    la = LatentMixer(4, 48, 32, 56, 80, 0.12, Rotation(1e5, 32, True, 4.0, (1024.0, 32.0, 1.0)), q_rank=112, gate_heads=True)
+    moe = ExpertMix(24, 3, 96, 6, 2, 160)
+    layers = (LayerSpec(a, Gelu(448)), LayerSpec(la, moe), LayerSpec(a, moe), LayerSpec(dataclasses.replace(la, kv_from=1), moe))
+    return StackConfig("fitatar-mini", "Fitatar", vocab=1024, width=288, layers=layers, embed_scale=10.0, two_norms=True, logit_cap=20.0, max_ctx=4096)
+
+
+def fitatar_bench(name: str, width: int, ff: int, heads: int, kv_heads: int, expert_ff: int, experts: int = 64, top: int = 6, shared: int = 2,
+                  n_layers: int = 8, vocab: int = 65536) -> StackConfig:
+    """Layers of a real model's size: a dense layer, then mixtures of experts; every fourth mixer is latent attention, the later
+    ones on the latents of the first."""
+    a = GroupedMixer(heads, kv_heads, 128, 128, 128 ** -0.5, qk_norm=False, bias=False, rot=Rotation(1e6, 64, factor=4.0), sink=True, gate=True)
+    la = LatentMixer(heads, 128, 64, 128, 512, 192 ** -0.5, Rotation(1e6, 64, True, 8.0, (4096.0, 32.0, 1.0)), q_rank=1536, gate_heads=True)
+    moe = ExpertMix(experts, top, expert_ff, 8, 4, shared * expert_ff)
+    layers = []
+    for i in range(n_layers):
+        m = dataclasses.replace(la, kv_from=None if i < 4 else 1) if i % 4 == 1 else a
+        layers.append(LayerSpec(m, moe if i else Gelu(ff)))
+    return StackConfig(name, "Fitatar", vocab=vocab, width=width, layers=tuple(layers), embed_scale=width ** 0.5, two_norms=True, logit_cap=30.0)
+
+
+NAMED = {"fitatar-mini": fitatar_mini,
+         "fitatar-2k": lambda: fitatar_bench("fitatar-2k", 2048, 8192, 16, 4, 1024),
+         "fitatar-4k": lambda: fitatar_bench("fitatar-4k", 4096, 16384, 32, 8, 1536),
+         "fitatar-5k": lambda: fitatar_bench("fitatar-5k", 5120, 20480, 40, 8, 2048),
+         "tepavik-mini": tepavik_mini,
          "tepavik-2k": lambda: tepavik_bench("tepavik-2k", 2048, 8192, 16, 4),
          "tepavik-4k": lambda: tepavik_bench("tepavik-4k", 4096, 16384, 32, 8),
          "tepavik-5k": lambda: tepavik_bench("tepavik-5k", 5120, 20480, 40, 8),

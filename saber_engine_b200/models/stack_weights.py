@@ -2,10 +2,13 @@
 layouts its kernels read.
 
 Side by side (parallel residual), a layer needs two linears.  `proj` holds every row that reads the normed stream:
-the mixer's segments (each starting at a multiple of 8 rows, the whole padded to 256), then the feed-forward's rows
-as tiles of 128 gate and 128 up rows of the same features.  `out` holds the mixer's output columns and the down
-columns side by side, so that one product adds both sublayers to the stream.  One after the other, `proj` and `out`
-belong to the mixer alone and `up` and `down` to the feed-forward behind its own norm.
+the mixer's segments (each starting at a multiple of 8 rows, the whole padded to 256; a latent that queries come from has
+whole tiles of its own ahead of them), then the feed-forward's rows as tiles of 256: 128 gate and 128 up rows of the same
+features, 256 up rows, or 248 up rows and the row of their gate.  `out` holds the mixer's output columns and the down
+columns side by side, so that one product adds both sublayers to the stream.  Where the feed-forward reads a norm of its
+own, its rows (a router's first) start at a tile of their own and multiply the second operand.  One after the other, `proj` and
+`out` belong to the mixer alone and `up` and `down` to the feed-forward behind its own norm.  The routed experts of a mixture
+are stacks of tiles, expert after expert.
 """
 from __future__ import annotations
 
@@ -20,7 +23,7 @@ from typing import Callable, Optional
 import torch
 
 from ..ops import layouts as L
-from .stack_config import ClampedGlu, DeltaMixer, LatentMixer, OuterMixer, StackConfig
+from .stack_config import ClampedGlu, DeltaMixer, ExpertMix, Gelu, GroupedMixer, LatentMixer, OuterMixer, StackConfig
 
 _ST_DTYPES = {"BF16": torch.bfloat16, "F32": torch.float32, "F16": torch.float16, "I32": torch.int32, "I64": torch.int64}
 
@@ -61,11 +64,9 @@ def tensor_shapes(cfg: StackConfig) -> dict:
             t[f"{p}mix.{name}"] = shape
         t[p + "mix.o"] = (w, m.out_features)
         if l.mlp is not None:
-            if not cfg.parallel:
+            if not cfg.parallel or cfg.two_norms:
                 t[p + "norm2"] = (w,)
-            for name in ("gate", "up") if isinstance(l.mlp, ClampedGlu) else ("up",):
-                t[f"{p}mlp.{name}"] = (l.mlp.ff, w)
-            t[p + "mlp.down"] = (w, l.mlp.ff)
+            t.update({f"{p}mlp.{name}": shape for name, shape in l.mlp.shapes(w).items()})
     t["final.norm"], t["head"] = (w,), (cfg.vocab, w)
     return t
 
@@ -75,7 +76,7 @@ def random_tensor(name: str, shape: tuple, g: torch.Generator, device, norm_offs
     if leaf in ("norm1", "norm2", "norm"):
         around = norm_offset if ".mix." not in name else 0.0            # (a mixer's own norm is stored plain)
         return torch.full(shape, 1.0 - around, dtype=torch.bfloat16, device=device)
-    if leaf == "D":
+    if leaf in ("D", "sink"):
         return torch.ones(shape, dtype=torch.bfloat16, device=device)
     if leaf == "b":
         return torch.zeros(shape, dtype=torch.bfloat16, device=device)
@@ -106,13 +107,23 @@ class StackLayer:
     out: Linear
     off: dict                        # segment name -> first column of the projection
     n_plain: int                     # columns of the projection's stored part
-    act_tile0: int                   # first gate | up tile
+    act_tile0: int                   # first feed-forward tile
     act_k0: int                      # first feed-forward column of `out`'s operand
     extra: dict = field(default_factory=dict)
     bias: Optional[torch.Tensor] = None     # fp32, of the projection's stored columns
-    norm2: Optional[torch.Tensor] = None    # feed-forward behind the mixer: its norm and linears
-    up: Optional[Linear] = None
+    norm2: Optional[torch.Tensor] = None    # the feed-forward's own norm
+    up: Optional[Linear] = None             # feed-forward behind the mixer: its linears
     down: Optional[Linear] = None
+    tile2: int = 0                          # first tile of the rows behind norm2 (side by side)
+    lat_tiles: int = 0                      # tiles of the latent that queries come from
+    carry: Optional[Linear] = None          # the linear from that latent to the queries
+    act_bias: Optional[torch.Tensor] = None # fp32, of the feed-forward's rows
+    out_bias: Optional[torch.Tensor] = None # fp32, of `out`
+    experts_up: Optional[Linear] = None     # stacks of routed experts: N_pad and K of one
+    experts_down: Optional[Linear] = None
+
+    def linears(self) -> list:
+        return [x for x in (self.proj, self.out, self.up, self.down, self.carry, self.experts_up, self.experts_down) if x is not None]
 
 
 @dataclass
@@ -127,7 +138,7 @@ class StackWeights:
     def nbytes(self) -> int:
         tot = self.embed.numel() * self.embed.element_size() + self.head.nbytes() + (self.loop_in.nbytes() if self.loop_in else 0)
         for l in self.layers:
-            tot += sum(x.nbytes() for x in (l.proj, l.out, l.up, l.down) if x is not None) + sum(t.numel() * t.element_size() for t in l.extra.values())
+            tot += sum(x.nbytes() for x in l.linears()) + sum(t.numel() * t.element_size() for t in l.extra.values())
         return tot
 
 
@@ -140,14 +151,37 @@ def pack_linear(rows: torch.Tensor, dtype: torch.dtype) -> Linear:
     return Linear(L.tile_weight_int8(rows.to(torch.bfloat16).contiguous().view(torch.int8).reshape(n, k * 2)), n, k)
 
 
-def project_layout(mixer, mlp: Optional[ClampedGlu]) -> tuple:
-    """(segment offsets, stored columns, first gate | up tile, rows in all)."""
-    off, n = {}, 0
-    for name, rows in mixer.segments():
+def pack_experts(rows: torch.Tensor, dtype: torch.dtype) -> Linear:
+    """rows [experts, N_pad, K]: one expert's tiles after the other's."""
+    e, n, k = rows.shape
+    return Linear(pack_linear(rows.reshape(e * n, k), dtype).w, n, k)
+
+
+@dataclass
+class ProjectLayout:
+    off: dict            # segment -> first row
+    n_plain: int         # rows whose results are stored
+    tile2: int           # first tile behind the second norm
+    tile0: int           # first feed-forward tile
+    rows: int            # in all
+    lat_tiles: int
+
+
+def project_layout(mixer, mlp, two_norms: bool = False) -> ProjectLayout:
+    """mlp: the feed-forward beside the mixer, or None."""
+    off, n, lat = {}, 0, 0
+    for i, (name, rows) in enumerate(mixer.segments()):
         off[name] = n
         n = (n + rows + 7) // 8 * 8
+        if i == 0 and mixer.q_rank:
+            n = L.round_up(n, 256)
+            lat = n // 256
+    tile2 = (n + 255) // 256
+    if two_norms and isinstance(mlp, ExpertMix):
+        off["router"] = tile2 * 256
+        n = (off["router"] + mlp.experts + 7) // 8 * 8
     tile0 = (n + 255) // 256
-    return off, n, tile0, (tile0 + ((mlp.ff + 127) // 128 if mlp is not None else 0)) * 256
+    return ProjectLayout(off, n, tile2, tile0, (tile0 + (mlp.tiles if mlp is not None else 0)) * 256, lat)
 
 
 def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dtype, device) -> StackWeights:
@@ -170,8 +204,9 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.", l.mixer
         beside = l.mlp if cfg.parallel else None
-        off, n_plain, tile0, rows = project_layout(m, beside)
-        r, seg_rows, bias = zeros(rows, KW), dict(m.segments()), None
+        lay = project_layout(m, beside, cfg.two_norms)
+        off, n_plain, tile0 = lay.off, lay.n_plain, lay.tile0
+        r, seg_rows, bias = zeros(lay.rows, KW), dict(m.segments()), None
         for name, tensor, first in m.sources():
             r[off[name]: off[name] + seg_rows[name], :W] = t(f"{p}mix.{tensor}")[first: first + seg_rows[name]]
         if m.biases():
@@ -180,17 +215,39 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
                 if name in m.biases():
                     bias[off[name]: off[name] + seg_rows[name]] = f32(f"{p}mix.{tensor}.b")
         mix_k = L.round_up(m.out_features, 64)
-        ff_k = L.round_up(l.mlp.ff, 128) if beside is not None else 0
+        ff_k = L.round_up(beside.inner, 128 if isinstance(beside, ClampedGlu) else 64) if beside is not None else 0
         o = zeros(NW, mix_k + ff_k)
         o[:W, : m.out_features] = t(p + "mix.o")
-        if beside is not None:
+        act_bias = out_bias = ex_up = ex_down = None
+        if isinstance(beside, ClampedGlu):
             gu = r[tile0 * 256:].view(-1, 2, 128, KW)                  # [tile][gate | up][feature][K]
             for half, name in enumerate(("gate", "up")):
                 full = zeros(ff_k, KW)
                 full[: l.mlp.ff, :W] = t(f"{p}mlp.{name}")
                 gu[:, half] = full.view(-1, 128, KW)
             o[:W, mix_k: mix_k + l.mlp.ff] = t(p + "mlp.down")
-        extra = {}
+        elif isinstance(beside, ExpertMix):
+            r[off["router"]: off["router"] + beside.experts, :W] = t(p + "mlp.router")
+            if beside.shared:
+                full = zeros(beside.tiles * beside.per_tile, KW)
+                full[: beside.shared, :W] = t(p + "mlp.shared.up")
+                tiles = r[tile0 * 256:].view(-1, 256, KW)
+                tiles[:, : beside.per_tile] = full.view(-1, beside.per_tile, KW)
+                tiles[:, beside.per_tile, :W] = t(p + "mlp.shared.sg")[0]
+                o[:W, mix_k: mix_k + beside.shared] = t(p + "mlp.shared.down")
+            eu, ed = zeros(beside.experts, L.round_up(beside.ff, 256) * KW), zeros(beside.experts, NW * L.round_up(beside.ff, 64))
+            eu, ed = eu.view(beside.experts, -1, KW), ed.view(beside.experts, NW, -1)
+            for e in range(beside.experts):
+                eu[e, : beside.ff, :W], ed[e, :W, : beside.ff] = t(f"{p}mlp.e{e}.up"), t(f"{p}mlp.e{e}.down")
+            ex_up, ex_down = pack_experts(eu, dtype), pack_experts(ed, dtype)
+            del eu, ed
+        elif beside is not None:
+            r[tile0 * 256: tile0 * 256 + beside.ff, :W] = t(p + "mlp.up")
+            o[:W, mix_k: mix_k + beside.ff] = t(p + "mlp.down")
+            if isinstance(beside, Gelu):
+                act_bias, out_bias = torch.zeros(beside.tiles * 256, dtype=torch.float32, device=dev), f32(p + "mlp.down.b")
+                act_bias[: beside.ff] = f32(p + "mlp.up.b")
+        extra, carry = {}, None
         if isinstance(m, DeltaMixer):
             extra["conv"] = torch.cat([f32(f"{p}mix.{n}.conv") for n in ("q", "k", "v")]).contiguous()
             for n in ("A_log", "dt_bias", "norm"):
@@ -206,14 +263,25 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
                     c = f32(f"{p}mix.{n}")
                     extra[key] = torch.cat([c[vd + kd:], c[vd: vd + kd], c[:vd]]).contiguous()
         elif isinstance(m, LatentMixer):
-            extra["dkv_norm"] = f32(p + "mix.dkv.norm")
+            if m.kv_from is None:
+                extra["dkv_norm"] = f32(p + "mix.dkv.norm")
+            if m.q_rank:
+                extra["dq_norm"] = f32(p + "mix.dq.norm")
+                c = zeros(L.round_up(m.query_rows, 256), L.round_up(m.q_rank, 64))
+                c[: m.query_rows, : m.q_rank] = t(p + "mix.uq")
+                carry = pack_linear(c, dtype)
             for n in ("uk", "uv"):                                     # row stride: the padded latent
                 full = t(f"{p}mix.{n}")
                 extra[n] = torch.zeros(full.shape[0], m.rank_pad, dtype=dtype, device=dev)
                 extra[n][:, : m.kv_rank] = full
-            half = m.rot_dim // 2
-            extra["freq"] = torch.tensor([m.rot_base ** (-2.0 * j / m.rot_dim) for j in range(half)] or [1.0], dtype=torch.float32, device=dev)
-        lw = StackLayer(norm(p + "norm1"), pack_linear(r, dtype), pack_linear(o, dtype), off, n_plain, tile0, mix_k, extra, bias)
+        elif isinstance(m, GroupedMixer) and m.sink:
+            extra["sink"] = f32(p + "mix.sink")
+        if getattr(m, "rot", None) is not None:
+            extra["freq"] = torch.tensor(m.rot.frequencies() or [1.0], dtype=torch.float32, device=dev)
+        lw = StackLayer(norm(p + "norm1"), pack_linear(r, dtype), pack_linear(o, dtype), off, n_plain, tile0, mix_k, extra, bias,
+                        tile2=lay.tile2, lat_tiles=lay.lat_tiles, carry=carry, act_bias=act_bias, out_bias=out_bias, experts_up=ex_up, experts_down=ex_down)
+        if beside is not None and cfg.two_norms:
+            lw.norm2 = norm(p + "norm2")
         del r, o
         if l.mlp is not None and not cfg.parallel:
             ff = l.mlp.ff

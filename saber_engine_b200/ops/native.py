@@ -141,7 +141,8 @@ class PickMergeParams(C.Structure):
 class MoeRouteParams(C.Structure):
     _fields_ = [("logits", P), ("topk_id", P), ("topk_w", P), ("counts", P), ("offsets", P), ("cursors", P),
                 ("tiles", P), ("ntiles", P), ("src_row", P), ("slot_of", P), ("M", I), ("ld", I), ("E", I),
-                ("top_k", I), ("nt", I), ("rows_cap", I), ("e_lo", I), ("e_n", I), ("norm_topk", I)]
+                ("top_k", I), ("nt", I), ("rows_cap", I), ("e_lo", I), ("e_n", I), ("norm_topk", I),
+                ("logits_f32", P), ("live", P), ("groups", I), ("keep", I)]
 
 
 class MoeCombineParams(C.Structure):
@@ -173,17 +174,20 @@ class Operand(C.Structure):
 class LinEpi(C.Structure):
     _fields_ = [("stream", I), ("ss", P), ("ss_n", I), ("inv_width", F), ("eps", F), ("out", P), ("ldo", I), ("n_plain", I),
                 ("act_tile0", I), ("act", Operand), ("act_k0", I), ("act_kind", I), ("limit", F), ("alpha", F), ("x", P), ("ldx", I), ("width", I),
-                ("add", I), ("bias", P), ("norm_w", P), ("op", Operand), ("op_k0", I), ("ss_out", P), ("ss_out_n", I)]
+                ("add", I), ("bias", P), ("norm_w", P), ("op", Operand), ("op_k0", I), ("ss_out", P), ("ss_out_n", I),
+                ("lat_tiles", I), ("lat_n", I), ("lat", Operand), ("lat_w", P), ("lat_ss", P), ("lat_ss_n", I), ("act_bias", P), ("cap", F),
+                ("norm_w2", P), ("op2", Operand), ("y", P), ("slot_of", P), ("route_w", P), ("routes", I), ("ldy", I), ("y_f32", I), ("out_bf16", I)]
 
 
 class LinParams(C.Structure):
-    _fields_ = [("w", P), ("a", P), ("ws", P), ("counters", P), ("err", P), ("M", I), ("M_pad", I), ("N_pad", I), ("K", I), ("nt", I),
-                ("splits", I), ("fp32", I), ("fuse", I), ("mtiles", I), ("e", LinEpi)]
+    _fields_ = [("w", P), ("a", P), ("a2", P), ("ws", P), ("counters", P), ("err", P), ("M", I), ("M_pad", I), ("N_pad", I), ("K", I), ("nt", I),
+                ("splits", I), ("fp32", I), ("fuse", I), ("mtiles", I), ("a2_tile0", I), ("group_tiles", P), ("group_ntiles", P), ("group_rows", P), ("src_row", P),
+                ("group_w_stride", U64), ("group_max", I), ("e", LinEpi)]
 
 
 class StreamEmbedParams(C.Structure):
     _fields_ = [("table", P), ("table_f32", I), ("vocab", I), ("ids", P), ("M", I), ("width", I), ("scale", F), ("x", P), ("x0", Operand),
-                ("x0_k0", I), ("norm_w", P), ("op", Operand), ("op_k0", I), ("ss_out", P), ("ss_out_n", I)]
+                ("x0_k0", I), ("norm_w", P), ("op", Operand), ("op_k0", I), ("ss_out", P), ("ss_out_n", I), ("norm_w2", P), ("op2", Operand)]
 
 
 class StreamNormParams(C.Structure):
@@ -198,7 +202,8 @@ class DeltaParams(C.Structure):
 
 
 class MlaParams(C.Structure):
-    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("dkv_off", I), ("g_off", I), ("dkv_norm", P), ("freq", P), ("w_uk", P), ("w_uv", P),
+    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("dkv_off", I), ("g_off", I), ("q", P), ("ldq", I), ("gate_heads", I), ("interleaved", I),
+                ("rot_amp", F), ("dkv_norm", P), ("freq", P), ("w_uk", P), ("w_uv", P),
                 ("cache", P), ("q_eff", P), ("o_part", P), ("ml", P), ("k_exp", P), ("v_exp", P), ("slot_map", P), ("pos", P),
                 ("cu_rows", P), ("kv_len", P), ("block_table", P), ("out", Operand), ("out_k0", I), ("M", I), ("nseq", I), ("H", I),
                 ("D", I), ("R", I), ("V", I), ("C", I), ("CP", I), ("RP", I), ("DP", I), ("VP", I), ("page", I), ("n_blocks", I),
@@ -214,7 +219,8 @@ class SsdParams(C.Structure):
 
 
 class GqaParams(C.Structure):
-    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("k_off", I), ("v_off", I), ("cache", P), ("q", P), ("o_part", P), ("ml", P),
+    _fields_ = [("x", P), ("ldx", I), ("q_off", I), ("k_off", I), ("v_off", I), ("g_off", I), ("rot", I), ("rot_amp", F), ("freq", P), ("sink", P),
+                ("cache", P), ("q", P), ("o_part", P), ("ml", P),
                 ("counters", P), ("slot_map", P), ("pos", P), ("cu_rows", P), ("kv_len", P), ("block_table", P), ("out", Operand),
                 ("out_k0", I), ("M", I), ("nseq", I), ("H", I), ("G", I), ("D", I), ("DK", I), ("KP", I), ("V", I), ("VP", I), ("page", I),
                 ("n_blocks", I), ("max_blocks", I), ("splits", I), ("f32", I), ("form", I), ("max_rows", I), ("qk_norm", I), ("chunk", I),

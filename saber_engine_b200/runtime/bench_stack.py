@@ -17,7 +17,7 @@ import torch
 from ..models import config as C
 from ..models.hybrid import HybridModel
 from ..models.stack import StackModel
-from ..models.stack_config import (ClampedGlu, DeltaMixer, GroupedMixer, LatentMixer, LayerSpec, OuterMixer, StackConfig)
+from ..models.stack_config import (ClampedGlu, DeltaMixer, GroupedMixer, LatentMixer, LayerSpec, OuterMixer, Rotation, StackConfig)
 from ..models.step import SeqStep, run_bucket
 
 SIZES = ("renosun-2k", "renosun-4k", "renosun-5k", "tepavik-2k", "tepavik-4k", "tepavik-5k")
@@ -41,7 +41,7 @@ def like_renosun(cfg: StackConfig) -> StackConfig:
     a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, GroupedMixer))
     mlp = ClampedGlu(cfg.layers[0].mlp.ff * 2 // 3 // 128 * 128, 7.0)
     d = LayerSpec(DeltaMixer(a.heads, a.heads // 2, 128, 128, 4), mlp)
-    la = LayerSpec(LatentMixer(a.heads, 128, 64, 128, 512, 192 ** -0.5, 1e6), mlp)
+    la = LayerSpec(LatentMixer(a.heads, 128, 64, 128, 512, 192 ** -0.5, Rotation(1e6, 64)), mlp)
     return StackConfig(f"renosun-like-{cfg.name}", "Renosun", vocab=cfg.vocab, width=cfg.width,
                        layers=tuple(la if isinstance(l.mixer, GroupedMixer) else d for l in cfg.layers), max_ctx=cfg.max_ctx)
 

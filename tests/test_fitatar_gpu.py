@@ -35,6 +35,7 @@ ALONE = {
     "experts_without_groups": [R.latent(mlp=R.moe(groups=1, keep=1, experts=10, top=4, ff=24))],
     "experts_without_shared": [R.attention(mlp=R.moe(shared=0, ff=136))],
     "one_of_many_experts": [R.attention(mlp=R.moe(experts=72, groups=9, keep=1, top=1, shared=248))],
+    "odd_width": [R.attention(mlp=R.dense(50)), R.latent(mlp=R.moe(ff=12, shared=20))],
     "groups_of_one": [R.attention(mlp=R.moe(experts=7, groups=7, keep=4, top=4, shared=249))],
 }
 
@@ -42,7 +43,7 @@ ALONE = {
 @pytest.mark.parametrize("name", ALONE)
 @pytest.mark.parametrize("dtype", [F32, BF16])
 def test_mechanism_alone_residual_stream(name, dtype):
-    cfg = R.config(ALONE[name])
+    cfg = R.config(ALONE[name], **({"width": 91} if name == "odd_width" else {}))
     t = R.tensors(cfg, seed=3)
     toks = R.tokens(cfg, 140)
     trace = []
@@ -144,7 +145,7 @@ def test_project_linear_parts(M, K, lat, plain, ff, splits, fuse, kind):
     want = torch.relu(z) ** 2 * torch.sigmoid(a2.double() @ gate.double().T * r) if kind == 2 else O.gelu(z + act_bias[:ff].cpu().double())
     got = _rows(act, M)
     _near(got[:, 64: 64 + ff], want, 0.01)
-    assert torch.all(got[:, :64] == 5.0) and torch.all(got[:, 64 + ff:] == 0)
+    assert torch.all(got[:, :64] == 5.0) and torch.all(got[:, 64 + ff: 64 + (n - tile0) * per] == 0)      # (columns past the tiles meet zero weights)
 
 
 def _route(z, top, groups, keep, nt, live):
@@ -336,7 +337,7 @@ def test_one_key_far_back_and_at_page_edges(dtype, kind):
         want = orc.forward(toks)
         without = list(toks)
         without[place] = 2
-        assert R.error(orc.forward(without)[-1:], want[-1:]) > 0.3               # the answer hangs on that one key
+        assert R.error(orc.forward(without)[-1:], want[-1:]) > 0.2               # the answer hangs on that one key
         for eng in engs:
             for cuts in ([n], [n - 1, 1], [n - 2, 2], [max(1, place), 1, 2, 200, 255, 1]):
                 assert R.error(R.feed(eng, "r", toks, cuts)[-1:], want[-1:]) < tol, (place, cuts)

@@ -111,7 +111,7 @@ def main() -> int:
     ap.add_argument("--no-extra-arms", action="store_true", help="skip the NVFP4 side arm of the 27B run")
     ap.add_argument("--no-single", action="store_true", help="skip the single-stream side measurement")
     ap.add_argument("--stack", default="", metavar="NAMES", help="instead of the headline workload: prefill and decode throughput of these layer-by-layer "
-                    "models (comma separated, or 'all'), each beside the hybrid decoder at equal layer sizes, with a roofline per launch group")
+                    "models (comma separated, or 'all'), each beside its closest relatives at equal layer sizes, with a roofline per launch group")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)

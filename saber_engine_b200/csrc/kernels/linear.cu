@@ -46,27 +46,45 @@ __device__ __forceinline__ float stored(const LinEpi& e, int n, float v) {      
 
 constexpr int kGatedTile = 248;           // features of a tile of act_kind 2; row 248 of the tile is their gate
 
-// v[0..7] += sum over the routes of token m of their weight times the expert's row, columns from n on
-__device__ __forceinline__ void add_routes(const LinEpi& e, int m, int n, float (&v)[8]) {
-#pragma unroll 4
-  for (int k = 0; k < e.routes; ++k) {
-    const int r = e.slot_of[m * e.routes + k];
-    if (r < 0) continue;
-    const float w = e.route_w[m * e.routes + k];
-    if (e.y_f32) {
-      const float4* y = reinterpret_cast<const float4*>(static_cast<const float*>(e.y) + static_cast<size_t>(r) * e.ldy + n);
-      const float4 a = __ldcg(y), b = __ldcg(y + 1);
-      v[0] = fmaf(w, a.x, v[0]); v[1] = fmaf(w, a.y, v[1]); v[2] = fmaf(w, a.z, v[2]); v[3] = fmaf(w, a.w, v[3]);
-      v[4] = fmaf(w, b.x, v[4]); v[5] = fmaf(w, b.y, v[5]); v[6] = fmaf(w, b.z, v[6]); v[7] = fmaf(w, b.w, v[7]);
-    } else {
-      const uint4 q = __ldcg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(e.y) + static_cast<size_t>(r) * e.ldy + n));
-      const uint32_t u[4] = {q.x, q.y, q.z, q.w};
+// x[i] (eight stream values of rows m + 8 i, columns from n on) += the sum over the rows' routes of weight times expert row.  A lane holds
+// a route of each row; sixteen pieces of expert rows are requested together.
+__device__ __forceinline__ void add_routes(const LinEpi& e, int m, int rows, int n, bool cols, int lane, float4 (&x)[4][2]) {
+  int slot[4];
+  float wt[4];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        v[2 * i] = fmaf(w, __uint_as_float(u[i] << 16), v[2 * i]);
-        v[2 * i + 1] = fmaf(w, __uint_as_float(u[i] & 0xFFFF0000u), v[2 * i + 1]);
+  for (int i = 0; i < 4; ++i) {
+    const bool in = 8 * i < rows && lane < e.routes;
+    slot[i] = in ? e.slot_of[(m + 8 * i) * e.routes + lane] : -1;
+    wt[i] = in ? e.route_w[(m + 8 * i) * e.routes + lane] : 0.f;
+  }
+  const __nv_bfloat16* y = static_cast<const __nv_bfloat16*>(e.y) + n;
+  for (int k0 = 0; k0 < e.routes; k0 += 4) {
+    uint4 q[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int r = __shfl_sync(0xffffffffu, slot[i], (k0 + k) & 31);
+        q[i][k] = make_uint4(0u, 0u, 0u, 0u);
+        if (cols && r >= 0) q[i][k] = __ldcg(reinterpret_cast<const uint4*>(y + static_cast<size_t>(r) * e.ldy));
       }
-    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float w = __shfl_sync(0xffffffffu, wt[i], (k0 + k) & 31);
+        const uint4 u = q[i][k];
+        float4& a = x[i][0];
+        float4& b = x[i][1];
+        a.x = fmaf(w, __uint_as_float(u.x << 16), a.x);
+        a.y = fmaf(w, __uint_as_float(u.x & 0xFFFF0000u), a.y);
+        a.z = fmaf(w, __uint_as_float(u.y << 16), a.z);
+        a.w = fmaf(w, __uint_as_float(u.y & 0xFFFF0000u), a.w);
+        b.x = fmaf(w, __uint_as_float(u.z << 16), b.x);
+        b.y = fmaf(w, __uint_as_float(u.z & 0xFFFF0000u), b.y);
+        b.z = fmaf(w, __uint_as_float(u.w << 16), b.z);
+        b.w = fmaf(w, __uint_as_float(u.w & 0xFFFF0000u), b.w);
+      }
   }
 }
 
@@ -81,8 +99,8 @@ __device__ __forceinline__ float row_rms_scale(const LinEpi& e, int m, int lane)
 }
 
 // One finished row of a 256-column tile, by a warp.  acc(c): the eight (project, stream) or four (gated unit)
-// accumulators from column c on.  sc: the row's scale (project); x0, x1: this lane's eight values of the stream row
-// (stream, when the linear adds to it), fetched by the caller ahead of time.
+// accumulators from column c on.  sc: the row's scale (project); x0, x1: this lane's eight values of the stream row and what
+// joins it (stream, when the linear adds to it), fetched by the caller ahead of time.
 template <typename Acc>
 __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& acc, int m, int tile_n, int lane, float sc, float4 x0, float4 x1) {
   const int n0 = tile_n * 256;
@@ -177,7 +195,6 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
     float* xr = e.x + static_cast<size_t>(m) * e.ldx + n;
     const float4 a = acc(lane * 8), b = acc(lane * 8 + 4);
     float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
-    if (e.y != nullptr) add_routes(e, m, n, v);
     if (e.add) {
       v[0] += x0.x; v[1] += x0.y; v[2] += x0.z; v[3] += x0.w;
       v[4] += x1.x; v[5] += x1.y; v[6] += x1.z; v[7] += x1.w;
@@ -220,8 +237,8 @@ __device__ __forceinline__ void linear_tile_epilogue(const LinEpi& e, const floa
       x[i][0] = x[i][1] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (addx && r < rows) {
         const float4* xr = reinterpret_cast<const float4*>(e.x + static_cast<size_t>(mb + r) * e.ldx + n);
-        x[i][0] = xr[0];
-        x[i][1] = xr[1];
+        x[i][0] = __ldcg(xr);                     // (what joins it may come from the CTA of another part)
+        x[i][1] = __ldcg(xr + 1);
       }
     }
 #pragma unroll
@@ -234,9 +251,34 @@ __device__ __forceinline__ void linear_tile_epilogue(const LinEpi& e, const floa
   }
 }
 
+// The routed rows of a tile join its stream rows in memory while the main loop runs (the epilogue then reads them there).
+__device__ __forceinline__ void linear_tile_routes(const LinEpi& e, int mb, int rows, int tile_n, int w, int lane) {
+  const int n = tile_n * 256 + lane * 8;
+  for (int r0 = w; r0 < rows; r0 += 32) {
+    float4 x[4][2];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      x[i][0] = x[i][1] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (n < e.width && r0 + 8 * i < rows) {
+        const float4* xr = reinterpret_cast<const float4*>(e.x + static_cast<size_t>(mb + r0 + 8 * i) * e.ldx + n);
+        x[i][0] = __ldcg(xr);
+        x[i][1] = __ldcg(xr + 1);
+      }
+    }
+    add_routes(e, mb + r0, rows - r0, n, n < e.width, lane, x);
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (n < e.width && r0 + 8 * i < rows) {
+        float4* xr = reinterpret_cast<float4*>(e.x + static_cast<size_t>(mb + r0 + 8 * i) * e.ldx + n);
+        __stcg(xr, x[i][0]);
+        __stcg(xr + 1, x[i][1]);
+      }
+  }
+}
+
 // kGroup: 0 a plain product, 1 a grouped one, 2 a grouped one whose operand rows are gathered by the epilogue warps
 template <int kMT, int kGroup>
-__global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_constant__ LinParams p, const int stages) {
+__global__ void __launch_bounds__(kLinThreads, 1) lin_bf16_kernel(const __grid_constant__ LinParams p, const int stages) {
   extern __shared__ uint8_t smem_raw[];
   // one round of CTAs: the successor may take the SMs this grid leaves idle or frees (until its own wait it touches
   // weights only)
@@ -290,7 +332,8 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
     // ---------------------------------------------------------------- producer
     if (lane == 0) {
       constexpr bool kCopyA = kGroup != 2;
-      const uint32_t tx = kLinTile + (kCopyA ? abytes : 0u);
+      const uint32_t acopy = kGroup == 0 ? abytes : static_cast<uint32_t>((group.z + 7) & ~7) * 128u;   // a group's own rows
+      const uint32_t tx = kLinTile + (kCopyA ? acopy : 0u);
       const uint64_t pol = gridDim.x > 1 ? l2_policy_evict_normal() : l2_policy_evict_first();
       const uint8_t* wp = static_cast<const uint8_t*>(p.w) + group.x * p.group_w_stride + (static_cast<size_t>(tile_n) * KB + kb0) * kLinTile;
       const uint8_t* ap = static_cast<const uint8_t*>(p.a2 != nullptr && tile_n >= p.a2_tile0 ? p.a2 : p.a) +
@@ -305,7 +348,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
       pdl_wait();
       if constexpr (kCopyA)
         for (int it = 0; it < pre; ++it) {
-          bulk_g2s(a_smem + it * abytes, ap, abytes, bar_full + 8 * it);
+          bulk_g2s(a_smem + it * abytes, ap, acopy, bar_full + 8 * it);
           ap += a_step;
         }
       int issued = pre, s = pre == stages ? 0 : pre;
@@ -315,7 +358,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
         if (!mbar_wait(bar_empty + 8 * s, ph ^ 1u, p.err, kErrWaitEmpty)) { ok = false; break; }
         mbar_arrive_expect_tx(bar_full + 8 * s, tx);
         bulk_g2s_hint(w_smem + s * kLinTile, wp, kLinTile, bar_full + 8 * s, pol);
-        if constexpr (kCopyA) bulk_g2s(a_smem + s * abytes, ap, abytes, bar_full + 8 * s);
+        if constexpr (kCopyA) bulk_g2s(a_smem + s * abytes, ap, acopy, bar_full + 8 * s);
         wp += kLinTile;
         ap += a_step;
         issued = it + 1;
@@ -342,6 +385,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
         const uint64_t b_desc = desc_hi | static_cast<uint64_t>((w_addr & 0x3FFFFu) >> 4);
 #pragma unroll
         for (int j2 = 0; j2 < kMT; ++j2) {
+          if (kGroup != 0 && j2 > 0 && j2 * p.nt >= group.z) break;
           const uint32_t dj = tmem_d + static_cast<uint32_t>(j2) * 256u;
           const uint64_t aj = a_desc + static_cast<uint64_t>(j2) * (static_cast<uint64_t>(p.nt) * 128u >> 4);
           mma_f16_ss(dj, aj, b_desc, idesc, it != 0 ? 1u : 0u);
@@ -366,14 +410,15 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
     const LinEpi& e = p.e;
     pdl_wait();
     if constexpr (kGroup == 2) {
-      // operand rows: up to four 16-byte pieces of every k-block per thread, three k-blocks in flight
-      constexpr int kLag = 2;                     // (below the number of stages)
-      const uint8_t* src[4];
-      uint32_t dst[4];
-      bool live[4];
+      // operand rows: up to 4 kMT 16-byte pieces of every k-block per thread
+      constexpr int kLag = kMT == 2 ? 1 : 2;      // (two below the number of stages: the tensor cores always have a k-block)
+      constexpr int kPieces = 4 * kMT;
+      const uint8_t* src[kPieces];
+      uint32_t dst[kPieces];
+      bool live[kPieces];
       const size_t a_step = static_cast<size_t>(p.M_pad) * 128;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
+      for (int i = 0; i < kPieces; ++i) {
         const int r = (te + 256 * i) >> 3, c = te & 7;
         live[i] = r < group.z;
         const int m = live[i] ? max(p.src_row[m0 + r], 0) : 0;
@@ -392,7 +437,7 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
         if (it >= stages) ok = __all_sync(0xffffffffu, mbar_wait(bar_empty + 8 * s, ph ^ 1u, p.err, kErrWaitEmpty));
         if (!ok) break;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
+        for (int i = 0; i < kPieces; ++i) {
           if (live[i]) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst[i] + s * abytes), "l"(src[i]) : "memory");
           src[i] += a_step;
         }
@@ -419,6 +464,9 @@ __global__ void __launch_bounds__(kLinThreads) lin_bf16_kernel(const __grid_cons
       }
       scale_s[te] = sc;
     }
+    if constexpr (kGroup == 0)
+      if (e.y != nullptr && split == 0)
+        for (int j2 = 0; j2 < kMT; ++j2) linear_tile_routes(e, m0 + j2 * p.nt, min(p.nt, p.M - m0 - j2 * p.nt), tile_n, warp - 2, lane);
     bool ok = mbar_wait(bar_acc, 0, p.err, kErrWaitAcc);
     if (!ok) abort_s = 1u;
     named_bar_sync(1, 256);
@@ -680,6 +728,8 @@ extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t strea
   using namespace saber;
   const LinEpi& e = p->e;
   if (p->M <= 0 || (p->N_pad & 255) || (p->K & 63) || p->K <= 0 || (p->M > p->M_pad && p->group_tiles == nullptr)) return static_cast<int>(cudaErrorInvalidValue);
+  if (e.y != nullptr && (!e.stream || !e.add || e.routes < 1 || e.routes > 32 || e.slot_of == nullptr || e.route_w == nullptr || e.y_f32 != p->fp32 || (e.ldy & 7)))
+    return static_cast<int>(cudaErrorInvalidValue);
   if (e.stream ? (e.width > p->N_pad || (e.ldx & 31) || e.x == nullptr)
                : (e.n_plain > e.act_tile0 * 256 || e.act_tile0 * 256 > p->N_pad || (e.ldo & 3)))
     return static_cast<int>(cudaErrorInvalidValue);
@@ -716,11 +766,14 @@ extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t strea
     cudaError_t r = cudaFuncSetAttribute(lin_bf16_kernel<1, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
     if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<2, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
     if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<1, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<2, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<2, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
     if (r == cudaSuccess) r = cudaFuncSetAttribute(lin_bf16_kernel<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
     if (r != cudaSuccess) return static_cast<int>(r);
     ready[dev] = true;
   }
-  const bool pair = !grouped && p->mtiles == 2 && p->splits == 1 && p->nt == 128 && (p->M_pad / 128) % 2 == 0;
+  const bool pair = p->mtiles == 2 && p->splits == 1 && p->nt == 128 && (grouped || (p->M_pad / 128) % 2 == 0);
+  if (grouped && p->mtiles == 2 && !pair) return static_cast<int>(cudaErrorInvalidValue);      // (the table's tiles would not fit)
   const int abytes = p->nt * 128 * (pair ? 2 : 1);
   int stages = (kSmem - 1024) / (static_cast<int>(kLinTile) + abytes);
   if (stages > kLinMaxStages) stages = kLinMaxStages;
@@ -728,10 +781,11 @@ extern "C" int saber_linear_launch(const saber::LinParams* p, cudaStream_t strea
   const int tiles_m = pair ? (p->M + 255) / 256 : (p->M + p->nt - 1) / p->nt;
   const dim3 grid(tiles_m, p->N_pad / 256, p->splits);
   const dim3 ggrid(grouped ? p->group_max : 1, p->N_pad / 256, 1);
-  cudaError_t r = grouped && p->src_row ? launch(lin_bf16_kernel<1, 2>, ggrid, dim3(kLinThreads), smem, stream, 2, q, stages)
-                  : grouped             ? launch(lin_bf16_kernel<1, 1>, ggrid, dim3(kLinThreads), smem, stream, 2, q, stages)
-                  : pair                ? launch(lin_bf16_kernel<2, 0>, grid, dim3(kLinThreads), smem, stream, 2, q, stages)
-                                        : launch(lin_bf16_kernel<1, 0>, grid, dim3(kLinThreads), smem, stream, 2, q, stages);
+  auto go = [&](auto kernel, const dim3& g) { return launch(kernel, g, dim3(kLinThreads), smem, stream, 2, q, stages); };
+  cudaError_t r;
+  if (grouped && p->src_row) r = pair ? go(lin_bf16_kernel<2, 2>, ggrid) : go(lin_bf16_kernel<1, 2>, ggrid);
+  else if (grouped) r = pair ? go(lin_bf16_kernel<2, 1>, ggrid) : go(lin_bf16_kernel<1, 1>, ggrid);
+  else r = pair ? go(lin_bf16_kernel<2, 0>, grid) : go(lin_bf16_kernel<1, 0>, grid);
   if (r != cudaSuccess || p->fuse) return static_cast<int>(r);
   return static_cast<int>(launch(lin_epi_kernel, dim3(p->M), dim3(256), 0, stream, 0, *p));
 }

@@ -58,7 +58,7 @@ struct LinEpi {
 };
 
 // group_tiles: a grouped product.  Row tile i is {expert, first row, rows}: rows of the (expert-major) output, each tile
-// against the weight rows of its expert (group_w_stride bytes apart), at most nt rows (fp32: 64).  group_rows: the token of every
+// against the weight rows of its expert (group_w_stride bytes apart), at most nt mtiles rows (fp32: 64).  group_rows: the token of every
 // output row, -1 between the experts' rows.  src_row: the same array where the operand's (and ss's) rows are tokens; null: they
 // lie in output order.
 struct LinParams {

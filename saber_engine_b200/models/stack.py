@@ -139,7 +139,7 @@ class StackModel:
         p, sc = N.LinParams(), self.scratch
         p.w, p.a, p.err, p.counters = lin.w.data_ptr(), a.data_ptr(), sc.err.data_ptr(), sc.counters.data_ptr()
         p.ws = (ws if ws is not None else sc.ws).data_ptr()
-        p.M, p.M_pad, p.N_pad, p.K, p.splits, p.mtiles = ew["rows"], a_rows, lin.N_pad, lin.K, 1, 1
+        p.M, p.M_pad, p.N_pad, p.K, p.splits, p.mtiles = ew["rows"], a_rows, lin.N_pad, lin.K, 1, ew["mtiles"]
         p.nt, p.fp32, p.fuse = ew["nt"], int(self.f32), int(self.fuse)
         p.group_tiles, p.group_ntiles, p.group_rows, p.group_max = (*(ew[k].data_ptr() for k in ("tiles", "ntiles", "src_row")), ew["max_tiles"])
         p.src_row = ew["src_row"].data_ptr() if gather else None
@@ -303,12 +303,16 @@ class StackModel:
             return {}
         dev, W = self.device, self.cfg.width
         i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=dev)       # noqa: E731
-        nt = 64 if self.f32 else L.token_tile(M)
+        nt, mtiles = 64 if self.f32 else L.token_tile(M), 1
+        if nt == 128 and M * max(f.top for f in ms) > 96 * max(f.experts for f in ms):     # a weight tile for 256 rows
+            mtiles = 2
+        tile = nt * mtiles
         per = [(M * f.top, min(f.experts, M * f.top)) for f in ms]            # routes, experts that can have one
         rows = L.round_up(max(r + 15 * e for r, e in per), 16)
-        pad = rows + 128                                                      # (a tile's copies may run past the live rows)
+        pad = L.round_up(rows, 128)
         top, E, ff = max(f.top for f in ms), max(f.experts for f in ms), max(L.round_up(f.ff, 64) for f in ms)
-        return {"nt": nt, "rows": rows, "pad": pad, "max_tiles": max(e + r // nt for r, e in per), "tiles": i32(max(e + r // nt for r, e in per), 4),
+        most = max(e + r // tile for r, e in per)
+        return {"nt": nt, "mtiles": mtiles, "rows": rows, "pad": pad, "max_tiles": most, "tiles": i32(most, 4),
                 "ntiles": i32(2), "src_row": i32(pad), "topk_id": i32(M * top), "slot_of": i32(M * top), "counts": i32(E), "offsets": i32(E + 1), "cursors": i32(E),
                 "topk_w": torch.zeros(M * top, dtype=torch.float32, device=dev), "act": torch.zeros(pad * ff, dtype=self.dtype, device=dev),
                 "y": torch.zeros(rows * L.round_up(W, 8), dtype=self.dtype, device=dev)}
@@ -319,7 +323,7 @@ class StackModel:
         p.logits_f32, p.ld, p.M, p.E, p.top_k = proj.data_ptr() + 4 * lw.off["router"], proj.stride(0), M, f.experts, f.top
         p.topk_id, p.topk_w, p.counts, p.offsets, p.cursors, p.tiles, p.ntiles, p.src_row, p.slot_of = \
             (ew[k].data_ptr() for k in ("topk_id", "topk_w", "counts", "offsets", "cursors", "tiles", "ntiles", "src_row", "slot_of"))
-        p.nt, p.rows_cap, p.e_lo, p.e_n, p.live, p.groups, p.keep = ew["nt"], ew["src_row"].numel(), 0, f.experts, live, f.groups, f.keep
+        p.nt, p.rows_cap, p.e_lo, p.e_n, p.live, p.groups, p.keep = ew["nt"] * ew["mtiles"], ew["src_row"].numel(), 0, f.experts, live, f.groups, f.keep
         prog.add_moe_route(p, tag=f"{tag}.route")
         e = N.LinEpi()
         self._row_norm(e, ss)

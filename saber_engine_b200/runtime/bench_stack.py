@@ -1,5 +1,6 @@
 """Throughput of a layer-by-layer model beside its closest relatives at equal layer sizes: Renosun beside the int4
-hybrid decoder, Tepavik beside Renosun and the hybrid decoder.
+hybrid decoder, Tepavik beside Renosun and the hybrid decoder, Fitatar beside Tepavik (grouped-query attention), Renosun (latent
+attention) and the hybrid decoder with a mixture of experts.
 
 Prefill: a cold prompt in portions of one rung (device-timed).  Decode: `streams` sequences at the prompt's length,
 one row each (no drafter on either side).  Then every group of launches of one step on its own: the group's
@@ -17,10 +18,11 @@ import torch
 from ..models import config as C
 from ..models.hybrid import HybridModel
 from ..models.stack import StackModel
-from ..models.stack_config import (ClampedGlu, DeltaMixer, GroupedMixer, LatentMixer, LayerSpec, OuterMixer, Rotation, StackConfig)
+from ..models.stack_config import (ClampedGlu, DeltaMixer, GroupedMixer, ExpertMix, LatentMixer, LayerSpec, OuterMixer, Rotation, SquaredRelu,
+                                   StackConfig)
 from ..models.step import SeqStep, run_bucket
 
-SIZES = ("renosun-2k", "renosun-4k", "renosun-5k", "tepavik-2k", "tepavik-4k", "tepavik-5k")
+SIZES = ("renosun-2k", "renosun-4k", "renosun-5k", "tepavik-2k", "tepavik-4k", "tepavik-5k", "fitatar-2k", "fitatar-4k", "fitatar-5k")
 
 
 def peaks() -> tuple:
@@ -32,7 +34,21 @@ def peaks() -> tuple:
 
 
 def like_models(cfg: StackConfig) -> list:
-    return [like_hybrid(cfg)] if cfg.arch == "Renosun" else [like_renosun(cfg), like_hybrid(cfg)]
+    makers = {"Renosun": [like_hybrid], "Tepavik": [like_renosun, like_hybrid], "Fitatar": [like_tepavik, like_renosun, like_hybrid]}[cfg.arch]
+    return [make(cfg) for make in makers]
+
+
+def experts_of(cfg: StackConfig):
+    return next((l.mlp for l in cfg.layers if isinstance(l.mlp, ExpertMix)), None)
+
+
+def like_tepavik(cfg: StackConfig) -> StackConfig:
+    """Tepavik attention layers only, over every earlier key, with the same heads; the feed-forward as wide as what a token meets."""
+    a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, GroupedMixer))
+    f = experts_of(cfg)
+    l = LayerSpec(GroupedMixer(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, 30.0, 0), SquaredRelu(f.top * f.ff + f.shared))
+    return StackConfig(f"tepavik-like-{cfg.name}", "Tepavik", vocab=cfg.vocab, width=cfg.width, layers=(l,) * len(cfg.layers), parallel=False,
+                       norm_offset=1.0, max_ctx=cfg.max_ctx)
 
 
 def like_renosun(cfg: StackConfig) -> StackConfig:
@@ -43,19 +59,20 @@ def like_renosun(cfg: StackConfig) -> StackConfig:
     d = LayerSpec(DeltaMixer(a.heads, a.heads // 2, 128, 128, 4), mlp)
     la = LayerSpec(LatentMixer(a.heads, 128, 64, 128, 512, 192 ** -0.5, Rotation(1e6, 64)), mlp)
     return StackConfig(f"renosun-like-{cfg.name}", "Renosun", vocab=cfg.vocab, width=cfg.width,
-                       layers=tuple(la if isinstance(l.mixer, GroupedMixer) else d for l in cfg.layers), max_ctx=cfg.max_ctx)
+                       layers=tuple(la if isinstance(l.mixer, LatentMixer if cfg.arch == "Fitatar" else GroupedMixer) else d for l in cfg.layers),
+                       max_ctx=cfg.max_ctx)
 
 
 def like_hybrid(cfg: StackConfig) -> C.HybridConfig:
-    """The hybrid decoder with the same width, feed-forward, recurrent heads of 128 and number of layer runs; its gated GQA
+    """The hybrid decoder with the same width, feed-forward or experts, recurrent heads of 128 and number of layer runs; its gated GQA
     attention has the same query width in heads of 256 and a quarter as many key heads."""
     a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, (LatentMixer, GroupedMixer)))
     d = next((l.mixer for l in cfg.layers if isinstance(l.mixer, DeltaMixer)), None)
     kh, vh, ff = (d.kv_heads, d.heads, cfg.layers[0].mlp.ff) if d else (a.heads // 2, a.heads, cfg.layers[0].mlp.ff * 2 // 3 // 256 * 256)
-    nq = max(4, a.heads * a.dim // 256)
+    nq, f = max(4, a.heads * a.dim // 256), experts_of(cfg)
     return C.HybridConfig(name=f"hybrid-like-{cfg.name}", n_layers=len(cfg.runs), hidden=cfg.width, n_q_heads=nq, n_kv_heads=max(1, nq // 4),
                           head_dim=256, ffn_inter=ff, vocab=cfg.vocab, gdn_k_heads=kh, gdn_v_heads=vh,
-                          gdn_head_dim=128, max_ctx=cfg.max_ctx)
+                          gdn_head_dim=128, max_ctx=cfg.max_ctx, moe=None if f is None else C.MoEConfig(f.experts, f.top, f.ff, f.shared, True))
 
 
 def mixer_name(m) -> str:
@@ -72,17 +89,21 @@ def _groups(model, b) -> dict:
         for i, t in enumerate(tags):
             part = t.split(".")
             if part[0][0] == "R" and part[0][1:].isdigit() and part[-1] != "digest":
-                m = model.cfg.layers[int(part[1][1:])].mixer
-                label = part[2] if part[2] in ("project", "out", "up", "down", "loop_in") else "mixer"
-                key = label if label in ("up", "down", "loop_in") else f"{label}:{mixer_name(m)}"
+                spec = model.cfg.layers[int(part[1][1:])]
+                alone = ("up", "down", "loop_in", "carry", "route", "experts_up", "experts_down")
+                label = part[2] if part[2] in ("project", "out", *alone) else "mixer"
+                key = label if label in alone else f"{label}:{mixer_name(spec.mixer)}" + ("+experts" if label != "mixer" and isinstance(spec.mlp, ExpertMix) else "")
                 out.setdefault(key, []).append((i, i + 1))
             elif t == "lm_head":
                 out["lm_head"] = [(i, i + 1)]
         return out
     layers = sorted({int(t[1:].split(".")[0]) for t in tags if t[0] == "L" and t[1].isdigit()})
     span = lambda li, keys: [i for i, t in enumerate(tags) if t.startswith(f"L{li}.") and any(k in t for k in keys)]   # noqa: E731
+    moe = model.cfg.moe is not None
     spec = {"delta": ("gdn.conv", "gdn.rec", "gdn.norm", "gdn.step"), "attention": ("attn.rope", "attn.core", "attn.gate", "attn.quant"),
-            "linears": ("in_norm", "in_proj", "attn.qkv", "out_proj", "o_proj", "post_norm", "mlp")}
+            "linears": ("in_norm", "in_proj", "attn.qkv", "out_proj", "o_proj", "post_norm", *(() if moe else ("mlp",)))}
+    if moe:
+        spec["experts"] = (".moe.",)
     for g, keys in spec.items():
         out[g] = []
         for li in layers:
@@ -125,14 +146,25 @@ def _roof(nbytes: float, flops: float) -> float:
 
 def stack_costs(cfg: StackConfig, M: int, nseq: int, ctx_pairs: float, ctx_tokens: float) -> dict:
     """Algorithmic (bytes, FLOPs) per launch group.  ctx_pairs: visible (row, key) pairs; ctx_tokens: keys read."""
-    W, out = cfg.width, {"loop_in": (4 * cfg.width ** 2 + M * 10 * cfg.width, 4.0 * M * cfg.width ** 2)}
+    W, head_rows = cfg.width, min(M, 8)
+    out = {"loop_in": (4 * cfg.width ** 2 + M * 10 * cfg.width, 4.0 * M * cfg.width ** 2)}
     for l in cfg.layers:
-        m, ff = l.mixer, l.mlp.ff
-        name = mixer_name(m)
-        segs = sum(n for _, n in m.segments())
-        n, k = (segs + 2 * ff, m.out_features + ff) if cfg.parallel else (segs, m.out_features)
-        out[f"project:{name}"] = (2 * n * W + M * (2 * W + 4 * segs + (2 * ff if cfg.parallel else 0)), 2.0 * M * n * W)
-        out[f"out:{name}"] = (2 * k * W + M * (2 * k + 8 * W + 2 * W), 2.0 * M * k * W)
+        m, ff, f = l.mixer, l.mlp.inner, l.mlp
+        name, mix = mixer_name(m), isinstance(f, ExpertMix)
+        tail = "+experts" if mix else ""
+        segs = sum(n for _, n in m.segments()) + (f.experts if mix else 0)
+        up_rows = ff * (2 if isinstance(f, ClampedGlu) else 1)
+        n, k = (segs + up_rows, m.out_features + ff) if cfg.parallel else (segs, m.out_features)
+        ops = 2 if cfg.two_norms else 1                        # operands of the stream
+        out[f"project:{name}{tail}"] = (2 * n * W + M * (2 * W * ops + 4 * segs + (2 * ff if cfg.parallel else 0)), 2.0 * M * n * W)
+        out[f"out:{name}{tail}"] = (2 * k * W + M * (2 * k + 8 * W + 2 * W * ops + (2 * f.top * W if mix else 0)), 2.0 * M * k * W)
+        if mix:
+            routes, met = M * f.top, f.experts * (1 - (1 - f.top / f.experts) ** M)       # experts that some token chooses, choices alike
+            out["route"] = (M * (4 * f.experts + 16 * f.top), 0.0)
+            out["experts_up"] = (2 * met * f.ff * W + M * 2 * W + routes * 2 * f.ff, 2.0 * routes * f.ff * W)
+            out["experts_down"] = (2 * met * f.ff * W + routes * 2 * (f.ff + W), 2.0 * routes * f.ff * W)
+        if m.q_rank:
+            out["carry"] = (2 * m.q_rank * m.query_rows + M * (2 * m.q_rank + 4 * m.query_rows), 2.0 * M * m.q_rank * m.query_rows)
         out["up"] = (2 * ff * W + M * (2 * W + 2 * ff), 2.0 * M * ff * W)
         out["down"] = (2 * ff * W + M * (2 * ff + 8 * W + 2 * W), 2.0 * M * ff * W)
         if isinstance(m, (DeltaMixer, OuterMixer)):
@@ -148,7 +180,7 @@ def stack_costs(cfg: StackConfig, M: int, nseq: int, ctx_pairs: float, ctx_token
                 pair = 2.0 * m.heads * (2 * m.kv_rank + m.rot_dim)
             out[f"mixer:{name}"] = (2 * ctx_tokens * (m.kv_rank + m.rot_dim) + 2 * m.heads * (m.dim + m.vdim) * m.kv_rank
                                     + M * (4 * m.heads * (m.dim + m.rot_dim + m.vdim) + 2 * m.heads * m.vdim), ctx_pairs * pair + carry)
-    out["lm_head"] = (2 * cfg.vocab * W, 2.0 * min(M, 8) * cfg.vocab * W)
+    out["lm_head"] = (2 * cfg.vocab * W, 2.0 * head_rows * cfg.vocab * W)
     return out
 
 
@@ -158,6 +190,13 @@ def hybrid_costs(cfg: C.HybridConfig, M: int, nseq: int, ctx_pairs: float, ctx_t
     lin = H * (sh.gdn_in_n + 2 * sh.ffn_inter) + H * (sh.gdn_out_k + sh.ffn_inter)
     out = {"linears": (0.5 * lin + M * (2 * sh.gdn_in_n + sh.gdn_out_k + sh.ffn_inter + 12 * H), 2.0 * M * lin)}
     out["delta"] = (2 * 4 * nseq * sh.gdn_v_heads * D * D + M * (2 * sh.gdn_in_n + sh.gdn_out_k), M * sh.gdn_v_heads * D * D * 8.0)
+    if cfg.moe is not None:
+        f = cfg.moe
+        met, mats = f.n_experts * (1 - (1 - f.top_k / f.n_experts) ** M), 3 * f.expert_inter * H
+        lin -= 3 * H * sh.ffn_inter
+        out["linears"] = (0.5 * lin + M * (2 * sh.gdn_in_n + sh.gdn_out_k + 12 * H), 2.0 * M * lin)
+        out["experts"] = (0.5 * (met * mats + 3 * f.shared_inter * H) + f.n_experts * H + M * f.top_k * (2 * H + 2 * 4 * f.expert_inter + 2 * H) + M * 4 * H,
+                          2.0 * M * (f.top_k * mats + 3 * f.shared_inter * H))
     out["attention"] = (2 * ctx_tokens * sh.n_kv_heads * cfg.head_dim + M * (2 * sh.qkv_n + sh.o_k), ctx_pairs * 4.0 * sh.n_q_heads * cfg.head_dim)
     return out
 

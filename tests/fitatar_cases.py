@@ -55,10 +55,10 @@ CASES = {
 
 
 def _chosen_apart(z, f, margin):
-    """Whether the expert choice of router logits z [E] would survive a disturbance of `margin` of their spread."""
+    """Whether the expert choice of router logits z [E] would survive a disturbance of `margin` of the largest of them."""
     r = f["router"]
     g, size = r["groups"]["count"], r["experts"] // r["groups"]["count"]
-    m = margin * float(z.std()) if len(z) > 1 else 0.0
+    m = margin * float(z.abs().max())
     best = z.view(g, size).max(1).values
     order = torch.argsort(best, descending=True)
     if r["groups"]["keep"] < g and best[order[r["groups"]["keep"] - 1]] - best[order[r["groups"]["keep"]]] < m:
@@ -96,6 +96,6 @@ def tensors(cfg: dict, seed: int = 0, code: int = 12) -> dict:
     routers = [(out[f"l{i}.mlp.router"].double()[:, :code] * out[f"l{i}.norm2"].double()[:code], l["mlp"]) for i, l in enumerate(cfg["layers"])
                if l["mlp"] and l["mlp"]["kind"] == "moe"]
     for v in range(cfg["vocab"] if routers else 0):
-        while not all(_chosen_apart(w @ out["embed"][v, :code].double(), f, 0.04) for w, f in routers):
+        while not all(_chosen_apart(w @ out["embed"][v, :code].double(), f, 0.02) for w, f in routers):
             out["embed"][v, :code] = torch.randn(code, generator=g).to(torch.bfloat16)
     return out

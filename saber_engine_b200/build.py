@@ -27,7 +27,7 @@ NVCC_FLAGS = [
 ]
 # Sources whose results are held to fp32 accuracy: CUDA's accurate math functions, IEEE division and
 # square root, denormals kept.
-PRECISE = {"linear.cu", "moe.cu", "delta.cu", "mla.cu", "mla_mma.cu", "flash_tc.cu", "gqa.cu", "ssd.cu", "ssd_chunk.cu"}
+PRECISE = {"linear.cu", "moe.cu", "delta.cu", "mla.cu", "mla_mma.cu", "flash_tc.cu", "gqa.cu", "ssd.cu", "ssd_chunk.cu", "cdelta.cu", "join.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-march=x86-64-v3"]
 
 

@@ -22,10 +22,12 @@
 
 #include "../comm/comm.h"
 #include "../kernels/attn.h"
+#include "../kernels/cdelta.h"
 #include "../kernels/delta.h"
 #include "../kernels/gdn.h"
 #include "../kernels/gemm_i8.h"
 #include "../kernels/gqa.h"
+#include "../kernels/join.h"
 #include "../kernels/linear.h"
 #include "../kernels/mla.h"
 #include "../kernels/moe.h"
@@ -71,12 +73,14 @@ struct OpDelta { saber::DeltaParams p; int single_row; };
 struct OpMla { saber::MlaParams p; };
 struct OpSsd { saber::SsdParams p; int single_row; };
 struct OpGqa { saber::GqaParams p; };
+struct OpCdelta { saber::CdeltaParams p; int single_row; };
+struct OpJoin { saber::JoinParams p; };
 struct OpMoeGather { const int8_t* q; const float* scale; int M_pad; const int32_t* src_row; const int32_t* ntiles;
                      int8_t* q_out; float* scale_out; int rows_cap, M_pad_out, K, to_fp8; };
 
 using Op = std::variant<OpGemm, OpRow, OpEmbed, OpGdnConv, OpGdnRec, OpRope, OpAttn, OpArgmax,
                         OpSeam, OpVerify, OpMemset, OpCopy, OpAllReduce, OpExpand, OpAdvance, OpPickMerge, OpMoeRoute, OpMoeCombine, OpMoeGather, OpDigest, OpDigestClear, OpGdnChunk, OpLogitGather, OpSampleSeam, OpGdnStep, OpSeamMerge, OpDraftIndex,
-                        OpLinear, OpStreamEmbed, OpStreamNorm, OpDelta, OpMla, OpSsd, OpGqa>;
+                        OpLinear, OpStreamEmbed, OpStreamNorm, OpDelta, OpMla, OpSsd, OpGqa, OpCdelta, OpJoin>;
 
 struct Entry {
   Op op;
@@ -140,6 +144,8 @@ int launch(const Op& op, cudaStream_t s) {
         else if constexpr (std::is_same_v<T, OpMla>) return saber_mla_launch(&o.p, s);
         else if constexpr (std::is_same_v<T, OpSsd>) return saber_ssd_launch(&o.p, o.single_row, s);
         else if constexpr (std::is_same_v<T, OpGqa>) return saber_gqa_launch(&o.p, s);
+        else if constexpr (std::is_same_v<T, OpCdelta>) return saber_cdelta_launch(&o.p, o.single_row, s);
+        else if constexpr (std::is_same_v<T, OpJoin>) return saber_join_launch(&o.p, s);
         else if constexpr (std::is_same_v<T, OpMoeGather>)
           return saber_moe_gather_launch(o.q, o.scale, o.M_pad, o.src_row, o.ntiles, o.q_out, o.scale_out, o.rows_cap,
                                          o.M_pad_out, o.K, o.to_fp8, s);
@@ -308,6 +314,12 @@ int saber_program_add_mla(void* h, const saber::MlaParams* p, const char* tag) {
 }
 int saber_program_add_ssd(void* h, const saber::SsdParams* p, int single_row, const char* tag) {
   return add(h, OpSsd{*p, single_row}, saber_ssd_launches(p, single_row), tag);
+}
+int saber_program_add_cdelta(void* h, const saber::CdeltaParams* p, int single_row, const char* tag) {
+  return add(h, OpCdelta{*p, single_row}, saber_cdelta_launches(single_row), tag);
+}
+int saber_program_add_join(void* h, const saber::JoinParams* p, const char* tag) {
+  return add(h, OpJoin{*p}, 1, tag);
 }
 int saber_program_add_gqa(void* h, const saber::GqaParams* p, const char* tag) {
   return add(h, OpGqa{*p}, saber_gqa_launches(p), tag);

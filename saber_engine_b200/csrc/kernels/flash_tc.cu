@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
   const int m0 = r0 + qt * 128, rows = min(128, nrows - qt * 128);
   const int pos0 = p.kv_len[j] - nrows + qt * 128;                  // position of the tile's first row
   const int keys = pos0 + rows;
-  const int first = p.chunk > 0 ? pos0 - pos0 % p.chunk : 0;        // first key any row of the tile sees
+  const int first = first_key(pos0, p.chunk, p.window);             // first key any row of the tile sees
   const int b0 = first / kTcKeys, blocks = (keys + kTcKeys - 1) / kTcKeys - b0;
   const uint32_t q_s = (smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t kbytes = static_cast<uint32_t>(KB) * 16384u, vbytes = static_cast<uint32_t>(VP) * 256u;
@@ -190,8 +190,8 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
     }
     // (a row may meet blocks ahead of its first key: the maximum starts finite so that differences stay numbers)
     float mx = kTcNone, used = kTcNone, l = 0.f;
-    const int low = p.chunk > 0 ? (pos0 + row) - (pos0 + row) % p.chunk : 0;   // first key of this row
-    const int low_last = p.chunk > 0 ? (pos0 + q4 * 32 + 31) - (pos0 + q4 * 32 + 31) % p.chunk : 0;
+    const int low = first_key(pos0 + row, p.chunk, p.window);       // first key of this row
+    const int low_last = first_key(pos0 + q4 * 32 + 31, p.chunk, p.window);
     // A wait that runs out ends both warps of a row: the one that gives up arrives at their next meeting without waiting.
     auto give_up = [&]() {
       abort_s[q4] = 1u;
@@ -306,7 +306,7 @@ __global__ void __launch_bounds__(kTcThreads) flash_tc_kernel(const __grid_const
       const bool live = row < rows;
       float den = half_s[blocks & 1][0][row] + half_s[blocks & 1][1][row];
       if (p.sink != nullptr) den += ex2(p.sink[h] * kTcLog2e - used * sc);        // (infinite: the sink takes everything)
-      float inv = 1.f / den;
+      float inv = p.out_scale / den;
       const float* g = p.gate == nullptr ? nullptr : p.gate + static_cast<size_t>(live ? m : m0) * p.ldg + (p.gate_heads ? h : h * p.V);
       if (g != nullptr && p.gate_heads) {
         inv /= 1.f + expf(-g[0]);

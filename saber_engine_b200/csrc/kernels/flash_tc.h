@@ -22,6 +22,8 @@ struct FlashParams {
   int out_k0;
   int nseq, H, G, DK, V, VP, n_blocks, max_blocks, max_rows;
   int chunk;                  // > 0: a row sees the keys of its own chunk of positions only
+  int window;                 // > 0: a row sees the last `window` keys only, its own among them
+  float out_scale;
   float scale, softcap;       // softcap > 0: scores cap tanh(scale s / cap)
   float bound;                // no |q . k| is larger (0: not known)
   uint32_t* err;

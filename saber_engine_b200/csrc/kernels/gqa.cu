@@ -1,5 +1,7 @@
 // Grouped-query attention over tiled pages.
 //
+//   conv     where q, k and v pass a convolution: the convolved rows with the weights of q and k, their sums of squares, normed
+//            values; the kernels behind it read these rows instead of the projections
 //   append   keys (normed) and values of this step's rows into their pages; for the tcgen05 form also the queries
 //   form 2   flash_tc.cu: prompt portions
 //   form 1   decoding and short portions: the query heads of a key head are the rows of an `mma.sync` tile, pages arrive
@@ -36,8 +38,13 @@ template <> struct Page<float> {
 __device__ __forceinline__ size_t page_block(const GqaParams& p, int page, int g) {
   return (static_cast<size_t>(page) * p.G + g) * kPage * (p.KP + p.VP);
 }
-// reciprocal root mean square of D values (a warp), 1 without the norm
-__device__ __forceinline__ float head_scale(const GqaParams& p, const float* x, int lane) {
+// which of row m's two sums of squares over all heads belongs to x's part
+__device__ __forceinline__ float row_scale(const GqaParams& p, int m, int isk) {
+  return 1.f / sqrtf(p.row_ss[2 * m + isk] / static_cast<float>((isk ? p.G : p.H) * p.D) + p.eps);
+}
+// reciprocal root mean square of the D values of a head of row m (a warp), 1 without the norm
+__device__ __forceinline__ float head_scale(const GqaParams& p, const float* x, int m, int isk, int lane) {
+  if (p.taps > 0) return row_scale(p, m, isk);
   if (!p.qk_norm) return 1.f;
   float sq = 0.f;
   for (int d = lane; d < p.D; d += 32) sq = fmaf(x[d], x[d], sq);
@@ -45,14 +52,109 @@ __device__ __forceinline__ float head_scale(const GqaParams& p, const float* x, 
 }
 
 __device__ __forceinline__ float gated(const GqaParams& p, int m, int h, int v, float y) {
-  if (p.g_off < 0) return y;
-  return y / (1.f + expf(-p.x[static_cast<size_t>(m) * p.ldx + p.g_off + h * p.V + v]));
+  y *= p.out_scale;
+  if (p.gate == nullptr) return y;
+  return y / (1.f + expf(-p.gate[static_cast<size_t>(m) * p.ld_gate + h * p.V + v]));
 }
 
-// Four rows of a head from x on (rows past n repeat the last), divided by their root mean square and rotated by the tables
+// slot of a sequence (< 0: none)
+__device__ __forceinline__ int gqa_slot(const GqaParams& p, int j) {
+  const int s = p.slots[j];
+  if (s >= p.n_slots) {
+    if (p.err) atomicCAS(p.err, 0u, static_cast<uint32_t>(kErrBadIndex));
+    return -1;
+  }
+  return s;
+}
+struct ConvChannels {                             // q | k | v
+  int nq, nk, nv;
+  __device__ __forceinline__ explicit ConvChannels(const GqaParams& p) : nq(p.H * p.D), nk(p.G * p.D), nv(p.G * p.V) {}
+  __device__ __forceinline__ int all() const { return nq + nk + nv; }
+  __device__ __forceinline__ int column(const GqaParams& p, int c) const { return c < nq ? p.rq_off + c : c < nq + nk ? p.rk_off + c - nq : p.rv_off + c - nq - nk; }
+};
+
+// The last rows of sequence j become the ring's (they are the inputs of the next portion's first convolutions).
+__device__ __forceinline__ void conv_ring(const GqaParams& p, int j) {
+  const int r0 = p.cu_rows[j], n = p.cu_rows[j + 1] - r0, slot = n > 0 ? gqa_slot(p, j) : -1;
+  if (slot < 0) return;
+  const ConvChannels ch(p);
+  float* hist = p.hist + static_cast<size_t>(slot) * p.taps * ch.all();
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ch.all(); c += gridDim.y * blockDim.x)
+    for (int t = max(0, n - p.taps); t < n; ++t)
+      hist[static_cast<size_t>(p.pos[r0 + t] % p.taps) * ch.all() + c] = p.raw[static_cast<size_t>(r0 + t) * p.ld_raw + ch.column(p, c)];
+}
+
+constexpr int kConvThreads = 512;
+
+// grid M, 512 threads: a row.  Columns of cx from x = q, k_off = k, v_off = v on (as the kernels behind it read them).
+__global__ void __launch_bounds__(kConvThreads) gqa_conv_kernel(const __grid_constant__ GqaParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[2][kConvThreads / 32];
+  const int m = blockIdx.x, j = mla_seq_of_row(p.cu_rows, p.nseq, m), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (j < 0) return;
+  const int slot = gqa_slot(p, j), t = m - p.cu_rows[j], pos = p.pos[m];
+  const ConvChannels ch(p);
+  const int C = ch.all();
+  float* hist = slot < 0 ? nullptr : p.hist + static_cast<size_t>(slot) * p.taps * C;
+  const float* raw = p.raw + static_cast<size_t>(m) * p.ld_raw;
+  auto conv = [&](int c) {
+    const int col = ch.column(p, c);
+    const float* w = p.conv_w + static_cast<size_t>(c) * p.taps;
+    const float x = raw[col];
+    float s = x * w[p.taps - 1];
+    for (int back = 1; back < p.taps; ++back) {
+      float u = 0.f;
+      if (back <= t) u = raw[col - static_cast<ptrdiff_t>(back) * p.ld_raw];
+      else if (back <= pos && hist != nullptr) u = hist[static_cast<size_t>((pos - back) % p.taps) * C + c];
+      s = fmaf(u, w[p.taps - 1 - back], s);
+    }
+    if (p.max_rows == 1 && hist != nullptr) hist[static_cast<size_t>(pos % p.taps) * C + c] = x;    // (no token of this step reads that row)
+    return s;
+  };
+  float* o = p.cx + static_cast<size_t>(m) * p.ldc;
+  float sq[2] = {0.f, 0.f};
+#pragma unroll
+  for (int isk = 0; isk < 2; ++isk) {
+    const int n = isk ? ch.nk : ch.nq, first = isk ? ch.nq : 0;
+    const float* w = isk ? p.k_w : p.q_w;
+    float* d = o + (isk ? p.k_off : p.q_off);
+#pragma unroll 4
+    for (int c = threadIdx.x; c < n; c += kConvThreads) {
+      const float s = conv(first + c);
+      sq[isk] = fmaf(s, s, sq[isk]);
+      d[c] = s * w[c];
+    }
+  }
+  for (int g = warp; g < p.G; g += kConvThreads / 32) {
+    float s2 = 0.f;
+    float* d = o + p.v_off + g * p.V;
+    for (int v = lane; v < p.V; v += 32) {
+      const float s = conv(ch.nq + ch.nk + g * p.V + v);
+      s2 = fmaf(s, s, s2);
+      d[v] = s;
+    }
+    if (!p.v_norm) continue;
+    s2 = 1.f / sqrtf(mla_warp_sum(s2) / static_cast<float>(p.V) + p.eps);
+    for (int v = lane; v < p.V; v += 32) d[v] *= s2;
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    sq[i] = mla_warp_sum(sq[i]);
+    if (lane == 0) red[i][warp] = sq[i];
+  }
+  __syncthreads();
+  if (threadIdx.x < 2) {
+    float s = 0.f;
+    for (int w = 0; w < kConvThreads / 32; ++w) s += red[threadIdx.x][w];
+    p.row_ss[2 * m + threadIdx.x] = s;
+  }
+}
+
+// Four rows of a head from x on, the first of them row m (rows past n repeat the last), divided by their root mean square and rotated by the tables
 // at t (rot floats a row); put(row, d, four values) takes the pieces.  D a multiple of 4, at most 256; rot a multiple of 8.
 template <typename Put>
-__device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x, int n, int lane, const float* t, const Put& put) {
+__device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x, int n, int m, int isk, int lane, const float* t, const Put& put) {
   float4 v[4][2];
   float sq[4];
 #pragma unroll
@@ -64,12 +166,12 @@ __device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x,
     }
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
-    if (!p.qk_norm) break;
+    if (!p.qk_norm || p.taps > 0) break;
     sq[r] = 0.f;
 #pragma unroll
     for (int u = 0; u < 2; ++u) sq[r] += v[r][u].x * v[r][u].x + v[r][u].y * v[r][u].y + v[r][u].z * v[r][u].z + v[r][u].w * v[r][u].w;
   }
-  if (p.qk_norm)
+  if (p.qk_norm && p.taps == 0)
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1)
 #pragma unroll
@@ -94,14 +196,14 @@ __device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x,
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
     if (r >= n) break;
-    const float s = p.qk_norm ? 1.f / sqrtf(sq[r] / static_cast<float>(p.D) + p.eps) : 1.f;
+    const float s = p.taps > 0 ? row_scale(p, m + r, isk) : p.qk_norm ? 1.f / sqrtf(sq[r] / static_cast<float>(p.D) + p.eps) : 1.f;
 #pragma unroll
     for (int u = 0; u < 2; ++u) put(r, u * 128 + lane * 4, make_float4(v[r][u].x * s, v[r][u].y * s, v[r][u].z * s, v[r][u].w * s));
   }
 }
 __device__ __forceinline__ uint2 pack4(float4 v) { return make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
 
-// grid (ceil(M / 8), ceil(items / 8)), 256 threads; a warp per (head, eight rows): query heads (tcgen05 form only), then
+// grid (ceil(M / 8), ceil(items / 8)) and, behind a convolution, nseq more columns that update the rings; 256 threads; a warp per (head, eight rows): query heads (tcgen05 form only), then
 // key heads, then value heads.  Eight values of neighbouring tokens leave as one 16-byte piece where a page allows it.
 template <typename T>
 __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__ GqaParams p) {
@@ -110,6 +212,10 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
   const int lane = threadIdx.x & 31;
   int item = blockIdx.y * 8 + (threadIdx.x >> 5);
   const int m0 = blockIdx.x * 8, n = min(8, p.M - m0);
+  if (n <= 0) {
+    conv_ring(p, static_cast<int>(blockIdx.x) - (p.M + 7) / 8);
+    return;
+  }
   const bool fast = sizeof(T) == 2 && (p.D & 3) == 0 && p.D <= 256 && (p.rot & 7) == 0;
   if (p.rot > 0) {
     for (int r = threadIdx.x >> 5; r < n; r += 8) rotary_table(rot_s + r * p.rot, p.freq, p.rot, p.rot_amp, p.pos[m0 + r], lane, 32);
@@ -121,14 +227,14 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
       const float* x0 = p.x + static_cast<size_t>(m0) * p.ldx + p.q_off + item * p.D;
       if (fast) {
         for (int r0 = 0; r0 < n; r0 += 4)
-          normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
+          normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, m0 + r0, 0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
             if (d < p.DK) *reinterpret_cast<uint2*>(q0 + static_cast<size_t>(r0 + r) * p.H * p.DK + d) = pack4(v);      // (zeros from D on)
           });
         return;
       }
       for (int r = 0; r < n; ++r) {
         const float* x = x0 + static_cast<size_t>(r) * p.ldx;
-        const float s = head_scale(p, x, lane);
+        const float s = head_scale(p, x, m0 + r, 0, lane);
         for (int d = lane; d < p.DK; d += 32) q0[static_cast<size_t>(r) * p.H * p.DK + d] = __float2bfloat16(d < p.D ? rotary_half(x, d, rot_s + r * p.rot, p.rot) * s : 0.f);
       }
       return;
@@ -153,7 +259,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
 #pragma unroll
       for (int r0 = 0; r0 < 8; r0 += 4) {
         if (r0 >= n) break;
-        normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
+        normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, m0 + r0, 1, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
           const int s = r == 0 ? slot[r0] : r == 1 ? slot[r0 + 1] : r == 2 ? slot[r0 + 2] : slot[r0 + 3];
           if (s >= 0 && d < p.D)
             *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.cache) + page_block(p, s / kPage, g) + bf16_key_at(s % kPage, d)) = pack4(v);
@@ -165,7 +271,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
       const int s = p.slot_map[m0 + r];
       if (s < 0 || s >= p.n_blocks * kPage) continue;
       const float* x = x0 + static_cast<size_t>(r) * p.ldx;
-      const float sc = head_scale(p, x, lane);
+      const float sc = head_scale(p, x, m0 + r, 1, lane);
       const size_t b = page_block(p, s / kPage, g);
       for (int d = lane; d < p.D; d += 32) Page<T>::store(p.cache, b + Page<T>::key(p, s % kPage, d), rotary_half(x, d, rot_s + r * p.rot, p.rot) * sc);
     }
@@ -205,7 +311,7 @@ __global__ void __launch_bounds__(128) gqa_row_kernel(const __grid_constant__ Gq
   const float* x = p.x + static_cast<size_t>(m) * p.ldx + p.q_off + h * p.D;
   float* rot_s = o + p.V;
   if (warp == 0) {
-    const float s = head_scale(p, x, lane);
+    const float s = head_scale(p, x, m, 0, lane);
     if (lane == 0) scale_s = s;
   }
   if (p.rot > 0) rotary_table(rot_s, p.freq, p.rot, p.rot_amp, p.pos[m], threadIdx.x, 128);
@@ -216,7 +322,7 @@ __global__ void __launch_bounds__(128) gqa_row_kernel(const __grid_constant__ Gq
     sm[d] = sizeof(T) == 2 ? __bfloat162float(__float2bfloat16(q)) : q;
   }
   for (int v = threadIdx.x; v < p.V; v += 128) o[v] = 0.f;
-  const int pos = p.pos[m], low = p.chunk > 0 ? pos - pos % p.chunk : 0;
+  const int pos = p.pos[m], low = first_key(pos, p.chunk, p.window);
   float mx = -INFINITY, l = 0.f;
   for (int pg = low / kPage; pg <= pos / kPage; ++pg) {
     const size_t b = page_block(p, page_at(p, j, pg), g);
@@ -260,7 +366,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
   const int j = mla_seq_of_row(p.cu_rows, p.nseq, m);
   if (j < 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hq = p.H / p.G;
-  const int pos = p.pos[m], low = p.chunk > 0 ? pos - pos % p.chunk : 0;
+  const int pos = p.pos[m], low = first_key(pos, p.chunk, p.window);
   const int page0 = low / kPage, pages = pos / kPage + 1 - page0;
   const int per = (pages + p.splits - 1) / p.splits;
   const int pa = page0 + sp * per, n = min(per, page0 + pages - pa);       // this CTA's pages (n <= 0: none)
@@ -294,7 +400,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
   }
   for (int r = warp; r < MT * 16; r += 4) {
     const float* x = xr + p.q_off + (g * hq + min(r, hq - 1)) * p.D;
-    const float s = head_scale(p, x, lane);
+    const float s = head_scale(p, x, m, 0, lane);
     for (int d = lane * 2; d < p.DK; d += 64) {
       const float a = r < hq && d < p.D ? rotary_half(x, d, rot_s, p.rot) * s : 0.f, b = r < hq && d + 1 < p.D ? rotary_half(x, d + 1, rot_s, p.rot) * s : 0.f;
       asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_s + r * qs + d * 2), "r"(pack2(a, b)) : "memory");
@@ -308,7 +414,7 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
     __nv_bfloat16* c = static_cast<__nv_bfloat16*>(p.cache) + (live ? page_block(p, slot / kPage, g) : 0);
     if (warp == 0) {
       const float* x = xr + p.k_off + g * p.D;
-      const float s = head_scale(p, x, lane);
+      const float s = head_scale(p, x, m, 1, lane);
       for (int d = lane; d < p.D; d += 32) {
         new_s[d] = __float2bfloat16(rotary_half(x, d, rot_s, p.rot) * s);
         if (live) c[bf16_key_at(slot % kPage, d)] = new_s[d];
@@ -520,14 +626,31 @@ static int split_mt(const GqaParams& p, cudaStream_t s) {
 }
 
 static int append_items(const GqaParams& p) {
-  if (p.form == 1 && p.max_rows == 1) return 0;                     // the attention kernel appends by itself
+  if (p.form == 1 && p.max_rows == 1) return 0;                     // the attention kernel appends by itself (the convolution kernel updates its rings)
   return (p.form == 2 ? p.H : 0) + (p.k_off >= 0 ? 2 * p.G : 0);
 }
 
 template <typename T>
-static int gqa_go(const GqaParams& p, cudaStream_t stream) {
+static int gqa_go(GqaParams p, cudaStream_t stream) {
+  p.gate = p.g_off < 0 ? nullptr : p.x + p.g_off;
+  p.ld_gate = p.ldx;
+  if (p.taps > 0) {
+    p.raw = p.x;
+    p.ld_raw = p.ldx;
+    p.rq_off = p.q_off;
+    p.rk_off = p.k_off;
+    p.rv_off = p.v_off;
+    p.x = p.cx;
+    p.ldx = p.ldc;
+    p.q_off = 0;
+    p.k_off = (p.H * p.D + 7) & ~7;
+    p.v_off = p.k_off + ((p.G * p.D + 7) & ~7);
+    const cudaError_t e = launch(gqa_conv_kernel, dim3(p.M), dim3(kConvThreads), 0, stream, 2, p);
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
   if (const int items = append_items(p)) {
-    const cudaError_t e = launch(gqa_append_kernel<T>, dim3((p.M + 7) / 8, (items + 7) / 8), dim3(256), 8 * p.rot * 4, stream, 0, p);
+    const int rings = p.taps > 0 && p.max_rows > 1 ? p.nseq : 0;
+    const cudaError_t e = launch(gqa_append_kernel<T>, dim3((p.M + 7) / 8 + rings, (items + 7) / 8), dim3(256), 8 * p.rot * 4, stream, 0, p);
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   if (p.form == 0)
@@ -556,8 +679,10 @@ static int gqa_go(const GqaParams& p, cudaStream_t stream) {
   f.chunk = p.chunk;
   f.scale = p.scale;
   f.softcap = p.softcap;
-  f.gate = p.g_off < 0 ? nullptr : p.x + p.g_off;
-  f.ldg = p.ldx;
+  f.gate = p.gate;
+  f.ldg = p.ld_gate;
+  f.window = p.window;
+  f.out_scale = p.out_scale;
   f.sink = p.sink;
   f.bound = p.qk_norm ? 1.02f * p.D : 0.f;        // (two vectors of root mean square one, and the rounding to bf16)
   f.err = p.err;
@@ -573,13 +698,17 @@ extern "C" int saber_gqa_form(const saber::GqaParams* p) {
   return saber_flash_tc_ok(p->page, p->DK, p->VP, p->scale, p->softcap) ? 2 : 1;
 }
 
-extern "C" int saber_gqa_launches(const saber::GqaParams* p) { return saber::append_items(*p) ? 2 : 1; }
+extern "C" int saber_gqa_launches(const saber::GqaParams* p) { return (p->taps > 0 ? 1 : 0) + (saber::append_items(*p) ? 2 : 1); }
 
 extern "C" int saber_gqa_launch(const saber::GqaParams* p, cudaStream_t stream) {
   using namespace saber;
   if (p->M <= 0 || p->G <= 0 || p->H % p->G || p->page != kPage || p->D > p->DK || p->DK > p->KP || p->V > p->VP || p->cache == nullptr ||
       p->D > 2048 || p->V > 2048 || p->rot < 0 || (p->rot & 1) || p->rot > p->D || p->rot > 1024 || (p->rot > 0 && p->freq == nullptr) || p->form < 0 || p->form > saber_gqa_form(p) || (p->form == 2 && p->q == nullptr) ||
       (p->form == 1 && (p->splits < 1 || p->splits > 32 || (p->splits > 1 && (p->o_part == nullptr || p->ml == nullptr || p->counters == nullptr)))))
+    return static_cast<int>(cudaErrorInvalidValue);
+  if (p->window < 0 || (p->window > 0 && p->chunk > 0) ||
+      (p->taps > 0 && (p->k_off < 0 || p->conv_w == nullptr || p->q_w == nullptr || p->k_w == nullptr || p->hist == nullptr || p->slots == nullptr ||
+                       p->cx == nullptr || p->row_ss == nullptr || (p->ldc & 7) || p->ldc < ((p->H * p->D + 7) & ~7) + ((p->G * p->D + 7) & ~7) + p->G * p->V)))
     return static_cast<int>(cudaErrorInvalidValue);
   return p->f32 ? gqa_go<float>(*p, stream) : gqa_go<__nv_bfloat16>(*p, stream);
 }

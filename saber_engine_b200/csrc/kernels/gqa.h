@@ -3,10 +3,13 @@
 //
 //   q, k    optionally divided by their root mean square over D (qk_norm), then rotated (rot > 0: the first rot values, halves
 //           layout)
+//   taps    > 0: q, k and v first pass a causal convolution of their own over the tokens; q and k are then normed over all heads at once
+//           (weights q_w, k_w), values per head (v_norm)
 //   score   scale q . k, then cap tanh(score / cap) when softcap > 0
 //   sink    exp(sink[h]) joins the denominator of head h
 //   gate    the output times sigmoid of column g_off + h V + v of x
-//   mask    keys j <= i; chunk > 0: of the same chunk of positions as i only, j >= i - i % chunk
+//   mask    keys j <= i; chunk > 0: of the same chunk of positions as i only, j >= i - i % chunk; window > 0: the last
+//           `window` ones only, i itself among them
 //
 // A page holds, per key / value head, the keys and then the values of its 64 tokens.  bf16: in the order the
 // tensor-core kernels multiply in place, keys [D / 64][64 tokens][128 bytes], values transposed [VP][64 tokens], both
@@ -45,6 +48,22 @@ struct GqaParams {
   int qk_norm, chunk;
   float scale, softcap, eps;
   uint32_t* err;
+  int window;
+  float out_scale;            // factor of the output
+  // convolution (taps > 0).  Inputs of a slot form a ring: the one of position p is row p % taps.
+  int taps, v_norm, n_slots, ldc;
+  const float* conv_w;        // [C][taps], C = H D + G D + G V in q | k | v order, last column: the current token
+  const float* q_w;           // [H D]
+  const float* k_w;           // [G D]
+  float* hist;                // [n_slots][taps][C]
+  const int32_t* slots;       // [nseq]
+  float* cx;                  // scratch [M][ldc]: the convolved rows, q | k | v from multiples of 8 on
+  float* row_ss;              // scratch [M][2]: sums of squares of q and k
+  // set at the launch
+  const float* gate;          // column 0 of the gate in row 0
+  int ld_gate;
+  const float* raw;           // the rows ahead of the convolution
+  int ld_raw, rq_off, rk_off, rv_off;
 };
 
 }  // namespace saber

@@ -32,6 +32,13 @@ __device__ __forceinline__ float clamped_glu(float gate, float up, float limit, 
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
 }
 
+// A gated unit of act_kind 0, 4 or 5.
+__device__ __forceinline__ float gated_unit(const LinEpi& e, float gate, float up) {
+  if (e.act_kind == 4) return 0.5f * gate * (1.f + tanhf(0.79788456080286536f * fmaf(0.044715f * gate * gate, gate, gate))) * up;
+  if (e.act_kind == 5) return gate / (1.f + expf(-gate)) * up;
+  return clamped_glu(gate, up, e.limit, e.alpha);
+}
+
 __device__ __forceinline__ float relu_squared(float x) {
   const float r = fmaxf(x, 0.f);
   return r * r;
@@ -184,8 +191,8 @@ __device__ __forceinline__ void linear_row_epilogue(const LinEpi& e, const Acc& 
     } else {
       const float4 g = acc(lane * 4), u = acc(128 + lane * 4);
       operand_store4(e.act, m, e.act_k0 + (tile_n - e.act_tile0) * 128 + lane * 4,
-                     make_float4(clamped_glu(g.x * sc, u.x * sc, e.limit, e.alpha), clamped_glu(g.y * sc, u.y * sc, e.limit, e.alpha),
-                                 clamped_glu(g.z * sc, u.z * sc, e.limit, e.alpha), clamped_glu(g.w * sc, u.w * sc, e.limit, e.alpha)));
+                     make_float4(gated_unit(e, g.x * sc, u.x * sc), gated_unit(e, g.y * sc, u.y * sc), gated_unit(e, g.z * sc, u.z * sc),
+                                 gated_unit(e, g.w * sc, u.w * sc)));
     }
     return;
   }
@@ -650,7 +657,7 @@ __global__ void __launch_bounds__(256) lin_epi_kernel(const __grid_constant__ Li
     }
     for (int i = threadIdx.x; i < (tiles - e.act_tile0) * 128; i += 256) {
       const float* t = acc + static_cast<size_t>(e.act_tile0 + (i >> 7)) * 256 + (i & 127);
-      operand_store1(e.act, m, e.act_k0 + i, clamped_glu(t[0] * sc, t[128] * sc, e.limit, e.alpha));
+      operand_store1(e.act, m, e.act_k0 + i, gated_unit(e, t[0] * sc, t[128] * sc));
     }
     return;
   }

@@ -18,6 +18,7 @@ namespace saber {
 //              act_kind 1  y = max(up, 0)^2, 256 features a tile
 //              act_kind 2  y = sigmoid(g) max(up, 0)^2, 248 features a tile and their gate's row g behind them
 //              act_kind 3  y = gelu(up + act_bias) (by the error function), 256 features a tile
+//              act_kind 4, 5  y = gelu(gate) up (by tanh), y = silu(gate) up, 128 gate then 128 up features a tile
 //            The first lat_tiles tiles are a latent of lat_n values instead: the operand `lat` takes lat_w times the
 //            value, lat_ss its sums of squares per 128 columns.  cap > 0: stored values become cap tanh(value / cap).
 //   stream   x[m][n] = (add ? x[m][n] : 0) + bias[n] + acc, and the operand of the next linear:

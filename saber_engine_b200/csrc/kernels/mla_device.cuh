@@ -25,6 +25,11 @@ __device__ __forceinline__ int mla_seq_of_row(const int32_t* cu, int nseq, int m
 __device__ __forceinline__ float mla_gate(const MlaParams& p, int m, int h, int v) {
   return p.x[static_cast<size_t>(m) * p.ldx + p.g_off + (p.gate_heads ? h : h * p.V + v)];
 }
+// first key that the query at a position sees: of its chunk of positions, among the last `window`, or all (0, 0)
+__device__ __forceinline__ int first_key(int pos, int chunk, int window) {
+  if (window > 0) return max(0, pos - window + 1);
+  return chunk > 0 ? pos - pos % chunk : 0;
+}
 // physical page of the i-th page of sequence j (bounds-checked: an entry outside the pool is recorded and read as page 0)
 template <typename Params>
 __device__ __forceinline__ int page_at(const Params& p, int j, int i) {

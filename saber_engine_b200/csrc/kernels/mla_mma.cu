@@ -551,6 +551,7 @@ static int flash_go(const MlaParams& p, cudaStream_t stream) {
   cudaError_t e = launch(mla_expand_kernel, dim3(2 * 148), dim3(256), 3 * kExpStage, stream, 0, p);
   if (e == cudaSuccess && p.expand == 2) {
     FlashParams f = {};
+    f.out_scale = 1.f;
     f.q = p.q_eff;
     f.k = p.k_exp;
     f.v = p.v_exp;

@@ -18,6 +18,92 @@ constexpr int kMoeTpMaxTiles = kTpMaxTiles;   // same flag regions as the row-pa
 
 __device__ __forceinline__ float e_safe(float x, float mx) { return x == -INFINITY ? 0.f : __expf(x - mx); }
 
+__device__ __forceinline__ float moe_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+// Routes by sigmoid scores with a correction of the choice (MoeRouteParams::sigmoid).
+template <int kPer, typename Add>
+__device__ __forceinline__ void moe_sigmoid_row(const MoeRouteParams& p, int m, int lane, const Add& add) {
+  const float* z = p.logits_f32 + static_cast<size_t>(m) * p.ld;
+  float v[kPer];                                    // choice scores (they may be negative)
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
+    const int e = i * 32 + lane;
+    v[i] = e < p.E ? moe_sigmoid(z[e]) + (p.correction != nullptr ? p.correction[e] : 0.f) : -INFINITY;
+  }
+  // largest of the values with their bit in `among`, entry i * 32 + lane below n; the lower entry wins ties (n: none is a number)
+  auto best = [&](const float (&x)[kPer], uint32_t among, int n, float& bv, int& be) {
+    bv = -INFINITY;
+    be = n;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i)
+      if ((among >> i & 1u) && i * 32 + lane < n && x[i] > bv) { bv = x[i]; be = i * 32 + lane; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+      if (ov > bv || (ov == bv && oe < be)) { bv = ov; be = oe; }
+    }
+  };
+  const uint32_t all = kPer == 32 ? 0xffffffffu : (1u << (kPer & 31)) - 1u;
+  uint32_t open = all;
+  if (p.groups > 1 && p.keep < p.groups) {
+    const int size = p.E / p.groups;
+    float strength[kPer];                           // entry i * 32 + lane: a group
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) strength[i] = -INFINITY;
+    for (int g = 0; g < p.groups; ++g) {
+      uint32_t in = 0u;
+#pragma unroll
+      for (int i = 0; i < kPer; ++i) {
+        const int e = i * 32 + lane;
+        if (e >= g * size && e < (g + 1) * size) in |= 1u << i;
+      }
+      float a, b = 0.f;
+      int ea, eb;
+      best(v, in, p.E, a, ea);
+      if (size > 1) {
+        if ((ea & 31) == lane) in &= ~(1u << (ea >> 5 & 31));
+        best(v, in, p.E, b, eb);
+      }
+#pragma unroll
+      for (int i = 0; i < kPer; ++i)
+        if (i * 32 + lane == g) strength[i] = a + b;
+    }
+    uint32_t left = all;
+    open = 0u;
+    for (int k = 0; k < p.keep; ++k) {
+      float bv;
+      int g;
+      best(strength, left, p.groups, bv, g);
+      if (g >= p.groups) break;                     // (scores that are no numbers)
+      if ((g & 31) == lane) left &= ~(1u << (g >> 5));
+#pragma unroll
+      for (int i = 0; i < kPer; ++i) {
+        const int e = i * 32 + lane;
+        if (e >= g * size && e < (g + 1) * size) open |= 1u << i;
+      }
+    }
+  }
+  float sum = 0.f, mine_w = 0.f;
+  int mine_e = -1;                                  // lane k holds route k
+  for (int k = 0; k < p.top_k; ++k) {
+    float bv;
+    int be;
+    best(v, open, p.E, bv, be);
+    if (be >= p.E) break;
+    if ((be & 31) == lane) open &= ~(1u << (be >> 5));
+    const float s = moe_sigmoid(z[be]);             // (the score itself; the choice's had the correction)
+    sum += s;
+    if (lane == k) { mine_w = s; mine_e = be; }
+  }
+  if (lane < p.top_k) {
+    p.topk_id[m * p.top_k + lane] = mine_e;
+    p.topk_w[m * p.top_k + lane] = mine_w / (sum + 1e-20f) * p.scale;
+    const int le = mine_e - p.e_lo;
+    if (mine_e >= 0 && le >= 0 && le < p.e_n) add(le);
+  }
+}
+
 // The routes of token m, by one warp; kPer * 32 experts at most.  add(expert) counts a route of a local expert.
 template <int kPer, typename Add>
 __device__ __forceinline__ void moe_topk_row(const MoeRouteParams& p, int m, int lane, const Add& add) {
@@ -26,6 +112,10 @@ __device__ __forceinline__ void moe_topk_row(const MoeRouteParams& p, int m, int
       p.topk_id[m * p.top_k + k] = -1;
       p.topk_w[m * p.top_k + k] = 0.f;
     }
+    return;
+  }
+  if (p.sigmoid) {
+    moe_sigmoid_row<kPer>(p, m, lane, add);
     return;
   }
   float v[kPer];
@@ -322,6 +412,7 @@ extern "C" int saber_moe_route_launches(const saber::MoeRouteParams* p) { return
 
 extern "C" int saber_moe_route_launch(const saber::MoeRouteParams* p, cudaStream_t stream) {
   using namespace saber;
+  if (p->sigmoid && p->logits_f32 == nullptr) return static_cast<int>(cudaErrorInvalidValue);
   if (p->E < 1 || p->E > 1024 || p->e_n > 1024 || p->top_k > kMoeMaxTopK || p->top_k < 1 || p->nt < 16 || (p->nt & 15) ||
       (p->groups > 1 && (p->E % p->groups || p->keep < 1 || p->keep * (p->E / p->groups) < p->top_k)))
     return static_cast<int>(cudaErrorInvalidValue);

@@ -26,6 +26,11 @@ struct MoeRouteParams {
   const float* logits_f32;
   const int32_t* live;           // rows from *live on are padding and take no route (null: every row is live)
   int groups, keep;              // groups > 1: only experts of the `keep` groups of neighbours whose best score is best
+  // sigmoid: scores are sigmoids of the logits one by one; the choice is made by score + correction[e], a group counts by the sum of its
+  // two largest of these, and the weights are the chosen scores over their sum (+ 1e-20), times `scale`
+  int sigmoid;
+  const float* correction;       // [E] or null
+  float scale;
 };
 
 struct MoeCombineParams {

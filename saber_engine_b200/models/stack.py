@@ -6,14 +6,17 @@ launch of its own.
   parallel    x <- x + mixer(norm(x)) + ff(norm(x)): two linears around the mixer's kernels.  Two norms: the same, the rows of the
               feed-forward multiply a second operand
   sequential  x <- x + mixer(norm1(x)); x <- x + ff(norm2(x)): two linears around the mixer, two for the feed-forward
-Launches of a mixer in decoding: delta rule 1, decayed outer products 1, grouped-query attention 1, latent attention 5 (6 where
+  joined      x <- x + c norm(mixer(blend of norm(x) with the token before)); x <- x + c norm(ff(norm(x))): a sublayer's result is whole
+              rows ahead of the stream, so that a row kernel stands between the linears (`join.cu`): it norms the result, adds it, norms
+              the stream and, ahead of a mixer, blends.  Mixers may stand side by side between the same two linears
+Launches of a mixer in decoding: delta rule 1, decayed outer products 1, grouped-query attention 1 (2 behind a convolution), latent attention 5 (6 where
 queries come from a latent of their own); a pass of a looped block adds one linear, routed experts add 3 (routing and two grouped
 products: the output linear's epilogue adds the experts' rows to the stream).
 
 Every row of every bucket is committed (no drafter): a decode bucket is one row per sequence, a prefill bucket
 is `width` ragged rows of up to `nseq` sequences, single decoded tokens beside portions of prompts included.
 Caches and states belong to a layer RUN: the pages of an attention run (a run may read those of an earlier one), the
-slots of a recurrent run.
+slots of a recurrent run, of a convolution's inputs and of the last token's row where tokens are blended.
 """
 from __future__ import annotations
 
@@ -26,7 +29,7 @@ from ..ops import functional as F
 from ..ops import layouts as L
 from ..ops import native as N
 from . import stack_weights as SW
-from .stack_config import DeltaMixer, ExpertMix, GroupedMixer, LatentMixer, OuterMixer, StackConfig
+from .stack_config import ChannelDeltaMixer, DeltaMixer, ExpertMix, GroupedMixer, LatentMixer, OuterMixer, StackConfig
 from .step import BlobLayout, Bucket, finish_bucket, head_outputs, plp_outputs, seam_outputs
 
 
@@ -59,23 +62,27 @@ class StackModel:
         else:
             self.w = SW.random_init(cfg, dtype, dev, seed)
         self.n_slots = max_seqs + 1                       # slot 0 is the null slot
-        self.kv, self.state, self.hist = {}, {}, {}
+        self.kv, self.state, self.hist, self.before = {}, {}, {}, {}
         for r in cfg.runs:
-            m = cfg.layers[r.layer].mixer
-            if isinstance(m, LatentMixer):
-                if m.kv_from is None:
-                    self.kv[r.index] = torch.zeros(self.kv_blocks, cfg.page_tokens, m.rank_pad + m.rot_pad, dtype=dtype, device=dev)
-            elif isinstance(m, GroupedMixer):
-                if m.kv_from is None:                     # the padding of a page stays zero: the kernels multiply it
-                    self.kv[r.index] = torch.zeros(self.kv_blocks, m.kv_heads, cfg.page_tokens * (m.key_pad + m.vdim_pad), dtype=dtype, device=dev)
-            else:
-                self.state[r.index] = torch.zeros(self.n_slots, m.heads, m.vdim_pad, m.dim_pad, dtype=torch.float32, device=dev)
+            if cfg.token_shift:
+                self.before[r.index] = torch.zeros(self.n_slots, cfg.width, dtype=torch.float32, device=dev)
+            for pre, m, _ in cfg.layers[r.layer].mixer.parts():
+                key = self._key(r, pre)
+                if isinstance(m, LatentMixer):
+                    if m.kv_from is None:
+                        self.kv[key] = torch.zeros(self.kv_blocks, cfg.page_tokens, m.rank_pad + m.rot_pad, dtype=dtype, device=dev)
+                    continue
+                if isinstance(m, GroupedMixer):
+                    if m.kv_from is None:                 # the padding of a page stays zero: the kernels multiply it
+                        self.kv[key] = torch.zeros(self.kv_blocks, m.kv_heads, cfg.page_tokens * (m.key_pad + m.vdim_pad), dtype=dtype, device=dev)
+                else:
+                    self.state[key] = torch.zeros(self.n_slots, m.heads, m.vdim_pad, m.dim_pad, dtype=torch.float32, device=dev)
                 if m.taps:
-                    self.hist[r.index] = torch.zeros(self.n_slots, m.taps, m.channels, dtype=torch.float32, device=dev)
+                    self.hist[key] = torch.zeros(self.n_slots, m.taps, m.channels, dtype=torch.float32, device=dev)
         # expanded keys / values of the pages a prompt portion sees: scratch of one layer run at a time, in
         # physical page order (absent when it would not fit its budget: the absorbed form serves then)
         self.k_exp = self.v_exp = None
-        lat = [l.mixer for l in cfg.layers if isinstance(l.mixer, LatentMixer)]
+        lat = [m for m in cfg.mixers() if isinstance(m, LatentMixer)]
         tokens = self.kv_blocks * cfg.page_tokens
         if lat and not self.f32 and tokens * cfg.expanded_token_bytes() <= expand_bytes:
             self.k_exp = torch.zeros(tokens * max(m.heads * m.key_tile for m in lat), dtype=dtype, device=dev)
@@ -85,6 +92,11 @@ class StackModel:
         torch.cuda.synchronize(dev)                       # buckets run on a stream of their own
 
     # ------------------------------------------------------------------------------ state
+    @staticmethod
+    def _key(run, prefix: str):
+        """Name of a mixer's caches and states: the layer run, and the part where mixers stand side by side."""
+        return run.index if not prefix else f"{run.index}.{prefix[:-1]}"
+
     def reset_slot(self, slot: int) -> None:
         with torch.cuda.stream(self.stream):
             for t in self.slot_tensors().values():
@@ -94,7 +106,7 @@ class StackModel:
         return {f"kv.{i}": t for i, t in self.kv.items()}
 
     def slot_tensors(self) -> dict:
-        return {**{f"state.{i}": t for i, t in self.state.items()}, **{f"hist.{i}": t for i, t in self.hist.items()}}
+        return {f"{name}.{i}": t for name, d in (("state", self.state), ("hist", self.hist), ("before", self.before)) for i, t in d.items()}
 
     def snapshot_views(self, slot: int) -> dict:
         return {k: t[slot] for k, t in self.slot_tensors().items()}
@@ -102,7 +114,7 @@ class StackModel:
     def state_bytes(self) -> dict:
         size = lambda d: sum(t.numel() * t.element_size() for t in d.values())    # noqa: E731
         exp = 0 if self.k_exp is None else (self.k_exp.numel() + self.v_exp.numel()) * 2
-        return {"weights": self.w.nbytes(), "kv_pool": size(self.kv), "state": size(self.state) + size(self.hist),
+        return {"weights": self.w.nbytes(), "kv_pool": size(self.kv), "state": size(self.state) + size(self.hist) + size(self.before),
                 "expanded_kv_scratch": exp}
 
     # ------------------------------------------------------------------------------ builders
@@ -192,12 +204,12 @@ class StackModel:
 
         # ---- activation buffers
         x = f32(M, L.round_up(W, 32))
-        ss = f32(L.padded_rows(M), (W + 127) // 128)
+        ss = f32(L.padded_rows(M), (W + 127) // 128) if not cfg.post_norms else None
         h = self._operand_buf(M, KW)
         h2 = self._operand_buf(M, KW) if cfg.two_norms else None
-        loop_op = self._operand_buf(M, 2 * KW) if cfg.loop is not None else None
+        loop_op = self._operand_buf(M, 2 * KW) if cfg.loop is not None and cfg.loop_linear else None
         mid = self._operand_buf(M, max(l.out.K for l in w.layers))
-        ups = [l for l in w.layers if l.up is not None]
+        ups = [l for l in w.layers if l.down is not None]
         ff = self._operand_buf(M, max(l.down.K for l in ups)) if ups else None
         ldp = max(L.round_up(l.n_plain, 8) for l in w.layers)
         proj = f32(M, ldp)
@@ -214,6 +226,15 @@ class StackModel:
         if self.race_check == "shadow":
             digests = torch.zeros(len(cfg.runs) + 1, dtype=torch.int64, device=dev)
             prog.digest_clear(digests, len(cfg.runs) + 1, tag="digest.clear")
+
+        if cfg.post_norms:
+            arenas = dict(x=x, h=h, mid=mid, ff=ff, proj=proj, work=work, experts=experts, ws=ws, digests=digests)
+            x = self._joined_layers(prog, M, nseq, decode, lay, at, arenas)
+            keep.append(arenas)
+            b = self._head(prog, key, kind, nseq, width, M, lay, at, blob, blob_host, x, h, None, ws, keep + [digests], seam, plp, capture)
+            b.arenas = [a for a in (arenas["x"], arenas["x2"], arenas["y"], h, mid, ff, proj) if a is not None]
+            b.digests, b.x = digests, x
+            return b
 
         h_op = self._operand(h, M, KW)
         h2_op = self._operand(h2, M, KW) if h2 is not None else None
@@ -262,17 +283,10 @@ class StackModel:
                 e.lat_ss, e.lat_ss_n = work["lat_ss"].data_ptr(), 2 * lw.lat_tiles
             self._linear(prog, lw.proj, h, M, e, ws, f"{t}.project", second=(h2, lw.tile2) if cfg.two_norms and spec.mlp is not None else None)
             if lw.experts_up is not None:
-                self._experts(prog, lw, spec.mlp, h2, ss, proj, M, at(lay.cu_rows + nseq), experts, ws, t)
+                self._experts(prog, lw, spec.mlp, h2, ss, proj.data_ptr() + 4 * lw.off["router"], proj.stride(0), M, at(lay.cu_rows + nseq), experts, ws, t)
             if lw.carry is not None:
                 self._carry_queries(prog, lw, spec.mixer, work, M, ws, f"{t}.carry")
-            if isinstance(spec.mixer, DeltaMixer):
-                prog.delta(self._delta_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work), decode, tag=f"{t}.delta")
-            elif isinstance(spec.mixer, OuterMixer):
-                prog.ssd(self._outer_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode), decode, tag=f"{t}.outer")
-            elif isinstance(spec.mixer, GroupedMixer):
-                prog.gqa(self._gqa_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode), tag=f"{t}.attention")
-            else:
-                prog.mla(self._mla_params(run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode), tag=f"{t}.latent_attention")
+            self._mixers(prog, run, lw, spec.mixer, proj, m_op, M, nseq, lay, at, work, decode, t)
             nxt = runs[i + 1] if i + 1 < len(runs) else None
             tgt = target(nxt)
             if lw.up is None:
@@ -295,6 +309,99 @@ class StackModel:
         b.digests, b.x = digests, x
         return b
 
+    def _mixers(self, prog, run, lw, mixer, proj, m_op, M, nseq, lay, at, work, decode, t: str) -> None:
+        for pre, m, scale in mixer.parts():
+            part, key, k0 = lw.part(pre), self._key(run, pre), lw.mix_k0[pre]
+            if isinstance(m, DeltaMixer):
+                prog.delta(self._delta_params(run, lw, m, proj, m_op, M, nseq, lay, at, work), decode, tag=f"{t}.delta")
+            elif isinstance(m, ChannelDeltaMixer):
+                prog.cdelta(self._cdelta_params(key, part, m, proj, m_op, k0, scale, M, nseq, lay, at, work), decode, tag=f"{t}.channel_delta")
+            elif isinstance(m, OuterMixer):
+                prog.ssd(self._outer_params(run, lw, m, proj, m_op, M, nseq, lay, at, work, decode), decode, tag=f"{t}.outer")
+            elif isinstance(m, GroupedMixer):
+                cache = self.kv[key if pre else self.cfg.pages_of(run)]
+                prog.gqa(self._gqa_params(key, cache, part, m, proj, m_op, k0, scale, M, nseq, lay, at, work, decode), tag=f"{t}.attention")
+            else:
+                prog.mla(self._mla_params(run, lw, m, proj, m_op, M, nseq, lay, at, work, decode), tag=f"{t}.latent_attention")
+
+    def _joined_layers(self, prog, M: int, nseq: int, decode: bool, lay, at, ar: dict) -> torch.Tensor:
+        """Layers whose sublayers' results are normed ahead of the stream; returns the stream's buffer behind the last.  A row kernel
+        that blends tokens reads the stream of neighbouring rows, so it writes another buffer than it reads."""
+        cfg, w, dev = self.cfg, self.w, self.device
+        W, KW, wide = cfg.width, L.round_up(cfg.width, 64), L.round_up(cfg.width, 8)
+        x, ws, live = ar["x"], ar["ws"], at(lay.cu_rows + nseq)
+        ar["x2"] = other = torch.zeros_like(x) if cfg.token_shift else x
+        ar["y"] = y = torch.zeros(M, wide, dtype=torch.float32, device=dev)
+        E = max([l.up_plain for l in w.layers], default=0)
+        ar["logits"] = logits = torch.zeros(M, max(8, E), dtype=torch.float32, device=dev)
+        h_op, experts = self._operand(ar["h"], M, KW), ar["experts"]
+
+        def plain(out: torch.Tensor, n: int, lin: SW.Linear, bias=None) -> N.LinEpi:
+            e = N.LinEpi()
+            e.out, e.ldo, e.n_plain, e.act_tile0, e.bias = out.data_ptr(), out.stride(0), n, lin.N_pad // 256, N.ptr(bias)
+            return e
+
+        def join(tag: str, norm_w, result=None, run=None) -> None:
+            """result: (post norm, whether `y` holds product rows, feed-forward with routed rows or None).  run: the layer run that
+            reads the row (None: a feed-forward or the head)."""
+            nonlocal x, other
+            p = N.JoinParams()
+            p.M, p.width, p.ldx, p.rows, p.nseq, p.n_slots = M, W, x.stride(0), self._join_rows(M, decode), nseq, self.n_slots
+            if result is None:
+                p.table, p.table_f32, p.vocab, p.ids, p.embed_scale = w.embed.data_ptr(), int(self.f32), cfg.vocab, at(lay.ids), cfg.embed_scale
+            else:
+                post, product, f = result
+                p.post_w, p.mult = post.data_ptr(), cfg.residual_mult
+                if product:
+                    p.y, p.ldy = y.data_ptr(), y.stride(0)
+                if f is not None:
+                    p.routed, p.slot_of, p.route_w = (experts[k].data_ptr() for k in ("y", "slot_of", "topk_w"))
+                    p.routes, p.ldr, p.routed_f32 = f.top, wide, int(self.f32)
+            p.norm_w, p.op, p.eps, p.err = norm_w.data_ptr(), h_op, cfg.eps, self.scratch.err.data_ptr()
+            p.x = p.x_out = x.data_ptr()
+            p.cu_rows, p.slots, p.pos = at(lay.cu_rows), at(lay.slots), at(lay.pos)
+            if run is not None:
+                if run.enter is not None:
+                    p.step = w.loop_step[run.enter].data_ptr()
+                if cfg.token_shift:
+                    p.shift, p.state, p.x_out = w.layers[run.layer].shift.data_ptr(), self.before[run.index].data_ptr(), other.data_ptr()
+                    x, other = other, x
+            prog.join(p, tag=tag)
+
+        runs = cfg.runs
+        join("embed", w.layers[runs[0].layer].norm, run=runs[0])
+        for i, run in enumerate(runs):
+            lw, spec, t = w.layers[run.layer], cfg.layers[run.layer], f"R{run.index}.L{run.layer}"
+            e = plain(ar["proj"], lw.n_plain, lw.proj, lw.bias)
+            self._linear(prog, lw.proj, ar["h"], M, e, ws, f"{t}.project")
+            self._mixers(prog, run, lw, spec.mixer, ar["proj"], self._operand(ar["mid"], M, lw.out.K), M, nseq, lay, at, ar["work"], decode, t)
+            self._linear(prog, lw.out, ar["mid"], M, plain(y, wide, lw.out, lw.out_bias), ws, f"{t}.out")
+            result, f = (lw.post1, True, None), spec.mlp
+            if f is not None:
+                join(f"{t}.join", lw.norm2, result)
+                e = N.LinEpi()
+                e.out, e.ldo, e.n_plain, e.act_tile0 = logits.data_ptr(), logits.stride(0), lw.up_plain, lw.up_tile0
+                if lw.down is not None:
+                    e.act, e.act_kind = self._operand(ar["ff"], M, lw.down.K), f.act_kind
+                self._linear(prog, lw.up, ar["h"], M, e, ws, f"{t}.up")
+                mix = f if isinstance(f, ExpertMix) else None
+                if mix is not None:
+                    self._experts(prog, lw, mix, ar["h"], None, logits.data_ptr() + 4 * lw.up_off["router"], logits.stride(0), M, live, experts, ws, t)
+                if lw.down is not None:
+                    self._linear(prog, lw.down, ar["ff"], M, plain(y, wide, lw.down), ws, f"{t}.down")
+                result = (lw.post2, lw.down is not None, mix)
+            nxt = runs[i + 1] if i + 1 < len(runs) else None
+            join(f"{t}.{'end' if f is not None else 'join'}", w.final_norm if nxt is None else w.layers[nxt.layer].norm, result, nxt)
+            if ar["digests"] is not None:
+                prog.digest(x, x.numel() * 4, ar["digests"].data_ptr() + 8 * run.index, tag=f"{t}.digest")
+        return x
+
+    def _join_rows(self, M: int, decode: bool) -> int:
+        """Rows of a CTA of the row kernel: several share the row ahead of them, while its rows fit."""
+        if decode or M < 256:
+            return 1
+        return next((r for r in (4, 2) if (r + 2) * L.round_up(self.cfg.width, 4) * 4 <= 110 << 10), 1)
+
     # ---- routed experts
     def _expert_scratch(self, M: int) -> dict:
         """Routing tables and routed rows of a bucket, sized for the largest mixture.  Every expert's rows start at a multiple of 16."""
@@ -310,24 +417,27 @@ class StackModel:
         per = [(M * f.top, min(f.experts, M * f.top)) for f in ms]            # routes, experts that can have one
         rows = L.round_up(max(r + 15 * e for r, e in per), 16)
         pad = L.round_up(rows, 128)
-        top, E, ff = max(f.top for f in ms), max(f.experts for f in ms), max(L.round_up(f.ff, 64) for f in ms)
+        top, E, ff = max(f.top for f in ms), max(f.experts for f in ms), max(L.round_up(f.ff, f.k_step) for f in ms)
         most = max(e + r // tile for r, e in per)
         return {"nt": nt, "mtiles": mtiles, "rows": rows, "pad": pad, "max_tiles": most, "tiles": i32(most, 4),
                 "ntiles": i32(2), "src_row": i32(pad), "topk_id": i32(M * top), "slot_of": i32(M * top), "counts": i32(E), "offsets": i32(E + 1), "cursors": i32(E),
                 "topk_w": torch.zeros(M * top, dtype=torch.float32, device=dev), "act": torch.zeros(pad * ff, dtype=self.dtype, device=dev),
                 "y": torch.zeros(rows * L.round_up(W, 8), dtype=self.dtype, device=dev)}
 
-    def _experts(self, prog, lw, f: ExpertMix, h2, ss, proj, M: int, live, ew: dict, ws, tag: str) -> None:
-        """Routes of the step, then the experts' rows; their weighted sum is left to the output linear."""
+    def _experts(self, prog, lw, f: ExpertMix, h2, ss, logits: int, ld: int, M: int, live, ew: dict, ws, tag: str) -> None:
+        """Routes of the step, then the experts' rows; their weighted sum is left to the output linear or the row kernel.
+        ss: sums of squares of the operand's rows (None: they are divided already)."""
         p = N.MoeRouteParams()
-        p.logits_f32, p.ld, p.M, p.E, p.top_k = proj.data_ptr() + 4 * lw.off["router"], proj.stride(0), M, f.experts, f.top
+        p.logits_f32, p.ld, p.M, p.E, p.top_k = logits, ld, M, f.experts, f.top
+        p.sigmoid, p.correction, p.scale = int(f.sigmoid), N.ptr(lw.correction), f.scale
         p.topk_id, p.topk_w, p.counts, p.offsets, p.cursors, p.tiles, p.ntiles, p.src_row, p.slot_of = \
             (ew[k].data_ptr() for k in ("topk_id", "topk_w", "counts", "offsets", "cursors", "tiles", "ntiles", "src_row", "slot_of"))
         p.nt, p.rows_cap, p.e_lo, p.e_n, p.live, p.groups, p.keep = ew["nt"] * ew["mtiles"], ew["src_row"].numel(), 0, f.experts, live, f.groups, f.keep
         prog.add_moe_route(p, tag=f"{tag}.route")
         e = N.LinEpi()
-        self._row_norm(e, ss)
-        e.act, e.act_kind = N.Operand(ew["act"].data_ptr(), ew["pad"], lw.experts_down.K, int(self.f32)), 1
+        if ss is not None:
+            self._row_norm(e, ss)
+        e.act, e.act_kind = N.Operand(ew["act"].data_ptr(), ew["pad"], lw.experts_down.K, int(self.f32)), f.expert_act_kind
         self._grouped_linear(prog, lw.experts_up, h2, L.padded_rows(M), ew, True, e, ws, f"{tag}.experts_up")
         e = N.LinEpi()
         e.out, e.ldo, e.n_plain, e.act_tile0 = ew["y"].data_ptr(), L.round_up(self.cfg.width, 8), L.round_up(self.cfg.width, 8), lw.experts_down.N_pad // 256
@@ -345,7 +455,7 @@ class StackModel:
     def _mixer_scratch(self, M: int, nseq: int, decode: bool) -> dict:
         """Scratch shared by the layers of a bucket, sized for the largest of them."""
         f32 = lambda n: torch.zeros(max(1, n), dtype=torch.float32, device=self.device)   # noqa: E731
-        ms = [l.mixer for l in self.cfg.layers]
+        ms = self.cfg.mixers()
         de, la = [m for m in ms if isinstance(m, (DeltaMixer, OuterMixer))], [m for m in ms if isinstance(m, LatentMixer)]
         outer, gr = [m for m in ms if isinstance(m, OuterMixer)], [m for m in ms if isinstance(m, GroupedMixer)]
         mx = lambda it: max(it, default=0)    # noqa: E731
@@ -360,6 +470,14 @@ class StackModel:
             wk["chunk"] = f32(mx(floats.values()))
         elif outer:
             wk["o"] = f32(M * mx(m.heads * m.vdim_pad for m in outer))
+        cd, conv = [m for m in ms if isinstance(m, ChannelDeltaMixer)], [m for m in gr if m.taps]
+        if cd and not decode:
+            blk = M // 4 + nseq
+            wk["cd_rec"] = f32(blk * mx(m.heads * (17 * m.dim_pad + 32) for m in cd))
+            wk["cd_v"] = f32(blk * mx(m.heads * ((m.vdim_pad + 15) // 16) * 64 for m in cd))
+            wk["cd_o"] = f32(M * mx(m.heads * m.vdim_pad for m in cd))
+        if conv:
+            wk["conv_x"], wk["conv_ss"] = f32(M * mx(self._conv_width(m) for m in conv)), f32(2 * M)
         if outer or gr:                                   # arrivals at the end of a row: zero between launches
             wk["counters"] = torch.zeros(max(nseq * mx(m.norm_groups for m in outer), M * mx(m.kv_heads for m in gr)), dtype=torch.int32, device=self.device)
         if gr:
@@ -417,7 +535,8 @@ class StackModel:
 
     def _gqa_splits(self, m: GroupedMixer, M: int) -> int:
         """Key splits: fill the SMs twice, never more parts than pages a row can see."""
-        span = self.max_ctx if m.chunk == 0 else min(self.max_ctx, m.chunk + self.cfg.page_tokens - 1)
+        part = m.chunk or m.window                        # keys a row sees at most
+        span = self.max_ctx if part == 0 else min(self.max_ctx, part + self.cfg.page_tokens - 1)
         pages = (span + self.cfg.page_tokens - 1) // self.cfg.page_tokens
         return max(1, min(32, pages, 2 * F.device_sms() // max(1, M * m.kv_heads)))
 
@@ -436,15 +555,38 @@ class StackModel:
         p.groups, p.gate_first, p.eps, p.err = m.norm_groups, int(m.gate_first), self.cfg.eps, self.scratch.err.data_ptr()
         return p
 
-    def _gqa_params(self, run, lw, m: GroupedMixer, proj, m_op, M, nseq, lay, at, wk, decode) -> N.GqaParams:
+    @staticmethod
+    def _conv_width(m: GroupedMixer) -> int:
+        """Columns of the convolved rows: q | k | v, each from a multiple of 8 on."""
+        return sum(L.round_up(n, 8) for name, n in m.segments() if name != "g")
+
+    def _cdelta_params(self, key, lw, m: ChannelDeltaMixer, proj, m_op, k0, scale, M, nseq, lay, at, wk) -> N.CdeltaParams:
+        p, x = N.CdeltaParams(), lw.extra
+        p.x, p.ldx = proj.data_ptr(), proj.stride(0)
+        p.r_off, p.k_off, p.v_off, p.a_off, p.l_off, p.g_off = (lw.off[k] for k in ("r", "k", "v", "a", "w1", "g"))
+        p.w2, p.w2_f32, p.rank, p.w0, p.norm_w = x["w2"].data_ptr(), int(self.f32), m.rank, x["w0"].data_ptr(), x["norm"].data_ptr()
+        p.state = self.state[key].data_ptr()
+        p.rec, p.vb, p.o = (N.ptr(wk.get(k)) for k in ("cd_rec", "cd_v", "cd_o"))
+        p.cu_rows, p.slots, p.pos = at(lay.cu_rows), at(lay.slots), at(lay.pos)
+        p.out, p.out_k0, p.out_scale, p.M, p.nseq = m_op, k0, scale, M, nseq
+        p.H, p.D, p.DP, p.VP, p.n_slots = m.heads, m.dim, m.dim_pad, m.vdim_pad, self.n_slots
+        p.eps, p.unit_eps, p.err = self.cfg.eps, m.unit_eps, self.scratch.err.data_ptr()
+        return p
+
+    def _gqa_params(self, key, cache, lw, m: GroupedMixer, proj, m_op, k0, scale, M, nseq, lay, at, wk, decode) -> N.GqaParams:
         p = self._gqa_sizes(m)
         p.x, p.ldx = proj.data_ptr(), proj.stride(0)
         p.q_off, p.k_off, p.v_off, p.g_off = lw.off["q"], lw.off.get("k", -1), lw.off.get("v", -1), lw.off.get("g", -1)
         p.freq, p.sink = N.ptr(lw.extra.get("freq")), N.ptr(lw.extra.get("sink"))
-        p.cache, p.q = self.kv[self.cfg.pages_of(run)].data_ptr(), wk["gqa_q"].data_ptr()
+        p.cache, p.q = cache.data_ptr(), wk["gqa_q"].data_ptr()
+        p.window, p.out_scale, p.taps = m.window, scale, m.taps
+        if m.taps:
+            p.conv_w, p.q_w, p.k_w = (lw.extra[k].data_ptr() for k in ("conv", "q_norm", "k_norm"))
+            p.hist, p.slots, p.n_slots, p.v_norm = self.hist[key].data_ptr(), at(lay.slots), self.n_slots, 1
+            p.cx, p.ldc, p.row_ss = wk["conv_x"].data_ptr(), self._conv_width(m), wk["conv_ss"].data_ptr()
         p.o_part, p.ml, p.counters = wk["gqa_o"].data_ptr(), wk["gqa_ml"].data_ptr(), wk["counters"].data_ptr()
         p.slot_map, p.pos, p.cu_rows, p.kv_len, p.block_table = (at(o) for o in (lay.slot_map, lay.pos, lay.cu_rows, lay.kv_len, lay.block_table))
-        p.out, p.out_k0, p.M, p.nseq = m_op, 0, M, nseq
+        p.out, p.out_k0, p.M, p.nseq = m_op, k0, M, nseq
         p.n_blocks, p.max_blocks, p.max_rows = self.kv_blocks, self.max_blocks, 1 if decode else M
         p.form = self._gqa_form(m, M, decode)
         p.splits = self._gqa_splits(m, M) if p.form == 1 else 1
@@ -497,7 +639,7 @@ class StackModel:
 
         def head(a, rows, dst, normed: bool, tag):
             e = N.LinEpi()
-            if not normed:
+            if not normed and ss is not None:            # (the row kernel has divided its rows already)
                 self._row_norm(e, ss)
             e.out, e.ldo, e.n_plain, e.act_tile0, e.cap = dst.data_ptr(), dst.stride(0), V, w.head.N_pad // 256, cfg.logit_cap
             self._linear(prog, w.head, a, rows, e, ws, tag)

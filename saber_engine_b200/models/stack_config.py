@@ -10,6 +10,7 @@ import dataclasses
 import json
 import math
 import os
+import struct
 from dataclasses import dataclass
 from pathlib import Path
 from typing import Optional
@@ -52,6 +53,7 @@ class Mixer:
     """What a layer asks of its mixer.  `segments` are the rows of the input projection, in order."""
     kind = ""
     kv_from: Optional[int] = None     # layer whose pages this mixer reads (it has none of its own)
+    out_bias = False
     q_rank = 0                        # > 0: the first segment is a latent of this size, normed and carried on by a linear of its own
 
     def segments(self) -> list:
@@ -65,6 +67,14 @@ class Mixer:
     def biases(self) -> list:
         """Segments whose tensor has a bias beside it (its name with '.b')."""
         return []
+
+    def parts(self) -> list:
+        """(prefix of names, mixer, factor of its result): several where mixers stand side by side."""
+        return [("", self, 1.0)]
+
+    def out_tensors(self) -> list:
+        """(output tensor, its input features, whether it has a bias) of every part."""
+        return [("o", self.out_features, self.out_bias)]
 
     def extra_shapes(self) -> dict:
         """Tensors beside the projections, name -> shape."""
@@ -255,8 +265,9 @@ class OuterMixer(Mixer):
 @dataclass(frozen=True)
 class GroupedMixer(Mixer):
     """Grouped-query attention: q and k over their root mean square per head, rotated, capped scores, keys of the query's own
-    chunk of positions, a learned number per head in the denominator, an output gate; each where asked for.  kv_from: the pages
-    of that layer are read, with this layer's queries and mask."""
+    chunk of positions or of a sliding window, a learned number per head in the denominator, an output gate; each where asked for.
+    taps: q, k and v pass a causal convolution of their own; q and k are then normed over all their heads at once, with weights,
+    and values per head.  kv_from: the pages of that layer are read, with this layer's queries and mask."""
     heads: int
     kv_heads: int
     dim: int
@@ -270,7 +281,14 @@ class GroupedMixer(Mixer):
     rot: Optional[Rotation] = None
     sink: bool = False
     gate: bool = False                # sigmoid of a projection, value by value
+    window: int = 0                   # > 0: the last `window` keys, the query's own among them
+    taps: int = 0
+    out_bias: bool = False
     kind = "attention"
+
+    @property
+    def channels(self) -> int:        # convolution channels q | k | v
+        return (self.heads + self.kv_heads) * self.dim + self.kv_heads * self.vdim
 
     @property
     def out_features(self) -> int:
@@ -296,16 +314,100 @@ class GroupedMixer(Mixer):
         return [name for name, _ in self.segments() if name != "g"] if self.bias else []
 
     def extra_shapes(self) -> dict:
-        return {"sink": (self.heads,)} if self.sink else {}
+        t = {"sink": (self.heads,)} if self.sink else {}
+        if self.taps:
+            rows = dict(self.segments())
+            t.update({f"{n}.conv": (rows[n], self.taps) for n in ("q", "k", "v")})
+            t.update({f"{n}.norm": (rows[n],) for n in ("q", "k")})
+        return t
+
+    def slot_bytes(self) -> int:
+        return 4 * self.taps * self.channels
 
     def page_token_bytes(self, elem: int) -> int:
         return 0 if self.kv_from is not None else elem * self.kv_heads * (self.key_pad + self.vdim_pad)
+
+
+@dataclass(frozen=True)
+class ChannelDeltaMixer(Mixer):
+    """Delta rule with a decay and a removal rate per head and key channel, keys and values of one size: S <- diag(w) S - (a u) (u^T S)
+    + k v^T with the unit key u, both terms of the old state; o = S^T r.  Decays come through `rank` values shared by the heads."""
+    heads: int
+    dim: int
+    rank: int
+    unit_eps: float = 1e-6            # inside the root of the unit norm of k
+    kind = "channel_delta"
+    taps = 0
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def dim_pad(self) -> int:
+        return _scan_width(self.dim, "delta mixer")
+
+    @property
+    def vdim_pad(self) -> int:
+        return (self.dim + 7) // 8 * 8
+
+    def segments(self) -> list:
+        n = self.out_features
+        return [("r", n), ("k", n), ("v", n), ("a", n), ("w1", self.rank), ("g", n)]
+
+    def biases(self) -> list:
+        return ["a"]
+
+    def extra_shapes(self) -> dict:
+        n = self.out_features
+        return {"w2": (n, self.rank), "w0": (n,), "norm": (n,)}
+
+    def slot_bytes(self) -> int:
+        return 4 * self.heads * self.vdim_pad * self.dim_pad
+
+
+@dataclass(frozen=True)
+class SideBySideMixer(Mixer):
+    """Two mixers over the same rows: left_scale * left + right_scale * right."""
+    left: Mixer
+    right: Mixer
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    kind = "side_by_side"
+
+    def parts(self) -> list:
+        return [("left.", self.left, self.left_scale), ("right.", self.right, self.right_scale)]
+
+    def _all(self, what) -> list:
+        return [(pre + name, *rest) for pre, m, _ in self.parts() for name, *rest in what(m)]
+
+    def segments(self) -> list:
+        return self._all(lambda m: m.segments())
+
+    def sources(self) -> list:
+        return [(pre + seg, pre + tensor, first) for pre, m, _ in self.parts() for seg, tensor, first in m.sources()]
+
+    def biases(self) -> list:
+        return [pre + name for pre, m, _ in self.parts() for name in m.biases()]
+
+    def extra_shapes(self) -> dict:
+        return dict(self._all(lambda m: m.extra_shapes().items()))
+
+    def out_tensors(self) -> list:
+        return self._all(lambda m: m.out_tensors())
+
+    def slot_bytes(self) -> int:
+        return self.left.slot_bytes() + self.right.slot_bytes()
+
+    def page_token_bytes(self, elem: int) -> int:
+        return self.left.page_token_bytes(elem) + self.right.page_token_bytes(elem)
 
 
 class FeedForward:
     """What a layer asks of its feed-forward.  Its rows are tiles of 256 behind the mixer's: `per_tile` features each."""
     act_kind = 0                      # the linear epilogue's activation
     per_tile = 256
+    k_step = 64                       # the activation's width goes up to a multiple of this
     limit = alpha = 0.0
 
     @property
@@ -327,7 +429,7 @@ class ClampedGlu(FeedForward):
     ff: int
     limit: float
     alpha: float = 1.702
-    per_tile = 128
+    per_tile = k_step = 128
 
     def shapes(self, width: int) -> dict:
         return {"gate": (self.ff, width), **super().shapes(width)}
@@ -350,31 +452,79 @@ class Gelu(FeedForward):
         return {"up": (self.ff, width), "up.b": (self.ff,), "down": (width, self.ff), "down.b": (width,)}
 
 
+GATED_ACTS = {"gelu_tanh": 4, "silu": 5}
+
+
+@dataclass(frozen=True)
+class GatedUnit(FeedForward):
+    """y = act(gate) up; act: gelu (by tanh) or silu."""
+    ff: int
+    act: str = "silu"
+    per_tile = k_step = 128
+
+    @property
+    def act_kind(self) -> int:
+        return GATED_ACTS[self.act]
+
+    def shapes(self, width: int) -> dict:
+        return {"gate": (self.ff, width), **super().shapes(width)}
+
+
 @dataclass(frozen=True)
 class ExpertMix(FeedForward):
-    """Mixture of squared-ReLU experts: softmax over `experts` scores, the `top` best of the `keep` groups of neighbours whose best
-    score is best, weighted by their scores as they are.  shared: the size of one more expert for every token, times the
-    sigmoid of a number of its own."""
+    """Mixture of experts: softmax over `experts` scores, the `top` best of the `keep` groups of neighbours whose best
+    score is best, weighted by their scores as they are; experts are squared ReLUs.  shared: the size of one more expert for every
+    token, times the sigmoid of a number of its own.
+    gated: experts are gated silu units, the shared one is added as it is.
+    sigmoid: scores are sigmoids; a correction per expert joins them for the choice, where a group counts by the sum of its two best;
+    the weights are the chosen scores over their sum, times `scale`."""
     experts: int
     top: int
     ff: int
     groups: int = 1
     keep: int = 1
     shared: int = 0
-    act_kind = 2
-    per_tile = 248                    # and the shared expert's gate row behind them
+    gated: bool = False
+    sigmoid: bool = False
+    scale: float = 1.0
+
+    @property
+    def act_kind(self) -> int:        # of the shared expert
+        return GATED_ACTS["silu"] if self.gated else 2
+
+    @property
+    def expert_act_kind(self) -> int:
+        return GATED_ACTS["silu"] if self.gated else 1
+
+    @property
+    def per_tile(self) -> int:        # not gated: and the shared expert's gate row behind them
+        return 128 if self.gated else 248
+
+    @property
+    def k_step(self) -> int:
+        return 128 if self.gated else 64
 
     @property
     def inner(self) -> int:
         return self.shared
 
+    @property
+    def matrices(self) -> tuple:      # of an expert, ahead of `down`
+        return ("gate", "up") if self.gated else ("up",)
+
     def shapes(self, width: int) -> dict:
         t = {}
         for e in range(self.experts):
-            t[f"e{e}.up"], t[f"e{e}.down"] = (self.ff, width), (width, self.ff)
+            t.update({f"e{e}.{n}": (self.ff, width) for n in self.matrices})
+            t[f"e{e}.down"] = (width, self.ff)
         t["router"] = (self.experts, width)
+        if self.sigmoid:
+            t["correction"] = (self.experts,)
         if self.shared:
-            t.update({"shared.up": (self.shared, width), "shared.down": (width, self.shared), "shared.sg": (1, width)})
+            t.update({f"shared.{n}": (self.shared, width) for n in self.matrices})
+            t["shared.down"] = (width, self.shared)
+            if not self.gated:
+                t["shared.sg"] = (1, width)
         return t
 
 
@@ -413,7 +563,11 @@ class StackConfig:
     two_norms: bool = False           # side by side: the feed-forward reads a norm of its own
     logit_cap: float = 0.0            # logits become cap tanh(logits / cap)
     norm_offset: float = 0.0          # norms multiply by offset + weight
+    post_norms: bool = False          # one after the other: a sublayer's result is normed, too, before it joins the stream
+    residual_mult: float = 1.0        # and multiplied by this
+    token_shift: bool = False         # what a mixer reads is blended with the token before
     loop: Optional[LoopSpec] = None
+    loop_linear: bool = True          # a pass starts with a linear over [stream; embedding], else with its vector only
     page_tokens: int = 64
     max_ctx: int = 32768
     source: Optional[str] = None      # folder the description was read from
@@ -437,6 +591,10 @@ class StackConfig:
                     out.append(LayerRun(len(out), i, enter))
         return tuple(out)
 
+    def mixers(self) -> list:
+        """Every mixer of every layer."""
+        return [m for l in self.layers for _, m, _ in l.mixer.parts()]
+
     def __post_init__(self):
         if not self.layers:
             raise ValueError(f"{self.name}: no layers")
@@ -451,7 +609,23 @@ class StackConfig:
                 raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / norm_groups {m.norm_groups} / decay {m.decay}")
             if isinstance(m, GroupedMixer):
                 self._check_grouped(i, m)
-            if not self.parallel and isinstance(l.mlp, (Gelu, ExpertMix)):
+            if isinstance(m, SideBySideMixer):
+                if not self.post_norms or any(x.kv_from is not None for _, x, _ in m.parts()):
+                    raise ValueError(f"{self.name}: layer {i}: mixers side by side stand ahead of normed results and have pages of their own")
+                for _, x, _ in m.parts():
+                    if isinstance(x, GroupedMixer):
+                        self._check_grouped(i, x)
+            if isinstance(m, ChannelDeltaMixer) and not self.post_norms:
+                raise ValueError(f"{self.name}: layer {i}: a channel delta rule stands ahead of a normed result")
+            for _, x, _ in m.parts():
+                if isinstance(x, ChannelDeltaMixer) and not (x.heads >= 1 and 1 <= x.dim <= 512 and 1 <= x.rank <= 2048):
+                    raise ValueError(f"{self.name}: layer {i}: heads {x.heads} / dim {x.dim} / rank {x.rank}")
+            if self.post_norms:
+                if l.mlp is not None and not (isinstance(l.mlp, GatedUnit) or (isinstance(l.mlp, ExpertMix) and l.mlp.gated)):
+                    raise ValueError(f"{self.name}: layer {i}: ahead of normed results feed-forwards are gated units or mixtures of them")
+            elif isinstance(l.mlp, GatedUnit) or (isinstance(l.mlp, ExpertMix) and l.mlp.gated):
+                raise ValueError(f"{self.name}: layer {i}: {type(l.mlp).__name__} stands ahead of a normed result only")
+            elif not self.parallel and isinstance(l.mlp, (Gelu, ExpertMix)):
                 raise ValueError(f"{self.name}: layer {i}: {type(l.mlp).__name__} stands beside its mixer only")
             if isinstance(l.mlp, ExpertMix):
                 self._check_experts(i, l.mlp)
@@ -461,12 +635,16 @@ class StackConfig:
                 self._check_source(i, m, lambda s: (s.kv_rank, s.rot_dim, s.rot))
         if self.two_norms and (not self.parallel or self.loop is not None):
             raise ValueError(f"{self.name}: a second norm needs layers side by side and no loop")
+        if self.post_norms and (self.parallel or self.width > 16384 or any(not isinstance(m, (GroupedMixer, ChannelDeltaMixer)) for m in self.mixers())):
+            raise ValueError(f"{self.name}: normed results join a stream of up to 16384 values, one sublayer after the other; mixers are attention and channel delta rules")
+        if not self.post_norms and (self.token_shift or self.residual_mult != 1.0 or not self.loop_linear):
+            raise ValueError(f"{self.name}: blended tokens, factors and passes without a linear come with normed results")
 
     def _check_experts(self, i: int, f: ExpertMix) -> None:
         if not (1 <= f.experts <= 1024 and 1 <= f.top <= 32 and f.groups >= 1 and f.experts % f.groups == 0 and 1 <= f.keep <= f.groups
                 and f.top <= f.experts // f.groups * f.keep):
             raise ValueError(f"{self.name}: layer {i}: top {f.top} of {f.experts} experts in {f.keep} of {f.groups} groups")
-        if not self.two_norms:
+        if not self.two_norms and not self.post_norms:
             raise ValueError(f"{self.name}: layer {i}: a mixture of experts reads a norm of its own")
 
     def _check_source(self, i: int, m: Mixer, sizes) -> None:
@@ -478,8 +656,12 @@ class StackConfig:
             raise ValueError(f"{self.name}: layer {i} cannot read the keys and values of layer {m.kv_from}")
 
     def _check_grouped(self, i: int, m: GroupedMixer) -> None:
-        if m.heads % m.kv_heads or m.chunk < 0 or m.dim > 2048 or m.vdim > 2048:
-            raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / chunk {m.chunk} / dim {m.dim} / vdim {m.vdim}")
+        if m.heads % m.kv_heads or m.chunk < 0 or m.window < 0 or (m.chunk and m.window) or m.dim > 2048 or m.vdim > 2048:
+            raise ValueError(f"{self.name}: layer {i}: heads {m.heads} / kv_heads {m.kv_heads} / chunk {m.chunk} / window {m.window} / dim {m.dim} / vdim {m.vdim}")
+        if m.taps and (m.kv_from is not None or m.qk_norm or m.gate or not self.post_norms):
+            raise ValueError(f"{self.name}: layer {i}: a convolution of q, k and v comes with keys of its own, without a norm per head or a gate")
+        if m.out_bias and not self.post_norms:
+            raise ValueError(f"{self.name}: layer {i}: a bias behind the output stands ahead of a normed result")
         if m.rot is not None and (m.rot.dims % 2 or m.rot.dims > min(m.dim, 1024) or m.rot.interleaved):
             raise ValueError(f"{self.name}: layer {i}: rotation of {m.rot.dims} of {m.dim} values")
         self._check_source(i, m, lambda s: (s.kv_heads, s.dim, s.vdim, s.rot))
@@ -494,7 +676,7 @@ class StackConfig:
         return sum(self.layers[r.layer].mixer.page_token_bytes(elem) for r in self.runs)
 
     def slot_bytes(self) -> int:
-        return sum(self.layers[r.layer].mixer.slot_bytes() for r in self.runs)
+        return sum(self.layers[r.layer].mixer.slot_bytes() + (4 * self.width if self.token_shift else 0) for r in self.runs)
 
     def expanded_token_bytes(self, elem: int = 2) -> int:
         return max([l.mixer.expanded_token_bytes(elem) for l in self.layers if isinstance(l.mixer, LatentMixer)], default=0)
@@ -505,6 +687,16 @@ class StackConfig:
     def expert_row_bytes(self, rows: int, elem: int = 2) -> int:
         """Scratch of the routed rows of a step (one layer at a time)."""
         return max([rows * l.mlp.top * elem * (l.mlp.ff + self.width) for l in self.layers if isinstance(l.mlp, ExpertMix)], default=0)
+
+    def scan_row_bytes(self, rows: int) -> int:
+        """Scratch of the prompt scans of channel delta rules and of convolved queries, keys and values (one layer at a time)."""
+        n = [0]
+        for m in self.mixers():
+            if isinstance(m, ChannelDeltaMixer):
+                n.append(m.heads * (17 * m.dim_pad + 32 + 4 * m.vdim_pad + 64) // 4 + m.heads * m.vdim_pad)
+            elif isinstance(m, GroupedMixer) and m.taps:
+                n.append(m.channels + 32)
+        return 4 * rows * max(n)
 
     def param_count(self) -> int:
         from .stack_weights import tensor_shapes
@@ -518,7 +710,7 @@ class StackConfig:
 
 
 # ------------------------------------------------------------------------------------ Renosun
-def renosun_from_json(doc: dict, name: str = "renosun", source: Optional[str] = None, max_ctx: int = 32768) -> StackConfig:
+def renosun_from_json(doc: dict, name: str = "renosun", source: Optional[str] = None, max_ctx: int = 32768, shapes: Optional[dict] = None) -> StackConfig:
     layers = []
     for i, l in enumerate(doc["layers"]):
         m = l["mixer"]
@@ -543,7 +735,7 @@ def renosun_from_json(doc: dict, name: str = "renosun", source: Optional[str] = 
 
 
 # ------------------------------------------------------------------------------------ Tepavik
-def tepavik_from_json(doc: dict, name: str = "tepavik", source: Optional[str] = None, max_ctx: int = 32768) -> StackConfig:
+def tepavik_from_json(doc: dict, name: str = "tepavik", source: Optional[str] = None, max_ctx: int = 32768, shapes: Optional[dict] = None) -> StackConfig:
     layers = []
     for i, l in enumerate(doc["layers"]):
         m = l["mixer"]
@@ -567,7 +759,7 @@ def tepavik_from_json(doc: dict, name: str = "tepavik", source: Optional[str] = 
 
 
 # ------------------------------------------------------------------------------------ Fitatar
-def fitatar_from_json(doc: dict, name: str = "fitatar", source: Optional[str] = None, max_ctx: int = 32768) -> StackConfig:
+def fitatar_from_json(doc: dict, name: str = "fitatar", source: Optional[str] = None, max_ctx: int = 32768, shapes: Optional[dict] = None) -> StackConfig:
     layers = []
     for i, l in enumerate(doc["layers"]):
         m, f = l["mixer"], l.get("mlp")
@@ -594,10 +786,42 @@ def fitatar_from_json(doc: dict, name: str = "fitatar", source: Optional[str] = 
                        source=source, max_ctx=max_ctx)
 
 
-ARCHITECTURES = {"Renosun": renosun_from_json, "Tepavik": tepavik_from_json, "Fitatar": fitatar_from_json}
+# ------------------------------------------------------------------------------------ Sofunex
+def sofunex_from_json(doc: dict, name: str = "sofunex", source: Optional[str] = None, max_ctx: int = 32768, shapes: Optional[dict] = None) -> StackConfig:
+    layers = []
+    for i, l in enumerate(doc["layers"]):
+        m, f = l["mixer"], l.get("mlp")
+        if l["type"] != "parallel":
+            raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
+        a, d, w1 = m["left"], m["right"], f"l{i}.mix.right.w1"
+        if shapes is None or w1 not in shapes:
+            raise ValueError(f"layer {i}: the size of tensor {w1!r} is missing (decays pass through that many values)")
+        left = GroupedMixer(a["heads"], a["kv_heads"], a["dim"], a["vdim"], float(a["scale"]), qk_norm=False, rot=Rotation.from_json(a["rot"]),
+                            window=(a.get("mask") or {}).get("size", 0), taps=a["conv"], out_bias=True)
+        mixer = SideBySideMixer(left, ChannelDeltaMixer(d["heads"], d["dim"], shapes[w1][0]), float(m["left_scale"]), float(m["right_scale"]))
+        if f is None:
+            mlp = None
+        elif f["kind"] == "dense":
+            mlp = GatedUnit(f["ff"], "gelu_tanh")
+        elif f["kind"] == "moe":
+            r, g = f["router"], f["router"].get("groups") or {}
+            mlp = ExpertMix(r["experts"], r["top"], f["expert"]["ff"], g.get("count", 1), g.get("keep", 1), (f.get("shared") or {}).get("ff", 0),
+                            gated=True, sigmoid=True, scale=float(r["scale"]))
+        else:
+            raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+        layers.append(LayerSpec(mixer, mlp))
+    lp = doc.get("loop")
+    return StackConfig(name=name, arch="Sofunex", vocab=doc["vocab"], width=doc["width"], layers=tuple(layers), eps=float(doc["norm"]["eps"]),
+                       embed_scale=float(doc["embedding"]["scale"]), parallel=False, post_norms=True, residual_mult=float(doc["residual_mult"]),
+                       token_shift=True, loop=None if lp is None else LoopSpec(lp["start"], lp["stop"], lp["times"]), loop_linear=False,
+                       source=source, max_ctx=max_ctx)
+
+
+ARCHITECTURES = {"Renosun": renosun_from_json, "Tepavik": tepavik_from_json, "Fitatar": fitatar_from_json, "Sofunex": sofunex_from_json}
 
 
 def from_json(doc: dict, **kw) -> StackConfig:
+    """shapes: sizes of the model's tensors by name, where its description alone does not settle all of them."""
     arch = doc.get("architecture")
     if arch not in ARCHITECTURES:
         raise KeyError(f"unknown architecture {arch!r}; known: {sorted(ARCHITECTURES)}")
@@ -611,7 +835,16 @@ def is_model_dir(path: str) -> bool:
 def load_dir(path: str) -> StackConfig:
     """The description in a model folder (config.json beside model.safetensors)."""
     p = Path(path)
-    return from_json(json.loads((p / "config.json").read_text()), name=p.resolve().name, source=str(p))
+    return from_json(json.loads((p / "config.json").read_text()), name=p.resolve().name, source=str(p), shapes=file_shapes(p / "model.safetensors"))
+
+
+def file_shapes(path) -> Optional[dict]:
+    """Tensor sizes of a safetensors file, from its header (None: there is no such file)."""
+    if not os.path.isfile(path):
+        return None
+    with open(path, "rb") as f:
+        (n,) = struct.unpack("<Q", f.read(8))
+        return {name: tuple(d["shape"]) for name, d in json.loads(f.read(n)).items() if name != "__metadata__"}
 
 
 # ---- built-in descriptions (random weights)
@@ -681,7 +914,34 @@ def fitatar_bench(name: str, width: int, ff: int, heads: int, kv_heads: int, exp
     return StackConfig(name, "Fitatar", vocab=vocab, width=width, layers=tuple(layers), embed_scale=width ** 0.5, two_norms=True, logit_cap=30.0)
 
 
-NAMED = {"fitatar-mini": fitatar_mini,
+def sofunex_mini() -> StackConfig:
+    """Small sizes for smoke tests and demos."""
+    def mix(heads, kv_heads, window):
+        a = GroupedMixer(heads, kv_heads, 48, 40, 0.14, qk_norm=False, rot=Rotation(1e4, 32, factor=2.0), window=window, taps=4, out_bias=True)
+        return SideBySideMixer(a, ChannelDeltaMixer(5, 56, 24), 0.7, 0.4)
+    dense, moe = GatedUnit(448, "gelu_tanh"), ExpertMix(12, 3, 96, 3, 2, 160, gated=True, sigmoid=True, scale=1.5)
+    layers = (LayerSpec(mix(6, 2, 192), dense), LayerSpec(mix(4, 4, 100), moe), LayerSpec(mix(6, 2, 192), moe), LayerSpec(mix(4, 1, 192), dense))
+    return StackConfig("sofunex-mini", "Sofunex", vocab=1024, width=288, layers=layers, embed_scale=10.0, parallel=False, post_norms=True,
+                       residual_mult=0.5, token_shift=True, loop=LoopSpec(1, 3, 2), loop_linear=False, max_ctx=4096)
+
+
+def sofunex_bench(name: str, width: int, ff: int, heads: int, kv_heads: int, expert_ff: int, experts: int = 64, top: int = 6, shared: int = 2,
+                  window: int = 8192, n_layers: int = 8, vocab: int = 65536) -> StackConfig:
+    """Layers of a real model's size: attention and a delta rule of the stream's width side by side; a dense layer in four, else
+    mixtures of experts; the third and fourth layer run twice."""
+    a = GroupedMixer(heads, kv_heads, 128, 128, 128 ** -0.5, qk_norm=False, rot=Rotation(1e6, 128, factor=4.0), window=window, taps=4, out_bias=True)
+    mixer = SideBySideMixer(a, ChannelDeltaMixer(heads, 128, 96), 0.6, 0.6)
+    moe = ExpertMix(experts, top, expert_ff, 8, 4, shared * expert_ff, gated=True, sigmoid=True, scale=2.0)
+    layers = tuple(LayerSpec(mixer, moe if i % 4 else GatedUnit(ff, "gelu_tanh")) for i in range(n_layers))
+    return StackConfig(name, "Sofunex", vocab=vocab, width=width, layers=layers, embed_scale=width ** 0.5, parallel=False, post_norms=True,
+                       residual_mult=0.3, token_shift=True, loop=LoopSpec(2, 4, 2), loop_linear=False)
+
+
+NAMED = {"sofunex-mini": sofunex_mini,
+         "sofunex-2k": lambda: sofunex_bench("sofunex-2k", 2048, 6144, 16, 4, 768),
+         "sofunex-4k": lambda: sofunex_bench("sofunex-4k", 4096, 12288, 32, 8, 1024),
+         "sofunex-5k": lambda: sofunex_bench("sofunex-5k", 5120, 13824, 40, 8, 1536),
+         "fitatar-mini": fitatar_mini,
          "fitatar-2k": lambda: fitatar_bench("fitatar-2k", 2048, 8192, 16, 4, 1024),
          "fitatar-4k": lambda: fitatar_bench("fitatar-4k", 4096, 16384, 32, 8, 1536),
          "fitatar-5k": lambda: fitatar_bench("fitatar-5k", 5120, 20480, 40, 8, 2048),

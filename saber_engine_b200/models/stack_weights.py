@@ -7,11 +7,13 @@ whole tiles of its own ahead of them), then the feed-forward's rows as tiles of 
 features, 256 up rows, or 248 up rows and the row of their gate.  `out` holds the mixer's output columns and the down
 columns side by side, so that one product adds both sublayers to the stream.  Where the feed-forward reads a norm of its
 own, its rows (a router's first) start at a tile of their own and multiply the second operand.  One after the other, `proj` and
-`out` belong to the mixer alone and `up` and `down` to the feed-forward behind its own norm.  The routed experts of a mixture
-are stacks of tiles, expert after expert.
+`out` belong to the mixer alone and `up` and `down` to the feed-forward behind its own norm (a router's rows ahead of the shared
+expert's).  Mixers side by side share `proj` and `out`, part after part.  The routed experts of a mixture are stacks of tiles,
+expert after expert.
 """
 from __future__ import annotations
 
+import dataclasses
 import json
 import math
 import mmap
@@ -23,7 +25,7 @@ from typing import Callable, Optional
 import torch
 
 from ..ops import layouts as L
-from .stack_config import ClampedGlu, DeltaMixer, ExpertMix, Gelu, GroupedMixer, LatentMixer, OuterMixer, StackConfig
+from .stack_config import ChannelDeltaMixer, ClampedGlu, DeltaMixer, ExpertMix, Gelu, GroupedMixer, LatentMixer, OuterMixer, StackConfig
 
 _ST_DTYPES = {"BF16": torch.bfloat16, "F32": torch.float32, "F16": torch.float16, "I32": torch.int32, "I64": torch.int64}
 
@@ -50,11 +52,17 @@ def tensor_shapes(cfg: StackConfig) -> dict:
     """Tensor names and shapes."""
     w, t = cfg.width, {"embed": (cfg.vocab, cfg.width)}
     if cfg.loop is not None:
-        t["loop.in"], t["loop.step"] = (w, 2 * w), (cfg.loop.times, w)
+        if cfg.loop_linear:
+            t["loop.in"] = (w, 2 * w)
+        t["loop.step"] = (cfg.loop.times, w)
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.", l.mixer
         rows, bias = dict(m.segments()), m.biases()
         t[p + "norm1"] = (w,)
+        if cfg.post_norms:
+            t[p + "norm1b"] = (w,)
+        if cfg.token_shift:
+            t[p + "shift"] = (w,)
         for seg, tensor, first in m.sources():
             have = t.get(f"{p}mix.{tensor}", (0, w))[0]
             t[f"{p}mix.{tensor}"] = (max(have, first + rows[seg]), w)
@@ -62,10 +70,15 @@ def tensor_shapes(cfg: StackConfig) -> dict:
                 t[f"{p}mix.{tensor}.b"] = (rows[seg],)
         for name, shape in m.extra_shapes().items():
             t[f"{p}mix.{name}"] = shape
-        t[p + "mix.o"] = (w, m.out_features)
+        for name, features, has_bias in m.out_tensors():
+            t[f"{p}mix.{name}"] = (w, features)
+            if has_bias:
+                t[f"{p}mix.{name}.b"] = (w,)
         if l.mlp is not None:
             if not cfg.parallel or cfg.two_norms:
                 t[p + "norm2"] = (w,)
+            if cfg.post_norms:
+                t[p + "norm2b"] = (w,)
             t.update({f"{p}mlp.{name}": shape for name, shape in l.mlp.shapes(w).items()})
     t["final.norm"], t["head"] = (w,), (cfg.vocab, w)
     return t
@@ -73,13 +86,17 @@ def tensor_shapes(cfg: StackConfig) -> dict:
 
 def random_tensor(name: str, shape: tuple, g: torch.Generator, device, norm_offset: float = 0.0) -> torch.Tensor:
     leaf = name.rsplit(".", 1)[-1]
-    if leaf in ("norm1", "norm2", "norm"):
+    if leaf in ("norm1", "norm2", "norm", "norm1b", "norm2b"):
         around = norm_offset if ".mix." not in name else 0.0            # (a mixer's own norm is stored plain)
         return torch.full(shape, 1.0 - around, dtype=torch.bfloat16, device=device)
     if leaf in ("D", "sink"):
         return torch.ones(shape, dtype=torch.bfloat16, device=device)
-    if leaf == "b":
+    if leaf in ("b", "correction"):
         return torch.zeros(shape, dtype=torch.bfloat16, device=device)
+    if leaf == "shift":
+        return torch.rand(shape, generator=g, device=device).bfloat16()
+    if leaf == "w0":
+        return (torch.rand(shape, generator=g, device=device) * 6 - 7).bfloat16()
     if leaf == "A_log":
         return torch.log(torch.rand(shape, generator=g, device=device) * 15 + 1).bfloat16()
     if leaf == "dt_bias":
@@ -121,6 +138,21 @@ class StackLayer:
     out_bias: Optional[torch.Tensor] = None # fp32, of `out`
     experts_up: Optional[Linear] = None     # stacks of routed experts: N_pad and K of one
     experts_down: Optional[Linear] = None
+    up_off: dict = field(default_factory=dict)      # stored columns of `up` (a router's)
+    up_plain: int = 0
+    up_tile0: int = 0                       # first tile of its activations
+    post1: Optional[torch.Tensor] = None    # norms of the sublayers' results (these and the rows below padded to 8)
+    post2: Optional[torch.Tensor] = None
+    shift: Optional[torch.Tensor] = None    # blend with the token before
+    correction: Optional[torch.Tensor] = None
+    mix_k0: dict = field(default_factory=dict)      # part of the mixer -> first column of `out`'s operand
+
+    def part(self, prefix: str) -> "StackLayer":
+        """One of the mixers side by side: its own names in `off` and `extra`."""
+        if not prefix:
+            return self
+        own = lambda d: {k[len(prefix):]: v for k, v in d.items() if k.startswith(prefix)}     # noqa: E731
+        return dataclasses.replace(self, off=own(self.off), extra=own(self.extra))
 
     def linears(self) -> list:
         return [x for x in (self.proj, self.out, self.up, self.down, self.carry, self.experts_up, self.experts_down) if x is not None]
@@ -184,6 +216,14 @@ def project_layout(mixer, mlp, two_norms: bool = False) -> ProjectLayout:
     return ProjectLayout(off, n, tile2, tile0, (tile0 + (mlp.tiles if mlp is not None else 0)) * 256, lat)
 
 
+def gated_rows(gate: torch.Tensor, up: torch.Tensor, KW: int) -> torch.Tensor:
+    """gate, up [ff, width] -> [tiles * 256, KW]: tiles of 128 gate and 128 up rows of the same features."""
+    ff, W = gate.shape
+    out = torch.zeros(L.round_up(ff, 128), 2, KW, dtype=gate.dtype, device=gate.device)
+    out[:ff, 0, :W], out[:ff, 1, :W] = gate, up
+    return out.view(-1, 128, 2, KW).transpose(1, 2).reshape(-1, KW)
+
+
 def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dtype, device) -> StackWeights:
     """Device layouts from `get(name)` (a tensor of the shape in `tensor_shapes`)."""
     dev = torch.device(device)
@@ -200,6 +240,86 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
     W = cfg.width
     KW, NW = L.round_up(W, 64), L.round_up(W, 256)
     zeros = lambda n, k: torch.zeros(n, k, dtype=torch.bfloat16 if dtype != torch.float32 else torch.float32, device=dev)   # noqa: E731
+    wide = L.round_up(W, 8)
+
+    def row(name: str) -> torch.Tensor:
+        """A vector of the stream's width, zeros up to a multiple of 8."""
+        out = torch.zeros(wide, dtype=torch.float32, device=dev)
+        out[:W] = f32(name)
+        return out
+
+    def experts(p: str, f: ExpertMix) -> tuple:
+        """The stacks of a mixture's routed experts."""
+        eu = zeros(f.experts, (L.round_up(f.ff, 128) * 2 if f.gated else L.round_up(f.ff, 256)) * KW).view(f.experts, -1, KW)
+        ed = zeros(f.experts, NW * L.round_up(f.ff, f.k_step)).view(f.experts, NW, -1)
+        for e in range(f.experts):
+            if f.gated:
+                eu[e] = gated_rows(t(f"{p}mlp.e{e}.gate").to(eu.dtype), t(f"{p}mlp.e{e}.up").to(eu.dtype), KW)
+            else:
+                eu[e, : f.ff, :W] = t(f"{p}mlp.e{e}.up")
+            ed[e, :W, : f.ff] = t(f"{p}mlp.e{e}.down")
+        return pack_experts(eu, dtype), pack_experts(ed, dtype)
+
+    def mixer_tensors(m, p: str) -> tuple:
+        """Tensors beside the projections as a mixer's kernels read them, and the linear from a query latent."""
+        extra, carry = {}, None
+        if isinstance(m, DeltaMixer):
+            extra["conv"] = torch.cat([f32(f"{p}{n}.conv") for n in ("q", "k", "v")]).contiguous()
+            for n in ("A_log", "dt_bias", "norm"):
+                extra[n] = f32(f"{p}{n}")
+        elif isinstance(m, OuterMixer):
+            for n in ("norm", *(("A_log", "dt_bias", "D") if m.decay is None else ())):
+                extra[n] = f32(f"{p}{n}")
+            if m.decay is not None:
+                extra["decay"] = torch.tensor(m.decay, dtype=torch.float32, device=dev)
+            if m.taps:                                                 # stored v | k | q, read q | k | v
+                kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
+                for n, key in (("conv", "conv"), ("conv.b", "conv_b")):
+                    c = f32(f"{p}{n}")
+                    extra[key] = torch.cat([c[vd + kd:], c[vd: vd + kd], c[:vd]]).contiguous()
+        elif isinstance(m, LatentMixer):
+            if m.kv_from is None:
+                extra["dkv_norm"] = f32(p + "dkv.norm")
+            if m.q_rank:
+                extra["dq_norm"] = f32(p + "dq.norm")
+                c = zeros(L.round_up(m.query_rows, 256), L.round_up(m.q_rank, 64))
+                c[: m.query_rows, : m.q_rank] = t(p + "uq")
+                carry = pack_linear(c, dtype)
+            for n in ("uk", "uv"):                                     # row stride: the padded latent
+                full = t(f"{p}{n}")
+                extra[n] = torch.zeros(full.shape[0], m.rank_pad, dtype=dtype, device=dev)
+                extra[n][:, : m.kv_rank] = full
+        elif isinstance(m, GroupedMixer):
+            if m.sink:
+                extra["sink"] = f32(p + "sink")
+            if m.taps:
+                extra["conv"] = torch.cat([f32(f"{p}{n}.conv") for n in ("q", "k", "v")]).contiguous()
+                extra["q_norm"], extra["k_norm"] = f32(p + "q.norm"), f32(p + "k.norm")
+        elif isinstance(m, ChannelDeltaMixer):
+            extra["w2"] = t(p + "w2").T.to(dtype).contiguous()         # [rank][channel]
+            extra["w0"], extra["norm"] = f32(p + "w0"), f32(p + "norm")
+        if getattr(m, "rot", None) is not None:
+            extra["freq"] = torch.tensor(m.rot.frequencies() or [1.0], dtype=torch.float32, device=dev)
+        return extra, carry
+
+    def gated_feed_forward(lw: StackLayer, p: str, f) -> None:
+        """`up`: a router's rows as stored columns, then tiles of gate and up rows; `down`."""
+        mix, at = isinstance(f, ExpertMix), "shared." if isinstance(f, ExpertMix) else ""
+        if mix:
+            lw.up_off, lw.up_plain = {"router": 0}, L.round_up(f.experts, 8)
+            lw.experts_up, lw.experts_down = experts(p, f)
+            lw.correction = f32(p + "mlp.correction") if f.sigmoid else None
+        lw.up_tile0 = (lw.up_plain + 255) // 256
+        u = zeros((lw.up_tile0 + (f.tiles if f.inner else 0)) * 256, KW)
+        if mix:
+            u[: f.experts, :W] = t(p + "mlp.router")
+        if f.inner:
+            u[lw.up_tile0 * 256:] = gated_rows(t(f"{p}mlp.{at}gate").to(u.dtype), t(f"{p}mlp.{at}up").to(u.dtype), KW)
+            d = zeros(NW, L.round_up(f.inner, 128))
+            d[:W, : f.inner] = t(f"{p}mlp.{at}down")
+            lw.down = pack_linear(d, dtype)
+        lw.up = pack_linear(u, dtype)
+
     layers = []
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.", l.mixer
@@ -214,17 +334,19 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
             for name, tensor, first in m.sources():
                 if name in m.biases():
                     bias[off[name]: off[name] + seg_rows[name]] = f32(f"{p}mix.{tensor}.b")
-        mix_k = L.round_up(m.out_features, 64)
-        ff_k = L.round_up(beside.inner, 128 if isinstance(beside, ClampedGlu) else 64) if beside is not None else 0
+        mix_k0, mix_k = {}, 0
+        for (pre, _, _), (_, features, _) in zip(m.parts(), m.out_tensors()):
+            mix_k0[pre] = mix_k
+            mix_k += L.round_up(features, 64)
+        ff_k = L.round_up(beside.inner, beside.k_step) if beside is not None else 0
         o = zeros(NW, mix_k + ff_k)
-        o[:W, : m.out_features] = t(p + "mix.o")
         act_bias = out_bias = ex_up = ex_down = None
+        for (pre, _, scale), (name, features, has_bias) in zip(m.parts(), m.out_tensors()):
+            o[:W, mix_k0[pre]: mix_k0[pre] + features] = t(f"{p}mix.{name}")
+            if has_bias:                                               # (the parts' factors are on their results otherwise)
+                out_bias = scale * row(f"{p}mix.{name}.b") + (0 if out_bias is None else out_bias)
         if isinstance(beside, ClampedGlu):
-            gu = r[tile0 * 256:].view(-1, 2, 128, KW)                  # [tile][gate | up][feature][K]
-            for half, name in enumerate(("gate", "up")):
-                full = zeros(ff_k, KW)
-                full[: l.mlp.ff, :W] = t(f"{p}mlp.{name}")
-                gu[:, half] = full.view(-1, 128, KW)
+            r[tile0 * 256:] = gated_rows(t(p + "mlp.gate").to(r.dtype), t(p + "mlp.up").to(r.dtype), KW)
             o[:W, mix_k: mix_k + l.mlp.ff] = t(p + "mlp.down")
         elif isinstance(beside, ExpertMix):
             r[off["router"]: off["router"] + beside.experts, :W] = t(p + "mlp.router")
@@ -235,12 +357,7 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
                 tiles[:, : beside.per_tile] = full.view(-1, beside.per_tile, KW)
                 tiles[:, beside.per_tile, :W] = t(p + "mlp.shared.sg")[0]
                 o[:W, mix_k: mix_k + beside.shared] = t(p + "mlp.shared.down")
-            eu, ed = zeros(beside.experts, L.round_up(beside.ff, 256) * KW), zeros(beside.experts, NW * L.round_up(beside.ff, 64))
-            eu, ed = eu.view(beside.experts, -1, KW), ed.view(beside.experts, NW, -1)
-            for e in range(beside.experts):
-                eu[e, : beside.ff, :W], ed[e, :W, : beside.ff] = t(f"{p}mlp.e{e}.up"), t(f"{p}mlp.e{e}.down")
-            ex_up, ex_down = pack_experts(eu, dtype), pack_experts(ed, dtype)
-            del eu, ed
+            ex_up, ex_down = experts(p, beside)
         elif beside is not None:
             r[tile0 * 256: tile0 * 256 + beside.ff, :W] = t(p + "mlp.up")
             o[:W, mix_k: mix_k + beside.ff] = t(p + "mlp.down")
@@ -248,42 +365,22 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
                 act_bias, out_bias = torch.zeros(beside.tiles * 256, dtype=torch.float32, device=dev), f32(p + "mlp.down.b")
                 act_bias[: beside.ff] = f32(p + "mlp.up.b")
         extra, carry = {}, None
-        if isinstance(m, DeltaMixer):
-            extra["conv"] = torch.cat([f32(f"{p}mix.{n}.conv") for n in ("q", "k", "v")]).contiguous()
-            for n in ("A_log", "dt_bias", "norm"):
-                extra[n] = f32(f"{p}mix.{n}")
-        elif isinstance(m, OuterMixer):
-            for n in ("norm", *(("A_log", "dt_bias", "D") if m.decay is None else ())):
-                extra[n] = f32(f"{p}mix.{n}")
-            if m.decay is not None:
-                extra["decay"] = torch.tensor(m.decay, dtype=torch.float32, device=dev)
-            if m.taps:                                                 # stored v | k | q, read q | k | v
-                kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
-                for n, key in (("conv", "conv"), ("conv.b", "conv_b")):
-                    c = f32(f"{p}mix.{n}")
-                    extra[key] = torch.cat([c[vd + kd:], c[vd: vd + kd], c[:vd]]).contiguous()
-        elif isinstance(m, LatentMixer):
-            if m.kv_from is None:
-                extra["dkv_norm"] = f32(p + "mix.dkv.norm")
-            if m.q_rank:
-                extra["dq_norm"] = f32(p + "mix.dq.norm")
-                c = zeros(L.round_up(m.query_rows, 256), L.round_up(m.q_rank, 64))
-                c[: m.query_rows, : m.q_rank] = t(p + "mix.uq")
-                carry = pack_linear(c, dtype)
-            for n in ("uk", "uv"):                                     # row stride: the padded latent
-                full = t(f"{p}mix.{n}")
-                extra[n] = torch.zeros(full.shape[0], m.rank_pad, dtype=dtype, device=dev)
-                extra[n][:, : m.kv_rank] = full
-        elif isinstance(m, GroupedMixer) and m.sink:
-            extra["sink"] = f32(p + "mix.sink")
-        if getattr(m, "rot", None) is not None:
-            extra["freq"] = torch.tensor(m.rot.frequencies() or [1.0], dtype=torch.float32, device=dev)
-        lw = StackLayer(norm(p + "norm1"), pack_linear(r, dtype), pack_linear(o, dtype), off, n_plain, tile0, mix_k, extra, bias,
-                        tile2=lay.tile2, lat_tiles=lay.lat_tiles, carry=carry, act_bias=act_bias, out_bias=out_bias, experts_up=ex_up, experts_down=ex_down)
+        for pre, m, _ in l.mixer.parts():
+            own, carried = mixer_tensors(m, f"{p}mix.{pre}")
+            extra.update({pre + k: v for k, v in own.items()})
+            carry = carry or carried
+        lw = StackLayer(row(p + "norm1") if cfg.post_norms else norm(p + "norm1"), pack_linear(r, dtype), pack_linear(o, dtype), off, n_plain, tile0, mix_k, extra, bias,
+                        tile2=lay.tile2, lat_tiles=lay.lat_tiles, carry=carry, act_bias=act_bias, out_bias=out_bias, experts_up=ex_up, experts_down=ex_down, mix_k0=mix_k0)
         if beside is not None and cfg.two_norms:
             lw.norm2 = norm(p + "norm2")
         del r, o
-        if l.mlp is not None and not cfg.parallel:
+        if cfg.post_norms:
+            lw.post1 = row(p + "norm1b")
+            lw.shift = row(p + "shift") if cfg.token_shift else None
+            if l.mlp is not None:
+                lw.norm2, lw.post2 = row(p + "norm2"), row(p + "norm2b")
+                gated_feed_forward(lw, p, l.mlp)
+        elif l.mlp is not None and not cfg.parallel:
             ff = l.mlp.ff
             u, d = zeros(L.round_up(ff, 256), KW), zeros(NW, L.round_up(ff, 64))
             u[:ff, :W], d[:W, :ff] = t(p + "mlp.up"), t(p + "mlp.down")
@@ -292,8 +389,11 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
         layers.append(lw)
     head = zeros(L.round_up(cfg.vocab, 256), KW)
     head[: cfg.vocab, :W] = t("head")
-    out = StackWeights(t("embed").to(dtype).contiguous(), layers, norm("final.norm"), pack_linear(head, dtype))
-    if cfg.loop is not None:
+    out = StackWeights(t("embed").to(dtype).contiguous(), layers, row("final.norm") if cfg.post_norms else norm("final.norm"), pack_linear(head, dtype))
+    if cfg.loop is not None and not cfg.loop_linear:
+        out.loop_step = torch.zeros(cfg.loop.times, wide, dtype=torch.float32, device=dev)
+        out.loop_step[:, :W] = f32("loop.step")
+    elif cfg.loop is not None:
         li = t("loop.in")
         r = zeros(NW, 2 * KW)
         r[:W, :W], r[:W, KW: KW + W] = li[:, :W], li[:, W:]

@@ -142,7 +142,7 @@ class MoeRouteParams(C.Structure):
     _fields_ = [("logits", P), ("topk_id", P), ("topk_w", P), ("counts", P), ("offsets", P), ("cursors", P),
                 ("tiles", P), ("ntiles", P), ("src_row", P), ("slot_of", P), ("M", I), ("ld", I), ("E", I),
                 ("top_k", I), ("nt", I), ("rows_cap", I), ("e_lo", I), ("e_n", I), ("norm_topk", I),
-                ("logits_f32", P), ("live", P), ("groups", I), ("keep", I)]
+                ("logits_f32", P), ("live", P), ("groups", I), ("keep", I), ("sigmoid", I), ("correction", P), ("scale", F)]
 
 
 class MoeCombineParams(C.Structure):
@@ -224,7 +224,23 @@ class GqaParams(C.Structure):
                 ("counters", P), ("slot_map", P), ("pos", P), ("cu_rows", P), ("kv_len", P), ("block_table", P), ("out", Operand),
                 ("out_k0", I), ("M", I), ("nseq", I), ("H", I), ("G", I), ("D", I), ("DK", I), ("KP", I), ("V", I), ("VP", I), ("page", I),
                 ("n_blocks", I), ("max_blocks", I), ("splits", I), ("f32", I), ("form", I), ("max_rows", I), ("qk_norm", I), ("chunk", I),
-                ("scale", F), ("softcap", F), ("eps", F), ("err", P)]
+                ("scale", F), ("softcap", F), ("eps", F), ("err", P), ("window", I), ("out_scale", F), ("taps", I), ("v_norm", I), ("n_slots", I), ("ldc", I),
+                ("conv_w", P), ("q_w", P), ("k_w", P), ("hist", P), ("slots", P), ("cx", P), ("row_ss", P), ("gate", P), ("ld_gate", I), ("raw", P),
+                ("ld_raw", I), ("rq_off", I), ("rk_off", I), ("rv_off", I)]
+
+
+class CdeltaParams(C.Structure):
+    _fields_ = [("x", P), ("ldx", I), ("r_off", I), ("k_off", I), ("v_off", I), ("a_off", I), ("l_off", I), ("g_off", I), ("w2", P), ("w2_f32", I),
+                ("rank", I), ("w0", P), ("norm_w", P), ("state", P), ("rec", P), ("vb", P), ("o", P), ("cu_rows", P), ("slots", P), ("pos", P),
+                ("out", Operand), ("out_k0", I), ("M", I), ("nseq", I), ("H", I), ("D", I), ("DP", I), ("VP", I), ("n_slots", I), ("eps", F),
+                ("unit_eps", F), ("out_scale", F), ("err", P)]
+
+
+class JoinParams(C.Structure):
+    _fields_ = [("y", P), ("routed", P), ("slot_of", P), ("route_w", P), ("post_w", P), ("step", P), ("table", P), ("ids", P), ("x", P), ("x_out", P),
+                ("norm_w", P), ("op", Operand), ("shift", P), ("state", P), ("cu_rows", P), ("slots", P), ("pos", P), ("M", I), ("width", I), ("ldx", I),
+                ("ldy", I), ("ldr", I), ("routes", I), ("routed_f32", I), ("table_f32", I), ("vocab", I), ("nseq", I), ("n_slots", I), ("rows", I),
+                ("mult", F), ("embed_scale", F), ("eps", F), ("err", P)]
 
 
 def lib() -> C.CDLL:
@@ -362,6 +378,10 @@ def _declare(L: C.CDLL) -> None:
         "saber_ssd_chunk_floats": (C.c_size_t, [C.POINTER(SsdParams)]),
         "saber_gqa_form": (I, [C.POINTER(GqaParams)]),
         "saber_gqa_launch": (I, [C.POINTER(GqaParams), S]),
+        "saber_cdelta_launch": (I, [C.POINTER(CdeltaParams), I, S]),
+        "saber_join_launch": (I, [C.POINTER(JoinParams), S]),
+        "saber_program_add_cdelta": (I, [P, C.POINTER(CdeltaParams), I, C.c_char_p]),
+        "saber_program_add_join": (I, [P, C.POINTER(JoinParams), C.c_char_p]),
         "saber_program_add_ssd": (I, [P, C.POINTER(SsdParams), I, C.c_char_p]),
         "saber_program_add_gqa": (I, [P, C.POINTER(GqaParams), C.c_char_p]),
         "saber_program_add_linear": (I, [P, C.POINTER(LinParams), C.c_char_p]),
@@ -551,6 +571,13 @@ class Program:
 
     def gqa(self, p: "GqaParams", tag: str = "gqa") -> int:
         return self._L.saber_program_add_gqa(self._h, C.byref(p), tag.encode())
+
+    # the delta rule with rates per key channel; normed results joining the stream
+    def cdelta(self, p: "CdeltaParams", single_row: bool, tag: str = "cdelta") -> int:
+        return self._L.saber_program_add_cdelta(self._h, C.byref(p), int(single_row), tag.encode())
+
+    def join(self, p: "JoinParams", tag: str = "join") -> int:
+        return self._L.saber_program_add_join(self._h, C.byref(p), tag.encode())
 
     # ---- execution ---------------------------------------------------------------------------
     @property

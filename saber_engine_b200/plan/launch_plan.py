@@ -273,6 +273,7 @@ def _resolve_stack(manifest: Manifest, device: DeviceProfile, cfg: StackConfig) 
     led.bill("recurrent_state_slots", (manifest.max_seqs + 1) * cfg.slot_bytes())
     led.bill("prefix_cache_snapshots", manifest.prefix_cache_mib << 20)
     led.bill("activation_arenas", rows * 4 * (3 * cfg.width + 3 * cfg.widest_project() + max(l.mlp.inner if l.mlp else 0 for l in cfg.layers)) * 2)
+    led.bill("scan_rows", cfg.scan_row_bytes(rows))
     led.bill("expert_rows", 2 * cfg.expert_row_bytes(rows))
     led.bill("logits", max(manifest.decode_batches) * cfg.vocab * 4 * 2)
     led.bill("splitk_scratch", 256 * 262144 * 4)

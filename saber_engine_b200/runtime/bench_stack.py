@@ -1,6 +1,7 @@
 """Throughput of a layer-by-layer model beside its closest relatives at equal layer sizes: Renosun beside the int4
 hybrid decoder, Tepavik beside Renosun and the hybrid decoder, Fitatar beside Tepavik (grouped-query attention), Renosun (latent
-attention) and the hybrid decoder with a mixture of experts.
+attention) and the hybrid decoder with a mixture of experts, Sofunex beside Fitatar (grouped-query attention, experts), Renosun (delta
+rule) and the hybrid decoder with a mixture of experts.
 
 Prefill: a cold prompt in portions of one rung (device-timed).  Decode: `streams` sequences at the prompt's length,
 one row each (no drafter on either side).  Then every group of launches of one step on its own: the group's
@@ -18,11 +19,12 @@ import torch
 from ..models import config as C
 from ..models.hybrid import HybridModel
 from ..models.stack import StackModel
-from ..models.stack_config import (ClampedGlu, DeltaMixer, GroupedMixer, ExpertMix, LatentMixer, LayerSpec, OuterMixer, Rotation, SquaredRelu,
-                                   StackConfig)
+from ..models.stack_config import (ChannelDeltaMixer, ClampedGlu, DeltaMixer, Gelu, GroupedMixer, ExpertMix, LatentMixer, LayerSpec, OuterMixer, Rotation,
+                                   SideBySideMixer, SquaredRelu, StackConfig)
 from ..models.step import SeqStep, run_bucket
 
-SIZES = ("renosun-2k", "renosun-4k", "renosun-5k", "tepavik-2k", "tepavik-4k", "tepavik-5k", "fitatar-2k", "fitatar-4k", "fitatar-5k")
+SIZES = ("renosun-2k", "renosun-4k", "renosun-5k", "tepavik-2k", "tepavik-4k", "tepavik-5k", "fitatar-2k", "fitatar-4k", "fitatar-5k", "sofunex-2k",
+         "sofunex-4k", "sofunex-5k")
 
 
 def peaks() -> tuple:
@@ -34,12 +36,28 @@ def peaks() -> tuple:
 
 
 def like_models(cfg: StackConfig) -> list:
-    makers = {"Renosun": [like_hybrid], "Tepavik": [like_renosun, like_hybrid], "Fitatar": [like_tepavik, like_renosun, like_hybrid]}[cfg.arch]
+    makers = {"Renosun": [like_hybrid], "Tepavik": [like_renosun, like_hybrid], "Fitatar": [like_tepavik, like_renosun, like_hybrid],
+              "Sofunex": [like_fitatar, like_renosun, like_hybrid]}[cfg.arch]
     return [make(cfg) for make in makers]
 
 
 def experts_of(cfg: StackConfig):
     return next((l.mlp for l in cfg.layers if isinstance(l.mlp, ExpertMix)), None)
+
+
+def mixer_of(cfg: StackConfig, *kinds):
+    return next((m for m in cfg.mixers() if isinstance(m, kinds)), None)
+
+
+def like_fitatar(cfg: StackConfig) -> StackConfig:
+    """Fitatar with the same attention heads, a layer for every layer run, and feed-forwards of the same bytes: its matrices are two, half as
+    wide again, where the other has three."""
+    a, layers = mixer_of(cfg, GroupedMixer), []
+    m = GroupedMixer(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, qk_norm=False, bias=False, rot=a.rot, sink=True, gate=True)
+    for r in cfg.runs:
+        f = cfg.layers[r.layer].mlp
+        layers.append(LayerSpec(m, ExpertMix(f.experts, f.top, f.ff * 3 // 2, f.groups, f.keep, f.shared * 3 // 2) if isinstance(f, ExpertMix) else Gelu(f.ff * 3 // 2)))
+    return StackConfig(f"fitatar-like-{cfg.name}", "Fitatar", vocab=cfg.vocab, width=cfg.width, layers=tuple(layers), two_norms=True, max_ctx=cfg.max_ctx)
 
 
 def like_tepavik(cfg: StackConfig) -> StackConfig:
@@ -54,7 +72,11 @@ def like_tepavik(cfg: StackConfig) -> StackConfig:
 def like_renosun(cfg: StackConfig) -> StackConfig:
     """Renosun with the same width, vocabulary, layers of each sort and attention heads; its gated feed-forward has three
     matrices where the other has two."""
-    a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, GroupedMixer))
+    a = mixer_of(cfg, GroupedMixer)
+    if cfg.arch == "Sofunex":                                  # delta layers only, as many key heads as value heads; gated units on both sides
+        c = mixer_of(cfg, ChannelDeltaMixer)
+        d = LayerSpec(DeltaMixer(c.heads, c.heads, c.dim, c.dim, 4), ClampedGlu(cfg.layers[0].mlp.ff, 7.0))
+        return StackConfig(f"renosun-like-{cfg.name}", "Renosun", vocab=cfg.vocab, width=cfg.width, layers=(d,) * len(cfg.runs), max_ctx=cfg.max_ctx)
     mlp = ClampedGlu(cfg.layers[0].mlp.ff * 2 // 3 // 128 * 128, 7.0)
     d = LayerSpec(DeltaMixer(a.heads, a.heads // 2, 128, 128, 4), mlp)
     la = LayerSpec(LatentMixer(a.heads, 128, 64, 128, 512, 192 ** -0.5, Rotation(1e6, 64)), mlp)
@@ -66,8 +88,7 @@ def like_renosun(cfg: StackConfig) -> StackConfig:
 def like_hybrid(cfg: StackConfig) -> C.HybridConfig:
     """The hybrid decoder with the same width, feed-forward or experts, recurrent heads of 128 and number of layer runs; its gated GQA
     attention has the same query width in heads of 256 and a quarter as many key heads."""
-    a = next(l.mixer for l in cfg.layers if isinstance(l.mixer, (LatentMixer, GroupedMixer)))
-    d = next((l.mixer for l in cfg.layers if isinstance(l.mixer, DeltaMixer)), None)
+    a, d = mixer_of(cfg, LatentMixer, GroupedMixer), mixer_of(cfg, DeltaMixer)
     kh, vh, ff = (d.kv_heads, d.heads, cfg.layers[0].mlp.ff) if d else (a.heads // 2, a.heads, cfg.layers[0].mlp.ff * 2 // 3 // 256 * 256)
     nq, f = max(4, a.heads * a.dim // 256), experts_of(cfg)
     return C.HybridConfig(name=f"hybrid-like-{cfg.name}", n_layers=len(cfg.runs), hidden=cfg.width, n_q_heads=nq, n_kv_heads=max(1, nq // 4),
@@ -90,8 +111,12 @@ def _groups(model, b) -> dict:
             part = t.split(".")
             if part[0][0] == "R" and part[0][1:].isdigit() and part[-1] != "digest":
                 spec = model.cfg.layers[int(part[1][1:])]
-                alone = ("up", "down", "loop_in", "carry", "route", "experts_up", "experts_down")
+                alone = ("loop_in", "carry", "route", "experts_up", "experts_down", "join", "end", "up", "down")
                 label = part[2] if part[2] in ("project", "out", *alone) else "mixer"
+                if isinstance(spec.mixer, SideBySideMixer):
+                    tail = "+experts" if isinstance(spec.mlp, ExpertMix) and label in ("up", "down", "end") else ""
+                    out.setdefault(f"mixer:{part[2]}" if label == "mixer" else label + tail, []).append((i, i + 1))
+                    continue
                 key = label if label in alone else f"{label}:{mixer_name(spec.mixer)}" + ("+experts" if label != "mixer" and isinstance(spec.mlp, ExpertMix) else "")
                 out.setdefault(key, []).append((i, i + 1))
             elif t == "lm_head":
@@ -146,6 +171,8 @@ def _roof(nbytes: float, flops: float) -> float:
 
 def stack_costs(cfg: StackConfig, M: int, nseq: int, ctx_pairs: float, ctx_tokens: float) -> dict:
     """Algorithmic (bytes, FLOPs) per launch group.  ctx_pairs: visible (row, key) pairs; ctx_tokens: keys read."""
+    if cfg.post_norms:
+        return joined_costs(cfg, M, nseq, ctx_pairs, ctx_tokens)
     W, head_rows = cfg.width, min(M, 8)
     out = {"loop_in": (4 * cfg.width ** 2 + M * 10 * cfg.width, 4.0 * M * cfg.width ** 2)}
     for l in cfg.layers:
@@ -181,6 +208,35 @@ def stack_costs(cfg: StackConfig, M: int, nseq: int, ctx_pairs: float, ctx_token
             out[f"mixer:{name}"] = (2 * ctx_tokens * (m.kv_rank + m.rot_dim) + 2 * m.heads * (m.dim + m.vdim) * m.kv_rank
                                     + M * (4 * m.heads * (m.dim + m.rot_dim + m.vdim) + 2 * m.heads * m.vdim), ctx_pairs * pair + carry)
     out["lm_head"] = (2 * cfg.vocab * W, 2.0 * head_rows * cfg.vocab * W)
+    return out
+
+
+def joined_costs(cfg: StackConfig, M: int, nseq: int, ctx_pairs: float, ctx_tokens: float) -> dict:
+    """The same for layers whose sublayers' results are normed ahead of the stream."""
+    W, head_rows = cfg.width, min(M, 8)
+    out = {"lm_head": (2 * cfg.vocab * W, 2.0 * head_rows * cfg.vocab * W)}
+    lin = lambda n, k, stored: (2 * n * k + M * (2 * k + stored), 2.0 * M * n * k)       # noqa: E731  (bytes a row leaves with)
+    for l in cfg.layers:
+        f, segs = l.mlp, sum(n for _, n in l.mixer.segments())
+        out["project"], out["out"] = lin(segs, W, 4 * segs), lin(W, sum(n for _, n, _ in l.mixer.out_tensors()), 4 * W)
+        out["join"] = out["end"] = (M * 14 * W, 0.0)                                     # result, stream, stream, operand
+        for _, m, _ in l.mixer.parts():
+            rows = sum(n for _, n in m.segments())
+            if isinstance(m, ChannelDeltaMixer):
+                out["mixer:channel_delta"] = (2 * 4 * nseq * m.heads * m.dim ** 2 + M * (4 * rows + 2 * m.out_features), M * m.heads * m.dim ** 2 * 9.0)
+            else:
+                part = min(1.0, m.window * nseq / max(ctx_tokens, 1)) if m.window else 1.0
+                out["mixer:attention"] = (2 * part * ctx_tokens * m.kv_heads * (m.dim + m.vdim) + M * (4 * rows + 2 * m.out_features),
+                                          part * ctx_pairs * 2.0 * m.heads * (m.dim + m.vdim))
+        if isinstance(f, ExpertMix):
+            routes, met = M * f.top, f.experts * (1 - (1 - f.top / f.experts) ** M)       # experts that some token chooses, choices alike
+            out["route"] = (M * (4 * f.experts + 16 * f.top), 0.0)
+            out["experts_up"] = (4 * met * f.ff * W + M * 2 * W + routes * 2 * f.ff, 4.0 * routes * f.ff * W)
+            out["experts_down"] = (2 * met * f.ff * W + routes * 2 * (f.ff + W), 2.0 * routes * f.ff * W)
+            out["up+experts"], out["down+experts"] = lin(f.experts + 2 * f.shared, W, 4 * f.experts + 2 * f.shared), lin(W, f.shared, 4 * W)
+            out["end+experts"] = (M * (14 * W + 2 * f.top * W), 0.0)
+        elif f is not None:
+            out["up"], out["down"] = lin(2 * f.ff, W, 2 * f.ff), lin(W, f.ff, 4 * W)
     return out
 
 

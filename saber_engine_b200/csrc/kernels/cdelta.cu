@@ -1,9 +1,10 @@
 // Delta rule with a decay and a removal rate per key channel, free head sizes, fp32 throughout.
 //
 // Prompt portions (ragged rows, any length), in blocks of four tokens: three launches.
-//   prep   decays, unit keys and removal rates, and per block everything that does not depend on the state
-//   scan   the recurrence.  Columns of the state are independent, so a warp owns four value columns for the whole portion: sixteen
-//          lanes split the key dimension, two lane groups take two columns each, the state stays in registers.  With
+//   prep   decays, unit keys and removal rates, and per block everything that does not depend on the state.  W2 tanh(l) of sixteen
+//          tokens is a product on the tensor cores: W2 is bf16, tanh(l) enters as three bf16 parts (24 bits), sums are fp32
+//   scan   the recurrence.  Columns of the state are independent, so a warp owns eight value columns for the whole portion: eight
+//          lanes split the key dimension, four lane groups take two columns each, the state stays in registers.  With
 //          D_ij = w_{j+1} .. w_i (products of decays channel by channel, no quotients), b_i = -rate_i u_i and p_i = u_i^T S_{i-1}:
 //              p_i = (u_i D_{i-1,0})^T S_0 + sum_{j<i} (u_i . D_{i-1,j} k_j) v_j + (u_i . D_{i-1,j} b_j) p_j
 //              o_i = (r_i D_i0)^T S_0 + sum_{j<=i} (r_i . D_ij k_j) v_j + (r_i . D_ij b_j) p_j
@@ -14,20 +15,24 @@
 // Decoding (one row per sequence): all of it in one launch, a CTA per (head, sequence).
 #include "cdelta.h"
 #include "launch.cuh"
+#include "mla_device.cuh"
 #include "ptx_sm100.cuh"
 #include "scan_records.cuh"
 
 namespace saber {
 
 // Record of a block and head, contiguous (one bulk copy): u D_{i-1,0} [4][DP] | r D_i0 [4][DP] | D_4j k [4][DP] | D_4j b [4][DP] |
-// D_40 [DP] | 32 dot products.  Missing tokens of the last block have k = r = v = b = u = 0 and decay 1.
-constexpr int kCdDots = 32;
-__host__ __device__ constexpr int cd_words(int DP) { return 17 * DP + kCdDots; }
+// D_40 [DP] | the dot products: u . D k below the diagonal (6), u . D b (6), 4 unused, r . D k [4][4], r . D b [4][4] (zeros above the
+// diagonal).  Missing tokens of the last block have k = r = v = b = u = 0 and decay 1.
+constexpr int kCdDots = 32;              // those that are not zero by position
+constexpr int kCdTail = 64;                // (records of whole 128 bytes)
+__host__ __device__ constexpr int cd_words(int DP) { return 17 * DP + kCdTail; }
 __host__ __device__ constexpr int cd_uk(int i, int j) { return kk_at(i, j); }                       // j < i
 __host__ __device__ constexpr int cd_ub(int i, int j) { return 6 + kk_at(i, j); }
 __host__ __device__ constexpr int cd_rk(int i, int j) { return 12 + i * (i + 1) / 2 + j; }          // j <= i
 __host__ __device__ constexpr int cd_rb(int i, int j) { return 22 + i * (i + 1) / 2 + j; }
-constexpr int kCdVWords = kBlk * kCols;
+constexpr int kCdCols = 32;              // value columns of a scan CTA
+constexpr int kCdVWords = kBlk * kCdCols;
 constexpr float kCdRate = 0.60653065971263342f;  // exp(-1/2)
 
 __device__ __forceinline__ int cd_slot(const CdeltaParams& p, int j) {
@@ -46,12 +51,15 @@ __device__ __forceinline__ bool cd_block_of_slot(const CdeltaParams& p, int slot
   }
   return false;
 }
-__device__ __forceinline__ float cd_w2(const CdeltaParams& p, int q, int c) {
-  const size_t i = static_cast<size_t>(q) * (p.H * p.D) + c;
-  return p.w2_f32 ? static_cast<const float*>(p.w2)[i] : __bfloat162float(static_cast<const __nv_bfloat16*>(p.w2)[i]);
+__host__ __device__ constexpr int cd_rank_pad(int rank) { return (rank + 15) & ~15; }
+// four values of channel c's row of W2, from q (a multiple of 4) on
+__device__ __forceinline__ float4 cd_w2(const CdeltaParams& p, int c, int q) {
+  const size_t i = static_cast<size_t>(c) * cd_rank_pad(p.rank) + q;
+  if (p.w2_f32) return *reinterpret_cast<const float4*>(static_cast<const float*>(p.w2) + i);
+  const uint2 u = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.w2) + i);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
 }
-__device__ __forceinline__ float cd_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float cd_decay(float z) { return expf(-kCdRate * cd_sigmoid(z)); }
+__device__ __forceinline__ float cd_decay(float z) { return expf(-kCdRate * sigmoid_f32(z)); }
 
 // Sums over the warp of 32 values a lane: lane n gets the sum of value n (a halving exchange, 31 shuffles).
 __device__ __forceinline__ float warp_sums32(float (&v)[32], int lane) {
@@ -67,92 +75,110 @@ __device__ __forceinline__ float warp_sums32(float (&v)[32], int lane) {
   return v[0];
 }
 
-// grid (blocks, ceil(H / 4)), 128 threads; a warp per (block, head); shared memory: tanh of the four tokens' `rank` values
-template <int NI>
-__global__ void __launch_bounds__(128) cdelta_prep_kernel(const __grid_constant__ CdeltaParams p) {
-  pdl_wait();
-  extern __shared__ float4 sm4[];                  // [rank] values of four tokens
-  const int lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5);
-  int j, blk;
-  if (!cd_block_of_slot(p, blockIdx.x, j, blk)) return;
-  if (cd_slot(p, j) < 0) return;
-  constexpr int DP = NI * 32;
-  const int m = p.cu_rows[j] + blk * kBlk, rows = min(kBlk, p.cu_rows[j + 1] - m);
-  const float* x = p.x + static_cast<size_t>(m) * p.ldx;
-  for (int q = threadIdx.x; q < p.rank; q += 128) {
-    float t[kBlk];
+// A store that no load has to wait for (the caller never reads what it writes).
+__device__ __forceinline__ void store_f32(float* p, float v) { asm volatile("st.global.f32 [%0], %1;" ::"l"(p), "f"(v)); }
+
+// The same over eight lanes and values (7 shuffles): lane lg of its eight gets value lg in v[0].
+__device__ __forceinline__ void scan_sums8(float (&v)[8], int lg) {
 #pragma unroll
-    for (int r = 0; r < kBlk; ++r) t[r] = r < rows ? tanhf(x[static_cast<size_t>(r) * p.ldx + p.l_off + q]) : 0.f;
-    sm4[q] = make_float4(t[0], t[1], t[2], t[3]);
+  for (int o = 4; o > 0; o >>= 1) {
+    const bool up = (lg & o) != 0;
+#pragma unroll
+    for (int e = 0; e < o; ++e) {
+      const float keep = up ? v[o + e] : v[e], give = up ? v[e] : v[o + e];
+      v[e] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+    }
   }
-  __syncthreads();
-  if (h >= p.H) return;
-  float inv[kBlk];
+}
+
+// Records of a block (rows live tokens from x on) and head h, by a warp.  mid(): what comes between the loads of the head's projections
+// and their use.  z(i, c, out): the arguments of the decays of channel c (32 i + lane
+// inside the head) of the four tokens, w0 not yet in them.
+template <int NI, typename Mid, typename Z>
+__device__ __forceinline__ void cd_records(const CdeltaParams& p, const float* x, int rows, int h, int slot, int lane, const Mid& mid, const Z& zget) {
+  constexpr int DP = NI * 32;
+  constexpr bool kHold = NI <= 4;                  // every load of the block at once, else of 32 channels at a time
+  const float* xr[kBlk];                           // (rows past the live ones repeat the last, channels past the head its first: not used)
+#pragma unroll
+  for (int r = 0; r < kBlk; ++r) xr[r] = x + static_cast<size_t>(min(r, rows - 1)) * p.ldx + h * p.D;
+  float kh[kHold ? NI : 1][kBlk], ah[kHold ? NI : 1][kBlk], rh[kHold ? NI : 1][kBlk], vh[kHold ? NI : 1][kBlk], w0[kHold ? NI : 1], inv[kBlk];
+  if constexpr (kHold) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int dc = i * 32 + lane < p.D ? i * 32 + lane : 0;
+#pragma unroll
+      for (int r = 0; r < kBlk; ++r) {
+        kh[i][r] = xr[r][p.k_off + dc];
+        ah[i][r] = xr[r][p.a_off + dc];
+        rh[i][r] = xr[r][p.r_off + dc];
+        vh[i][r] = xr[r][p.v_off + dc];
+      }
+      w0[i] = p.w0[h * p.D + dc];
+    }
+  }
+  mid();
 #pragma unroll
   for (int r = 0; r < kBlk; ++r) inv[r] = 0.f;
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
-    const int d = i * 32 + lane;
+    const int d = i * 32 + lane, dc = d < p.D ? d : 0;
 #pragma unroll
     for (int r = 0; r < kBlk; ++r) {
-      const float k = d < p.D && r < rows ? x[static_cast<size_t>(r) * p.ldx + p.k_off + h * p.D + d] : 0.f;
-      inv[r] = fmaf(k, k, inv[r]);
+      const float k = kHold ? kh[kHold ? i : 0][r] : xr[r][p.k_off + dc];
+      inv[r] = fmaf(d < p.D ? k : 0.f, k, inv[r]);
     }
   }
 #pragma unroll
   for (int r = 0; r < kBlk; ++r) inv[r] = 1.f / sqrtf(warp_sum_f(inv[r]) + p.unit_eps);
-  float* o = p.rec + (static_cast<size_t>(blockIdx.x) * p.H + h) * cd_words(DP);
+  float* o = p.rec + (static_cast<size_t>(slot) * p.H + h) * cd_words(DP);
   float dots[kCdDots];
 #pragma unroll
   for (int e = 0; e < kCdDots; ++e) dots[e] = 0.f;
-#pragma unroll 1
+  constexpr int kUnroll = kHold ? NI : 1;
+#pragma unroll kUnroll
   for (int i = 0; i < NI; ++i) {
-    const int d = i * 32 + lane, c = h * p.D + d;
-    float w[kBlk], k[kBlk], b[kBlk], u[kBlk], rr[kBlk];
+    const int d = i * 32 + lane, c = h * p.D + d, dc = d < p.D ? d : 0;
+    float w[kBlk], k[kBlk], b[kBlk], u[kBlk], rr[kBlk], z[kBlk];
     const bool in = d < p.D;
-    {
-      const float z0 = in ? p.w0[c] : 0.f;
-      float z[kBlk] = {z0, z0, z0, z0};
-      if (in) {
-#pragma unroll 8
-        for (int q = 0; q < p.rank; ++q) {
-          const float f = cd_w2(p, q, c);
-          const float4 t = sm4[q];
-          z[0] = fmaf(f, t.x, z[0]);
-          z[1] = fmaf(f, t.y, z[1]);
-          z[2] = fmaf(f, t.z, z[2]);
-          z[3] = fmaf(f, t.w, z[3]);
-        }
-      }
+    if constexpr (!kHold) {
+      w0[0] = p.w0[h * p.D + dc];
 #pragma unroll
       for (int r = 0; r < kBlk; ++r) {
-        const bool live = in && r < rows;
-        const float* xr = x + static_cast<size_t>(r) * p.ldx;
-        w[r] = live ? cd_decay(z[r]) : 1.f;
-        k[r] = live ? xr[p.k_off + c] : 0.f;
-        u[r] = k[r] * inv[r];
-        b[r] = live ? -cd_sigmoid(xr[p.a_off + c]) * u[r] : 0.f;
-        rr[r] = live ? xr[p.r_off + c] : 0.f;
+        kh[0][r] = xr[r][p.k_off + dc];
+        ah[0][r] = xr[r][p.a_off + dc];
+        rh[0][r] = xr[r][p.r_off + dc];
       }
     }
-    // row i of the triangle against j = i, i - 1, ..: the product of the decays between them grows by one at a time
+    zget(i, in ? c : -1, z);
+#pragma unroll
+    for (int r = 0; r < kBlk; ++r) {
+      const bool live = in && r < rows;
+      const int ih = kHold ? i : 0;
+      const float dec = cd_decay(z[r] + w0[ih]), rate = sigmoid_f32(ah[ih][r]);
+      w[r] = live ? dec : 1.f;
+      k[r] = live ? kh[ih][r] : 0.f;
+      u[r] = k[r] * inv[r];
+      b[r] = -rate * u[r];
+      rr[r] = live ? rh[ih][r] : 0.f;
+    }
+    // row t of the triangle against j = t, t - 1, ..: the product of the decays between them grows by one at a time
 #pragma unroll
     for (int t = 0; t < kBlk; ++t) {
-      float g = 1.f;                               // D_tj (read-outs), then D_{t-1,j}: the same ahead of w_t
+      float g = 1.f;                               // D_{t-1,j}
       dots[cd_rk(t, t)] = fmaf(rr[t], k[t], dots[cd_rk(t, t)]);
       dots[cd_rb(t, t)] = fmaf(rr[t], b[t], dots[cd_rb(t, t)]);
+      const float rw = rr[t] * w[t];
 #pragma unroll
       for (int jj = t - 1; jj >= 0; --jj) {
-        const float gk = g * k[jj], gb = g * b[jj];          // D_{t-1,jj}
+        const float gk = g * k[jj], gb = g * b[jj];
         dots[cd_uk(t, jj)] = fmaf(u[t], gk, dots[cd_uk(t, jj)]);
         dots[cd_ub(t, jj)] = fmaf(u[t], gb, dots[cd_ub(t, jj)]);
-        const float rw = rr[t] * w[t];
         dots[cd_rk(t, jj)] = fmaf(rw, gk, dots[cd_rk(t, jj)]);
         dots[cd_rb(t, jj)] = fmaf(rw, gb, dots[cd_rb(t, jj)]);
         g *= w[jj];
       }
       o[t * DP + d] = u[t] * g;                    // g is D_{t-1,0} now
-      o[(kBlk + t) * DP + d] = rr[t] * w[t] * g;
+      o[(kBlk + t) * DP + d] = rw * g;
     }
     float g = 1.f;
 #pragma unroll
@@ -164,23 +190,158 @@ __global__ void __launch_bounds__(128) cdelta_prep_kernel(const __grid_constant_
     o[4 * kBlk * DP + d] = g;
   }
   const float mine = warp_sums32(dots, lane);
-  o[(4 * kBlk + 1) * DP + lane] = mine;
-  const int groups = (p.VP + kCols - 1) / kCols;
-  for (int d = lane; d < groups * kCols; d += 32) {
-    float* vo = p.vb + ((static_cast<size_t>(blockIdx.x) * p.H + h) * groups + d / kCols) * kCdVWords + d % kCols;
+  {
+    float* tail = o + (4 * kBlk + 1) * DP;
+    const int e = lane < 12 ? 0 : lane < 22 ? lane - 12 : lane - 22;                    // r . D k and r . D b in rows of four
+    const int row = e >= 6 ? 3 : e >= 3 ? 2 : e >= 1 ? 1 : 0, at = 4 * row + e - row * (row + 1) / 2;
+    tail[lane < 12 ? lane : lane < 22 ? 16 + at : 32 + at] = mine;
+    if (lane < 12) tail[(lane < 6 ? 16 : 32) + (lane % 6 < 3 ? lane % 6 + 1 : lane % 6 < 5 ? lane % 6 + 3 : 11)] = 0.f;      // 1, 2, 3, 6, 7, 11
+  }
+  const int groups = (p.VP + kCdCols - 1) / kCdCols;
 #pragma unroll
-    for (int r = 0; r < kBlk; ++r) vo[r * kCols] = d < p.D && r < rows ? x[static_cast<size_t>(r) * p.ldx + p.v_off + h * p.D + d] : 0.f;
+  for (int gr = 0; gr < NI; ++gr) {                // (never more than the key's pieces of 32)
+    if (gr >= groups) break;
+    const int d = gr * kCdCols + lane;
+    float* vo = p.vb + ((static_cast<size_t>(slot) * p.H + h) * groups + gr) * kCdVWords + lane;
+#pragma unroll
+    for (int r = 0; r < kBlk; ++r) {
+      const float v = kHold ? vh[kHold ? gr : 0][r] : xr[r][p.v_off + (d < p.D ? d : 0)];
+      vo[r * kCdCols] = d < p.D && r < rows ? v : 0.f;
+    }
+  }
+}
+
+// grid (blocks, ceil(H / 4)), 128 threads; a warp per (block, head); shared memory: tanh of the four tokens' `rank` values
+template <int NI>
+__global__ void __launch_bounds__(128) cdelta_prep_kernel(const __grid_constant__ CdeltaParams p) {
+  pdl_wait();
+  extern __shared__ float4 sm4[];                  // [rank, padded] values of four tokens
+  const int lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5), RK = cd_rank_pad(p.rank);
+  int j, blk;
+  if (!cd_block_of_slot(p, blockIdx.x, j, blk)) return;
+  if (cd_slot(p, j) < 0) return;
+  const int m = p.cu_rows[j] + blk * kBlk, rows = min(kBlk, p.cu_rows[j + 1] - m);
+  const float* x = p.x + static_cast<size_t>(m) * p.ldx;
+  for (int q = threadIdx.x; q < RK; q += 128) {
+    float t[kBlk];
+#pragma unroll
+    for (int r = 0; r < kBlk; ++r) t[r] = r < rows && q < p.rank ? tanhf(x[static_cast<size_t>(r) * p.ldx + p.l_off + q]) : 0.f;
+    sm4[q] = make_float4(t[0], t[1], t[2], t[3]);
+  }
+  __syncthreads();
+  if (h >= p.H) return;
+  cd_records<NI>(p, x, rows, h, blockIdx.x, lane, [] {}, [&](int, int c, float (&z)[kBlk]) {
+#pragma unroll
+    for (int r = 0; r < kBlk; ++r) z[r] = 0.f;
+    if (c < 0) return;
+#pragma unroll 2
+    for (int q = 0; q < RK; q += 4) {
+      const float4 f = cd_w2(p, c, q);
+      const float fa[4] = {f.x, f.y, f.z, f.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float4 t = sm4[q + e];
+        z[0] = fmaf(fa[e], t.x, z[0]);
+        z[1] = fmaf(fa[e], t.y, z[1]);
+        z[2] = fmaf(fa[e], t.z, z[2]);
+        z[3] = fmaf(fa[e], t.w, z[3]);
+      }
+    }
+  });
+}
+
+constexpr int kCdMmaRank = 256;          // largest padded rank of the tensor-core form
+constexpr int kCdMmaHeads = 4;           // heads of a CTA
+
+// The same for bf16 W2, grid (ceil(blocks / 4), ceil(H / kCdMmaHeads)), 128 threads: four blocks (sixteen tokens), a warp per block; the
+// product W2 tanh(l) of a head by all four warps.  Shared memory: tanh in three parts [3][16][RK + 8] bf16, products [16][DP + 4].
+template <int NI>
+__global__ void __launch_bounds__(128) cdelta_prep_mma_kernel(const __grid_constant__ CdeltaParams p) {
+  pdl_wait();
+  constexpr int DP = NI * 32, ZS = DP + 4;
+  extern __shared__ float4 sm4[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, RK = cd_rank_pad(p.rank);
+  const uint32_t ts = smem_u32(sm4), t_row = static_cast<uint32_t>(RK + 8) * 2u, t_part = 16u * t_row;
+  float* zs = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(sm4) + 3 * t_part);
+  const int slot = blockIdx.x * 4 + warp;
+  int j, blk, rows = 0;
+  const float* x = p.x;
+  if (cd_block_of_slot(p, slot, j, blk) && cd_slot(p, j) >= 0) {
+    const int m = p.cu_rows[j] + blk * kBlk;
+    rows = min(kBlk, p.cu_rows[j + 1] - m);
+    x += static_cast<size_t>(m) * p.ldx;
+  }
+  if (__syncthreads_or(rows) == 0) return;
+#pragma unroll
+  for (int r = 0; r < kBlk; ++r)
+    for (int q = lane; q < RK; q += 32) {
+      float t = r < rows && q < p.rank ? tanhf(x[static_cast<size_t>(r) * p.ldx + p.l_off + q]) : 0.f;
+#pragma unroll
+      for (int part = 0; part < 3; ++part) {
+        const __nv_bfloat16 v = __float2bfloat16(t);
+        asm volatile("st.shared.b16 [%0], %1;" ::"r"(ts + part * t_part + (warp * kBlk + r) * t_row + q * 2), "h"(__bfloat16_as_ushort(v)) : "memory");
+        t -= __bfloat162float(v);
+      }
+    }
+  const uint32_t a_row = ts + static_cast<uint32_t>(lane & 15) * t_row + ((lane >> 4) << 4);
+  const __nv_bfloat16* w2 = static_cast<const __nv_bfloat16*>(p.w2);
+  const int h1 = min(p.H, (static_cast<int>(blockIdx.y) + 1) * kCdMmaHeads);
+  for (int h = blockIdx.y * kCdMmaHeads; h < h1; ++h) {
+    auto product = [&] {
+      __syncthreads();                               // (tanh is there; the products of the head before are read)
+      float acc[NI][4] = {};
+      const __nv_bfloat16* wr[NI];
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int d = (warp * NI + i) * 8 + (lane >> 2);
+        wr[i] = w2 + static_cast<size_t>(h * p.D + (d < p.D ? d : 0)) * RK + (lane & 3) * 2;
+      }
+      uint32_t nb[NI][2];                            // the next step's pieces of W2
+      auto fetch = [&](int k0) {
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          nb[i][0] = *reinterpret_cast<const uint32_t*>(wr[i] + k0);
+          nb[i][1] = *reinterpret_cast<const uint32_t*>(wr[i] + k0 + 8);
+        }
+      };
+      fetch(0);
+      for (int k0 = 0; k0 < RK; k0 += 16) {
+        uint32_t a[3][4], bb[NI][2];
+#pragma unroll
+        for (int i = 0; i < NI; ++i) { bb[i][0] = nb[i][0]; bb[i][1] = nb[i][1]; }
+        if (k0 + 16 < RK) fetch(k0 + 16);
+#pragma unroll
+        for (int part = 0; part < 3; ++part) ldsm4(a[part], a_row + part * t_part + k0 * 2);
+#pragma unroll
+        for (int i = 0; i < NI; ++i)                 // (channels past the head: numbers that nothing reads)
+#pragma unroll
+          for (int part = 2; part >= 0; --part) mma16816(acc[i], a[part], bb[i][0], bb[i][1]);
+      }
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        float* d = zs + (lane >> 2) * ZS + (warp * NI + i) * 8 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(d) = make_float2(acc[i][0], acc[i][1]);
+        *reinterpret_cast<float2*>(d + 8 * ZS) = make_float2(acc[i][2], acc[i][3]);
+      }
+      __syncthreads();
+    };
+    if (rows > 0)
+      cd_records<NI>(p, x, rows, h, slot, lane, product, [&](int i, int, float (&z)[kBlk]) {
+#pragma unroll
+        for (int r = 0; r < kBlk; ++r) z[r] = zs[(warp * kBlk + r) * ZS + i * 32 + lane];
+      });
+    else product();
   }
 }
 
 constexpr int kCdStages = 4;             // blocks of four tokens in flight
 constexpr int kCdScanThreads = 160;
 
-// grid (nseq, H, ceil(VP / 16)), 160 threads: four warps of four value columns, each at its own pace, and a warp whose first lane
+// grid (nseq, H, ceil(VP / 32)), 160 threads: four warps of eight value columns, each at its own pace, and a warp whose first lane
 // keeps the copies going
-template <int NJ>
+template <int NI>
 __global__ void __launch_bounds__(kCdScanThreads) cdelta_scan_kernel(const __grid_constant__ CdeltaParams p) {
-  constexpr int DP = NJ * 64;
+  constexpr int DP = NI * 32;
   constexpr int kRec = cd_words(DP);
   constexpr int kStageWords = kRec + kCdVWords;
   extern __shared__ float4 sm4[];
@@ -192,10 +353,10 @@ __global__ void __launch_bounds__(kCdScanThreads) cdelta_scan_kernel(const __gri
   if (n <= 0) return;
   const int slot = cd_slot(p, j);
   if (slot < 0) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
-  const int vb = blockIdx.z * kCols, groups = (p.VP + kCols - 1) / kCols;
-  const int cl = warp * 4 + (lane >> 4) * 2;       // column inside the CTA's 16
-  const bool on = vb + warp * 4 < p.VP;            // VP is a multiple of 8
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 7;
+  const int vb = blockIdx.z * kCdCols, groups = (p.VP + kCdCols - 1) / kCdCols;
+  const int cl = warp * 8 + (lane >> 3) * 2;       // columns inside the CTA's 32
+  const bool on = vb + warp * 8 < p.VP;            // VP is a multiple of 8
   const int blocks = (n + kBlk - 1) / kBlk;
   const uint32_t bar = smem_u32(bars), bar_free = bar + 8 * kCdStages;
   const uint32_t sm_u = smem_u32(sm);
@@ -226,19 +387,19 @@ __global__ void __launch_bounds__(kCdScanThreads) cdelta_scan_kernel(const __gri
     }
     return;
   }
-  f32x2 S[NJ][2][2] = {};                          // [64 keys][pair of keys][column]
+  f32x2 S[NI][2][2] = {};                          // [32 keys][pair of keys][column]
   float* st = p.state + ((static_cast<size_t>(slot) * p.H + h) * p.VP + vb + cl) * DP;
   if (on) {
 #pragma unroll
     for (int c = 0; c < 2; ++c)
 #pragma unroll
-      for (int i = 0; i < NJ; ++i) {
-        const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4);
+      for (int i = 0; i < NI; ++i) {
+        const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(st + static_cast<size_t>(c) * DP + i * 32 + lg * 4);
         S[i][0][c] = f.x;
         S[i][1][c] = f.y;
       }
   }
-  const int tok = lg >> 2, col = (lg >> 1) & 1;    // whose read-out value this lane keeps (lanes 2i, 2i + 1 share one)
+  const int tok = lg >> 1, col = lg & 1;           // whose values this lane keeps
   float* out = p.o + (static_cast<size_t>(r0 + tok) * p.H + h) * p.VP + vb + cl + col;
   const size_t out_step = static_cast<size_t>(kBlk) * p.H * p.VP;
   for (int blk = 0; blk < blocks; ++blk) {
@@ -247,14 +408,14 @@ __global__ void __launch_bounds__(kCdScanThreads) cdelta_scan_kernel(const __gri
     const float* b = sm + s * kStageWords;
     const float* vrec = b + kRec;
     if (on) {
-      float sk[kBlk][2], sq[kBlk][2];
+      float sk[kBlk][2], sq[8];                    // [token][column]
 #pragma unroll
       for (int r = 0; r < kBlk; ++r) {
         f32x2 a[2] = {}, c[2] = {};
 #pragma unroll
-        for (int i = 0; i < NJ; ++i) {
-          const ulonglong2 u4 = *reinterpret_cast<const ulonglong2*>(b + r * DP + i * 64 + lg * 4);
-          const ulonglong2 r4 = *reinterpret_cast<const ulonglong2*>(b + (kBlk + r) * DP + i * 64 + lg * 4);
+        for (int i = 0; i < NI; ++i) {
+          const ulonglong2 u4 = *reinterpret_cast<const ulonglong2*>(b + r * DP + i * 32 + lg * 4);
+          const ulonglong2 r4 = *reinterpret_cast<const ulonglong2*>(b + (kBlk + r) * DP + i * 32 + lg * 4);
 #pragma unroll
           for (int v = 0; v < 2; ++v) {
             a[v] = fma_f2(S[i][0][v], u4.x, a[v]);
@@ -267,79 +428,71 @@ __global__ void __launch_bounds__(kCdScanThreads) cdelta_scan_kernel(const __gri
         for (int v = 0; v < 2; ++v) {
           const float2 e = unpack_f2(a[v]), f = unpack_f2(c[v]);
           sk[r][v] = e.x + e.y;
-          sq[r][v] = f.x + f.y;
+          sq[r * 2 + v] = f.x + f.y;
         }
       }
 #pragma unroll
-      for (int o = 1; o < 16; o <<= 1)
+      for (int o = 1; o < 8; o <<= 1)
 #pragma unroll
         for (int r = 0; r < kBlk; ++r)
 #pragma unroll
           for (int v = 0; v < 2; ++v) sk[r][v] += __shfl_xor_sync(0xffffffffu, sk[r][v], o);
-      // read-out values by halving exchange (4 + 2 + 1 + 1 shuffles)
-      float mine;
-      {
-        float t4[4], t2[2];
-        const bool b3 = (lg & 8) != 0, b2 = (lg & 4) != 0, b1 = (lg & 2) != 0;
+      scan_sums8(sq, lg);
+      const float* tail = b + (4 * kBlk + 1) * DP;
+      float pr[48], held[kBlk][2], val[kBlk][2];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {              // tokens 0, 1 stay with b3 = 0; tokens 2, 3 with b3 = 1
-          const float keep = b3 ? sq[2 + (e >> 1)][e & 1] : sq[e >> 1][e & 1];
-          const float give = b3 ? sq[e >> 1][e & 1] : sq[2 + (e >> 1)][e & 1];
-          t4[e] = keep + __shfl_xor_sync(0xffffffffu, give, 8);
-        }
+      for (int e = 0; e < 48; e += 4)
+        if (e != 12) *reinterpret_cast<float4*>(pr + e) = *reinterpret_cast<const float4*>(tail + e);
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const float keep = b2 ? t4[2 + e] : t4[e], give = b2 ? t4[e] : t4[2 + e];
-          t2[e] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
-        }
-        const float keep = b1 ? t2[1] : t2[0], give = b1 ? t2[0] : t2[1];
-        mine = keep + __shfl_xor_sync(0xffffffffu, give, 2);
-        mine += __shfl_xor_sync(0xffffffffu, mine, 1);
+      for (int i = 0; i < kBlk; ++i) {
+        const float2 v = *reinterpret_cast<const float2*>(vrec + i * kCdCols + cl);
+        val[i][0] = v.x;
+        val[i][1] = v.y;
       }
-      float pr[kCdDots], held[kBlk][2], val[kBlk][2];
-#pragma unroll
-      for (int e = 0; e < kCdDots; e += 4) *reinterpret_cast<float4*>(pr + e) = *reinterpret_cast<const float4*>(b + (4 * kBlk + 1) * DP + e);
       float o = 0.f;
 #pragma unroll
       for (int i = 0; i < kBlk; ++i) {
-        const float2 v = *reinterpret_cast<const float2*>(vrec + i * kCols + cl);
-        val[i][0] = v.x;
-        val[i][1] = v.y;
-        float h0 = sk[i][0], h1 = sk[i][1], t = mine;
 #pragma unroll
-        for (int jj = 0; jj < i; ++jj) {
-          h0 = fmaf(pr[cd_uk(i, jj)], val[jj][0], fmaf(pr[cd_ub(i, jj)], held[jj][0], h0));
-          h1 = fmaf(pr[cd_uk(i, jj)], val[jj][1], fmaf(pr[cd_ub(i, jj)], held[jj][1], h1));
+        for (int v = 0; v < 2; ++v) {
+          float a = sk[i][v];
+#pragma unroll
+          for (int jj = 0; jj < i; ++jj) a = fmaf(pr[cd_uk(i, jj)], val[jj][v], a);      // (what does not wait for `held` first)
+#pragma unroll
+          for (int jj = 0; jj < i; ++jj) a = fmaf(pr[cd_ub(i, jj)], held[jj][v], a);
+          held[i][v] = a;
         }
-        held[i][0] = h0;
-        held[i][1] = h1;
+        float t = sq[0];
 #pragma unroll
         for (int jj = 0; jj <= i; ++jj)
-          t = fmaf(pr[cd_rk(i, jj)], col ? val[jj][1] : val[jj][0], fmaf(pr[cd_rb(i, jj)], col ? held[jj][1] : held[jj][0], t));
+          t = fmaf(pr[16 + 4 * i + jj], col ? val[jj][1] : val[jj][0], fmaf(pr[32 + 4 * i + jj], col ? held[jj][1] : held[jj][0], t));
         o = tok == i ? t : o;
       }
-      if ((lg & 1) == 0 && blk * kBlk + tok < n) out[blk * out_step] = o;
+      if (blk * kBlk + tok < n) store_f32(out + blk * out_step, o);
+      f32x2 v2[kBlk][2], p2[kBlk][2];
 #pragma unroll
-      for (int i = 0; i < NJ; ++i) {
-        const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(b + 4 * kBlk * DP + i * 64 + lg * 4);
+      for (int r = 0; r < kBlk; ++r)
+#pragma unroll
+        for (int v = 0; v < 2; ++v) {
+          v2[r][v] = pack_f2(val[r][v], val[r][v]);
+          p2[r][v] = pack_f2(held[r][v], held[r][v]);
+        }
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(b + 4 * kBlk * DP + i * 32 + lg * 4);
 #pragma unroll
         for (int v = 0; v < 2; ++v) {
           S[i][0][v] = mul_f2(S[i][0][v], g4.x);
           S[i][1][v] = mul_f2(S[i][1][v], g4.y);
         }
-      }
 #pragma unroll
-      for (int r = 0; r < kBlk; ++r) {
-        const f32x2 v0 = pack_f2(val[r][0], val[r][0]), v1 = pack_f2(val[r][1], val[r][1]);
-        const f32x2 p0 = pack_f2(held[r][0], held[r][0]), p1 = pack_f2(held[r][1], held[r][1]);
+        for (int r = 0; r < kBlk; ++r) {
+          const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(b + (2 * kBlk + r) * DP + i * 32 + lg * 4);
+          const ulonglong2 b4 = *reinterpret_cast<const ulonglong2*>(b + (3 * kBlk + r) * DP + i * 32 + lg * 4);
 #pragma unroll
-        for (int i = 0; i < NJ; ++i) {
-          const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(b + (2 * kBlk + r) * DP + i * 64 + lg * 4);
-          const ulonglong2 b4 = *reinterpret_cast<const ulonglong2*>(b + (3 * kBlk + r) * DP + i * 64 + lg * 4);
-          S[i][0][0] = fma_f2(p0, b4.x, fma_f2(v0, k4.x, S[i][0][0]));
-          S[i][0][1] = fma_f2(p1, b4.x, fma_f2(v1, k4.x, S[i][0][1]));
-          S[i][1][0] = fma_f2(p0, b4.y, fma_f2(v0, k4.y, S[i][1][0]));
-          S[i][1][1] = fma_f2(p1, b4.y, fma_f2(v1, k4.y, S[i][1][1]));
+          for (int v = 0; v < 2; ++v) {
+            S[i][0][v] = fma_f2(p2[r][v], b4.x, fma_f2(v2[r][v], k4.x, S[i][0][v]));
+            S[i][1][v] = fma_f2(p2[r][v], b4.y, fma_f2(v2[r][v], k4.y, S[i][1][v]));
+          }
         }
       }
     }
@@ -350,8 +503,8 @@ __global__ void __launch_bounds__(kCdScanThreads) cdelta_scan_kernel(const __gri
 #pragma unroll
     for (int c = 0; c < 2; ++c)
 #pragma unroll
-      for (int i = 0; i < NJ; ++i)
-        *reinterpret_cast<ulonglong2*>(st + static_cast<size_t>(c) * DP + i * 64 + lg * 4) = make_ulonglong2(S[i][0][c], S[i][1][c]);
+      for (int i = 0; i < NI; ++i)
+        *reinterpret_cast<ulonglong2*>(st + static_cast<size_t>(c) * DP + i * 32 + lg * 4) = make_ulonglong2(S[i][0][c], S[i][1][c]);
   }
 }
 
@@ -370,11 +523,11 @@ __global__ void __launch_bounds__(256) cdelta_out_kernel(const __grid_constant__
     for (int v = lane * 4; v < p.D; v += 128) {
       const float4 a = *reinterpret_cast<const float4*>(o + v), b = *reinterpret_cast<const float4*>(g + v), c = *reinterpret_cast<const float4*>(w + v);
       operand_store4(p.out, m, p.out_k0 + h * p.D + v,
-                     make_float4(a.x * r * c.x * cd_sigmoid(b.x), a.y * r * c.y * cd_sigmoid(b.y), a.z * r * c.z * cd_sigmoid(b.z), a.w * r * c.w * cd_sigmoid(b.w)));
+                     make_float4(a.x * r * c.x * sigmoid_f32(b.x), a.y * r * c.y * sigmoid_f32(b.y), a.z * r * c.z * sigmoid_f32(b.z), a.w * r * c.w * sigmoid_f32(b.w)));
     }
     return;
   }
-  for (int v = lane; v < p.D; v += 32) operand_store1(p.out, m, p.out_k0 + h * p.D + v, o[v] * r * w[v] * cd_sigmoid(g[v]));
+  for (int v = lane; v < p.D; v += 32) operand_store1(p.out, m, p.out_k0 + h * p.D + v, o[v] * r * w[v] * sigmoid_f32(g[v]));
 }
 
 template <int NI>
@@ -407,8 +560,8 @@ __global__ void __launch_bounds__(256) cdelta_step_kernel(const __grid_constant_
   float* bs = ws + DP;                             // -rate u
   float* ks = bs + DP;                             // key
   float* zs = ks + DP;                             // [kCdParts][DP]
-  float* ts = zs + kCdParts * DP;                  // [rank, to a multiple of 4] tanh of the shared values
-  float* vs = ts + ((p.rank + 3) & ~3);            // VP
+  float* ts = zs + kCdParts * DP;                  // [rank, padded] tanh of the shared values
+  float* vs = ts + cd_rank_pad(p.rank);            // VP
   float* os = vs + p.VP;                           // VP
   __shared__ float red[3][8];
   const int h = blockIdx.x, j = blockIdx.y;
@@ -424,7 +577,7 @@ __global__ void __launch_bounds__(256) cdelta_step_kernel(const __grid_constant_
   pdl_wait();
   if (slot < 0) return;
   const float* x = p.x + static_cast<size_t>(m) * p.ldx;
-  for (int q = threadIdx.x; q < p.rank; q += nt) ts[q] = tanhf(x[p.l_off + q]);
+  for (int q = threadIdx.x; q < cd_rank_pad(p.rank); q += nt) ts[q] = q < p.rank ? tanhf(x[p.l_off + q]) : 0.f;
   float sum[3] = {0.f, 0.f, 0.f};                  // k . k, r . k, r . rate k
   for (int d = threadIdx.x; d < DP; d += nt) {
     float k = 0.f, r = 0.f, a = 0.f;
@@ -432,7 +585,7 @@ __global__ void __launch_bounds__(256) cdelta_step_kernel(const __grid_constant_
       const int c = h * p.D + d;
       k = x[p.k_off + c];
       r = x[p.r_off + c];
-      a = cd_sigmoid(x[p.a_off + c]);
+      a = sigmoid_f32(x[p.a_off + c]);
     }
     ks[d] = k;
     rs[d] = r;
@@ -454,14 +607,16 @@ __global__ void __launch_bounds__(256) cdelta_step_kernel(const __grid_constant_
     for (int w = 0; w < nw; ++w) sum[i] += red[i][w];
   }
   const float inv = 1.f / sqrtf(sum[0] + p.unit_eps), rk = sum[1], rb = -inv * sum[2];
-  const int per = (p.rank + kCdParts - 1) / kCdParts;
+  const int RK = cd_rank_pad(p.rank), per = RK / kCdParts;
   for (int i = threadIdx.x; i < kCdParts * DP; i += nt) {
     const int part = i / DP, d = i - part * DP;
     float z = 0.f;
     if (d < p.D) {
-      const int q1 = min(p.rank, (part + 1) * per);
-#pragma unroll 8
-      for (int q = part * per; q < q1; ++q) z = fmaf(cd_w2(p, q, h * p.D + d), ts[q], z);
+#pragma unroll 6
+      for (int q = part * per; q < (part + 1) * per; q += 4) {
+        const float4 f = cd_w2(p, h * p.D + d, q), t = *reinterpret_cast<const float4*>(ts + q);
+        z = fmaf(f.x, t.x, fmaf(f.y, t.y, fmaf(f.z, t.z, fmaf(f.w, t.w, z))));
+      }
     }
     zs[i] = z;
   }
@@ -528,7 +683,7 @@ __global__ void __launch_bounds__(256) cdelta_step_kernel(const __grid_constant_
   for (int w = 0; w < nw; ++w) s2 += red[0][w];
   const float r = p.out_scale / sqrtf(s2 / static_cast<float>(p.D) + p.eps);
   for (int v = threadIdx.x; v < p.D; v += nt)
-    operand_store1(p.out, m, p.out_k0 + h * p.D + v, os[v] * r * p.norm_w[h * p.D + v] * cd_sigmoid(x[p.g_off + h * p.D + v]));
+    operand_store1(p.out, m, p.out_k0 + h * p.D + v, os[v] * r * p.norm_w[h * p.D + v] * sigmoid_f32(x[p.g_off + h * p.D + v]));
 }
 
 template <typename Kernel>
@@ -547,14 +702,21 @@ static int cdelta_go(const CdeltaParams& p, bool single, cudaStream_t stream) {
   constexpr int NI = NJ * 2, DP = NJ * 64;
   if (single) {
     const int warps = min(8, p.VP / 8);
-    const int smem = ((5 + kCdParts) * DP + ((p.rank + 3) & ~3) + 2 * p.VP) * 4;
+    const int smem = ((5 + kCdParts) * DP + cd_rank_pad(p.rank) + 2 * p.VP) * 4;
     return static_cast<int>(launch(cdelta_step_kernel<NI>, dim3(p.H, p.nseq), dim3(32 * warps), smem, stream, 2, p));
   }
   static bool ready[64];
   constexpr int smem = kCdStages * (cd_words(DP) + kCdVWords) * 4;
-  cudaError_t e = cd_allow(cdelta_scan_kernel<NJ>, ready, smem);
-  if (e == cudaSuccess) e = launch(cdelta_prep_kernel<NI>, dim3(p.M / kBlk + p.nseq, (p.H + 3) / 4), dim3(128), p.rank * 16, stream, 0, p);
-  if (e == cudaSuccess) e = launch(cdelta_scan_kernel<NJ>, dim3(p.nseq, p.H, (p.VP + kCols - 1) / kCols), dim3(kCdScanThreads), smem, stream, 0, p);
+  cudaError_t e = cd_allow(cdelta_scan_kernel<NI>, ready, smem);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  const int blocks = p.M / kBlk + p.nseq, RK = cd_rank_pad(p.rank);
+  bool mma = false;
+  if constexpr (DP <= 256) mma = !p.w2_f32 && RK <= kCdMmaRank;
+  if constexpr (DP <= 256)
+    if (mma)
+      e = launch(cdelta_prep_mma_kernel<NI>, dim3((blocks + 3) / 4, (p.H + kCdMmaHeads - 1) / kCdMmaHeads), dim3(128), 3 * 16 * (RK + 8) * 2 + 16 * (DP + 4) * 4, stream, 0, p);
+  if (!mma) e = launch(cdelta_prep_kernel<NI>, dim3(blocks, (p.H + 3) / 4), dim3(128), RK * 16, stream, 0, p);
+  if (e == cudaSuccess) e = launch(cdelta_scan_kernel<NI>, dim3(p.nseq, p.H, (p.VP + kCdCols - 1) / kCdCols), dim3(kCdScanThreads), smem, stream, 0, p);
   if (e == cudaSuccess) e = launch(cdelta_out_kernel, dim3(p.M, (p.H + 7) / 8), dim3(256), 0, stream, 0, p);
   return static_cast<int>(e);
 }

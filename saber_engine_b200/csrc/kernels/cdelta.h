@@ -15,13 +15,13 @@ namespace saber {
 struct CdeltaParams {
   const float* x;             // [M][ldx] projections of this step's rows
   int ldx, r_off, k_off, v_off, a_off, l_off, g_off;
-  const void* w2;             // [rank][H D], bf16 (w2_f32: fp32)
+  const void* w2;             // [H D][rank, zeros up to a multiple of 16], bf16 (w2_f32: fp32)
   int w2_f32, rank;
   const float* w0;            // [H D]
   const float* norm_w;        // [H D]
   float* state;               // [n_slots][H][VP][DP] (pads stay zero)
-  float* rec;                 // scratch [M / 4 + nseq][H][17 DP + 32]: blocks of four tokens, see cdelta.cu
-  float* vb;                  // scratch [M / 4 + nseq][H][ceil(VP / 16)][64]
+  float* rec;                 // scratch [M / 4 + nseq][H][17 DP + 64]: blocks of four tokens, see cdelta.cu
+  float* vb;                  // scratch [M / 4 + nseq][H][ceil(VP / 32)][128]
   float* o;                   // scratch [M][H][VP]
   const int32_t* cu_rows;     // [nseq + 1]
   const int32_t* slots;       // [nseq], < 0: padding sequence

@@ -38,13 +38,19 @@ template <> struct Page<float> {
 __device__ __forceinline__ size_t page_block(const GqaParams& p, int page, int g) {
   return (static_cast<size_t>(page) * p.G + g) * kPage * (p.KP + p.VP);
 }
-// which of row m's two sums of squares over all heads belongs to x's part
-__device__ __forceinline__ float row_scale(const GqaParams& p, int m, int isk) {
-  return 1.f / sqrtf(p.row_ss[2 * m + isk] / static_cast<float>((isk ? p.G : p.H) * p.D) + p.eps);
+// reciprocal root mean square of row m's queries (isk: keys) over all heads, by a warp
+constexpr int kConvPart = 256;            // columns of a partial sum
+__host__ __device__ constexpr int conv_parts(int n) { return (n + kConvPart - 1) / kConvPart; }
+__device__ __forceinline__ float row_scale(const GqaParams& p, int m, int isk, int lane) {
+  const int pq = conv_parts(p.H * p.D), pk = conv_parts(p.G * p.D);
+  const float* ss = p.row_ss + static_cast<size_t>(m) * (pq + pk) + (isk ? pq : 0);
+  float s = 0.f;
+  for (int i = lane; i < (isk ? pk : pq); i += 32) s += ss[i];
+  return 1.f / sqrtf(mla_warp_sum(s) / static_cast<float>((isk ? p.G : p.H) * p.D) + p.eps);
 }
 // reciprocal root mean square of the D values of a head of row m (a warp), 1 without the norm
 __device__ __forceinline__ float head_scale(const GqaParams& p, const float* x, int m, int isk, int lane) {
-  if (p.taps > 0) return row_scale(p, m, isk);
+  if (p.taps > 0) return row_scale(p, m, isk, lane);
   if (!p.qk_norm) return 1.f;
   float sq = 0.f;
   for (int d = lane; d < p.D; d += 32) sq = fmaf(x[d], x[d], sq);
@@ -84,77 +90,152 @@ __device__ __forceinline__ void conv_ring(const GqaParams& p, int j) {
       hist[static_cast<size_t>(p.pos[r0 + t] % p.taps) * ch.all() + c] = p.raw[static_cast<size_t>(r0 + t) * p.ld_raw + ch.column(p, c)];
 }
 
-constexpr int kConvThreads = 512;
+constexpr int kConvRows = 8;              // rows of a strip
 
-// grid M, 512 threads: a row.  Columns of cx from x = q, k_off = k, v_off = v on (as the kernels behind it read them).
-__global__ void __launch_bounds__(kConvThreads) gqa_conv_kernel(const __grid_constant__ GqaParams p) {
+template <int VEC> struct ConvVec;
+template <> struct ConvVec<4> { typedef float4 T; };
+template <> struct ConvVec<1> { typedef float T; };
+__device__ __forceinline__ float4 conv_fma(float4 a, float4 b, float4 c) {
+  return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w));
+}
+__device__ __forceinline__ float conv_fma(float a, float b, float c) { return fmaf(a, b, c); }
+__device__ __forceinline__ float conv_dot(float4 a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+__device__ __forceinline__ float conv_dot(float a) { return a * a; }
+__device__ __forceinline__ float4 conv_mul(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float conv_mul(float a, float b) { return a * b; }
+__device__ __forceinline__ float4 conv_scale(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
+__device__ __forceinline__ float conv_scale(float a, float s) { return a * s; }
+
+// Up to kConvRows neighbouring rows of one sequence: the first is row m (its t-th of this step, at position pos).
+struct ConvRun {
+  int m, n, t, pos;
+  float* hist;                            // of the slot, or null
+};
+// Channels c .. c + VEC - 1 (column col of the rows) of a run, convolved.  TAPS: their number when known at compile time, else 0.
+template <int VEC, int TAPS, int ROWS>
+__device__ __forceinline__ void conv_run(const GqaParams& p, const ConvRun& run, int C, int c, int col, typename ConvVec<VEC>::T (&y)[ROWS]) {
+  typedef typename ConvVec<VEC>::T V;
+  const float* x = p.raw + static_cast<size_t>(run.m) * p.ld_raw + col;
+  const float* w = p.conv_w + c;
+  auto input = [&](int i) -> V {          // of row m + i, earlier ones from the ring
+    if (run.t + i >= 0) return *reinterpret_cast<const V*>(x + static_cast<ptrdiff_t>(i) * p.ld_raw);
+    if (run.pos + i >= 0 && run.hist != nullptr) return *reinterpret_cast<const V*>(run.hist + static_cast<size_t>((run.pos + i) % p.taps) * C + c);
+    return V{};
+  };
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) y[r] = V{};
+  if constexpr (TAPS > 0) {
+    V u[TAPS - 1 + ROWS], f[TAPS];
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) f[i] = *reinterpret_cast<const V*>(w + static_cast<size_t>(i) * C);
+#pragma unroll
+    for (int i = 0; i < TAPS - 1 + ROWS; ++i) u[i] = i - (TAPS - 1) < run.n ? input(i - (TAPS - 1)) : V{};
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) y[r] = conv_fma(u[r + i], f[i], y[r]);
+  } else {
+    for (int i = 0; i < p.taps; ++i) {
+      const V f = *reinterpret_cast<const V*>(w + static_cast<size_t>(i) * C);
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r)
+        if (r < run.n) y[r] = conv_fma(input(r - (p.taps - 1) + i), f, y[r]);
+    }
+  }
+  if (p.max_rows == 1 && run.hist != nullptr)                      // (no token of this step reads that row)
+    *reinterpret_cast<V*>(run.hist + static_cast<size_t>(run.pos % p.taps) * C + c) = input(0);
+}
+
+// grid (ceil(M / ROWS), ceil(items / 4)), 128 threads; a warp per strip of rows and item: 256 columns of q, then of k, then a value
+// head.  Columns of cx from 0 = q, k_off = k, v_off = v on (as the kernels behind it read them).
+template <int VEC, int TAPS, int ROWS>
+__global__ void __launch_bounds__(128) gqa_conv_kernel(const __grid_constant__ GqaParams p) {
   pdl_trigger();
   pdl_wait();
-  __shared__ float red[2][kConvThreads / 32];
-  const int m = blockIdx.x, j = mla_seq_of_row(p.cu_rows, p.nseq, m), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (j < 0) return;
-  const int slot = gqa_slot(p, j), t = m - p.cu_rows[j], pos = p.pos[m];
+  typedef typename ConvVec<VEC>::T V;
+  const int lane = threadIdx.x & 31, item = blockIdx.y * 4 + (threadIdx.x >> 5);
   const ConvChannels ch(p);
-  const int C = ch.all();
-  float* hist = slot < 0 ? nullptr : p.hist + static_cast<size_t>(slot) * p.taps * C;
-  const float* raw = p.raw + static_cast<size_t>(m) * p.ld_raw;
-  auto conv = [&](int c) {
-    const int col = ch.column(p, c);
-    const float* w = p.conv_w + static_cast<size_t>(c) * p.taps;
-    const float x = raw[col];
-    float s = x * w[p.taps - 1];
-    for (int back = 1; back < p.taps; ++back) {
-      float u = 0.f;
-      if (back <= t) u = raw[col - static_cast<ptrdiff_t>(back) * p.ld_raw];
-      else if (back <= pos && hist != nullptr) u = hist[static_cast<size_t>((pos - back) % p.taps) * C + c];
-      s = fmaf(u, w[p.taps - 1 - back], s);
-    }
-    if (p.max_rows == 1 && hist != nullptr) hist[static_cast<size_t>(pos % p.taps) * C + c] = x;    // (no token of this step reads that row)
-    return s;
-  };
-  float* o = p.cx + static_cast<size_t>(m) * p.ldc;
-  float sq[2] = {0.f, 0.f};
+  const int C = ch.all(), pq = conv_parts(ch.nq), pk = conv_parts(ch.nk);
+  if (item >= pq + pk + p.G) return;
+  const int end = min(p.M, (static_cast<int>(blockIdx.x) + 1) * ROWS);
+  for (int m = blockIdx.x * ROWS; m < end;) {
+    const int j = mla_seq_of_row(p.cu_rows, p.nseq, m);
+    if (j < 0) return;                                              // (padding rows come last)
+    const int slot = gqa_slot(p, j);
+    const ConvRun run = {m, min(end, p.cu_rows[j + 1]) - m, m - p.cu_rows[j], p.pos[m], slot < 0 ? nullptr : p.hist + static_cast<size_t>(slot) * p.taps * C};
+    m += run.n;
+    float* o = p.cx + static_cast<size_t>(run.m) * p.ldc;
+    float sq[ROWS];
 #pragma unroll
-  for (int isk = 0; isk < 2; ++isk) {
-    const int n = isk ? ch.nk : ch.nq, first = isk ? ch.nq : 0;
-    const float* w = isk ? p.k_w : p.q_w;
-    float* d = o + (isk ? p.k_off : p.q_off);
-#pragma unroll 4
-    for (int c = threadIdx.x; c < n; c += kConvThreads) {
-      const float s = conv(first + c);
-      sq[isk] = fmaf(s, s, sq[isk]);
-      d[c] = s * w[c];
-    }
-  }
-  for (int g = warp; g < p.G; g += kConvThreads / 32) {
-    float s2 = 0.f;
-    float* d = o + p.v_off + g * p.V;
-    for (int v = lane; v < p.V; v += 32) {
-      const float s = conv(ch.nq + ch.nk + g * p.V + v);
-      s2 = fmaf(s, s, s2);
-      d[v] = s;
-    }
-    if (!p.v_norm) continue;
-    s2 = 1.f / sqrtf(mla_warp_sum(s2) / static_cast<float>(p.V) + p.eps);
-    for (int v = lane; v < p.V; v += 32) d[v] *= s2;
-  }
+    for (int r = 0; r < ROWS; ++r) sq[r] = 0.f;
+    if (item < pq + pk) {
+      const bool isk = item >= pq;
+      const int first = (isk ? item - pq : item) * kConvPart, n = min(isk ? ch.nk : ch.nq, first + kConvPart);
+      const float* w = isk ? p.k_w : p.q_w;
+      for (int c = first + lane * VEC; c < n; c += 32 * VEC) {
+        V y[ROWS];
+        conv_run<VEC, TAPS, ROWS>(p, run, C, (isk ? ch.nq : 0) + c, (isk ? p.rk_off : p.rq_off) + c, y);
+        const V f = *reinterpret_cast<const V*>(w + c);
+        float* d = o + (isk ? p.k_off : p.q_off) + c;
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    sq[i] = mla_warp_sum(sq[i]);
-    if (lane == 0) red[i][warp] = sq[i];
-  }
-  __syncthreads();
-  if (threadIdx.x < 2) {
-    float s = 0.f;
-    for (int w = 0; w < kConvThreads / 32; ++w) s += red[threadIdx.x][w];
-    p.row_ss[2 * m + threadIdx.x] = s;
+        for (int r = 0; r < ROWS; ++r)
+          if (r < run.n) {
+            sq[r] += conv_dot(y[r]);
+            *reinterpret_cast<V*>(d + static_cast<size_t>(r) * p.ldc) = conv_mul(y[r], f);
+          }
+      }
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) {
+        sq[r] = mla_warp_sum(sq[r]);
+        if (lane == 0 && r < run.n) p.row_ss[static_cast<size_t>(run.m + r) * (pq + pk) + item] = sq[r];
+      }
+    } else {
+      const int g = item - pq - pk;
+      float* d = o + p.v_off + g * p.V;
+      for (int v = lane * VEC; v < p.V; v += 32 * VEC) {
+        V y[ROWS];
+        conv_run<VEC, TAPS, ROWS>(p, run, C, ch.nq + ch.nk + g * p.V + v, p.rv_off + g * p.V + v, y);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+          if (r < run.n) {
+            sq[r] += conv_dot(y[r]);
+            *reinterpret_cast<V*>(d + static_cast<size_t>(r) * p.ldc + v) = y[r];
+          }
+      }
+      if (!p.v_norm) continue;
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) sq[r] = 1.f / sqrtf(mla_warp_sum(sq[r]) / static_cast<float>(p.V) + p.eps);
+      for (int v = lane * VEC; v < p.V; v += 32 * VEC)              // (a lane's own values)
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+          if (r < run.n) {
+            V* a = reinterpret_cast<V*>(d + static_cast<size_t>(r) * p.ldc + v);
+            *a = conv_scale(*a, sq[r]);
+          }
+    }
   }
 }
 
-// Four rows of a head from x on, the first of them row m (rows past n repeat the last), divided by their root mean square and rotated by the tables
+template <int VEC, int TAPS>
+static cudaError_t conv_rows_go(const GqaParams& p, cudaStream_t stream) {
+  const int items = conv_parts(p.H * p.D) + conv_parts(p.G * p.D) + p.G;
+  if (p.max_rows == 1) return launch(gqa_conv_kernel<VEC, TAPS, 1>, dim3(p.M, (items + 3) / 4), dim3(128), 0, stream, 2, p);
+  return launch(gqa_conv_kernel<VEC, TAPS, kConvRows>, dim3((p.M + kConvRows - 1) / kConvRows, (items + 3) / 4), dim3(128), 0, stream, 2, p);
+}
+static cudaError_t conv_go(const GqaParams& p, cudaStream_t stream) {
+  if (((p.H * p.D) & 3) || ((p.G * p.D) & 3) || (p.V & 3)) return conv_rows_go<1, 0>(p, stream);
+  switch (p.taps) {
+    case 2: return conv_rows_go<4, 2>(p, stream);
+    case 3: return conv_rows_go<4, 3>(p, stream);
+    case 4: return conv_rows_go<4, 4>(p, stream);
+    default: return conv_rows_go<4, 0>(p, stream);
+  }
+}
+
+// Four rows of a head from x on (scale: their reciprocal root mean squares where they are known; rows past n repeat the last), divided by their root mean square and rotated by the tables
 // at t (rot floats a row); put(row, d, four values) takes the pieces.  D a multiple of 4, at most 256; rot a multiple of 8.
 template <typename Put>
-__device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x, int n, int m, int isk, int lane, const float* t, const Put& put) {
+__device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x, int n, const float* scale, int lane, const float* t, const Put& put) {
   float4 v[4][2];
   float sq[4];
 #pragma unroll
@@ -196,7 +277,7 @@ __device__ __forceinline__ void normed_rows4(const GqaParams& p, const float* x,
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
     if (r >= n) break;
-    const float s = p.taps > 0 ? row_scale(p, m + r, isk) : p.qk_norm ? 1.f / sqrtf(sq[r] / static_cast<float>(p.D) + p.eps) : 1.f;
+    const float s = p.taps > 0 ? scale[r] : p.qk_norm ? 1.f / sqrtf(sq[r] / static_cast<float>(p.D) + p.eps) : 1.f;
 #pragma unroll
     for (int u = 0; u < 2; ++u) put(r, u * 128 + lane * 4, make_float4(v[r][u].x * s, v[r][u].y * s, v[r][u].z * s, v[r][u].w * s));
   }
@@ -217,8 +298,18 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
     return;
   }
   const bool fast = sizeof(T) == 2 && (p.D & 3) == 0 && p.D <= 256 && (p.rot & 7) == 0;
-  if (p.rot > 0) {
-    for (int r = threadIdx.x >> 5; r < n; r += 8) rotary_table(rot_s + r * p.rot, p.freq, p.rot, p.rot_amp, p.pos[m0 + r], lane, 32);
+  __shared__ float scale_s[2][8];                 // behind a convolution: of the rows' queries and keys
+  if (p.rot > 0 || p.taps > 0) {
+    for (int r = threadIdx.x >> 5; r < n; r += 8) {
+      if (p.rot > 0) rotary_table(rot_s + r * p.rot, p.freq, p.rot, p.rot_amp, p.pos[m0 + r], lane, 32);
+      if (p.taps > 0) {
+        const float a = row_scale(p, m0 + r, 0, lane), b = row_scale(p, m0 + r, 1, lane);
+        if (lane == 0) {
+          scale_s[0][r] = a;
+          scale_s[1][r] = b;
+        }
+      }
+    }
     __syncthreads();
   }
   if (p.form == 2) {
@@ -227,7 +318,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
       const float* x0 = p.x + static_cast<size_t>(m0) * p.ldx + p.q_off + item * p.D;
       if (fast) {
         for (int r0 = 0; r0 < n; r0 += 4)
-          normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, m0 + r0, 0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
+          normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, scale_s[0] + r0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
             if (d < p.DK) *reinterpret_cast<uint2*>(q0 + static_cast<size_t>(r0 + r) * p.H * p.DK + d) = pack4(v);      // (zeros from D on)
           });
         return;
@@ -259,7 +350,7 @@ __global__ void __launch_bounds__(256) gqa_append_kernel(const __grid_constant__
 #pragma unroll
       for (int r0 = 0; r0 < 8; r0 += 4) {
         if (r0 >= n) break;
-        normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, m0 + r0, 1, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
+        normed_rows4(p, x0 + static_cast<size_t>(r0) * p.ldx, n - r0, scale_s[1] + r0, lane, rot_s + r0 * p.rot, [&](int r, int d, float4 v) {
           const int s = r == 0 ? slot[r0] : r == 1 ? slot[r0 + 1] : r == 2 ? slot[r0 + 2] : slot[r0 + 3];
           if (s >= 0 && d < p.D)
             *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.cache) + page_block(p, s / kPage, g) + bf16_key_at(s % kPage, d)) = pack4(v);
@@ -398,9 +489,10 @@ __global__ void __launch_bounds__(128) gqa_split_kernel(const __grid_constant__ 
     rotary_table(rot_s, p.freq, p.rot, p.rot_amp, pos, threadIdx.x, 128);
     __syncthreads();
   }
+  const float qs_all = p.taps > 0 ? row_scale(p, m, 0, lane) : 1.f;
   for (int r = warp; r < MT * 16; r += 4) {
     const float* x = xr + p.q_off + (g * hq + min(r, hq - 1)) * p.D;
-    const float s = head_scale(p, x, m, 0, lane);
+    const float s = p.taps > 0 ? qs_all : head_scale(p, x, m, 0, lane);
     for (int d = lane * 2; d < p.DK; d += 64) {
       const float a = r < hq && d < p.D ? rotary_half(x, d, rot_s, p.rot) * s : 0.f, b = r < hq && d + 1 < p.D ? rotary_half(x, d + 1, rot_s, p.rot) * s : 0.f;
       asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_s + r * qs + d * 2), "r"(pack2(a, b)) : "memory");
@@ -645,7 +737,7 @@ static int gqa_go(GqaParams p, cudaStream_t stream) {
     p.q_off = 0;
     p.k_off = (p.H * p.D + 7) & ~7;
     p.v_off = p.k_off + ((p.G * p.D + 7) & ~7);
-    const cudaError_t e = launch(gqa_conv_kernel, dim3(p.M), dim3(kConvThreads), 0, stream, 2, p);
+    const cudaError_t e = conv_go(p, stream);
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   if (const int items = append_items(p)) {

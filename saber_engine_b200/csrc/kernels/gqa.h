@@ -52,13 +52,13 @@ struct GqaParams {
   float out_scale;            // factor of the output
   // convolution (taps > 0).  Inputs of a slot form a ring: the one of position p is row p % taps.
   int taps, v_norm, n_slots, ldc;
-  const float* conv_w;        // [C][taps], C = H D + G D + G V in q | k | v order, last column: the current token
+  const float* conv_w;        // [taps][C], C = H D + G D + G V in q | k | v order, last row: the current token
   const float* q_w;           // [H D]
   const float* k_w;           // [G D]
   float* hist;                // [n_slots][taps][C]
   const int32_t* slots;       // [nseq]
   float* cx;                  // scratch [M][ldc]: the convolved rows, q | k | v from multiples of 8 on
-  float* row_ss;              // scratch [M][2]: sums of squares of q and k
+  float* row_ss;              // scratch [M][ceil(H D / 256) + ceil(G D / 256)]: sums of squares of 256 columns each, q's then k's
   // set at the launch
   const float* gate;          // column 0 of the gate in row 0
   int ld_gate;

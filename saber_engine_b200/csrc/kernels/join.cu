@@ -22,23 +22,32 @@ __device__ __forceinline__ float dot4(float4 a) { return a.x * a.x + a.y * a.y +
 __device__ __forceinline__ float4 join_result(const JoinParams& p, int m, int c) {
   float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
   if (p.y != nullptr) z = *reinterpret_cast<const float4*>(p.y + static_cast<size_t>(m) * p.ldy + c);
-  if (p.routed != nullptr) {
-#pragma unroll 4
-    for (int k = 0; k < p.routes; ++k) {
-      const int r = p.slot_of[m * p.routes + k];
-      if (r < 0) continue;
-      const float w = p.route_w[m * p.routes + k];
-      const size_t at = static_cast<size_t>(r) * p.ldr + c;
-      float4 v;
-      if (p.routed_f32) {
-        v = *reinterpret_cast<const float4*>(static_cast<const float*>(p.routed) + at);
-      } else {
-        const uint2 u = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.routed) + at);
-        v = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
+  if (p.routed != nullptr)
+    for (int k0 = 0; k0 < p.routes; k0 += 4) {      // four rows requested together
+      int slot[4];
+      float w[4];
+      float4 v[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int at = m * p.routes + min(k0 + i, p.routes - 1);
+        slot[i] = p.slot_of[at];
+        w[i] = p.route_w[at];
       }
-      z = make_float4(fmaf(w, v.x, z.x), fmaf(w, v.y, z.y), fmaf(w, v.z, z.z), fmaf(w, v.w, z.w));
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const size_t at = static_cast<size_t>(max(slot[i], 0)) * p.ldr + c;
+        if (p.routed_f32) {
+          v[i] = *reinterpret_cast<const float4*>(static_cast<const float*>(p.routed) + at);
+        } else {
+          const uint2 u = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.routed) + at);
+          v[i] = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (slot[i] >= 0 && k0 + i < p.routes)
+          z = make_float4(fmaf(w[i], v[i].x, z.x), fmaf(w[i], v[i].y, z.y), fmaf(w[i], v[i].z, z.z), fmaf(w[i], v[i].w, z.w));
     }
-  }
   return z;
 }
 

@@ -473,11 +473,11 @@ class StackModel:
         cd, conv = [m for m in ms if isinstance(m, ChannelDeltaMixer)], [m for m in gr if m.taps]
         if cd and not decode:
             blk = M // 4 + nseq
-            wk["cd_rec"] = f32(blk * mx(m.heads * (17 * m.dim_pad + 32) for m in cd))
-            wk["cd_v"] = f32(blk * mx(m.heads * ((m.vdim_pad + 15) // 16) * 64 for m in cd))
+            wk["cd_rec"] = f32(blk * mx(m.heads * (17 * m.dim_pad + 64) for m in cd))
+            wk["cd_v"] = f32(blk * mx(m.heads * ((m.vdim_pad + 31) // 32) * 128 for m in cd))
             wk["cd_o"] = f32(M * mx(m.heads * m.vdim_pad for m in cd))
         if conv:
-            wk["conv_x"], wk["conv_ss"] = f32(M * mx(self._conv_width(m) for m in conv)), f32(2 * M)
+            wk["conv_x"], wk["conv_ss"] = f32(M * mx(self._conv_width(m) for m in conv)), f32(M * mx(self._conv_parts(m) for m in conv))
         if outer or gr:                                   # arrivals at the end of a row: zero between launches
             wk["counters"] = torch.zeros(max(nseq * mx(m.norm_groups for m in outer), M * mx(m.kv_heads for m in gr)), dtype=torch.int32, device=self.device)
         if gr:
@@ -559,6 +559,11 @@ class StackModel:
     def _conv_width(m: GroupedMixer) -> int:
         """Columns of the convolved rows: q | k | v, each from a multiple of 8 on."""
         return sum(L.round_up(n, 8) for name, n in m.segments() if name != "g")
+
+    @staticmethod
+    def _conv_parts(m: GroupedMixer) -> int:
+        """Partial sums of squares of a convolved row: 256 columns of q, then of k."""
+        return sum((n + 255) // 256 for name, n in m.segments() if name in ("q", "k"))
 
     def _cdelta_params(self, key, lw, m: ChannelDeltaMixer, proj, m_op, k0, scale, M, nseq, lay, at, wk) -> N.CdeltaParams:
         p, x = N.CdeltaParams(), lw.extra

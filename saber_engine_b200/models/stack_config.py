@@ -693,7 +693,7 @@ class StackConfig:
         n = [0]
         for m in self.mixers():
             if isinstance(m, ChannelDeltaMixer):
-                n.append(m.heads * (17 * m.dim_pad + 32 + 4 * m.vdim_pad + 64) // 4 + m.heads * m.vdim_pad)
+                n.append(m.heads * (17 * m.dim_pad + 64 + 4 * m.vdim_pad + 128) // 4 + m.heads * m.vdim_pad)
             elif isinstance(m, GroupedMixer) and m.taps:
                 n.append(m.channels + 32)
         return 4 * rows * max(n)

@@ -293,10 +293,11 @@ def build(cfg: StackConfig, get: Callable[[str], torch.Tensor], dtype: torch.dty
             if m.sink:
                 extra["sink"] = f32(p + "sink")
             if m.taps:
-                extra["conv"] = torch.cat([f32(f"{p}{n}.conv") for n in ("q", "k", "v")]).contiguous()
+                extra["conv"] = torch.cat([f32(f"{p}{n}.conv") for n in ("q", "k", "v")]).T.contiguous()     # [tap][channel]
                 extra["q_norm"], extra["k_norm"] = f32(p + "q.norm"), f32(p + "k.norm")
         elif isinstance(m, ChannelDeltaMixer):
-            extra["w2"] = t(p + "w2").T.to(dtype).contiguous()         # [rank][channel]
+            extra["w2"] = torch.zeros(m.out_features, L.round_up(m.rank, 16), dtype=dtype, device=dev)
+            extra["w2"][:, : m.rank] = t(p + "w2")
             extra["w0"], extra["norm"] = f32(p + "w0"), f32(p + "norm")
         if getattr(m, "rot", None) is not None:
             extra["freq"] = torch.tensor(m.rot.frequencies() or [1.0], dtype=torch.float32, device=dev)

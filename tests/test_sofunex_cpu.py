@@ -99,7 +99,8 @@ def test_packed_linears_hold_every_row_once(name):
             assert k0 % 64 == 0 and torch.equal(lw.out.w[:W, k0: k0 + n], t[f"{p}mix.{side}.o"].float())
         assert torch.allclose(lw.out_bias[:W], l.mixer.left_scale * t[p + "mix.left.o.b"].float()) and not lw.out_bias[W:].any()
         right, left = lw.part("right."), lw.part("left.")
-        assert torch.equal(right.extra["w2"], t[p + "mix.right.w2"].float().T) and set(left.off) == {"q", "k", "v"} and "conv" in left.extra
+        assert not right.extra["w2"][:, l.mixer.right.rank:].any() and torch.equal(left.extra["conv"].T, torch.cat([t[f"{p}mix.left.{n}.conv"] for n in "qkv"]).float())
+        assert torch.equal(right.extra["w2"][:, : l.mixer.right.rank], t[p + "mix.right.w2"].float()) and set(left.off) == {"q", "k", "v"} and "conv" in left.extra
         for got_row, key in ((lw.norm, "norm1"), (lw.post1, "norm1b"), (lw.shift, "shift"), *(((lw.norm2, "norm2"), (lw.post2, "norm2b")) if f else ())):
             assert got_row.numel() % 8 == 0 and torch.equal(got_row[:W], t[p + key].float()) and not got_row[W:].any()
         got = sum(float(x.w.abs().sum()) for x in lw.linears())

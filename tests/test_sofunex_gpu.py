@@ -83,7 +83,7 @@ def _delta(H, D, rank, lens, pieces, w2_f32, seed, decays=None):
         offs[name], at = at, (at + k + 7) // 8 * 8
     xs = [rnd(T, ld) for T in lens]
     S = len(lens)
-    dev = dict(state=torch.zeros(S + 1, H, VP, DP, device="cuda"), w2=w2.T.contiguous().to(F32 if w2_f32 else BF16).cuda(), w0=w0.cuda(),
+    dev = dict(state=torch.zeros(S + 1, H, VP, DP, device="cuda"), w2=torch.nn.functional.pad(w2, (0, -rank % 16)).to(F32 if w2_f32 else BF16).contiguous().cuda(), w0=w0.cuda(),
                norm=(1 + 0.3 * rnd(n)).cuda())
     outs = [[] for _ in lens]
     done = [0] * S
@@ -101,8 +101,8 @@ def _delta(H, D, rank, lens, pieces, w2_f32, seed, decays=None):
         i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")          # noqa: E731
         single = all(k == 1 for _, k in todo)
         blk = M // 4 + nseq
-        buf = dict(x=x.cuda(), cu=i32(cu), slots=i32(slots + [-1]), pos=pos.cuda(), rec=torch.zeros(blk * H * (17 * DP + 32), device="cuda"),
-                   vb=torch.zeros(blk * H * ((VP + 15) // 16) * 64, device="cuda"), o=torch.zeros(M * H * VP, device="cuda"),
+        buf = dict(x=x.cuda(), cu=i32(cu), slots=i32(slots + [-1]), pos=pos.cuda(), rec=torch.zeros(blk * H * (17 * DP + 64), device="cuda"),
+                   vb=torch.zeros(blk * H * ((VP + 31) // 32) * 128, device="cuda"), o=torch.zeros(M * H * VP, device="cuda"),
                    out=torch.full((M, n + 64), 7.0, device="cuda"), err=torch.zeros(1, dtype=torch.int32, device="cuda"))
         p = NN.CdeltaParams()
         p.x, p.ldx, p.w2, p.w2_f32, p.rank, p.w0, p.norm_w, p.state = buf["x"].data_ptr(), ld, dev["w2"].data_ptr(), int(w2_f32), rank, dev["w0"].data_ptr(), \
@@ -137,8 +137,9 @@ def _delta(H, D, rank, lens, pieces, w2_f32, seed, decays=None):
 def test_channel_delta_rule(H, D, rank):
     """Ragged portions, single tokens and mixtures of them; read-outs and states."""
     lens = [90, 33, 5, 1]
-    for pieces in ([[90, 33, 5, 1]], [[1, 1, 1, 1]] * 90, [[2, 7, 1, 1], [61, 1, 3, 0], [5, 20, 2, 0], [30, 30, 0, 0]]):
-        got, want, st, states = _delta(H, D, rank, lens, pieces, len(pieces) == 1, H + D)
+    ragged = [[2, 7, 1, 1], [61, 1, 3, 0], [5, 20, 2, 0], [30, 30, 0, 0]]
+    for pieces, w2_f32 in (([[90, 33, 5, 1]], True), ([[1, 1, 1, 1]] * 90, False), (ragged, False), (ragged, True)):
+        got, want, st, states = _delta(H, D, rank, lens, pieces, w2_f32, H + D)
         for j in range(4):
             assert len(got[j]) == lens[j]
             _near(got[j], want[j], 2e-5)

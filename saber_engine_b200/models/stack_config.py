@@ -806,13 +806,13 @@ def sofunex_from_json(doc: dict, name: str = "sofunex", source: Optional[str] = 
         elif f["kind"] == "moe":
             r, g = f["router"], f["router"].get("groups") or {}
             mlp = ExpertMix(r["experts"], r["top"], f["expert"]["ff"], g.get("count", 1), g.get("keep", 1), (f.get("shared") or {}).get("ff", 0),
-                            gated=True, sigmoid=True, scale=float(r["scale"]))
+                            gated=True, sigmoid=True, scale=float(r.get("scale", 1.0)))
         else:
             raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
         layers.append(LayerSpec(mixer, mlp))
     lp = doc.get("loop")
     return StackConfig(name=name, arch="Sofunex", vocab=doc["vocab"], width=doc["width"], layers=tuple(layers), eps=float(doc["norm"]["eps"]),
-                       embed_scale=float(doc["embedding"]["scale"]), parallel=False, post_norms=True, residual_mult=float(doc["residual_mult"]),
+                       embed_scale=float(doc["embedding"]["scale"]), parallel=False, post_norms=True, residual_mult=float(doc.get("residual_mult", 1.0)),
                        token_shift=True, loop=None if lp is None else LoopSpec(lp["start"], lp["stop"], lp["times"]), loop_linear=False,
                        source=source, max_ctx=max_ctx)
 

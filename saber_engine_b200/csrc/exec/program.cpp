@@ -37,6 +37,7 @@
 
 extern "C" int saber_digest_launch(const void* buf, size_t bytes, unsigned long long* out, cudaStream_t stream);
 extern "C" int saber_digest_clear_launch(unsigned long long* out, int n, cudaStream_t stream);
+extern "C" void saber_pdl_plain_next();
 
 namespace {
 
@@ -86,6 +87,8 @@ struct Entry {
   Op op;
   int launches;      // kernel/memset/memcpy nodes this op contributes to a captured graph
   std::string tag;   // label for explain / tracing
+  bool side = false; // runs beside the ops that follow, up to the next one with `join`
+  bool join = false;
 };
 
 struct Program {
@@ -94,7 +97,27 @@ struct Program {
   cudaGraphExec_t exec = nullptr;
   int captured_nodes = -1;
   int last_failed_op = -1;
+  cudaStream_t side = nullptr;       // of the ops that run beside others
+  cudaEvent_t forked = nullptr, done = nullptr;
 };
+
+// The side stream's work and the main stream's next op wait for what the other has been given so far.
+int fork_side(Program* pr, cudaStream_t s) {
+  cudaError_t e = cudaSuccess;
+  if (pr->side == nullptr) {
+    e = cudaStreamCreateWithFlags(&pr->side, cudaStreamNonBlocking);
+    if (e == cudaSuccess) e = cudaEventCreateWithFlags(&pr->forked, cudaEventDisableTiming);
+    if (e == cudaSuccess) e = cudaEventCreateWithFlags(&pr->done, cudaEventDisableTiming);
+  }
+  if (e == cudaSuccess) e = cudaEventRecord(pr->forked, s);
+  if (e == cudaSuccess) e = cudaStreamWaitEvent(pr->side, pr->forked, 0);
+  return static_cast<int>(e);
+}
+int join_side(Program* pr, cudaStream_t s) {
+  cudaError_t e = cudaEventRecord(pr->done, pr->side);
+  if (e == cudaSuccess) e = cudaStreamWaitEvent(s, pr->done, 0);
+  return static_cast<int>(e);
+}
 
 int launch(const Op& op, cudaStream_t s) {
   return std::visit(
@@ -171,6 +194,9 @@ void saber_program_destroy(void* h) {
   if (!pr) return;
   if (pr->exec) cudaGraphExecDestroy(pr->exec);
   if (pr->graph) cudaGraphDestroy(pr->graph);
+  if (pr->done) cudaEventDestroy(pr->done);
+  if (pr->forked) cudaEventDestroy(pr->forked);
+  if (pr->side) cudaStreamDestroy(pr->side);
   delete pr;
 }
 
@@ -328,6 +354,15 @@ int saber_program_add_allreduce(void* h, const saber::AllReduceParams* p, const 
   return add(h, OpAllReduce{*p}, 1, tag);
 }
 
+// Op `i` runs on a stream of its own beside the ops that follow it (side), or is the first that waits for those (join).
+int saber_program_mark(void* h, int i, int side, int join) {
+  auto* pr = static_cast<Program*>(h);
+  if (i < 0 || i >= static_cast<int>(pr->ops.size())) return static_cast<int>(cudaErrorInvalidValue);
+  pr->ops[i].side = side != 0;
+  pr->ops[i].join = join != 0;
+  return 0;
+}
+
 int saber_program_num_ops(void* h) { return static_cast<int>(static_cast<Program*>(h)->ops.size()); }
 
 int saber_program_declared_launches(void* h) {
@@ -343,14 +378,36 @@ const char* saber_program_op_tag(void* h, int i) {
 
 int saber_program_last_failed_op(void* h) { return static_cast<Program*>(h)->last_failed_op; }
 
-// Eager walk of ops [first, last). Returns 0 or the CUDA error of the first failing launch.
+// Eager walk of ops [first, last). Returns 0 or the CUDA error of the first failing launch.  Side ops whose join lies outside the range
+// run in line.
 int saber_program_run_range(void* h, int first, int last, cudaStream_t stream) {
   auto* pr = static_cast<Program*>(h);
   const int n = static_cast<int>(pr->ops.size());
   if (last < 0 || last > n) last = n;
+  int joins = -1;                    // the last op of the range that joins
+  for (int i = first; i < last; ++i)
+    if (pr->ops[i].join) joins = i;
+  bool open = false;
   for (int i = first; i < last; ++i) {
-    const int e = launch(pr->ops[i].op, stream);
-    if (e != 0) { pr->last_failed_op = i; return e; }
+    const Entry& en = pr->ops[i];
+    int e = 0;
+    if (en.join && open) {
+      e = join_side(pr, stream);
+      open = false;
+      saber_pdl_plain_next();
+    }
+    const bool side = en.side && i < joins;
+    if (e == 0 && side && !open) {
+      e = fork_side(pr, stream);
+      open = true;
+      saber_pdl_plain_next();
+    }
+    if (e == 0) e = launch(en.op, side ? pr->side : stream);
+    if (e != 0) {
+      if (open) join_side(pr, stream);
+      pr->last_failed_op = i;
+      return e;
+    }
   }
   return 0;
 }

@@ -18,6 +18,7 @@ namespace saber {
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
+bool pdl_take_plain();    // whether this thread's next launch follows kernels of several streams (then it is an ordinary one)
 int pdl_enabled();   // process-wide switch (launch.cu): 0 off, 1 every kernel, 2 only launches that ask for it
 
 template <typename... KArgs, typename... Args>
@@ -32,10 +33,12 @@ inline cudaError_t launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_
   cfg.stream = stream;
   cudaLaunchAttribute attr[2];
   unsigned n = 0;
+  const bool plain = pdl_take_plain();
   if (cooperative) {
     attr[n].id = cudaLaunchAttributeCooperative;
     attr[n].val.cooperative = 1;
     ++n;
+  } else if (plain) {
   } else if (pdl_enabled() == 1 || (pdl_enabled() == 2 && wants_pdl)) {
     // (a cooperative grid must be resident as a whole when it starts: it is launched serialised)
     attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;

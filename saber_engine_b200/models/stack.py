@@ -9,7 +9,7 @@ launch of its own.
   joined      x <- x + c norm(mixer(blend of norm(x) with the token before)); x <- x + c norm(ff(norm(x))): a sublayer's result is whole
               rows ahead of the stream, so that a row kernel stands between the linears (`join.cu`): it norms the result, adds it, norms
               the stream and, ahead of a mixer, blends.  Mixers may stand side by side between the same two linears
-Launches of a mixer in decoding: delta rule 1, decayed outer products 1, grouped-query attention 1 (2 behind a convolution), latent attention 5 (6 where
+Launches of a mixer in decoding (of mixers side by side, the first on a stream of its own): delta rule 1, decayed outer products 1, grouped-query attention 1 (2 behind a convolution), latent attention 5 (6 where
 queries come from a latent of their own); a pass of a looped block adds one linear, routed experts add 3 (routing and two grouped
 products: the output linear's epilogue adds the experts' rows to the stream).
 
@@ -36,12 +36,14 @@ from .step import BlobLayout, Bucket, finish_bucket, head_outputs, plp_outputs, 
 class StackModel:
     def __init__(self, cfg: StackConfig, device="cuda", max_seqs: int = 8, max_ctx: Optional[int] = None, kv_blocks: Optional[int] = None,
                  weights: Optional[SW.StackWeights] = None, seed: int = 0, dtype: torch.dtype = torch.bfloat16, fuse: bool = True,
-                 expand_bytes: int = 24 << 30, race_check: str = "off", attn_impl: str = "tc"):
+                 expand_bytes: int = 24 << 30, race_check: str = "off", attn_impl: str = "tc", side_stream: bool = True):
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("dtype must be bfloat16 or float32")
         if attn_impl not in ("tc", "mma"):
             raise ValueError("attn_impl must be 'tc' or 'mma'")
-        self.attn_impl = attn_impl
+        # side_stream: mixers side by side run beside each other in decoding (in prompts each fills the SMs, and the scan's few warps
+        # would wait for the other's)
+        self.attn_impl, self.side_stream = attn_impl, side_stream
         if race_check not in ("off", "shadow"):
             raise ValueError("race_check must be 'off' or 'shadow'")
         self.cfg, self.tp, self.rank, self.comm = cfg, 1, 0, None
@@ -374,8 +376,12 @@ class StackModel:
             lw, spec, t = w.layers[run.layer], cfg.layers[run.layer], f"R{run.index}.L{run.layer}"
             e = plain(ar["proj"], lw.n_plain, lw.proj, lw.bias)
             self._linear(prog, lw.proj, ar["h"], M, e, ws, f"{t}.project")
+            at0 = prog.num_ops
             self._mixers(prog, run, lw, spec.mixer, ar["proj"], self._operand(ar["mid"], M, lw.out.K), M, nseq, lay, at, ar["work"], decode, t)
+            mixers = prog.num_ops - at0
             self._linear(prog, lw.out, ar["mid"], M, plain(y, wide, lw.out, lw.out_bias), ws, f"{t}.out")
+            if decode and self.side_stream and mixers == 2:    # (they read the same rows and write columns of their own)
+                prog.beside(at0, at0 + 1, at0 + 2)
             result, f = (lw.post1, True, None), spec.mlp
             if f is not None:
                 join(f"{t}.join", lw.norm2, result)

@@ -389,6 +389,7 @@ def _declare(L: C.CDLL) -> None:
         "saber_program_add_stream_norm": (I, [P, C.POINTER(StreamNormParams), C.c_char_p]),
         "saber_program_add_delta": (I, [P, C.POINTER(DeltaParams), I, C.c_char_p]),
         "saber_program_add_mla": (I, [P, C.POINTER(MlaParams), C.c_char_p]),
+        "saber_program_mark": (I, [P, I, I, I]),
         "saber_program_num_ops": (I, [P]),
         "saber_program_declared_launches": (I, [P]),
         "saber_program_op_tag": (C.c_char_p, [P, I]),
@@ -578,6 +579,12 @@ class Program:
 
     def join(self, p: "JoinParams", tag: str = "join") -> int:
         return self._L.saber_program_add_join(self._h, C.byref(p), tag.encode())
+
+    def beside(self, first: int, last: int, join: int) -> None:
+        """Ops first .. last - 1 run on a stream of their own beside those from `last` on; op `join` is the first that waits for them."""
+        for i in range(first, last):
+            check(self._L.saber_program_mark(self._h, i, 1, 0), "mark")
+        check(self._L.saber_program_mark(self._h, join, 0, 1), "mark")
 
     # ---- execution ---------------------------------------------------------------------------
     @property

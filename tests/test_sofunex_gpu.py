@@ -589,6 +589,16 @@ def test_long_decoding_over_page_borders():
         assert R.error(R.feed(eng, "r", toks, [10, 1]), want) < R.TOL[dtype]
 
 
+def test_mixers_beside_each_other_and_in_line_agree():
+    """Captured and eager, with the first mixer on a stream of its own or not: the same numbers."""
+    cfg = R.CASES["every_kind"]
+    t = R.tensors(cfg, 13)
+    toks = R.tokens(cfg, 80)
+    got = [R.feed(R.engine(cfg, t, BF16, capture=capture, side_stream=side), "r", toks, [40, 1]) for side in (True, False) for capture in (True, False)]
+    assert R.error(got[0], O.Oracle(cfg, t).forward(toks)) < R.TOL[BF16]
+    assert all(torch.equal(g, got[0]) for g in got[1:])
+
+
 def test_unfused_linears_agree():
     cfg = R.CASES["every_kind"]
     t = R.tensors(cfg, 11)

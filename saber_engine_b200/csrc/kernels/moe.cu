@@ -105,7 +105,7 @@ __device__ __forceinline__ void moe_sigmoid_row(const MoeRouteParams& p, int m, 
 }
 
 // The routes of token m, by one warp; kPer * 32 experts at most.  add(expert) counts a route of a local expert.
-template <int kPer, typename Add>
+template <int kPer, bool kSigmoid, typename Add>
 __device__ __forceinline__ void moe_topk_row(const MoeRouteParams& p, int m, int lane, const Add& add) {
   if (p.live != nullptr && m >= *p.live) {
     for (int k = lane; k < p.top_k; k += 32) {
@@ -114,7 +114,7 @@ __device__ __forceinline__ void moe_topk_row(const MoeRouteParams& p, int m, int
     }
     return;
   }
-  if (p.sigmoid) {
+  if constexpr (kSigmoid) {
     moe_sigmoid_row<kPer>(p, m, lane, add);
     return;
   }
@@ -189,11 +189,11 @@ __device__ __forceinline__ void moe_topk_row(const MoeRouteParams& p, int m, int
 }
 
 // grid = ceil(M / 8), block 256: one warp per token.
-template <int kPer>
+template <int kPer, bool kSigmoid>
 __global__ void __launch_bounds__(256) moe_topk_kernel(const MoeRouteParams p) {
   pdl_wait();
   const int m = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (m < p.M) moe_topk_row<kPer>(p, m, threadIdx.x & 31, [&](int e) { atomicAdd(p.counts + e, 1); });
+  if (m < p.M) moe_topk_row<kPer, kSigmoid>(p, m, threadIdx.x & 31, [&](int e) { atomicAdd(p.counts + e, 1); });
 }
 
 // One block of 1024 threads (one per local expert): exclusive scans of the padded row counts and of
@@ -248,7 +248,7 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const MoeRouteParams p) 
 }
 
 // One block for a few tokens: scores, plan and placement in one launch.
-template <int kPer>
+template <int kPer, bool kSigmoid>
 __global__ void __launch_bounds__(1024) moe_route_few_kernel(const MoeRouteParams p) {
   pdl_trigger();
   pdl_wait();
@@ -257,7 +257,7 @@ __global__ void __launch_bounds__(1024) moe_route_few_kernel(const MoeRouteParam
   counts[t] = 0;
   for (int i = t; i < p.rows_cap; i += 1024) p.src_row[i] = -1;
   __syncthreads();
-  for (int m = t >> 5; m < p.M; m += 32) moe_topk_row<kPer>(p, m, t & 31, [&](int e) { atomicAdd(counts + e, 1); });
+  for (int m = t >> 5; m < p.M; m += 32) moe_topk_row<kPer, kSigmoid>(p, m, t & 31, [&](int e) { atomicAdd(counts + e, 1); });
   __syncthreads();
   const int c = counts[t];
   int rows_total, tiles_total;
@@ -398,13 +398,17 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const MoeCombineParams
 namespace saber {
 static bool moe_few(const MoeRouteParams& p) { return p.logits_f32 != nullptr && p.M <= 64; }
 
-template <int kPer>
-static int moe_route_go(const MoeRouteParams& p, cudaStream_t stream) {
-  if (moe_few(p)) return static_cast<int>(launch(moe_route_few_kernel<kPer>, dim3(1), dim3(1024), 0, stream, 2, p));
-  launch(moe_topk_kernel<kPer>, dim3((p.M + 7) / 8), dim3(256), 0, stream, 0, p);
+template <int kPer, bool kSigmoid>
+static int moe_route_form(const MoeRouteParams& p, cudaStream_t stream) {
+  if (moe_few(p)) return static_cast<int>(launch(moe_route_few_kernel<kPer, kSigmoid>, dim3(1), dim3(1024), 0, stream, 2, p));
+  launch(moe_topk_kernel<kPer, kSigmoid>, dim3((p.M + 7) / 8), dim3(256), 0, stream, 0, p);
   launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, 0, p);
   launch(moe_place_kernel, dim3((p.M * p.top_k + 255) / 256), dim3(256), 0, stream, 0, p);
   return static_cast<int>(cudaGetLastError());
+}
+template <int kPer>
+static int moe_route_go(const MoeRouteParams& p, cudaStream_t stream) {
+  return p.sigmoid ? moe_route_form<kPer, true>(p, stream) : moe_route_form<kPer, false>(p, stream);
 }
 }  // namespace saber
 

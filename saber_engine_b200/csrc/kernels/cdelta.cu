@@ -288,7 +288,7 @@ __global__ void __launch_bounds__(128) cdelta_prep_mma_kernel(const __grid_const
   const int h1 = min(p.H, (static_cast<int>(blockIdx.y) + 1) * kCdMmaHeads);
   for (int h = blockIdx.y * kCdMmaHeads; h < h1; ++h) {
     auto product = [&] {
-      __syncthreads();                               // (tanh is there; the products of the head before are read)
+      named_bar_sync(1, 128);                        // (tanh is there; the products of the head before are read)
       float acc[NI][4] = {};
       const __nv_bfloat16* wr[NI];
 #pragma unroll
@@ -323,7 +323,7 @@ __global__ void __launch_bounds__(128) cdelta_prep_mma_kernel(const __grid_const
         *reinterpret_cast<float2*>(d) = make_float2(acc[i][0], acc[i][1]);
         *reinterpret_cast<float2*>(d + 8 * ZS) = make_float2(acc[i][2], acc[i][3]);
       }
-      __syncthreads();
+      named_bar_sync(1, 128);                        // (warps with and without a block meet here)
     };
     if (rows > 0)
       cd_records<NI>(p, x, rows, h, slot, lane, product, [&](int i, int, float (&z)[kBlk]) {
